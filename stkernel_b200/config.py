@@ -13,8 +13,9 @@ from __future__ import annotations
 
 import dataclasses
 import json
+import math
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Sequence, Tuple
+from typing import Any, Dict, List, Mapping, Optional, Sequence, Tuple, Union
 
 
 class ConfigError(ValueError):
@@ -101,6 +102,16 @@ class ModelConfig:
     rms_norm_eps: float = 1e-6
     rope_theta: float = 10000.0
     max_position_embeddings: int = 430000
+
+    # ---- model-family interface (shared with HybridConfig) ------------
+    family = "dsv4"                         # key of models/registry.py (a class attribute, not a field)
+
+    def check_engine(self, e: "EngineConfig") -> None:
+        """Engine settings this architecture cannot run with."""
+        if self.num_attention_heads % e.parallel.tp_size:
+            raise ConfigError("tp_size must divide num_attention_heads")
+        if self.o_groups % e.parallel.tp_size and e.parallel.tp_size % self.o_groups:
+            raise ConfigError("tp_size and o_groups must divide one another")
 
     # ---- derived -----------------------------------------------------
     @property
@@ -211,6 +222,324 @@ def tiny_config(**over: Any) -> ModelConfig:
     return cfg
 
 
+# ----------------------------------------------------------------------------
+# decoders described layer by layer
+# ----------------------------------------------------------------------------
+@dataclass(frozen=True)
+class YarnScaling:
+    """YaRN context extension of a rotary embedding: frequencies below the `slow` bound are divided by `factor`, those
+    above the `fast` bound stay, with a linear ramp between them; cos and sin are scaled by 1 + 0.1 ln(factor)."""
+    factor: float
+    original: float              # context length the unscaled frequencies were made for
+    fast: float                  # full turns over `original` above which a frequency is kept
+    slow: float                  # full turns over `original` below which a frequency is divided by `factor`
+
+
+@dataclass(frozen=True)
+class RotaryConfig:
+    """Rotation of the first `dims` dimensions of a head, dimension i paired with i + dims/2."""
+    base: float
+    dims: int
+    scaling: Optional[YarnScaling] = None
+
+    def frequencies(self) -> Tuple[List[float], float]:
+        """-> (radians per position of every pair, factor on cos and sin)."""
+        d = self.dims
+        f = [self.base ** (-2.0 * i / d) for i in range(d // 2)]
+        s = self.scaling
+        if s is None:
+            return f, 1.0
+        at = lambda turns: d * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+        lo = max(math.floor(at(s.fast)), 0)
+        hi = min(math.ceil(at(s.slow)), d - 1)
+        span = max(hi - lo, 0.001)
+        out = []
+        for i, x in enumerate(f):
+            r = min(max((i - lo) / span, 0.0), 1.0)
+            out.append(x / s.factor * r + x * (1.0 - r))
+        return out, 0.1 * math.log(s.factor) + 1.0
+
+
+@dataclass(frozen=True)
+class AttentionMixer:
+    """Grouped-query sliding-window attention whose values are the unrotated keys (no value projection), with a tanh cap
+    on the scaled scores and one learned sink per head in the softmax denominator."""
+    heads: int
+    kv_heads: int
+    dim: int
+    window: int                  # keys a position sees, itself included
+    scale: float
+    rotary: Optional[RotaryConfig] = None
+    softcap: float = 0.0         # 0: scores are not capped
+    sink: bool = True
+    kind = "attention"
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def rot_dims(self) -> int:
+        return self.rotary.dims if self.rotary is not None else 0
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.dim
+
+
+@dataclass(frozen=True)
+class MlstmMixer:
+    """Matrix-memory recurrence with exponential input gate and running-maximum stabiliser (mLSTM)."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float              # tanh cap of both gate pre-activations
+    kind = "mlstm"
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class DenseMlp:
+    """W_down(silu(W_gate h) * W_up h)."""
+    ff: int
+
+
+@dataclass(frozen=True)
+class HybridLayer:
+    mixer: Union[AttentionMixer, MlstmMixer]
+    mlp: Optional[DenseMlp] = None
+    weights_of: Optional[int] = None      # layer whose tensors this one runs with (cache and state are its own)
+
+
+@dataclass(frozen=True)
+class HybridConfig:
+    """A decoder given as a list of layers, each with its own mixer (attention or recurrence) and optional feed-forward.
+    Both sublayers read one layer norm's output and are added to an fp32 residual together (parallel block)."""
+    vocab_size: int
+    hidden_size: int
+    layers: Tuple[HybridLayer, ...]
+    norm_eps: float = 1e-6
+    embedding_scale: float = 1.0
+    dtype: str = "bfloat16"               # "bfloat16": projections and activations; "float32": everything
+    max_position_embeddings: int = 1 << 30
+    architecture: str = "Timalorn"
+    family = "hybrid"
+    # fields of the other family that family-neutral code asks for
+    n_mtp_layers = 0
+    n_routed_experts = 0
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    def weight_layer(self, i: int) -> int:
+        """The layer whose tensors layer i uses (itself unless `weights_of` says otherwise)."""
+        seen = set()
+        while self.layers[i].weights_of is not None:
+            if i in seen:
+                raise ConfigError(f"layers[{i}].weights_of refers to itself")
+            seen.add(i)
+            i = self.layers[i].weights_of
+        return i
+
+    def windows(self) -> List[int]:
+        """Distinct attention windows, one page group each."""
+        return sorted({l.mixer.window for l in self.layers if l.mixer.kind == "attention"})
+
+    def validate(self) -> None:
+        def positive(name: str, v: Any, integer: bool = True) -> None:
+            ok = (isinstance(v, int) if integer else isinstance(v, (int, float))) and not isinstance(v, bool)
+            if not ok or not math.isfinite(v) or v <= 0:
+                raise ConfigError(f"{name}: {v!r} must be a positive {'integer' if integer else 'number'}")
+
+        positive("vocab_size", self.vocab_size)
+        positive("hidden_size", self.hidden_size)
+        positive("norm_eps", self.norm_eps, False)
+        if not isinstance(self.embedding_scale, (int, float)) or not math.isfinite(self.embedding_scale):
+            raise ConfigError("embedding_scale must be a finite number")
+        if self.dtype not in ("bfloat16", "float32"):
+            raise ConfigError(f"unknown dtype {self.dtype!r}")
+        if not self.layers:
+            raise ConfigError("layers must not be empty")
+        for i, l in enumerate(self.layers):
+            at, m = f"layers[{i}]", l.mixer
+            for f in ("heads", "dim"):
+                positive(f"{at}.mixer.{f}", getattr(m, f))
+            if m.kind == "attention":
+                positive(f"{at}.mixer.kv_heads", m.kv_heads)
+                positive(f"{at}.mixer.mask.size", m.window)
+                if not isinstance(m.scale, (int, float)) or not math.isfinite(m.scale):
+                    raise ConfigError(f"{at}.mixer.scale must be a finite number")
+                if m.heads % m.kv_heads:
+                    raise ConfigError(f"{at}.mixer: kv_heads must divide heads")
+                if m.softcap < 0 or not math.isfinite(m.softcap):
+                    raise ConfigError(f"{at}.mixer.softcap must not be negative")
+                if m.dim > 1024:
+                    raise ConfigError(f"{at}.mixer.dim: at most 1024")
+                if m.rotary is not None:
+                    r = m.rotary
+                    positive(f"{at}.mixer.rot.base", r.base, False)
+                    positive(f"{at}.mixer.rot.dims", r.dims)
+                    if r.dims % 2 or r.dims > m.dim:
+                        raise ConfigError(f"{at}.mixer.rot.dims must be even and at most dim")
+                    if r.scaling is not None:
+                        for f in ("factor", "original", "fast", "slow"):
+                            positive(f"{at}.mixer.rot.scaling.{f}", getattr(r.scaling, f), False)
+            else:
+                positive(f"{at}.mixer.vdim", m.vdim)
+                positive(f"{at}.mixer.gate_cap", m.gate_cap, False)
+                if m.dim > 1024:
+                    raise ConfigError(f"{at}.mixer.dim: at most 1024")
+            if l.mlp is not None:
+                positive(f"{at}.mlp.ff", l.mlp.ff)
+            if l.weights_of is not None:
+                j = l.weights_of
+                if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < len(self.layers):
+                    raise ConfigError(f"{at}.weights_of: no layer {j!r}")
+                src = self.layers[self.weight_layer(i)]
+                if src.mixer != m or src.mlp != l.mlp:
+                    raise ConfigError(f"{at} must equal layer {j}, whose weights it uses")
+
+    def check_engine(self, e: "EngineConfig") -> None:
+        p = e.parallel
+        if p.tp_size != 1 or p.pp_size != 1 or p.dcp_size != 1:
+            raise ConfigError(f"{self.architecture} runs on one GPU (no tensor, pipeline or context parallelism)")
+        if e.spec.method != "none":
+            raise ConfigError(f"{self.architecture} has no draft layers for speculative decoding")
+        if p.eplb_record or p.eplb_redundant:
+            raise ConfigError(f"{self.architecture} has no experts to balance")
+
+
+def _take(d: Any, at: str, required: Sequence[str], optional: Sequence[str] = ()) -> Dict[str, Any]:
+    """The keys of a JSON object, none missing and none unknown."""
+    if not isinstance(d, Mapping):
+        raise ConfigError(f"{at}: {d!r} is not an object")
+    for k in required:
+        if k not in d:
+            raise ConfigError(f"{at}: {k} is missing")
+    unknown = set(d) - set(required) - set(optional)
+    if unknown:
+        raise ConfigError(f"{at}: unknown keys {sorted(unknown)}")
+    return dict(d)
+
+
+def timalorn_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> HybridConfig:
+    """The `config.json` of a Timalorn model: parallel blocks of windowed attention and mLSTM layers."""
+    for k in ("vocab", "width", "layers", "norm", "embedding"):
+        if k not in d:
+            raise ConfigError(f"config.json: {k} is missing")
+    if not isinstance(d["layers"], Sequence) or isinstance(d["layers"], str):
+        raise ConfigError("config.json: layers is not a list")
+    layers: List[HybridLayer] = []
+    for i, l in enumerate(d["layers"]):
+        at = f"layers[{i}]"
+        l = _take(l, at, ("type", "mixer"), ("mlp", "weights_of"))
+        if l["type"] == "attention":
+            m = _take(l["mixer"], f"{at}.mixer", ("heads", "kv_heads", "dim", "mask", "scale"),
+                      ("vdim", "rot", "softcap"))
+            if m.get("vdim", m["dim"]) != m["dim"]:
+                raise ConfigError(f"{at}.mixer.vdim: the values are the keys, so it must equal dim")
+            rot = None
+            if m.get("rot") is not None:
+                r = _take(m["rot"], f"{at}.mixer.rot", ("base", "dims"), ("scaling",))
+                sc = r.get("scaling")
+                if sc is not None:
+                    sc = YarnScaling(**_take(sc, f"{at}.mixer.rot.scaling", ("factor", "original", "fast", "slow")))
+                rot = RotaryConfig(r["base"], r["dims"], sc)
+            mixer: Union[AttentionMixer, MlstmMixer] = AttentionMixer(
+                m["heads"], m["kv_heads"], m["dim"], _take(m["mask"], f"{at}.mixer.mask", ("size",))["size"], m["scale"], rot,
+                m.get("softcap") or 0.0)
+        elif l["type"] == "mlstm":
+            mixer = MlstmMixer(**_take(l["mixer"], f"{at}.mixer", ("heads", "dim", "vdim", "gate_cap")))
+        else:
+            raise ConfigError(f"{at}.type: unknown mixer {l['type']!r}")
+        mlp = None
+        if l.get("mlp") is not None:
+            p = _take(l["mlp"], f"{at}.mlp", ("kind", "ff"))
+            if p["kind"] != "dense":
+                raise ConfigError(f"{at}.mlp.kind: unknown feed-forward {p['kind']!r}")
+            mlp = DenseMlp(p["ff"])
+        layers.append(HybridLayer(mixer, mlp, l.get("weights_of")))
+    cfg = HybridConfig(d["vocab"], d["width"], tuple(layers), _take(d["norm"], "norm", ("eps",))["eps"],
+                       _take(d["embedding"], "embedding", ("scale",))["scale"], dtype)
+    cfg.validate()
+    return cfg
+
+
+def timalorn_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
+    """The inverse of `timalorn_config_from_json`."""
+    layers = []
+    for l in cfg.layers:
+        m = l.mixer
+        if m.kind == "attention":
+            mixer: Dict[str, Any] = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.dim,
+                                     "mask": {"size": m.window}, "scale": m.scale, "softcap": m.softcap}
+            if m.rotary is not None:
+                mixer["rot"] = {"base": m.rotary.base, "dims": m.rotary.dims}
+                if m.rotary.scaling is not None:
+                    mixer["rot"]["scaling"] = dataclasses.asdict(m.rotary.scaling)
+        else:
+            mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "gate_cap": m.gate_cap}
+        d: Dict[str, Any] = {"type": m.kind, "mixer": mixer,
+                             "mlp": {"kind": "dense", "ff": l.mlp.ff} if l.mlp is not None else None}
+        if l.weights_of is not None:
+            d["weights_of"] = l.weights_of
+        layers.append(d)
+    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "layers": layers,
+            "norm": {"eps": cfg.norm_eps}, "embedding": {"scale": cfg.embedding_scale}}
+
+
+def hybrid_config_from_dict(d: Mapping[str, Any]) -> HybridConfig:
+    """The inverse of `dataclasses.asdict(HybridConfig)` (the "model" section of an EngineConfig dictionary)."""
+    d = dict(d)
+    layers = []
+    for l in d.pop("layers"):
+        m = dict(l["mixer"])
+        if "kv_heads" in m:
+            r = m.pop("rotary", None)
+            if r is not None:
+                r = dict(r)
+                sc = r.pop("scaling", None)
+                r = RotaryConfig(**r, scaling=YarnScaling(**sc) if sc is not None else None)
+            mixer: Union[AttentionMixer, MlstmMixer] = AttentionMixer(**m, rotary=r)
+        else:
+            mixer = MlstmMixer(**m)
+        layers.append(HybridLayer(mixer, DenseMlp(**l["mlp"]) if l.get("mlp") is not None else None, l.get("weights_of")))
+    cfg = HybridConfig(layers=tuple(layers), **d)
+    cfg.validate()
+    return cfg
+
+
+def hybrid_stack(n_layers: int, width: int, heads: int, kv_heads: int, dim: int, window: int, ff: int, vocab: int,
+                 mlstm_heads: int, mlstm_dim: int, mlstm_vdim: int, attention_every: int = 2, dtype: str = "bfloat16",
+                 yarn: Optional[YarnScaling] = None, rot_dims: Optional[int] = None) -> HybridConfig:
+    """A Timalorn-shaped decoder of `n_layers` with one attention layer in every `attention_every` (the rest mLSTM)."""
+    att = AttentionMixer(heads, kv_heads, dim, window, dim ** -0.5, RotaryConfig(10000.0, rot_dims or dim // 2, yarn), 50.0)
+    rec = MlstmMixer(mlstm_heads, mlstm_dim, mlstm_vdim, 15.0)
+    layers = tuple(HybridLayer(att if i % attention_every == attention_every - 1 else rec, DenseMlp(ff))
+                   for i in range(n_layers))
+    cfg = HybridConfig(vocab, width, layers, 1e-6, math.sqrt(width), dtype)
+    cfg.validate()
+    return cfg
+
+
+def tiny_hybrid_config(**over: Any) -> HybridConfig:
+    """CPU-sized Timalorn-shaped decoder: mLSTM, attention, a second attention layer with the first one's weights, and an
+    mLSTM layer without feed-forward."""
+    att = AttentionMixer(4, 2, 24, 40, 0.2, RotaryConfig(5000.0, 8, YarnScaling(4.0, 64, 8.0, 1.0)), 30.0)
+    rec = MlstmMixer(3, 16, 24, 9.0)
+    kw: Dict[str, Any] = dict(vocab_size=300, hidden_size=88, norm_eps=1e-5, embedding_scale=7.5,
+                              layers=(HybridLayer(rec, DenseMlp(104)), HybridLayer(att, DenseMlp(104)),
+                                      HybridLayer(att, DenseMlp(104), 1), HybridLayer(rec, None)))
+    kw.update(over)
+    cfg = HybridConfig(**kw)
+    cfg.validate()
+    return cfg
+
+
 @dataclass(frozen=True)
 class ParallelConfig:
     tp_size: int = 1
@@ -309,7 +638,7 @@ class KernelConfig:
 
 @dataclass(frozen=True)
 class EngineConfig:
-    model: ModelConfig = field(default_factory=ModelConfig)
+    model: Union[ModelConfig, "HybridConfig"] = field(default_factory=ModelConfig)
     parallel: ParallelConfig = field(default_factory=ParallelConfig)
     cache: CacheConfig = field(default_factory=CacheConfig)
     sched: SchedulerConfig = field(default_factory=SchedulerConfig)
@@ -320,10 +649,7 @@ class EngineConfig:
     def validate(self) -> "EngineConfig":
         for part in (self.model, self.parallel, self.cache, self.sched, self.spec, self.kernels):
             part.validate()
-        if self.model.num_attention_heads % self.parallel.tp_size:
-            raise ConfigError("tp_size must divide num_attention_heads")
-        if self.model.o_groups % self.parallel.tp_size and self.parallel.tp_size % self.model.o_groups:
-            raise ConfigError("tp_size and o_groups must divide one another")
+        self.model.check_engine(self)
         if self.spec.method == "dspark" and self.parallel.pp_size > 1:
             # The reference refuses DSpark under pipeline parallelism
             # (overlay/dspark_utils_v2.py:158-159).
@@ -355,8 +681,9 @@ class EngineConfig:
         unknown = set(d) - known
         if unknown:
             raise ConfigError(f"unknown EngineConfig sections: {sorted(unknown)}")
+        m = d.get("model")
         return EngineConfig(
-            model=build(ModelConfig, d.get("model")),
+            model=hybrid_config_from_dict(m) if isinstance(m, Mapping) and "layers" in m else build(ModelConfig, m),
             parallel=build(ParallelConfig, d.get("parallel")),
             cache=build(CacheConfig, d.get("cache")),
             sched=build(SchedulerConfig, d.get("sched")),

@@ -1,0 +1,177 @@
+// Residual-side kernels of the parallel block (models/hybrid.py): scaled embedding into an fp32 residual, residual add fused
+// with the next layer norm, and the feed-forward half of the joined sublayer buffer.
+#define STK_PDL_CLASS 4
+#include "common.cuh"
+
+namespace stk {
+
+template <typename T> __device__ __forceinline__ float ld_act(const T* p);
+template <> __device__ __forceinline__ float ld_act<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float ld_act<__nv_bfloat16>(const __nv_bfloat16* p) { return bf16_to_f(*p); }
+template <typename T> __device__ __forceinline__ void st_act(T* p, float v);
+template <> __device__ __forceinline__ void st_act<float>(float* p, float v) { *p = v; }
+template <> __device__ __forceinline__ void st_act<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+template <typename E>
+__global__ void __launch_bounds__(256)
+embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed, float* __restrict__ x, long long ldx, int W,
+                    int vocab, float scale, int* status) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const long long id = ids[t];
+  const bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0) set_status(status, kBadIndex, t);
+  for (int i = threadIdx.x; i < W; i += blockDim.x)
+    x[t * ldx + i] = ok ? ld_act(embed + id * W + i) * scale : 0.f;
+}
+
+// x[r] += y[r]; h[t] = layer_norm(x[r]) * w with r = rows ? rows[t] : t (with `rows` the sum is not written back).  The
+// row stays in shared memory between the three passes (mean, squared deviations, output), all in fp32.
+template <typename O>
+__global__ void __launch_bounds__(256)
+add_layer_norm_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy,
+                      const float* __restrict__ w, O* __restrict__ h, long long ldh, int W, int width, float eps,
+                      const int64_t* __restrict__ rows) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_trigger();
+  const long long r = rows != nullptr ? rows[blockIdx.x] : static_cast<long long>(blockIdx.x);
+  float* xr = x + r * ldx;
+  const float* yr = y != nullptr ? y + r * ldy : nullptr;
+  const bool store = yr != nullptr && rows == nullptr;
+  float s = 0.f;
+  if ((W & 3) == 0 && (ldx & 3) == 0 && (ldy & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      float4 v = *reinterpret_cast<const float4*>(xr + i);
+      if (yr != nullptr) {
+        const float4 u = *reinterpret_cast<const float4*>(yr + i);
+        v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+        if (store) *reinterpret_cast<float4*>(xr + i) = v;
+      }
+      *reinterpret_cast<float4*>(row + i) = v;
+      s += (v.x + v.y) + (v.z + v.w);
+    }
+  } else {
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+      float v = xr[i];
+      if (yr != nullptr) {
+        v += yr[i];
+        if (store) xr[i] = v;
+      }
+      row[i] = v;
+      s += v;
+    }
+  }
+  const float mean = block_sum(s, red) / static_cast<float>(W);
+  float q = 0.f;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float d = row[i] - mean;
+    q = fmaf(d, d, q);
+  }
+  const float inv = 1.f / sqrtf(block_sum(q, red) / static_cast<float>(W) + eps);
+  O* hr = h + blockIdx.x * ldh;
+  if (sizeof(O) == 2 && (width & 1) == 0 && (ldh & 1) == 0) {
+    for (int i = threadIdx.x * 2; i < width; i += blockDim.x * 2) {
+      const float a = i < W ? (row[i] - mean) * inv * w[i] : 0.f;
+      const float b = i + 1 < W ? (row[i + 1] - mean) * inv * w[i + 1] : 0.f;
+      *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(hr) + i) = __floats2bfloat162_rn(a, b);
+    }
+  } else {
+    for (int i = threadIdx.x; i < width; i += blockDim.x) st_act(hr + i, i < W ? (row[i] - mean) * inv * w[i] : 0.f);
+  }
+}
+
+// out[t, mix : o0) = 0, out[t, o0 + j] = silu(gate_j) * up_j for j < ff, zero up to `cols`.
+template <typename A>
+__global__ void __launch_bounds__(256)
+join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int ff, A* __restrict__ out, long long ldo, int mix,
+                int o0, int cols) {
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.y;
+  const A* pg = proj + t * ldp + go;
+  const A* pu = proj + t * ldp + uo;
+  A* o = out + t * ldo;
+  const int base = blockIdx.x * blockDim.x * 8 + threadIdx.x * 8;      // eight columns per thread, from o0 on
+  if (blockIdx.x == 0)
+    for (int i = mix + threadIdx.x; i < o0; i += blockDim.x) st_act(o + i, 0.f);
+  const int n = cols - o0;
+  if (base >= n) return;
+  if (sizeof(A) == 2 && base + 8 <= ff && (ldo & 7) == 0 && (ldp & 7) == 0) {
+    const uint4 gv = *reinterpret_cast<const uint4*>(pg + base), uv = *reinterpret_cast<const uint4*>(pu + base);
+    const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+    const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uv);
+    uint4 ov;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
+      o2[j] = __floats2bfloat162_rn(g.x / (1.f + __expf(-g.x)) * u.x, g.y / (1.f + __expf(-g.y)) * u.y);
+    }
+    *reinterpret_cast<uint4*>(o + o0 + base) = ov;
+    return;
+  }
+  for (int j = base; j < base + 8 && j < n; ++j) {
+    float v = 0.f;
+    if (j < ff) {
+      const float g = ld_act(pg + j);
+      v = g / (1.f + expf(-g)) * ld_act(pu + j);
+    }
+    st_act(o + o0 + j, v);
+  }
+}
+
+}  // namespace stk
+
+using namespace stk;
+
+STK_API int stk_embed_scaled(const int64_t* ids, const void* embed, int embed_fp32, float* x, long long ldx, int T, int W,
+                             int vocab, float scale, int* status, void* stream) {
+  if (T <= 0) return 0;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (embed_fp32)
+    launch_pdl(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, ids, (const float*)embed, x, ldx, W, vocab, scale, status);
+  else
+    launch_pdl(embed_scaled_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, ids, (const __nv_bfloat16*)embed, x, ldx, W, vocab,
+               scale, status);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+STK_API int stk_add_layer_norm(float* x, long long ldx, const float* y, long long ldy, const float* w, void* h, int h_fp32,
+                               long long ldh, int T, int W, int width, float eps, const int64_t* rows, void* stream) {
+  if (T <= 0) return 0;
+  const size_t smem = static_cast<size_t>(W) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (smem > 40 * 1024) {
+    if (cudaFuncSetAttribute(add_layer_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=
+            cudaSuccess ||
+        cudaFuncSetAttribute(add_layer_norm_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=
+            cudaSuccess)
+      return -3;
+  }
+  if (h_fp32)
+    launch_pdl(add_layer_norm_kernel<float>, dim3(T), dim3(256), smem, st, x, ldx, y, ldy, w, (float*)h, ldh, W, width, eps, rows);
+  else
+    launch_pdl(add_layer_norm_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, st, x, ldx, y, ldy, w, (__nv_bfloat16*)h, ldh, W,
+               width, eps, rows);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+STK_API int stk_join_glu(const void* proj, long long ldp, int gate_off, int up_off, int ff, void* out, long long ldo, int fp32,
+                         int mixer_dim, int ff_off, int cols, int T, void* stream) {
+  if (T <= 0) return 0;
+  if (T > 65535) return -1;
+  const int n = cols - ff_off;
+  const dim3 grid(n > 0 ? (n + 2047) / 2048 : 1, T);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (fp32)
+    launch_pdl(join_glu_kernel<float>, grid, dim3(256), 0, st, (const float*)proj, ldp, gate_off, up_off, ff, (float*)out, ldo,
+               mixer_dim, ff_off, cols);
+  else
+    launch_pdl(join_glu_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)proj, ldp, gate_off, up_off, ff,
+               (__nv_bfloat16*)out, ldo, mixer_dim, ff_off, cols);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}

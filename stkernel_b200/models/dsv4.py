@@ -13,7 +13,6 @@ Parallel layout (one rank per GPU, `tp` ranks):
 """
 from __future__ import annotations
 
-import hashlib
 import os
 from dataclasses import dataclass, field
 from typing import Callable, Dict, List, Optional, Tuple
@@ -31,58 +30,13 @@ from ..ops.functional import LinearWeight
 from ..ops.scratch import side_branch
 from ..runtime.planning import (dcp_global_row, dcp_local_index, dcp_local_rows, dcp_owner, pp_layer_range, sp_gather_sizes,
                                 split_indexer_prefill_chunks)
+from .decoder import Decoder
+from .sources import DictSource, RandomSource, WeightSource  # noqa: F401  (public names of this module)
 from .dsv4_oracle import index_cache_computes
 from .weights import compressor_slots
 
 BF16 = torch.bfloat16
 F32 = torch.float32
-
-
-# ----------------------------------------------------------------------------
-# weight sources
-# ----------------------------------------------------------------------------
-class WeightSource:
-    """Hands out fp32 master tensors by checkpoint name."""
-
-    def get(self, name: str, shape: Tuple[int, ...], device) -> torch.Tensor:
-        raise NotImplementedError
-
-
-class DictSource(WeightSource):
-    def __init__(self, tensors: Dict[str, torch.Tensor]):
-        self.t = tensors
-
-    def get(self, name, shape, device):
-        t = self.t[name]
-        assert tuple(t.shape) == tuple(shape), (name, t.shape, shape)
-        return t.to(device)
-
-
-class RandomSource(WeightSource):
-    """Random-init weights: every tensor is a pure function of (seed, name), so replicated
-    tensors agree across ranks without communication."""
-
-    def __init__(self, seed: int = 0, std: float = 0.02):
-        self.seed, self.std = seed, std
-
-    def _gen(self, name: str, device) -> torch.Generator:
-        h = int.from_bytes(hashlib.sha256(f"{self.seed}:{name}".encode()).digest()[:7], "little")
-        g = torch.Generator(device=device)
-        g.manual_seed(h)
-        return g
-
-    def get(self, name, shape, device):
-        dev = torch.device(device)
-        g = self._gen(name, dev)
-        if name.endswith("tid2eid"):
-            return torch.randint(0, 1 << 30, shape, generator=g, device=dev, dtype=torch.int64)
-        if name.endswith("norm.weight") or name.endswith("_scale"):
-            return torch.ones(shape, device=dev)
-        if name.endswith("_base") or name.endswith("attn_sink"):
-            return torch.zeros(shape, device=dev)
-        if name.endswith("gate.bias"):
-            return torch.rand(shape, generator=g, device=dev) * 0.2 - 0.1
-        return torch.randn(shape, generator=g, device=dev) * self.std
 
 
 # ----------------------------------------------------------------------------
@@ -326,21 +280,16 @@ def dcp_merge_candidates(gids: torch.Tensor, vals: torch.Tensor, k: int) -> torc
     return torch.where(top[:, :k] > float("-inf"), ids, torch.full_like(ids, -1))
 
 
-class DSV4Model:
+class DSV4Model(Decoder):
     def __init__(self, cfg: ModelConfig, weights: ModelWeights, kv, comm=None, tp_rank: int = 0, tp_size: int = 1):
+        dev = weights.embed.device
+        super().__init__(dev, comm, tp_rank, tp_size)
         self.cfg = cfg
         self.w = weights
         self.kv = kv
-        self.comm = comm
-        self.tp_rank, self.tp_size = tp_rank, tp_size
-        dev = weights.embed.device
-        self.device = dev
+        self.vocab_start = weights.vocab_start
         self.inv = Fn.inv_freq(cfg.qk_rope_head_dim, cfg.rope_theta, dev)
         self.topk_buffer: Optional[torch.Tensor] = None     # IndexCache: shared by consecutive C4A layers
-        self.pipe = None                                     # parallel.pipeline.PipeStage when the model is one stage of several
-        self.pipe_defer = False                              # the engine exchanges a step's tokens when it finishes the step
-        self.want_logprobs: Optional[int] = None             # set by the engine for a step that reports log-probabilities
-        self.last_logprobs = None                            # (sampled token's, top values, top ids) of that step
         self.aux_layers: Tuple[int, ...] = ()
         self.aux_out: List[torch.Tensor] = []
         self.stats = {"sp_steps": 0, "mla_token_parallel_calls": 0, "dcp_topk_merges": 0}     # which paths ran (tests)
@@ -351,7 +300,6 @@ class DSV4Model:
         self._dcp_lt: Optional[torch.Tensor] = None
         self._dcp_stages: Dict[tuple, PagedCache] = {}
         self.dcp_stage_bytes = int(os.environ.get("STK_DCP_STAGE_MB", "64")) << 20
-        self.load_recorder = None           # parallel.eplb.LoadRecorder when expert load is being recorded
         # Sequence-parallel indexer: with TP the indexer weights are replicated, so each rank scores only its
         # share of a large step's rows and the top-k rows are all-gathered (overlay/attention.py
         # `_indexer_sp_owned_ranges` in the reference; here every row of a step is split evenly, which is exact
@@ -825,6 +773,19 @@ class DSV4Model:
         return Fn.mhc_post(f, X, post, comb)
 
     # ---- whole model -------------------------------------------------------------
+    def build_meta(self, buf, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False,
+                   spans: Tuple[int, int] = (1, 1)) -> StepMeta:
+        tok_req, positions, first, last, sm = A.token_maps(buf.d_qstart, buf.d_rows, buf.d_start, n_req, t_pad,
+                                                           self.kv.swa.table_dev)
+        swa_slots, swa_lens = A.swa_indices(positions, tok_req, self.kv.swa.table_dev, self.cfg.sliding_window)
+        return StepMeta(buf.d_tokens[:t_pad], tok_req, positions, first, last, sm, swa_slots, swa_lens, max_comp_rows,
+                        pure_decode=pure_decode)
+
+    def decode_bucket(self, max_comp_rows: int) -> int:
+        # compressed-row bound baked into the graph: next multiple of 2048 with 64 rows of headroom,
+        # so a sequence crosses into a new graph only every 8192 tokens
+        return ((max_comp_rows + 64) // 2048 + 1) * 2048
+
     def forward_hidden(self, meta: StepMeta) -> torch.Tensor:
         """-> final residual streams [T, hc, H]."""
         cfg = self.cfg
@@ -876,66 +837,19 @@ class DSV4Model:
             X = self.comm.all_gather_dim0(X)
         return X
 
-    def head_hidden(self, X: torch.Tensor) -> torch.Tensor:
+    def head_hidden(self, X: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         cfg = self.cfg
+        if rows is not None:
+            X = X.index_select(0, rows)
         h = Fn.hc_head(X, *self.w.hc_head, cfg.rms_norm_eps, cfg.hc_eps)
         return Fn.rms_norm(h, self.w.norm, cfg.rms_norm_eps)
 
+    def local_logits(self, h: torch.Tensor) -> torch.Tensor:
+        return Fn.linear(h, self.w.head, tag="head")
+
     def compute_logits(self, h: torch.Tensor) -> torch.Tensor:
         """h [n, H] -> logits [n, V] (vocab shards gathered across ranks)."""
-        lg = Fn.linear(h, self.w.head, tag="head")
+        lg = self.local_logits(h)
         if self.tp_size > 1 and self.comm is not None:
             lg = self.comm.all_gather_last_dim(lg)[:, :self.cfg.vocab_size]
         return lg
-
-    def sample(self, h: torch.Tensor, temp: torch.Tensor, seed: torch.Tensor, pos: torch.Tensor,
-               top_k: Optional[torch.Tensor] = None, top_p: Optional[torch.Tensor] = None,
-               agreed_status: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """Head hidden states [n, H] -> sampled tokens [n] (seeded Gumbel arg-max).  Under tensor parallelism the
-        logits stay sharded: every rank takes the noisy arg-max of its vocabulary shard and the ranks exchange one
-        candidate per row (no logits all-gather); truncated sampling (top-k / top-p) needs the whole row and gathers."""
-        from ..ops import sampling as S
-        n = h.shape[0]
-        if self.want_logprobs is not None:
-            # log-probabilities asked for: the whole rows are needed anyway (gathered across ranks); the token is the one
-            # the sharded arg-max would pick (same noise, same logits)
-            lg = self.compute_logits(h)
-            toks, _ = S.gumbel_argmax(lg, temp, seed, pos, top_k=top_k, top_p=top_p)
-            lp = torch.log_softmax(lg.float(), dim=-1)
-            top_lp, top_ids = lp.topk(max(1, min(self.want_logprobs, lp.shape[1])), dim=-1)
-            self.last_logprobs = (lp.gather(1, toks.view(-1, 1).long()).squeeze(1), top_lp, top_ids)
-            return toks
-        ll = None
-        if self.tp_size > 1 and top_k is None and top_p is None and h.is_cuda and n <= 256:
-            ll = self._ll_any(3 * n)
-        if ll is not None:
-            lg = Fn.linear(h, self.w.head, tag="head")
-            toks, _ = S.gumbel_argmax(lg, temp, seed, pos, vocab_start=self.w.vocab_start, ll=ll, agreed_status=agreed_status)
-            return toks
-        toks, _ = S.gumbel_argmax(self.compute_logits(h), temp, seed, pos, top_k=top_k, top_p=top_p)
-        return toks
-
-    def forward_sample(self, meta: StepMeta, logit_rows: Optional[torch.Tensor], temp, seed, pos, top_k=None, top_p=None,
-                       agreed_status=None) -> torch.Tensor:
-        """Sampled tokens for the selected token rows (all rows when logit_rows is None)."""
-        X = self.forward_hidden(meta)
-        pipe = self.pipe
-        if pipe is not None and not pipe.last:
-            # an earlier stage: the step's tokens come back from the last one (now, or when the engine finishes the
-            # step if the exchange is deferred)
-            n = logit_rows.shape[0] if logit_rows is not None else meta.token_ids.shape[0]
-            toks = torch.zeros(n, dtype=torch.int64, device=meta.token_ids.device)
-            return toks if self.pipe_defer else pipe.broadcast_from_last(toks)
-        if logit_rows is not None:
-            X = X.index_select(0, logit_rows)
-        toks = self.sample(self.head_hidden(X), temp, seed, pos, top_k, top_p, agreed_status)
-        if pipe is None or self.pipe_defer:
-            return toks.contiguous() if pipe is not None else toks
-        return pipe.broadcast_from_last(toks.contiguous())
-
-    def forward(self, meta: StepMeta, logit_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """Logits for the selected token rows (all rows when logit_rows is None)."""
-        X = self.forward_hidden(meta)
-        if logit_rows is not None:
-            X = X.index_select(0, logit_rows)
-        return self.compute_logits(self.head_hidden(X))

@@ -28,9 +28,10 @@ from typing import Any, Dict, Iterable, List, Optional, Tuple
 
 import torch
 
-from ..config import FP8_BLOCK, ModelConfig, model_config_from_hf
+from ..config import FP8_BLOCK, ModelConfig
 from ..ops import reference as R
-from .dsv4 import WeightSource
+from .registry import family_of, load_model_config  # noqa: F401
+from .sources import WeightSource
 from .weights import weight_shapes
 
 _DTYPES = {"F32": (torch.float32, 4), "F16": (torch.float16, 2), "BF16": (torch.bfloat16, 2), "I64": (torch.int64, 8),
@@ -194,18 +195,15 @@ class CheckpointSource(WeightSource):
             raise ValueError(f"{name}: checkpoint shape {tuple(out.shape)} != expected {tuple(shape)}")
         return out
 
-    def missing(self, cfg: ModelConfig) -> List[str]:
-        return [n for n in weight_shapes(cfg) if n not in self.index]
+    def missing(self, cfg) -> List[str]:
+        return [n for n in family_of(cfg).weight_shapes(cfg) if n not in self.index]
 
-    def unexpected(self, cfg: ModelConfig) -> List[str]:
-        want = set(weight_shapes(cfg))
+    def unexpected(self, cfg) -> List[str]:
+        want = set(family_of(cfg).weight_shapes(cfg))
         return [n for n in self.index.keys() if n not in want and not n.endswith(".scale")]
 
 
-def load_model_config(path: str) -> ModelConfig:
-    with open(os.path.join(path, "config.json")) as f:
-        return model_config_from_hf(json.load(f))
-
+# `load_model_config` (from the registry) is part of this module's interface: config.json next to the shards
 
 # ---------------------------------------------------------------------------------------
 # TP shard plan

@@ -1,0 +1,53 @@
+"""Where model weights come from: a dictionary, seeded random tensors, or a checkpoint (`loader.CheckpointSource`)."""
+from __future__ import annotations
+
+import hashlib
+from typing import Dict, Tuple
+
+import torch
+
+
+class WeightSource:
+    """Hands out fp32 master tensors by checkpoint name."""
+
+    def get(self, name: str, shape: Tuple[int, ...], device) -> torch.Tensor:
+        raise NotImplementedError
+
+
+class DictSource(WeightSource):
+    def __init__(self, tensors: Dict[str, torch.Tensor]):
+        self.t = tensors
+
+    def get(self, name, shape, device):
+        t = self.t[name]
+        assert tuple(t.shape) == tuple(shape), (name, t.shape, shape)
+        return t.to(device)
+
+
+class RandomSource(WeightSource):
+    """Random-init weights: every tensor is a pure function of (seed, name), so replicated
+    tensors agree across ranks without communication."""
+
+    def __init__(self, seed: int = 0, std: float = 0.02):
+        self.seed, self.std = seed, std
+
+    def _gen(self, name: str, device) -> torch.Generator:
+        h = int.from_bytes(hashlib.sha256(f"{self.seed}:{name}".encode()).digest()[:7], "little")
+        g = torch.Generator(device=device)
+        g.manual_seed(h)
+        return g
+
+    def get(self, name, shape, device):
+        dev = torch.device(device)
+        g = self._gen(name, dev)
+        if name.endswith("tid2eid"):
+            return torch.randint(0, 1 << 30, shape, generator=g, device=dev, dtype=torch.int64)
+        if name.endswith(("norm.weight", "_scale", ".norm", ".norm1")):
+            return torch.ones(shape, device=dev)
+        if name.endswith(".f.b"):
+            return 3.0 + 3.0 * torch.rand(shape, generator=g, device=dev)      # forget gates of a recurrence start near one
+        if name.endswith(("_base", "attn_sink", ".sink", ".i.b")):
+            return torch.zeros(shape, device=dev)
+        if name.endswith("gate.bias"):
+            return torch.rand(shape, generator=g, device=dev) * 0.2 - 0.1
+        return torch.randn(shape, generator=g, device=dev) * self.std

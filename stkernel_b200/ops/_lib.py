@@ -11,7 +11,7 @@ import ctypes
 import os
 import re
 from pathlib import Path
-from typing import Any, Dict, Optional
+from typing import Any, Dict, Optional, Sequence
 
 import torch
 
@@ -47,6 +47,19 @@ def available() -> bool:
     return _LIB_PATH.exists()
 
 
+def use_family(name: str, files: Optional[Sequence[str]]) -> None:
+    """Load the library that serves one model family: the whole one when it is built and current, else one of just these
+    sources, compiled now if need be.  Before the first kernel of the process."""
+    global _LIB_PATH
+    from ..csrc import build as B
+    if _lib is not None or files is None or B.is_current(_LIB_PATH):
+        return
+    path = B.library_path(name)
+    if not B.is_current(path, files):
+        B.build(only=files, name=name)
+    _LIB_PATH = path
+
+
 def lib() -> ctypes.CDLL:
     global _lib
     if _lib is None:
@@ -56,7 +69,11 @@ def lib() -> ctypes.CDLL:
                 "on a GPU machine)")
         _lib = ctypes.CDLL(str(_LIB_PATH), mode=os.RTLD_GLOBAL if hasattr(os, "RTLD_GLOBAL") else ctypes.DEFAULT_MODE)
         for name, (ret, types) in _parse_signatures().items():
-            fn = getattr(_lib, name)
+            fn = getattr(_lib, name, None)
+            if fn is None:                        # a family library holds only what that family launches
+                if _LIB_PATH.name == "libstk_b200.so":
+                    raise RuntimeError(f"{_LIB_PATH} has no {name}: rebuild it (`python -m stkernel_b200.csrc.build`)")
+                continue
             fn.argtypes = types
             fn.restype = ret
     return _lib

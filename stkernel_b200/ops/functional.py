@@ -43,7 +43,7 @@ def cpu_act_dtype() -> torch.dtype:
 # ----------------------------------------------------------------------------
 @dataclass
 class LinearWeight:
-    """[N, K] weight in its storage format: bf16, or e4m3 with 128x128 fp32 block scales."""
+    """[N, K] weight in its storage format: bf16, e4m3 with 128x128 fp32 block scales, or fp32 (true fp32 products)."""
     w: torch.Tensor
     scale: Optional[torch.Tensor] = None
 
@@ -64,7 +64,7 @@ class LinearWeight:
         if dense_dtype == "fp8":
             q, s = R.quant_fp8_block128_weight(w.to(device=device, dtype=F32), ue8m0=ue8m0)
             return LinearWeight(q.contiguous(), s.contiguous())
-        return LinearWeight(w.to(device=device, dtype=BF16).contiguous())
+        return LinearWeight(w.to(device=device, dtype=F32 if dense_dtype == "float32" else BF16).contiguous())
 
     def dequant(self) -> torch.Tensor:
         if self.is_fp8:
@@ -184,6 +184,8 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
     norm = (weight, eps): x is RMS-normalised first (inside the weight-streaming kernel for decode-sized batches).
     ll: an `LLExchange`; the bf16 result is a per-rank partial sum that goes into the folded all-reduce and an
     `LLPending` is returned instead of a tensor (row-parallel layers at decode sizes)."""
+    if lw.w.dtype == F32:
+        return _linear_f32(x, lw, out)
     if (norm is not None or ll is not None) and not isinstance(x, QuantAct) and x.is_cuda:
         t0, (n0, k0) = x.shape[0], lw.w.shape
         if groups == 1 and ar_ctx is None and out_dtype == BF16 and _skinny_ok(x, t0, k0, lw.is_fp8, n0 // max(groups, 1), n0) and (ll is None or n0 % 2 == 0):
@@ -254,6 +256,21 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
               xa.scale if is_fp8 else None, xa.scale.stride(0) if is_fp8 else 0, splits, ws, cnt,
               _lib.status_buffer(), sms, groups, ctypes.addressof(ar_ctx) if ar_ctx is not None else None,
               _lib.stream())
+    return out
+
+
+def _linear_f32(x: torch.Tensor, lw: LinearWeight, out: Optional[torch.Tensor]) -> torch.Tensor:
+    """fp32 x fp32 -> fp32 on the CUDA cores (no tf32 anywhere): models that run in float32."""
+    t, (n, k) = x.shape[0], lw.w.shape
+    if not x.is_cuda:
+        y = x.to(F32) @ lw.w.t()
+        if out is not None:
+            out.copy_(y)
+            return out
+        return y
+    if out is None:
+        out = torch.empty(t, n, dtype=F32, device=x.device)
+    _lib.call("stk_linear_f32", lw.w, lw.w.stride(0), x, x.stride(0), out, out.stride(0), t, n, k, _lib.stream())
     return out
 
 

@@ -1,0 +1,215 @@
+"""Ops of the hybrid decoder: scaled embedding and add + layer norm on an fp32 residual, paged windowed attention whose
+values are the unrotated keys, mLSTM recurrence, and the parallel block's joined sublayer outputs.
+
+Activations are bf16, or fp32 in a float32 model (every kernel here has both forms; the fp32 forms use no reduced-precision
+products).  Residual, norms, scores and softmax, gates and recurrent state are fp32 in either.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional, Tuple
+
+import torch
+
+from . import _lib
+from . import reference as R
+from .cache import PAGE
+from .functional import cpu_act_dtype
+from .scratch import scratch
+
+BF16 = torch.bfloat16
+F32 = torch.float32
+
+# spans of at most this many tokens are attended token by token (the kernel of decode steps); longer ones in query tiles
+ATTN_TOKEN_SPAN = 4
+# spans of at least this many tokens run the recurrence in chunks on the tensor cores (bf16 models)
+MLSTM_CHUNK_SPAN = 24
+MLSTM_CHUNK = 64
+
+
+def act_dtype(dtype: str, device) -> torch.dtype:
+    if dtype == "float32":
+        return F32
+    return BF16 if torch.device(device).type == "cuda" else cpu_act_dtype()
+
+
+def _is32(t: torch.Tensor) -> int:
+    return 1 if t.dtype == F32 else 0
+
+
+# ----------------------------------------------------------------------------
+# residual
+# ----------------------------------------------------------------------------
+def embed_scaled(ids: torch.Tensor, embed: torch.Tensor, scale: float) -> torch.Tensor:
+    """ids [T] -> fp32 residual [T, W] = embed[id] * scale."""
+    if not ids.is_cuda:
+        ok = (ids >= 0) & (ids < embed.shape[0])
+        return torch.where(ok[:, None], embed[ids.clamp(0, embed.shape[0] - 1)].to(F32) * scale, torch.zeros(1))
+    t, w = ids.shape[0], embed.shape[1]
+    x = torch.empty(t, w, dtype=F32, device=ids.device)
+    _lib.call("stk_embed_scaled", ids, embed, _is32(embed), x, w, t, w, embed.shape[0], float(scale), _lib.status_buffer(),
+              _lib.stream())
+    return x
+
+
+def add_layer_norm(x: torch.Tensor, y: Optional[torch.Tensor], w: torch.Tensor, eps: float, width: int, dtype: torch.dtype,
+                   rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += y (fp32, in place; y None: nothing to add), then the layer norm of x in `dtype`, zero-padded to `width` columns.
+    rows: only these rows are normed (and the addition is not written back)."""
+    w_n = x.shape[1]
+    if not x.is_cuda:
+        if rows is not None:
+            x = x[rows]
+            x = x + y[rows] if y is not None else x
+        elif y is not None:
+            x += y
+        h = torch.zeros(x.shape[0], width, dtype=dtype)
+        h[:, :w_n] = R.layer_norm(x, w, eps).to(dtype)
+        return h
+    t = x.shape[0] if rows is None else rows.shape[0]
+    h = torch.empty(t, width, dtype=dtype, device=x.device)
+    _lib.call("stk_add_layer_norm", x, x.stride(0), y, y.stride(0) if y is not None else 0, w, h, _is32(h), width, t, w_n, width,
+              float(eps), rows, _lib.stream())
+    return h
+
+
+# ----------------------------------------------------------------------------
+# step description
+# ----------------------------------------------------------------------------
+@dataclass
+class HybridMeta:
+    """Device-side description of one ragged step (decode rows and prompt portions alike)."""
+    token_ids: torch.Tensor        # [T] int64
+    tok_req: torch.Tensor          # [T] int32 request row, -1 padding
+    positions: torch.Tensor        # [T] int64, -1 padding
+    first_pos: torch.Tensor        # [T] int32 first position of the token's span in this step
+    last_pos: torch.Tensor         # [T] int32
+    query_start: torch.Tensor      # [n_req + 1] int32
+    req_rows: torch.Tensor         # [n_req] int32
+    start_pos: torch.Tensor        # [n_req] int32
+    n_req: int
+    max_span: int                  # longest span of the step (host knowledge: which kernels have work)
+    pure_decode: bool = False      # every span is one token
+    min_span: int = 1
+
+
+# ----------------------------------------------------------------------------
+# windowed attention
+# ----------------------------------------------------------------------------
+@dataclass
+class AttentionParams:
+    """Constants of one attention layer on the device."""
+    heads: int
+    kv_heads: int
+    dim: int
+    window: int
+    scale: float
+    softcap: float
+    freq: torch.Tensor             # [rot_dims / 2] fp32 radians per position
+    mag: float
+    sink: Optional[torch.Tensor]   # [heads] fp32
+
+
+def window_attention(proj: torch.Tensor, q_off: int, k_off: int, a: AttentionParams, meta: HybridMeta, table: torch.Tensor,
+                     cache: torch.Tensor, out: torch.Tensor) -> None:
+    """proj [T, *] holds q at column q_off and k at k_off.  Inserts the tokens' rows into the paged cache and writes the
+    attention output of every token into out[:, : heads * dim] (a view of the joined sublayer buffer)."""
+    t = proj.shape[0]
+    h, g, d = a.heads, a.kv_heads, a.dim
+    if not proj.is_cuda:
+        q = proj[:, q_off:q_off + h * d].reshape(t, h, d)
+        k = proj[:, k_off:k_off + g * d].reshape(t, g, d)
+        R.window_kv_insert(k, meta.positions, meta.tok_req, table, cache, a.freq, a.mag)
+        o = R.window_attention(q, meta.positions, meta.tok_req, table, cache, a.freq, a.mag, a.window, a.scale, a.softcap,
+                               a.sink)
+        out[:, :h * d] = o.flatten(1).to(out.dtype)
+        return
+    rd = 2 * a.freq.numel()
+    common = (proj, proj.stride(0), q_off, k_off, meta.positions, meta.tok_req, table, table.stride(0), cache, cache.shape[3],
+              a.freq, rd, float(a.mag), h, g, d)
+    _lib.call("stk_window_kv_insert", *common, _is32(proj), t, _lib.stream())
+    tail = (a.window, float(a.scale), float(a.softcap), a.sink, out, out.stride(0))
+    if _is32(proj) or d > 256 or cache.shape[3] % 8:
+        _lib.call("stk_window_attention_simt", *common, *tail, _is32(proj), t, _lib.stream())
+        return
+    token_span = ATTN_TOKEN_SPAN if meta.max_span > ATTN_TOKEN_SPAN else meta.max_span
+    if meta.min_span <= token_span:
+        splits = _lib.query("stk_window_attention_splits", t, h, g, a.window, _lib.sm_count())
+        part = scratch("wattn.part", (splits * t * h * (d + 2),), F32, proj.device) if splits > 1 else None
+        _lib.call("stk_window_attention_tokens", *common, *tail, meta.first_pos, meta.last_pos, token_span, splits, part, t,
+                  _lib.stream())
+    if meta.max_span > token_span:
+        _lib.call("stk_window_attention_tiles", *common, *tail, meta.query_start, meta.req_rows, meta.start_pos, meta.n_req,
+                  token_span + 1, t, _lib.stream())
+
+
+# ----------------------------------------------------------------------------
+# mLSTM
+# ----------------------------------------------------------------------------
+@dataclass
+class MlstmParams:
+    heads: int
+    dim: int
+    vdim: int
+    cap: float
+    gate_bias: torch.Tensor        # [2 * heads] fp32: input gates, forget gates
+    norm: torch.Tensor             # [heads * vdim] fp32
+    eps: float
+
+
+def mlstm(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, gates: torch.Tensor, p: MlstmParams,
+          meta: HybridMeta, state: Tuple[torch.Tensor, torch.Tensor, torch.Tensor], out: torch.Tensor,
+          glu: Optional[Tuple[int, int, int]]) -> None:
+    """Runs the step's tokens through the recurrence (state updated) and writes norm(o) * sigmoid(g) into
+    out[:, : heads * vdim].  gates [T, 2 * heads] fp32 projections.  glu: see `join_glu` (done by the same launch)."""
+    t = proj.shape[0]
+    h, d, v = p.heads, p.dim, p.vdim
+    S, n, m = state
+    if not proj.is_cuda:
+        seg = lambda o, w: proj[:, o:o + h * w].reshape(t, h, w)
+        o = R.mlstm_scan(seg(q_off, d), seg(k_off, d), seg(v_off, v), gates, p.gate_bias, p.cap, meta.tok_req, meta.first_pos,
+                         meta.positions, S, n, m)
+        out[:, :h * v] = R.head_norm_gate(o, p.norm, proj[:, g_off:g_off + h * v], p.eps).to(out.dtype)
+        join_glu(proj, out, h * v, glu)
+        return
+    dev = proj.device
+    num = scratch("mlstm.num", (t, h * v), F32, dev)
+    den = scratch("mlstm.den", (t, h), F32, dev)
+    mt = scratch("mlstm.m", (t, h), F32, dev)
+    chunked = not _is32(proj) and meta.max_span >= MLSTM_CHUNK_SPAN and d <= 256
+    args = (proj, proj.stride(0), q_off, k_off, v_off, gates, p.gate_bias, float(p.cap), meta.query_start, meta.req_rows,
+            meta.start_pos, meta.n_req, S, n, m, num, den, mt, h, d, v)
+    if not chunked or meta.min_span < MLSTM_CHUNK_SPAN:
+        _lib.call("stk_mlstm_scan", *args, _is32(proj), 1, (MLSTM_CHUNK_SPAN - 1) if chunked else 1 << 30, t, _lib.stream())
+    if chunked:
+        L = MLSTM_CHUNK
+        chunks = t // L + meta.n_req
+        a_ws = scratch("mlstm.gates", (chunks * h * _lib.query("stk_mlstm_gate_slot"),), F32, dev)
+        u_ws = scratch("mlstm.states", (chunks * h * d * (v + 1),), F32, dev)
+        _lib.call("stk_mlstm_chunks", *args, MLSTM_CHUNK_SPAN, a_ws, u_ws, chunks, t, _lib.stream())
+    go, uo, ff = glu if glu is not None else (0, 0, 0)
+    _lib.call("stk_mlstm_finish", num, den, mt, m, p.norm, float(p.eps), meta.tok_req, meta.positions, meta.last_pos, proj,
+              proj.stride(0), g_off, out, out.stride(0), _is32(proj), h, v, go, uo, ff, out_offset(h * v), out.shape[1], t,
+              _lib.stream())
+
+
+def out_offset(mixer_dim: int) -> int:
+    """Column of the joined sublayer buffer where the feed-forward activation starts."""
+    return (mixer_dim + 15) // 16 * 16
+
+
+def join_glu(proj: torch.Tensor, out: torch.Tensor, mixer_dim: int, glu: Optional[Tuple[int, int, int]]) -> None:
+    """out[:, out_offset(mixer_dim):] = silu(gate) * up with (gate, up) at columns glu[0], glu[1] of proj, glu[2] wide (None:
+    no feed-forward); columns of `out` between and after the two parts become zero."""
+    o0 = out_offset(mixer_dim)
+    go, uo, ff = glu if glu is not None else (0, 0, 0)
+    if not proj.is_cuda:
+        out[:, mixer_dim:] = 0
+        if ff:
+            gate, up = proj[:, go:go + ff].to(F32), proj[:, uo:uo + ff].to(F32)
+            out[:, o0:o0 + ff] = (torch.nn.functional.silu(gate) * up).to(out.dtype)
+        return
+    if out.shape[1] == mixer_dim:
+        return
+    _lib.call("stk_join_glu", proj, proj.stride(0), go, uo, ff, out, out.stride(0), _is32(proj), mixer_dim, o0, out.shape[1],
+              proj.shape[0], _lib.stream())

@@ -569,3 +569,101 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w13: 
         act = swiglu_clamp(gu[:, :inter], gu[:, inter:], limit)
         out[tok] += (act @ w2[e].to(F32).t()) * wt[:, None]
     return out
+
+
+# ----------------------------------------------------------------------------
+# layers of the hybrid decoder (paged windowed attention, mLSTM, parallel block)
+# ----------------------------------------------------------------------------
+def layer_norm(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    """fp32 layer norm with a weight and no bias."""
+    xf = x.to(F32)
+    c = xf - xf.mean(-1, keepdim=True)
+    return c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * w.to(F32)
+
+
+def rotate_half_head(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, mag: float) -> torch.Tensor:
+    """x [T, heads, D]: the first 2 * len(freq) dimensions rotated (dimension i with i + len(freq)), fp32."""
+    d = freq.numel()
+    xf = x.to(F32)
+    if d == 0:
+        return xf
+    a = positions.to(F32)[:, None] * freq.to(F32)[None]
+    c, s = (torch.cos(a) * mag)[:, None], (torch.sin(a) * mag)[:, None]
+    u, v = xf[..., :d], xf[..., d:2 * d]
+    return torch.cat([u * c - v * s, v * c + u * s, xf[..., 2 * d:]], -1)
+
+
+def window_kv_insert(k: torch.Tensor, positions, tok_req, table, cache, freq, mag: float) -> None:
+    """k [T, G, D] -> cache [pages, G, PAGE, row]: the key as projected, then its rotated head."""
+    page_rows = cache.shape[2]
+    d, rd = k.shape[-1], 2 * freq.numel()
+    rot = rotate_half_head(k, positions, freq, mag)[..., :rd]
+    for t in range(k.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        pg = int(table[r, p // page_rows])
+        if pg < 0:
+            continue
+        cache[pg, :, p % page_rows, :d] = k[t].to(cache.dtype)
+        cache[pg, :, p % page_rows, d:d + rd] = rot[t].to(cache.dtype)
+
+
+def window_attention(q: torch.Tensor, positions, tok_req, table, cache, freq, mag: float, window: int, scale: float,
+                     softcap: float, sink: Optional[torch.Tensor]) -> torch.Tensor:
+    """q [T, H, D] (unrotated) against the paged rows of each token's window -> [T, H, D] fp32."""
+    t_n, h, d = q.shape
+    g, page_rows = cache.shape[1], cache.shape[2]
+    rd = 2 * freq.numel()
+    qr = rotate_half_head(q, positions, freq, mag).to(q.dtype).to(F32)
+    out = torch.zeros(t_n, h, d, dtype=F32)
+    for t in range(t_n):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        at = torch.arange(max(0, p - window + 1), p + 1)
+        rows = cache[table[r, at // page_rows].long(), :, at % page_rows].to(F32)        # [n, G, row]
+        v = rows[..., :d]
+        k = torch.cat([rows[..., d:d + rd], rows[..., rd:d]], -1)
+        s = torch.einsum("ghd,ngd->ghn", qr[t].view(g, h // g, d), k) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
+        s = s.view(h, -1)
+        if sink is not None:
+            s = torch.cat([s, sink.to(F32)[:, None]], -1)
+        w = torch.softmax(s, -1)[:, :at.numel()]
+        out[t] = torch.einsum("ghn,ngd->ghd", w.view(g, h // g, -1), v).reshape(h, d)
+    return out
+
+
+def mlstm_scan(q, k, v, gates, gate_bias, cap: float, tok_req, first_pos, positions, S, n, m):
+    """One step's tokens through the recurrence.  q, k [T, H, D], v [T, H, V], gates [T, 2H] (input gates, forget gates;
+    before bias and cap), state S [rows, H, D, V], n [rows, H, D], m [rows, H] updated in place.  A span that starts at
+    position 0 starts from zeros.  -> output [T, H, V] fp32 (before the norm)."""
+    t_n, h, d = q.shape
+    pre = cap * torch.tanh((gates.to(F32) + gate_bias.to(F32)) / cap)
+    ig, fg = pre[:, :h], torch.nn.functional.logsigmoid(pre[:, h:])
+    out = torch.zeros(t_n, h, v.shape[-1], dtype=F32)
+    for t in range(t_n):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        if p == 0:
+            S[r].zero_()
+            n[r].zero_()
+            m[r].zero_()
+        m_new = torch.maximum(fg[t] + m[r], ig[t])
+        a, b = torch.exp(fg[t] + m[r] - m_new), torch.exp(ig[t] - m_new)
+        kf, qf = k[t].to(F32), q[t].to(F32) * d ** -0.5
+        S[r] = a[:, None, None] * S[r] + b[:, None, None] * kf[:, :, None] * v[t].to(F32)[:, None, :]
+        n[r] = a[:, None] * n[r] + b[:, None] * kf
+        m[r] = m_new
+        den = torch.maximum((n[r] * qf).sum(-1).abs(), torch.exp(-m_new)) + 1e-6
+        out[t] = torch.einsum("hdv,hd->hv", S[r], qf) / den[:, None]
+    return out
+
+
+def head_norm_gate(o: torch.Tensor, w: torch.Tensor, g: torch.Tensor, eps: float) -> torch.Tensor:
+    """o [T, H, V] fp32: every head divided by its root mean square, times w [H*V] and sigmoid(g [T, H*V])."""
+    y = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps)
+    return y.flatten(1) * w.to(F32) * torch.sigmoid(g.to(F32))

@@ -16,11 +16,10 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from ..config import EngineConfig
-from ..models.dsv4 import DSV4Model, ModelWeights, StepMeta
-from ..ops import attention as A
+from ..models.registry import family_of
 from ..ops import sampling as S
 from ..ops.cache import PAGE
-from .kv import KVManager, OutOfPages, memory_pool_tokens, size_pools
+from .kv import CacheManager, OutOfPages
 from .metrics import Metrics
 
 
@@ -101,7 +100,7 @@ class ScheduledSeq:
 class Scheduler:
     """Decode-first continuous batching with chunked prefill and page-aware admission."""
 
-    def __init__(self, cfg: EngineConfig, kv: KVManager, prefix_cache=None):
+    def __init__(self, cfg: EngineConfig, kv: CacheManager, prefix_cache=None):
         self.cfg = cfg
         self.kv = kv
         self.prefix_cache = prefix_cache
@@ -231,7 +230,7 @@ class StepBuffers:
 
 
 class Engine:
-    def __init__(self, cfg: EngineConfig, weights: ModelWeights, device, comm=None, tp_rank: int = 0,
+    def __init__(self, cfg: EngineConfig, weights, device, comm=None, tp_rank: int = 0,
                  max_context: Optional[int] = None, draft_weights=None, mask_token_id: int = 0, pipe=None):
         """pipe: a `parallel.pipeline.PipeStage` when this engine is one pipeline stage (its `weights` then hold the
         stage's layers only, `build_model_weights(layer_range=pipe.layer_range(...))`).  Every stage runs the same
@@ -245,22 +244,6 @@ class Engine:
         dcp = cfg.parallel.dcp_size
         if dcp > 1 and (dcp != cfg.parallel.tp_size or comm is None):
             raise ValueError("dcp_size must be 1 or tp_size (the context-parallel ranks are the tensor-parallel group)")
-        pool_tokens = cfg.cache.kv_pool_tokens
-        if pool_tokens is None and cfg.cache.size_by_memory and self.device.type == "cuda":
-            free, total = torch.cuda.mem_get_info(self.device)
-            lo_hi = pipe.layer_range(cfg.model.num_hidden_layers) if pipe is not None else (0, cfg.model.num_hidden_layers)
-            pool_tokens = memory_pool_tokens(cfg.model, cfg.cache.gpu_memory_utilization, free, total, ctx,
-                                             list(range(*lo_hi)), dcp)
-            if comm is not None or pipe is not None:
-                # every rank (and every stage) runs the same scheduler: they must agree on the pool, so take the smallest
-                import torch.distributed as dist
-                seen = [None] * dist.get_world_size()
-                dist.all_gather_object(seen, pool_tokens)
-                pool_tokens = min(seen)
-        pools = size_pools(cfg.model, sc.max_num_seqs, ctx, sc.max_num_batched_tokens, dcp, pool_tokens)
-        if cfg.cache.num_pages is not None:
-            pools["swa_pages"] = max(pools["swa_pages"], cfg.cache.num_pages)
-        has_c128 = any(cfg.model.layer_kind(i) == "c128a" for i in range(cfg.model.num_hidden_layers))
         spec_on = cfg.spec.method == "dspark"
         n_spec = cfg.spec.num_speculative_tokens if spec_on else 0
         if spec_on and draft_weights is None:
@@ -278,15 +261,12 @@ class Engine:
                                  f"[{weights.layer_offset}, {weights.layer_offset + len(weights.layers)})")
         elif cfg.parallel.pp_size > 1:
             raise ValueError("ParallelConfig.pp_size > 1 needs a PipeStage")
-        stage_layers = list(range(*pipe.layer_range(cfg.model.num_hidden_layers))) if pipe is not None else None
-        self.kv = KVManager(cfg.model, self.device, sc.max_num_seqs, ctx + 64, pools["swa_pages"] + (sc.max_num_seqs if spec_on else 0),
-                            pools["c4_pages"], pools["c128_pages"] if has_c128 else 0, sc.max_num_batched_tokens,
-                            layers=stage_layers, extra_swa_layers=cfg.model.n_mtp_layers if spec_on else 0, spec_tokens=n_spec,
-                            dcp_rank=tp_rank if dcp > 1 else 0, dcp_size=dcp)
-        self.model = DSV4Model(cfg.model, weights, self.kv, comm, tp_rank, cfg.parallel.tp_size)
+        family = family_of(cfg.model)
+        self.kv = family.make_cache(cfg, self.device, ctx, comm, tp_rank, pipe)
+        self.model = family.make_model(cfg, weights, self.kv, comm, tp_rank)
         self.model.pipe = pipe
         self.prefix_cache = None
-        if cfg.cache.enable_prefix_caching:
+        if cfg.cache.enable_prefix_caching and family.prefix_cache:
             from .prefix_cache import PrefixCache
             pc = PrefixCache(self.kv)
             self.prefix_cache = pc if pc.enabled else None
@@ -313,6 +293,7 @@ class Engine:
             from ..parallel.eplb import LoadRecorder
             self.model.load_recorder = LoadRecorder(cfg.model.num_hidden_layers, cfg.model.n_routed_experts, self.device)
         self.metrics = Metrics()
+        self._spans = (1, 1)                 # shortest and longest span of the staged step
         self.async_scheduling = sc.async_scheduling and not spec_on and pipe is None
         self._inflight = None                # asynchronous scheduling: the step that is launched and not read yet
         self._async_parity = 0
@@ -384,6 +365,64 @@ class Engine:
         while self.has_work():
             self.step()
         return [self.requests[i].output for i in ids]
+
+    # ---- given tokens (replay, scoring) ---------------------------------------------
+    def open_sequence(self, max_tokens: Optional[int] = None) -> Request:
+        """A request whose tokens the caller supplies step by step (`feed`) instead of sampling them.  It holds a request
+        row and cache pages like any other until `close_sequence`."""
+        if not self.kv.free_rows:
+            raise OutOfPages("no free request row")
+        req = Request(self._next_id, [], SamplingParams(max_tokens=0))
+        self._next_id += 1
+        req.row = self.kv.alloc_row()
+        self.kv.reserve(req.row, max_tokens or self.cfg.sched.max_model_len)
+        return req
+
+    def feed(self, spans: Sequence[Tuple[Request, Sequence[int], Sequence[int]]]) -> Optional[torch.Tensor]:
+        """One step over [(sequence, its next tokens, places among them whose logits are wanted)]: the step function of
+        generation with given tokens instead of sampled ones.  -> fp32 logits [wanted, vocab] on the device in the order of
+        the entries and places, or None when nothing is wanted."""
+        seqs: List[ScheduledSeq] = []
+        rows: List[int] = []
+        t = 0
+        for req, tokens, want in spans:
+            if not tokens:
+                continue
+            start = len(req.prompt)
+            if start + len(tokens) > self.cfg.sched.max_model_len:
+                raise ValueError("sequence exceeds max_model_len")
+            if any(not 0 <= w < len(tokens) for w in want):
+                raise ValueError("a wanted place is outside the step's tokens")
+            req.prompt.extend(int(x) for x in tokens)
+            seqs.append(ScheduledSeq(req, start, len(tokens), False))
+            rows += [t + w for w in want]
+            t += len(tokens)
+        if not seqs:
+            return None
+        if t > self.cfg.sched.max_num_batched_tokens or len(seqs) > self.cfg.sched.max_num_seqs:
+            raise ValueError("step exceeds max_num_batched_tokens or max_num_seqs")
+        t, n_req, _ = self._stage(seqs)
+        self._upload(t, n_req, 0)
+        max_comp_rows = max(1, max(s.start + s.n for s in seqs) // 4)
+        meta = self._build_meta(t, n_req, max_comp_rows, pure_decode=all(s.n == 1 for s in seqs))
+        X = self.model.forward_hidden(meta)
+        logits = None
+        if rows:
+            logits = self.model.compute_logits(self.model.head_hidden(X, torch.tensor(rows, device=self.device))).float()
+        self._queue_status_read()
+        if self.device.type == "cuda":
+            torch.cuda.current_stream().synchronize()
+        self._check_device_status()
+        for s in seqs:
+            s.req.num_computed = s.start + s.n
+        self.metrics.steps_total += 1
+        return logits
+
+    def close_sequence(self, req: Request) -> None:
+        """Give back what the sequence holds."""
+        if not req.finished:
+            req.finished = True
+            self.kv.free_row(req.row)
 
     # ---- device status ---------------------------------------------------------------
     def _agreed_status(self) -> Optional[torch.Tensor]:
@@ -464,6 +503,7 @@ class Engine:
                     trunc = trunc or r.params.truncates
                     ns += 1
         b.n_qstart[len(seqs)] = t
+        self._spans = (min(s.n for s in seqs), max(s.n for s in seqs))
         self.buf.truncating = trunc
         return t, len(seqs), ns
 
@@ -490,14 +530,8 @@ class Engine:
             b.event.record()
         self.h2d_bytes_last = d.h2d_bytes(t, n)
 
-    def _build_meta(self, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False) -> StepMeta:
-        b = self.buf
-        cfg = self.cfg.model
-        tok_req, positions, first, last, sm = A.token_maps(b.d_qstart, b.d_rows, b.d_start, n_req, t_pad,
-                                                           self.kv.swa.table_dev)
-        swa_slots, swa_lens = A.swa_indices(positions, tok_req, self.kv.swa.table_dev, cfg.sliding_window)
-        return StepMeta(b.d_tokens[:t_pad], tok_req, positions, first, last, sm, swa_slots, swa_lens, max_comp_rows,
-                        pure_decode=pure_decode)
+    def _build_meta(self, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False):
+        return self.model.build_meta(self.buf, t_pad, n_req, max_comp_rows, pure_decode, self._spans)
 
     def _run_model(self, t_pad: int, n_req: int, ns: int, max_comp_rows: int, identity_rows: bool = False) -> torch.Tensor:
         """-> sampled tokens [ns] (device).
@@ -727,7 +761,7 @@ class Engine:
         m = self.metrics
         m.num_requests_running = self.sched.num_running
         m.num_requests_waiting = self.sched.num_waiting
-        m.kv_cache_usage = self.kv.c4.pages_in_use / max(1, self.kv.c4.num_pages)
+        m.kv_cache_usage = self.kv.usage()
         pc = self.prefix_cache
         if pc is not None:
             m.prefix_cache_queries, m.prefix_cache_hits, m.prefix_cache_hit_tokens = pc.queries, pc.hits, pc.hit_tokens
@@ -846,7 +880,7 @@ class Engine:
             self.d_spec_temp[:nb].copy_(temps[:nb], non_blocking=True)
         full = nb == len(seqs) and all(s.n_sample == 1 + n_spec for s in seqs)
         if self.use_graphs and full and t <= self.cfg.sched.graph_cap and not self.buf.truncating:
-            rows_bucket = ((max_comp_rows + 64) // 2048 + 1) * 2048
+            rows_bucket = self.model.decode_bucket(max_comp_rows)
             key = ("spec", n_req, rows_bucket)
             g = self._graphs.get(key)
             if g is None:
@@ -907,9 +941,7 @@ class Engine:
         bucket = 1
         while bucket < n_req:
             bucket *= 2
-        # compressed-row bound baked into the graph: next multiple of 2048 with 64 rows of headroom,
-        # so a sequence crosses into a new graph only every 8192 tokens
-        rows_bucket = ((max_comp_rows + 64) // 2048 + 1) * 2048
+        rows_bucket = self.model.decode_bucket(max_comp_rows)
         key = (bucket, rows_bucket)
         if n_req < bucket:
             # padding rows: empty query ranges => request -1, nothing is read or written for them

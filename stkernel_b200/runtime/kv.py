@@ -25,7 +25,7 @@ from typing import Callable, Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import ModelConfig
+from ..config import HybridConfig, ModelConfig
 from ..ops.cache import PAGE, PagedCache
 from .planning import dcp_owner
 
@@ -182,7 +182,54 @@ class GroupTable:
         return below(self.hi[row]) - below(self.lo[row])
 
 
-class KVManager:
+class CacheManager:
+    """What the scheduler and the engine ask of any model family's caches: request rows, page groups, admission."""
+
+    def __init__(self, device, max_requests: int):
+        self.device = torch.device(device)
+        self.max_requests = max_requests
+        self.free_rows = list(range(max_requests - 1, -1, -1))
+        # context tokens promised to admitted requests, in whatever unit the family's admission counts (pages)
+        self.reserved: Dict[int, int] = {}
+
+    def groups(self) -> List[GroupTable]:
+        raise NotImplementedError
+
+    def alloc_row(self) -> int:
+        if not self.free_rows:
+            raise OutOfPages("no free request row")
+        return self.free_rows.pop()
+
+    def free_row(self, row: int) -> None:
+        for g in self.groups():
+            g.release_all(row)
+        self.reserved.pop(row, None)
+        self.free_rows.append(row)
+
+    def sync(self, parity: int = 0) -> None:
+        for g in self.groups():
+            g.sync(parity)
+
+    def reserve(self, row: int, context: int) -> None:
+        """Promise request `row` room for a context of `context` tokens."""
+
+    def prepare(self, row: int, start_pos: int, n_tokens: int, lookback: Optional[int] = None) -> None:
+        """Make resident what a step that appends positions [start, start+n) to request `row` touches."""
+        raise NotImplementedError
+
+    def fits(self, context: int) -> bool:
+        """Whether a request of this context could ever be admitted."""
+        return True
+
+    def can_admit(self, n_tokens: int, context: int) -> bool:
+        raise NotImplementedError
+
+    def usage(self) -> float:
+        """Share of the pages in use (the gauge of the serving metrics)."""
+        raise NotImplementedError
+
+
+class KVManager(CacheManager):
     """Owns the group tables, the per-layer cache tensors and the request-row allocator."""
 
     def __init__(self, cfg: ModelConfig, device, max_requests: int, max_model_len: int, swa_pages: int,
@@ -191,10 +238,9 @@ class KVManager:
         """dcp_size > 1: the ratio-4 caches (compressed latent rows and indexer keys, the part of the KV that grows
         with the context) are dealt page by page over the ranks; `c4_pages` is then this rank's pool.  The
         sliding-window and ratio-128 caches stay replicated (a window, and 1/32 of the ratio-4 rows)."""
+        super().__init__(device, max_requests)
         self.cfg = cfg
         self.dcp_rank, self.dcp_size = dcp_rank, dcp_size
-        self.device = torch.device(device)
-        self.max_requests = max_requests
         fp8 = cfg.kv_cache_dtype == "fp8_ds_mla"
         D, Rd = cfg.head_dim, cfg.qk_rope_head_dim
         # the block table spans the whole context; SWA residency is bounded by window + chunk
@@ -232,24 +278,14 @@ class KVManager:
             elif kind == "c128a":
                 self.comp_cache[li] = PagedCache.allocate(self.c128.num_pages, D, Rd, fp8, "latent", self.device)
                 self.comp_state[li] = torch.zeros(max_requests, ring128, 2 * D, dtype=torch.float32, device=self.device)
-        self.free_rows = list(range(max_requests - 1, -1, -1))
         self.spec_tokens = spec_tokens
-        # ratio-4 pages promised to admitted requests for their whole context (allocated page by page as they grow):
-        # admission counts the part not yet allocated as taken, so a pool smaller than max_requests x max_model_len
-        # makes requests wait instead of running out of pages in the middle of a step
-        self.reserved: Dict[int, int] = {}
+        # `reserved` holds the ratio-4 pages promised to admitted requests for their whole context (allocated page by
+        # page as they grow): admission counts the part not yet allocated as taken, so a pool smaller than
+        # max_requests x max_model_len makes requests wait instead of running out of pages in the middle of a step
 
     # ---- request rows -------------------------------------------------------
-    def alloc_row(self) -> int:
-        if not self.free_rows:
-            raise OutOfPages("no free request row")
-        return self.free_rows.pop()
-
-    def free_row(self, row: int) -> None:
-        for g in (self.swa, self.c4, self.c128):
-            g.release_all(row)
-        self.reserved.pop(row, None)
-        self.free_rows.append(row)
+    def groups(self) -> List[GroupTable]:
+        return [self.swa, self.c4, self.c128]
 
     def reserve(self, row: int, context: int) -> None:
         """Promise request `row` the ratio-4 pages of a context of `context` tokens."""
@@ -294,9 +330,8 @@ class KVManager:
         return (bool(self.free_rows) and len(self.swa.free) >= need_swa
                 and len(self.c4.free) - self.promised() >= need_c4)
 
-    def sync(self, parity: int = 0) -> None:
-        for g in (self.swa, self.c4, self.c128):
-            g.sync(parity)
+    def usage(self) -> float:
+        return self.c4.pages_in_use / max(1, self.c4.num_pages)
 
     def bytes_allocated(self) -> int:
         n = 0
@@ -305,6 +340,80 @@ class KVManager:
         for d in (self.comp_state, self.idx_state):
             n += sum(t.numel() * 4 for t in d.values())
         return n
+
+
+class HybridKVManager(CacheManager):
+    """Caches of a decoder described layer by layer (`HybridConfig`).
+
+    * attention layers: paged rows, one page group per distinct window (layers of the same window share the block table).
+      A page holds `[kv_heads, PAGE, row]`; a row is the projected key followed by the rotated copy of its first
+      `rot_dims` dimensions, padded to 16 bytes.  The projected key is the value, and with its rotated head replaced it is
+      the key, so nothing is stored twice.  Pages are released as they leave the window.
+    * mLSTM layers: per request row the matrix memory `[heads, dim, vdim]`, the normaliser `[heads, dim]` and the running
+      maximum `[heads]`, fp32.  Nothing is cleared when a row changes hands: a span that starts at position 0 reads zeros.
+    """
+
+    def __init__(self, cfg: HybridConfig, device, max_requests: int, max_model_len: int, max_chunk: int,
+                 extra_pages: int = 0):
+        super().__init__(device, max_requests)
+        self.cfg = cfg
+        dt = torch.float32 if cfg.dtype == "float32" else torch.bfloat16
+        self.max_model_len = max_model_len
+        pages_ctx = (max_model_len + PAGE - 1) // PAGE + 1
+        self.by_window: Dict[int, GroupTable] = {}
+        for w in cfg.windows():
+            pages = hybrid_pool_pages(w, max_requests, max_model_len, max_chunk) + extra_pages
+            self.by_window[w] = GroupTable(f"window{w}", pages, max_requests, pages_ctx, self.device, 1.0)
+        self.kv_cache: Dict[int, torch.Tensor] = {}
+        self.state: Dict[int, Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = {}
+        for li, l in enumerate(cfg.layers):
+            m = l.mixer
+            if m.kind == "attention":
+                g = self.by_window[m.window]
+                self.kv_cache[li] = torch.zeros(g.num_pages, m.kv_heads, PAGE, kv_row_width(m.dim, m.rot_dims), dtype=dt,
+                                                device=self.device)
+            else:
+                z = lambda *s: torch.zeros(max_requests, m.heads, *s, dtype=torch.float32, device=self.device)
+                self.state[li] = (z(m.dim, m.vdim), z(m.dim), z())
+
+    def groups(self) -> List[GroupTable]:
+        return list(self.by_window.values())
+
+    def group_of(self, layer: int) -> GroupTable:
+        return self.by_window[self.cfg.layers[layer].mixer.window]
+
+    def prepare(self, row: int, start_pos: int, n_tokens: int, lookback: Optional[int] = None) -> None:
+        end = start_pos + n_tokens
+        for w, g in self.by_window.items():
+            lo = max(0, start_pos - w + 1)
+            g.release_before(row, lo // PAGE)
+            g.ensure(row, lo // PAGE, (end - 1) // PAGE)
+
+    def can_admit(self, n_tokens: int, context: int) -> bool:
+        n = min(n_tokens, context)
+        return bool(self.free_rows) and all(len(g.free) >= n // PAGE + 2 for g in self.by_window.values())
+
+    def usage(self) -> float:
+        total = sum(g.num_pages for g in self.by_window.values())
+        if total == 0:
+            return (self.max_requests - len(self.free_rows)) / self.max_requests
+        return sum(g.pages_in_use for g in self.by_window.values()) / total
+
+    def bytes_allocated(self) -> int:
+        n = sum(t.numel() * t.element_size() for t in self.kv_cache.values())
+        return n + sum(t.numel() * 4 for st in self.state.values() for t in st)
+
+
+def kv_row_width(dim: int, rot_dims: int) -> int:
+    """Elements of a cached row (key as projected, rotated head), a multiple of 8 so that rows stay 16-byte aligned."""
+    return (dim + rot_dims + 7) // 8 * 8
+
+
+def hybrid_pool_pages(window: int, max_requests: int, max_context: int, max_chunk: int) -> int:
+    """Pages of one window group so that `max_requests` requests never run out: the window (or the whole context, if that
+    is shorter) of each, and one step's new tokens."""
+    span = min(window, max_context)
+    return max_requests * ((span + PAGE - 1) // PAGE + 2) + (max_chunk + PAGE - 1) // PAGE + 2
 
 
 def size_pools(cfg: ModelConfig, max_requests: int, max_context: int, max_chunk: int, dcp_size: int = 1,
