@@ -14,6 +14,8 @@ from ..ops import functional as Fn
 
 
 class Decoder:
+    recurrent = False          # running a step twice changes more than running it once (a state advances)
+
     def __init__(self, device, comm=None, tp_rank: int = 0, tp_size: int = 1):
         self.device = torch.device(device)
         self.comm = comm

@@ -177,6 +177,7 @@ class HybridModel(Decoder):
         self.kv = kv
         self.act = HB.act_dtype(cfg.dtype, self.device)
         self.width = _pad(cfg.hidden_size)
+        self.recurrent = any(l.mixer.kind == "mlstm" for l in cfg.layers)
         self.on_layer = None                # optional hook (layer index, residual [T, W] fp32) after each layer
 
     def build_meta(self, buf, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False,

@@ -1007,7 +1007,12 @@ class DecodeGraph:
     def __init__(self, eng: Engine, bucket: int, rows_bucket: int):
         self.eng = eng
         self.bucket = bucket
-        # warm-up outside capture (allocates scratch, configures kernels), then capture
+        # warm-up outside capture (allocates scratch, configures kernels), then capture.  A recurrent state must not advance
+        # here: such a model warms up on empty query ranges (every row is padding) and gets its ranges back for the replay.
+        qstart = eng.buf.d_qstart[:bucket + 1]
+        ranges = qstart.clone() if eng.model.recurrent else None
+        if ranges is not None:
+            qstart.zero_()
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -1021,6 +1026,8 @@ class DecodeGraph:
         with torch.cuda.graph(self.graph, stream=_capture_stream(eng.device)):
             self.out = eng._run_model(bucket, bucket, bucket, rows_bucket, identity_rows=True)
         self.launches_per_replay = _lib.launch_count - before
+        if ranges is not None:
+            qstart.copy_(ranges)
         _after_capture_rendezvous(eng)
 
     def replay(self) -> torch.Tensor:
