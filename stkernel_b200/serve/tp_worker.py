@@ -8,7 +8,7 @@ The engines advance in lockstep: before each step rank 0 broadcasts the control 
 them in the same order and calls `step()`, so schedulers, page tables and seeded samplers stay
 identical and the only device collectives are the model's own.  A follower that hears nothing for
 `--heartbeat-timeout` seconds exits instead of waiting forever in a collective.  With `--model`
-absent, random weights of the flagship architecture are served (benchmarks, tests).
+absent, random weights of the flagship architecture, or of the one in `--model-config`, are served (benchmarks, tests).
 
 Flag names follow the reference's serve script (launchers/start-hy4-tp4.sh:354-392).
 """
@@ -118,16 +118,22 @@ def follower_loop(engine: Engine, cpu_group, heartbeat_timeout: float = 120.0) -
 
 
 def build_engine(a, rank: int, world: int, device) -> Tuple[Engine, Any]:
-    from ..models.dsv4 import RandomSource, build_model_weights
+    from ..models.registry import config_from_json, family_of, load_model_config
+    from ..models.sources import RandomSource
     spec_cfg = SpecConfig()
     if a.speculative_config:
         sc = json.loads(a.speculative_config)
         spec_cfg = SpecConfig(method=sc.get("method", "dspark"), num_speculative_tokens=int(sc.get("num_speculative_tokens", 5)),
                               markov_topk=int(sc.get("markov_topk", 512)), markov_sideload=os.environ.get("STK_MARKOV_SIDELOAD", ""))
     if a.model:
-        from ..models.loader import CheckpointSource, load_model_config
-        mcfg = load_model_config(a.model)
+        from ..models.loader import CheckpointSource
+        mcfg = load_model_config(a.model, getattr(a, "dtype", "") or None)
         src = CheckpointSource(a.model)
+    elif getattr(a, "model_config", ""):
+        # random weights of an architecture given by its config.json
+        with open(a.model_config) as f:
+            mcfg = config_from_json(json.load(f), getattr(a, "dtype", "") or None)
+        src = RandomSource(0)
     else:
         n_mtp = 3 if spec_cfg.method == "dspark" else 0
         if a.tiny:
@@ -165,8 +171,10 @@ def build_engine(a, rank: int, world: int, device) -> Tuple[Engine, Any]:
             group = groups[pp_rank]
         comm = Communicator(group=group, device=device,
                             use_symm=pp == 1 and os.environ.get("STK_ONESHOT_AR", "1") == "1" and device.type == "cuda")
-    weights = build_model_weights(mcfg, src, device, tp_rank, tp, head_fp8=mcfg.dense_dtype == "fp8" and device.type == "cuda",
-                                  layer_range=layer_range)
+    if device.type == "cuda":
+        from ..ops import _lib
+        _lib.use_family(family_of(mcfg).name, family_of(mcfg).native_sources)
+    weights = family_of(mcfg).build_weights(mcfg, src, device, tp_rank, tp, layer_range=layer_range)
     draft = None
     if spec_cfg.method == "dspark":
         from ..spec.dspark import build_draft_weights
@@ -182,9 +190,12 @@ def build_engine(a, rank: int, world: int, device) -> Tuple[Engine, Any]:
     return eng, mcfg
 
 
-def main(argv: Optional[Sequence[str]] = None) -> int:
+def make_parser() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser()
     ap.add_argument("--model", default="")
+    ap.add_argument("--model-config", default="", help="without --model: config.json of the architecture to serve with random weights")
+    ap.add_argument("--dtype", choices=("", "bfloat16", "float32"), default="",
+                    help="compute type, for architectures that offer a choice (Timalorn: bfloat16 or float32)")
     ap.add_argument("--tokenizer", default="")
     ap.add_argument("--served-model-name", default="deepseek-v4-flash")
     ap.add_argument("--host", default="127.0.0.1")
@@ -212,8 +223,17 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     ap.add_argument("--layers", type=int, default=2, help="random-weight mode: decoder layers")
     ap.add_argument("--tiny", action="store_true", help="random-weight mode: CPU-sized architecture")
     ap.add_argument("--heartbeat-timeout", type=float, default=120.0)
-    a = ap.parse_args(argv)
+    return ap
 
+
+def make_tokenizer(a, mcfg) -> ChatTokenizer:
+    """The checkpoint's tokenizer, or bytes when there is none (random weights, a checkpoint of weights alone)."""
+    path = a.tokenizer or (a.model if a.model and os.path.exists(os.path.join(a.model, "tokenizer.json")) else "")
+    return ChatTokenizer(HFTokenizer(path) if path else ByteTokenizer(mcfg.vocab_size))
+
+
+def main(argv: Optional[Sequence[str]] = None) -> int:
+    a = make_parser().parse_args(argv)
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local = int(os.environ.get("LOCAL_RANK", "0"))
@@ -234,7 +254,7 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     if rank != 0:
         return follower_loop(eng, cpu_group, a.heartbeat_timeout)
     import uvicorn
-    tok = ChatTokenizer(HFTokenizer(a.tokenizer or a.model) if (a.tokenizer or a.model) else ByteTokenizer(mcfg.vocab_size))
+    tok = make_tokenizer(a, mcfg)
     kwargs = json.loads(a.default_chat_template_kwargs) if a.default_chat_template_kwargs else None
     app = create_app(eng, tok, a.served_model_name, default_thinking=a.default_thinking, profile_dir=a.profiler_dir,
                      default_chat_template_kwargs=kwargs,
