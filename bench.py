@@ -86,6 +86,16 @@ class ClockSampler:
                 "samples": len(self.samples), "power_w_max": max(float(s[2]) for s in self.samples)}
 
 
+def hybrid_arm(args) -> None:
+    import torch
+    from stkernel_b200.bench import hybrid_bench
+    torch.cuda.set_device(0)
+    with ClockSampler(0) as clocks:
+        res = hybrid_bench.run([int(x) for x in args.hybrid_sizes.split(",")])
+    print(hybrid_bench.render(res), file=sys.stderr)
+    print(json.dumps({"metric": "hybrid_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -98,7 +108,13 @@ def main() -> None:
     ap.add_argument("--skip-spec", action="store_true")
     ap.add_argument("--long-ctx", type=int, default=131072)
     ap.add_argument("--no-fused", action="store_true", help="NCCL-after-GEMM baseline collectives")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="instead of the flagship: the Timalorn decoder beside the flagship's architecture at equal width "
+                         "and depth, prefill, decode and per-kernel rooflines (one JSON line; table on stderr)")
+    ap.add_argument("--hybrid-sizes", default="2048,4096", help="widths for --hybrid")
     args = ap.parse_args()
+    if args.hybrid:
+        return hybrid_arm(args)
     if args.impl == "reference":
         return reference_arm(args)
 
