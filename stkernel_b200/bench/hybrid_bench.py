@@ -127,7 +127,7 @@ HYBRID_GROUPS = [("projections", ("gemm", "skinny")), ("window_attention", ("win
                  ("window_attention combine", ("window_attn_combine",)), ("kv insert", ("window_kv_insert",)),
                  ("add + layer norm", ("add_layer_norm",)), ("feed-forward join", ("join_glu",)),
                  ("mlstm scan", ("mlstm_scan_kernel",)), ("mlstm chunk states", ("mlstm_chunk_state",)),
-                 ("mlstm chunk scan", ("mlstm_chunk_scan",)), ("mlstm chunk outputs", ("mlstm_chunk_out",)),
+                 ("mlstm chunk gates", ("mlstm_chunk_gates",)), ("mlstm chunk outputs", ("mlstm_chunk_out",)),
                  ("mlstm finish", ("mlstm_finish",)), ("embedding", ("embed_scaled",))]
 DSV4_GROUPS = [("projections", ("gemm_", "skinny")), ("sparse attention", ("sparse_mla", "mla_decode")),
                ("sparse attention merge", ("mla_merge", "mla_combine")),
@@ -178,8 +178,8 @@ def hybrid_work(cfg: HybridConfig, spans: List[Tuple[int, int]], decode: bool) -
                 add("mlstm scan", 4.0 * T * H * D * V, 2 * state * len(spans) + T * H * (4.0 * D + 6.0 * V))
             else:
                 chunks = sum(-(-n // 64) for _, n in spans)
-                add("mlstm chunk states", 2.0 * T * H * D * V, T * H * 2.0 * (D + V) + chunks * state)
-                add("mlstm chunk scan", 0, 2 * chunks * state + 2 * state * len(spans))
+                add("mlstm chunk gates", 0, T * H * (8.0 + 12.0))
+                add("mlstm chunk states", 2.0 * T * H * D * V, T * H * 2.0 * (D + V) + chunks * state + 2 * state * len(spans))
                 add("mlstm chunk outputs", 2.0 * T * H * D * V + T * H * 64.0 * (D + V), T * H * (4.0 * D + 6.0 * V) + chunks * state)
             add("mlstm finish", 0, T * (H * V * (4.0 + 2 + 2) + 6.0 * ff))
     add("embedding", 0, T * W * 6.0)

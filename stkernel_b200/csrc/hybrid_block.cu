@@ -1,16 +1,9 @@
 // Residual-side kernels of the parallel block (models/hybrid.py): scaled embedding into an fp32 residual, residual add fused
 // with the next layer norm, and the feed-forward half of the joined sublayer buffer.
 #define STK_PDL_CLASS 4
-#include "common.cuh"
+#include "hybrid_block.cuh"
 
 namespace stk {
-
-template <typename T> __device__ __forceinline__ float ld_act(const T* p);
-template <> __device__ __forceinline__ float ld_act<float>(const float* p) { return *p; }
-template <> __device__ __forceinline__ float ld_act<__nv_bfloat16>(const __nv_bfloat16* p) { return bf16_to_f(*p); }
-template <typename T> __device__ __forceinline__ void st_act(T* p, float v);
-template <> __device__ __forceinline__ void st_act<float>(float* p, float v) { *p = v; }
-template <> __device__ __forceinline__ void st_act<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
 template <typename E>
 __global__ void __launch_bounds__(256)
@@ -97,30 +90,7 @@ join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int f
   const int base = blockIdx.x * blockDim.x * 8 + threadIdx.x * 8;      // eight columns per thread, from o0 on
   if (blockIdx.x == 0)
     for (int i = mix + threadIdx.x; i < o0; i += blockDim.x) st_act(o + i, 0.f);
-  const int n = cols - o0;
-  if (base >= n) return;
-  if (sizeof(A) == 2 && base + 8 <= ff && (ldo & 7) == 0 && (ldp & 7) == 0) {
-    const uint4 gv = *reinterpret_cast<const uint4*>(pg + base), uv = *reinterpret_cast<const uint4*>(pu + base);
-    const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
-    const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uv);
-    uint4 ov;
-    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
-      o2[j] = __floats2bfloat162_rn(g.x / (1.f + __expf(-g.x)) * u.x, g.y / (1.f + __expf(-g.y)) * u.y);
-    }
-    *reinterpret_cast<uint4*>(o + o0 + base) = ov;
-    return;
-  }
-  for (int j = base; j < base + 8 && j < n; ++j) {
-    float v = 0.f;
-    if (j < ff) {
-      const float g = ld_act(pg + j);
-      v = g / (1.f + expf(-g)) * ld_act(pu + j);
-    }
-    st_act(o + o0 + j, v);
-  }
+  glu_columns(pg, pu, o + o0, base, ff, cols - o0, (ldo & 7) == 0 && (ldp & 7) == 0);
 }
 
 }  // namespace stk

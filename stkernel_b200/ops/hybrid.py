@@ -185,7 +185,7 @@ def mlstm(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, ga
         L = MLSTM_CHUNK
         chunks = t // L + meta.n_req
         a_ws = scratch("mlstm.gates", (chunks * h * _lib.query("stk_mlstm_gate_slot"),), F32, dev)
-        u_ws = scratch("mlstm.states", (chunks * h * d * (v + 1),), F32, dev)
+        u_ws = scratch("mlstm.states", (chunks * h * _lib.query("stk_mlstm_state_slot", d, v),), F32, dev)
         _lib.call("stk_mlstm_chunks", *args, MLSTM_CHUNK_SPAN, a_ws, u_ws, chunks, t, _lib.stream())
     go, uo, ff = glu if glu is not None else (0, 0, 0)
     _lib.call("stk_mlstm_finish", num, den, mt, m, p.norm, float(p.eps), meta.tok_req, meta.positions, meta.last_pos, proj,
