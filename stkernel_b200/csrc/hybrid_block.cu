@@ -15,6 +15,18 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
   const long long id = ids[t];
   const bool ok = id >= 0 && id < vocab;
   if (!ok && threadIdx.x == 0) set_status(status, kBadIndex, t);
+  if (sizeof(E) == 2 && (W & 7) == 0 && (ldx & 3) == 0) {
+    for (int i = threadIdx.x * 8; i < W; i += blockDim.x * 8) {
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (ok) v = __ldg(reinterpret_cast<const uint4*>(embed + id * W + i));
+      float2 f[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) f[j] = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
+      *reinterpret_cast<float4*>(x + t * ldx + i) = make_float4(f[0].x * scale, f[0].y * scale, f[1].x * scale, f[1].y * scale);
+      *reinterpret_cast<float4*>(x + t * ldx + i + 4) = make_float4(f[2].x * scale, f[2].y * scale, f[3].x * scale, f[3].y * scale);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < W; i += blockDim.x)
     x[t * ldx + i] = ok ? ld_act(embed + id * W + i) * scale : 0.f;
 }
@@ -22,7 +34,7 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
 // x[r] += y[r]; h[t] = layer_norm(x[r]) * w with r = rows ? rows[t] : t (with `rows` the sum is not written back).  The
 // row stays in shared memory between the three passes (mean, squared deviations, output), all in fp32.
 template <typename O>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 add_layer_norm_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy,
                       const float* __restrict__ w, O* __restrict__ h, long long ldh, int W, int width, float eps,
                       const int64_t* __restrict__ rows) {
@@ -122,10 +134,12 @@ STK_API int stk_add_layer_norm(float* x, long long ldx, const float* y, long lon
             cudaSuccess)
       return -3;
   }
+  // few rows: a wide row is spread over more threads (the step waits for this kernel); many rows: more rows at once
+  const int threads = T > 148 || W <= 1024 ? 256 : (W <= 2048 ? 512 : 1024);
   if (h_fp32)
-    launch_pdl(add_layer_norm_kernel<float>, dim3(T), dim3(256), smem, st, x, ldx, y, ldy, w, (float*)h, ldh, W, width, eps, rows);
+    launch_pdl(add_layer_norm_kernel<float>, dim3(T), dim3(threads), smem, st, x, ldx, y, ldy, w, (float*)h, ldh, W, width, eps, rows);
   else
-    launch_pdl(add_layer_norm_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, st, x, ldx, y, ldy, w, (__nv_bfloat16*)h, ldh, W,
+    launch_pdl(add_layer_norm_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, st, x, ldx, y, ldy, w, (__nv_bfloat16*)h, ldh, W,
                width, eps, rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

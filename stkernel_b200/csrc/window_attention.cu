@@ -8,7 +8,7 @@
 //   window_attn_simt       any size and type, fp32 arithmetic throughout: one CTA per (token, head)
 //   window_attn_tokens     bf16, spans of a few tokens (decode): one CTA per (token, key/value head, key range); the heads of
 //                          the group are the 16 MMA rows, four warps take 16 of every 64 keys each
-//   window_attn_tiles      bf16, prompt portions: 64 rows (tokens x heads of the group) per CTA, key pages through two stages
+//   window_attn_tiles      bf16, prompt portions: 128 rows (tokens x heads of the group) per CTA, key pages through two stages
 // Probabilities enter the value product as bf16 pairs (high part and remainder), so they keep 16 mantissa bits.
 #define STK_PDL_CLASS 8
 #include "common.cuh"
@@ -39,35 +39,61 @@ __device__ __forceinline__ float cap_score(float s, float cap, float two_over_ca
   return cap - __fdividef(2.f * cap, 1.f + e);
 }
 
+// One warp per token; cos and sin of its position go through shared memory.  vec: rows and heads are 16-byte aligned bf16.
 template <typename A>
 __global__ void __launch_bounds__(128)
-window_kv_insert_kernel(const WinArgs a) {
-  __shared__ float2 cs[512];
+window_kv_insert_kernel(const WinArgs a, int T, int vec) {
+  extern __shared__ float2 cs_all[];                                        // [4][rd / 2]
   pdl_wait();
   pdl_trigger();
-  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long t = blockIdx.x * 4ll + warp;
+  if (t >= T) return;
   const int req = a.tok_req[t];
   const long long pos = a.positions[t];
   if (req < 0 || pos < 0) return;
   const int page = a.table[static_cast<long long>(req) * a.bt_stride + pos / kPage];
   if (page < 0) return;
   const int half = a.rd >> 1;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+  float2* cs = cs_all + warp * half;
+  for (int i = lane; i < half; i += 32) {
     float s, c;
     sincosf(static_cast<float>(pos) * a.freq[i], &s, &c);
     cs[i] = make_float2(c * a.mag, s * a.mag);
   }
-  __syncthreads();
+  __syncwarp();
   const A* k = reinterpret_cast<const A*>(a.proj) + t * a.ldp + a.k_off;
   A* base = reinterpret_cast<A*>(a.cache) + (static_cast<long long>(page) * a.G * kPage + pos % kPage) * a.row;
-  for (int e = threadIdx.x; e < a.G * a.D; e += blockDim.x) {
-    const int g = e / a.D, d = e % a.D;
-    base[static_cast<long long>(g) * kPage * a.row + d] = k[e];
+  const long long gstep = static_cast<long long>(kPage) * a.row;
+  if (sizeof(A) == 2 && vec) {
+    const int c8 = a.D >> 3, h8 = half >> 3;
+    for (int e = lane; e < a.G * c8; e += 32) {
+      const int g = e / c8, c = (e - g * c8) * 8;
+      *reinterpret_cast<uint4*>(base + g * gstep + c) = *reinterpret_cast<const uint4*>(k + g * a.D + c);
+    }
+    for (int e = lane; e < a.G * h8; e += 32) {
+      const int g = e / h8, c = (e - g * h8) * 8;
+      const uint4 uu = *reinterpret_cast<const uint4*>(k + g * a.D + c), vv = *reinterpret_cast<const uint4*>(k + g * a.D + half + c);
+      uint4 ru, rv;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 u = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&uu)[i]);
+        const float2 v = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&vv)[i]);
+        const float2 w0 = cs[c + 2 * i], w1 = cs[c + 2 * i + 1];
+        reinterpret_cast<__nv_bfloat162*>(&ru)[i] = __floats2bfloat162_rn(u.x * w0.x - v.x * w0.y, u.y * w1.x - v.y * w1.y);
+        reinterpret_cast<__nv_bfloat162*>(&rv)[i] = __floats2bfloat162_rn(v.x * w0.x + u.x * w0.y, v.y * w1.x + u.y * w1.y);
+      }
+      A* r = base + g * gstep + a.D;
+      *reinterpret_cast<uint4*>(r + c) = ru;
+      *reinterpret_cast<uint4*>(r + half + c) = rv;
+    }
+    return;
   }
-  for (int e = threadIdx.x; e < a.G * half; e += blockDim.x) {
+  for (int e = lane; e < a.G * a.D; e += 32) base[e / a.D * gstep + e % a.D] = k[e];
+  for (int e = lane; e < a.G * half; e += 32) {
     const int g = e / half, i = e % half;
     const float u = to_f(k[g * a.D + i]), v = to_f(k[g * a.D + half + i]);
-    A* r = base + static_cast<long long>(g) * kPage * a.row + a.D;
+    A* r = base + g * gstep + a.D;
     from_f(r + i, u * cs[i].x - v * cs[i].y);
     from_f(r + half + i, v * cs[i].x + u * cs[i].y);
   }
@@ -449,27 +475,39 @@ window_attn_combine_kernel(const WinArgs a, const int* __restrict__ first_pos, c
 }
 
 // ---- prompt portions --------------------------------------------------------------------------------
-constexpr int kTileRows = 64;
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
-template <int NV>
-__global__ void __launch_bounds__(128)
+// WARPS x 16 rows per CTA; scores and maxima in units of log2(e).
+template <int NV, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32, 2)
 window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, const int* __restrict__ req_rows,
                          const int* __restrict__ start_pos, int n_req, int min_span, int gs) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
+  constexpr int kThreads = WARPS * 32, kRows = WARPS * 16;
   const int stride = win_stride(a.row);
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);           // [64][stride]
-  __nv_bfloat16* st = qs + kTileRows * stride;                              // two stages of [64][stride]
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);           // [kRows][stride]
+  __nv_bfloat16* st = qs + kRows * stride;                                  // two stages of [64][stride]
   __shared__ int s_find[2];
   pdl_wait();
   pdl_trigger();
-  const int bq = kTileRows / gs;                                            // tokens per tile
+  const int bq = kRows / gs;                                                // tokens per tile
   if (threadIdx.x == 0) {
     int left = blockIdx.x, ri = -1;
     for (int i = 0; i < n_req; ++i) {
       const int n = query_start[i + 1] - query_start[i];
       if (n < min_span) continue;
       const int tiles = (n + bq - 1) / bq;
-      if (left < tiles) { ri = i; break; }
+      if (left < tiles) { ri = i; left = tiles - 1 - left; break; }        // the tiles with the most keys first
       left -= tiles;
     }
     s_find[0] = ri;
@@ -488,11 +526,13 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   auto tok_of = [&](int r) { const int q = r / gs; return q < n_tok ? q0 + off + q : -1; };
   auto head_of = [&](int r) { const int h = h0 + r % gs; return r / gs < n_tok && h < h_end ? h : -1; };
-  fill_queries(qs, stride, a, kTileRows, gs, reinterpret_cast<float2*>(st), tok_of, head_of, 128);
+  fill_queries(qs, stride, a, kRows, gs, reinterpret_cast<float2*>(st), tok_of, head_of, kThreads);
   __syncthreads();
-  zero_pad_columns(st, 2 * kPage, stride, a.row, 128);
+  zero_pad_columns(st, 2 * kPage, stride, a.row, kThreads);
   const int ks0 = a.rd / 16, ks1 = (a.D + a.rd + 15) / 16;
-  const float toc = a.softcap > 0.f ? 2.f / a.softcap : 0.f;
+  const bool capped = a.softcap > 0.f;
+  const float c_in = capped ? a.scale * 2.f * kLog2e / a.softcap : a.scale * kLog2e;
+  const float c_cap = a.softcap * kLog2e, c_two = -2.f * c_cap;
   float o[NV][4], m[2], l[2] = {0.f, 0.f};
   int rel[2];                                                               // the row's token within the tile
 #pragma unroll
@@ -500,7 +540,7 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
     const int row = warp * 16 + (lane >> 2) + r * 8;
     rel[r] = row / gs;
     const int h = head_of(row);
-    m[r] = h >= 0 && a.sink != nullptr ? a.sink[h] : -INFINITY;
+    m[r] = h >= 0 && a.sink != nullptr ? a.sink[h] * kLog2e : -INFINITY;
     // each of the four lanes of a row keeps a partial denominator: the sink is counted by one of them
     if (h >= 0 && a.sink != nullptr && (lane & 3) == 0) l[r] = 1.f;
   }
@@ -509,78 +549,89 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
 #pragma unroll
     for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
   const int pa = static_cast<int>(lo / kPage), pb = static_cast<int>(last / kPage) + 1;
-  load_page(st, stride, a, bt, g, pa, lo, last, 128);
+  load_page(st, stride, a, bt, g, pa, lo, last, kThreads);
   cp_async_commit();
+  const __nv_bfloat16* q_frag = qs + (warp * 16 + (lane & 15)) * stride + (lane >> 4) * 8;
   for (int lp = pa; lp < pb; ++lp) {
     const __nv_bfloat16* cur = st + ((lp - pa) & 1) * kPage * stride;
-    if (lp + 1 < pb) load_page(st + ((lp + 1 - pa) & 1) * kPage * stride, stride, a, bt, g, lp + 1, lo, last, 128);
+    cp_async_wait<0>();
+    __syncthreads();                                                        // this page is in; the other stage is free
+    if (lp + 1 < pb) load_page(st + ((lp + 1 - pa) & 1) * kPage * stride, stride, a, bt, g, lp + 1, lo, last, kThreads);
     cp_async_commit();
-    cp_async_wait<1>();
-    __syncthreads();
-    float s[4][2][4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) s[i][j][k] = 0.f;
-    for (int ks = ks0; ks < ks1; ++ks) {
-      uint32_t af[4];
-      ldsm4(af, qs + (warp * 16 + (lane & 15)) * stride + ks * 16 + (lane >> 4) * 8);
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        uint32_t bf[4];
-        ldsm4(bf, cur + (i * 16 + (lane >> 4) * 8 + (lane & 7)) * stride + ks * 16 + ((lane >> 3) & 1) * 8);
-        mma16816(s[i][0], af, bf[0], bf[1]);
-        mma16816(s[i][1], af, bf[2], bf[3]);
-      }
-    }
     const long long base = static_cast<long long>(lp) * kPage;
     const bool edge = base + kPage - 1 > first || base < last - a.window + 1;
     // key position relative to the tile's first token, so that the window test is on small ints
     const int kr = static_cast<int>(base - first) + (lane & 3) * 2;
-    float mx[2] = {m[0], m[1]};
+#pragma unroll 1
+    for (int kh = 0; kh < kPage; kh += 32) {
+      const __nv_bfloat16* keys = cur + kh * stride;
+      float s[2][2][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
+        for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          float v = s[i][j][k] * a.scale;
-          if (toc > 0.f) v = cap_score(v, a.softcap, toc);
-          if (edge) {
-            const int d = rel[k >> 1] - (kr + i * 16 + j * 8 + (k & 1));     // query position - key position
-            if (d < 0 || d >= a.window) v = -INFINITY;
+          for (int k = 0; k < 4; ++k) s[i][j][k] = 0.f;
+#pragma unroll 4
+      for (int ks = ks0; ks < ks1; ++ks) {
+        uint32_t af[4];
+        ldsm4(af, q_frag + ks * 16);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          uint32_t bf[4];
+          ldsm4(bf, keys + (i * 16 + (lane >> 4) * 8 + (lane & 7)) * stride + ks * 16 + ((lane >> 3) & 1) * 8);
+          mma16816(s[i][0], af, bf[0], bf[1]);
+          mma16816(s[i][1], af, bf[2], bf[3]);
+        }
+      }
+      float mx[2] = {m[0], m[1]};
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            float v = s[i][j][k] * c_in;
+            if (capped) v = fmaf(c_two, rcp(1.f + ex2(v)), c_cap);          // cap * tanh(score / cap)
+            if (edge) {
+              const int d = rel[k >> 1] - (kr + kh + i * 16 + j * 8 + (k & 1));   // query position - key position
+              if (d < 0 || d >= a.window) v = -INFINITY;
+            }
+            s[i][j][k] = v;
+            mx[k >> 1] = fmaxf(mx[k >> 1], v);
           }
-          s[i][j][k] = v;
-          mx[k >> 1] = fmaxf(mx[k >> 1], v);
+      bool grew = false;
+      float f[2];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+        grew = grew || mx[r] > m[r];
+        f[r] = mx[r] == -INFINITY ? 1.f : ex2(m[r] - mx[r]);
+        m[r] = mx[r];
+      }
+      if (__any_sync(0xffffffffu, grew)) {                                  // most key blocks leave every maximum as it is
+        l[0] *= f[0];
+        l[1] *= f[1];
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          o[j][0] *= f[0]; o[j][1] *= f[0]; o[j][2] *= f[1]; o[j][3] *= f[1];
         }
-    float f[2];
+      }
+      const float ms[2] = {m[0] == -INFINITY ? 0.f : m[0], m[1] == -INFINITY ? 0.f : m[1]};
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-      f[r] = mx[r] == -INFINITY ? 1.f : __expf(m[r] - mx[r]);
-      m[r] = mx[r];
-      l[r] *= f[r];
+      for (int i = 0; i < 2; ++i) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float p = ex2(s[i][j][k] - ms[k >> 1]);
+            s[i][j][k] = p;
+            l[k >> 1] += p;
+          }
+        value16<NV>(o, s[i], keys + i * 16 * stride, stride, a.D, lane);
+      }
     }
-#pragma unroll
-    for (int j = 0; j < NV; ++j) {
-      o[j][0] *= f[0]; o[j][1] *= f[0]; o[j][2] *= f[1]; o[j][3] *= f[1];
-    }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const float p = m[k >> 1] == -INFINITY ? 0.f : __expf(s[i][j][k] - m[k >> 1]);
-          s[i][j][k] = p;
-          l[k >> 1] += p;
-        }
-      value16<NV>(o, s[i], cur + i * 16 * stride, stride, a.D, lane);
-    }
-    __syncthreads();
   }
   cp_async_wait<0>();
 #pragma unroll
@@ -644,8 +695,12 @@ STK_API int stk_window_kv_insert(const void* proj, long long ldp, int q_off, int
   const WinArgs a = win_args(STK_WIN_CALL);
   if (!win_ok(a)) return -1;
   cudaStream_t st = (cudaStream_t)stream;
-  if (fp32) launch_pdl(window_kv_insert_kernel<float>, dim3(T), dim3(128), 0, st, a);
-  else launch_pdl(window_kv_insert_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, st, a);
+  const int vec = !fp32 && dim % 8 == 0 && rd % 16 == 0 && row % 8 == 0 && ldp % 8 == 0 && k_off % 8 == 0 &&
+                  ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0;
+  const dim3 grid((T + 3) / 4);
+  const size_t smem = static_cast<size_t>(2) * rd * sizeof(float2);
+  if (fp32) launch_pdl(window_kv_insert_kernel<float>, grid, dim3(128), smem, st, a, T, vec);
+  else launch_pdl(window_kv_insert_kernel<__nv_bfloat16>, grid, dim3(128), smem, st, a, T, vec);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -715,16 +770,22 @@ STK_API int stk_window_attention_tiles(const void* proj, long long ldp, int q_of
   if (T <= 0) return 0;
   const WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
   if (!win_mma_ok(a) || window < 1 || n_req < 1) return -1;
-  const int hg = heads / kv_heads, gs = hg < kTileRows ? hg : kTileRows, sub = (hg + gs - 1) / gs, bq = kTileRows / gs;
+  // eight warps of rows up to 128-wide heads, four above (their output accumulators fill the register file)
+  const int rows = dim <= 128 ? 128 : 64;
+  const int hg = heads / kv_heads, gs = hg < rows ? hg : rows, sub = (hg + gs - 1) / gs, bq = rows / gs;
   if (kv_heads * sub > 65535) return -2;
-  const size_t smem = static_cast<size_t>(kTileRows + 2 * kPage) * win_stride(row) * 2;
+  const size_t smem = static_cast<size_t>(rows + 2 * kPage) * win_stride(row) * 2;
   const dim3 grid(T / bq + n_req, kv_heads * sub);                     // upper bound over the ways to cut T tokens into spans
   cudaStream_t st = (cudaStream_t)stream;
 #define STK_WIN_TILE(NV)                                                                                                  \
-  if (cudaFuncSetAttribute(window_attn_tiles_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=       \
-      cudaSuccess)                                                                                                         \
-    return -3;                                                                                                             \
-  launch_pdl(window_attn_tiles_kernel<NV>, grid, dim3(128), smem, st, a, query_start, req_rows, start_pos, n_req, min_span, gs);
+  {                                                                                                                       \
+    constexpr int kW = NV <= 16 ? 8 : 4;                                                                                   \
+    if (cudaFuncSetAttribute(window_attn_tiles_kernel<NV, kW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) !=  \
+        cudaSuccess)                                                                                                       \
+      return -3;                                                                                                           \
+    launch_pdl(window_attn_tiles_kernel<NV, kW>, grid, dim3(kW * 32), smem, st, a, query_start, req_rows, start_pos, n_req, \
+               min_span, gs);                                                                                              \
+  }
   STK_WIN_DIM(STK_WIN_TILE)
 #undef STK_WIN_TILE
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
