@@ -123,7 +123,7 @@ def kernel_times(step, steps: int) -> Dict[str, List[float]]:
 
 # ---- rooflines ------------------------------------------------------------------------------------------
 # group -> (pattern in the kernel name); work per step below uses the same group names
-HYBRID_GROUPS = [("projections", ("gemm", "skinny")), ("window_attention", ("window_attn_tiles", "window_attn_tokens")),
+HYBRID_GROUPS = [("projections", ("gemm", "skinny")), ("window_attention", ("window_attn_tc", "window_attn_tiles", "window_attn_tokens")),
                  ("window_attention combine", ("window_attn_combine",)), ("kv insert", ("window_kv_insert",)),
                  ("add + layer norm", ("add_layer_norm",)), ("feed-forward join", ("join_glu",)),
                  ("mlstm scan", ("mlstm_scan_kernel",)), ("mlstm chunk states", ("mlstm_chunk_state",)),

@@ -11,22 +11,9 @@
 //   window_attn_tiles      bf16, prompt portions: 128 rows (tokens x heads of the group) per CTA, key pages through two stages
 // Probabilities enter the value product as bf16 pairs (high part and remainder), so they keep 16 mantissa bits.
 #define STK_PDL_CLASS 8
-#include "common.cuh"
+#include "window_attention.cuh"
 
 namespace stk {
-
-constexpr int kPage = 64;
-
-struct WinArgs {
-  const void* proj; long long ldp; int q_off, k_off;
-  const int64_t* positions; const int* tok_req;
-  const int* table; int bt_stride;
-  void* cache; int row;
-  const float* freq; int rd; float mag;
-  int H, G, D;
-  int window; float scale, softcap; const float* sink;
-  void* out; long long ldo;
-};
 
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return bf16_to_f(v); }
@@ -475,23 +462,11 @@ window_attn_combine_kernel(const WinArgs a, const int* __restrict__ first_pos, c
 }
 
 // ---- prompt portions --------------------------------------------------------------------------------
-constexpr float kLog2e = 1.4426950408889634f;
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ float rcp(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
 // WARPS x 16 rows per CTA; scores and maxima in units of log2(e).
 template <int NV, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32, 2)
 window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, const int* __restrict__ req_rows,
-                         const int* __restrict__ start_pos, int n_req, int min_span, int gs) {
+                         const int* __restrict__ start_pos, int n_req, int min_span, int max_span, int gs) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   constexpr int kThreads = WARPS * 32, kRows = WARPS * 16;
   const int stride = win_stride(a.row);
@@ -505,7 +480,7 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
     int left = blockIdx.x, ri = -1;
     for (int i = 0; i < n_req; ++i) {
       const int n = query_start[i + 1] - query_start[i];
-      if (n < min_span) continue;
+      if (n < min_span || n > max_span) continue;
       const int tiles = (n + bq - 1) / bq;
       if (left < tiles) { ri = i; left = tiles - 1 - left; break; }        // the tiles with the most keys first
       left -= tiles;
@@ -662,29 +637,6 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
 
 using namespace stk;
 
-static WinArgs win_args(const void* proj, long long ldp, int q_off, int k_off, const int64_t* positions, const int* tok_req,
-                        const int* table, int bt_stride, void* cache, int row, const float* freq, int rd, float mag, int heads,
-                        int kv_heads, int dim, int window = 0, float scale = 0.f, float softcap = 0.f,
-                        const float* sink = nullptr, void* out = nullptr, long long ldo = 0) {
-  WinArgs a;
-  a.proj = proj; a.ldp = ldp; a.q_off = q_off; a.k_off = k_off;
-  a.positions = positions; a.tok_req = tok_req;
-  a.table = table; a.bt_stride = bt_stride;
-  a.cache = cache; a.row = row;
-  a.freq = freq; a.rd = rd; a.mag = mag;
-  a.H = heads; a.G = kv_heads; a.D = dim;
-  a.window = window; a.scale = scale; a.softcap = softcap; a.sink = sink;
-  a.out = out; a.ldo = ldo;
-  return a;
-}
-static bool win_ok(const WinArgs& a) {
-  return a.H > 0 && a.G > 0 && a.D > 0 && a.H % a.G == 0 && a.rd >= 0 && (a.rd & 1) == 0 && a.rd <= a.D && a.D <= 1024 &&
-         a.row >= a.D + a.rd;
-}
-// tensor-core kernels: whole 16-byte rows, head size within the accumulators
-static bool win_mma_ok(const WinArgs& a) {
-  return win_ok(a) && a.D <= 256 && a.row % 8 == 0 && (reinterpret_cast<uintptr_t>(a.cache) & 15) == 0;
-}
 #define STK_WIN_CALL proj, ldp, q_off, k_off, positions, tok_req, table, bt_stride, cache, row, freq, rd, mag, heads, kv_heads, dim
 
 STK_API int stk_window_kv_insert(const void* proj, long long ldp, int q_off, int k_off, const int64_t* positions,
@@ -765,7 +717,7 @@ STK_API int stk_window_attention_tiles(const void* proj, long long ldp, int q_of
                                        const int* tok_req, const int* table, int bt_stride, void* cache, int row, const float* freq, int rd, float mag,
                                        int heads, int kv_heads, int dim,
                                        int window, float scale, float softcap, const float* sink, void* out, long long ldo,
-                                       const int* query_start, const int* req_rows, const int* start_pos, int n_req, int min_span,
+                                       const int* query_start, const int* req_rows, const int* start_pos, int n_req, int min_span, int max_span,
                                        int T, void* stream) {
   if (T <= 0) return 0;
   const WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
@@ -784,7 +736,7 @@ STK_API int stk_window_attention_tiles(const void* proj, long long ldp, int q_of
         cudaSuccess)                                                                                                       \
       return -3;                                                                                                           \
     launch_pdl(window_attn_tiles_kernel<NV, kW>, grid, dim3(kW * 32), smem, st, a, query_start, req_rows, start_pos, n_req, \
-               min_span, gs);                                                                                              \
+               min_span, max_span, gs);                                                                                              \
   }
   STK_WIN_DIM(STK_WIN_TILE)
 #undef STK_WIN_TILE

@@ -98,7 +98,8 @@ FAMILIES: Dict[str, ModelFamily] = {
     "dsv4": ModelFamily("dsv4", _dsv4_shapes, _dsv4_weights, _dsv4_cache, _dsv4_model, prefix_cache=True),
     "hybrid": ModelFamily("hybrid", _hybrid_shapes, _hybrid_weights, _hybrid_cache, _hybrid_model, prefix_cache=False,
                           native_sources=("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", "linear_f32.cu",
-                                          "hybrid_block.cu", "window_attention.cu", "mlstm.cu", "sampler.cu")),
+                                          "hybrid_block.cu", "window_attention.cu", "window_attention_tc.cu",
+                                          "mlstm.cu", "sampler.cu")),
 }
 
 # architecture name in config.json -> configuration parser

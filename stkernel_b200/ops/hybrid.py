@@ -22,6 +22,8 @@ F32 = torch.float32
 
 # spans of at most this many tokens are attended token by token (the kernel of decode steps); longer ones in query tiles
 ATTN_TOKEN_SPAN = 4
+# spans of at least this many tokens take the tcgen05 kernel where its sizes allow
+ATTN_TC_SPAN = 64
 # spans of at least this many tokens run the recurrence in chunks on the tensor cores (bf16 models)
 MLSTM_CHUNK_SPAN = 24
 MLSTM_CHUNK = 64
@@ -138,9 +140,15 @@ def window_attention(proj: torch.Tensor, q_off: int, k_off: int, a: AttentionPar
         part = scratch("wattn.part", (splits * t * h * (d + 2),), F32, proj.device) if splits > 1 else None
         _lib.call("stk_window_attention_tokens", *common, *tail, meta.first_pos, meta.last_pos, token_span, splits, part, t,
                   _lib.stream())
-    if meta.max_span > token_span:
-        _lib.call("stk_window_attention_tiles", *common, *tail, meta.query_start, meta.req_rows, meta.start_pos, meta.n_req,
-                  token_span + 1, t, _lib.stream())
+    spans = (meta.query_start, meta.req_rows, meta.start_pos, meta.n_req)
+    tc = (meta.max_span >= ATTN_TC_SPAN and out.stride(0) % 8 == 0
+          and _lib.query("stk_window_attention_tc_ok", h, g, d, rd, cache.shape[3]) == 1)
+    if meta.max_span > token_span and not (tc and meta.min_span >= ATTN_TC_SPAN):
+        _lib.call("stk_window_attention_tiles", *common, *tail, *spans, token_span + 1, ATTN_TC_SPAN - 1 if tc else 1 << 30, t,
+                  _lib.stream())
+    if tc:
+        _lib.call("stk_window_attention_tc", *common, *tail, *spans, ATTN_TC_SPAN, cache.shape[0], t, _lib.status_buffer(),
+                  _lib.stream())
 
 
 # ----------------------------------------------------------------------------
