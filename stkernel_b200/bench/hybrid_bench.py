@@ -302,3 +302,55 @@ def render(res: Dict) -> str:
                                  f"{x['gbs']:7.1f} GB/s" + (f"  special functions {x['sfu_us']} us" if "sfu_us" in x else ""))
                     lines.append(f"    {x['us']:9.1f} us {x['launches']:6.1f}x  {x['group']:26s}{extra}")
     return "\n".join(lines)
+
+
+def main() -> None:
+    """One op of a layer on its own (profilers): `python -m stkernel_b200.bench.hybrid_bench --op attention|mlstm`."""
+    import argparse
+    from ..ops import hybrid as HB
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--op", choices=("attention", "mlstm"), required=True)
+    ap.add_argument("--width", type=int, default=4096)
+    ap.add_argument("--tokens", type=int, default=4096)
+    ap.add_argument("--context", type=int, default=8192)
+    ap.add_argument("--repeat", type=int, default=3)
+    a = ap.parse_args()
+    dev = torch.device("cuda:0")
+    cfg = hybrid_config(a.width, 2, 1024)
+    g = torch.Generator(device=dev).manual_seed(0)
+    n, ctx = a.tokens, a.context
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    meta = HB.HybridMeta(torch.zeros(n, dtype=torch.int64, device=dev), torch.zeros(n, dtype=torch.int32, device=dev),
+                         torch.arange(ctx, ctx + n, device=dev), i32([ctx] * n), i32([ctx + n - 1] * n), i32([0, n]), i32([0]),
+                         i32([ctx]), 1, n, False, n)
+    m = next(l.mixer for l in cfg.layers if l.mixer.kind == a.op)
+    pages = (ctx + n) // 64 + 1
+    e0, e1 = (torch.cuda.Event(enable_timing=True) for _ in range(2))
+    if a.op == "attention":
+        proj = torch.randn(n, (m.heads + m.kv_heads) * m.dim, generator=g, device=dev).to(torch.bfloat16)
+        cache = torch.randn(pages, m.kv_heads, 64, m.dim + m.rot_dims, generator=g, device=dev).to(torch.bfloat16)
+        table = torch.arange(pages, dtype=torch.int32, device=dev).view(1, -1)
+        freq, mag = m.rotary.frequencies()
+        p = HB.AttentionParams(m.heads, m.kv_heads, m.dim, m.window, m.scale, m.softcap, torch.tensor(freq, device=dev), mag,
+                               torch.zeros(m.heads, device=dev))
+        out = torch.empty(n, m.out_dim, dtype=torch.bfloat16, device=dev)
+        run_op = lambda: HB.window_attention(proj, 0, m.heads * m.dim, p, meta, table, cache, out)
+    else:
+        qk, vv = m.heads * m.dim, m.heads * m.vdim
+        proj = torch.randn(n, 2 * qk + 2 * vv, generator=g, device=dev).to(torch.bfloat16)
+        gates = torch.randn(n, 2 * m.heads, generator=g, device=dev)
+        p = HB.MlstmParams(m.heads, m.dim, m.vdim, m.gate_cap, torch.zeros(2 * m.heads, device=dev), torch.ones(vv, device=dev), 1e-6)
+        st = tuple(torch.zeros(1, m.heads, *s, device=dev) for s in ((m.dim, m.vdim), (m.dim,), ()))
+        out = torch.empty(n, vv, dtype=torch.bfloat16, device=dev)
+        run_op = lambda: HB.mlstm(proj, 0, qk, 2 * qk, 2 * qk + vv, gates, p, meta, st, out, None)
+    for _ in range(a.repeat):
+        e0.record()
+        run_op()
+        e1.record()
+        torch.cuda.synchronize()
+    _lib.check_status()
+    print(f"{a.op} width {a.width} tokens {n} context {ctx}: {e0.elapsed_time(e1) * 1e3:.1f} us")
+
+
+if __name__ == "__main__":
+    main()

@@ -210,3 +210,82 @@ def test_mlstm(where, c):
                 assert e < (2e-5 if dt == F32 else 5e-3), (plan, sizes, r, e)
                 at[r] += sizes[r]
         assert all(torch.isnan(s[1]).all() for s in S)          # a row nobody owns is not touched
+
+
+# ---- the kernels of one layer agree with one another at sizes the oracle is too slow for --------------------
+LONG = [dict(H=8, G=2, D=128, R=64, win=300), dict(H=4, G=4, D=128, R=128, win=1000), dict(H=6, G=2, D=96, R=12, win=129),
+        dict(H=16, G=1, D=64, R=16, win=64), dict(H=5, G=1, D=112, R=6, win=500), dict(H=40, G=2, D=16, R=16, win=257),
+        dict(H=130, G=1, D=32, R=32, win=90), dict(H=4, G=2, D=72, R=8, win=400), dict(H=2, G=1, D=200, R=40, win=333)]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("c", LONG, ids=lambda c: "x".join(str(v) for v in c.values()))
+@pytest.mark.parametrize("cap,sink", [(20.0, True), (0.0, False)])
+def test_attention_kernels_agree_over_many_pages(c, cap, sink):
+    """Three requests in one step (a long portion that begins inside a page, a short one, a few tokens): the tensor-core kernels
+    against the fp32 one, over more pages than any ring of stages holds."""
+    from stkernel_b200.ops import _lib
+    dev = torch.device("cuda:0")
+    H, G, D, R, win = c["H"], c["G"], c["D"], c["R"], c["win"]
+    g = torch.Generator(device=dev).manual_seed(1)
+    spans = [(777, 0, 0), (1, 500, 3), (333, 1300, 1), (40, 130, 2), (3, 0, 4), (64, 64, 5)]
+    n = sum(s[0] for s in spans)
+    meta = one_request(0, 0, 0, dev, splits=spans)
+    pages = -(-1700 // 64)
+    cache = torch.zeros(6 * pages, G, 64, (D + R + 7) // 8 * 8, dtype=BF16, device=dev)
+    cache[..., :D + R] = torch.randn(6 * pages, G, 64, D + R, generator=g, device=dev)
+    table = torch.randperm(6 * pages, generator=torch.Generator().manual_seed(2)).view(6, pages).to(torch.int32).to(dev)
+    ko = (H * D + 15) // 16 * 16
+    proj = torch.randn(n, ko + (G * D + 15) // 16 * 16, generator=g, device=dev).to(BF16)
+    proj[::5, :H * D] *= 4
+    sk = torch.randn(H, generator=g, device=dev) * 3 if sink else None
+    freq = torch.rand(R // 2, generator=g, device=dev)
+    a = HB.AttentionParams(H, G, D, win, D ** -0.5, cap, freq, 1.1, sk)
+    out = torch.full((n, HB.out_offset(H * D)), float("nan"), dtype=BF16, device=dev)
+    HB.window_attention(proj, 0, ko, a, meta, table, cache, out)
+    ref = torch.empty_like(out)
+    _lib.call("stk_window_attention_simt", proj, proj.stride(0), 0, ko, meta.positions, meta.tok_req, table, table.stride(0), cache,
+              cache.shape[3], freq, R, 1.1, H, G, D, win, D ** -0.5, cap, sk, ref, ref.stride(0), 0, n, _lib.stream())
+    x, y = out[:, :H * D].float(), ref[:, :H * D].float()
+    assert torch.isfinite(x).all()
+    err = ((x - y).view(n, H, D).norm(dim=-1) / y.view(n, H, D).norm(dim=-1).clamp(min=1e-3)).amax(1)
+    # the tensor-core kernels round the rotated query and the row copy of it to bf16, the fp32 one only the row
+    assert err.max() < 6e-2 and err.mean() < 1e-2, int(err.argmax())
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("c", [dict(H=2, D=64, V=128), dict(H=3, D=40, V=72), dict(H=1, D=256, V=320), dict(H=2, D=24, V=13)],
+                         ids=lambda c: "x".join(str(v) for v in c.values()))
+def test_mlstm_chunks_agree_with_the_scan_over_many_chunks(c):
+    """More chunks than one pass of the gate chain holds, from a carried state, beside a fresh request and a decode row."""
+    dev = torch.device("cuda:0")
+    H, D, V = c["H"], c["D"], c["V"]
+    g = torch.Generator(device=dev).manual_seed(3)
+    spans = [(2300, 5, 2), (1, 70, 0), (130, 0, 3)]
+    n = sum(s[0] for s in spans)
+    meta = one_request(0, 0, 0, dev, splits=spans)
+    al = lambda x: (x + 15) // 16 * 16
+    offs = [0, al(H * D), 2 * al(H * D), 2 * al(H * D) + al(H * V)]
+    proj = torch.randn(n, offs[3] + al(H * V), generator=g, device=dev).to(BF16)
+    proj[:, :H * D] = (proj[:, offs[1]:offs[1] + H * D].float() + 0.4 * proj[:, :H * D].float()).to(BF16)
+    gates = torch.randn(n, 2 * H, generator=g, device=dev) * 3
+    gates[:, H:] += 4
+    p = HB.MlstmParams(H, D, V, 10.0, torch.zeros(2 * H, device=dev), torch.ones(H * V, device=dev), 1e-6)
+    init = [torch.randn(4, H, D, V, generator=g, device=dev), torch.randn(4, H, D, generator=g, device=dev),
+            torch.randn(4, H, generator=g, device=dev)]
+    outs, states = [], []
+    keep = HB.MLSTM_CHUNK_SPAN
+    try:
+        for span in (keep, 1 << 20):
+            HB.MLSTM_CHUNK_SPAN = span
+            st = [x.clone() for x in init]
+            out = torch.zeros(n, HB.out_offset(H * V), dtype=BF16, device=dev)
+            HB.mlstm(proj, *offs, gates, p, meta, st, out, None)
+            outs.append(out.double().cpu())
+            states.append([x.double().cpu() for x in st])
+    finally:
+        HB.MLSTM_CHUNK_SPAN = keep
+    assert rel(outs[0], outs[1]) < 4e-3
+    for x, y in zip(*states):
+        assert rel(x, y) < 2e-4
+    assert torch.equal(states[0][0][1], init[0][1].double().cpu())
