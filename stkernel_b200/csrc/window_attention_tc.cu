@@ -11,8 +11,8 @@
 //                    TMEM only when a row's maximum grew by more than 2^8), probabilities to shared memory as bf16 pairs
 //                    (high part and remainder, two products), row output from TMEM
 //
-// TMEM: per tile 64 columns of S and up to 128 of O.  Every mbarrier wait is bounded; on expiry the status word is set and the
-// CTA leaves.  Layout of the query rows: see window_attention.cu.
+// TMEM: per tile two buffers of 64 score columns (the next page's scores are ready when a softmax warp comes back for them)
+// and up to 128 columns of O.  Every mbarrier wait is bounded; on expiry the status word is set and the CTA leaves.  Layout of the query rows: see window_attention.cu.
 #define STK_PDL_CLASS 8
 #include "window_attention.cuh"
 
@@ -25,7 +25,7 @@ constexpr int kTcKvPanel = kPage * 128, kTcQPanel = kTcTileRows * 128, kTcPTile 
 
 struct alignas(8) WinTcBars {
   uint64_t loaded[kTcMaxStages], full[kTcMaxStages], empty[kTcMaxStages];
-  uint64_t s_full[2], p_full[2], pv_done[2];
+  uint64_t s_full[2][2], p_full[2], pv_done[2];             // [tile][score buffer], [tile]
   uint32_t tmem_base;
   int find[2];
 };
@@ -57,6 +57,7 @@ __device__ __forceinline__ uint64_t win_desc_mn(uint32_t smem_addr, uint32_t lbo
   return d;
 }
 
+template <bool kCap>
 __global__ void __launch_bounds__(kTcThreads, 1)
 window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs x) {
   extern __shared__ uint8_t smem_raw[];
@@ -87,7 +88,8 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
       mbar_init(&bars->empty[s], 1);
     }
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&bars->s_full[i], 1);
+      mbar_init(&bars->s_full[i][0], 1);
+      mbar_init(&bars->s_full[i][1], 1);
       mbar_init(&bars->p_full[i], 4);
       mbar_init(&bars->pv_done[i], 1);
     }
@@ -163,42 +165,39 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = bars->tmem_base;                           // S0 0, S1 64, O0 128, O1 256
+  const uint32_t tmem = bars->tmem_base;                           // scores of tile i, buffer b: i * 64 + b * 128; outputs: 256 + i * 128
 
   if (warp == 8) {
     // ------------------------------- loader -------------------------------
+    // A page is complete before the next one is asked for, so that a page never waits behind the release of a stage that only
+    // a later product gives back; the ring still runs stages ahead of the products.
     bool ok = true;
     const int n = page1 - page0;
-    for (int i = 0; i <= n && ok; ++i) {
-      if (i < n) {
-        const int st = i % x.stages;
-        if (i >= x.stages) ok = mbar_wait(&bars->empty[st], ((i / x.stages) - 1) & 1, x.status, 700);
-        if (!ok) break;
-        if (lane == 0) {
-          const int page = max(bt[page0 + i], 0);
-          mbar_expect_tx(&bars->loaded[st], x.panels * kTcKvPanel);
-          for (int p = 0; p < x.panels; ++p)
-            tma_load_2d(kv_s + (st * x.panels + p) * kTcKvPanel, &tm_kv, &bars->loaded[st], p * 64, (page * a.G + g) * kPage);
-        }
-        __syncwarp();
+    for (int i = 0; i < n && ok; ++i) {
+      const int st = i % x.stages;
+      if (i >= x.stages) ok = mbar_wait(&bars->empty[st], ((i / x.stages) - 1) & 1, x.status, 700);
+      if (!ok) break;
+      if (lane == 0) {
+        const int page = max(bt[page0 + i], 0);
+        mbar_expect_tx(&bars->loaded[st], x.panels * kTcKvPanel);
+        for (int p = 0; p < x.panels; ++p)
+          tma_load_2d(kv_s + (st * x.panels + p) * kTcKvPanel, &tm_kv, &bars->loaded[st], p * 64, (page * a.G + g) * kPage);
       }
-      if (i > 0) {
-        const int j = i - 1, st = j % x.stages;
-        ok = mbar_wait(&bars->loaded[st], (j / x.stages) & 1, x.status, 701);
-        if (!ok) break;
-        const long long base = static_cast<long long>(page0 + j) * kPage;
-        if (base < key_lo || base + kPage - 1 > key_hi) {
-          for (int e = lane; e < kPage * x.panels * 8; e += 32) {
-            const int r = e / (x.panels * 8), c = e - r * (x.panels * 8);
-            if (base + r < key_lo || base + r > key_hi)
-              *reinterpret_cast<uint4*>(kv_s + (st * x.panels + (c >> 3)) * kTcKvPanel + r * 128 + ((c & 7) << 4)) =
-                  make_uint4(0, 0, 0, 0);
-          }
-          fence_proxy_async();
+      __syncwarp();
+      ok = mbar_wait(&bars->loaded[st], (i / x.stages) & 1, x.status, 701);
+      if (!ok) break;
+      const long long base = static_cast<long long>(page0 + i) * kPage;
+      if (base < key_lo || base + kPage - 1 > key_hi) {
+        for (int e = lane; e < kPage * x.panels * 8; e += 32) {
+          const int r = e / (x.panels * 8), c = e - r * (x.panels * 8);
+          if (base + r < key_lo || base + r > key_hi)
+            *reinterpret_cast<uint4*>(kv_s + (st * x.panels + (c >> 3)) * kTcKvPanel + r * 128 + ((c & 7) << 4)) =
+                make_uint4(0, 0, 0, 0);
         }
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&bars->full[st]);
+        fence_proxy_async();
       }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->full[st]);
     }
     if (!ok && lane == 0) {
       // leave no copy in flight: the ring's outstanding loads land before the CTA's shared memory goes away
@@ -215,11 +214,13 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
       const int ks0 = a.rd / 16, ks1 = (a.D + a.rd + 15) / 16;
       int done[2] = {0, 0};
       bool ok = true;
-      for (int lp = page0 - 1; lp < page1 && ok; ++lp) {
-        const int n = lp - page0, st = n % x.stages, sn = (n + 1) % x.stages;
+      // pages that the scores run ahead of the outputs; page lp + lead must fit the ring beside page lp
+      const int lead = x.stages > 2 ? 2 : 1;
+      for (int lp = page0 - lead; lp < page1 && ok; ++lp) {
+        const int n = lp - page0, st = n % x.stages, sn = (n + lead) % x.stages;
         bool waited = false;
         for (int i = 0; i < 2 && ok; ++i) {
-          const bool now = lp >= pa[i] && lp < pb[i], next = lp + 1 >= pa[i] && lp + 1 < pb[i];
+          const bool now = lp >= pa[i] && lp < pb[i], next = lp + lead >= pa[i] && lp + lead < pb[i];
           if (now) {
             ok = mbar_wait(&bars->p_full[i], done[i] & 1, x.status, 710 + i);
             if (!ok) break;
@@ -227,18 +228,19 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
           }
           if (next) {
             if (!waited) {
-              ok = mbar_wait(&bars->full[sn], ((n + 1) / x.stages) & 1, x.status, 712);
+              ok = mbar_wait(&bars->full[sn], ((n + lead) / x.stages) & 1, x.status, 712);
               if (!ok) break;
               tc_fence_after();
               waited = true;
             }
             const uint8_t* kv = kv_s + sn * x.panels * kTcKvPanel;
+            const int buf = (lp + lead - pa[i]) & 1;
             for (int ks = ks0; ks < ks1; ++ks) {
               const uint64_t ad = umma_desc_sw128(smem_u32(q_s + (i * x.q_panels + (ks >> 2) - x.q_panel0) * kTcQPanel)) + 2 * (ks & 3);
               const uint64_t bd = umma_desc_sw128(smem_u32(kv + (ks >> 2) * kTcKvPanel)) + 2 * (ks & 3);
-              umma_f16(tmem + i * 64, ad, bd, idesc_qk, ks > ks0 ? 1u : 0u);
+              umma_f16(tmem + i * 64 + buf * 128, ad, bd, idesc_qk, ks > ks0 ? 1u : 0u);
             }
-            umma_commit(&bars->s_full[i]);
+            umma_commit(&bars->s_full[i][buf]);
           }
           if (now) {
             const uint8_t* kv = kv_s + st * x.panels * kTcKvPanel;
@@ -248,7 +250,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
               for (int kk = 0; kk < 4; ++kk) {
                 const uint64_t ad = umma_desc_sw128(smem_u32(p_s + (2 * i + part) * kTcPTile)) + 2 * kk;
                 const uint64_t bd = win_desc_mn(smem_u32(kv + kk * 2048), kTcKvPanel);
-                umma_f16(tmem + 128 + i * 128, ad, bd, idesc_pv, (done[i] > 0 || part > 0 || kk > 0) ? 1u : 0u);
+                umma_f16(tmem + 256 + i * 128, ad, bd, idesc_pv, (done[i] > 0 || part > 0 || kk > 0) ? 1u : 0u);
               }
             umma_commit(&bars->pv_done[i]);
             ++done[i];
@@ -262,11 +264,10 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
     // ------------------------------- softmax -------------------------------
     const int tile = warp >> 2, r = (warp & 3) * 32 + lane;
     const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
-    const uint32_t ts = tmem + tile * 64 + lanes, to = tmem + 128 + tile * 128 + lanes;
+    const uint32_t ts = tmem + tile * 64 + lanes, to = tmem + 256 + tile * 128 + lanes;
     const int q = r / x.gs, h = h0 + (r - q * x.gs);
     const bool row_ok = q < n_tok[tile] && q < bq && h < h_end;
-    const bool capped = a.softcap > 0.f;
-    const float c_in = capped ? a.scale * 2.f * kLog2e / a.softcap : a.scale * kLog2e;
+    const float c_in = kCap ? a.scale * 2.f * kLog2e / a.softcap : a.scale * kLog2e;
     const float c_cap = a.softcap * kLog2e, c_two = -2.f * c_cap;
     float m = row_ok && a.sink != nullptr ? a.sink[h] * kLog2e : -INFINITY, l = row_ok && a.sink != nullptr ? 1.f : 0.f;
     const long long last = first[tile] + n_tok[tile] - 1;
@@ -275,14 +276,14 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
     bool ok = true;
     int k = 0;
     for (int lp = pa[tile]; lp < pb[tile] && ok; ++lp, ++k) {
-      ok = mbar_wait(&bars->s_full[tile], k & 1, x.status, 720);
+      ok = mbar_wait(&bars->s_full[tile][k & 1], (k >> 1) & 1, x.status, 720);
       if (!ok) break;
       tc_fence_after();
       float v[64];
       {
         uint32_t s0[32], s1[32];
-        tmem_ld_32x32(ts, s0);
-        tmem_ld_32x32(ts + 32, s1);
+        tmem_ld_32x32(ts + (k & 1) * 128, s0);
+        tmem_ld_32x32(ts + (k & 1) * 128 + 32, s1);
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
@@ -293,15 +294,21 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
       const long long base = static_cast<long long>(lp) * kPage;
       const bool edge = base + kPage - 1 > first[tile] || base < last - a.window + 1;
       const int d0 = static_cast<int>(first[tile] + q - base);              // query position - key position of column 0
-      float mx = -INFINITY;
+      // cap * tanh(score / cap), in units of log2(e)
 #pragma unroll
       for (int j = 0; j < 64; ++j) {
-        float s = v[j] * c_in;
-        if (capped) s = fmaf(c_two, rcp(1.f + ex2(s)), c_cap);              // cap * tanh(score / cap)
-        if (edge && (d0 - j < 0 || d0 - j >= a.window)) s = -INFINITY;
-        v[j] = s;
-        mx = fmaxf(mx, s);
+        const float u = v[j] * c_in;
+        v[j] = kCap ? fmaf(c_two, rcp(1.f + ex2(u)), c_cap) : u;
       }
+      if (edge) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j)
+          if (d0 - j < 0 || d0 - j >= a.window) v[j] = -INFINITY;
+      }
+      float mx4[4] = {v[0], v[1], v[2], v[3]};
+#pragma unroll
+      for (int j = 4; j < 64; ++j) mx4[j & 3] = fmaxf(mx4[j & 3], v[j]);
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       const bool grow = mx > m + 8.f || (m == -INFINITY && mx > -INFINITY);
       const bool any = __any_sync(0xffffffffu, grow);
       if (k > 0) {
@@ -327,13 +334,14 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
         }
       }
       const float ms = m == -INFINITY ? 0.f : m;
+      float ls[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int c = 0; c < 8; ++c) {
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const float p0 = ex2(v[c * 8 + 2 * j] - ms), p1 = ex2(v[c * 8 + 2 * j + 1] - ms);
-          l += p0 + p1;
+          ls[j] += p0 + p1;
           const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
           const float2 hf = __bfloat1622float2(hb);
           const __nv_bfloat162 lb = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
@@ -344,6 +352,7 @@ window_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const WinTcArgs
         *reinterpret_cast<uint4*>(p_hi + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
         *reinterpret_cast<uint4*>(p_lo + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
+      l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
       fence_proxy_async();
       tc_fence_before();
       __syncwarp();
@@ -419,9 +428,11 @@ STK_API int stk_window_attention_tc(const void* proj, long long ldp, int q_off, 
   if (smem < 118 * 1024) smem = 118 * 1024;                          // one CTA per SM: it owns all of tensor memory
   CUtensorMap tm;
   if (make_tmap_2d(&tm, cache, 2, num_pages * kv_heads * kPage, row, row, kPage) != 0) return -3;
-  if (cudaFuncSetAttribute(window_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
+  if (cudaFuncSetAttribute(window_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
+      cudaFuncSetAttribute(window_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
     return -3;
   const dim3 grid(T / (2 * bq) + n_req, kv_heads * sub);
-  launch_pdl(window_attn_tc_kernel, grid, dim3(kTcThreads), smem, (cudaStream_t)stream, tm, x);
+  if (softcap > 0.f) launch_pdl(window_attn_tc_kernel<true>, grid, dim3(kTcThreads), smem, (cudaStream_t)stream, tm, x);
+  else launch_pdl(window_attn_tc_kernel<false>, grid, dim3(kTcThreads), smem, (cudaStream_t)stream, tm, x);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

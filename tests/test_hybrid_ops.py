@@ -213,7 +213,8 @@ def test_mlstm(where, c):
 
 
 # ---- the kernels of one layer agree with one another at sizes the oracle is too slow for --------------------
-LONG = [dict(H=8, G=2, D=128, R=64, win=300), dict(H=4, G=4, D=128, R=128, win=1000), dict(H=6, G=2, D=96, R=12, win=129),
+LONG = [dict(H=8, G=2, D=128, R=64, win=300), dict(H=4, G=4, D=128, R=128, win=1000), dict(H=4, G=2, D=128, R=12, win=700),
+        dict(H=3, G=1, D=128, R=120, win=200), dict(H=6, G=2, D=96, R=12, win=129),
         dict(H=16, G=1, D=64, R=16, win=64), dict(H=5, G=1, D=112, R=6, win=500), dict(H=40, G=2, D=16, R=16, win=257),
         dict(H=130, G=1, D=32, R=32, win=90), dict(H=4, G=2, D=72, R=8, win=400), dict(H=2, G=1, D=200, R=40, win=333)]
 
