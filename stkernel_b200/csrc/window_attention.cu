@@ -440,24 +440,29 @@ window_attn_combine_kernel(const WinArgs a, const int* __restrict__ first_pos, c
                            const float* __restrict__ part, int splits, int T) {
   pdl_wait();
   pdl_trigger();
+  __shared__ float s_m[64], s_w[64], s_l[64];                               // at most 64 ranges
   const int h = blockIdx.x, t = blockIdx.y;
   if (a.tok_req[t] < 0 || a.positions[t] < 0 || last_pos[t] - first_pos[t] + 1 > max_span) return;
   const long long step = static_cast<long long>(T) * a.H * (a.D + 2);
   const float* p = part + (static_cast<long long>(t) * a.H + h) * (a.D + 2);
-  float m = a.sink != nullptr ? a.sink[h] : -INFINITY;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, p[s * step + a.D]);
-  float l = a.sink != nullptr ? __expf(a.sink[h] - m) : 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float ms = p[s * step + a.D];
-    if (ms != -INFINITY) l = fmaf(__expf(ms - m), p[s * step + a.D + 1], l);
+  const int s = threadIdx.x;
+  if (s < splits) {
+    s_m[s] = p[s * step + a.D];
+    s_l[s] = p[s * step + a.D + 1];
   }
-  for (int c = threadIdx.x; c < a.D; c += blockDim.x) {
+  __syncthreads();
+  float m = a.sink != nullptr ? a.sink[h] : -INFINITY;
+  for (int i = 0; i < splits; ++i) m = fmaxf(m, s_m[i]);
+  if (s < splits) s_w[s] = s_m[s] == -INFINITY ? 0.f : __expf(s_m[s] - m);
+  __syncthreads();
+  float l = a.sink != nullptr ? __expf(a.sink[h] - m) : 0.f;
+  for (int i = 0; i < splits; ++i) l = fmaf(s_w[i], s_l[i], l);
+  const float inv = 1.f / l;
+  for (int c = s; c < a.D; c += blockDim.x) {
     float v = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float ms = p[s * step + a.D];
-      if (ms != -INFINITY) v = fmaf(__expf(ms - m), p[s * step + c], v);
-    }
-    reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h * a.D + c] = __float2bfloat16(v / l);
+#pragma unroll 8
+    for (int i = 0; i < splits; ++i) v = fmaf(s_w[i], p[i * step + c], v);
+    reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h * a.D + c] = __float2bfloat16(v * inv);
   }
 }
 
@@ -695,7 +700,7 @@ STK_API int stk_window_attention_tokens(const void* proj, long long ldp, int q_o
                                         void* stream) {
   if (T <= 0) return 0;
   const WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
-  if (!win_mma_ok(a) || window < 1 || splits < 1 || (splits > 1 && part == nullptr) || T > 65535) return -1;
+  if (!win_mma_ok(a) || window < 1 || splits < 1 || splits > 64 || (splits > 1 && part == nullptr) || T > 65535) return -1;
   const int sub = (heads / kv_heads + 15) / 16;
   if (kv_heads * sub > 65535) return -2;
   const size_t smem = static_cast<size_t>(16 + 2 * kPage) * win_stride(row) * 2;

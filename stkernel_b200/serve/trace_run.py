@@ -2,14 +2,14 @@
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N
 
-Standard input, one JSON object a line:
+Steps arrive as lines of JSON on standard input:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "chat-1", "tokens": [812, 44], "want": [1]}], "end": ["chat-0"]}
 
-`entries` are the requests of the step with their next tokens and the places among them whose logits are wanted; `end` are the
-requests that are finished after it (their cache pages and state rows are given back).  The wanted logits go to
-OUT/<step>.f32 as little-endian fp32 [wanted, vocab], in the order of the entries and places, and `done <step>` is printed
-when the step is complete.
+An entry feeds a request its next tokens and names the places among them whose logits are to be written; `end` lists requests
+that are over once the step has run, so their pages and rows become free.  OUT/<step>.f32 receives the logits (little-endian
+fp32, one vocabulary-long row per place, in the order of the entries and their places); `done <step>` on standard output says
+that the step is complete.
 
 The model, its step function, caches and kernels are the engine's own (`Engine.feed`); nothing is sampled.  In bfloat16 they
 are what serving uses, in float32 every operand is fp32.  Exit code 3: the architecture has no float32 form.
@@ -120,7 +120,7 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     ap.add_argument("--model", required=True, help="folder with config.json and safetensors")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16")
     ap.add_argument("--out", required=True, help="folder for <step>.f32")
-    ap.add_argument("--max-tokens", type=int, default=8192, help="most tokens that live requests hold at any time")
+    ap.add_argument("--max-tokens", type=int, default=8192, help="bound on the tokens of all open requests together (sizes the cache)")
     a = ap.parse_args(argv)
     engine = build_engine(a.model, a.dtype, a.max_tokens)
     run(engine, sys.stdin, a.out, lambda n: print(f"done {n}", flush=True))
