@@ -225,6 +225,9 @@ def tiny_config(**over: Any) -> ModelConfig:
 # ----------------------------------------------------------------------------
 # decoders described layer by layer
 # ----------------------------------------------------------------------------
+FULL_CONTEXT = 1 << 40       # window of an attention layer that sees every earlier position
+
+
 @dataclass(frozen=True)
 class YarnScaling:
     """YaRN context extension of a rotary embedding: frequencies below the `slow` bound are divided by `factor`, those
@@ -237,10 +240,12 @@ class YarnScaling:
 
 @dataclass(frozen=True)
 class RotaryConfig:
-    """Rotation of the first `dims` dimensions of a head, dimension i paired with i + dims/2."""
+    """Rotation of the first `dims` dimensions of a head: dimension i paired with i + dims/2, or with its neighbour
+    (2i with 2i + 1) when `interleaved`."""
     base: float
     dims: int
     scaling: Optional[YarnScaling] = None
+    interleaved: bool = False
 
     def frequencies(self) -> Tuple[List[float], float]:
         """-> (radians per position of every pair, factor on cos and sin)."""
@@ -288,6 +293,28 @@ class AttentionMixer:
 
 
 @dataclass(frozen=True)
+class LatentAttentionMixer:
+    """Causal attention over low-rank latents: queries come out of a normed latent of size q_rank, keys and values are read out
+    of a normed latent of size kv_rank per token (per head `dim` unrotated key dimensions and `vdim` value dimensions) plus one
+    rotated key part of rot_dim dimensions that all heads share.  A head's output is multiplied by the sigmoid of a gate."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rotary: Optional[RotaryConfig] = None
+    kv_from: Optional[int] = None         # layer whose cached latents and rotated key parts this one attends over
+    kind = "latent_attention"
+    window = FULL_CONTEXT
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
 class MlstmMixer:
     """Matrix-memory recurrence with exponential input gate and running-maximum stabiliser (mLSTM)."""
     heads: int
@@ -303,21 +330,40 @@ class MlstmMixer:
 
 @dataclass(frozen=True)
 class DenseMlp:
-    """W_down(silu(W_gate h) * W_up h)."""
+    """W_down(act(W_gate h) * W_up h)."""
     ff: int
+    act: str = "silu"                     # "silu" | "relu"
+    kind = "dense"
+
+
+@dataclass(frozen=True)
+class MoeMlp:
+    """`top` of `experts` feed-forward layers W_down relu(W_up h)^2 per token, chosen by the largest router logits (bias
+    included) and weighted by the softmax over the chosen logits."""
+    experts: int
+    top: int
+    ff: int
+    kind = "moe"
+
+
+Mixer = Union[AttentionMixer, MlstmMixer, LatentAttentionMixer]
+Mlp = Union[DenseMlp, MoeMlp]
 
 
 @dataclass(frozen=True)
 class HybridLayer:
-    mixer: Union[AttentionMixer, MlstmMixer]
-    mlp: Optional[DenseMlp] = None
+    mixer: Mixer
+    mlp: Optional[Mlp] = None
     weights_of: Optional[int] = None      # layer whose tensors this one runs with (cache and state are its own)
 
 
 @dataclass(frozen=True)
 class HybridConfig:
     """A decoder given as a list of layers, each with its own mixer (attention or recurrence) and optional feed-forward.
-    Both sublayers read one layer norm's output and are added to an fp32 residual together (parallel block)."""
+
+    block "parallel":  both sublayers read one layer norm's output and are added to the fp32 residual together;
+    block "post_norm": the sublayers follow one another, read the residual itself, and their outputs are RMS-normed before
+                       they are added to it."""
     vocab_size: int
     hidden_size: int
     layers: Tuple[HybridLayer, ...]
@@ -326,6 +372,7 @@ class HybridConfig:
     dtype: str = "bfloat16"               # "bfloat16": projections and activations; "float32": everything
     max_position_embeddings: int = 1 << 30
     architecture: str = "Timalorn"
+    block: str = "parallel"               # "parallel" | "post_norm"
     family = "hybrid"
     # fields of the other family that family-neutral code asks for
     n_mtp_layers = 0
@@ -346,8 +393,17 @@ class HybridConfig:
         return i
 
     def windows(self) -> List[int]:
-        """Distinct attention windows, one page group each."""
-        return sorted({l.mixer.window for l in self.layers if l.mixer.kind == "attention"})
+        """Distinct attention windows, one page group each (FULL_CONTEXT: pages stay until the request ends)."""
+        return sorted({l.mixer.window for l in self.layers if l.mixer.kind != "mlstm"})
+
+    def cache_layer(self, i: int) -> int:
+        """The layer whose cache layer i reads (itself unless `kv_from` says otherwise)."""
+        j = getattr(self.layers[i].mixer, "kv_from", None)
+        return i if j is None else j
+
+    def mechanisms(self) -> Tuple[str, ...]:
+        """Kinds of mixers and feed-forwards in this model, which decide what kernels it needs."""
+        return tuple(sorted({l.mixer.kind for l in self.layers} | {l.mlp.kind for l in self.layers if l.mlp is not None}))
 
     def validate(self) -> None:
         def positive(name: str, v: Any, integer: bool = True) -> None:
@@ -364,37 +420,71 @@ class HybridConfig:
             raise ConfigError(f"unknown dtype {self.dtype!r}")
         if not self.layers:
             raise ConfigError("layers must not be empty")
+        if self.block not in ("parallel", "post_norm"):
+            raise ConfigError(f"unknown block {self.block!r}")
+
+        def rotary(at: str, r: RotaryConfig, dim: int, of: str) -> None:
+            positive(f"{at}.rot.base", r.base, False)
+            positive(f"{at}.rot.dims", r.dims)
+            if r.dims % 2 or r.dims > dim:
+                raise ConfigError(f"{at}.rot.dims must be even and at most {of}")
+            if r.scaling is not None:
+                for f in ("factor", "original", "fast", "slow"):
+                    positive(f"{at}.rot.scaling.{f}", getattr(r.scaling, f), False)
+
         for i, l in enumerate(self.layers):
             at, m = f"layers[{i}]", l.mixer
+            if self.block == "parallel" and (m.kind == "latent_attention" or (l.mlp is not None and l.mlp.kind != "dense")):
+                raise ConfigError(f"{at}: {m.kind} with this feed-forward is not available in parallel blocks")
             for f in ("heads", "dim"):
                 positive(f"{at}.mixer.{f}", getattr(m, f))
+            if m.dim > 1024:
+                raise ConfigError(f"{at}.mixer.dim: at most 1024")
+            if m.kind in ("attention", "latent_attention") and (not isinstance(m.scale, (int, float)) or isinstance(m.scale, bool)
+                                                                or not math.isfinite(m.scale)):
+                raise ConfigError(f"{at}.mixer.scale must be a finite number")
             if m.kind == "attention":
                 positive(f"{at}.mixer.kv_heads", m.kv_heads)
                 positive(f"{at}.mixer.mask.size", m.window)
-                if not isinstance(m.scale, (int, float)) or not math.isfinite(m.scale):
-                    raise ConfigError(f"{at}.mixer.scale must be a finite number")
                 if m.heads % m.kv_heads:
                     raise ConfigError(f"{at}.mixer: kv_heads must divide heads")
                 if m.softcap < 0 or not math.isfinite(m.softcap):
                     raise ConfigError(f"{at}.mixer.softcap must not be negative")
-                if m.dim > 1024:
-                    raise ConfigError(f"{at}.mixer.dim: at most 1024")
                 if m.rotary is not None:
-                    r = m.rotary
-                    positive(f"{at}.mixer.rot.base", r.base, False)
-                    positive(f"{at}.mixer.rot.dims", r.dims)
-                    if r.dims % 2 or r.dims > m.dim:
-                        raise ConfigError(f"{at}.mixer.rot.dims must be even and at most dim")
-                    if r.scaling is not None:
-                        for f in ("factor", "original", "fast", "slow"):
-                            positive(f"{at}.mixer.rot.scaling.{f}", getattr(r.scaling, f), False)
+                    rotary(f"{at}.mixer", m.rotary, m.dim, "dim")
+            elif m.kind == "latent_attention":
+                for f in ("vdim", "q_rank", "kv_rank"):
+                    positive(f"{at}.mixer.{f}", getattr(m, f))
+                if m.rot_dim != 0:
+                    positive(f"{at}.mixer.rot_dim", m.rot_dim)
+                if m.kv_rank + m.rot_dim > 2048 or m.vdim > 1024:
+                    raise ConfigError(f"{at}.mixer: kv_rank + rot_dim must be at most 2048, vdim at most 1024")
+                if m.rotary is not None:
+                    rotary(f"{at}.mixer", m.rotary, m.rot_dim, "rot_dim")
+                if (m.rotary.dims if m.rotary is not None else 0) != m.rot_dim:
+                    raise ConfigError(f"{at}.mixer.rot.dims must equal rot_dim")
+                j = m.kv_from
+                if j is not None:
+                    if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < i:
+                        raise ConfigError(f"{at}.mixer.kv_from: {j!r} is not an earlier layer")
+                    src = self.layers[j].mixer
+                    if (src.kind != "latent_attention" or src.kv_from is not None
+                            or (src.kv_rank, src.rot_dim, src.rotary) != (m.kv_rank, m.rot_dim, m.rotary)):
+                        raise ConfigError(f"{at}.mixer.kv_from: layer {j} must cache latents of its own of the same kv_rank, "
+                                          "rot_dim and rotation")
             else:
                 positive(f"{at}.mixer.vdim", m.vdim)
                 positive(f"{at}.mixer.gate_cap", m.gate_cap, False)
-                if m.dim > 1024:
-                    raise ConfigError(f"{at}.mixer.dim: at most 1024")
             if l.mlp is not None:
                 positive(f"{at}.mlp.ff", l.mlp.ff)
+                if l.mlp.kind == "dense":
+                    if l.mlp.act not in ("silu", "relu"):
+                        raise ConfigError(f"{at}.mlp.act: unknown activation {l.mlp.act!r}")
+                else:
+                    positive(f"{at}.mlp.router.experts", l.mlp.experts)
+                    positive(f"{at}.mlp.router.top", l.mlp.top)
+                    if l.mlp.top > l.mlp.experts or l.mlp.top > 32 or l.mlp.experts > 512:
+                        raise ConfigError(f"{at}.mlp.router: top must be at most experts and 32, experts at most 512")
             if l.weights_of is not None:
                 j = l.weights_of
                 if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < len(self.layers):
@@ -410,29 +500,37 @@ class HybridConfig:
         if e.spec.method != "none":
             raise ConfigError(f"{self.architecture} has no draft layers for speculative decoding")
         if p.eplb_record or p.eplb_redundant:
-            raise ConfigError(f"{self.architecture} has no experts to balance")
+            raise ConfigError(f"{self.architecture} has no expert placement to balance")
 
 
 def _take(d: Any, at: str, required: Sequence[str], optional: Sequence[str] = ()) -> Dict[str, Any]:
-    """The keys of a JSON object, none missing and none unknown."""
+    """The keys of a JSON object, none missing and none unknown (an unknown key that is null or false asks for nothing)."""
     if not isinstance(d, Mapping):
         raise ConfigError(f"{at}: {d!r} is not an object")
     for k in required:
         if k not in d:
             raise ConfigError(f"{at}: {k} is missing")
-    unknown = set(d) - set(required) - set(optional)
+    unknown = {k for k in unknown_keys(d, required, optional) if d[k] is not None and d[k] is not False}
     if unknown:
         raise ConfigError(f"{at}: unknown keys {sorted(unknown)}")
-    return dict(d)
+    return {k: v for k, v in d.items() if k not in unknown_keys(d, required, optional)}
 
 
-def timalorn_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> HybridConfig:
-    """The `config.json` of a Timalorn model: parallel blocks of windowed attention and mLSTM layers."""
+def unknown_keys(d: Mapping[str, Any], required: Sequence[str], optional: Sequence[str]) -> set:
+    return set(d) - set(required) - set(optional)
+
+
+def _check_model_keys(d: Mapping[str, Any]) -> None:
     for k in ("vocab", "width", "layers", "norm", "embedding"):
         if k not in d:
             raise ConfigError(f"config.json: {k} is missing")
     if not isinstance(d["layers"], Sequence) or isinstance(d["layers"], str):
         raise ConfigError("config.json: layers is not a list")
+
+
+def timalorn_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> HybridConfig:
+    """The `config.json` of a Timalorn model: parallel blocks of windowed attention and mLSTM layers."""
+    _check_model_keys(d)
     layers: List[HybridLayer] = []
     for i, l in enumerate(d["layers"]):
         at = f"layers[{i}]"
@@ -449,7 +547,7 @@ def timalorn_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> 
                 if sc is not None:
                     sc = YarnScaling(**_take(sc, f"{at}.mixer.rot.scaling", ("factor", "original", "fast", "slow")))
                 rot = RotaryConfig(r["base"], r["dims"], sc)
-            mixer: Union[AttentionMixer, MlstmMixer] = AttentionMixer(
+            mixer: Mixer = AttentionMixer(
                 m["heads"], m["kv_heads"], m["dim"], _take(m["mask"], f"{at}.mixer.mask", ("size",))["size"], m["scale"], rot,
                 m.get("softcap") or 0.0)
         elif l["type"] == "mlstm":
@@ -492,22 +590,77 @@ def timalorn_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
             "norm": {"eps": cfg.norm_eps}, "embedding": {"scale": cfg.embedding_scale}}
 
 
+def domilix_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> HybridConfig:
+    """The `config.json` of a Domilix model: latent attention (cached latents may be shared between layers), dense or
+    mixture-of-experts feed-forwards, RMS norms on the sublayers' outputs."""
+    _check_model_keys(d)
+    layers: List[HybridLayer] = []
+    for i, l in enumerate(d["layers"]):
+        at = f"layers[{i}]"
+        l = _take(l, at, ("type", "mixer"), ("mlp",))
+        if l["type"] != "latent_attention":
+            raise ConfigError(f"{at}.type: unknown mixer {l['type']!r}")
+        m = _take(l["mixer"], f"{at}.mixer", ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale"), ("rot", "kv_from"))
+        rot = m.pop("rot", None)
+        if rot is not None:
+            rot = RotaryConfig(**_take(rot, f"{at}.mixer.rot", ("base", "dims")), interleaved=True)
+        mlp: Optional[Mlp] = None
+        if l.get("mlp") is not None:
+            p = l["mlp"]
+            kind = p.get("kind") if isinstance(p, Mapping) else None
+            if kind == "dense":
+                mlp = DenseMlp(_take(p, f"{at}.mlp", ("kind", "ff"))["ff"], "relu")
+            elif kind == "moe":
+                p = _take(p, f"{at}.mlp", ("kind", "expert", "router"))
+                r = _take(p["router"], f"{at}.mlp.router", ("experts", "top"))
+                mlp = MoeMlp(r["experts"], r["top"], _take(p["expert"], f"{at}.mlp.expert", ("ff",))["ff"])
+            else:
+                raise ConfigError(f"{at}.mlp.kind: unknown feed-forward {kind!r}")
+        layers.append(HybridLayer(LatentAttentionMixer(**m, rotary=rot), mlp))
+    cfg = HybridConfig(d["vocab"], d["width"], tuple(layers), _take(d["norm"], "norm", ("eps",))["eps"],
+                       _take(d["embedding"], "embedding", ("scale",))["scale"], dtype, architecture="Domilix", block="post_norm")
+    cfg.validate()
+    return cfg
+
+
+def domilix_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
+    """The inverse of `domilix_config_from_json`."""
+    layers = []
+    for l in cfg.layers:
+        m = l.mixer
+        mixer: Dict[str, Any] = {k: getattr(m, k) for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale")}
+        if m.rotary is not None:
+            mixer["rot"] = {"base": m.rotary.base, "dims": m.rotary.dims}
+        if m.kv_from is not None:
+            mixer["kv_from"] = m.kv_from
+        p = l.mlp
+        mlp = None if p is None else {"kind": "dense", "ff": p.ff} if p.kind == "dense" else \
+            {"kind": "moe", "expert": {"ff": p.ff}, "router": {"experts": p.experts, "top": p.top}}
+        layers.append({"type": m.kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "layers": layers,
+            "norm": {"eps": cfg.norm_eps}, "embedding": {"scale": cfg.embedding_scale}}
+
+
 def hybrid_config_from_dict(d: Mapping[str, Any]) -> HybridConfig:
     """The inverse of `dataclasses.asdict(HybridConfig)` (the "model" section of an EngineConfig dictionary)."""
     d = dict(d)
     layers = []
     for l in d.pop("layers"):
         m = dict(l["mixer"])
+        r = m.pop("rotary", None)
+        if r is not None:
+            r = dict(r)
+            sc = r.pop("scaling", None)
+            r = RotaryConfig(**r, scaling=YarnScaling(**sc) if sc is not None else None)
         if "kv_heads" in m:
-            r = m.pop("rotary", None)
-            if r is not None:
-                r = dict(r)
-                sc = r.pop("scaling", None)
-                r = RotaryConfig(**r, scaling=YarnScaling(**sc) if sc is not None else None)
-            mixer: Union[AttentionMixer, MlstmMixer] = AttentionMixer(**m, rotary=r)
+            mixer: Mixer = AttentionMixer(**m, rotary=r)
+        elif "kv_rank" in m:
+            mixer = LatentAttentionMixer(**m, rotary=r)
         else:
             mixer = MlstmMixer(**m)
-        layers.append(HybridLayer(mixer, DenseMlp(**l["mlp"]) if l.get("mlp") is not None else None, l.get("weights_of")))
+        p = l.get("mlp")
+        mlp: Optional[Mlp] = None if p is None else MoeMlp(**p) if "experts" in p else DenseMlp(**p)
+        layers.append(HybridLayer(mixer, mlp, l.get("weights_of")))
     cfg = HybridConfig(layers=tuple(layers), **d)
     cfg.validate()
     return cfg
@@ -522,6 +675,38 @@ def hybrid_stack(n_layers: int, width: int, heads: int, kv_heads: int, dim: int,
     layers = tuple(HybridLayer(att if i % attention_every == attention_every - 1 else rec, DenseMlp(ff))
                    for i in range(n_layers))
     cfg = HybridConfig(vocab, width, layers, 1e-6, math.sqrt(width), dtype)
+    cfg.validate()
+    return cfg
+
+
+def latent_stack(n_layers: int, width: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, ff: int,
+                 experts: int, top: int, expert_ff: int, vocab: int, share_from: Optional[int] = None,
+                 dtype: str = "bfloat16") -> HybridConfig:
+    """A Domilix-shaped decoder: the first layer's feed-forward is dense, the others' are mixtures of experts (experts 0: all
+    dense); layers after `share_from` attend over that layer's latents."""
+    rot = RotaryConfig(10000.0, rot_dim, interleaved=True) if rot_dim else None
+    layers = []
+    for i in range(n_layers):
+        src = share_from if share_from is not None and i > share_from else None
+        mixer = LatentAttentionMixer(heads, dim, rot_dim, vdim, q_rank, kv_rank, (dim + rot_dim) ** -0.5, rot, src)
+        layers.append(HybridLayer(mixer, DenseMlp(ff, "relu") if i == 0 or experts == 0 else MoeMlp(experts, top, expert_ff)))
+    cfg = HybridConfig(vocab, width, tuple(layers), 1e-5, 1.0, dtype, architecture="Domilix", block="post_norm")
+    cfg.validate()
+    return cfg
+
+
+def tiny_latent_config(**over: Any) -> HybridConfig:
+    """CPU-sized Domilix-shaped decoder: dense, mixture of experts over the first layer's latents, and a layer without
+    feed-forward."""
+    rot = RotaryConfig(3000.0, 12, interleaved=True)
+    own = LatentAttentionMixer(3, 20, 12, 28, 40, 36, 0.21, rot)
+    kw: Dict[str, Any] = dict(vocab_size=300, hidden_size=88, norm_eps=2e-5, embedding_scale=1.5, architecture="Domilix",
+                              block="post_norm",
+                              layers=(HybridLayer(own, DenseMlp(104, "relu")),
+                                      HybridLayer(dataclasses.replace(own, heads=2, kv_from=0), MoeMlp(6, 2, 40)),
+                                      HybridLayer(own, None)))
+    kw.update(over)
+    cfg = HybridConfig(**kw)
     cfg.validate()
     return cfg
 

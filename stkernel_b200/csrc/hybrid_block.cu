@@ -1,20 +1,25 @@
-// Residual-side kernels of the parallel block (models/hybrid.py): scaled embedding into an fp32 residual, residual add fused
-// with the next layer norm, and the feed-forward half of the joined sublayer buffer.
+// Residual-side kernels of the layer-by-layer decoders (models/hybrid.py): scaled embedding into an fp32 residual, residual add
+// fused with the next norm (parallel block), norm of a sublayer's output fused with the residual add (post-norm block), and the
+// feed-forward half of the joined sublayer buffer.
 #define STK_PDL_CLASS 4
 #include "hybrid_block.cuh"
 
 namespace stk {
 
+// h != nullptr: the row also in the compute type E, zero-padded to `width` columns.
 template <typename E>
 __global__ void __launch_bounds__(256)
 embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed, float* __restrict__ x, long long ldx, int W,
-                    int vocab, float scale, int* status) {
+                    int vocab, float scale, E* __restrict__ h, long long ldh, int width, int* status) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
   const long long id = ids[t];
   const bool ok = id >= 0 && id < vocab;
   if (!ok && threadIdx.x == 0) set_status(status, kBadIndex, t);
+  if (h != nullptr)
+    for (int i = threadIdx.x; i < width; i += blockDim.x)
+      st_act(h + t * ldh + i, ok && i < W ? ld_act(embed + id * W + i) * scale : 0.f);
   if (sizeof(E) == 2 && (W & 7) == 0 && (ldx & 3) == 0) {
     for (int i = threadIdx.x * 8; i < W; i += blockDim.x * 8) {
       uint4 v = make_uint4(0, 0, 0, 0);
@@ -31,13 +36,14 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
     x[t * ldx + i] = ok ? ld_act(embed + id * W + i) * scale : 0.f;
 }
 
-// x[r] += y[r]; h[t] = layer_norm(x[r]) * w with r = rows ? rows[t] : t (with `rows` the sum is not written back).  The
-// row stays in shared memory between the three passes (mean, squared deviations, output), all in fp32.
+// x[r] += y[r]; h[t] = norm(x[r]) * w with r = rows ? rows[t] : t (with `rows` the sum is not written back).  The
+// row stays in shared memory between the three passes (mean, squared deviations, output), all in fp32.  center: layer norm,
+// otherwise RMS norm (no mean).
 template <typename O>
 __global__ void __launch_bounds__(1024)
 add_layer_norm_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy,
                       const float* __restrict__ w, O* __restrict__ h, long long ldh, int W, int width, float eps,
-                      const int64_t* __restrict__ rows) {
+                      const int64_t* __restrict__ rows, int center) {
   extern __shared__ __align__(16) float row[];
   __shared__ float red[32];
   pdl_wait();
@@ -69,7 +75,8 @@ add_layer_norm_kernel(float* __restrict__ x, long long ldx, const float* __restr
       s += v;
     }
   }
-  const float mean = block_sum(s, red) / static_cast<float>(W);
+  s = block_sum(s, red);                                  // also publishes the row
+  const float mean = center ? s / static_cast<float>(W) : 0.f;
   float q = 0.f;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     const float d = row[i] - mean;
@@ -88,11 +95,119 @@ add_layer_norm_kernel(float* __restrict__ x, long long ldx, const float* __restr
   }
 }
 
-// out[t, mix : o0) = 0, out[t, o0 + j] = silu(gate_j) * up_j for j < ff, zero up to `cols`.
+// x[t] += rms_norm(y[t]) * w and h[t] = x[t] in the compute type, zero-padded to `width` columns (h may be null).  y is either
+// one fp32 row per token, or the weighted sum of `top` expert rows: row pair_row[t * top + j] (t * top + j when pair_row is
+// null) times weights[t * top + j].
+template <typename A>
+struct PostNormArgs {
+  float* x; long long ldx;
+  const float* y; long long ldy;
+  const A* pairs; long long ldp; const int* pair_row; const float* weights; int top;
+  const float* w; float eps;
+  A* h; long long ldh;
+  int W, width;
+};
+
+template <typename A>
+__global__ void __launch_bounds__(1024)
+post_norm_add_kernel(const PostNormArgs<A> a) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[32];
+  __shared__ long long src[32];
+  __shared__ float wt[32];
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.x;
+  float q = 0.f;
+  if (a.pairs != nullptr) {
+    if (static_cast<int>(threadIdx.x) < a.top) {
+      const long long p = t * a.top + threadIdx.x;
+      const int r = a.pair_row != nullptr ? a.pair_row[p] : static_cast<int>(p);
+      src[threadIdx.x] = r < 0 ? 0 : r * a.ldp;
+      wt[threadIdx.x] = r < 0 ? 0.f : a.weights[p];
+    }
+    __syncthreads();
+    if (sizeof(A) == 2 && (a.W & 7) == 0 && (a.ldp & 7) == 0) {
+      for (int i = threadIdx.x * 8; i < a.W; i += blockDim.x * 8) {
+        float s[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) s[k] = 0.f;
+        for (int j = 0; j < a.top; ++j) {
+          const uint4 v = *reinterpret_cast<const uint4*>(a.pairs + src[j] + i);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float2 f = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[k]);
+            s[2 * k] = fmaf(wt[j], f.x, s[2 * k]);
+            s[2 * k + 1] = fmaf(wt[j], f.y, s[2 * k + 1]);
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) q = fmaf(s[k], s[k], q);
+        *reinterpret_cast<float4*>(row + i) = make_float4(s[0], s[1], s[2], s[3]);
+        *reinterpret_cast<float4*>(row + i + 4) = make_float4(s[4], s[5], s[6], s[7]);
+      }
+    } else {
+      for (int i = threadIdx.x; i < a.W; i += blockDim.x) {
+        float s = 0.f;
+        for (int j = 0; j < a.top; ++j) s = fmaf(wt[j], ld_act(a.pairs + src[j] + i), s);
+        row[i] = s;
+        q = fmaf(s, s, q);
+      }
+    }
+  } else if ((a.W & 3) == 0 && (a.ldy & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(a.y + t * a.ldy + i);
+      *reinterpret_cast<float4*>(row + i) = v;
+      q = fmaf(v.x, v.x, q); q = fmaf(v.y, v.y, q); q = fmaf(v.z, v.z, q); q = fmaf(v.w, v.w, q);
+    }
+  } else {
+    for (int i = threadIdx.x; i < a.W; i += blockDim.x) {
+      const float v = a.y[t * a.ldy + i];
+      row[i] = v;
+      q = fmaf(v, v, q);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(q, red) / static_cast<float>(a.W) + a.eps);
+  float* xr = a.x + t * a.ldx;
+  A* hr = a.h != nullptr ? a.h + t * a.ldh : nullptr;
+  if ((a.W & 3) == 0 && (a.ldx & 3) == 0 && (a.ldh & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
+      float4 v = *reinterpret_cast<const float4*>(xr + i);
+      const float4 r = *reinterpret_cast<const float4*>(row + i);
+      const float4 w = *reinterpret_cast<const float4*>(a.w + i);
+      v.x = fmaf(r.x * inv, w.x, v.x);
+      v.y = fmaf(r.y * inv, w.y, v.y);
+      v.z = fmaf(r.z * inv, w.z, v.z);
+      v.w = fmaf(r.w * inv, w.w, v.w);
+      *reinterpret_cast<float4*>(xr + i) = v;
+      if (hr != nullptr) {
+        if (sizeof(A) == 2) {
+          __nv_bfloat162 b[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+          *reinterpret_cast<uint2*>(hr + i) = *reinterpret_cast<const uint2*>(b);
+        } else {
+          *reinterpret_cast<float4*>(hr + i) = v;
+        }
+      }
+    }
+    if (hr != nullptr)
+      for (int i = a.W + threadIdx.x; i < a.width; i += blockDim.x) st_act(hr + i, 0.f);
+    return;
+  }
+  for (int i = threadIdx.x; i < (hr != nullptr ? a.width : a.W); i += blockDim.x) {
+    float v = 0.f;
+    if (i < a.W) {
+      v = fmaf(row[i] * inv, a.w[i], xr[i]);
+      xr[i] = v;
+    }
+    if (hr != nullptr) st_act(hr + i, v);
+  }
+}
+
+// out[t, mix : o0) = 0, out[t, o0 + j] = act(gate_j) * up_j for j < ff, zero up to `cols`.  relu: act is relu, else silu.
 template <typename A>
 __global__ void __launch_bounds__(256)
 join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int ff, A* __restrict__ out, long long ldo, int mix,
-                int o0, int cols) {
+                int o0, int cols, int relu) {
   pdl_wait();
   pdl_trigger();
   const long long t = blockIdx.y;
@@ -102,7 +217,7 @@ join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int f
   const int base = blockIdx.x * blockDim.x * 8 + threadIdx.x * 8;      // eight columns per thread, from o0 on
   if (blockIdx.x == 0)
     for (int i = mix + threadIdx.x; i < o0; i += blockDim.x) st_act(o + i, 0.f);
-  glu_columns(pg, pu, o + o0, base, ff, cols - o0, (ldo & 7) == 0 && (ldp & 7) == 0);
+  glu_columns(pg, pu, o + o0, base, ff, cols - o0, (ldo & 7) == 0 && (ldp & 7) == 0, relu);
 }
 
 }  // namespace stk
@@ -110,19 +225,20 @@ join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int f
 using namespace stk;
 
 STK_API int stk_embed_scaled(const int64_t* ids, const void* embed, int embed_fp32, float* x, long long ldx, int T, int W,
-                             int vocab, float scale, int* status, void* stream) {
+                             int vocab, float scale, void* h, long long ldh, int width, int* status, void* stream) {
   if (T <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   if (embed_fp32)
-    launch_pdl(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, ids, (const float*)embed, x, ldx, W, vocab, scale, status);
+    launch_pdl(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, ids, (const float*)embed, x, ldx, W, vocab, scale, (float*)h,
+               ldh, width, status);
   else
     launch_pdl(embed_scaled_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, ids, (const __nv_bfloat16*)embed, x, ldx, W, vocab,
-               scale, status);
+               scale, (__nv_bfloat16*)h, ldh, width, status);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 STK_API int stk_add_layer_norm(float* x, long long ldx, const float* y, long long ldy, const float* w, void* h, int h_fp32,
-                               long long ldh, int T, int W, int width, float eps, const int64_t* rows, void* stream) {
+                               long long ldh, int T, int W, int width, float eps, const int64_t* rows, int center, void* stream) {
   if (T <= 0) return 0;
   const size_t smem = static_cast<size_t>(W) * sizeof(float);
   if (smem > 200 * 1024) return -2;
@@ -137,15 +253,16 @@ STK_API int stk_add_layer_norm(float* x, long long ldx, const float* y, long lon
   // few rows: a wide row is spread over more threads (the step waits for this kernel); many rows: more rows at once
   const int threads = T > 148 || W <= 1024 ? 256 : (W <= 2048 ? 512 : 1024);
   if (h_fp32)
-    launch_pdl(add_layer_norm_kernel<float>, dim3(T), dim3(threads), smem, st, x, ldx, y, ldy, w, (float*)h, ldh, W, width, eps, rows);
+    launch_pdl(add_layer_norm_kernel<float>, dim3(T), dim3(threads), smem, st, x, ldx, y, ldy, w, (float*)h, ldh, W, width, eps, rows,
+               center);
   else
     launch_pdl(add_layer_norm_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, st, x, ldx, y, ldy, w, (__nv_bfloat16*)h, ldh, W,
-               width, eps, rows);
+               width, eps, rows, center);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 STK_API int stk_join_glu(const void* proj, long long ldp, int gate_off, int up_off, int ff, void* out, long long ldo, int fp32,
-                         int mixer_dim, int ff_off, int cols, int T, void* stream) {
+                         int mixer_dim, int ff_off, int cols, int relu, int T, void* stream) {
   if (T <= 0) return 0;
   if (T > 65535) return -1;
   const int n = cols - ff_off;
@@ -153,9 +270,35 @@ STK_API int stk_join_glu(const void* proj, long long ldp, int gate_off, int up_o
   cudaStream_t st = (cudaStream_t)stream;
   if (fp32)
     launch_pdl(join_glu_kernel<float>, grid, dim3(256), 0, st, (const float*)proj, ldp, gate_off, up_off, ff, (float*)out, ldo,
-               mixer_dim, ff_off, cols);
+               mixer_dim, ff_off, cols, relu);
   else
     launch_pdl(join_glu_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)proj, ldp, gate_off, up_off, ff,
-               (__nv_bfloat16*)out, ldo, mixer_dim, ff_off, cols);
+               (__nv_bfloat16*)out, ldo, mixer_dim, ff_off, cols, relu);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// pairs == nullptr: y [T, W] fp32 rows.  Otherwise the weighted sum of each token's `top` expert rows in the compute type.
+STK_API int stk_post_norm_add(float* x, long long ldx, const float* y, long long ldy, const void* pairs, long long ldp,
+                              const int* pair_row, const float* weights, int top, const float* w, float eps, void* h, long long ldh,
+                              int W, int width, int fp32, int T, void* stream) {
+  if (T <= 0) return 0;
+  const size_t smem = static_cast<size_t>(W) * sizeof(float);
+  if (smem > 200 * 1024 || top > 32 || (pairs == nullptr) == (y == nullptr)) return -2;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (smem > 40 * 1024) {
+    if (cudaFuncSetAttribute(post_norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(post_norm_add_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=
+            cudaSuccess)
+      return -3;
+  }
+  const int threads = T > 148 || W <= 1024 ? 256 : (W <= 2048 ? 512 : 1024);
+  if (fp32) {
+    const PostNormArgs<float> a{x, ldx, y, ldy, (const float*)pairs, ldp, pair_row, weights, top, w, eps, (float*)h, ldh, W, width};
+    launch_pdl(post_norm_add_kernel<float>, dim3(T), dim3(threads), smem, st, a);
+  } else {
+    const PostNormArgs<__nv_bfloat16> a{x,   ldx, y, ldy, (const __nv_bfloat16*)pairs, ldp, pair_row, weights, top,
+                                        w, eps, (__nv_bfloat16*)h, ldh, W, width};
+    launch_pdl(post_norm_add_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, st, a);
+  }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -11,9 +11,11 @@ template <typename T> __device__ __forceinline__ void st_act(T* p, float v);
 template <> __device__ __forceinline__ void st_act<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void st_act<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
-// o[j] = silu(gate_j) * up_j for j < ff, zero for ff <= j < n: the eight columns from `base` on.  vec: 16-byte accesses allowed.
+// o[j] = act(gate_j) * up_j for j < ff, zero for ff <= j < n: the eight columns from `base` on.  vec: 16-byte accesses allowed.
+// relu: act is relu, else silu.
 template <typename A>
-__device__ __forceinline__ void glu_columns(const A* pg, const A* pu, A* o, int base, int ff, int n, bool vec) {
+__device__ __forceinline__ void glu_columns(const A* pg, const A* pu, A* o, int base, int ff, int n, bool vec,
+                                            int relu = 0) {
   if (base >= n) return;
   if (sizeof(A) == 2 && base + 8 <= ff && vec) {
     const uint4 gv = *reinterpret_cast<const uint4*>(pg + base), uv = *reinterpret_cast<const uint4*>(pu + base);
@@ -24,7 +26,8 @@ __device__ __forceinline__ void glu_columns(const A* pg, const A* pu, A* o, int 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
-      o2[j] = __floats2bfloat162_rn(g.x / (1.f + __expf(-g.x)) * u.x, g.y / (1.f + __expf(-g.y)) * u.y);
+      o2[j] = relu ? __floats2bfloat162_rn(fmaxf(g.x, 0.f) * u.x, fmaxf(g.y, 0.f) * u.y)
+                   : __floats2bfloat162_rn(g.x / (1.f + __expf(-g.x)) * u.x, g.y / (1.f + __expf(-g.y)) * u.y);
     }
     *reinterpret_cast<uint4*>(o + base) = ov;
     return;
@@ -33,7 +36,7 @@ __device__ __forceinline__ void glu_columns(const A* pg, const A* pu, A* o, int 
     float v = 0.f;
     if (j < ff) {
       const float g = ld_act(pg + j);
-      v = g / (1.f + expf(-g)) * ld_act(pu + j);
+      v = (relu ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * ld_act(pu + j);
     }
     st_act(o + j, v);
   }

@@ -5,6 +5,7 @@
 // scores = sigmoid | sqrt(softplus) of the fp32 gate logits; selection by score + bias (or by a token-id hash table
 // with bounds checks); weights from the unbiased score, renormalised and scaled (topkGatingSoftplusSqrt /
 // fused_topk_bias and the hash-MoE lookup of overlay/nvidia_model.py:806-827).
+// Scoring 2 (softmax over the chosen): score = logit + bias, weights = softmax of the selected scores.
 #pragma once
 #include "common.cuh"
 
@@ -40,15 +41,16 @@ __device__ __forceinline__ void route_token_impl(const RouterArgs& r, const floa
       const float x = kCg ? __ldcg(row + e) : row[e];
       float s;
       if (r.scoring == 0) s = 1.f / (1.f + __expf(-x));
-      else s = sqrtf(x > 20.f ? x : log1pf(__expf(x)));
+      else if (r.scoring == 1) s = sqrtf(x > 20.f ? x : log1pf(__expf(x)));
+      else s = x + (r.bias ? r.bias[e] : 0.f);
       sc[i] = s;
-      sel[i] = s + (r.bias ? r.bias[e] : 0.f);
+      sel[i] = r.scoring == 2 ? s : s + (r.bias ? r.bias[e] : 0.f);
     } else {
       sc[i] = 0.f;
       sel[i] = -INFINITY;
     }
   }
-  float wsum = 0.f;
+  float wsum = 0.f, top = 0.f;
   float my_w = 0.f;      // lane j keeps the j-th selected weight
   int my_id = -1;
   if (r.tid2eid != nullptr) {
@@ -98,6 +100,10 @@ __device__ __forceinline__ void route_token_impl(const RouterArgs& r, const floa
         if (i * 32 + lane == best_e) { s = sc[i]; sel[i] = -INFINITY; }
       }
       s = __shfl_sync(0xffffffffu, s, best_e & 31);
+      if (r.scoring == 2) {
+        if (j == 0) top = s;
+        s = expf(s - top);
+      }
       wsum += s;
       if (lane == j) { my_w = s; my_id = best_e; }
     }

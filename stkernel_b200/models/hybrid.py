@@ -1,11 +1,16 @@
-"""Decoder described layer by layer (`HybridConfig`): attention and recurrent mixers in parallel blocks.
+"""Decoder described layer by layer (`HybridConfig`): attention and recurrent mixers, in parallel or post-norm blocks.
 
-A layer is two matrix products.  Everything that reads the layer's norm (mixer projections, feed-forward gate and up) is one
+Parallel block: a layer is two matrix products.  Everything that reads the layer's norm (mixer projections, feed-forward gate and up) is one
 weight `w_in`; everything that is added to the residual (mixer output and feed-forward down projection) is one weight `w_out`
 over the joined activations, so the sum of both sublayers is formed inside that product, and the fp32 residual is touched
 once per layer, by the kernel that also norms it for the next layer:
 
     h = norm(x += y_prev);  p = h W_in^T;  c = [mixer(p) | silu(p.gate) * p.up];  y = c W_out^T  (fp32)
+
+Post-norm block: both sublayers read the residual itself (its copy h in the compute type) and one kernel per sublayer norms the
+output, adds it to the fp32 residual and leaves the next copy; a mixture of experts' weighted sum is formed in that kernel too:
+
+    h = x += norm1(mixer(h));  h = x += norm2(ff(h))
 
 Segments of both weights start on 16-column boundaries (zero-padded), whatever the configured sizes.
 """
@@ -20,6 +25,8 @@ from ..config import HybridConfig, HybridLayer
 from ..ops import attention as A
 from ..ops import functional as Fn
 from ..ops import hybrid as HB
+from ..ops import latent as LA
+from ..ops import moe as MO
 from ..ops.functional import LinearWeight
 from ..utils.spans import span
 from .decoder import Decoder
@@ -47,6 +54,16 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
             out[f"{p}.mix.q"] = ((m.heads * m.dim, W), "bf16")
             out[f"{p}.mix.k"] = ((m.kv_heads * m.dim, W), "bf16")
             out[f"{p}.mix.sink"] = ((m.heads,), "bf16")
+        elif m.kind == "latent_attention":
+            out[f"{p}.mix.dq"] = ((m.q_rank, W), "bf16")
+            out[f"{p}.mix.dq.norm"] = ((m.q_rank,), "bf16")
+            out[f"{p}.mix.uq"] = ((m.heads * (m.dim + m.rot_dim), m.q_rank), "bf16")
+            if m.kv_from is None:
+                out[f"{p}.mix.dkv"] = ((m.kv_rank + m.rot_dim, W), "bf16")
+                out[f"{p}.mix.dkv.norm"] = ((m.kv_rank,), "bf16")
+            out[f"{p}.mix.uk"] = ((m.heads * m.dim, m.kv_rank), "bf16")
+            out[f"{p}.mix.uv"] = ((m.heads * m.vdim, m.kv_rank), "bf16")
+            out[f"{p}.mix.g"] = ((m.heads, W), "bf16")
         else:
             out[f"{p}.mix.q"] = ((m.heads * m.dim, W), "bf16")
             out[f"{p}.mix.k"] = ((m.heads * m.dim, W), "bf16")
@@ -58,9 +75,18 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
                 out[f"{p}.mix.{g}.b"] = ((m.heads,), "bf16")
         out[f"{p}.mix.o"] = ((W, m.out_dim), "bf16")
         if l.mlp is not None:
-            out[f"{p}.mlp.gate"] = ((l.mlp.ff, W), "bf16")
-            out[f"{p}.mlp.up"] = ((l.mlp.ff, W), "bf16")
-            out[f"{p}.mlp.down"] = ((W, l.mlp.ff), "bf16")
+            if cfg.block == "post_norm":
+                out[f"{p}.norm2"] = ((W,), "bf16")
+            if l.mlp.kind == "dense":
+                out[f"{p}.mlp.gate"] = ((l.mlp.ff, W), "bf16")
+                out[f"{p}.mlp.up"] = ((l.mlp.ff, W), "bf16")
+                out[f"{p}.mlp.down"] = ((W, l.mlp.ff), "bf16")
+            else:
+                for e in range(l.mlp.experts):
+                    out[f"{p}.mlp.e{e}.up"] = ((l.mlp.ff, W), "bf16")
+                    out[f"{p}.mlp.e{e}.down"] = ((W, l.mlp.ff), "bf16")
+                out[f"{p}.mlp.router"] = ((l.mlp.experts, W), "bf16")
+                out[f"{p}.mlp.router.b"] = ((l.mlp.experts,), "bf16")
     out["final.norm"] = ((W,), "bf16")
     out["head"] = ((cfg.vocab_size, W), "bf16")
     return out
@@ -96,7 +122,15 @@ class BlockWeights:
     seg: Dict[str, int]                     # first column of each segment of the w_in product
     attention: Optional[HB.AttentionParams] = None
     mlstm: Optional[HB.MlstmParams] = None
+    latent: Optional[LA.LatentParams] = None
     w_gates: Optional[LinearWeight] = None  # [2 * heads, pad(W)]: input and forget gate of the recurrence (fp32 results)
+    # post-norm blocks: the feed-forward has weights of its own
+    norm2: Optional[torch.Tensor] = None    # fp32 [W]
+    w_gate_up: Optional[LinearWeight] = None
+    w_down: Optional[LinearWeight] = None
+    router: Optional[LinearWeight] = None   # [experts, pad(W)]
+    router_bias: Optional[torch.Tensor] = None          # fp32 [experts]
+    experts: Optional[MO.PlainExperts] = None
 
 
 @dataclass
@@ -121,6 +155,30 @@ def _stack(parts: List[Tuple[str, torch.Tensor]], width: int, dtype) -> Tuple[Li
     return LinearWeight(w), seg
 
 
+def _spread(w: torch.Tensor, heads: int, rows: int, pad_rows: int, width: int, dtype) -> torch.Tensor:
+    """[heads * rows, K] -> [heads * pad_rows, width]: zero rows after each head's, zero columns after K."""
+    out = torch.zeros(heads, pad_rows, width, dtype=dtype, device=w.device)
+    out[:, :rows, :w.shape[1]] = w.view(heads, rows, -1).to(dtype)
+    return out.view(heads * pad_rows, width)
+
+
+def build_latent(cfg: HybridConfig, get, m, dt, device) -> LA.LatentParams:
+    H, D, R, C, Q = m.heads, m.dim, m.rot_dim, m.kv_rank, m.q_rank
+    dp, cp, vp = LA.head_pads(m)
+    f32 = lambda n: get(n).to(F32).contiguous()
+    uq = get("mix.uq").view(H, D + R, Q)
+    w_uq = torch.zeros(H * dp + _pad(H * R), _pad(Q), dtype=dt, device=device)
+    w_uq[:H * dp] = _spread(uq[:, :D].reshape(H * D, Q), H, D, dp, _pad(Q), dt)
+    if R:
+        w_uq[H * dp:H * dp + H * R, :Q] = uq[:, D:].reshape(H * R, Q).to(dt)
+    w_uk = _spread(get("mix.uk").view(H, D, C).transpose(1, 2).reshape(H * C, D), H, C, cp, dp, dt)
+    w_uv = _spread(get("mix.uv"), H, m.vdim, vp, cp, dt)
+    freq = m.rotary.frequencies()[0] if m.rotary is not None else []
+    return LA.LatentParams(H, D, R, m.vdim, Q, C, m.scale, cfg.norm_eps, dp, cp, vp, LA.split_frequencies(freq, device),
+                           f32("mix.dq.norm"), f32("mix.dkv.norm") if m.kv_from is None else None, LinearWeight(w_uq),
+                           LinearWeight(w_uk), LinearWeight(w_uv))
+
+
 def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWeights:
     l: HybridLayer = cfg.layers[i]
     shapes = weight_shapes(cfg)
@@ -128,28 +186,63 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
     f32 = lambda n: get(n).to(F32).contiguous()
     dt = F32 if cfg.dtype == "float32" else BF16
     m, W = l.mixer, cfg.hidden_size
-    names = ["q", "k"] + (["v", "g"] if m.kind == "mlstm" else [])
+    joined = l.mlp if cfg.block == "parallel" else None              # the feed-forward shares the mixer's two products
+    if m.kind == "latent_attention":
+        names = ["dq", "dkv", "g"] if m.kv_from is None else ["dq", "g"]
+    else:
+        names = ["q", "k"] + (["v", "g"] if m.kind == "mlstm" else [])
     parts = [(n, get(f"mix.{n}")) for n in names]
-    if l.mlp is not None:
+    if joined is not None:
         parts += [("gate", get("mlp.gate")), ("up", get("mlp.up"))]
     w_in, seg = _stack(parts, _pad(W), dt)
-    off = HB.out_offset(m.out_dim)
-    w_out = torch.zeros(W, off + (_pad(l.mlp.ff) if l.mlp is not None else 0), dtype=dt, device=device)
-    w_out[:, :m.out_dim] = get("mix.o").to(dt)
-    if l.mlp is not None:
-        w_out[:, off:off + l.mlp.ff] = get("mlp.down").to(dt)
+    if m.kind == "latent_attention":
+        vp = LA.head_pads(m)[2]
+        w_out = torch.zeros(W, m.heads, vp, dtype=dt, device=device)
+        w_out[:, :, :m.vdim] = get("mix.o").view(W, m.heads, m.vdim).to(dt)
+        w_out = w_out.view(W, m.heads * vp)
+    else:
+        off = HB.out_offset(m.out_dim)
+        w_out = torch.zeros(W, off + (_pad(joined.ff) if joined is not None else 0), dtype=dt, device=device)
+        w_out[:, :m.out_dim] = get("mix.o").to(dt)
+        if joined is not None:
+            w_out[:, off:off + joined.ff] = get("mlp.down").to(dt)
     b = BlockWeights(f32("norm1"), w_in, LinearWeight(w_out), seg)
     if m.kind == "attention":
         freq, mag = m.rotary.frequencies() if m.rotary is not None else ([], 1.0)
         b.attention = HB.AttentionParams(m.heads, m.kv_heads, m.dim, m.window, m.scale, m.softcap,
                                          torch.tensor(freq, dtype=torch.float64).to(F32).to(device), mag,
                                          f32("mix.sink") if m.sink else None)
+    elif m.kind == "latent_attention":
+        b.latent = build_latent(cfg, get, m, dt, device)
     else:
         b.w_gates, _ = _stack([("i", torch.cat([get("mix.i"), get("mix.f")], 0))], _pad(W), dt)
         b.w_gates = LinearWeight(b.w_gates.w[:2 * m.heads])
         b.mlstm = HB.MlstmParams(m.heads, m.dim, m.vdim, m.gate_cap, torch.cat([f32("mix.i.b"), f32("mix.f.b")]).contiguous(),
                                  f32("mix.norm"), cfg.norm_eps)
+    if l.mlp is not None and joined is None:
+        build_feed_forward(b, l.mlp, get, W, dt, device)
     return b
+
+
+def build_feed_forward(b: BlockWeights, mlp, get, W: int, dt, device) -> None:
+    b.norm2 = get("norm2").to(F32).contiguous()
+    ff = _pad(mlp.ff)
+    if mlp.kind == "dense":
+        b.w_gate_up, seg = _stack([("gate", get("mlp.gate")), ("up", get("mlp.up"))], _pad(W), dt)
+        b.seg.update(seg)
+        down = torch.zeros(W, ff, dtype=dt, device=device)
+        down[:, :mlp.ff] = get("mlp.down").to(dt)
+        b.w_down = LinearWeight(down)
+        return
+    up = torch.zeros(mlp.experts, ff, _pad(W), dtype=dt, device=device)
+    down = torch.zeros(mlp.experts, _pad(W), ff, dtype=dt, device=device)
+    for e in range(mlp.experts):
+        up[e, :mlp.ff, :W] = get(f"mlp.e{e}.up").to(dt)
+        down[e, :W, :mlp.ff] = get(f"mlp.e{e}.down").to(dt)
+    b.experts = MO.PlainExperts(up, down)
+    router, _ = _stack([("router", get("mlp.router"))], _pad(W), dt)
+    b.router = LinearWeight(router.w[:mlp.experts])
+    b.router_bias = get("mlp.router.b").to(F32).contiguous()
 
 
 def build_hybrid_weights(cfg: HybridConfig, src: WeightSource, device) -> HybridWeights:
@@ -184,31 +277,91 @@ class HybridModel(Decoder):
                    spans: Tuple[int, int] = (1, 1)) -> HB.HybridMeta:
         tok_req, positions, first, last = A.token_maps(buf.d_qstart, buf.d_rows, buf.d_start, n_req, t_pad)
         return HB.HybridMeta(buf.d_tokens[:t_pad], tok_req, positions, first, last, buf.d_qstart, buf.d_rows, buf.d_start, n_req,
-                             spans[1], pure_decode, spans[0])
+                             spans[1], pure_decode, spans[0], 4 * max_comp_rows + 4)
+
+    def decode_bucket(self, max_comp_rows: int) -> int:
+        # full-context attention splits the key range by the longest context a graph serves: one graph per power of two
+        if self.kv.full is None:
+            return 0
+        bucket = 256
+        while bucket < max_comp_rows + 1:
+            bucket *= 2
+        return bucket
 
     def layer(self, li: int, x: torch.Tensor, y: Optional[torch.Tensor], meta: HB.HybridMeta) -> torch.Tensor:
-        """Adds the previous layer's output y to the residual x (in place) and returns this layer's output [T, W] fp32."""
+        """Parallel block: adds the previous layer's output y to the residual x (in place) and returns this layer's output
+        [T, W] fp32."""
         cfg, b = self.cfg, self.w.layers[li]
         m, mlp = cfg.layers[li].mixer, cfg.layers[li].mlp
-        t = x.shape[0]
         h = HB.add_layer_norm(x, y, b.norm, cfg.norm_eps, self.width, self.act)
-        p = Fn.linear(h, b.w_in, tag="in")
-        c = torch.empty(t, b.w_out.in_features, dtype=self.act, device=x.device)
         glu = (b.seg["gate"], b.seg["up"], mlp.ff) if mlp is not None else None
+        c = self.mix(li, h, meta, glu, mlp.act if mlp is not None else "silu")
+        return Fn.linear(c, b.w_out, out_dtype=F32, tag="out")
+
+    def mix(self, li: int, h: torch.Tensor, meta: HB.HybridMeta, glu: Optional[Tuple[int, int, int]] = None,
+            act: str = "silu") -> torch.Tensor:
+        """Mixer output of layer li (before its output projection), joined with the feed-forward activation where the block
+        shares its products (glu)."""
+        b, m = self.w.layers[li], self.cfg.layers[li].mixer
+        t = h.shape[0]
+        if m.kind == "latent_attention":
+            p = Fn.linear(h, b.w_in, out_dtype=F32, tag="in")
+            src = self.cfg.cache_layer(li)
+            table, cache = self.kv.group_of(src).table_dev, self.kv.kv_cache[src]
+            cq = LA.latent_prep(p, b.seg["dq"], b.seg.get("dkv", -1), b.latent, meta, table, cache, self.act)
+            q = Fn.linear(cq, b.latent.w_uq, tag="uq")
+            with span("latent_attention", t):
+                return LA.latent_attention(q, p[:, b.seg["g"]:b.seg["g"] + m.heads], b.latent, meta, table, cache)
+        p = Fn.linear(h, b.w_in, tag="in")
+        c = torch.empty(t, b.w_out.in_features, dtype=self.act, device=h.device)
         if m.kind == "attention":
             with span("window_attention", t):
                 HB.window_attention(p, b.seg["q"], b.seg["k"], b.attention, meta, self.kv.group_of(li).table_dev,
                                     self.kv.kv_cache[li], c)
-                HB.join_glu(p, c, m.out_dim, glu)
+                HB.join_glu(p, c, m.out_dim, glu, act)
         else:
             with span("mlstm", t):
                 gates = Fn.linear(h, b.w_gates, out_dtype=F32, tag="gates")
                 HB.mlstm(p, b.seg["q"], b.seg["k"], b.seg["v"], b.seg["g"], gates, b.mlstm, meta, self.kv.state[li], c, glu)
-        return Fn.linear(c, b.w_out, out_dtype=F32, tag="out")
+        return c
+
+    def feed_forward(self, li: int, h: torch.Tensor):
+        """Feed-forward output of a post-norm layer: fp32 rows, or expert rows whose sum the norm forms."""
+        b, mlp = self.w.layers[li], self.cfg.layers[li].mlp
+        if mlp.kind == "dense":
+            p = Fn.linear(h, b.w_gate_up, tag="gate_up")
+            c = torch.empty(h.shape[0], b.w_down.in_features, dtype=self.act, device=h.device)
+            HB.join_glu(p, c, 0, (b.seg["gate"], b.seg["up"], mlp.ff), mlp.act)
+            return Fn.linear(c, b.w_down, out_dtype=F32, tag="down")
+        with span("experts", h.shape[0]):
+            routed = Fn.gate_route(h, b.router, b.router_bias, mlp.top, "softmax_topk", True, 1.0)
+            if routed is None:
+                logits = Fn.linear(h, b.router, out_dtype=F32, tag="router")
+                routed = MO.router(logits, b.router_bias, mlp.top, "softmax_topk", True, 1.0)
+            return MO.plain_experts(h, *routed, b.experts)
+
+    def post_norm_layer(self, li: int, x: torch.Tensor, h: torch.Tensor, meta: HB.HybridMeta) -> torch.Tensor:
+        """Adds both sublayers to the residual x (in place); h is x in the compute type, as is the result."""
+        cfg, b = self.cfg, self.w.layers[li]
+        y = Fn.linear(self.mix(li, h, meta), b.w_out, out_dtype=F32, tag="out")
+        h = HB.post_norm_add(x, y, b.norm, cfg.norm_eps, self.width, self.act)
+        if cfg.layers[li].mlp is not None:
+            h = HB.post_norm_add(x, self.feed_forward(li, h), b.norm2, cfg.norm_eps, self.width, self.act)
+        return h
 
     def forward_hidden(self, meta: HB.HybridMeta):
-        """-> (residual before the last layer's output, that output), both [T, W] fp32: the sum is formed where it is normed."""
-        x = HB.embed_scaled(meta.token_ids, self.w.embed, self.cfg.embedding_scale)
+        """-> (residual before the last layer's output, that output), both [T, W] fp32: the sum is formed where it is normed.
+        Post-norm blocks: (residual, None)."""
+        cfg = self.cfg
+        if cfg.block == "post_norm":
+            h = torch.empty(meta.token_ids.shape[0], self.width, dtype=self.act, device=self.device)
+            x = HB.embed_scaled(meta.token_ids, self.w.embed, cfg.embedding_scale, h)
+            for li in range(len(self.w.layers)):
+                h = self.post_norm_layer(li, x, h, meta)
+                if self.on_layer is not None:
+                    self.on_layer(li, x.clone())
+            return x, None
+        x = HB.embed_scaled(meta.token_ids, self.w.embed, cfg.embedding_scale)
         y = None
         for li in range(len(self.w.layers)):
             y = self.layer(li, x, y, meta)
@@ -218,7 +371,8 @@ class HybridModel(Decoder):
 
     def head_hidden(self, X, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         x, y = X
-        return HB.add_layer_norm(x, y, self.w.norm, self.cfg.norm_eps, self.width, self.act, rows=rows)
+        return HB.add_layer_norm(x, y, self.w.norm, self.cfg.norm_eps, self.width, self.act, rows=rows,
+                                 center=self.cfg.block == "parallel")
 
     def compute_logits(self, h: torch.Tensor) -> torch.Tensor:
         return Fn.linear(h, self.w.head, out_dtype=F32, tag="head")

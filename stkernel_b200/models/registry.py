@@ -13,7 +13,7 @@ from typing import Any, Callable, Dict, Mapping, Optional, Tuple
 
 import torch
 
-from ..config import ConfigError, EngineConfig, model_config_from_hf, timalorn_config_from_json
+from ..config import ConfigError, EngineConfig, domilix_config_from_json, model_config_from_hf, timalorn_config_from_json
 
 
 @dataclass(frozen=True)
@@ -24,7 +24,8 @@ class ModelFamily:
     make_cache: Callable[..., Any]             # (engine cfg, device, context, comm, tp_rank, pipe) -> cache manager
     make_model: Callable[..., Any]             # (engine cfg, weights, cache, comm, tp_rank) -> Decoder
     prefix_cache: bool                         # prefixes can be kept and adopted
-    native_sources: Optional[Tuple[str, ...]] = None    # .cu files its steps need (None: the whole library)
+    # cfg -> (name, .cu files) of the library that holds just the kernels its steps need; None: the whole library
+    native_sources: Optional[Callable[[Any], Tuple[str, Tuple[str, ...]]]] = None
 
 
 # ---- DeepSeek-V4-style -----------------------------------------------------------------------
@@ -84,9 +85,16 @@ def _hybrid_weights(cfg, src, device, tp_rank=0, tp_size=1, layer_range=None):
 
 
 def _hybrid_cache(cfg: EngineConfig, device, ctx: int, comm, tp_rank: int, pipe):
-    from ..runtime.kv import HybridKVManager
+    from ..runtime.kv import HybridKVManager, hybrid_bytes_per_context_token
     sc = cfg.sched
-    return HybridKVManager(cfg.model, device, sc.max_num_seqs, ctx + 64, sc.max_num_batched_tokens, cfg.cache.num_pages or 0)
+    pool_tokens = cfg.cache.kv_pool_tokens
+    per_token = hybrid_bytes_per_context_token(cfg.model)
+    if pool_tokens is None and cfg.cache.size_by_memory and device.type == "cuda" and per_token:
+        free, total = torch.cuda.mem_get_info(device)
+        budget = cfg.cache.gpu_memory_utilization * total - (total - free)
+        pool_tokens = max(ctx, int(budget / per_token))
+    return HybridKVManager(cfg.model, device, sc.max_num_seqs, ctx + 64, sc.max_num_batched_tokens, cfg.cache.num_pages or 0,
+                           pool_tokens)
 
 
 def _hybrid_model(cfg: EngineConfig, weights, kv, comm, tp_rank: int):
@@ -94,18 +102,36 @@ def _hybrid_model(cfg: EngineConfig, weights, kv, comm, tp_rank: int):
     return HybridModel(cfg.model, weights, kv)
 
 
+_HYBRID_SOURCES = ("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", "linear_f32.cu", "hybrid_block.cu", "sampler.cu")
+_MECHANISM_SOURCES = {"attention": ("window_attention.cu", "window_attention_tc.cu"), "mlstm": ("mlstm.cu",), "dense": (),
+                      "latent_attention": ("latent_attention.cu",),
+                      "moe": ("moe.cu", "moe_plain.cu", "gate_cluster.cu")}
+
+
+def _hybrid_sources(cfg) -> Tuple[str, Tuple[str, ...]]:
+    kinds = [k for k in cfg.mechanisms() if _MECHANISM_SOURCES[k]]
+    return "-".join(["hybrid"] + kinds), _HYBRID_SOURCES + tuple(f for k in kinds for f in _MECHANISM_SOURCES[k])
+
+
 FAMILIES: Dict[str, ModelFamily] = {
     "dsv4": ModelFamily("dsv4", _dsv4_shapes, _dsv4_weights, _dsv4_cache, _dsv4_model, prefix_cache=True),
     "hybrid": ModelFamily("hybrid", _hybrid_shapes, _hybrid_weights, _hybrid_cache, _hybrid_model, prefix_cache=False,
-                          native_sources=("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", "linear_f32.cu",
-                                          "hybrid_block.cu", "window_attention.cu", "window_attention_tc.cu",
-                                          "mlstm.cu", "sampler.cu")),
+                          native_sources=_hybrid_sources),
 }
 
 # architecture name in config.json -> configuration parser
 ARCHITECTURES: Dict[str, Callable[..., Any]] = {
     "Timalorn": timalorn_config_from_json,
+    "Domilix": domilix_config_from_json,
 }
+
+
+def use_native(cfg) -> None:
+    """Load the kernels a model needs (compiling them when the checkout has none); before the first kernel of the process."""
+    f = family_of(cfg)
+    if f.native_sources is not None:
+        from ..ops import _lib
+        _lib.use_family(*f.native_sources(cfg))
 
 
 def family_of(cfg) -> ModelFamily:

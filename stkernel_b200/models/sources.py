@@ -42,11 +42,11 @@ class RandomSource(WeightSource):
         g = self._gen(name, dev)
         if name.endswith("tid2eid"):
             return torch.randint(0, 1 << 30, shape, generator=g, device=dev, dtype=torch.int64)
-        if name.endswith(("norm.weight", "_scale", ".norm", ".norm1")):
+        if name.endswith(("norm.weight", "_scale", ".norm", ".norm1", ".norm2")):
             return torch.ones(shape, device=dev)
         if name.endswith(".f.b"):
             return 3.0 + 3.0 * torch.rand(shape, generator=g, device=dev)      # forget gates of a recurrence start near one
-        if name.endswith(("_base", "attn_sink", ".sink", ".i.b")):
+        if name.endswith(("_base", "attn_sink", ".sink", ".i.b", ".router.b")):
             return torch.zeros(shape, device=dev)
         if name.endswith("gate.bias"):
             return torch.rand(shape, generator=g, device=dev) * 0.2 - 0.1

@@ -185,7 +185,7 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
     ll: an `LLExchange`; the bf16 result is a per-rank partial sum that goes into the folded all-reduce and an
     `LLPending` is returned instead of a tensor (row-parallel layers at decode sizes)."""
     if lw.w.dtype == F32:
-        return _linear_f32(x, lw, out)
+        return _linear_f32(x, lw, out, groups)
     if (norm is not None or ll is not None) and not isinstance(x, QuantAct) and x.is_cuda:
         t0, (n0, k0) = x.shape[0], lw.w.shape
         if groups == 1 and ar_ctx is None and out_dtype == BF16 and _skinny_ok(x, t0, k0, lw.is_fp8, n0 // max(groups, 1), n0) and (ll is None or n0 % 2 == 0):
@@ -259,9 +259,16 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
     return out
 
 
-def _linear_f32(x: torch.Tensor, lw: LinearWeight, out: Optional[torch.Tensor]) -> torch.Tensor:
+def _linear_f32(x: torch.Tensor, lw: LinearWeight, out: Optional[torch.Tensor], groups: int = 1) -> torch.Tensor:
     """fp32 x fp32 -> fp32 on the CUDA cores (no tf32 anywhere): models that run in float32."""
     t, (n, k) = x.shape[0], lw.w.shape
+    if groups > 1:
+        if out is None:
+            out = torch.empty(t, n, dtype=F32, device=x.device)
+        m = n // groups
+        for g in range(groups):
+            _linear_f32(x[:, g * k:(g + 1) * k], LinearWeight(lw.w[g * m:(g + 1) * m]), out[:, g * m:(g + 1) * m])
+        return out
     if not x.is_cuda:
         y = x.to(F32) @ lw.w.t()
         if out is not None:
@@ -288,6 +295,9 @@ def _gate_cluster_ok() -> bool:
     return _gate_cluster_state[d]
 
 
+SCORING = {"sigmoid": 0, "sqrtsoftplus": 1, "softmax_topk": 2}
+
+
 def gate_route(x: torch.Tensor, w_gate: LinearWeight, bias, top_k: int, scoring: str, renorm: bool, scaling: float,
                tid2eid=None, token_ids=None):
     """Router gate projection and expert selection in one launch for decode-sized batches (the CTA that finishes the
@@ -306,7 +316,7 @@ def gate_route(x: torch.Tensor, w_gate: LinearWeight, bias, top_k: int, scoring:
             and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and _gate_cluster_ok()):
         # one 16-CTA cluster: the logits meet in distributed shared memory instead of global memory
         _lib.call("stk_gate_route_cluster", w, w.stride(0), x, x.stride(0), t, e, k, bias, tid2eid, token_ids, vocab, ids,
-                  wts, top_k, 0 if scoring == "sigmoid" else 1, 1 if renorm else 0, float(scaling), _lib.status_buffer(),
+                  wts, top_k, SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(),
                   _lib.stream())
         return ids, wts
     cnt = _route_counters.get(dev.index)
@@ -316,7 +326,7 @@ def gate_route(x: torch.Tensor, w_gate: LinearWeight, bias, top_k: int, scoring:
     _lib.call("stk_skinny_linear_fused", w_gate.w, w_gate.w.stride(0), 1 if w_gate.is_fp8 else 0, w_gate.scale,
               w_gate.scale.stride(0) if w_gate.is_fp8 else 0, x, x.stride(0), logits, logits.stride(0), t, e, k, 1,
               _lib.sm_count(), None, 0.0, None, 2, cnt, bias, tid2eid, token_ids, vocab, ids, wts, top_k,
-              0 if scoring == "sigmoid" else 1, 1 if renorm else 0, float(scaling), _lib.status_buffer(), _lib.stream())
+              SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(), _lib.stream())
     return ids, wts
 
 

@@ -1,5 +1,6 @@
-"""Ops of the hybrid decoder: scaled embedding and add + layer norm on an fp32 residual, paged windowed attention whose
-values are the unrotated keys, mLSTM recurrence, and the parallel block's joined sublayer outputs.
+"""Ops of the layer-by-layer decoders: scaled embedding, add + norm and norm + add on an fp32 residual, paged windowed attention
+whose values are the unrotated keys, mLSTM recurrence, and the parallel block's joined sublayer outputs.  (Latent attention:
+`ops/latent.py`; experts: `ops/moe.py`.)
 
 Activations are bf16, or fp32 in a float32 model (every kernel here has both forms; the fp32 forms use no reduced-precision
 products).  Residual, norms, scores and softmax, gates and recurrent state are fp32 in either.
@@ -42,22 +43,27 @@ def _is32(t: torch.Tensor) -> int:
 # ----------------------------------------------------------------------------
 # residual
 # ----------------------------------------------------------------------------
-def embed_scaled(ids: torch.Tensor, embed: torch.Tensor, scale: float) -> torch.Tensor:
-    """ids [T] -> fp32 residual [T, W] = embed[id] * scale."""
+def embed_scaled(ids: torch.Tensor, embed: torch.Tensor, scale: float, h: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """ids [T] -> fp32 residual [T, W] = embed[id] * scale.  h [T, width]: receives the rows in the compute type as well,
+    zero-padded."""
+    t, w = ids.shape[0], embed.shape[1]
     if not ids.is_cuda:
         ok = (ids >= 0) & (ids < embed.shape[0])
-        return torch.where(ok[:, None], embed[ids.clamp(0, embed.shape[0] - 1)].to(F32) * scale, torch.zeros(1))
-    t, w = ids.shape[0], embed.shape[1]
+        x = torch.where(ok[:, None], embed[ids.clamp(0, embed.shape[0] - 1)].to(F32) * scale, torch.zeros(1))
+        if h is not None:
+            h.zero_()
+            h[:, :w] = x.to(h.dtype)
+        return x
     x = torch.empty(t, w, dtype=F32, device=ids.device)
-    _lib.call("stk_embed_scaled", ids, embed, _is32(embed), x, w, t, w, embed.shape[0], float(scale), _lib.status_buffer(),
-              _lib.stream())
+    _lib.call("stk_embed_scaled", ids, embed, _is32(embed), x, w, t, w, embed.shape[0], float(scale), h,
+              h.stride(0) if h is not None else 0, h.shape[1] if h is not None else 0, _lib.status_buffer(), _lib.stream())
     return x
 
 
 def add_layer_norm(x: torch.Tensor, y: Optional[torch.Tensor], w: torch.Tensor, eps: float, width: int, dtype: torch.dtype,
-                   rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   rows: Optional[torch.Tensor] = None, center: bool = True) -> torch.Tensor:
     """x += y (fp32, in place; y None: nothing to add), then the layer norm of x in `dtype`, zero-padded to `width` columns.
-    rows: only these rows are normed (and the addition is not written back)."""
+    rows: only these rows are normed (and the addition is not written back).  center False: RMS norm."""
     w_n = x.shape[1]
     if not x.is_cuda:
         if rows is not None:
@@ -66,12 +72,36 @@ def add_layer_norm(x: torch.Tensor, y: Optional[torch.Tensor], w: torch.Tensor, 
         elif y is not None:
             x += y
         h = torch.zeros(x.shape[0], width, dtype=dtype)
-        h[:, :w_n] = R.layer_norm(x, w, eps).to(dtype)
+        h[:, :w_n] = (R.layer_norm if center else R.rms_norm)(x, w, eps).to(dtype)
         return h
     t = x.shape[0] if rows is None else rows.shape[0]
     h = torch.empty(t, width, dtype=dtype, device=x.device)
     _lib.call("stk_add_layer_norm", x, x.stride(0), y, y.stride(0) if y is not None else 0, w, h, _is32(h), width, t, w_n, width,
-              float(eps), rows, _lib.stream())
+              float(eps), rows, 1 if center else 0, _lib.stream())
+    return h
+
+
+def post_norm_add(x: torch.Tensor, y, w: torch.Tensor, eps: float, width: int, dtype: torch.dtype) -> torch.Tensor:
+    """x += rms_norm(y) * w (fp32, in place) -> x in `dtype`, zero-padded to `width` columns.  y: fp32 [T, W], or `ExpertRows`
+    whose weighted sum over each token's pairs is normed."""
+    t, w_n = x.shape
+    rows = None if isinstance(y, torch.Tensor) else y
+    if not x.is_cuda:
+        if rows is not None:
+            k = rows.weights.shape[1]
+            at = rows.pair_row.long() if rows.pair_row is not None else torch.arange(t * k)
+            y = (rows.y[at].to(F32).view(t, k, -1)[..., :w_n] * rows.weights[..., None]).sum(1)
+        x += R.rms_norm(y, w, eps)
+        h = torch.zeros(t, width, dtype=dtype)
+        h[:, :w_n] = x.to(dtype)
+        return h
+    h = torch.empty(t, width, dtype=dtype, device=x.device)
+    common = (w, float(eps), h, h.stride(0), w_n, width, _is32(h), t, _lib.stream())
+    if rows is None:
+        _lib.call("stk_post_norm_add", x, x.stride(0), y, y.stride(0), None, 0, None, None, 0, *common)
+    else:
+        _lib.call("stk_post_norm_add", x, x.stride(0), None, 0, rows.y, rows.y.stride(0), rows.pair_row, rows.weights,
+                  rows.weights.shape[1], *common)
     return h
 
 
@@ -93,6 +123,7 @@ class HybridMeta:
     max_span: int                  # longest span of the step (host knowledge: which kernels have work)
     pure_decode: bool = False      # every span is one token
     min_span: int = 1
+    max_context: int = 1 << 30     # no token of the step sees more keys (host knowledge: how far to split the key range)
 
 
 # ----------------------------------------------------------------------------
@@ -206,8 +237,9 @@ def out_offset(mixer_dim: int) -> int:
     return (mixer_dim + 15) // 16 * 16
 
 
-def join_glu(proj: torch.Tensor, out: torch.Tensor, mixer_dim: int, glu: Optional[Tuple[int, int, int]]) -> None:
-    """out[:, out_offset(mixer_dim):] = silu(gate) * up with (gate, up) at columns glu[0], glu[1] of proj, glu[2] wide (None:
+def join_glu(proj: torch.Tensor, out: torch.Tensor, mixer_dim: int, glu: Optional[Tuple[int, int, int]],
+             act: str = "silu") -> None:
+    """out[:, out_offset(mixer_dim):] = act(gate) * up with (gate, up) at columns glu[0], glu[1] of proj, glu[2] wide (None:
     no feed-forward); columns of `out` between and after the two parts become zero."""
     o0 = out_offset(mixer_dim)
     go, uo, ff = glu if glu is not None else (0, 0, 0)
@@ -215,9 +247,10 @@ def join_glu(proj: torch.Tensor, out: torch.Tensor, mixer_dim: int, glu: Optiona
         out[:, mixer_dim:] = 0
         if ff:
             gate, up = proj[:, go:go + ff].to(F32), proj[:, uo:uo + ff].to(F32)
-            out[:, o0:o0 + ff] = (torch.nn.functional.silu(gate) * up).to(out.dtype)
+            gate = torch.relu(gate) if act == "relu" else torch.nn.functional.silu(gate)
+            out[:, o0:o0 + ff] = (gate * up).to(out.dtype)
         return
     if out.shape[1] == mixer_dim:
         return
     _lib.call("stk_join_glu", proj, proj.stride(0), go, uo, ff, out, out.stride(0), _is32(proj), mixer_dim, o0, out.shape[1],
-              proj.shape[0], _lib.stream())
+              1 if act == "relu" else 0, proj.shape[0], _lib.stream())

@@ -9,7 +9,7 @@ import torch
 from . import _lib
 from . import reference as R
 from .scratch import scratch
-from .functional import cpu_act_dtype
+from .functional import SCORING, cpu_act_dtype
 
 BF16 = torch.bfloat16
 F32 = torch.float32
@@ -82,7 +82,7 @@ def router(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scori
     w = torch.empty(t, top_k, dtype=F32, device=logits.device)
     vocab = tid2eid.shape[0] if tid2eid is not None else 0
     _lib.call("stk_router", logits, logits.stride(0), bias, tid2eid, token_ids, vocab, ids, w, t, e, top_k,
-              0 if scoring == "sigmoid" else 1, 1 if renorm else 0, float(scaling), _lib.status_buffer(), _lib.stream())
+              SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(), _lib.stream())
     return ids, w
 
 
@@ -146,3 +146,39 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, ew: E
     out = torch.empty(t, h, dtype=BF16, device=dev)
     _lib.call("stk_moe_combine", y, weights, pair_row, shared, out, t, h, k, None, st)
     return out
+
+
+# ----------------------------------------------------------------------------
+# experts without a gate, in the compute type
+# ----------------------------------------------------------------------------
+@dataclass
+class PlainExperts:
+    """y = W_down relu(W_up x)^2 per expert: up [E, F, K], down [E, W, F], bf16 or fp32, K and F padded to whole 16-byte units."""
+    up: torch.Tensor
+    down: torch.Tensor
+
+    @property
+    def num(self) -> int:
+        return self.up.shape[0]
+
+
+@dataclass
+class ExpertRows:
+    """Outputs of every (token, chosen expert) pair and where they lie: row pair_row[p] of y, or row p when pair_row is None."""
+    y: torch.Tensor
+    pair_row: Optional[torch.Tensor]
+    weights: torch.Tensor                  # [T, k] fp32
+
+
+def plain_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, ex: PlainExperts) -> ExpertRows:
+    """x [T, K] through its chosen experts ids [T, k]; the weighted sum is left to the consumer."""
+    t, k = ids.shape
+    n_pairs, (e_n, inter, width), out_w = t * k, ex.up.shape, ex.down.shape[1]
+    if not x.is_cuda:
+        return ExpertRows(R.plain_experts(x, ids, ex.up, ex.down, x.dtype), None, weights)
+    st, f32 = _lib.stream(), 1 if x.dtype == F32 else 0
+    act = torch.empty(n_pairs, inter, dtype=x.dtype, device=x.device)
+    y = torch.empty(n_pairs, out_w, dtype=x.dtype, device=x.device)
+    _lib.call("stk_expert_rows", x, x.stride(0), k, ex.up, ids, e_n, act, inter, inter, inter, width, 1, f32, n_pairs, st)
+    _lib.call("stk_expert_rows", act, inter, 1, ex.down, ids, e_n, y, out_w, out_w, out_w, inter, 0, f32, n_pairs, st)
+    return ExpertRows(y, None, weights)

@@ -413,14 +413,21 @@ def router_scores(logits: torch.Tensor, scoring: str) -> torch.Tensor:
         return torch.sigmoid(lf)
     if scoring == "sqrtsoftplus":
         return torch.sqrt(torch.nn.functional.softplus(lf))
+    if scoring == "softmax_topk":
+        return lf
     raise ValueError(scoring)
 
 
 def route(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str, renorm: bool,
           scaling: float, hash_ids: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """-> (expert ids [T, k] int32, weights [T, k] fp32).  Selection uses score+bias,
-    weights use the unbiased score.  hash_ids [T, k] (already looked up) overrides selection."""
+    weights use the unbiased score (except "softmax_topk").  hash_ids [T, k] (already looked up) overrides selection."""
     scores = router_scores(logits, scoring)
+    if scoring == "softmax_topk":
+        # the bias belongs to the logits: the softmax over the chosen ones sees it too
+        z = scores + bias.to(F32)[None] if bias is not None else scores
+        ids = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :top_k]
+        return ids.to(torch.int32), torch.softmax(torch.gather(z, 1, ids), -1) * scaling
     if hash_ids is not None:
         ids = hash_ids.long()
     else:
@@ -667,3 +674,61 @@ def head_norm_gate(o: torch.Tensor, w: torch.Tensor, g: torch.Tensor, eps: float
     """o [T, H, V] fp32: every head divided by its root mean square, times w [H*V] and sigmoid(g [T, H*V])."""
     y = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps)
     return y.flatten(1) * w.to(F32) * torch.sigmoid(g.to(F32))
+
+
+# ----------------------------------------------------------------------------
+# latent attention over paged latents, ungated experts, post-norm residual
+# ----------------------------------------------------------------------------
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
+    """x [T, ..., R]: neighbours (2i, 2i + 1) rotated by position * (freq[0, i] + freq[1, i]), fp32 result."""
+    if x.shape[-1] == 0:
+        return x.to(F32)
+    a = positions.to(torch.float64)[:, None] * (freq[0].double() + freq[1].double())[None]
+    return apply_rope_interleaved(x, torch.cos(a).to(F32), torch.sin(a).to(F32))
+
+
+def latent_insert(c: torch.Tensor, k: torch.Tensor, rot_off: int, positions, tok_req, table, cache) -> None:
+    """c [T, C], k [T, R] (rotated) -> rows of cache [pages, PAGE, row]: latent, zeros, key part, zeros."""
+    page_rows = cache.shape[1]
+    for t in range(c.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        pg = int(table[r, p // page_rows])
+        if pg < 0:
+            continue
+        dst = cache[pg, p % page_rows]
+        dst.zero_()
+        dst[:c.shape[1]] = c[t].to(cache.dtype)
+        dst[rot_off:rot_off + k.shape[1]] = k[t].to(cache.dtype)
+
+
+def latent_attention(qa: torch.Tensor, qr: torch.Tensor, rot_off: int, positions, tok_req, table, cache, freq,
+                     scale: float) -> torch.Tensor:
+    """qa [T, H, C] queries in latent space, qr [T, H, R] before rotation -> softmax-weighted latents [T, H, C] fp32."""
+    t_n, h, c = qa.shape
+    page_rows = cache.shape[1]
+    qr = rotate_pairs(qr, positions, freq).to(qa.dtype).to(F32)
+    out = torch.zeros(t_n, h, c, dtype=F32)
+    for t in range(t_n):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        at = torch.arange(0, p + 1)
+        rows = cache[table[r, at // page_rows].long(), at % page_rows].to(F32)
+        s = qa[t].to(F32) @ rows[:, :c].t() + qr[t] @ rows[:, rot_off:rot_off + qr.shape[-1]].t()
+        out[t] = torch.softmax(s * scale, -1) @ rows[:, :c]
+    return out
+
+
+def plain_experts(x: torch.Tensor, ids: torch.Tensor, up: torch.Tensor, down: torch.Tensor, act_dtype) -> torch.Tensor:
+    """x [T, K] through expert ids [T, k] of up [E, F, K], down [E, W, F]: relu squared between them -> pair rows [T * k, W]."""
+    t, k = ids.shape
+    out = torch.zeros(t * k, down.shape[1], dtype=act_dtype)
+    flat = ids.reshape(-1).long()
+    xp = x.to(F32).repeat_interleave(k, 0)
+    for e in flat.unique().tolist():
+        at = (flat == e).nonzero().flatten()
+        z = torch.relu(xp[at] @ up[e].to(F32).t())
+        out[at] = ((z * z).to(act_dtype).to(F32) @ down[e].to(F32).t()).to(act_dtype)
+    return out

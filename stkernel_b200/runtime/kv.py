@@ -25,8 +25,9 @@ from typing import Callable, Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import HybridConfig, ModelConfig
+from ..config import FULL_CONTEXT, HybridConfig, ModelConfig
 from ..ops.cache import PAGE, PagedCache
+from ..ops.latent import latent_row
 from .planning import dcp_owner
 
 
@@ -349,12 +350,17 @@ class HybridKVManager(CacheManager):
       A page holds `[kv_heads, PAGE, row]`; a row is the projected key followed by the rotated copy of its first
       `rot_dims` dimensions, padded to 16 bytes.  The projected key is the value, and with its rotated head replaced it is
       the key, so nothing is stored twice.  Pages are released as they leave the window.
+    * latent-attention layers: paged rows of one latent and one rotated key part (`ops/latent.py`), in the page group of the
+      full context, whose pages stay until the request ends.  A layer that attends over another layer's latents has none.
     * mLSTM layers: per request row the matrix memory `[heads, dim, vdim]`, the normaliser `[heads, dim]` and the running
       maximum `[heads]`, fp32.  Nothing is cleared when a row changes hands: a span that starts at position 0 reads zeros.
+
+    pool_tokens caps the full-context group at this many tokens over all requests together; admission then promises every
+    request the pages of its whole context and makes others wait.
     """
 
     def __init__(self, cfg: HybridConfig, device, max_requests: int, max_model_len: int, max_chunk: int,
-                 extra_pages: int = 0):
+                 extra_pages: int = 0, pool_tokens: Optional[int] = None):
         super().__init__(device, max_requests)
         self.cfg = cfg
         dt = torch.float32 if cfg.dtype == "float32" else torch.bfloat16
@@ -363,7 +369,13 @@ class HybridKVManager(CacheManager):
         self.by_window: Dict[int, GroupTable] = {}
         for w in cfg.windows():
             pages = hybrid_pool_pages(w, max_requests, max_model_len, max_chunk) + extra_pages
-            self.by_window[w] = GroupTable(f"window{w}", pages, max_requests, pages_ctx, self.device, 1.0)
+            name = f"window{w}"
+            if w >= FULL_CONTEXT:
+                name = "full"
+                if pool_tokens is not None:
+                    pages = min(pages, max(-(-pool_tokens // PAGE), pages_ctx))
+            self.by_window[w] = GroupTable(name, pages, max_requests, pages_ctx, self.device, 1.0)
+        self.full = self.by_window.get(FULL_CONTEXT)
         self.kv_cache: Dict[int, torch.Tensor] = {}
         self.state: Dict[int, Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = {}
         for li, l in enumerate(cfg.layers):
@@ -372,6 +384,10 @@ class HybridKVManager(CacheManager):
                 g = self.by_window[m.window]
                 self.kv_cache[li] = torch.zeros(g.num_pages, m.kv_heads, PAGE, kv_row_width(m.dim, m.rot_dims), dtype=dt,
                                                 device=self.device)
+            elif m.kind == "latent_attention":
+                if m.kv_from is None:
+                    self.kv_cache[li] = torch.zeros(self.full.num_pages, PAGE, latent_row(m.kv_rank, m.rot_dim)[0], dtype=dt,
+                                                    device=self.device)
             else:
                 z = lambda *s: torch.zeros(max_requests, m.heads, *s, dtype=torch.float32, device=self.device)
                 self.state[li] = (z(m.dim, m.vdim), z(m.dim), z())
@@ -389,9 +405,27 @@ class HybridKVManager(CacheManager):
             g.release_before(row, lo // PAGE)
             g.ensure(row, lo // PAGE, (end - 1) // PAGE)
 
+    # ---- admission: the full-context group promises whole contexts --------------------------------
+    @staticmethod
+    def full_pages(context: int) -> int:
+        return context // PAGE + 1
+
+    def reserve(self, row: int, context: int) -> None:
+        if self.full is not None:
+            self.reserved[row] = self.full_pages(context)
+
+    def promised(self) -> int:
+        """Full-context pages promised to running requests and not allocated yet."""
+        return sum(max(0, need - self.full.held(row)) for row, need in self.reserved.items())
+
+    def fits(self, context: int) -> bool:
+        return self.full is None or self.full_pages(context) <= self.full.num_pages
+
     def can_admit(self, n_tokens: int, context: int) -> bool:
         n = min(n_tokens, context)
-        return bool(self.free_rows) and all(len(g.free) >= n // PAGE + 2 for g in self.by_window.values())
+        if not self.free_rows or any(len(g.free) < n // PAGE + 2 for w, g in self.by_window.items() if w < FULL_CONTEXT):
+            return False
+        return self.full is None or len(self.full.free) - self.promised() >= self.full_pages(context)
 
     def usage(self) -> float:
         total = sum(g.num_pages for g in self.by_window.values())
@@ -402,6 +436,13 @@ class HybridKVManager(CacheManager):
     def bytes_allocated(self) -> int:
         n = sum(t.numel() * t.element_size() for t in self.kv_cache.values())
         return n + sum(t.numel() * 4 for st in self.state.values() for t in st)
+
+
+def hybrid_bytes_per_context_token(cfg: HybridConfig) -> int:
+    """Bytes of full-context cache that one token of context costs (windows and recurrent states are bounded)."""
+    es = 4 if cfg.dtype == "float32" else 2
+    return sum(latent_row(l.mixer.kv_rank, l.mixer.rot_dim)[0] * es for l in cfg.layers
+               if l.mixer.kind == "latent_attention" and l.mixer.kv_from is None)
 
 
 def kv_row_width(dim: int, rot_dims: int) -> int:

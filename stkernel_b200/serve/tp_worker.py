@@ -118,7 +118,7 @@ def follower_loop(engine: Engine, cpu_group, heartbeat_timeout: float = 120.0) -
 
 
 def build_engine(a, rank: int, world: int, device) -> Tuple[Engine, Any]:
-    from ..models.registry import config_from_json, family_of, load_model_config
+    from ..models.registry import config_from_json, family_of, load_model_config, use_native
     from ..models.sources import RandomSource
     spec_cfg = SpecConfig()
     if a.speculative_config:
@@ -172,8 +172,7 @@ def build_engine(a, rank: int, world: int, device) -> Tuple[Engine, Any]:
         comm = Communicator(group=group, device=device,
                             use_symm=pp == 1 and os.environ.get("STK_ONESHOT_AR", "1") == "1" and device.type == "cuda")
     if device.type == "cuda":
-        from ..ops import _lib
-        _lib.use_family(family_of(mcfg).name, family_of(mcfg).native_sources)
+        use_native(mcfg)
     weights = family_of(mcfg).build_weights(mcfg, src, device, tp_rank, tp, layer_range=layer_range)
     draft = None
     if spec_cfg.method == "dspark":

@@ -30,7 +30,7 @@ def build_engine(model: str, dtype: str, max_tokens: int):
     """The engine as the server builds it, sized for `max_tokens` live tokens."""
     from ..config import ConfigError, EngineConfig, SchedulerConfig
     from ..models.loader import CheckpointSource
-    from ..models.registry import family_of, load_model_config
+    from ..models.registry import family_of, load_model_config, use_native
     import torch
     try:
         cfg = load_model_config(model, dtype)
@@ -42,8 +42,7 @@ def build_engine(model: str, dtype: str, max_tokens: int):
     if not torch.cuda.is_available():
         raise RuntimeError("trace_run needs a CUDA device")
     family = family_of(cfg)
-    from ..ops import _lib
-    _lib.use_family(family.name, family.native_sources)
+    use_native(cfg)
     device = torch.device("cuda:0")
     torch.cuda.set_device(device)
     context = max(64, max_tokens)
