@@ -1,7 +1,11 @@
 // Mixture-of-experts feed-forward with ungated experts, y = W_down relu(W_up x)^2, weights in the compute type (bf16 or fp32).
 //
 //   expert_rows      one CTA per (pair, block of output rows): a warp streams whole weight rows and dots them with the pair's
-//                    activations, fp32 accumulation.  Decode-sized batches, and every batch of a float32 model.
+//                    activations, fp32 accumulation.  A handful of pairs, and every batch of a float32 model.
+//   experts_slim     tcgen05, pairs sorted by expert: 128 weight rows x 16..64 tokens per tile (few tokens per expert: the
+//                    time is that of streaming the weights)
+//   experts_wide     tcgen05, pairs sorted by expert: 256 tokens (two accumulators that share the weight tile; one when the
+//                    expert has no more than 128 left) x 256 weight rows
 // A pair is one (token, chosen expert).  The weighted sum over a token's pairs is formed where it is normed (hybrid_block.cu).
 #define STK_PDL_CLASS 1024
 #include "common.cuh"
@@ -69,6 +73,314 @@ expert_rows_kernel(const A* __restrict__ x, long long ldx, int div, const A* __r
   }
 }
 
+// ---- pairs sorted by expert ----------------------------------------------------------------------
+int make_tmap_2d(CUtensorMap* tm, const void* base, int elem_bytes, long long rows, long long cols, long long ld, int box_rows);
+
+// sorted row q <- activations of token sorted[q] / topk
+__global__ void __launch_bounds__(128)
+expert_gather_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const int* __restrict__ sorted, int topk,
+                     __nv_bfloat16* __restrict__ xs, int K) {
+  pdl_wait();
+  pdl_trigger();
+  const long long q = blockIdx.x;
+  const uint4* src = reinterpret_cast<const uint4*>(x + static_cast<long long>(sorted[q] / topk) * ldx);
+  uint4* dst = reinterpret_cast<uint4*>(xs + q * K);
+  for (int i = threadIdx.x; i < K / 8; i += blockDim.x) dst[i] = src[i];
+}
+
+struct ExpertArgs {
+  const int* offsets;      // [E + 1] first sorted row of every expert
+  int E, N, k_blocks, tiles_n;
+  __nv_bfloat16* out;      // [P, ldo]
+  long long ldo;
+  int square;
+  int* status;
+};
+constexpr int kMaxExperts = 512;
+
+struct alignas(8) ExpertBars {
+  uint64_t full[8], empty[8], tmem_full[2], tmem_empty[2];
+  uint32_t tmem_base;
+};
+
+// first[e]: tiles of the experts before e, for tiles of `rows` tokens (first[E] = all tiles).
+__device__ __forceinline__ void expert_tiles(int* first, const int* offsets, int E, int rows, int tiles_n) {
+  if (threadIdx.x < 32) {
+    int run = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int n = e < E ? (offsets[e + 1] - offsets[e] + rows - 1) / rows * tiles_n : 0;
+      int incl = n;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, incl, o);
+        if (static_cast<int>(threadIdx.x) >= o) incl += v;
+      }
+      if (e < E) first[e] = run + incl - n;
+      run += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (threadIdx.x == 0) first[E] = run;
+  }
+}
+
+__device__ __forceinline__ uint32_t expert_pack(uint32_t a, uint32_t b, int square) {
+  float x = __uint_as_float(a), y = __uint_as_float(b);
+  if (square) {
+    x = x > 0.f ? x * x : 0.f;
+    y = y > 0.f ? y * y : 0.f;
+  }
+  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+template <int BT>
+struct SlimCfg {
+  static constexpr int kStageBytes = 128 * 128 + BT * 128;
+  static constexpr int kStages = 8;
+  static constexpr int kTmemCols = 2 * BT <= 32 ? 32 : 2 * BT <= 64 ? 64 : 128;
+};
+
+template <int BT>
+__global__ void __launch_bounds__(192, 1)
+experts_slim_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const ExpertArgs a) {
+  using Cfg = SlimCfg<BT>;
+  constexpr int kStages = Cfg::kStages;
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ int first[kMaxExperts + 1];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* smem_b = smem + kStages * 128 * 128;
+  ExpertBars* bars = reinterpret_cast<ExpertBars*>(smem_b + kStages * BT * 128);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 64) {
+    for (int s = 0; s < kStages; ++s) {
+      mbar_init(&bars->full[s], 1);
+      mbar_init(&bars->empty[s], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&bars->tmem_full[i], 1);
+      mbar_init(&bars->tmem_empty[i], 4);
+    }
+    fence_barrier_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(&bars->tmem_base, Cfg::kTmemCols);
+    tmem_relinquish();
+  }
+  pdl_wait();
+  pdl_trigger();
+  expert_tiles(first, a.offsets, a.E, BT, a.tiles_n);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = bars->tmem_base;
+  const int units = first[a.E];
+  if (warp == 0) {
+    if (lane == 0) {
+      int seq = 0, e = 0;
+      bool ok = true;
+      for (int u = blockIdx.x; u < units && ok; u += gridDim.x) {
+        while (u >= first[e + 1]) ++e;
+        const int r = u - first[e], tt = r / a.tiles_n, tn = r - tt * a.tiles_n;
+        for (int kb = 0; kb < a.k_blocks; ++kb, ++seq) {
+          const int st = seq % kStages;
+          if (!mbar_wait(&bars->empty[st], ((seq / kStages) & 1) ^ 1, a.status, 940)) { ok = false; break; }
+          mbar_expect_tx(&bars->full[st], Cfg::kStageBytes);
+          tma_load_2d(smem + st * 128 * 128, &tm_w, &bars->full[st], kb * 64, e * a.N + tn * 128);
+          tma_load_2d(smem_b + st * BT * 128, &tm_x, &bars->full[st], kb * 64, a.offsets[e] + tt * BT);
+        }
+      }
+      if (!ok)
+        for (int s = max(0, seq - kStages); s < seq; ++s) mbar_wait(&bars->full[s % kStages], (s / kStages) & 1, nullptr, 0);
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t kIdesc = umma_idesc(1u, 1u, 128, BT);
+      int seq = 0, i = 0;
+      bool ok = true;
+      for (int u = blockIdx.x; u < units && ok; u += gridDim.x, ++i) {
+        if (!mbar_wait(&bars->tmem_empty[i & 1], ((i >> 1) & 1) ^ 1, a.status, 941)) break;
+        tc_fence_after();
+        for (int kb = 0; kb < a.k_blocks; ++kb, ++seq) {
+          const int st = seq % kStages;
+          if (!mbar_wait(&bars->full[st], (seq / kStages) & 1, a.status, 942)) { ok = false; break; }
+          tc_fence_after();
+          const uint64_t ad = umma_desc_sw128(smem_u32(smem + st * 128 * 128));
+          const uint64_t bd = umma_desc_sw128(smem_u32(smem_b + st * BT * 128));
+#pragma unroll
+          for (int k = 0; k < 4; ++k) umma_f16(tmem + (i & 1) * BT, ad + 2 * k, bd + 2 * k, kIdesc, (kb > 0 || k > 0) ? 1u : 0u);
+          umma_commit(&bars->empty[st]);
+        }
+        if (ok) umma_commit(&bars->tmem_full[i & 1]);
+      }
+    }
+  } else {
+    const int q = warp & 3;
+    int i = 0, e = 0;
+    for (int u = blockIdx.x; u < units; u += gridDim.x, ++i) {
+      while (u >= first[e + 1]) ++e;
+      const int r = u - first[e], tt = r / a.tiles_n, tn = r - tt * a.tiles_n;
+      if (!mbar_wait(&bars->tmem_full[i & 1], (i >> 1) & 1, a.status, 943)) break;
+      tc_fence_after();
+      const int n = tn * 128 + q * 32 + lane, valid = min(BT, a.offsets[e + 1] - a.offsets[e] - tt * BT);
+      __nv_bfloat16* o = a.out + (static_cast<long long>(a.offsets[e]) + tt * BT) * a.ldo + n;
+#pragma unroll
+      for (int c = 0; c < BT; c += 16) {
+        uint32_t v[16];
+        tmem_ld_32x16(tmem + (i & 1) * BT + c + (static_cast<uint32_t>(q * 32) << 16), v);
+        tmem_ld_wait();
+        if (n < a.N) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c + j < valid) {
+              float f = __uint_as_float(v[j]);
+              if (a.square) f = f > 0.f ? f * f : 0.f;
+              o[(c + j) * a.ldo] = __float2bfloat16(f);
+            }
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->tmem_empty[i & 1]);
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::kTmemCols);
+  }
+}
+
+constexpr int kXwStages = 3, kXwStageBytes = 2 * 128 * 128 + 256 * 128;
+
+__global__ void __launch_bounds__(320, 1)
+experts_wide_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const ExpertArgs a) {
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ int first[kMaxExperts + 1];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  ExpertBars* bars = reinterpret_cast<ExpertBars*>(smem + kXwStages * kXwStageBytes);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 64) {
+    for (int s = 0; s < kXwStages; ++s) {
+      mbar_init(&bars->full[s], 1);
+      mbar_init(&bars->empty[s], 1);
+    }
+    mbar_init(&bars->tmem_full[0], 1);
+    mbar_init(&bars->tmem_empty[0], 8);
+    fence_barrier_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(&bars->tmem_base, 512);
+    tmem_relinquish();
+  }
+  pdl_wait();
+  pdl_trigger();
+  expert_tiles(first, a.offsets, a.E, 256, a.tiles_n);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = bars->tmem_base;
+  const int units = first[a.E];
+  if (warp == 0) {
+    if (lane == 0) {
+      int seq = 0, e = 0;
+      bool ok = true;
+      for (int u = blockIdx.x; u < units && ok; u += gridDim.x) {
+        while (u >= first[e + 1]) ++e;
+        const int r = u - first[e], tt = r / a.tiles_n, tn = r - tt * a.tiles_n;
+        const int row = a.offsets[e] + tt * 256;
+        const bool two = a.offsets[e + 1] - row > 128;
+        for (int kb = 0; kb < a.k_blocks; ++kb, ++seq) {
+          const int st = seq % kXwStages;
+          if (!mbar_wait(&bars->empty[st], ((seq / kXwStages) & 1) ^ 1, a.status, 950)) { ok = false; break; }
+          mbar_expect_tx(&bars->full[st], kXwStageBytes - (two ? 0 : 128 * 128));
+          uint8_t* s = smem + st * kXwStageBytes;
+          tma_load_2d(s, &tm_x, &bars->full[st], kb * 64, row);
+          if (two) tma_load_2d(s + 128 * 128, &tm_x, &bars->full[st], kb * 64, row + 128);
+          tma_load_2d(s + 2 * 128 * 128, &tm_w, &bars->full[st], kb * 64, e * a.N + tn * 256);
+        }
+      }
+      if (!ok)
+        for (int s = max(0, seq - kXwStages); s < seq; ++s) mbar_wait(&bars->full[s % kXwStages], (s / kXwStages) & 1, nullptr, 0);
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t kIdesc = umma_idesc(1u, 1u, 128, 256);
+      int seq = 0, i = 0, e = 0;
+      bool ok = true;
+      for (int u = blockIdx.x; u < units && ok; u += gridDim.x, ++i) {
+        while (u >= first[e + 1]) ++e;
+        const bool two = a.offsets[e + 1] - a.offsets[e] - (u - first[e]) / a.tiles_n * 256 > 128;
+        if (!mbar_wait(&bars->tmem_empty[0], (i & 1) ^ 1, a.status, 951)) break;
+        tc_fence_after();
+        for (int kb = 0; kb < a.k_blocks; ++kb, ++seq) {
+          const int st = seq % kXwStages;
+          if (!mbar_wait(&bars->full[st], (seq / kXwStages) & 1, a.status, 952)) { ok = false; break; }
+          tc_fence_after();
+          const uint8_t* s = smem + st * kXwStageBytes;
+          const uint64_t a0 = umma_desc_sw128(smem_u32(s)), a1 = umma_desc_sw128(smem_u32(s + 128 * 128));
+          const uint64_t bd = umma_desc_sw128(smem_u32(s + 2 * 128 * 128));
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const uint32_t acc = (kb > 0 || k > 0) ? 1u : 0u;
+            umma_f16(tmem, a0 + 2 * k, bd + 2 * k, kIdesc, acc);
+            if (two) umma_f16(tmem + 256, a1 + 2 * k, bd + 2 * k, kIdesc, acc);
+          }
+          umma_commit(&bars->empty[st]);
+        }
+        if (ok) umma_commit(&bars->tmem_full[0]);
+      }
+    }
+  } else {
+    const int q = warp & 3, half = (warp - 2) >> 2;                 // the warp's TMEM lanes, its half of the columns
+    int i = 0, e = 0;
+    for (int u = blockIdx.x; u < units; u += gridDim.x, ++i) {
+      while (u >= first[e + 1]) ++e;
+      const int r = u - first[e], tt = r / a.tiles_n, tn = r - tt * a.tiles_n;
+      if (!mbar_wait(&bars->tmem_full[0], i & 1, a.status, 953)) break;
+      tc_fence_after();
+      const int row0 = a.offsets[e] + tt * 256, left = a.offsets[e + 1] - row0;
+      for (int m = 0; m < (left > 128 ? 2 : 1); ++m) {
+        const int t = m * 128 + q * 32 + lane;
+        __nv_bfloat16* o = a.out + static_cast<long long>(row0 + (t < left ? t : 0)) * a.ldo + tn * 256;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          uint32_t v[32];
+          const int col = half * 128 + c * 32;
+          tmem_ld_32x32(tmem + m * 256 + col + (static_cast<uint32_t>(q * 32) << 16), v);
+          tmem_ld_wait();
+          if (t < left) {
+#pragma unroll
+            for (int j = 0; j < 32; j += 8)
+              if (tn * 256 + col + j < a.N)                          // N is a multiple of 8
+                *reinterpret_cast<uint4*>(o + col + j) =
+                    make_uint4(expert_pack(v[j], v[j + 1], a.square), expert_pack(v[j + 2], v[j + 3], a.square),
+                               expert_pack(v[j + 4], v[j + 5], a.square), expert_pack(v[j + 6], v[j + 7], a.square));
+          }
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->tmem_empty[0]);
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+template <int BT>
+static int launch_slim(const CUtensorMap& tw, const CUtensorMap& tx, const ExpertArgs& a, int grid, cudaStream_t st) {
+  const int smem = SlimCfg<BT>::kStages * SlimCfg<BT>::kStageBytes + 256 + 1024;
+  static_assert(sizeof(ExpertBars) <= 256, "barrier block");
+  if (cudaFuncSetAttribute(experts_slim_kernel<BT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
+  launch_pdl(experts_slim_kernel<BT>, dim3(grid), dim3(192), smem, st, tw, tx, a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 }  // namespace stk
 
 using namespace stk;
@@ -94,4 +406,46 @@ STK_API int stk_expert_rows(const void* x, long long ldx, int div, const void* W
                  (__nv_bfloat16*)out + (long long)p0 * ldo, ldo, N, n_pad, K, square);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+STK_API int stk_expert_gather(const void* x, long long ldx, const int* sorted, int topk, void* xs, int K, int n_pairs, void* stream) {
+  if (n_pairs <= 0) return 0;
+  if (K % 8 || ldx % 8 || topk < 1) return -1;
+  launch_pdl(expert_gather_kernel, dim3(n_pairs), dim3(128), 0, (cudaStream_t)stream, (const __nv_bfloat16*)x, ldx, sorted, topk,
+             (__nv_bfloat16*)xs, K);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// xs [n_pairs, K] sorted by expert, W [E, N, K], out [n_pairs, ldo]; bf16.  The tile follows the average number of pairs an expert has.
+STK_API int stk_experts(const void* xs, int n_pairs, const void* W, const int* offsets, int E, int N, int K, void* out, long long ldo,
+                        int square, int sm_count, int* status, void* stream) {
+  if (n_pairs <= 0) return 0;
+  if (E < 1 || E > kMaxExperts || N % 8 || K % 8 || ldo % 8 || static_cast<long long>(E) * N >= (1ll << 31) ||
+      ((reinterpret_cast<uintptr_t>(xs) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out)) & 15))
+    return -1;
+  const int avg = n_pairs / E;
+  const bool wide = avg > 64 && N >= 128;
+  const int bt = avg <= 8 ? 16 : avg <= 24 ? 32 : 64;
+  CUtensorMap tw, tx;
+  if (make_tmap_2d(&tw, W, 2, static_cast<long long>(E) * N, K, K, wide ? 256 : 128) != 0) return -2;
+  if (make_tmap_2d(&tx, xs, 2, n_pairs, K, K, wide ? 128 : bt) != 0) return -2;
+  ExpertArgs a;
+  a.offsets = offsets; a.E = E; a.N = N; a.k_blocks = (K + 63) / 64; a.tiles_n = wide ? (N + 255) / 256 : (N + 127) / 128;
+  a.out = (__nv_bfloat16*)out; a.ldo = ldo; a.square = square; a.status = status;
+  cudaStream_t st = (cudaStream_t)stream;
+  // no more CTAs than there can be tiles
+  const int rows = wide ? 256 : bt;
+  const long long most = (static_cast<long long>(n_pairs) / rows + (n_pairs < E ? n_pairs : E)) * a.tiles_n;
+  const int grid = most < sm_count ? static_cast<int>(most) : sm_count;
+  if (wide) {
+    const int smem = kXwStages * kXwStageBytes + 256 + 1024;
+    if (cudaFuncSetAttribute(experts_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
+    launch_pdl(experts_wide_kernel, dim3(grid), dim3(320), smem, st, tw, tx, a);
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  }
+  switch (bt) {
+    case 16: return launch_slim<16>(tw, tx, a, grid, st);
+    case 32: return launch_slim<32>(tw, tx, a, grid, st);
+    default: return launch_slim<64>(tw, tx, a, grid, st);
+  }
 }

@@ -29,8 +29,9 @@ class Decoder:
 
     # ---- what a family provides --------------------------------------------------
     def build_meta(self, buf, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False,
-                   spans: Tuple[int, int] = (1, 1)):
-        """Device-side description of the staged step.  spans = (shortest, longest) span, known on the host."""
+                   spans: Tuple = (1, 1)):
+        """Device-side description of the staged step.  spans = (shortest, longest[, all as (start, tokens)]) spans,
+        known on the host."""
         raise NotImplementedError
 
     def decode_bucket(self, max_comp_rows: int) -> int:

@@ -173,10 +173,18 @@ def build_latent(cfg: HybridConfig, get, m, dt, device) -> LA.LatentParams:
         w_uq[H * dp:H * dp + H * R, :Q] = uq[:, D:].reshape(H * R, Q).to(dt)
     w_uk = _spread(get("mix.uk").view(H, D, C).transpose(1, 2).reshape(H * C, D), H, C, cp, dp, dt)
     w_uv = _spread(get("mix.uv"), H, m.vdim, vp, cp, dt)
+    w_ukv = None
+    if dt == BF16 and torch.device(device).type == "cuda" and LA.prompt_ok(m):
+        # prompts expand keys and values from the latent columns of gathered rows
+        v64, cols = (m.vdim + 63) // 64 * 64, LA.latent_row(C, R)[1]
+        both = torch.zeros(H, dp + v64, cols, dtype=dt, device=device)
+        both[:, :D, :C] = get("mix.uk").view(H, D, C).to(dt)
+        both[:, dp:dp + m.vdim, :C] = get("mix.uv").view(H, m.vdim, C).to(dt)
+        w_ukv = LinearWeight(both.view(H * (dp + v64), cols))
     freq = m.rotary.frequencies()[0] if m.rotary is not None else []
     return LA.LatentParams(H, D, R, m.vdim, Q, C, m.scale, cfg.norm_eps, dp, cp, vp, LA.split_frequencies(freq, device),
                            f32("mix.dq.norm"), f32("mix.dkv.norm") if m.kv_from is None else None, LinearWeight(w_uq),
-                           LinearWeight(w_uk), LinearWeight(w_uv))
+                           LinearWeight(w_uk), LinearWeight(w_uv), w_ukv)
 
 
 def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWeights:
@@ -274,10 +282,10 @@ class HybridModel(Decoder):
         self.on_layer = None                # optional hook (layer index, residual [T, W] fp32) after each layer
 
     def build_meta(self, buf, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False,
-                   spans: Tuple[int, int] = (1, 1)) -> HB.HybridMeta:
+                   spans: Tuple = (1, 1)) -> HB.HybridMeta:
         tok_req, positions, first, last = A.token_maps(buf.d_qstart, buf.d_rows, buf.d_start, n_req, t_pad)
         return HB.HybridMeta(buf.d_tokens[:t_pad], tok_req, positions, first, last, buf.d_qstart, buf.d_rows, buf.d_start, n_req,
-                             spans[1], pure_decode, spans[0], 4 * max_comp_rows + 4)
+                             spans[1], pure_decode, spans[0], spans[2] if len(spans) > 2 else None, max_context=4 * max_comp_rows + 4)
 
     def decode_bucket(self, max_comp_rows: int) -> int:
         # full-context attention splits the key range by the longest context a graph serves: one graph per power of two

@@ -104,7 +104,7 @@ def _hybrid_model(cfg: EngineConfig, weights, kv, comm, tp_rank: int):
 
 _HYBRID_SOURCES = ("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", "linear_f32.cu", "hybrid_block.cu", "sampler.cu")
 _MECHANISM_SOURCES = {"attention": ("window_attention.cu", "window_attention_tc.cu"), "mlstm": ("mlstm.cu",), "dense": (),
-                      "latent_attention": ("latent_attention.cu",),
+                      "latent_attention": ("latent_attention.cu", "latent_tokens_tc.cu", "latent_prompt_tc.cu"),
                       "moe": ("moe.cu", "moe_plain.cu", "gate_cluster.cu")}
 
 

@@ -7,7 +7,7 @@ products).  Residual, norms, scores and softmax, gates and recurrent state are f
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Optional, Tuple
 
 import torch
@@ -123,6 +123,8 @@ class HybridMeta:
     max_span: int                  # longest span of the step (host knowledge: which kernels have work)
     pure_decode: bool = False      # every span is one token
     min_span: int = 1
+    spans: Optional[Tuple[Tuple[int, int], ...]] = None      # (start, tokens) of every request, when the host knows them
+    gathered: dict = field(default_factory=dict)             # cached rows that a layer copied out of their pages for this step
     max_context: int = 1 << 30     # no token of the step sees more keys (host knowledge: how far to split the key range)
 
 

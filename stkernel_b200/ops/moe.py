@@ -177,6 +177,21 @@ def plain_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, ex:
     if not x.is_cuda:
         return ExpertRows(R.plain_experts(x, ids, ex.up, ex.down, x.dtype), None, weights)
     st, f32 = _lib.stream(), 1 if x.dtype == F32 else 0
+    if not f32 and n_pairs > DIRECT_MAX_PAIRS:
+        dev = x.device
+        sorted_p = scratch("moe.sorted", (n_pairs,), I32, dev)
+        pair_row = torch.empty(n_pairs, dtype=I32, device=dev)
+        offsets = scratch("moe.offsets", (e_n + 1,), I32, dev)
+        sorted_e = scratch("moe.sorted_e", (n_pairs,), I32, dev)
+        counts = scratch("moe.counts", (((n_pairs + 255) // 256) * e_n,), I32, dev) if n_pairs > 2048 else None
+        _lib.call("stk_moe_align", ids, n_pairs, 0, e_n, sorted_p, pair_row, offsets, sorted_e, counts, st)
+        xs = scratch("moe.plain.xs", (n_pairs, width), BF16, dev)
+        act = scratch("moe.plain.act", (n_pairs, inter), BF16, dev)
+        y = torch.empty(n_pairs, out_w, dtype=BF16, device=dev)
+        _lib.call("stk_expert_gather", x, x.stride(0), sorted_p, k, xs, width, n_pairs, st)
+        for a, w, o, n, kk, square in ((xs, ex.up, act, inter, width, 1), (act, ex.down, y, out_w, inter, 0)):
+            _lib.call("stk_experts", a, n_pairs, w, offsets, e_n, n, kk, o, n, square, _lib.sm_count(), _lib.status_buffer(), st)
+        return ExpertRows(y, pair_row, weights)
     act = torch.empty(n_pairs, inter, dtype=x.dtype, device=x.device)
     y = torch.empty(n_pairs, out_w, dtype=x.dtype, device=x.device)
     _lib.call("stk_expert_rows", x, x.stride(0), k, ex.up, ids, e_n, act, inter, inter, inter, width, 1, f32, n_pairs, st)

@@ -293,7 +293,7 @@ class Engine:
             from ..parallel.eplb import LoadRecorder
             self.model.load_recorder = LoadRecorder(cfg.model.num_hidden_layers, cfg.model.n_routed_experts, self.device)
         self.metrics = Metrics()
-        self._spans = (1, 1)                 # shortest and longest span of the staged step
+        self._spans = (1, 1)                 # shortest and longest span of the staged step, then (start, tokens) of each
         self.async_scheduling = sc.async_scheduling and not spec_on and pipe is None
         self._inflight = None                # asynchronous scheduling: the step that is launched and not read yet
         self._async_parity = 0
@@ -503,7 +503,7 @@ class Engine:
                     trunc = trunc or r.params.truncates
                     ns += 1
         b.n_qstart[len(seqs)] = t
-        self._spans = (min(s.n for s in seqs), max(s.n for s in seqs))
+        self._spans = (min(s.n for s in seqs), max(s.n for s in seqs), tuple((s.start, s.n) for s in seqs))
         self.buf.truncating = trunc
         return t, len(seqs), ns
 
