@@ -11,11 +11,13 @@ This is the engine's equivalent of the reference's eager scratch pool
 from __future__ import annotations
 
 from contextlib import contextmanager
-from typing import Dict, Sequence, Tuple
+from typing import Dict, List, Sequence, Tuple
 
 import torch
 
 _pool: Dict[Tuple[str, str], torch.Tensor] = {}
+# buffers that were outgrown: captured graphs may still hold their addresses
+_outgrown: List[torch.Tensor] = []
 _frozen = False
 _branch = ""
 
@@ -52,6 +54,8 @@ def scratch(name: str, shape: Sequence[int], dtype: torch.dtype, device, zero: b
             raise RuntimeError(f"scratch buffer {name!r} would grow after graphs were captured")
         cap = max(nbytes, 2 * buf.numel() if buf is not None else 0)
         cap = (cap + 255) // 256 * 256
+        if buf is not None:
+            _outgrown.append(buf)
         buf = torch.zeros(cap, dtype=torch.uint8, device=device) if zero else torch.empty(cap, dtype=torch.uint8, device=device)
         _pool[key] = buf
     return buf[:n * torch.empty((), dtype=dtype).element_size()].view(dtype).view(*shape)
@@ -59,7 +63,8 @@ def scratch(name: str, shape: Sequence[int], dtype: torch.dtype, device, zero: b
 
 def reset() -> None:
     _pool.clear()
+    _outgrown.clear()
 
 
 def total_bytes() -> int:
-    return sum(b.numel() for b in _pool.values())
+    return sum(b.numel() for b in list(_pool.values()) + _outgrown)

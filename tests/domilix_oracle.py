@@ -15,7 +15,7 @@ def rms(v, eps):
 def rotate_pairs(vec, position, rot):
     """vec [..., D] at one position: neighbours (2i, 2i + 1) of the first rot.dims values turn by position * base^(-2i/dims)."""
     out = vec.clone()
-    for i in range(rot["dims"] // 2):
+    for i in range(rot["dims"] // 2 if rot else 0):
         a = position * rot["base"] ** (-2.0 * i / rot["dims"])
         c, s = math.cos(a), math.sin(a)
         u, v = vec[..., 2 * i], vec[..., 2 * i + 1]
@@ -29,7 +29,7 @@ def queries(h, w, p, m, eps):
     T, H, D, R = h.shape[0], m["heads"], m["dim"], m["rot_dim"]
     low = rms(h @ w[p + "dq"].T, eps) * w[p + "dq.norm"]
     q = (low @ w[p + "uq"].T).reshape(T, H, D + R)
-    turned = torch.stack([rotate_pairs(q[t, :, D:], t, m["rot"]) for t in range(T)])
+    turned = torch.stack([rotate_pairs(q[t, :, D:], t, m.get("rot")) for t in range(T)])
     return q[:, :, :D], turned
 
 
@@ -38,7 +38,7 @@ def latents(h, w, p, m, eps):
     C = m["kv_rank"]
     z = h @ w[p + "dkv"].T
     c = rms(z[:, :C], eps) * w[p + "dkv.norm"]
-    return c, torch.stack([rotate_pairs(z[t, C:], t, m["rot"]) for t in range(z.shape[0])])
+    return c, torch.stack([rotate_pairs(z[t, C:], t, m.get("rot")) for t in range(z.shape[0])])
 
 
 def softmax_row(s):
