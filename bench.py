@@ -96,6 +96,16 @@ def hybrid_arm(args) -> None:
     print(json.dumps({"metric": "hybrid_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
 
 
+def latent_arm(args) -> None:
+    import torch
+    from stkernel_b200.bench import hybrid_bench, latent_bench
+    torch.cuda.set_device(0)
+    with ClockSampler(0) as clocks:
+        res = latent_bench.run([int(x) for x in args.latent_sizes.split(",")], beside=not args.latent_alone)
+    print(hybrid_bench.render(res), file=sys.stderr)
+    print(json.dumps({"metric": "latent_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -112,9 +122,16 @@ def main() -> None:
                     help="instead of the flagship: the Timalorn decoder beside the flagship's architecture at equal width "
                          "and depth, prefill, decode and per-kernel rooflines (one JSON line; table on stderr)")
     ap.add_argument("--hybrid-sizes", default="2048,4096", help="widths for --hybrid")
+    ap.add_argument("--latent", action="store_true",
+                    help="instead of the flagship: the Domilix decoder beside the flagship's architecture at equal width, depth "
+                         "and expert counts, prefill, decode and per-kernel rooflines (one JSON line; table on stderr)")
+    ap.add_argument("--latent-sizes", default="2048,4096", help="widths for --latent")
+    ap.add_argument("--latent-alone", action="store_true", help="with --latent: without the flagship's architecture beside it")
     args = ap.parse_args()
     if args.hybrid:
         return hybrid_arm(args)
+    if args.latent:
+        return latent_arm(args)
     if args.impl == "reference":
         return reference_arm(args)
 
