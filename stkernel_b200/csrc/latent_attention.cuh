@@ -41,6 +41,60 @@ __device__ __forceinline__ void lat_st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void lat_st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ float lat_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
+
+// ---- issue of tensor-core products by a converged warp -----------------------------------------------
+// The whole warp runs the issuing code with warp-uniform operands (descriptors are their low words; the high word is the same for
+// every 128-byte-swizzled operand here) and one elected lane executes the instruction: a few instructions per product, which
+// small products need to keep the tensor pipe busy.
+constexpr uint32_t kDescHi = (1024u >> 4) | (1u << 14) | (2u << 29);      // 8-row groups 1024 bytes apart, version, 128-byte swizzle
+__device__ __forceinline__ uint32_t desc_lo(uint32_t smem_addr, uint32_t lbo_bytes = 16) {
+  return ((smem_addr & 0x3FFFF) >> 4) | ((lbo_bytes >> 4) << 16);
+}
+// D[tmem] (+)= A[smem] * B[smem]
+__device__ __forceinline__ void mma_ss(uint32_t d, uint32_t a_lo, uint32_t b_lo, uint32_t idesc, uint32_t acc, uint32_t lead) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t.reg .b64 a, b;\n\t"
+      "setp.ne.b32 p, %5, 0;\n\tsetp.ne.b32 q, %6, 0;\n\t"
+      "mov.b64 a, {%1, %3};\n\tmov.b64 b, {%2, %3};\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %4, p;\n\t}"
+      ::"r"(d), "r"(a_lo), "r"(b_lo), "r"(kDescHi), "r"(idesc), "r"(acc), "r"(lead)
+      : "memory");
+}
+// D[tmem] (+)= A[tmem] * B[smem]
+__device__ __forceinline__ void mma_ts(uint32_t d, uint32_t a_tmem, uint32_t b_lo, uint32_t idesc, uint32_t acc, uint32_t lead) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t.reg .b64 b;\n\t"
+      "setp.ne.b32 p, %5, 0;\n\tsetp.ne.b32 q, %6, 0;\n\t"
+      "mov.b64 b, {%2, %3};\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], b, %4, p;\n\t}"
+      ::"r"(d), "r"(a_tmem), "r"(b_lo), "r"(kDescHi), "r"(idesc), "r"(acc), "r"(lead)
+      : "memory");
+}
+__device__ __forceinline__ void mma_commit(uint64_t* bar, uint32_t lead) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+      ::"r"(smem_u32(bar)), "r"(lead) : "memory");
+}
+
+// packed pairs of fp32
+__device__ __forceinline__ uint64_t pack2(float x, float y) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 }  // namespace stk
 
 static inline stk::LatArgs lat_args(const void* qa, long long ldqa, int cp, const void* qr, long long ldqr, const float* gate,

@@ -47,15 +47,6 @@ struct LpArgs {
   int* status;
 };
 
-// D[tmem] (+)= A[tmem] * B[smem desc]
-__device__ __forceinline__ void umma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
 __device__ __forceinline__ void lp_st16(uint32_t taddr, const uint32_t (&r)[16]) {
   asm volatile(
       "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
@@ -70,17 +61,6 @@ __device__ __forceinline__ float lp_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// MN-major operand of one 64-column panel, 128-byte swizzle: 8-row groups 1024 bytes apart along K.
-__device__ __forceinline__ uint64_t lp_desc_mn(uint32_t smem_addr) {
-  uint64_t d = 0;
-  d |= static_cast<uint64_t>((smem_addr & 0x3FFFF) >> 4);
-  d |= static_cast<uint64_t>(kLpPanel >> 4) << 16;
-  d |= static_cast<uint64_t>(1024 >> 4) << 32;
-  d |= static_cast<uint64_t>(1) << 46;
-  d |= static_cast<uint64_t>(2) << 61;
-  return d;
-}
-
 // One CTA per 128 rows of the gathered matrix.
 __global__ void __launch_bounds__(256)
 latent_rows_kernel(const int* __restrict__ query_start, const int* __restrict__ req_rows, const int* __restrict__ start_pos, int n_req,
@@ -233,69 +213,88 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     __syncwarp();
   } else if (warp == 9) {
     // ------------------------------- MMA issuer -------------------------------
-    if (lane == 0) {
-      const uint32_t idesc_qk = umma_idesc(1u, 1u, 128, 128);
-      const uint32_t idesc_pv = umma_idesc(1u, 1u, 128, 64) | (1u << 16);         // B is MN-major
-      const int r_steps = (a.R + 15) / 16;
-      bool ok = mbar_wait(&bars->q_full, 0, a.status, 810);
-      int k_seen = 0, v_seen = 0;                                  // blocks whose key / value panels have been waited for
-      auto wait_panels = [&](int b, int j0, int n, int& seen) {
-        if (seen > b) return true;
-        for (int j = 0; j < n; ++j) {
-          const int seq = b * per + j0 + j;
-          if (!mbar_wait(&bars->full[seq % a.slots], (seq / a.slots) & 1, a.status, 811)) return false;
-        }
-        tc_fence_after();
-        seen = b + 1;
-        return true;
-      };
-      auto scores = [&](int i, int b) {
-        if (!wait_panels(b, 0, kp, k_seen)) return false;
-        uint32_t acc = 0;
-        for (int j = 0; j < kp; ++j) {
-          const uint64_t ad = umma_desc_sw128(smem_u32(q_s + (i * kp + j) * kLpPanel));
-          const uint64_t bd = umma_desc_sw128(smem_u32(ring + ((b * per + j) % a.slots) * kLpPanel));
-          const int steps = j < a.d_panels ? min(4, a.d_steps - j * 4) : min(4, r_steps - (j - a.d_panels) * 4);
-          for (int ks = 0; ks < steps; ++ks) {
-            umma_f16(tmem + i * 128, ad + 2 * ks, bd + 2 * ks, idesc_qk, acc);
-            acc = 1;
-          }
-        }
-        umma_commit(&bars->s_full[i]);
-        return true;
-      };
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-        if (ok && nb[i] > 0) ok = scores(i, 0);
-      if (ok)
-        for (int j = 0; j < kp; ++j) umma_commit(&bars->empty[j % a.slots]);
-      for (int b = 0; b < nb_max && ok; ++b) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          if (!ok || b >= nb[i]) continue;
-          ok = mbar_wait(&bars->p_full[i], b & 1, a.status, 812);
-          if (!ok) continue;
+    const uint32_t lead = elect_one() ? 1u : 0u, tm = __shfl_sync(0xffffffffu, tmem, 0);
+    constexpr uint32_t kIdescS = umma_idesc(1u, 1u, 128, 128);
+    constexpr uint32_t kIdescO1 = umma_idesc(1u, 1u, 128, 64) | (1u << 16), kIdescO2 = umma_idesc(1u, 1u, 128, 128) | (1u << 16);
+    constexpr uint32_t kStep = kLpPanel >> 4;                      // a panel in descriptor units
+    const uint32_t q_lo = desc_lo(smem_u32(q_s)), k_lo = desc_lo(smem_u32(ring)), v_lo = desc_lo(smem_u32(ring), kLpPanel);
+    bool ok = mbar_wait(&bars->q_full, 0, a.status, 810);
+    struct At { int slot; uint32_t par; };
+    auto ahead = [&](At c, int n) {
+      c.slot += n;
+      if (c.slot >= a.slots) { c.slot -= a.slots; c.par ^= 1u; }
+      return c;
+    };
+    At cur{0, 0u};                                                 // first panel of block b
+    auto scores = [&](int i, At c, bool wait) {
+      for (int j = 0; j < kp; ++j) {
+        const At p = ahead(c, j);
+        if (wait) {
+          if (!mbar_wait(&bars->full[p.slot], p.par, a.status, 811)) return false;
           tc_fence_after();
-          ok = wait_panels(b, kp, a.v_panels, v_seen);
-          if (!ok) continue;
+        }
+        const uint32_t al = q_lo + (i * kp + j) * kStep, bl = k_lo + p.slot * kStep;
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) mma_ss(tm + i * 128, al + 2 * ks, bl + 2 * ks, kIdescS, ks > 0 ? 1u : (j > 0 ? 1u : 0u), lead);
+      }
+      mma_commit(&bars->s_full[i], lead);
+      return true;
+    };
+    if (ok) ok = scores(0, cur, true);
+    if (ok && nb[1] > 0) ok = scores(1, cur, false);
+    if (ok)
+      for (int j = 0; j < kp; ++j) mma_commit(&bars->empty[j], lead);
+    for (int b = 0; b < nb_max && ok; ++b) {
+      const At next = ahead(cur, per), v0 = ahead(cur, kp);
+      bool v_seen = false, k_seen = false;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        if (!ok || b >= nb[i]) continue;
+        ok = mbar_wait(&bars->p_full[i], b & 1, a.status, 812);
+        tc_fence_after();
+        if (ok && !v_seen) {
+          for (int j = 0; j < a.v_panels && ok; ++j) {
+            const At p = ahead(v0, j);
+            ok = mbar_wait(&bars->full[p.slot], p.par, a.status, 813);
+          }
+          tc_fence_after();
+          v_seen = true;
+        }
+        if (!ok) continue;
+        const uint32_t first_acc = b > 0 ? 1u : 0u;
+        if (a.v_panels == 2 && v0.slot + 1 < a.slots) {
+          // both value panels side by side: one product of 128 columns
+          const uint32_t bl = v_lo + v0.slot * kStep;
+#pragma unroll
+          for (int part = 0; part < 2; ++part)
+#pragma unroll
+            for (int kk = 0; kk < 8; ++kk)
+              mma_ts(tm + 256 + i * 128, tm + i * 128 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, bl + kk * 128, kIdescO2,
+                     part + kk > 0 ? 1u : first_acc, lead);
+        } else {
           for (int vj = 0; vj < a.v_panels; ++vj) {
-            const uint8_t* v = ring + ((b * per + kp + vj) % a.slots) * kLpPanel;
+            const uint32_t bl = v_lo + ahead(v0, vj).slot * kStep;
 #pragma unroll
             for (int part = 0; part < 2; ++part)
 #pragma unroll
               for (int kk = 0; kk < 8; ++kk)
-                umma_f16_ts(tmem + 256 + i * 128 + vj * 64, tmem + i * 128 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8,
-                            lp_desc_mn(smem_u32(v + kk * 2048)), idesc_pv, (b > 0 || part > 0 || kk > 0) ? 1u : 0u);
+                mma_ts(tm + 256 + i * 128 + vj * 64, tm + i * 128 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, bl + kk * 128,
+                       kIdescO1, part + kk > 0 ? 1u : first_acc, lead);
           }
-          if (b + 1 == nb[i]) umma_commit(&bars->o_full[i]);
-          else ok = scores(i, b + 1);
         }
-        if (ok) {
-          for (int j = 0; j < a.v_panels; ++j) umma_commit(&bars->empty[(b * per + kp + j) % a.slots]);
-          if (b + 1 < nb_max)
-            for (int j = 0; j < kp; ++j) umma_commit(&bars->empty[((b + 1) * per + j) % a.slots]);
+        if (b + 1 == nb[i]) {
+          mma_commit(&bars->o_full[i], lead);
+        } else {
+          ok = scores(i, next, !k_seen);
+          k_seen = true;
         }
       }
+      if (ok) {
+        for (int j = 0; j < a.v_panels; ++j) mma_commit(&bars->empty[ahead(v0, j).slot], lead);
+        if (b + 1 < nb_max)
+          for (int j = 0; j < kp; ++j) mma_commit(&bars->empty[ahead(next, j).slot], lead);
+      }
+      cur = next;
     }
     __syncwarp();
   } else {
@@ -305,31 +304,40 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const uint32_t ts = tmem + tile * 128 + lanes, to = tmem + 256 + tile * 128 + lanes;
     const int t_first = tile ? first[1] : first[0], t_blocks = tile ? nb[1] : nb[0], t_tok = tile ? n_tok[1] : n_tok[0];
     const float c_in = a.scale * kLpLog2e;
+    const bool flip = c_in < 0.f;                                  // a negative scale: the largest score is the smallest product
+    const uint32_t masked = __float_as_uint(flip ? INFINITY : -INFINITY);
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int b = 0; b < t_blocks && ok; ++b) {
       ok = mbar_wait(&bars->s_full[tile], b & 1, a.status, 820);
       if (!ok) break;
       tc_fence_after();
-      const int d0 = t_first + r - b * kLpTile;                // keys 0 .. d0 of the block are visible
+      const int d0 = t_first + r - b * kLpTile;                    // keys 0 .. d0 of the block are visible
       const bool edge = b * kLpTile + kLpTile - 1 > t_first;
-      float mx = -INFINITY;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t s[32];
-        tmem_ld_32x32(ts + c * 32, s);
+      uint32_t s[2][32];                                           // 64 scores of the row at a time
+      auto fetch = [&](int half) {
+        tmem_ld_32x32(ts + half * 64, s[0]);
+        tmem_ld_32x32(ts + half * 64 + 32, s[1]);
         tmem_ld_wait();
-        float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
         if (edge) {
 #pragma unroll
-          for (int j = 0; j < 32; ++j)
-            m4[j & 3] = fmaxf(m4[j & 3], c * 32 + j <= d0 ? __uint_as_float(s[j]) * c_in : -INFINITY);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 32; ++j) m4[j & 3] = fmaxf(m4[j & 3], __uint_as_float(s[j]) * c_in);
+          for (int j = 0; j < 64; ++j)
+            if (half * 64 + j > d0) s[j >> 5][j & 31] = masked;
         }
-        mx = fmaxf(mx, fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])));
-      }
+      };
+      auto largest = [&]() {
+        float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+        for (int j = 0; j < 64; ++j) {
+          const float v = __uint_as_float(s[j >> 5][j & 31]);
+          m4[j & 3] = fmaxf(m4[j & 3], flip ? -v : v);
+        }
+        return fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+      };
+      fetch(0);
+      float mx = largest();
+      fetch(1);
+      mx = fmaxf(mx, largest()) * fabsf(c_in);
       const bool grow = mx > m + 8.f || (m == -INFINITY && mx > -INFINITY);
       if (__any_sync(0xffffffffu, grow)) {
         const float f = grow ? (m == -INFINITY ? 0.f : lp_ex2(m - mx)) : 1.f;
@@ -349,29 +357,37 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         }
       }
       const float ms = m == -INFINITY ? 0.f : m;
-      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+      const uint64_t c2 = pack2(c_in, c_in), m2 = pack2(-ms, -ms), minus = pack2(-1.f, -1.f);
+      uint64_t sum2[2] = {0ull, 0ull};
+      auto weigh = [&](int half) {
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t s[32], hi[16], lo[16];
-        tmem_ld_32x32(ts + c * 32, s);
-        tmem_ld_wait();
+        for (int c = 0; c < 2; ++c) {
+          uint32_t hi[16], lo[16];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          float p0 = lp_ex2(fmaf(__uint_as_float(s[2 * j]), c_in, -ms)), p1 = lp_ex2(fmaf(__uint_as_float(s[2 * j + 1]), c_in, -ms));
-          if (edge) {
-            p0 = c * 32 + 2 * j <= d0 ? p0 : 0.f;
-            p1 = c * 32 + 2 * j + 1 <= d0 ? p1 : 0.f;
+          for (int j = 0; j < 16; ++j) {
+            float p0, p1;
+            unpack2(fma2(pack2(__uint_as_float(s[c][2 * j]), __uint_as_float(s[c][2 * j + 1])), c2, m2), p0, p1);
+            p0 = lp_ex2(p0);
+            p1 = lp_ex2(p1);
+            const uint64_t p2 = pack2(p0, p1);
+            sum2[j & 1] = add2(sum2[j & 1], p2);
+            const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
+            hi[j] = *reinterpret_cast<const uint32_t*>(&hb);
+            float r0, r1;
+            unpack2(fma2(pack2(__uint_as_float(hi[j] << 16), __uint_as_float(hi[j] & 0xffff0000u)), minus, p2), r0, r1);
+            const __nv_bfloat162 lb = __floats2bfloat162_rn(r0, r1);
+            lo[j] = *reinterpret_cast<const uint32_t*>(&lb);
           }
-          ls[j & 3] += p0 + p1;
-          const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
-          const float2 hf = __bfloat1622float2(hb);
-          const __nv_bfloat162 lb = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
-          hi[j] = *reinterpret_cast<const uint32_t*>(&hb);
-          lo[j] = *reinterpret_cast<const uint32_t*>(&lb);
+          lp_st16(ts + (half * 2 + c) * 32, hi);
+          lp_st16(ts + (half * 2 + c) * 32 + 16, lo);
         }
-        lp_st16(ts + c * 32, hi);
-        lp_st16(ts + c * 32 + 16, lo);
-      }
+      };
+      weigh(1);
+      fetch(0);
+      weigh(0);
+      float ls[4];
+      unpack2(sum2[0], ls[0], ls[1]);
+      unpack2(sum2[1], ls[2], ls[3]);
       l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
       lp_st_wait();
       tc_fence_before();

@@ -7,7 +7,7 @@
 //                    panel (the rotated part) has two buffers of its own
 //   MMA warp         S^T[key, column] = rows . Q^T as the panels arrive; O^T[dim, column] += rows^T . P with the same panels as
 //                    MN-major operand, 128 dims at a time, giving each pair of panels back as soon as its dims are done
-//   softmax warps    one key per thread: column maxima over the lanes, probabilities to shared memory as bf16 pairs (high parts
+//   softmax warps    eight, one key and half of the columns per thread: column maxima over the lanes, probabilities to shared memory as bf16 pairs (high parts
 //                    and remainders are 2N columns of one product), O rescaled only when a column's maximum grew by more than 2^8
 //
 // Each CTA writes an unnormalised partial result; latent_merge joins the splits and applies the output gate.  Rows behind the last
@@ -21,7 +21,7 @@ namespace stk {
 
 int make_tmap_2d(CUtensorMap* tm, const void* base, int elem_bytes, long long rows, long long cols, long long ld, int box_rows);
 
-constexpr int kLtBlock = 128, kLtPanel = kLtBlock * 128, kLtThreads = 192, kLtMaxPairs = 6;
+constexpr int kLtBlock = 128, kLtPanel = kLtBlock * 128, kLtThreads = 320, kLtMaxPairs = 6;
 constexpr float kLtLog2e = 1.4426950408889634f;
 
 struct LtArgs {
@@ -29,7 +29,7 @@ struct LtArgs {
   const int* query_start; const int* req_rows; const int* start_pos;
   int n_req, max_span;
   int tq, hs;                            // tokens per tile, heads per group (tq * hs <= N)
-  int pairs, tail, slots, v_tiles, steps;   // panel pairs of a row, whether an odd panel follows, ring size, 128-dim tiles, 16-column steps
+  int pairs, tail, slots, v_tiles;       // panel pairs of a row, whether an odd panel follows, ring size, 128-dim tiles
   float* part;                           // [splits][T][H][C + 2]
   int T;
   int* status;
@@ -53,12 +53,12 @@ __device__ __forceinline__ bool lt_bar_all(bool ok) {
   asm volatile(
       "{\n\t.reg .pred p, q;\n\t"
       "setp.ne.s32 p, %1, 0;\n\t"
-      "barrier.cta.red.and.pred q, 1, 128, p;\n\t"
+      "barrier.cta.red.and.pred q, 1, 256, p;\n\t"
       "selp.s32 %0, 1, 0, q;\n\t}"
       : "=r"(r) : "r"(ok ? 1 : 0) : "memory");
   return r != 0;
 }
-__device__ __forceinline__ void lt_bar_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void lt_bar_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 __device__ __forceinline__ void lt_st16(uint32_t taddr, const uint32_t (&r)[16]) {
   asm volatile(
       "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
@@ -67,15 +67,19 @@ __device__ __forceinline__ void lt_st16(uint32_t taddr, const uint32_t (&r)[16])
       "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
       : "memory");
 }
-// MN-major operand of panel pairs, 128-byte swizzle: the two 64-column panels are one panel apart, 8-row groups 1024 bytes.
-__device__ __forceinline__ uint64_t lt_desc_mn(uint32_t smem_addr) {
-  uint64_t d = 0;
-  d |= static_cast<uint64_t>((smem_addr & 0x3FFFF) >> 4);
-  d |= static_cast<uint64_t>(kLtPanel >> 4) << 16;
-  d |= static_cast<uint64_t>(1024 >> 4) << 32;
-  d |= static_cast<uint64_t>(1) << 46;
-  d |= static_cast<uint64_t>(2) << 61;
-  return d;
+// 8 or 16 columns of the warp's 32 lanes
+template <int C>
+__device__ __forceinline__ void lt_ld(uint32_t taddr, uint32_t (&r)[C]) {
+  if constexpr (C == 16) {
+    tmem_ld_32x16(taddr, r);
+  } else {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+                 : "r"(taddr));
+  }
+}
+__device__ __forceinline__ void lt_cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
 template <int N>
@@ -95,7 +99,8 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
   float* m_ref = smax + 4 * N;                                      // [N]
   float* alpha = m_ref + N;                                         // [N]
   int* col_pos = reinterpret_cast<int*>(alpha + N);                 // [N] last key a column sees (-1: padding)
-  int* flags = col_pos + N;
+  int* col_row = col_pos + N;                                       // [N] token * heads + head of a column
+  int* flags = col_row + N;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   pdl_trigger();
@@ -128,7 +133,7 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
       bars->find[0] = ri;
       bars->find[1] = off * x.tq;
     }
-  } else if (threadIdx.x == 128) {
+  } else if (threadIdx.x == 288) {
     for (int s = 0; s < kLtMaxPairs; ++s) {
       mbar_init(&bars->full[s], 1);
       mbar_init(&bars->empty[s], 1);
@@ -138,7 +143,7 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
       mbar_init(&bars->tail_empty[i], 1);
       mbar_init(&bars->s_full[i], 1);
     }
-    mbar_init(&bars->p_full, 4);
+    mbar_init(&bars->p_full, 8);
     mbar_init(&bars->pv_done, 1);
     mbar_init(&bars->clean, 1);
     fence_barrier_init();
@@ -162,52 +167,79 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
     }
     return;
   }
-  if (warp == 5) {
+  const int* bt = a.table + static_cast<long long>(x.req_rows[ri]) * a.bt_stride;
+  auto load_pair = [&](int st, int d, int pg0, int pg1) {
+    mbar_expect_tx(&bars->full[st], 2 * kLtPanel);
+    uint8_t* dst = ring + st * 2 * kLtPanel;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      tma_load_2d(dst + j * kLtPanel, &tm_rows, &bars->full[st], (2 * d + j) * 64, pg0 * kLatPage);
+      tma_load_2d(dst + j * kLtPanel + kLtPanel / 2, &tm_rows, &bars->full[st], (2 * d + j) * 64, pg1 * kLatPage);
+    }
+  };
+  auto load_tail = [&](int st, int pg0, int pg1) {
+    mbar_expect_tx(&bars->tail_full[st], kLtPanel);
+    tma_load_2d(tails + st * kLtPanel, &tm_rows, &bars->tail_full[st], 2 * x.pairs * 64, pg0 * kLatPage);
+    tma_load_2d(tails + st * kLtPanel + kLtPanel / 2, &tm_rows, &bars->tail_full[st], 2 * x.pairs * 64, pg1 * kLatPage);
+  };
+  auto page_of = [&](int lp) { return lp <= p_last / kLatPage ? max(bt[lp], 0) : 0; };
+  if (warp == 8 && lane == 0) {
+    // the first block is on its way while the queries are laid out
+    const int pg0 = page_of(2 * b0), pg1 = page_of(2 * b0 + 1);
+    for (int d = 0; d < x.pairs; ++d) load_pair(d, d, pg0, pg1);
+    if (x.tail) load_tail(0, pg0, pg1);
+  }
+  if (warp == 9) {
     tmem_alloc(&bars->tmem_base, kTmemCols);
     tmem_relinquish();
   }
-  const int* bt = a.table + static_cast<long long>(x.req_rows[ri]) * a.bt_stride;
-  // cos and sin of the tile's positions (in the probabilities' memory, which comes later), columns' last keys
+  __syncwarp();
+  // latent parts of the queries, straight to their places
+  for (int n = warp; n < N; n += kLtThreads / 32) {
+    const int q = n / x.hs, hh = n - q * x.hs;
+    const bool valid = q < ntok && hh < nh;
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(a.qa) + (valid ? (tok0 + q) * a.ldqa + (h0 + hh) * a.cp : 0);
+    for (int cc = lane; cc < q_panels * 8; cc += 32) {
+      uint8_t* dst = q_s + (cc >> 3) * (N * 128) + n * 128 + (((cc & 7) ^ (n & 7)) << 4);
+      if (valid && cc * 8 < a.rot_off) lt_cp16(dst, src + cc * 8);
+      else if (!valid || cc * 8 >= a.rot_off + a.R) *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    }
+    if (lane == 0) {
+      col_pos[n] = valid ? p0 + q : -1;
+      col_row[n] = (tok0 + q) * a.H + h0 + hh;
+      m_ref[n] = -INFINITY;
+    }
+  }
+  // cos and sin of the tile's positions (in the probabilities' memory, which comes later)
   const int half = a.R >> 1;
   float2* cs = reinterpret_cast<float2*>(p_s);
   const bool table_fits = ntok * half * 8 <= 2 * 2 * N * 128;
   if (table_fits)
     for (int e = threadIdx.x; e < ntok * half; e += kLtThreads) cs[e] = lat_cos_sin(p0 + e / half, a.freq[e % half], a.freq[half + e % half]);
-  if (threadIdx.x < N) {
-    const int q = threadIdx.x / x.hs;
-    col_pos[threadIdx.x] = q < ntok && static_cast<int>(threadIdx.x) - q * x.hs < nh ? p0 + q : -1;
-    m_ref[threadIdx.x] = -INFINITY;
-    if (threadIdx.x < 2) flags[threadIdx.x] = 0;
-  }
+  if (threadIdx.x < 2) flags[threadIdx.x] = 0;
   __syncthreads();
   {
-    const int chunks = q_panels * 8;
+    const int chunks = (a.R + 7) / 8;
     for (int e = threadIdx.x; e < N * chunks; e += kLtThreads) {
-      const int n = e / chunks, cc = e - n * chunks, c = cc * 8;
-      const int q = n / x.hs, hh = n - q * x.hs;
+      const int n = e / chunks, rc = e - n * chunks, cc = (a.rot_off >> 3) + rc;
+      if (col_pos[n] < 0) continue;
+      const int q = n / x.hs;
+      const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(a.qr) + (tok0 + q) * a.ldqr + (h0 + n - q * x.hs) * a.R + rc * 8;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (q < ntok && hh < nh) {
-        const long long t = tok0 + q;
-        const int h = h0 + hh;
-        if (c < a.rot_off) {
-          v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.qa) + t * a.ldqa + h * a.cp + c);
-        } else if (c < a.rot_off + a.R) {
-          const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(a.qr) + t * a.ldqr + h * a.R + (c - a.rot_off);
-          __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&v);
+      __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&v);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const int k = ((c - a.rot_off) >> 1) + j;
-            if (k < half) {
-              const float2 w = table_fits ? cs[q * half + k] : lat_cos_sin(p0 + q, a.freq[k], a.freq[half + k]);
-              const float u = bf16_to_f(src[2 * j]), y = bf16_to_f(src[2 * j + 1]);
-              o[j] = __floats2bfloat162_rn(u * w.x - y * w.y, y * w.x + u * w.y);
-            }
-          }
+      for (int j = 0; j < 4; ++j) {
+        const int k = rc * 4 + j;
+        if (k < half) {
+          const float2 w = table_fits ? cs[q * half + k] : lat_cos_sin(p0 + q, a.freq[k], a.freq[half + k]);
+          const float u = bf16_to_f(src[2 * j]), y = bf16_to_f(src[2 * j + 1]);
+          o[j] = __floats2bfloat162_rn(u * w.x - y * w.y, y * w.x + u * w.y);
         }
       }
       *reinterpret_cast<uint4*>(q_s + (cc >> 3) * (N * 128) + n * 128 + (((cc & 7) ^ (n & 7)) << 4)) = v;
     }
   }
+  asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
   fence_proxy_async();
   tc_fence_before();
   __syncthreads();
@@ -218,32 +250,24 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
   // scores of the next block may be formed before this block's output when the ring holds two blocks
   const bool ahead = x.slots >= 2 * x.pairs;
 
-  if (warp == 4) {
+  if (warp == 8) {
     // ------------------------------- loader -------------------------------
     bool ok = true;
-    int seq = 0, done_b = b0;
+    int seq = x.pairs, done_b = b0 + 1;
     if (lane == 0) {
-      for (int b = b0; b < b1 && ok; ++b) {
-        const int pg0 = max(bt[2 * b], 0), pg1 = 2 * b + 1 <= p_last / kLatPage ? max(bt[2 * b + 1], 0) : 0;
+      for (int b = b0 + 1; b < b1 && ok; ++b) {
+        const int pg0 = page_of(2 * b), pg1 = page_of(2 * b + 1);
         for (int d = 0; d < x.pairs; ++d, ++seq) {
           const int st = seq % x.slots;
           if (seq >= x.slots) ok = mbar_wait(&bars->empty[st], ((seq / x.slots) - 1) & 1, x.status, 900);
           if (!ok) break;
-          mbar_expect_tx(&bars->full[st], 2 * kLtPanel);
-          uint8_t* dst = ring + st * 2 * kLtPanel;
-#pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            tma_load_2d(dst + j * kLtPanel, &tm_rows, &bars->full[st], (2 * d + j) * 64, pg0 * kLatPage);
-            tma_load_2d(dst + j * kLtPanel + kLtPanel / 2, &tm_rows, &bars->full[st], (2 * d + j) * 64, pg1 * kLatPage);
-          }
+          load_pair(st, d, pg0, pg1);
         }
         if (ok && x.tail) {
           const int i = b - b0, st = i & 1;
           if (i >= 2) ok = mbar_wait(&bars->tail_empty[st], ((i >> 1) - 1) & 1, x.status, 901);
           if (!ok) break;
-          mbar_expect_tx(&bars->tail_full[st], kLtPanel);
-          tma_load_2d(tails + st * kLtPanel, &tm_rows, &bars->tail_full[st], 2 * x.pairs * 64, pg0 * kLatPage);
-          tma_load_2d(tails + st * kLtPanel + kLtPanel / 2, &tm_rows, &bars->tail_full[st], 2 * x.pairs * 64, pg1 * kLatPage);
+          load_tail(st, pg0, pg1);
           done_b = b + 1;
         }
       }
@@ -272,106 +296,103 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
     if (!ok && lane == 0) {
       // leave no copy in flight: what was asked for lands before the CTA's shared memory goes away
       for (int s = max(0, seq - x.slots); s < seq; ++s) mbar_wait(&bars->full[s % x.slots], (s / x.slots) & 1, nullptr, 0);
-      for (int i = max(0, done_b - b0 - 2); i < done_b - b0; ++i) mbar_wait(&bars->tail_full[i & 1], (i >> 1) & 1, nullptr, 0);
+      for (int i = max(0, done_b - b0 - 2); x.tail && i < done_b - b0; ++i) mbar_wait(&bars->tail_full[i & 1], (i >> 1) & 1, nullptr, 0);
     }
     __syncwarp();
-  } else if (warp == 5) {
+  } else if (warp == 9) {
     // ------------------------------- MMA issuer -------------------------------
-    if (lane == 0) {
-      constexpr uint32_t kIdescS = umma_idesc(1u, 1u, 128, N);
-      constexpr uint32_t kIdescO = umma_idesc(1u, 1u, 128, 2 * N) | (1u << 15);           // A is MN-major
-      bool ok = true;
-      auto scores = [&](int b) {
-        const int i = b - b0;
-        if (ragged && b == b1 - 1) {
-          if (!mbar_wait(&bars->clean, 0, x.status, 910)) return false;
-        }
-        uint32_t acc = 0;
-        for (int d = 0; d < x.pairs; ++d) {
-          const int s = i * x.pairs + d, st = s % x.slots;
-          if (!mbar_wait(&bars->full[st], (s / x.slots) & 1, x.status, 911)) return false;
-          tc_fence_after();
-          for (int j = 0; j < 2; ++j) {
-            const uint64_t ad = umma_desc_sw128(smem_u32(ring + (st * 2 + j) * kLtPanel));
-            const uint64_t bd = umma_desc_sw128(smem_u32(q_s + (2 * d + j) * (N * 128)));
-            const int n = min(4, x.steps - (2 * d + j) * 4);
-            for (int ks = 0; ks < n; ++ks) {
-              umma_f16(tmem + (i & 1) * N, ad + 2 * ks, bd + 2 * ks, kIdescS, acc);
-              acc = 1;
-            }
-          }
-          if (d >= x.v_tiles) umma_commit(&bars->empty[st]);
-        }
-        if (x.tail) {
-          if (!mbar_wait(&bars->tail_full[i & 1], (i >> 1) & 1, x.status, 912)) return false;
-          tc_fence_after();
-          const uint64_t ad = umma_desc_sw128(smem_u32(tails + (i & 1) * kLtPanel));
-          const uint64_t bd = umma_desc_sw128(smem_u32(q_s + 2 * x.pairs * (N * 128)));
-          const int n = min(4, x.steps - 8 * x.pairs);
-          for (int ks = 0; ks < n; ++ks) {
-            umma_f16(tmem + (i & 1) * N, ad + 2 * ks, bd + 2 * ks, kIdescS, acc);
-            acc = 1;
-          }
-          umma_commit(&bars->tail_empty[i & 1]);
-        }
-        umma_commit(&bars->s_full[i & 1]);
-        return true;
-      };
-      ok = scores(b0);
-      for (int b = b0; b < b1 && ok; ++b) {
-        const int i = b - b0;
-        if (ahead && b + 1 < b1) ok = scores(b + 1);
-        if (!ok) break;
-        ok = mbar_wait(&bars->p_full, i & 1, x.status, 913);
-        if (!ok) break;
-        tc_fence_after();
-        for (int j = 0; j < x.v_tiles; ++j) {
-          const int st = (i * x.pairs + j) % x.slots;
-          const uint32_t rows = smem_u32(ring + st * 2 * kLtPanel);
-#pragma unroll
-          for (int kk = 0; kk < 8; ++kk) {
-            const uint64_t bd = umma_desc_sw128(smem_u32(p_s + (kk >> 2) * (2 * N * 128))) + 2 * (kk & 3);
-            umma_f16(tmem_o + j * 2 * N, lt_desc_mn(rows + kk * 2048), bd, kIdescO, (i > 0 || kk > 0) ? 1u : 0u);
-          }
-          umma_commit(&bars->empty[st]);
-        }
-        umma_commit(&bars->pv_done);
-        if (!ahead && b + 1 < b1) ok = scores(b + 1);
+    constexpr uint32_t kIdescS = umma_idesc(1u, 1u, 128, N);
+    constexpr uint32_t kIdescO = umma_idesc(1u, 1u, 128, 2 * N) | (1u << 15);             // A is MN-major
+    constexpr uint32_t kStep = kLtPanel >> 4, kQStep = (N * 128) >> 4;                    // panels in descriptor units
+    const uint32_t lead = elect_one() ? 1u : 0u, tm = __shfl_sync(0xffffffffu, tmem, 0);
+    const uint32_t k_lo = desc_lo(smem_u32(ring)), v_lo = desc_lo(smem_u32(ring), kLtPanel), t_lo = desc_lo(smem_u32(tails));
+    const uint32_t q_lo = desc_lo(smem_u32(q_s)), p_lo = desc_lo(smem_u32(p_s));
+    struct At { int slot; uint32_t par; };
+    auto ahead_of = [&](At c, int n) {
+      c.slot += n;
+      if (c.slot >= x.slots) { c.slot -= x.slots; c.par ^= 1u; }
+      return c;
+    };
+    auto scores = [&](int b, At c) {
+      const int i = b - b0;
+      if (ragged && b == b1 - 1) {
+        if (!mbar_wait(&bars->clean, 0, x.status, 910)) return false;
       }
+      const uint32_t d0 = tm + (i & 1) * N;
+      for (int d = 0; d < x.pairs; ++d) {
+        const At p = ahead_of(c, d);
+        if (!mbar_wait(&bars->full[p.slot], p.par, x.status, 911)) return false;
+        tc_fence_after();
+        const uint32_t al = k_lo + p.slot * 2 * kStep, bl = q_lo + d * 2 * kQStep;
+#pragma unroll
+        for (int ks = 0; ks < 8; ++ks)
+          mma_ss(d0, al + (ks >> 2) * kStep + 2 * (ks & 3), bl + (ks >> 2) * kQStep + 2 * (ks & 3), kIdescS,
+                 ks > 0 ? 1u : (d > 0 ? 1u : 0u), lead);
+        if (d >= x.v_tiles) mma_commit(&bars->empty[p.slot], lead);
+      }
+      if (x.tail) {
+        if (!mbar_wait(&bars->tail_full[i & 1], (i >> 1) & 1, x.status, 912)) return false;
+        tc_fence_after();
+        const uint32_t al = t_lo + (i & 1) * kStep, bl = q_lo + 2 * x.pairs * kQStep;
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) mma_ss(d0, al + 2 * ks, bl + 2 * ks, kIdescS, ks > 0 ? 1u : (x.pairs > 0 ? 1u : 0u), lead);
+        mma_commit(&bars->tail_empty[i & 1], lead);
+      }
+      mma_commit(&bars->s_full[i & 1], lead);
+      return true;
+    };
+    At cur{0, 0u};                                                  // first pair of block b
+    bool ok = scores(b0, cur);
+    for (int b = b0; b < b1 && ok; ++b) {
+      const int i = b - b0;
+      const At next = ahead_of(cur, x.pairs);
+      if (ahead && b + 1 < b1) ok = scores(b + 1, next);
+      if (ok) ok = mbar_wait(&bars->p_full, i & 1, x.status, 913);
+      if (!ok) break;
+      tc_fence_after();
+      for (int j = 0; j < x.v_tiles; ++j) {
+        const int st = ahead_of(cur, j).slot;
+        const uint32_t al = v_lo + st * 2 * kStep, dj = tm + 2 * N + j * 2 * N;
+#pragma unroll
+        for (int kk = 0; kk < 8; ++kk)
+          mma_ss(dj, al + kk * 128, p_lo + (kk >> 2) * 2 * kQStep + 2 * (kk & 3), kIdescO, kk > 0 ? 1u : (i > 0 ? 1u : 0u), lead);
+        mma_commit(&bars->empty[st], lead);
+      }
+      mma_commit(&bars->pv_done, lead);
+      if (!ahead && b + 1 < b1) ok = scores(b + 1, next);
+      cur = next;
     }
     __syncwarp();
   } else {
     // ------------------------------- softmax -------------------------------
-    const int row = warp * 32 + lane;
-    const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
+    constexpr int NH = N / 2;                                       // columns of this thread
+    const int row = (warp & 3) * 32 + lane, c0 = (warp >> 2) * NH;
+    const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const float c_in = a.scale * kLtLog2e;
-    float l[N];
+    float l[NH];
 #pragma unroll
-    for (int n = 0; n < N; ++n) l[n] = 0.f;
+    for (int n = 0; n < NH; ++n) l[n] = 0.f;
     bool ok = true;
     for (int b = b0; b < b1; ++b) {
       const int i = b - b0, key = b * kLtBlock + row;
       ok = ok && mbar_wait(&bars->s_full[i & 1], (i >> 1) & 1, x.status, 920);
       tc_fence_after();
-      const bool edge = b * kLtBlock + kLtBlock - 1 > p0;
-      float v[N];
-      auto load = [&]() {
+      float v[NH], keep[NH];
+      {
+        uint32_t r[NH];
+        lt_ld<NH>(tmem + (i & 1) * N + c0 + lanes, r);
+        tmem_ld_wait();
 #pragma unroll
-        for (int c = 0; c < N; c += 16) {
-          uint32_t r[16];
-          tmem_ld_32x16(tmem + (i & 1) * N + lanes + c, r);
-          tmem_ld_wait();
+        for (int n = 0; n < NH; ++n) v[n] = __uint_as_float(r[n]) * c_in;
+        if (b * kLtBlock + kLtBlock - 1 > p0) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[c + j] = __uint_as_float(r[j]) * c_in;
+          for (int n = 0; n < NH; ++n)
+            if (key > col_pos[c0 + n]) v[n] = -INFINITY;
         }
-        if (edge) {
+      }
 #pragma unroll
-          for (int n = 0; n < N; ++n)
-            if (key > col_pos[n]) v[n] = -INFINITY;
-        }
-      };
-      load();
-      bfly_reduce_store<N, true>(v, smax + warp * N, lane);
+      for (int n = 0; n < NH; ++n) keep[n] = v[n];
+      bfly_reduce_store<NH, true>(v, smax + (warp & 3) * N + c0, lane);
       ok = lt_bar_all(ok);
       if (!ok) break;
       if (threadIdx.x == 0) flags[(i + 1) & 1] = 0;
@@ -396,32 +417,34 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
       }
       if (flags[i & 1]) {
 #pragma unroll
-        for (int n = 0; n < N; ++n) l[n] *= alpha[n];
+        for (int n = 0; n < NH; ++n) l[n] *= alpha[c0 + n];
         if (i > 0) {
+          // high parts for the first four warps, remainders for the others
+          const uint32_t to = tmem_o + (warp >> 2) * N + lanes;
           for (int j = 0; j < x.v_tiles; ++j)
 #pragma unroll
-            for (int c = 0; c < 2 * N; c += 16) {
+            for (int c = 0; c < N; c += 16) {
               uint32_t o[16];
-              tmem_ld_32x16(tmem_o + j * 2 * N + c + lanes, o);
+              tmem_ld_32x16(to + j * 2 * N + c, o);
               tmem_ld_wait();
 #pragma unroll
-              for (int k = 0; k < 16; ++k) o[k] = __float_as_uint(__uint_as_float(o[k]) * alpha[(c + k) % N]);
-              lt_st16(tmem_o + j * 2 * N + c + lanes, o);
+              for (int k = 0; k < 16; ++k) o[k] = __float_as_uint(__uint_as_float(o[k]) * alpha[c + k]);
+              lt_st16(to + j * 2 * N + c, o);
             }
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
-      load();
-      uint8_t* dst = p_s + (row >> 6) * (2 * N * 128) + (row & 7) * 2;
+      uint8_t* dst = p_s + (row >> 6) * (2 * N * 128) + c0 * 128 + (row & 7) * 2;
       const int chunk = (row & 63) >> 3;
 #pragma unroll
-      for (int n = 0; n < N; ++n) {
-        const float mr = m_ref[n];
-        const float p = mr == -INFINITY ? 0.f : lt_ex2(v[n] - mr);
+      for (int n = 0; n < NH; ++n) {
+        const float mr = m_ref[c0 + n];
+        const float p = mr == -INFINITY ? 0.f : lt_ex2(keep[n] - mr);
         l[n] += p;
         const __nv_bfloat16 hi = __float2bfloat16(p);
-        *reinterpret_cast<__nv_bfloat16*>(dst + n * 128 + ((chunk ^ (n & 7)) << 4)) = hi;
-        *reinterpret_cast<__nv_bfloat16*>(dst + (N + n) * 128 + ((chunk ^ (n & 7)) << 4)) = __float2bfloat16(p - bf16_to_f(hi));
+        const int at = n * 128 + ((chunk ^ (n & 7)) << 4);
+        *reinterpret_cast<__nv_bfloat16*>(dst + at) = hi;
+        *reinterpret_cast<__nv_bfloat16*>(dst + N * 128 + at) = __float2bfloat16(p - bf16_to_f(hi));
       }
       fence_proxy_async();
       tc_fence_before();
@@ -430,10 +453,11 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
     }
     if (ok) ok = mbar_wait(&bars->pv_done, (b1 - 1 - b0) & 1, x.status, 922);
     tc_fence_after();
-    bfly_reduce_store<N, false>(l, smax + warp * N, lane);
+    bfly_reduce_store<NH, false>(l, smax + (warp & 3) * N + c0, lane);
     lt_bar_sync();
     if (ok) {
-      for (int j = 0; j < x.v_tiles; ++j) {
+      // the two halves of the warps take every other 128 dims
+      for (int j = warp >> 2; j < x.v_tiles; j += 2) {
         const int d = j * 128 + row;
 #pragma unroll
         for (int c = 0; c < N; c += 16) {
@@ -441,18 +465,17 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
           tmem_ld_32x16(tmem_o + j * 2 * N + c + lanes, u);
           tmem_ld_32x16(tmem_o + j * 2 * N + N + c + lanes, w);
           tmem_ld_wait();
+          if (d < a.C) {
 #pragma unroll
-          for (int k = 0; k < 16; ++k) {
-            const int n = c + k;
-            const int q = n / x.hs, hh = n - q * x.hs;
-            if (q < ntok && hh < nh && d < a.C)
-              part[(static_cast<long long>(tok0 + q) * a.H + h0 + hh) * (a.C + 2) + d] = __uint_as_float(u[k]) + __uint_as_float(w[k]);
+            for (int k = 0; k < 16; ++k)
+              if (col_pos[c + k] >= 0)
+                part[static_cast<long long>(col_row[c + k]) * (a.C + 2) + d] = __uint_as_float(u[k]) + __uint_as_float(w[k]);
           }
         }
       }
       if (threadIdx.x < N && col_pos[threadIdx.x] >= 0) {
-        const int n = threadIdx.x, q = n / x.hs, hh = n - q * x.hs;
-        float* o = part + (static_cast<long long>(tok0 + q) * a.H + h0 + hh) * (a.C + 2);
+        const int n = threadIdx.x;
+        float* o = part + static_cast<long long>(col_row[n]) * (a.C + 2);
         o[a.C] = m_ref[n];
         o[a.C + 1] = (smax[n] + smax[N + n]) + (smax[2 * N + n] + smax[3 * N + n]);
       }
@@ -460,18 +483,21 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == 9) {
     tc_fence_after();
     tmem_dealloc(tmem, kTmemCols);
   }
 }
 
 // One CTA per (token, head): joins the splits, normalises, gates; zeros behind the latent's dimensions and for padding tokens.
+constexpr int kLtMaxSplits = 64;
+
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part, int splits, const float* __restrict__ gate, long long ldg,
                     const int64_t* __restrict__ positions, const int* __restrict__ tok_req, const int* __restrict__ first_pos,
                     const int* __restrict__ last_pos, int max_span, int T, int H, int C, int cp, __nv_bfloat16* __restrict__ out,
                     long long ldo) {
+  __shared__ float wt[kLtMaxSplits];
   pdl_wait();
   pdl_trigger();
   const long long t = blockIdx.x;
@@ -484,22 +510,38 @@ latent_merge_kernel(const float* __restrict__ part, int splits, const float* __r
   if (last_pos[t] - first_pos[t] + 1 > max_span) return;
   const long long step = static_cast<long long>(T) * H * (C + 2);
   const float* p = part + (t * H + h) * (C + 2);
-  float m = -INFINITY;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, p[s * step + C]);
-  float l = 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float ms = p[s * step + C];
-    if (ms != -INFINITY) l = fmaf(lt_ex2(ms - m), p[s * step + C + 1], l);
+  if (threadIdx.x < 32) {
+    // the splits' weights: two per lane
+    float m[2], l[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int s = threadIdx.x + i * 32;
+      m[i] = s < splits ? p[s * step + C] : -INFINITY;
+      l[i] = s < splits ? p[s * step + C + 1] : 0.f;
+    }
+    const float mx = warp_max(fmaxf(m[0], m[1]));
+    float sum = 0.f, f[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      f[i] = m[i] == -INFINITY ? 0.f : lt_ex2(m[i] - mx);
+      sum = fmaf(f[i], l[i], sum);
+    }
+    const float g = (gate != nullptr ? lat_sigmoid(gate[t * ldg + h]) : 1.f) / warp_sum(sum);
+    wt[threadIdx.x] = f[0] * g;
+    wt[threadIdx.x + 32] = f[1] * g;
   }
-  const float g = (gate != nullptr ? lat_sigmoid(gate[t * ldg + h]) : 1.f) / l;
+  __syncthreads();
   for (int d = threadIdx.x; d < cp; d += blockDim.x) {
     float v = 0.f;
-    if (d < C)
+    if (d < C) {
+      // a split without keys left its columns unwritten
+#pragma unroll 8
       for (int s = 0; s < splits; ++s) {
-        const float ms = p[s * step + C];
-        if (ms != -INFINITY) v = fmaf(lt_ex2(ms - m), p[s * step + d], v);
+        const float w = wt[s];
+        v = fmaf(w, w != 0.f ? p[s * step + d] : 0.f, v);
       }
-    o[d] = __float2bfloat16(v * g);
+    }
+    o[d] = __float2bfloat16(v);
   }
 }
 
@@ -513,7 +555,7 @@ static LtShape lt_shape(int C, int row, int n) {
   s.pairs = panels / 2;
   s.tail = panels & 1;
   if (s.pairs < s.v_tiles) { s.pairs = s.v_tiles; s.tail = 0; }        // the values reach into the odd panel
-  const int fixed = (2 * s.pairs + s.tail) * n * 128 + 4 * n * 128 + (s.tail ? 2 * kLtPanel : 0) + 256 + 7 * n * 4 + 64 + 1024;
+  const int fixed = (2 * s.pairs + s.tail) * n * 128 + 4 * n * 128 + (s.tail ? 2 * kLtPanel : 0) + 256 + 8 * n * 4 + 64 + 1024;
   s.slots = (227 * 1024 - fixed) / (2 * kLtPanel);
   if (s.slots > kLtMaxPairs) s.slots = kLtMaxPairs;
   return s;
@@ -540,7 +582,7 @@ STK_API int stk_latent_tokens_splits(int T, int heads, int max_span, int context
   const int blocks = context / kLtBlock + 1;
   int best = 1;
   double cost = 1e30;
-  for (int s = 1; s <= 64 && s <= blocks; ++s) {
+  for (int s = 1; s <= kLtMaxSplits && s <= blocks; ++s) {
     const int waves = (tiles * s + sm_count - 1) / sm_count;
     const double c = static_cast<double>(waves) * ((blocks + s - 1) / s + 1.5) + 0.03 * s;
     if (c < cost - 1e-9) { cost = c; best = s; }
@@ -560,7 +602,7 @@ STK_API int stk_latent_tokens(const void* qa, long long ldqa, int cp, const void
   x.l = lat_args(qa, ldqa, cp, qr, ldqr, gate, ldg, positions, tok_req, table, bt_stride, cache, row, rot_off, freq, heads, kv_rank,
                  rot, scale, out, ldo);
   const int n = stk_latent_tokens_columns(heads, kv_rank, row, max_span);
-  if (!lat_ok(x.l) || n == 0 || splits < 1 || n_req < 1 || num_pages < 1 || ldqa % 8 || cp % 8 || rot_off % 8 || heads > 65535 ||
+  if (!lat_ok(x.l) || n == 0 || splits < 1 || splits > kLtMaxSplits || n_req < 1 || num_pages < 1 || ldqa % 8 || cp % 8 || rot_off % 8 || heads > 65535 ||
       ((reinterpret_cast<uintptr_t>(qa) | reinterpret_cast<uintptr_t>(cache)) & 15))
     return -1;
   const LtShape s = lt_shape(kv_rank, row, n);
@@ -568,12 +610,12 @@ STK_API int stk_latent_tokens(const void* qa, long long ldqa, int cp, const void
   x.hs = (heads + groups - 1) / groups;
   x.tq = max_span < 2 ? 1 : n / x.hs;
   x.query_start = query_start; x.req_rows = req_rows; x.start_pos = start_pos; x.n_req = n_req; x.max_span = max_span;
-  x.pairs = s.pairs; x.tail = s.tail; x.slots = s.slots; x.v_tiles = s.v_tiles; x.steps = (row + 15) / 16;
+  x.pairs = s.pairs; x.tail = s.tail; x.slots = s.slots; x.v_tiles = s.v_tiles;
   x.part = part; x.T = T; x.status = status;
   static_assert(sizeof(LtBars) <= 256, "barrier block");
   CUtensorMap tm;
   if (make_tmap_2d(&tm, cache, 2, num_pages * kLatPage, row, row, kLatPage) != 0) return -3;
-  int smem = s.slots * 2 * kLtPanel + (s.tail ? 2 * kLtPanel : 0) + (2 * s.pairs + s.tail) * n * 128 + 4 * n * 128 + 256 + 7 * n * 4 +
+  int smem = s.slots * 2 * kLtPanel + (s.tail ? 2 * kLtPanel : 0) + (2 * s.pairs + s.tail) * n * 128 + 4 * n * 128 + 256 + 8 * n * 4 +
              64 + 1024;
   if (smem < 118 * 1024) smem = 118 * 1024;                          // one CTA per SM: it owns all of tensor memory
   const int tiles = max_span < 2 ? min(T, n_req) : T / x.tq + n_req;
