@@ -495,33 +495,37 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUt
             const int nthr2 = kEpiWarps * 32;
             const int rows_valid = min(BT, a.T - tt * BT);
             const int cols_valid = min(128, a.N - tn * 128);
-            const bool vec_ok = (cols_valid == 128) && ((a.N & 3) == 0) && (a.out_vec_ok || a.ar_enabled);
+            const int cv = cols_valid >> 2;                  // vectors of a row (a tile at the edge of N has fewer than 32)
+            const bool vec_ok = ((a.N & 3) == 0) && (a.out_vec_ok || a.ar_enabled);
             if (vec_ok) {
               // four output vectors per thread at a time, so that 4 x (unrolled splits) loads are in flight: one vector
               // at a time left a reducing CTA at a few dozen GB/s
-              const int total = rows_valid * 32;
+              const int total = rows_valid * cv;
               for (int v0 = et2; v0 < total; v0 += nthr2 * 4) {
                 float4 s4[4];
+                int row4[4], col4[4];
+                const float* src[4];                        // the vector's place in split 0 (the last one's past the end)
 #pragma unroll
-                for (int u = 0; u < 4; ++u) s4[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+                for (int u = 0; u < 4; ++u) {
+                  s4[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+                  const int v = min(v0 + u * nthr2, total - 1);
+                  row4[u] = cv == 32 ? v >> 5 : v / cv;
+                  col4[u] = (v - row4[u] * cv) * 4;
+                  src[u] = a.workspace + static_cast<long long>(tt * BT + row4[u]) * a.N + tn * 128 + col4[u];
+                }
+                const long long split_step = static_cast<long long>(a.T) * a.N;
 #pragma unroll 4
                 for (int p = 0; p < a.splits; ++p) {
 #pragma unroll
                   for (int u = 0; u < 4; ++u) {
-                    const int v = v0 + u * nthr2;
-                    if (v < total) {
-                      const int r = v >> 5, c4 = (v & 31) * 4;
-                      const float4 x = __ldcg(reinterpret_cast<const float4*>(
-                          &a.workspace[(static_cast<long long>(p) * a.T + tt * BT + r) * a.N + tn * 128 + c4]));
-                      s4[u].x += x.x; s4[u].y += x.y; s4[u].z += x.z; s4[u].w += x.w;
-                    }
+                    const float4 x = __ldcg(reinterpret_cast<const float4*>(src[u] + p * split_step));
+                    s4[u].x += x.x; s4[u].y += x.y; s4[u].z += x.z; s4[u].w += x.w;
                   }
                 }
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
-                  const int v = v0 + u * nthr2;
-                  if (v >= total) break;
-                  const int r = v >> 5, c4 = (v & 31) * 4;
+                  if (v0 + u * nthr2 >= total) break;
+                  const int r = row4[u], c4 = col4[u];
                   const int t = tt * BT + r;
                   if (a.ar_enabled) {
                     if constexpr (Cfg::kArTileBytes > 0) {
@@ -702,6 +706,7 @@ gemm_wide_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
       tc_fence_after();
       // a thread owns one token row and, per chunk, 32 consecutive output features: 64 contiguous bytes of bf16
       const bool vec_ok = !a.out_fp32 && (a.ldo % 8 == 0) && ((reinterpret_cast<uintptr_t>(a.out) & 15) == 0);
+      const bool vec32_ok = (a.ldo % 4 == 0) && ((reinterpret_cast<uintptr_t>(a.out) & 15) == 0);
 #pragma unroll
       for (int m = 0; m < 2; ++m) {
         const int t = tt * 256 + m * 128 + q * 32 + lane;
@@ -727,9 +732,14 @@ gemm_wide_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
               }
             } else if (a.out_fp32) {
               float* o = reinterpret_cast<float*>(a.out) + static_cast<long long>(t) * a.ldo + n0;
+              if (vec32_ok && n0 + 32 <= a.N) {
 #pragma unroll
-              for (int j = 0; j < 32; ++j)
-                if (n0 + j < a.N) o[j] = __uint_as_float(r[j]);
+                for (int j = 0; j < 32; j += 4) *reinterpret_cast<uint4*>(o + j) = make_uint4(r[j], r[j + 1], r[j + 2], r[j + 3]);
+              } else {
+#pragma unroll
+                for (int j = 0; j < 32; ++j)
+                  if (n0 + j < a.N) o[j] = __uint_as_float(r[j]);
+              }
             } else {
               __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(a.out) + static_cast<long long>(t) * a.ldo + n0;
 #pragma unroll

@@ -489,7 +489,7 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
   }
 }
 
-// One CTA per (token, head): joins the splits, normalises, gates; zeros behind the latent's dimensions and for padding tokens.
+// One CTA per (token, head, part of the dims): joins the splits, normalises, gates; zeros behind the latent's dimensions and for padding tokens.
 constexpr int kLtMaxSplits = 64;
 
 __global__ void __launch_bounds__(128)
@@ -503,8 +503,9 @@ latent_merge_kernel(const float* __restrict__ part, int splits, const float* __r
   const long long t = blockIdx.x;
   const int h = blockIdx.y;
   __nv_bfloat16* o = out + t * ldo + h * cp;
+  const int d0 = blockIdx.z * blockDim.x + threadIdx.x, dstep = gridDim.z * blockDim.x;
   if (tok_req[t] < 0 || positions[t] < 0) {
-    for (int d = threadIdx.x; d < cp; d += blockDim.x) o[d] = __float2bfloat16(0.f);
+    for (int d = d0; d < cp; d += dstep) o[d] = __float2bfloat16(0.f);
     return;
   }
   if (last_pos[t] - first_pos[t] + 1 > max_span) return;
@@ -531,11 +532,11 @@ latent_merge_kernel(const float* __restrict__ part, int splits, const float* __r
     wt[threadIdx.x + 32] = f[1] * g;
   }
   __syncthreads();
-  for (int d = threadIdx.x; d < cp; d += blockDim.x) {
+  for (int d = d0; d < cp; d += dstep) {
     float v = 0.f;
     if (d < C) {
       // a split without keys left its columns unwritten
-#pragma unroll 8
+#pragma unroll 16
       for (int s = 0; s < splits; ++s) {
         const float w = wt[s];
         v = fmaf(w, w != 0.f ? p[s * step + d] : 0.f, v);
@@ -629,7 +630,9 @@ STK_API int stk_latent_tokens(const void* qa, long long ldqa, int cp, const void
     if (cudaFuncSetAttribute(latent_tokens_tc_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -3;
     launch_pdl(latent_tokens_tc_kernel<32>, grid, dim3(kLtThreads), smem, st, tm, x);
   }
-  launch_pdl(latent_merge_kernel, dim3(T, heads), dim3(128), 0, st, (const float*)part, splits, gate, ldg, positions, tok_req, first_pos,
+  // few rows: every 128 dims get a CTA of their own (each waits for as many loads as there are splits)
+  const int z = static_cast<long long>(T) * heads < 1024 ? (cp + 127) / 128 : 1;
+  launch_pdl(latent_merge_kernel, dim3(T, heads, z), dim3(128), 0, st, (const float*)part, splits, gate, ldg, positions, tok_req, first_pos,
              last_pos, max_span, T, heads, kv_rank, cp, (__nv_bfloat16*)out, ldo);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
