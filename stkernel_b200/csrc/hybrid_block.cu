@@ -17,10 +17,11 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
   const long long id = ids[t];
   const bool ok = id >= 0 && id < vocab;
   if (!ok && threadIdx.x == 0) set_status(status, kBadIndex, t);
+  const bool vec = sizeof(E) == 2 && (W & 7) == 0 && (ldx & 3) == 0 && (ldh & 7) == 0;
   if (h != nullptr)
-    for (int i = threadIdx.x; i < width; i += blockDim.x)
+    for (int i = (vec ? W : 0) + threadIdx.x; i < width; i += blockDim.x)
       st_act(h + t * ldh + i, ok && i < W ? ld_act(embed + id * W + i) * scale : 0.f);
-  if (sizeof(E) == 2 && (W & 7) == 0 && (ldx & 3) == 0) {
+  if (vec) {
     for (int i = threadIdx.x * 8; i < W; i += blockDim.x * 8) {
       uint4 v = make_uint4(0, 0, 0, 0);
       if (ok) v = __ldg(reinterpret_cast<const uint4*>(embed + id * W + i));
@@ -29,6 +30,12 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
       for (int j = 0; j < 4; ++j) f[j] = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
       *reinterpret_cast<float4*>(x + t * ldx + i) = make_float4(f[0].x * scale, f[0].y * scale, f[1].x * scale, f[1].y * scale);
       *reinterpret_cast<float4*>(x + t * ldx + i + 4) = make_float4(f[2].x * scale, f[2].y * scale, f[3].x * scale, f[3].y * scale);
+      if (h != nullptr) {
+        __align__(16) __nv_bfloat162 b[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) b[j] = __floats2bfloat162_rn(f[j].x * scale, f[j].y * scale);
+        *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(h) + t * ldh + i) = *reinterpret_cast<const uint4*>(b);
+      }
     }
     return;
   }
@@ -182,7 +189,7 @@ post_norm_add_kernel(const PostNormArgs<A> a) {
       *reinterpret_cast<float4*>(xr + i) = v;
       if (hr != nullptr) {
         if (sizeof(A) == 2) {
-          __nv_bfloat162 b[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+          __align__(8) __nv_bfloat162 b[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
           *reinterpret_cast<uint2*>(hr + i) = *reinterpret_cast<const uint2*>(b);
         } else {
           *reinterpret_cast<float4*>(hr + i) = v;

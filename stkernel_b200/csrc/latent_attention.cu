@@ -39,7 +39,11 @@ latent_prep_kernel(const PrepArgs a) {
 #pragma unroll
   for (int j = 0; j < 16; ++j) {
     const int i = i0 + j * 128;
-    v[j] = i < n ? src[i] : 0.f;
+    v[j] = j * 128 < n && i < n ? src[i] : 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j < 16; ++j) {
+    if (j * 128 >= n) break;
     ss = fmaf(v[j], v[j], ss);
   }
   for (int i = i0 + 16 * 128; i < n; i += 128) ss = fmaf(src[i], src[i], ss);
@@ -53,6 +57,7 @@ latent_prep_kernel(const PrepArgs a) {
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
       const int i = i0 + j * 128;
+      if (j * 128 >= a.q_width) break;
       if (i < a.q_width) lat_st(o + i, i < a.Q ? v[j] * inv * a.wq[i] : 0.f);
     }
     for (int i = i0 + 16 * 128; i < a.q_width; i += 128) lat_st(o + i, i < a.Q ? src[i] * inv * a.wq[i] : 0.f);
@@ -69,6 +74,7 @@ latent_prep_kernel(const PrepArgs a) {
 #pragma unroll
   for (int j = 0; j < 16; ++j) {
     const int i = i0 + j * 128;
+    if (j * 128 >= a.rot_off) break;
     if (i < a.rot_off) lat_st(o + i, i < a.C ? v[j] * inv * a.wkv[i] : 0.f);
   }
   for (int i = i0 + 16 * 128; i < a.rot_off; i += 128) lat_st(o + i, i < a.C ? src[i] * inv * a.wkv[i] : 0.f);

@@ -61,7 +61,8 @@ __device__ __forceinline__ float lp_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// One CTA per 128 rows of the gathered matrix.
+// kRowParts CTAs per 128 rows of the gathered matrix.
+constexpr int kRowParts = 8;
 __global__ void __launch_bounds__(256)
 latent_rows_kernel(const int* __restrict__ query_start, const int* __restrict__ req_rows, const int* __restrict__ start_pos, int n_req,
                    int min_span, const int* __restrict__ table, int bt_stride, const __nv_bfloat16* __restrict__ cache, int row,
@@ -84,10 +85,12 @@ latent_rows_kernel(const int* __restrict__ query_start, const int* __restrict__ 
   __syncthreads();
   const int ri = found[0], j0 = found[1] * kLpTile, ctx = found[2];
   const int chunks = row >> 3;
-  uint4* dst = reinterpret_cast<uint4*>(out + static_cast<long long>(blockIdx.x) * kLpTile * row);
+  constexpr int kRows = kLpTile / kRowParts;
+  const int part = blockIdx.y * kRows;
+  uint4* dst = reinterpret_cast<uint4*>(out + (static_cast<long long>(blockIdx.x) * kLpTile + part) * row);
   const int* bt = ri >= 0 ? table + static_cast<long long>(req_rows[ri]) * bt_stride : nullptr;
-  for (int e = threadIdx.x; e < kLpTile * chunks; e += blockDim.x) {
-    const int r = e / chunks, c = e - r * chunks, j = j0 + r;
+  for (int e = threadIdx.x; e < kRows * chunks; e += blockDim.x) {
+    const int r = e / chunks, c = e - r * chunks, j = j0 + part + r;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (ri >= 0 && j < ctx) {
       const int page = bt[j / kLatPage];
@@ -452,7 +455,7 @@ STK_API int stk_latent_rows(const int* query_start, const int* req_rows, const i
                             const int* table, int bt_stride, const void* cache, int row, void* out, long long rows, void* stream) {
   if (rows <= 0) return 0;
   if (rows % kLpTile || row % 8) return -1;
-  launch_pdl(latent_rows_kernel, dim3(static_cast<unsigned>(rows / kLpTile)), dim3(256), 0, (cudaStream_t)stream, query_start,
+  launch_pdl(latent_rows_kernel, dim3(static_cast<unsigned>(rows / kLpTile), kRowParts), dim3(256), 0, (cudaStream_t)stream, query_start,
              req_rows, start_pos, n_req, min_span, table, bt_stride, (const __nv_bfloat16*)cache, row, (__nv_bfloat16*)out);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
