@@ -28,7 +28,7 @@ MAX_SEQUENCES = 64           # live requests
 
 def build_engine(model: str, dtype: str, max_tokens: int):
     """The engine as the server builds it, sized for `max_tokens` live tokens."""
-    from ..config import ConfigError, EngineConfig, SchedulerConfig
+    from ..config import CacheConfig, ConfigError, EngineConfig, SchedulerConfig
     from ..models.loader import CheckpointSource
     from ..models.registry import family_of, load_model_config, use_native
     import torch
@@ -47,8 +47,10 @@ def build_engine(model: str, dtype: str, max_tokens: int):
     torch.cuda.set_device(device)
     context = max(64, max_tokens)
     step = min(MAX_STEP, context)
-    ecfg = EngineConfig(model=cfg, sched=SchedulerConfig(max_model_len=context, max_num_seqs=min(MAX_SEQUENCES, context),
-                                                         max_num_batched_tokens=step)).validate()
+    seqs = min(MAX_SEQUENCES, context)
+    # the live tokens all together, and the page every sequence leaves partly filled
+    ecfg = EngineConfig(model=cfg, sched=SchedulerConfig(max_model_len=context, max_num_seqs=seqs, max_num_batched_tokens=step),
+                        cache=CacheConfig(kv_pool_tokens=context + 64 * seqs)).validate()
     weights = family.build_weights(cfg, CheckpointSource(model), device)
     from ..runtime.engine import Engine
     return Engine(ecfg, weights, device, max_context=context)
