@@ -329,6 +329,89 @@ class MlstmMixer:
 
 
 @dataclass(frozen=True)
+class QueryTemperature:
+    """Queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: float
+
+
+@dataclass(frozen=True)
+class GroupedAttentionMixer:
+    """Grouped-query causal attention over the full context with key and value projections of their own sizes and no rotation.
+
+    qk_norm: queries and keys are divided by their root mean square per head; null_sink: the softmax has one more key of score 0
+    and no value; gate: the heads' outputs are multiplied element by element with the sigmoid of a projection of the same input."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    q_temp: Optional[QueryTemperature] = None
+    bias: bool = True                     # q, k and v projections have biases
+    qk_norm: bool = True
+    null_sink: bool = True
+    gate: bool = True
+    kind = "grouped_attention"
+    window = FULL_CONTEXT
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class RetentionMixer:
+    """Linear attention with a fixed decay per head: S <- decay S + k v^T, read with the query; queries and keys are rotated,
+    every head's read-out is divided by its root mean square and multiplied with silu of a gate."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]
+    rotary: Optional[RotaryConfig] = None
+    kind = "retention"
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class Mamba2Mixer:
+    """Mamba-2: a short causal convolution over (x, B, C), then S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x per head; the
+    gated output is RMS-normed in norm_groups equal parts.  Heads share B and C within each of `groups` groups."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int                             # taps, the current token's included
+    norm_groups: int
+    kind = "mamba2"
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_dim(self) -> int:
+        return self.out_dim + 2 * self.groups * self.state
+
+
+@dataclass(frozen=True)
+class ParallelMixer:
+    """Two mixers over the same input: left_scale * left + right_scale * right.  At most one of them keeps a cache and at most
+    one a recurrent state."""
+    left: GroupedAttentionMixer
+    right: RetentionMixer
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind = "parallel"
+
+    @property
+    def out_dim(self) -> int:
+        return self.left.out_dim + self.right.out_dim
+
+
+@dataclass(frozen=True)
 class DenseMlp:
     """W_down(act(W_gate h) * W_up h)."""
     ff: int
@@ -338,16 +421,48 @@ class DenseMlp:
 
 @dataclass(frozen=True)
 class MoeMlp:
-    """`top` of `experts` feed-forward layers W_down relu(W_up h)^2 per token, chosen by the largest router logits (bias
-    included) and weighted by the softmax over the chosen logits."""
+    """`top` of `experts` feed-forward layers W_down act(W_up h) per token, chosen by the largest router logits (bias included)
+    and weighted by the softmax over the chosen logits (which is the softmax over all of them, renormalised); a shared expert of
+    the same form, if there is one, is added for every token."""
     experts: int
     top: int
     ff: int
+    act: str = "relu2"                    # "relu2" (relu squared) | "gelu" (exact)
+    router_bias: bool = True
+    shared_ff: int = 0                    # 0: no shared expert
     kind = "moe"
 
+    @property
+    def shared_parts(self) -> int:
+        """The shared expert runs as this many always-chosen experts (W_down act(W_up h) is a sum over slices of its columns)."""
+        return 0 if not self.shared_ff else min(-(-self.shared_ff // self.ff), 8, 32 - self.top)
 
-Mixer = Union[AttentionMixer, MlstmMixer, LatentAttentionMixer]
+    @property
+    def expert_width(self) -> int:
+        """Hidden columns of a stored expert: those of an expert, or of a part of the shared one if that is wider."""
+        return self.ff if not self.shared_ff else max(self.ff, -(-self.shared_ff // self.shared_parts))
+
+
+Mixer = Union[AttentionMixer, MlstmMixer, LatentAttentionMixer, GroupedAttentionMixer, RetentionMixer, Mamba2Mixer, ParallelMixer]
 Mlp = Union[DenseMlp, MoeMlp]
+
+ATTENTION_KINDS = ("attention", "latent_attention", "grouped_attention")
+RECURRENT_KINDS = ("mlstm", "retention", "mamba2")
+
+
+def mixer_parts(m: Mixer) -> Tuple[Mixer, ...]:
+    """The mixers a layer runs (a parallel mixer's two sides, otherwise itself)."""
+    return (m.left, m.right) if m.kind == "parallel" else (m,)
+
+
+def attention_part(m: Mixer) -> Optional[Mixer]:
+    """The part of a mixer that keeps a paged cache."""
+    return next((p for p in mixer_parts(m) if p.kind in ATTENTION_KINDS), None)
+
+
+def recurrent_part(m: Mixer) -> Optional[Mixer]:
+    """The part of a mixer that keeps a recurrent state."""
+    return next((p for p in mixer_parts(m) if p.kind in RECURRENT_KINDS), None)
 
 
 @dataclass(frozen=True)
@@ -363,7 +478,10 @@ class HybridConfig:
 
     block "parallel":  both sublayers read one layer norm's output and are added to the fp32 residual together;
     block "post_norm": the sublayers follow one another, read the residual itself, and their outputs are RMS-normed before
-                       they are added to it."""
+                       they are added to it;
+    block "streams":   several residual streams; a sublayer reads the layer norm (with bias) of a weighted sum of them, and every
+                       stream becomes a weighted sum of all of them plus a multiple of the sublayer's output.  The model's
+                       output is the sum of the streams."""
     vocab_size: int
     hidden_size: int
     layers: Tuple[HybridLayer, ...]
@@ -372,7 +490,10 @@ class HybridConfig:
     dtype: str = "bfloat16"               # "bfloat16": projections and activations; "float32": everything
     max_position_embeddings: int = 1 << 30
     architecture: str = "Timalorn"
-    block: str = "parallel"               # "parallel" | "post_norm"
+    block: str = "parallel"               # "parallel" | "post_norm" | "streams"
+    streams: int = 1                      # residual streams ("streams" blocks)
+    tied_head: bool = False               # logits are read with the embedding table
+    logit_scale: float = 1.0
     family = "hybrid"
     # fields of the other family that family-neutral code asks for
     n_mtp_layers = 0
@@ -394,7 +515,8 @@ class HybridConfig:
 
     def windows(self) -> List[int]:
         """Distinct attention windows, one page group each (FULL_CONTEXT: pages stay until the request ends)."""
-        return sorted({l.mixer.window for l in self.layers if l.mixer.kind != "mlstm"})
+        parts = [attention_part(l.mixer) for l in self.layers]
+        return sorted({p.window for p in parts if p is not None})
 
     def cache_layer(self, i: int) -> int:
         """The layer whose cache layer i reads (itself unless `kv_from` says otherwise)."""
@@ -403,7 +525,8 @@ class HybridConfig:
 
     def mechanisms(self) -> Tuple[str, ...]:
         """Kinds of mixers and feed-forwards in this model, which decide what kernels it needs."""
-        return tuple(sorted({l.mixer.kind for l in self.layers} | {l.mlp.kind for l in self.layers if l.mlp is not None}))
+        return tuple(sorted({p.kind for l in self.layers for p in mixer_parts(l.mixer)}
+                            | {l.mlp.kind for l in self.layers if l.mlp is not None}))
 
     def validate(self) -> None:
         def positive(name: str, v: Any, integer: bool = True) -> None:
@@ -414,13 +537,20 @@ class HybridConfig:
         positive("vocab_size", self.vocab_size)
         positive("hidden_size", self.hidden_size)
         positive("norm_eps", self.norm_eps, False)
-        if not isinstance(self.embedding_scale, (int, float)) or not math.isfinite(self.embedding_scale):
-            raise ConfigError("embedding_scale must be a finite number")
+        def number(name: str, v: Any) -> None:
+            if not isinstance(v, (int, float)) or isinstance(v, bool) or not math.isfinite(v):
+                raise ConfigError(f"{name} must be a finite number")
+
+        number("embedding_scale", self.embedding_scale)
+        number("logit_scale", self.logit_scale)
+        positive("streams", self.streams)
+        if self.streams > 8 or (self.streams != 1 and self.block != "streams"):
+            raise ConfigError("streams: at most 8, and 1 unless the block is \"streams\"")
         if self.dtype not in ("bfloat16", "float32"):
             raise ConfigError(f"unknown dtype {self.dtype!r}")
         if not self.layers:
             raise ConfigError("layers must not be empty")
-        if self.block not in ("parallel", "post_norm"):
+        if self.block not in ("parallel", "post_norm", "streams"):
             raise ConfigError(f"unknown block {self.block!r}")
 
         def rotary(at: str, r: RotaryConfig, dim: int, of: str) -> None:
@@ -432,59 +562,107 @@ class HybridConfig:
                 for f in ("factor", "original", "fast", "slow"):
                     positive(f"{at}.rot.scaling.{f}", getattr(r.scaling, f), False)
 
-        for i, l in enumerate(self.layers):
-            at, m = f"layers[{i}]", l.mixer
-            if self.block == "parallel" and (m.kind == "latent_attention" or (l.mlp is not None and l.mlp.kind != "dense")):
-                raise ConfigError(f"{at}: {m.kind} with this feed-forward is not available in parallel blocks")
-            for f in ("heads", "dim"):
-                positive(f"{at}.mixer.{f}", getattr(m, f))
-            if m.dim > 1024:
-                raise ConfigError(f"{at}.mixer.dim: at most 1024")
-            if m.kind in ("attention", "latent_attention") and (not isinstance(m.scale, (int, float)) or isinstance(m.scale, bool)
-                                                                or not math.isfinite(m.scale)):
-                raise ConfigError(f"{at}.mixer.scale must be a finite number")
+        def mixer(at: str, i: int, m: Mixer) -> None:
+            """at: name of the mixer's section."""
+            positive(f"{at}.heads", m.heads)
+            if m.kind != "mamba2":
+                positive(f"{at}.dim", m.dim)
+                if m.dim > 1024:
+                    raise ConfigError(f"{at}.dim: at most 1024")
+            if m.kind in ATTENTION_KINDS:
+                number(f"{at}.scale", m.scale)
             if m.kind == "attention":
-                positive(f"{at}.mixer.kv_heads", m.kv_heads)
-                positive(f"{at}.mixer.mask.size", m.window)
+                positive(f"{at}.kv_heads", m.kv_heads)
+                positive(f"{at}.mask.size", m.window)
                 if m.heads % m.kv_heads:
-                    raise ConfigError(f"{at}.mixer: kv_heads must divide heads")
+                    raise ConfigError(f"{at}: kv_heads must divide heads")
                 if m.softcap < 0 or not math.isfinite(m.softcap):
-                    raise ConfigError(f"{at}.mixer.softcap must not be negative")
+                    raise ConfigError(f"{at}.softcap must not be negative")
                 if m.rotary is not None:
-                    rotary(f"{at}.mixer", m.rotary, m.dim, "dim")
+                    rotary(at, m.rotary, m.dim, "dim")
             elif m.kind == "latent_attention":
                 for f in ("vdim", "q_rank", "kv_rank"):
-                    positive(f"{at}.mixer.{f}", getattr(m, f))
+                    positive(f"{at}.{f}", getattr(m, f))
                 if m.rot_dim != 0:
-                    positive(f"{at}.mixer.rot_dim", m.rot_dim)
+                    positive(f"{at}.rot_dim", m.rot_dim)
                 if m.kv_rank + m.rot_dim > 2048 or m.vdim > 1024:
-                    raise ConfigError(f"{at}.mixer: kv_rank + rot_dim must be at most 2048, vdim at most 1024")
+                    raise ConfigError(f"{at}: kv_rank + rot_dim must be at most 2048, vdim at most 1024")
                 if m.rotary is not None:
-                    rotary(f"{at}.mixer", m.rotary, m.rot_dim, "rot_dim")
+                    rotary(at, m.rotary, m.rot_dim, "rot_dim")
                 if (m.rotary.dims if m.rotary is not None else 0) != m.rot_dim:
-                    raise ConfigError(f"{at}.mixer.rot.dims must equal rot_dim")
+                    raise ConfigError(f"{at}.rot.dims must equal rot_dim")
                 j = m.kv_from
                 if j is not None:
                     if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < i:
-                        raise ConfigError(f"{at}.mixer.kv_from: {j!r} is not an earlier layer")
+                        raise ConfigError(f"{at}.kv_from: {j!r} is not an earlier layer")
                     src = self.layers[j].mixer
                     if (src.kind != "latent_attention" or src.kv_from is not None
                             or (src.kv_rank, src.rot_dim, src.rotary) != (m.kv_rank, m.rot_dim, m.rotary)):
-                        raise ConfigError(f"{at}.mixer.kv_from: layer {j} must cache latents of its own of the same kv_rank, "
+                        raise ConfigError(f"{at}.kv_from: layer {j} must cache latents of its own of the same kv_rank, "
                                           "rot_dim and rotation")
+            elif m.kind == "grouped_attention":
+                positive(f"{at}.kv_heads", m.kv_heads)
+                positive(f"{at}.vdim", m.vdim)
+                if m.vdim > 1024:
+                    raise ConfigError(f"{at}.vdim: at most 1024")
+                if m.heads % m.kv_heads:
+                    raise ConfigError(f"{at}: kv_heads must divide heads")
+                if m.q_temp is not None:
+                    number(f"{at}.q_temp.coef", m.q_temp.coef)
+                    positive(f"{at}.q_temp.every", m.q_temp.every, False)
+            elif m.kind == "retention":
+                positive(f"{at}.vdim", m.vdim)
+                if not isinstance(m.decay, tuple) or len(m.decay) != m.heads:
+                    raise ConfigError(f"{at}.decay: one number per head")
+                for d in m.decay:
+                    positive(f"{at}.decay", d, False)
+                if m.rotary is not None:
+                    rotary(at, m.rotary, m.dim, "dim")
+            elif m.kind == "mamba2":
+                for f in ("vdim", "state", "groups", "conv", "norm_groups"):
+                    positive(f"{at}.{f}", getattr(m, f))
+                if m.state > 1024 or m.conv > 64:
+                    raise ConfigError(f"{at}: state must be at most 1024, conv at most 64")
+                if m.heads % m.groups:
+                    raise ConfigError(f"{at}: groups must divide heads")
+                if m.out_dim % m.norm_groups:
+                    raise ConfigError(f"{at}: norm_groups must divide heads * vdim")
             else:
-                positive(f"{at}.mixer.vdim", m.vdim)
-                positive(f"{at}.mixer.gate_cap", m.gate_cap, False)
+                positive(f"{at}.vdim", m.vdim)
+                positive(f"{at}.gate_cap", m.gate_cap, False)
+
+        for i, l in enumerate(self.layers):
+            at, m = f"layers[{i}]", l.mixer
+            if self.block == "parallel" and (m.kind not in ("attention", "mlstm") or (l.mlp is not None and l.mlp.kind != "dense")):
+                raise ConfigError(f"{at}: {m.kind} with this feed-forward is not available in parallel blocks")
+            if m.kind == "parallel":
+                number(f"{at}.mixer.left_scale", m.left_scale)
+                number(f"{at}.mixer.right_scale", m.right_scale)
+                if m.left.kind != "grouped_attention" or m.right.kind != "retention":
+                    raise ConfigError(f"{at}.mixer: grouped attention beside retention is what this build combines")
+                mixer(f"{at}.mixer.left", i, m.left)
+                mixer(f"{at}.mixer.right", i, m.right)
+            else:
+                if m.kind in ("grouped_attention", "retention"):
+                    raise ConfigError(f"{at}.type: {m.kind} is one side of a parallel mixer")
+                mixer(f"{at}.mixer", i, m)
             if l.mlp is not None:
                 positive(f"{at}.mlp.ff", l.mlp.ff)
                 if l.mlp.kind == "dense":
                     if l.mlp.act not in ("silu", "relu"):
                         raise ConfigError(f"{at}.mlp.act: unknown activation {l.mlp.act!r}")
                 else:
-                    positive(f"{at}.mlp.router.experts", l.mlp.experts)
-                    positive(f"{at}.mlp.router.top", l.mlp.top)
-                    if l.mlp.top > l.mlp.experts or l.mlp.top > 32 or l.mlp.experts > 512:
-                        raise ConfigError(f"{at}.mlp.router: top must be at most experts and 32, experts at most 512")
+                    p = l.mlp
+                    positive(f"{at}.mlp.router.experts", p.experts)
+                    positive(f"{at}.mlp.router.top", p.top)
+                    if p.act not in ("relu2", "gelu"):
+                        raise ConfigError(f"{at}.mlp.act: unknown activation {p.act!r}")
+                    if p.shared_ff != 0:
+                        positive(f"{at}.mlp.shared.ff", p.shared_ff)
+                    most = 31 if p.shared_ff else 32
+                    if p.top > p.experts or p.top > most or p.experts + p.shared_parts > 512:
+                        raise ConfigError(f"{at}.mlp.router: top must be at most experts and {most}, experts (and the parts of the "
+                                          "shared one) at most 512")
             if l.weights_of is not None:
                 j = l.weights_of
                 if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < len(self.layers):
@@ -520,8 +698,8 @@ def unknown_keys(d: Mapping[str, Any], required: Sequence[str], optional: Sequen
     return set(d) - set(required) - set(optional)
 
 
-def _check_model_keys(d: Mapping[str, Any]) -> None:
-    for k in ("vocab", "width", "layers", "norm", "embedding"):
+def _check_model_keys(d: Mapping[str, Any], more: Sequence[str] = ("embedding",)) -> None:
+    for k in ("vocab", "width", "layers", "norm") + tuple(more):
         if k not in d:
             raise ConfigError(f"config.json: {k} is missing")
     if not isinstance(d["layers"], Sequence) or isinstance(d["layers"], str):
@@ -641,26 +819,97 @@ def domilix_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
             "norm": {"eps": cfg.norm_eps}, "embedding": {"scale": cfg.embedding_scale}}
 
 
+def fanulix_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> HybridConfig:
+    """The `config.json` of a Fanulix model: residual streams over layers of Mamba-2, or of softmax attention beside retention, each
+    with an optional mixture of experts."""
+    _check_model_keys(d, ("streams", "logit_scale"))
+    layers: List[HybridLayer] = []
+    for i, l in enumerate(d["layers"]):
+        at = f"layers[{i}]"
+        l = _take(l, at, ("type", "mixer"), ("mlp",))
+        if l["type"] == "mamba2":
+            mixer: Mixer = Mamba2Mixer(**_take(l["mixer"], f"{at}.mixer", ("heads", "vdim", "state", "groups", "conv", "norm_groups")))
+        elif l["type"] == "parallel":
+            m = _take(l["mixer"], f"{at}.mixer", ("left", "right", "left_scale", "right_scale"))
+            a = _take(m["left"], f"{at}.mixer.left", ("heads", "kv_heads", "dim", "vdim", "scale", "q_temp"))
+            a["q_temp"] = QueryTemperature(**_take(a["q_temp"], f"{at}.mixer.left.q_temp", ("coef", "every")))
+            r = _take(m["right"], f"{at}.mixer.right", ("heads", "dim", "vdim", "decay", "rot"))
+            rot = RotaryConfig(**_take(r.pop("rot"), f"{at}.mixer.right.rot", ("base", "dims")))
+            if not isinstance(r["decay"], Sequence) or isinstance(r["decay"], str):
+                raise ConfigError(f"{at}.mixer.right.decay is not a list")
+            r["decay"] = tuple(r["decay"])
+            mixer = ParallelMixer(GroupedAttentionMixer(**a), RetentionMixer(**r, rotary=rot), m["left_scale"], m["right_scale"])
+        else:
+            raise ConfigError(f"{at}.type: unknown mixer {l['type']!r}")
+        mlp: Optional[Mlp] = None
+        if l.get("mlp") is not None:
+            p = _take(l["mlp"], f"{at}.mlp", ("kind", "expert", "router", "shared"))
+            if p["kind"] != "moe":
+                raise ConfigError(f"{at}.mlp.kind: unknown feed-forward {p['kind']!r}")
+            r = _take(p["router"], f"{at}.mlp.router", ("experts", "top"))
+            ff = [_take(p[k], f"{at}.mlp.{k}", ("ff",))["ff"] for k in ("expert", "shared")]
+            for k, v in (("expert", ff[0]), ("shared", ff[1]), ("router", r["top"])):
+                if not isinstance(v, int) or isinstance(v, bool) or v < 1:
+                    raise ConfigError(f"{at}.mlp.{k}: {v!r} must be a positive integer")
+            mlp = MoeMlp(r["experts"], r["top"], ff[0], "gelu", False, ff[1])
+        layers.append(HybridLayer(mixer, mlp))
+    cfg = HybridConfig(d["vocab"], d["width"], tuple(layers), _take(d["norm"], "norm", ("eps",))["eps"], 1.0, dtype,
+                       architecture="Fanulix", block="streams", streams=d["streams"], tied_head=True, logit_scale=d["logit_scale"])
+    cfg.validate()
+    return cfg
+
+
+def fanulix_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
+    """The inverse of `fanulix_config_from_json`."""
+    layers = []
+    for l in cfg.layers:
+        m, p = l.mixer, l.mlp
+        if m.kind == "mamba2":
+            mixer: Dict[str, Any] = dataclasses.asdict(m)
+        else:
+            a, r = m.left, m.right
+            left = {k: getattr(a, k) for k in ("heads", "kv_heads", "dim", "vdim", "scale")}
+            left["q_temp"] = dataclasses.asdict(a.q_temp)
+            right = {"heads": r.heads, "dim": r.dim, "vdim": r.vdim, "decay": list(r.decay),
+                     "rot": {"base": r.rotary.base, "dims": r.rotary.dims}}
+            mixer = {"left": left, "right": right, "left_scale": m.left_scale, "right_scale": m.right_scale}
+        mlp = None if p is None else {"kind": "moe", "expert": {"ff": p.ff}, "router": {"experts": p.experts, "top": p.top},
+                                      "shared": {"ff": p.shared_ff}}
+        layers.append({"type": m.kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "streams": cfg.streams,
+            "layers": layers, "norm": {"eps": cfg.norm_eps}, "logit_scale": cfg.logit_scale}
+
+
+def _mixer_from_dict(d: Mapping[str, Any]) -> Mixer:
+    m = dict(d)
+    if "left" in m:
+        return ParallelMixer(**{**m, "left": _mixer_from_dict(m["left"]), "right": _mixer_from_dict(m["right"])})
+    r = m.pop("rotary", None)
+    if r is not None:
+        r = dict(r)
+        sc = r.pop("scaling", None)
+        r = RotaryConfig(**r, scaling=YarnScaling(**sc) if sc is not None else None)
+    if "q_temp" in m:
+        return GroupedAttentionMixer(**{**m, "q_temp": QueryTemperature(**m["q_temp"]) if m["q_temp"] is not None else None})
+    if "decay" in m:
+        return RetentionMixer(**{**m, "decay": tuple(m["decay"])}, rotary=r)
+    if "state" in m:
+        return Mamba2Mixer(**m)
+    if "kv_heads" in m:
+        return AttentionMixer(**m, rotary=r)
+    if "kv_rank" in m:
+        return LatentAttentionMixer(**m, rotary=r)
+    return MlstmMixer(**m)
+
+
 def hybrid_config_from_dict(d: Mapping[str, Any]) -> HybridConfig:
     """The inverse of `dataclasses.asdict(HybridConfig)` (the "model" section of an EngineConfig dictionary)."""
     d = dict(d)
     layers = []
     for l in d.pop("layers"):
-        m = dict(l["mixer"])
-        r = m.pop("rotary", None)
-        if r is not None:
-            r = dict(r)
-            sc = r.pop("scaling", None)
-            r = RotaryConfig(**r, scaling=YarnScaling(**sc) if sc is not None else None)
-        if "kv_heads" in m:
-            mixer: Mixer = AttentionMixer(**m, rotary=r)
-        elif "kv_rank" in m:
-            mixer = LatentAttentionMixer(**m, rotary=r)
-        else:
-            mixer = MlstmMixer(**m)
         p = l.get("mlp")
         mlp: Optional[Mlp] = None if p is None else MoeMlp(**p) if "experts" in p else DenseMlp(**p)
-        layers.append(HybridLayer(mixer, mlp, l.get("weights_of")))
+        layers.append(HybridLayer(_mixer_from_dict(l["mixer"]), mlp, l.get("weights_of")))
     cfg = HybridConfig(layers=tuple(layers), **d)
     cfg.validate()
     return cfg
@@ -691,6 +940,39 @@ def latent_stack(n_layers: int, width: int, heads: int, dim: int, rot_dim: int, 
         mixer = LatentAttentionMixer(heads, dim, rot_dim, vdim, q_rank, kv_rank, (dim + rot_dim) ** -0.5, rot, src)
         layers.append(HybridLayer(mixer, DenseMlp(ff, "relu") if i == 0 or experts == 0 else MoeMlp(experts, top, expert_ff)))
     cfg = HybridConfig(vocab, width, tuple(layers), 1e-5, 1.0, dtype, architecture="Domilix", block="post_norm")
+    cfg.validate()
+    return cfg
+
+
+def streams_stack(n_layers: int, width: int, streams: int, heads: int, kv_heads: int, dim: int, vdim: int, ret_heads: int,
+                  ret_dim: int, ret_vdim: int, ssm_heads: int, ssm_vdim: int, ssm_state: int, ssm_groups: int, experts: int, top: int,
+                  expert_ff: int, shared_ff: int, vocab: int, conv: int = 4, parallel_every: int = 2,
+                  dtype: str = "bfloat16") -> HybridConfig:
+    """A Fanulix-shaped decoder: one layer of attention beside retention in every `parallel_every` (the rest Mamba-2), a mixture of
+    experts in each."""
+    decay = tuple(1.0 - 2.0 ** (-5.0 - 7.0 * i / max(1, ret_heads - 1)) for i in range(ret_heads))
+    both = ParallelMixer(GroupedAttentionMixer(heads, kv_heads, dim, vdim, dim ** -0.5, QueryTemperature(0.1, 4096)),
+                         RetentionMixer(ret_heads, ret_dim, ret_vdim, decay, RotaryConfig(10000.0, ret_dim)), 0.7, 0.6)
+    ssm = Mamba2Mixer(ssm_heads, ssm_vdim, ssm_state, ssm_groups, conv, ssm_groups)
+    mlp = MoeMlp(experts, top, expert_ff, "gelu", False, shared_ff)
+    layers = tuple(HybridLayer(both if i % parallel_every == parallel_every - 1 else ssm, mlp) for i in range(n_layers))
+    cfg = HybridConfig(vocab, width, layers, 1e-6, 1.0, dtype, architecture="Fanulix", block="streams", streams=streams, tied_head=True,
+                       logit_scale=0.5)
+    cfg.validate()
+    return cfg
+
+
+def tiny_streams_config(**over: Any) -> HybridConfig:
+    """CPU-sized Fanulix-shaped decoder: attention beside retention, Mamba-2, and a Mamba-2 layer without feed-forward."""
+    both = ParallelMixer(GroupedAttentionMixer(4, 2, 20, 28, 0.21, QueryTemperature(0.25, 24)),
+                         RetentionMixer(3, 16, 20, (0.9, 0.97, 0.995), RotaryConfig(3000.0, 12)), 0.8, 0.45)
+    kw: Dict[str, Any] = dict(vocab_size=300, hidden_size=88, norm_eps=2e-5, architecture="Fanulix", block="streams", streams=2,
+                              tied_head=True, logit_scale=0.6,
+                              layers=(HybridLayer(both, MoeMlp(6, 2, 40, "gelu", False, 72)),
+                                      HybridLayer(Mamba2Mixer(4, 24, 20, 2, 4, 2), MoeMlp(5, 3, 24, "gelu", False, 24)),
+                                      HybridLayer(Mamba2Mixer(3, 16, 12, 1, 3, 1), None)))
+    kw.update(over)
+    cfg = HybridConfig(**kw)
     cfg.validate()
     return cfg
 

@@ -248,6 +248,19 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// cos and sin of position * (hi + lo): the product's rounding error and the frequency's remainder, a small angle together, are
+// added by the angle-sum formulas, so the result is good to 32-bit resolution however far the position is.
+__device__ __forceinline__ float2 cos_sin_split(long long pos, float hi, float lo) {
+  const float p = static_cast<float>(pos);
+  const float a = p * hi;
+  const float e = fmaf(p, hi, -a) + p * lo;
+  float s, c;
+  sincosf(a, &s, &c);
+  const float e2 = e * e;
+  const float se = fmaf(-e * e2, 1.f / 6.f, e), ce = fmaf(e2, fmaf(e2, 1.f / 24.f, -0.5f), 1.f);
+  return make_float2(c * ce - s * se, s * ce + c * se);
+}
+
 // Block-wide sum through shared memory (red must hold 32 floats).
 __device__ __forceinline__ float block_sum(float v, float* red) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;

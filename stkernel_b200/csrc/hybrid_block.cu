@@ -1,15 +1,16 @@
 // Residual-side kernels of the layer-by-layer decoders (models/hybrid.py): scaled embedding into an fp32 residual, residual add
-// fused with the next norm (parallel block), norm of a sublayer's output fused with the residual add (post-norm block), and the
-// feed-forward half of the joined sublayer buffer.
+// fused with the next norm (parallel block), norm of a sublayer's output fused with the residual add (post-norm block), the update
+// of several residual streams fused with the norm of their next weighted sum (streams block), and the feed-forward half of the
+// joined sublayer buffer.
 #define STK_PDL_CLASS 4
 #include "hybrid_block.cuh"
 
 namespace stk {
 
-// h != nullptr: the row also in the compute type E, zero-padded to `width` columns.
+// h != nullptr: the row also in the compute type E, zero-padded to `width` columns.  copies: the row that many times, W apart.
 template <typename E>
 __global__ void __launch_bounds__(256)
-embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed, float* __restrict__ x, long long ldx, int W,
+embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed, float* __restrict__ x, long long ldx, int copies, int W,
                     int vocab, float scale, E* __restrict__ h, long long ldh, int width, int* status) {
   pdl_wait();
   pdl_trigger();
@@ -28,8 +29,11 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
       float2 f[4];
 #pragma unroll
       for (int j = 0; j < 4; ++j) f[j] = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
-      *reinterpret_cast<float4*>(x + t * ldx + i) = make_float4(f[0].x * scale, f[0].y * scale, f[1].x * scale, f[1].y * scale);
-      *reinterpret_cast<float4*>(x + t * ldx + i + 4) = make_float4(f[2].x * scale, f[2].y * scale, f[3].x * scale, f[3].y * scale);
+      for (int c = 0; c < copies; ++c) {
+        float* to = x + t * ldx + c * W + i;
+        *reinterpret_cast<float4*>(to) = make_float4(f[0].x * scale, f[0].y * scale, f[1].x * scale, f[1].y * scale);
+        *reinterpret_cast<float4*>(to + 4) = make_float4(f[2].x * scale, f[2].y * scale, f[3].x * scale, f[3].y * scale);
+      }
       if (h != nullptr) {
         __align__(16) __nv_bfloat162 b[4];
 #pragma unroll
@@ -39,8 +43,10 @@ embed_scaled_kernel(const int64_t* __restrict__ ids, const E* __restrict__ embed
     }
     return;
   }
-  for (int i = threadIdx.x; i < W; i += blockDim.x)
-    x[t * ldx + i] = ok ? ld_act(embed + id * W + i) * scale : 0.f;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = ok ? ld_act(embed + id * W + i) * scale : 0.f;
+    for (int c = 0; c < copies; ++c) x[t * ldx + c * W + i] = v;
+  }
 }
 
 // x[r] += y[r]; h[t] = norm(x[r]) * w with r = rows ? rows[t] : t (with `rows` the sum is not written back).  The
@@ -210,6 +216,172 @@ post_norm_add_kernel(const PostNormArgs<A> a) {
   }
 }
 
+// Streams x [*, S, W] fp32: x_t <- sum_s mix[s, t] x_s + write[t] y (y as in PostNormArgs, none at all if both are null), then
+// h = layer norm (weight w, bias b) of u = sum_s read[s] x_s, in the compute type, zero-padded to `width` columns.  rows: only these
+// rows, and the streams stay as they were.
+template <typename A>
+struct StreamArgs {
+  float* x;
+  const float* y; long long ldy;
+  const A* pairs; long long ldp; const int* pair_row; const float* weights; int top;
+  const float* mix; const float* write; const float* read;
+  const float* w; const float* b; float eps;
+  A* h; long long ldh;
+  int W, width;
+  const int64_t* rows;
+};
+
+// N consecutive columns of one row: the sublayer's output, all streams, their update; returns u in `row` and adds its sum.
+template <typename A, int S, int N>
+__device__ __forceinline__ float stream_columns(const StreamArgs<A>& a, float* xr, long long r, int i, const long long* src,
+                                                const float* wt, const float (&mix)[S][S], const float (&write)[S],
+                                                const float (&read)[S], float* row, bool has_y, bool store) {
+  float v[S][N], y[N];
+#pragma unroll
+  for (int s = 0; s < S; ++s) {
+    if constexpr (N == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(xr + s * a.W + i);
+      v[s][0] = f.x; v[s][1] = f.y; v[s][2] = f.z; v[s][3] = f.w;
+    } else {
+      v[s][0] = xr[s * a.W + i];
+    }
+  }
+  if (has_y) {
+#pragma unroll
+    for (int k = 0; k < N; ++k) y[k] = 0.f;
+    if (a.pairs != nullptr) {
+      for (int j = 0; j < a.top; ++j) {
+        const A* p = a.pairs + src[j] + i;
+        if constexpr (N == 4 && sizeof(A) == 2) {
+          const uint2 q = *reinterpret_cast<const uint2*>(p);
+          const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+          const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+          y[0] = fmaf(wt[j], f0.x, y[0]); y[1] = fmaf(wt[j], f0.y, y[1]);
+          y[2] = fmaf(wt[j], f1.x, y[2]); y[3] = fmaf(wt[j], f1.y, y[3]);
+        } else {
+#pragma unroll
+          for (int k = 0; k < N; ++k) y[k] = fmaf(wt[j], ld_act(p + k), y[k]);
+        }
+      }
+    } else if constexpr (N == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(a.y + r * a.ldy + i);
+      y[0] = f.x; y[1] = f.y; y[2] = f.z; y[3] = f.w;
+    } else {
+      y[0] = a.y[r * a.ldy + i];
+    }
+  }
+  float u[N], sum = 0.f;
+#pragma unroll
+  for (int k = 0; k < N; ++k) u[k] = 0.f;
+#pragma unroll
+  for (int t = 0; t < S; ++t) {
+    float n[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      if (has_y) {
+        n[k] = write[t] * y[k];
+#pragma unroll
+        for (int s = 0; s < S; ++s) n[k] = fmaf(mix[s][t], v[s][k], n[k]);
+      } else {
+        n[k] = v[t][k];
+      }
+      u[k] = fmaf(read[t], n[k], u[k]);
+    }
+    if (store) {
+      if constexpr (N == 4) *reinterpret_cast<float4*>(xr + t * a.W + i) = make_float4(n[0], n[1], n[2], n[3]);
+      else xr[t * a.W + i] = n[0];
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < N; ++k) {
+    row[i + k] = u[k];
+    sum += u[k];
+  }
+  return sum;
+}
+
+template <typename A, int S>
+__global__ void __launch_bounds__(1024)
+stream_norm_kernel(const StreamArgs<A> a) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[32];
+  __shared__ long long src[32];
+  __shared__ float wt[32];
+  pdl_wait();
+  pdl_trigger();
+  const long long r = a.rows != nullptr ? a.rows[blockIdx.x] : static_cast<long long>(blockIdx.x);
+  const bool has_y = a.y != nullptr || a.pairs != nullptr, store = has_y && a.rows == nullptr;
+  if (a.pairs != nullptr) {
+    if (static_cast<int>(threadIdx.x) < a.top) {
+      const long long p = r * a.top + threadIdx.x;
+      const int at = a.pair_row != nullptr ? a.pair_row[p] : static_cast<int>(p);
+      src[threadIdx.x] = at < 0 ? 0 : at * a.ldp;
+      wt[threadIdx.x] = at < 0 ? 0.f : a.weights[p];
+    }
+    __syncthreads();
+  }
+  float mix[S][S], write[S], read[S];
+#pragma unroll
+  for (int s = 0; s < S; ++s) {
+    read[s] = a.read[s];
+    write[s] = has_y ? a.write[s] : 0.f;
+#pragma unroll
+    for (int t = 0; t < S; ++t) mix[s][t] = has_y ? a.mix[s * S + t] : 0.f;
+  }
+  float* xr = a.x + r * S * a.W;
+  float sum = 0.f;
+  if ((a.W & 3) == 0 && (a.ldy & 3) == 0 && (a.ldp & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4)
+      sum += stream_columns<A, S, 4>(a, xr, r, i, src, wt, mix, write, read, row, has_y, store);
+  } else {
+    for (int i = threadIdx.x; i < a.W; i += blockDim.x)
+      sum += stream_columns<A, S, 1>(a, xr, r, i, src, wt, mix, write, read, row, has_y, store);
+  }
+  const float mean = block_sum(sum, red) / static_cast<float>(a.W);          // also publishes the row
+  float q = 0.f;
+  for (int i = threadIdx.x; i < a.W; i += blockDim.x) {
+    const float d = row[i] - mean;
+    q = fmaf(d, d, q);
+  }
+  const float inv = 1.f / sqrtf(block_sum(q, red) / static_cast<float>(a.W) + a.eps);
+  A* hr = a.h + blockIdx.x * a.ldh;
+  if (sizeof(A) == 2 && (a.width & 1) == 0 && (a.ldh & 1) == 0) {
+    for (int i = threadIdx.x * 2; i < a.width; i += blockDim.x * 2) {
+      const float c = i < a.W ? fmaf((row[i] - mean) * inv, a.w[i], a.b[i]) : 0.f;
+      const float d = i + 1 < a.W ? fmaf((row[i + 1] - mean) * inv, a.w[i + 1], a.b[i + 1]) : 0.f;
+      *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(hr) + i) = __floats2bfloat162_rn(c, d);
+    }
+  } else {
+    for (int i = threadIdx.x; i < a.width; i += blockDim.x)
+      st_act(hr + i, i < a.W ? fmaf((row[i] - mean) * inv, a.w[i], a.b[i]) : 0.f);
+  }
+}
+
+template <typename A, int S>
+static int launch_stream_norm(const StreamArgs<A>& a, int T, cudaStream_t st) {
+  const size_t smem = static_cast<size_t>(a.W) * sizeof(float);
+  if (smem > 40 * 1024 &&
+      cudaFuncSetAttribute(stream_norm_kernel<A, S>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+    return -3;
+  const int threads = T > 148 || a.W <= 1024 ? 256 : (a.W <= 2048 ? 512 : 1024);
+  launch_pdl(stream_norm_kernel<A, S>, dim3(T), dim3(threads), smem, st, a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <typename A>
+static int launch_streams(const StreamArgs<A>& a, int S, int T, cudaStream_t st) {
+  switch (S) {
+    case 1: return launch_stream_norm<A, 1>(a, T, st);
+    case 2: return launch_stream_norm<A, 2>(a, T, st);
+    case 3: return launch_stream_norm<A, 3>(a, T, st);
+    case 4: return launch_stream_norm<A, 4>(a, T, st);
+    case 5: return launch_stream_norm<A, 5>(a, T, st);
+    case 6: return launch_stream_norm<A, 6>(a, T, st);
+    case 7: return launch_stream_norm<A, 7>(a, T, st);
+    default: return launch_stream_norm<A, 8>(a, T, st);
+  }
+}
+
 // out[t, mix : o0) = 0, out[t, o0 + j] = act(gate_j) * up_j for j < ff, zero up to `cols`.  relu: act is relu, else silu.
 template <typename A>
 __global__ void __launch_bounds__(256)
@@ -231,15 +403,15 @@ join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int f
 
 using namespace stk;
 
-STK_API int stk_embed_scaled(const int64_t* ids, const void* embed, int embed_fp32, float* x, long long ldx, int T, int W,
+STK_API int stk_embed_scaled(const int64_t* ids, const void* embed, int embed_fp32, float* x, long long ldx, int copies, int T, int W,
                              int vocab, float scale, void* h, long long ldh, int width, int* status, void* stream) {
   if (T <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   if (embed_fp32)
-    launch_pdl(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, ids, (const float*)embed, x, ldx, W, vocab, scale, (float*)h,
+    launch_pdl(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, ids, (const float*)embed, x, ldx, copies, W, vocab, scale, (float*)h,
                ldh, width, status);
   else
-    launch_pdl(embed_scaled_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, ids, (const __nv_bfloat16*)embed, x, ldx, W, vocab,
+    launch_pdl(embed_scaled_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, ids, (const __nv_bfloat16*)embed, x, ldx, copies, W, vocab,
                scale, (__nv_bfloat16*)h, ldh, width, status);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
@@ -308,4 +480,25 @@ STK_API int stk_post_norm_add(float* x, long long ldx, const float* y, long long
     launch_pdl(post_norm_add_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, st, a);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// x [*, streams, W].  pairs == nullptr: y [*, W] fp32 rows (neither: the streams stay as they are).  mix [streams, streams] indexed
+// [from, to], write and read [streams].  T rows are normed: all, or those in `rows`.
+STK_API int stk_stream_norm(float* x, int streams, const float* y, long long ldy, const void* pairs, long long ldp, const int* pair_row,
+                            const float* weights, int top, const float* mix, const float* write, const float* read, const float* w,
+                            const float* b, float eps, void* h, long long ldh, int W, int width, int fp32, const int64_t* rows, int T,
+                            void* stream) {
+  if (T <= 0) return 0;
+  if (streams < 1 || streams > 8 || static_cast<size_t>(W) * sizeof(float) > 200 * 1024 || top > 32 ||
+      (pairs != nullptr && y != nullptr))
+    return -2;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (fp32) {
+    const StreamArgs<float> a{x, y, ldy, (const float*)pairs, ldp, pair_row, weights, top, mix, write, read, w, b, eps, (float*)h, ldh,
+                              W, width, rows};
+    return launch_streams(a, streams, T, st);
+  }
+  const StreamArgs<__nv_bfloat16> a{x, y, ldy, (const __nv_bfloat16*)pairs, ldp, pair_row, weights, top, mix, write, read, w, b, eps,
+                                    (__nv_bfloat16*)h, ldh, W, width, rows};
+  return launch_streams(a, streams, T, st);
 }

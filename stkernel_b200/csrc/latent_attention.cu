@@ -80,7 +80,7 @@ latent_prep_kernel(const PrepArgs a) {
   for (int i = i0 + 16 * 128; i < a.rot_off; i += 128) lat_st(o + i, i < a.C ? src[i] * inv * a.wkv[i] : 0.f);
   const int pairs = a.R >> 1;
   for (int i = i0; i < pairs; i += 128) {
-    const float2 w = lat_cos_sin(pos, a.freq[i], a.freq[pairs + i]);
+    const float2 w = cos_sin_split(pos, a.freq[i], a.freq[pairs + i]);
     const float x = src[a.C + 2 * i], y = src[a.C + 2 * i + 1];
     lat_st(o + a.rot_off + 2 * i, x * w.x - y * w.y);
     lat_st(o + a.rot_off + 2 * i + 1, y * w.x + x * w.y);
@@ -114,7 +114,7 @@ latent_attn_simt_kernel(const LatArgs a, const int* __restrict__ first_pos, cons
   for (int d = threadIdx.x; d < a.rot_off; d += blockDim.x) q[d] = d < a.C ? lat_f(qa[d]) : 0.f;
   const int pairs = a.R >> 1;
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const float2 w = lat_cos_sin(pos, a.freq[i], a.freq[pairs + i]);
+    const float2 w = cos_sin_split(pos, a.freq[i], a.freq[pairs + i]);
     const float x = lat_f(qr[2 * i]), y = lat_f(qr[2 * i + 1]);
     q[a.rot_off + 2 * i] = x * w.x - y * w.y;
     q[a.rot_off + 2 * i + 1] = y * w.x + x * w.y;

@@ -22,19 +22,6 @@ struct LatArgs {
   void* out; long long ldo;                       // latent read-outs: head h at columns h * cp
 };
 
-// cos and sin of position * (hi + lo): the product's rounding error and the frequency's remainder, a small angle together, are
-// added by the angle-sum formulas, so the result is good to 32-bit resolution however far the position is.
-__device__ __forceinline__ float2 lat_cos_sin(long long pos, float hi, float lo) {
-  const float p = static_cast<float>(pos);
-  const float a = p * hi;
-  const float e = fmaf(p, hi, -a) + p * lo;
-  float s, c;
-  sincosf(a, &s, &c);
-  const float e2 = e * e;
-  const float se = fmaf(-e * e2, 1.f / 6.f, e), ce = fmaf(e2, fmaf(e2, 1.f / 24.f, -0.5f), 1.f);
-  return make_float2(c * ce - s * se, s * ce + c * se);
-}
-
 __device__ __forceinline__ float lat_f(float v) { return v; }
 __device__ __forceinline__ float lat_f(__nv_bfloat16 v) { return bf16_to_f(v); }
 __device__ __forceinline__ void lat_st(float* p, float v) { *p = v; }

@@ -1,5 +1,6 @@
-// Latent attention of prompt portions on the 5th-generation tensor cores (bf16): keys and values of the whole context are
-// expanded from the cached latents first (a plain product), then each head is ordinary causal attention.
+// Causal attention of prompt portions over the full context on the 5th-generation tensor cores (bf16).  Latent attention: keys and
+// values of the whole context are expanded from the cached latents first (a plain product), then each head is ordinary causal
+// attention.  Grouped attention: the gathered rows themselves hold the keys and values of every key/value head.
 //
 //   latent_rows          the cached rows of every request with a long span, copied out of their pages into one matrix; each
 //                        request starts on a 128-row border and is padded with zero rows to the next one
@@ -42,7 +43,12 @@ struct LpArgs {
   int h0;                                              // first head of this launch
   int dp, d_panels, r_panels, v_panels, d_steps;       // panels of 64 columns; d_steps: 16-column steps of the unrotated part
   float scale;
-  __nv_bfloat16* out; long long ldo; int vp, vdim;
+  __nv_bfloat16* out; long long ldo; int vp, vdim;     // head h's output at columns h * vp; vw columns of it are written
+  int vw;
+  int h0_kv, heads_per_kv, kv_step, k_off, v_off;      // keys of a head at columns (h - h0_kv) / heads_per_kv * kv_step + k_off
+  const float* sink;                                   // per head: score of a key without value (nullptr: none)
+  const __nv_bfloat16* ogate; long long ldog;          // element-wise output gate logits, head h at columns h * vp (nullptr: none)
+  float out_scale;
   int slots;
   int* status;
 };
@@ -65,7 +71,7 @@ __device__ __forceinline__ float lp_ex2(float x) {
 constexpr int kRowParts = 8;
 __global__ void __launch_bounds__(256)
 latent_rows_kernel(const int* __restrict__ query_start, const int* __restrict__ req_rows, const int* __restrict__ start_pos, int n_req,
-                   int min_span, const int* __restrict__ table, int bt_stride, const __nv_bfloat16* __restrict__ cache, int row,
+                   int min_span, const int* __restrict__ table, int bt_stride, const __nv_bfloat16* __restrict__ cache, int G, int row,
                    __nv_bfloat16* __restrict__ out) {
   __shared__ int found[3];
   pdl_wait();
@@ -84,18 +90,18 @@ latent_rows_kernel(const int* __restrict__ query_start, const int* __restrict__ 
   }
   __syncthreads();
   const int ri = found[0], j0 = found[1] * kLpTile, ctx = found[2];
-  const int chunks = row >> 3;
+  const int per_head = row >> 3, chunks = G * per_head;            // a page is [G][kLatPage][row], an output row [G * row]
   constexpr int kRows = kLpTile / kRowParts;
   const int part = blockIdx.y * kRows;
-  uint4* dst = reinterpret_cast<uint4*>(out + (static_cast<long long>(blockIdx.x) * kLpTile + part) * row);
+  uint4* dst = reinterpret_cast<uint4*>(out + (static_cast<long long>(blockIdx.x) * kLpTile + part) * G * row);
   const int* bt = ri >= 0 ? table + static_cast<long long>(req_rows[ri]) * bt_stride : nullptr;
   for (int e = threadIdx.x; e < kRows * chunks; e += blockDim.x) {
-    const int r = e / chunks, c = e - r * chunks, j = j0 + part + r;
+    const int r = e / chunks, ce = e - r * chunks, g = ce / per_head, c = ce - g * per_head, j = j0 + part + r;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (ri >= 0 && j < ctx) {
       const int page = bt[j / kLatPage];
       if (page >= 0)
-        v = *reinterpret_cast<const uint4*>(cache + (static_cast<long long>(page) * kLatPage + j % kLatPage) * row + c * 8);
+        v = *reinterpret_cast<const uint4*>(cache + ((static_cast<long long>(page) * G + g) * kLatPage + j % kLatPage) * row + c * 8);
     }
     dst[e] = v;
   }
@@ -174,7 +180,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       uint32_t v = 0;
       if (c < pairs && r < (i ? n_tok[1] : n_tok[0])) {
         const __nv_bfloat16* src = a.qr + static_cast<long long>(q0 + off + rr) * a.ldqr + h * a.R + 2 * c;
-        const float2 w = lat_cos_sin((i ? first[1] : first[0]) + r, a.freq[c], a.freq[pairs + c]);
+        const float2 w = cos_sin_split((i ? first[1] : first[0]) + r, a.freq[c], a.freq[pairs + c]);
         const float x = bf16_to_f(src[0]), y = bf16_to_f(src[1]);
         const __nv_bfloat162 b = __floats2bfloat162_rn(x * w.x - y * w.y, y * w.x + x * w.y);
         v = *reinterpret_cast<const uint32_t*>(&b);
@@ -201,10 +207,10 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
           if (!ok) break;
           mbar_expect_tx(&bars->full[st], kLpPanel);
           const int y = seg + b * kLpTile;
-          const int e0 = hl * (a.dp + a.v_panels * 64);
-          if (j < a.d_panels) tma_load_2d(ring + st * kLpPanel, &tm_e, &bars->full[st], e0 + j * 64, y);
+          const int e0 = (h - a.h0_kv) / a.heads_per_kv * a.kv_step;
+          if (j < a.d_panels) tma_load_2d(ring + st * kLpPanel, &tm_e, &bars->full[st], e0 + a.k_off + j * 64, y);
           else if (j < kp) tma_load_2d(ring + st * kLpPanel, &tm_r, &bars->full[st], a.rot_off + (j - a.d_panels) * 64, y);
-          else tma_load_2d(ring + st * kLpPanel, &tm_e, &bars->full[st], e0 + a.dp + (j - kp) * 64, y);
+          else tma_load_2d(ring + st * kLpPanel, &tm_e, &bars->full[st], e0 + a.v_off + (j - kp) * 64, y);
         }
       }
       if (!ok) {
@@ -309,7 +315,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const float c_in = a.scale * kLpLog2e;
     const bool flip = c_in < 0.f;                                  // a negative scale: the largest score is the smallest product
     const uint32_t masked = __float_as_uint(flip ? INFINITY : -INFINITY);
-    float m = -INFINITY, l = 0.f;
+    float m = a.sink != nullptr ? a.sink[h] * kLpLog2e : -INFINITY, l = a.sink != nullptr ? 1.f : 0.f;
     bool ok = true;
     for (int b = 0; b < t_blocks && ok; ++b) {
       ok = mbar_wait(&bars->s_full[tile], b & 1, a.status, 820);
@@ -403,25 +409,48 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       if (ok) {
         const bool row_ok = r < t_tok;
         const long long t = q0 + off + tile * kLpTile + (row_ok ? r : 0);
-        const float g = (a.gate != nullptr ? lat_sigmoid(a.gate[t * a.ldg + h]) : 1.f) / l;
+        const float g = (a.gate != nullptr ? lat_sigmoid(a.gate[t * a.ldg + h]) : 1.f) * a.out_scale / l;
         __nv_bfloat16* out = a.out + t * a.ldo + h * a.vp;
+        const __nv_bfloat16* og = a.ogate != nullptr ? a.ogate + t * a.ldog + h * a.vp : nullptr;
+        const bool vec = ((a.vp | a.vw) & 7) == 0 && (a.ldo & 7) == 0 && (og == nullptr || ((a.ldog & 7) == 0 && (reinterpret_cast<uintptr_t>(og) & 15) == 0));
         for (int c = 0; c < a.v_panels * 64; c += 16) {
           uint32_t o[16];
+          __syncwarp();
           tmem_ld_32x16(to + c, o);
           tmem_ld_wait();
-          if (row_ok) {
-            uint32_t pk[8];
+          if (!row_ok) continue;
+          if (vec) {
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-              const __nv_bfloat162 v = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * g, __uint_as_float(o[2 * j + 1]) * g);
-              pk[j] = *reinterpret_cast<const uint32_t*>(&v);
+            for (int half = 0; half < 2; ++half) {
+              if (c + half * 8 >= a.vw) continue;
+              uint4 gv = make_uint4(0, 0, 0, 0);
+              if (og != nullptr) gv = *reinterpret_cast<const uint4*>(og + c + half * 8);
+              uint32_t pk[4];
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                float x = __uint_as_float(o[half * 8 + 2 * j]) * g, y = __uint_as_float(o[half * 8 + 2 * j + 1]) * g;
+                if (og != nullptr) {
+                  const float2 z = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&gv)[j]);
+                  x = __fdividef(x, 1.f + __expf(-z.x));
+                  y = __fdividef(y, 1.f + __expf(-z.y));
+                }
+                const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+                pk[j] = *reinterpret_cast<const uint32_t*>(&v);
+              }
+              *reinterpret_cast<uint4*>(out + c + half * 8) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
             }
-            *reinterpret_cast<uint4*>(out + c) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
-            *reinterpret_cast<uint4*>(out + c + 8) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (c + j < a.vw) {
+                float x = __uint_as_float(o[j]) * g;
+                if (og != nullptr) x *= lat_sigmoid(bf16_to_f(og[c + j]));
+                out[c + j] = __float2bfloat16(x);
+              }
           }
         }
         if (row_ok)
-          for (int c = a.v_panels * 64; c < a.vp; c += 8) *reinterpret_cast<uint4*>(out + c) = make_uint4(0, 0, 0, 0);
+          for (int c = a.v_panels * 64; c < a.vw; c += 8) *reinterpret_cast<uint4*>(out + c) = make_uint4(0, 0, 0, 0);
       }
     }
   }
@@ -450,13 +479,15 @@ STK_API int stk_latent_prompt_ok(int dim, int dp, int rot, int vdim, int row, in
   return lp_slots(dp, rot, vdim) >= per;
 }
 
-// rows: total rows of the gathered matrix (a multiple of 128).
+// rows: total rows of the gathered matrix (a multiple of 128).  Pages hold `heads` blocks of [64, row]; a gathered row is theirs
+// side by side.
 STK_API int stk_latent_rows(const int* query_start, const int* req_rows, const int* start_pos, int n_req, int min_span,
-                            const int* table, int bt_stride, const void* cache, int row, void* out, long long rows, void* stream) {
+                            const int* table, int bt_stride, const void* cache, int heads, int row, void* out, long long rows,
+                            void* stream) {
   if (rows <= 0) return 0;
-  if (rows % kLpTile || row % 8) return -1;
+  if (rows % kLpTile || row % 8 || heads < 1) return -1;
   launch_pdl(latent_rows_kernel, dim3(static_cast<unsigned>(rows / kLpTile), kRowParts), dim3(256), 0, (cudaStream_t)stream, query_start,
-             req_rows, start_pos, n_req, min_span, table, bt_stride, (const __nv_bfloat16*)cache, row, (__nv_bfloat16*)out);
+             req_rows, start_pos, n_req, min_span, table, bt_stride, (const __nv_bfloat16*)cache, heads, row, (__nv_bfloat16*)out);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -477,7 +508,9 @@ STK_API int stk_latent_prompt(const void* q, long long ldq, const void* qr, long
   a.query_start = query_start; a.start_pos = start_pos; a.n_req = n_req; a.min_span = min_span;
   a.freq = freq; a.R = rot; a.rot_off = rot_off; a.h0 = h0;
   a.dp = dp; a.d_panels = dp / 64; a.r_panels = (rot + 63) / 64; a.v_panels = (vdim + 63) / 64; a.d_steps = (dim + 15) / 16;
-  a.scale = scale; a.out = (__nv_bfloat16*)out; a.ldo = ldo; a.vp = vp; a.vdim = vdim; a.status = status;
+  a.scale = scale; a.out = (__nv_bfloat16*)out; a.ldo = ldo; a.vp = vp; a.vdim = vdim; a.vw = vp; a.status = status;
+  a.h0_kv = h0; a.heads_per_kv = 1; a.kv_step = dp + a.v_panels * 64; a.k_off = 0; a.v_off = dp;
+  a.sink = nullptr; a.ogate = nullptr; a.ldog = 0; a.out_scale = 1.f;
   a.slots = lp_slots(dp, rot, vdim);
   CUtensorMap tq, te, tr;
   const long long cols = static_cast<long long>(nh) * (dp + a.v_panels * 64);
@@ -491,5 +524,41 @@ STK_API int stk_latent_prompt(const void* q, long long ldq, const void* qr, long
   // at least 118 KB: one CTA per SM, it owns all of tensor memory
   launch_pdl(latent_prompt_tc_kernel, dim3(T / (2 * kLpTile) + n_req, nh), dim3(kLpThreads), smem < 118 * 1024 ? 118 * 1024 : smem,
              (cudaStream_t)stream, tq, te, tr, a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// Whether `stk_prompt_attention` covers a layer: values of at most 128 dimensions, a ring that holds a block's keys and values.
+STK_API int stk_prompt_attention_ok(int dim, int dp, int vdim, int row, int k_col) {
+  if (row % 8 || k_col % 8 || k_col < vdim || row < k_col + dim) return 0;
+  return stk_latent_prompt_ok(dim, dp, 0, vdim, row, 0);
+}
+
+// Spans of at least min_span tokens.  q: final queries, head h at columns h * dp (zeros behind dim); rows [n_rows, kv_heads * row]:
+// gathered cached rows, per key/value head value, then key from column k_col on.  out: head h at columns h * vdim.
+STK_API int stk_prompt_attention(const void* q, long long ldq, const int* query_start, const int* start_pos, int n_req, int min_span,
+                                 const void* rows, long long n_rows, int row, int k_col, const void* gate, long long ldg, float out_scale,
+                                 const float* sink, int heads, int kv_heads, int dim, int dp, int vdim, float scale, void* out,
+                                 long long ldo, int T, int* status, void* stream) {
+  if (T <= 0) return 0;
+  if (!stk_prompt_attention_ok(dim, dp, vdim, row, k_col) || n_req < 1 || n_rows < 1 || heads < 1 || heads > 65535 || kv_heads < 1 ||
+      heads % kv_heads || ldq % 8 || n_rows >= (1ll << 31) || ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(rows)) & 15))
+    return -1;
+  LpArgs a = {};
+  a.query_start = query_start; a.start_pos = start_pos; a.n_req = n_req; a.min_span = min_span;
+  a.dp = dp; a.d_panels = dp / 64; a.r_panels = 0; a.v_panels = (vdim + 63) / 64; a.d_steps = (dim + 15) / 16;
+  a.scale = scale; a.out = (__nv_bfloat16*)out; a.ldo = ldo; a.vp = vdim; a.vdim = vdim; a.vw = vdim; a.status = status;
+  a.h0_kv = 0; a.heads_per_kv = heads / kv_heads; a.kv_step = row; a.k_off = k_col; a.v_off = 0;
+  a.sink = sink; a.ogate = (const __nv_bfloat16*)gate; a.ldog = ldg; a.out_scale = out_scale;
+  a.slots = lp_slots(dp, 0, vdim);
+  if (reinterpret_cast<uintptr_t>(out) & 15) return -1;
+  CUtensorMap tq, te;
+  const long long cols = static_cast<long long>(kv_heads) * row;
+  if (make_tmap_2d(&tq, q, 2, T, static_cast<long long>(heads) * dp, ldq, kLpTile) != 0) return -3;
+  if (make_tmap_2d(&te, rows, 2, n_rows, cols, cols, kLpTile) != 0) return -3;
+  const int smem = 2 * a.d_panels * kLpPanel + a.slots * kLpPanel + 1024 + 1024;
+  if (cudaFuncSetAttribute(latent_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
+    return -3;
+  launch_pdl(latent_prompt_tc_kernel, dim3(T / (2 * kLpTile) + n_req, heads), dim3(kLpThreads), smem < 118 * 1024 ? 118 * 1024 : smem,
+             (cudaStream_t)stream, tq, te, te, a);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

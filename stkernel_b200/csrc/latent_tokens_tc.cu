@@ -215,7 +215,7 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
   float2* cs = reinterpret_cast<float2*>(p_s);
   const bool table_fits = ntok * half * 8 <= 2 * 2 * N * 128;
   if (table_fits)
-    for (int e = threadIdx.x; e < ntok * half; e += kLtThreads) cs[e] = lat_cos_sin(p0 + e / half, a.freq[e % half], a.freq[half + e % half]);
+    for (int e = threadIdx.x; e < ntok * half; e += kLtThreads) cs[e] = cos_sin_split(p0 + e / half, a.freq[e % half], a.freq[half + e % half]);
   if (threadIdx.x < 2) flags[threadIdx.x] = 0;
   __syncthreads();
   {
@@ -231,7 +231,7 @@ latent_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const LtArg
       for (int j = 0; j < 4; ++j) {
         const int k = rc * 4 + j;
         if (k < half) {
-          const float2 w = table_fits ? cs[q * half + k] : lat_cos_sin(p0 + q, a.freq[k], a.freq[half + k]);
+          const float2 w = table_fits ? cs[q * half + k] : cos_sin_split(p0 + q, a.freq[k], a.freq[half + k]);
           const float u = bf16_to_f(src[2 * j]), y = bf16_to_f(src[2 * j + 1]);
           o[j] = __floats2bfloat162_rn(u * w.x - y * w.y, y * w.x + u * w.y);
         }

@@ -1,0 +1,139 @@
+// Linear recurrences with a scalar decay per head and token,
+//
+//   S_t = exp(g_t) S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t  (+ skip v_t)        S [D, V] fp32 per head and request row
+//
+// shared by retention (retention.cu) and Mamba-2 (mamba2.cu).  A span that starts at position 0 starts from a zero state.
+//
+//   linear_scan_kernel     token by token, any size and type: one CTA per (32 or 64 value columns, head, request), the block of the
+//                          state in registers.  A `Front` supplies a token's q and k (in shared memory), v and decay: rotation,
+//                          convolution and step sizes happen on the way in.
+//   linear_chunk_*         spans of some length, bf16 operands (linear_scan.cu)
+#pragma once
+#include "hybrid_block.cuh"
+
+namespace stk {
+
+struct ScanArgs {
+  const int* query_start; const int* req_rows; const int* start_pos; int n_req;
+  float* S; float* o;                             // state [rows, H, D, V]; outputs [T, H, V]
+  int H, D, V;
+};
+
+constexpr int kScanThreads = 256, kScanRows = 8;
+
+// Front: static constexpr bool kValues (v comes through shared memory);
+//   float2 fill(t, i, pos, row, h, col0, cols, q, k, x)  token t = the i-th of its span; all threads; returns the decay and what its
+//                                                        rounding left over (a fixed decay's error would add up over the tokens)
+//   float value(t, h, col)                               v when !kValues
+//   float skip(h)                                        factor of v in the output
+template <typename Front, int NR, int VEC>
+__global__ void __launch_bounds__(kScanThreads)
+linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr int kCols = 32 * VEC;
+  float* q = sm;                                  // [D]
+  float* k = q + a.D;                             // [D]
+  float* x = k + a.D;                             // [kCols]
+  float* part = x + kCols;                        // [8][kCols]
+  pdl_wait();
+  pdl_trigger();
+  const int vb = blockIdx.x, h = blockIdx.y, ri = blockIdx.z;
+  const int q0 = a.query_start[ri], span = a.query_start[ri + 1] - q0;
+  if (span <= 0 || span < min_span || span > max_span) return;
+  const long long row = a.req_rows[ri];
+  const int start = a.start_pos[ri];
+  const int lane = threadIdx.x & 31, r = threadIdx.x >> 5;
+  const int col = vb * kCols + lane * VEC;
+  float* gS = a.S + (row * a.H + h) * static_cast<long long>(a.D) * a.V + col;
+  float S[NR][VEC];
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = r + j * kScanRows;
+    const bool in = start != 0 && d < a.D;
+    if (VEC == 2 && in && col + 1 < a.V) {
+      const float2 s = *reinterpret_cast<const float2*>(gS + static_cast<long long>(d) * a.V);
+      S[j][0] = s.x;
+      S[j][VEC - 1] = s.y;
+    } else {
+#pragma unroll
+      for (int c = 0; c < VEC; ++c) S[j][c] = in && col + c < a.V ? gS[static_cast<long long>(d) * a.V + c] : 0.f;
+    }
+  }
+  const float skip = f.skip(h);
+  for (int i = 0; i < span; ++i) {
+    const long long t = q0 + i;
+    __syncthreads();
+    const float2 decay = f.fill(t, i, start + i, row, h, vb * kCols, min(kCols, a.V - vb * kCols), q, k, x);
+    float v[VEC];
+    if (!Front::kValues) {
+#pragma unroll
+      for (int c = 0; c < VEC; ++c) v[c] = col + c < a.V ? f.value(t, h, col + c) : 0.f;
+    }
+    __syncthreads();
+    if (Front::kValues) {
+#pragma unroll
+      for (int c = 0; c < VEC; ++c) v[c] = col + c < a.V ? x[lane * VEC + c] : 0.f;
+    }
+    float acc[VEC];
+#pragma unroll
+    for (int c = 0; c < VEC; ++c) acc[c] = 0.f;
+#pragma unroll
+    for (int j = 0; j < NR; ++j) {
+      const int d = r + j * kScanRows;
+      if (d < a.D) {
+        const float kd = k[d], qd = q[d];
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) {
+          S[j][c] = fmaf(decay.x, S[j][c], fmaf(decay.y, S[j][c], kd * v[c]));
+          acc[c] = fmaf(qd, S[j][c], acc[c]);
+        }
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < VEC; ++c) part[r * kCols + lane * VEC + c] = acc[c];
+    __syncthreads();
+    const int oc = threadIdx.x;
+    if (oc < kCols && vb * kCols + oc < a.V) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < kScanRows; ++w) s += part[w * kCols + oc];
+      if (Front::kValues) s = fmaf(skip, x[oc], s);
+      a.o[(t * a.H + h) * a.V + vb * kCols + oc] = s;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = r + j * kScanRows;
+    if (d >= a.D) continue;
+    if (VEC == 2 && col + 1 < a.V) {
+      *reinterpret_cast<float2*>(gS + static_cast<long long>(d) * a.V) = make_float2(S[j][0], S[j][VEC - 1]);
+    } else {
+#pragma unroll
+      for (int c = 0; c < VEC; ++c)
+        if (col + c < a.V) gS[static_cast<long long>(d) * a.V + c] = S[j][c];
+    }
+  }
+}
+
+template <typename Front, int NR, int VEC>
+static int launch_scan_as(const Front& f, const ScanArgs& a, int min_span, int max_span, cudaStream_t st) {
+  constexpr int kCols = 32 * VEC;
+  const size_t smem = static_cast<size_t>(2 * a.D + (1 + kScanRows) * kCols) * sizeof(float);
+  launch_pdl(linear_scan_kernel<Front, NR, VEC>, dim3((a.V + kCols - 1) / kCols, a.H, a.n_req), dim3(kScanThreads), smem, st, f, a,
+             min_span, max_span);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// Spans of min_span .. max_span tokens, D up to 1024.
+template <typename Front>
+static int launch_scan(const Front& f, const ScanArgs& a, int min_span, int max_span, cudaStream_t st) {
+  if (a.H < 1 || a.H > 65535 || a.D < 1 || a.D > 1024 || a.V < 1 || a.n_req > 65535) return -1;
+  if (a.n_req <= 0) return 0;
+  const bool two = a.V >= 64 && a.V % 2 == 0;
+  if (a.D <= 64) return two ? launch_scan_as<Front, 8, 2>(f, a, min_span, max_span, st) : launch_scan_as<Front, 8, 1>(f, a, min_span, max_span, st);
+  if (a.D <= 128) return two ? launch_scan_as<Front, 16, 2>(f, a, min_span, max_span, st) : launch_scan_as<Front, 16, 1>(f, a, min_span, max_span, st);
+  if (a.D <= 256) return launch_scan_as<Front, 32, 1>(f, a, min_span, max_span, st);
+  return launch_scan_as<Front, 128, 1>(f, a, min_span, max_span, st);
+}
+
+}  // namespace stk

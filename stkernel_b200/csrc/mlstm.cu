@@ -18,11 +18,11 @@
 //                       tensor cores with the fp32 operand of each product as a bf16 pair (16 mantissa bits).
 // Sums of log gates reach hundreds, so they are formed in fp64 and kept as integer part + remainder: differences lose nothing.
 #define STK_PDL_CLASS 16
+#include "chunk_mma.cuh"
 #include "hybrid_block.cuh"
 
 namespace stk {
 
-constexpr int kChunk = 64;
 constexpr int kGateSlot = 3 * kChunk + 8;      // a (integer, remainder), F; A, F_end, m_start, M_end as (integer, remainder) pairs
 
 struct MlstmArgs {
@@ -127,101 +127,6 @@ mlstm_scan_kernel(const MlstmArgs a, int min_span, int max_span) {
 }
 
 // ---- chunks -------------------------------------------------------------------------------------------
-__device__ __forceinline__ void mls_ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mls_ldsm4_t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mls_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void mls_split(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) {
-  hi = __float2bfloat16(x);
-  lo = __float2bfloat16(x - bf16_to_f(hi));
-}
-__device__ __forceinline__ void mls_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 r = __floats2bfloat162_rn(x - f.x, y - f.y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&r);
-}
-
-// chunk index of the step -> (request, first chunk of the request, tokens [t0, t0 + n) of the step); false past the end
-struct ChunkRef { int ri, first, t0, n; };
-__device__ __forceinline__ bool find_chunk(const MlstmArgs& a, int min_span, int ci, ChunkRef& c) {
-  int base = 0;
-  for (int i = 0; i < a.n_req; ++i) {
-    const int q0 = a.query_start[i], span = a.query_start[i + 1] - q0;
-    if (span < min_span) continue;
-    const int nc = (span + kChunk - 1) / kChunk;
-    if (ci < base + nc) {
-      c.ri = i;
-      c.first = base;
-      c.t0 = q0 + (ci - base) * kChunk;
-      c.n = min(kChunk, span - (ci - base) * kChunk);
-      return true;
-    }
-    base += nc;
-  }
-  return false;
-}
-
-// rows [0, 64) x cols [0, width) of head columns into shared memory; rows >= n and columns >= width up to `cols` are zero
-__device__ __forceinline__ void load_rows(__nv_bfloat16* dst, int stride, int cols, const __nv_bfloat16* src, long long ld, int n,
-                                          int width, int nthreads) {
-  if ((width & 7) == 0 && (cols & 7) == 0 && (ld & 7) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
-    const int ch = cols >> 3;
-    for (int e = threadIdx.x; e < kChunk * ch; e += nthreads) {
-      const int r = e / ch, c = (e - r * ch) * 8;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (r < n && c < width) v = *reinterpret_cast<const uint4*>(src + r * ld + c);
-      *reinterpret_cast<uint4*>(dst + r * stride + c) = v;
-    }
-  } else {
-    for (int e = threadIdx.x; e < kChunk * cols; e += nthreads) {
-      const int r = e / cols, c = e - r * cols;
-      dst[r * stride + c] = r < n && c < width ? src[r * ld + c] : __float2bfloat16(0.f);
-    }
-  }
-}
-
-__device__ __forceinline__ void mls_cp16(void* dst, const void* src, bool valid) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void mls_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void mls_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-// Like load_rows, but asynchronous when the rows are 16-byte aligned.
-__device__ __forceinline__ void load_rows_async(__nv_bfloat16* dst, int stride, int cols, const __nv_bfloat16* src, long long ld,
-                                                int n, int width, int nthreads) {
-  if ((width & 7) == 0 && (cols & 7) == 0 && (ld & 7) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
-    const int ch = cols >> 3;
-    for (int e = threadIdx.x; e < kChunk * ch; e += nthreads) {
-      const int r = e / ch, c = (e - r * ch) * 8;
-      const bool ok = r < n && c < width;
-      mls_cp16(dst + r * stride + c, ok ? src + r * ld + c : src, ok);
-    }
-  } else {
-    load_rows(dst, stride, cols, src, ld, n, width, nthreads);
-  }
-}
-
-// chunks of request ri begin at this index of the step's chunk numbering
-__device__ __forceinline__ int first_chunk(const MlstmArgs& a, int min_span, int ri) {
-  int first = 0;
-  for (int i = 0; i < ri; ++i) {
-    const int s = a.query_start[i + 1] - a.query_start[i];
-    if (s >= min_span) first += (s + kChunk - 1) / kChunk;
-  }
-  return first;
-}
-
 // A chunk's state before its first token: [D][Vp] high parts, [D][Vp] remainders (bf16), then n[D] fp32; Vp = V rounded up to 8.
 // Slots are whole 16-byte units.
 __host__ __device__ inline long long state_slot_floats(int D, int V) {
@@ -236,7 +141,7 @@ mlstm_chunk_gates_kernel(const MlstmArgs a, int min_span, float* __restrict__ ga
   const int h = blockIdx.x, ri = blockIdx.y;
   const int q0 = a.query_start[ri], span = a.query_start[ri + 1] - q0;
   if (span < min_span || span <= 0) return;
-  const int first = first_chunk(a, min_span, ri), nc = (span + kChunk - 1) / kChunk;
+  const int first = first_chunk(a.query_start, min_span, ri), nc = (span + kChunk - 1) / kChunk;
   const int warp = threadIdx.x >> 5, l = threadIdx.x & 31;
   for (int c = warp; c < nc; c += 8) {
     const int t0 = q0 + c * kChunk, n = min(kChunk, span - c * kChunk);
@@ -305,8 +210,6 @@ mlstm_chunk_gates_kernel(const MlstmArgs a, int min_span, float* __restrict__ ga
 }
 
 // (2) states.  One CTA: 64 memory rows x 64 value columns of one head of one request, all its chunks in order.
-constexpr int kStStride = 72;
-
 __global__ void __launch_bounds__(128)
 mlstm_chunk_state_kernel(const MlstmArgs a, int min_span, const float* __restrict__ gate_ws, float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -322,7 +225,7 @@ mlstm_chunk_state_kernel(const MlstmArgs a, int min_span, const float* __restric
   const int vb = blockIdx.x, db = blockIdx.y, h = blockIdx.z % a.H, ri = blockIdx.z / a.H;
   const int q0 = a.query_start[ri], span = a.query_start[ri + 1] - q0;
   if (span < min_span || span <= 0) return;
-  const int first = first_chunk(a, min_span, ri), nc = (span + kChunk - 1) / kChunk;
+  const int first = first_chunk(a.query_start, min_span, ri), nc = (span + kChunk - 1) / kChunk;
   const long long row = a.req_rows[ri];
   const bool fresh = a.start_pos[ri] == 0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -462,7 +365,7 @@ mlstm_chunk_out_kernel(const MlstmArgs a, int min_span, const float* __restrict_
   pdl_wait();
   pdl_trigger();
   const int vb = blockIdx.x, ci = blockIdx.y, h = blockIdx.z;
-  if (threadIdx.x == 0) s_ok = find_chunk(a, min_span, ci, s_c) ? 1 : 0;
+  if (threadIdx.x == 0) s_ok = find_chunk(a.query_start, a.n_req, min_span, ci, s_c) ? 1 : 0;
   __syncthreads();
   if (!s_ok) return;
   const ChunkRef c = s_c;

@@ -1,4 +1,5 @@
-// Mixture-of-experts feed-forward with ungated experts, y = W_down relu(W_up x)^2, weights in the compute type (bf16 or fp32).
+// Mixture-of-experts feed-forward with ungated experts, y = W_down act(W_up x), act relu squared or the exact gelu, weights in the
+// compute type (bf16 or fp32).
 //
 //   expert_rows      one CTA per (pair, block of output rows): a warp streams whole weight rows and dots them with the pair's
 //                    activations, fp32 accumulation.  A handful of pairs, and every batch of a float32 model.
@@ -36,11 +37,18 @@ template <> struct Vec16<__nv_bfloat16> {
 
 constexpr int kRowsPerWarp = 4, kExpertWarps = 8;
 
-// out[pair, n] = act(x[pair / div] . W[expert(pair), n]) for n < N, zeros up to n_pad.  act: relu squared when `square`.
+// act 0: none, 1: relu squared, 2: gelu (exact)
+__device__ __forceinline__ float expert_act(float v, int act) {
+  if (act == 1) return v > 0.f ? v * v : 0.f;
+  if (act == 2) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  return v;
+}
+
+// out[pair, n] = act(x[pair / div] . W[expert(pair), n]) for n < N, zeros up to n_pad.
 template <typename A>
 __global__ void __launch_bounds__(kExpertWarps * 32)
 expert_rows_kernel(const A* __restrict__ x, long long ldx, int div, const A* __restrict__ W, long long estride,
-                   const int* __restrict__ ids, int E, A* __restrict__ out, long long ldo, int N, int n_pad, int K, int square) {
+                   const int* __restrict__ ids, int E, A* __restrict__ out, long long ldo, int N, int n_pad, int K, int act) {
   using V = Vec16<A>;
   pdl_wait();
   pdl_trigger();
@@ -68,7 +76,7 @@ expert_rows_kernel(const A* __restrict__ x, long long ldx, int div, const A* __r
 #pragma unroll
   for (int r = 0; r < kRowsPerWarp; ++r) {
     float v = warp_sum(acc[r]);
-    if (square) v = v > 0.f ? v * v : 0.f;
+    v = expert_act(v, act);
     if (lane == 0 && n0 + r < n_pad) out[pair * ldo + n0 + r] = V::round(ok && n0 + r < N ? v : 0.f);
   }
 }
@@ -93,7 +101,7 @@ struct ExpertArgs {
   int E, N, k_blocks, tiles_n;
   __nv_bfloat16* out;      // [P, ldo]
   long long ldo;
-  int square;
+  int act;
   int* status;
 };
 constexpr int kMaxExperts = 512;
@@ -123,12 +131,8 @@ __device__ __forceinline__ void expert_tiles(int* first, const int* offsets, int
   }
 }
 
-__device__ __forceinline__ uint32_t expert_pack(uint32_t a, uint32_t b, int square) {
-  float x = __uint_as_float(a), y = __uint_as_float(b);
-  if (square) {
-    x = x > 0.f ? x * x : 0.f;
-    y = y > 0.f ? y * y : 0.f;
-  }
+__device__ __forceinline__ uint32_t expert_pack(uint32_t a, uint32_t b, int act) {
+  const float x = expert_act(__uint_as_float(a), act), y = expert_act(__uint_as_float(b), act);
   const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
   return *reinterpret_cast<const uint32_t*>(&v);
 }
@@ -231,11 +235,7 @@ experts_slim_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
         if (n < a.N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (c + j < valid) {
-              float f = __uint_as_float(v[j]);
-              if (a.square) f = f > 0.f ? f * f : 0.f;
-              o[(c + j) * a.ldo] = __float2bfloat16(f);
-            }
+            if (c + j < valid) o[(c + j) * a.ldo] = __float2bfloat16(expert_act(__uint_as_float(v[j]), a.act));
         }
       }
       tc_fence_before();
@@ -354,8 +354,8 @@ experts_wide_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
             for (int j = 0; j < 32; j += 8)
               if (tn * 256 + col + j < a.N)                          // N is a multiple of 8
                 *reinterpret_cast<uint4*>(o + col + j) =
-                    make_uint4(expert_pack(v[j], v[j + 1], a.square), expert_pack(v[j + 2], v[j + 3], a.square),
-                               expert_pack(v[j + 4], v[j + 5], a.square), expert_pack(v[j + 6], v[j + 7], a.square));
+                    make_uint4(expert_pack(v[j], v[j + 1], a.act), expert_pack(v[j + 2], v[j + 3], a.act),
+                               expert_pack(v[j + 4], v[j + 5], a.act), expert_pack(v[j + 6], v[j + 7], a.act));
           }
         }
       }
@@ -387,7 +387,7 @@ using namespace stk;
 
 // x rows of K elements (K a multiple of 16 bytes' worth, rows 16-byte aligned), W [E, N, K].
 STK_API int stk_expert_rows(const void* x, long long ldx, int div, const void* W, const int* ids, int E, void* out, long long ldo,
-                            int N, int n_pad, int K, int square, int fp32, int n_pairs, void* stream) {
+                            int N, int n_pad, int K, int act, int fp32, int n_pairs, void* stream) {
   if (n_pairs <= 0) return 0;
   const int v = fp32 ? 4 : 8;
   if (K % v || ldx % v || div < 1 || N < 1 || n_pad < N || E < 1) return -1;
@@ -399,11 +399,11 @@ STK_API int stk_expert_rows(const void* x, long long ldx, int div, const void* W
     const int n = min(n_pairs - p0, 65520 / div * div);
     if (fp32)
       launch_pdl(expert_rows_kernel<float>, dim3(bx, n), dim3(kExpertWarps * 32), 0, st, (const float*)x + (long long)(p0 / div) * ldx,
-                 ldx, div, (const float*)W, (long long)N * K, ids + p0, E, (float*)out + (long long)p0 * ldo, ldo, N, n_pad, K, square);
+                 ldx, div, (const float*)W, (long long)N * K, ids + p0, E, (float*)out + (long long)p0 * ldo, ldo, N, n_pad, K, act);
     else
       launch_pdl(expert_rows_kernel<__nv_bfloat16>, dim3(bx, n), dim3(kExpertWarps * 32), 0, st,
                  (const __nv_bfloat16*)x + (long long)(p0 / div) * ldx, ldx, div, (const __nv_bfloat16*)W, (long long)N * K, ids + p0, E,
-                 (__nv_bfloat16*)out + (long long)p0 * ldo, ldo, N, n_pad, K, square);
+                 (__nv_bfloat16*)out + (long long)p0 * ldo, ldo, N, n_pad, K, act);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
@@ -418,7 +418,7 @@ STK_API int stk_expert_gather(const void* x, long long ldx, const int* sorted, i
 
 // xs [n_pairs, K] sorted by expert, W [E, N, K], out [n_pairs, ldo]; bf16.  The tile follows the average number of pairs an expert has.
 STK_API int stk_experts(const void* xs, int n_pairs, const void* W, const int* offsets, int E, int N, int K, void* out, long long ldo,
-                        int square, int sm_count, int* status, void* stream) {
+                        int act, int sm_count, int* status, void* stream) {
   if (n_pairs <= 0) return 0;
   if (E < 1 || E > kMaxExperts || N % 8 || K % 8 || ldo % 8 || static_cast<long long>(E) * N >= (1ll << 31) ||
       ((reinterpret_cast<uintptr_t>(xs) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out)) & 15))
@@ -431,7 +431,7 @@ STK_API int stk_experts(const void* xs, int n_pairs, const void* W, const int* o
   if (make_tmap_2d(&tx, xs, 2, n_pairs, K, K, wide ? 128 : bt) != 0) return -2;
   ExpertArgs a;
   a.offsets = offsets; a.E = E; a.N = N; a.k_blocks = (K + 63) / 64; a.tiles_n = wide ? (N + 255) / 256 : (N + 127) / 128;
-  a.out = (__nv_bfloat16*)out; a.ldo = ldo; a.square = square; a.status = status;
+  a.out = (__nv_bfloat16*)out; a.ldo = ldo; a.act = act; a.status = status;
   cudaStream_t st = (cudaStream_t)stream;
   // no more CTAs than there can be tiles
   const int rows = wide ? 256 : bt;

@@ -1,0 +1,185 @@
+// Retention: a linear recurrence (linear_scan.cuh) with a fixed decay per head over rotated queries and keys; every head's read-out
+// is divided by its root mean square and multiplied with silu of a gate.
+//
+//   retention_scan       decode rows, short spans, float32: rotation in fp32 on the way into the recurrence
+//   rotate_qk            long spans: rotated queries and scaled, rotated keys as bf16 pairs for the chunked form
+//   retention_finish     head norm, gate, factor
+#define STK_PDL_CLASS 16
+#include "linear_scan.cuh"
+
+namespace stk {
+
+struct RotArgs {
+  const void* proj; long long ldp; int q_off, k_off;
+  const float* freq; int pairs;                   // [2][pairs]: dimension i turns with i + pairs
+  float k_scale;
+};
+
+// Element d of a head after its rotation at position pos.
+template <typename A>
+__device__ __forceinline__ float rotated(const RotArgs& r, const A* x, int d, long long pos) {
+  const float v = ld_act(x + d);
+  if (d >= 2 * r.pairs) return v;
+  const int i = d < r.pairs ? d : d - r.pairs;
+  const float2 w = cos_sin_split(pos, r.freq[i], r.freq[r.pairs + i]);
+  return d < r.pairs ? v * w.x - ld_act(x + d + r.pairs) * w.y : v * w.x + ld_act(x + d - r.pairs) * w.y;
+}
+
+template <typename A>
+struct RetentionFront {
+  static constexpr bool kValues = false;
+  RotArgs r;
+  int v_off, D, V;
+  const float* decay;                             // [2][H]: the decays and what their rounding left over
+  int H;
+  __device__ __forceinline__ float skip(int) const { return 0.f; }
+  __device__ __forceinline__ float value(long long t, int h, int col) const {
+    return ld_act(reinterpret_cast<const A*>(r.proj) + t * r.ldp + v_off + h * V + col);
+  }
+  __device__ __forceinline__ float2 fill(long long t, int, long long pos, long long, int h, int, int, float* q, float* k, float*) const {
+    const A* p = reinterpret_cast<const A*>(r.proj) + t * r.ldp;
+    for (int e = threadIdx.x; e < 2 * D; e += kScanThreads) {
+      if (e < D) q[e] = rotated(r, p + r.q_off + h * D, e, pos);
+      else k[e - D] = rotated(r, p + r.k_off + h * D, e - D, pos) * r.k_scale;
+    }
+    return make_float2(decay[h], decay[H + h]);
+  }
+};
+
+// out [T][q high | q remainder | k high | k remainder][H * D8], zeros behind each head's D columns.  One CTA per token; the cos and
+// sin of its position are formed once for all heads.
+__global__ void __launch_bounds__(256)
+rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bfloat16* __restrict__ out, int H, int D, int D8) {
+  extern __shared__ float2 cs[];
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.x;
+  const long long pos = positions[t] < 0 ? 0 : positions[t];
+  for (int i = threadIdx.x; i < r.pairs; i += blockDim.x) cs[i] = cos_sin_split(pos, r.freq[i], r.freq[r.pairs + i]);
+  __syncthreads();
+  const __nv_bfloat16* p = reinterpret_cast<const __nv_bfloat16*>(r.proj) + t * r.ldp;
+  const int n = H * D8;
+  __nv_bfloat16* o = out + t * 4 * n;
+  for (int e = threadIdx.x; e < n; e += blockDim.x) {               // two columns, e / (D8 / 2) the (q or k, head)
+    const int half = D8 / 2, u = e / half, d0 = (e - u * half) * 2, isk = u >= H ? 1 : 0, h = u - isk * H;
+    const __nv_bfloat16* x = p + (isk ? r.k_off : r.q_off) + h * D;
+    float y[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int d = d0 + j;
+      float f = 0.f;
+      if (d < D) {
+        f = bf16_to_f(x[d]);
+        if (d < 2 * r.pairs) {
+          const float2 w = cs[d < r.pairs ? d : d - r.pairs];
+          f = d < r.pairs ? f * w.x - bf16_to_f(x[d + r.pairs]) * w.y : f * w.x + bf16_to_f(x[d - r.pairs]) * w.y;
+        }
+        if (isk) f *= r.k_scale;
+      }
+      y[j] = f;
+    }
+    const __nv_bfloat162 hi = __floats2bfloat162_rn(y[0], y[1]);
+    const float2 hf = __bfloat1622float2(hi);
+    __nv_bfloat16* dst = o + isk * 2 * n + h * D8 + d0;
+    *reinterpret_cast<__nv_bfloat162*>(dst) = hi;
+    *reinterpret_cast<__nv_bfloat162*>(dst + n) = __floats2bfloat162_rn(y[0] - hf.x, y[1] - hf.y);
+  }
+}
+
+// out[t, col + h * V + c] = o / rms(o over the head) * silu(g) * scale: one warp per (token, head).  Zeros into the columns left .. col
+// and behind the last head.
+template <typename A>
+__global__ void __launch_bounds__(256)
+retention_finish_kernel(const float* __restrict__ o, float eps, const int* __restrict__ tok_req, const int64_t* __restrict__ positions,
+                        const A* __restrict__ proj, long long ldp, int g_off, float scale, A* __restrict__ out, long long ldo, int left,
+                        int col, int cols, int H, int V, int T) {
+  pdl_wait();
+  pdl_trigger();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long th = blockIdx.x * 8ll + warp;
+  if (th >= static_cast<long long>(T) * H) return;
+  const long long t = th / H;
+  const int h = static_cast<int>(th - t * H);
+  A* to = out + t * ldo;
+  if (h == 0)
+    for (int c = left + lane; c < col; c += 32) st_act(to + c, 0.f);
+  if (h == H - 1)
+    for (int c = col + H * V + lane; c < cols; c += 32) st_act(to + c, 0.f);
+  to += col + h * V;
+  if (tok_req[t] < 0 || positions[t] < 0) {
+    for (int c = lane; c < V; c += 32) st_act(to + c, 0.f);
+    return;
+  }
+  const float* x = o + th * V;
+  const A* g = proj + t * ldp + g_off + h * V;
+  float ss = 0.f;
+  if (sizeof(A) == 2 && ((V | ldp | ldo | g_off | col) & 3) == 0) {
+    for (int c = lane * 4; c < V; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(x + c);
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+    const float r = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
+    for (int c = lane * 4; c < V; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(x + c);
+      const uint2 gu = *reinterpret_cast<const uint2*>(g + c);
+      const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu.x));
+      const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu.y));
+      uint2 pk;
+      *reinterpret_cast<__nv_bfloat162*>(&pk.x) =
+          __floats2bfloat162_rn(v.x * r * g0.x / (1.f + __expf(-g0.x)), v.y * r * g0.y / (1.f + __expf(-g0.y)));
+      *reinterpret_cast<__nv_bfloat162*>(&pk.y) =
+          __floats2bfloat162_rn(v.z * r * g1.x / (1.f + __expf(-g1.x)), v.w * r * g1.y / (1.f + __expf(-g1.y)));
+      *reinterpret_cast<uint2*>(to + c) = pk;
+    }
+    return;
+  }
+  for (int c = lane; c < V; c += 32) ss = fmaf(x[c], x[c], ss);
+  const float r = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
+  for (int c = lane; c < V; c += 32) {
+    const float z = ld_act(g + c);
+    st_act(to + c, x[c] * r * z / (1.f + expf(-z)));
+  }
+}
+
+}  // namespace stk
+
+using namespace stk;
+
+// Spans of min_span .. max_span tokens, token by token.
+STK_API int stk_retention_scan(const void* proj, long long ldp, int q_off, int k_off, int v_off, const float* freq, int pairs,
+                               float k_scale, const float* decay, const int* query_start, const int* req_rows, const int* start_pos,
+                               int n_req, float* S, float* o, int heads, int dim, int vdim, int fp32, int min_span, int max_span, int T,
+                               void* stream) {
+  if (T <= 0) return 0;
+  if (pairs < 0 || 2 * pairs > dim) return -1;
+  const ScanArgs a{query_start, req_rows, start_pos, n_req, S, o, heads, dim, vdim};
+  const RotArgs r{proj, ldp, q_off, k_off, freq, pairs, k_scale};
+  if (fp32) return launch_scan(RetentionFront<float>{r, v_off, dim, vdim, decay, heads}, a, min_span, max_span, (cudaStream_t)stream);
+  return launch_scan(RetentionFront<__nv_bfloat16>{r, v_off, dim, vdim, decay, heads}, a, min_span, max_span, (cudaStream_t)stream);
+}
+
+// out [T, 4, heads * d8] bf16: see rotate_qk_kernel.
+STK_API int stk_rotate_qk(const void* proj, long long ldp, int q_off, int k_off, const float* freq, int pairs, float k_scale,
+                          const int64_t* positions, void* out, int heads, int dim, int d8, int T, void* stream) {
+  if (T <= 0) return 0;
+  if (pairs < 0 || 2 * pairs > dim || d8 < dim || d8 % 8) return -1;
+  const RotArgs r{proj, ldp, q_off, k_off, freq, pairs, k_scale};
+  launch_pdl(rotate_qk_kernel, dim3(T), dim3(256), static_cast<size_t>(pairs) * sizeof(float2), (cudaStream_t)stream, r, positions,
+             (__nv_bfloat16*)out, heads, dim, d8);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+STK_API int stk_retention_finish(const float* o, float eps, const int* tok_req, const int64_t* positions, const void* proj, long long ldp,
+                                 int g_off, float scale, void* out, long long ldo, int left, int col, int cols, int fp32, int heads,
+                                 int vdim, int T, void* stream) {
+  if (T <= 0) return 0;
+  const dim3 grid(static_cast<unsigned>((static_cast<long long>(T) * heads + 7) / 8));
+  cudaStream_t st = (cudaStream_t)stream;
+  if (fp32)
+    launch_pdl(retention_finish_kernel<float>, grid, dim3(256), 0, st, o, eps, tok_req, positions, (const float*)proj, ldp, g_off, scale,
+               (float*)out, ldo, left, col, cols, heads, vdim, T);
+  else
+    launch_pdl(retention_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, eps, tok_req, positions, (const __nv_bfloat16*)proj, ldp,
+               g_off, scale, (__nv_bfloat16*)out, ldo, left, col, cols, heads, vdim, T);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}

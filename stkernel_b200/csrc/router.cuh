@@ -5,6 +5,7 @@
 // scores = sigmoid | sqrt(softplus) of the fp32 gate logits; selection by score + bias (or by a token-id hash table
 // with bounds checks); weights from the unbiased score, renormalised and scaled (topkGatingSoftplusSqrt /
 // fused_topk_bias and the hash-MoE lookup of overlay/nvidia_model.py:806-827).
+// `always` experts E, E + 1, ... are taken by every token with weight 1, behind the chosen ones.
 // Scoring 2 (softmax over the chosen): score = logit + bias, weights = softmax of the selected scores.
 #pragma once
 #include "common.cuh"
@@ -16,9 +17,9 @@ struct RouterArgs {
   const int* tid2eid;         // [vocab, topk] or nullptr
   const int64_t* token_ids;   // [T] (hash routing)
   int vocab;
-  int* ids;                   // [T, topk]
-  float* weights;             // [T, topk]
-  int E, topk, scoring, renorm;
+  int* ids;                   // [T, topk + always]
+  float* weights;             // [T, topk + always]
+  int E, topk, always, scoring, renorm;
   float scaling;
   int* status;
 };
@@ -108,11 +109,13 @@ __device__ __forceinline__ void route_token_impl(const RouterArgs& r, const floa
       if (lane == j) { my_w = s; my_id = best_e; }
     }
   }
-  if (lane < r.topk) {
+  const int n = r.topk + r.always;
+  if (lane < n) {
     float w = my_w;
     if (r.renorm) w = w / fmaxf(wsum, 1e-20f);
-    r.ids[t * r.topk + lane] = my_id;
-    r.weights[t * r.topk + lane] = w * r.scaling;
+    const bool chosen = lane < r.topk;
+    r.ids[t * n + lane] = chosen ? my_id : r.E + lane - r.topk;
+    r.weights[t * n + lane] = chosen ? w * r.scaling : 1.f;
   }
 }
 

@@ -3,6 +3,8 @@
 // A cached row is the projected key k[0 : D] followed by the rotated copy of k[0 : R] (R = rotated dimensions): the values
 // are the unrotated keys, so this one row serves as key and as value.  Scores contract over the whole row: the query is laid
 // out as [0 (R columns) | q[R : D] | rot(q)[0 : R]], so a tile of rows is used in shared memory exactly as it was copied.
+// Rows may also be [value (V columns) | zeros | key from column k_col on] with queries that are dense and final (rd = 0): scores
+// contract the key columns and outputs sum the value columns of the same tile.  An element-wise gate and a factor can follow.
 //
 //   window_kv_insert       rotates the new keys and writes their rows
 //   window_attn_simt       any size and type, fp32 arithmetic throughout: one CTA per (token, head)
@@ -100,12 +102,12 @@ window_attn_simt_kernel(const WinArgs a) {
   const int t = blockIdx.x, h = blockIdx.y, g = h / (a.H / a.G);
   const int req = a.tok_req[t];
   const long long pos = a.positions[t];
-  A* out = reinterpret_cast<A*>(a.out) + t * a.ldo + h * a.D;
+  A* out = reinterpret_cast<A*>(a.out) + t * a.ldo + h * a.V;
   if (req < 0 || pos < 0) {
-    for (int d = threadIdx.x; d < a.D; d += blockDim.x) from_f(out + d, 0.f);
+    for (int d = threadIdx.x; d < a.V; d += blockDim.x) from_f(out + d, 0.f);
     return;
   }
-  const A* qg = reinterpret_cast<const A*>(a.proj) + t * a.ldp + a.q_off + h * a.D;
+  const A* qg = reinterpret_cast<const A*>(a.proj) + t * a.ldp + a.q_off + h * a.q_step;
   const int half = a.rd >> 1;
   for (int d = threadIdx.x; d < a.D; d += blockDim.x) {
     float v = to_f(qg[d]);
@@ -137,7 +139,7 @@ window_attn_simt_kernel(const WinArgs a) {
     for (int j = warp; j < n; j += 4) {
       const A* r = row_of(k0 + j);
       float s = 0.f;
-      for (int d = lane; d < a.D; d += 32) s = fmaf(q[d], to_f(d < a.rd ? r[a.D + d] : r[d]), s);
+      for (int d = lane; d < a.D; d += 32) s = fmaf(q[d], to_f(d < a.rd ? r[a.D + d] : r[a.k_col - a.rd + d]), s);
       s = warp_sum(s) * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
       if (lane == 0) sc[j] = s;
@@ -162,7 +164,7 @@ window_attn_simt_kernel(const WinArgs a) {
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int d = threadIdx.x + i * 128;
-        if (d < a.D) acc[i] = fmaf(p, to_f(r[d]), acc[i]);
+        if (d < a.V) acc[i] = fmaf(p, to_f(r[d]), acc[i]);
       }
     }
     __syncthreads();
@@ -170,7 +172,7 @@ window_attn_simt_kernel(const WinArgs a) {
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
     const int d = threadIdx.x + i * 128;
-    if (d < a.D) from_f(out + d, acc[i] / l);
+    if (d < a.V) from_f(out + d, acc[i] / l * win_factor<A>(a, t, h, d));
   }
 }
 
@@ -238,9 +240,11 @@ __device__ __forceinline__ void fill_queries(__nv_bfloat16* qs, int stride, cons
     const int r = e / cols, c = e - r * cols;
     const int t = tok(r), h = head(r);
     float v = 0.f;
-    if (t >= 0 && h >= 0 && c >= a.rd && c < a.D + a.rd) {
-      const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.proj) + t * a.ldp + a.q_off + h * a.D;
-      if (c < a.D) {
+    if (t >= 0 && h >= 0 && c >= a.k_col && c < a.D + a.k_col) {
+      const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.proj) + t * a.ldp + a.q_off + h * a.q_step;
+      if (a.rd == 0) {
+        v = bf16_to_f(q[c - a.k_col]);
+      } else if (c < a.D) {
         v = bf16_to_f(q[c]);
       } else {
         const int d = c - a.D, i = d < half ? d : d - half;
@@ -299,7 +303,7 @@ __device__ __forceinline__ void value16(float (&o)[NV][4], const float (&p)[2][4
 }
 
 // ---- a few tokens per span ------------------------------------------------------------------------
-// part: [splits][T][H][D + 2] fp32 (unnormalised output, maximum, denominator) when splits > 1.
+// part: [splits][T][H][V + 2] fp32 (unnormalised output, maximum, denominator) when splits > 1.
 template <int NV>
 __global__ void __launch_bounds__(128)
 window_attn_tokens_kernel(const WinArgs a, const int* __restrict__ first_pos, const int* __restrict__ last_pos, int max_span,
@@ -319,8 +323,8 @@ window_attn_tokens_kernel(const WinArgs a, const int* __restrict__ first_pos, co
   const long long pos = a.positions[t];
   if (req < 0 || pos < 0) {
     if (split == 0)
-      for (int e = threadIdx.x; e < nh * a.D; e += 128)
-        reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h0 * a.D + e] = __float2bfloat16(0.f);
+      for (int e = threadIdx.x; e < nh * a.V; e += 128)
+        reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h0 * a.V + e] = __float2bfloat16(0.f);
     return;
   }
   if (last_pos[t] - first_pos[t] + 1 > max_span) return;
@@ -334,7 +338,7 @@ window_attn_tokens_kernel(const WinArgs a, const int* __restrict__ first_pos, co
                [&](int r) { return r < nh ? h0 + r : -1; }, 128);
   __syncthreads();
   zero_pad_columns(st, 2 * kPage, stride, a.row, 128);
-  const int ks0 = a.rd / 16, ks1 = (a.D + a.rd + 15) / 16;
+  const int ks0 = a.k_col / 16, ks1 = (a.D + a.k_col + 15) / 16;
   float o[NV][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll
   for (int j = 0; j < NV; ++j)
@@ -389,7 +393,7 @@ window_attn_tokens_kernel(const WinArgs a, const int* __restrict__ first_pos, co
     for (int j = 0; j < NV; ++j) {
       o[j][0] *= f[0]; o[j][1] *= f[0]; o[j][2] *= f[1]; o[j][3] *= f[1];
     }
-    value16<NV>(o, s, keys, stride, a.D, lane);
+    value16<NV>(o, s, keys, stride, a.V, lane);
     __syncthreads();
   }
   cp_async_wait<0>();
@@ -404,17 +408,17 @@ window_attn_tokens_kernel(const WinArgs a, const int* __restrict__ first_pos, co
       red_l[warp][(lane >> 2) + r * 8] = l[r];
     }
   }
-  float* ob = reinterpret_cast<float*>(st);                                  // [4][16][D]
+  float* ob = reinterpret_cast<float*>(st);                                  // [4][16][V]
 #pragma unroll
   for (int j = 0; j < NV; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int c = j * 8 + (lane & 3) * 2 + (i & 1), r = (lane >> 2) + (i >> 1) * 8;
-      if (c < a.D) ob[(warp * 16 + r) * a.D + c] = o[j][i];
+      if (c < a.V) ob[(warp * 16 + r) * a.V + c] = o[j][i];
     }
   __syncthreads();
-  for (int e = threadIdx.x; e < nh * a.D; e += 128) {
-    const int r = e / a.D, c = e - r * a.D, h = h0 + r;
+  for (int e = threadIdx.x; e < nh * a.V; e += 128) {
+    const int r = e / a.V, c = e - r * a.V, h = h0 + r;
     float mm = fmaxf(fmaxf(red_m[0][r], red_m[1][r]), fmaxf(red_m[2][r], red_m[3][r]));
     if (splits == 1 && a.sink != nullptr) mm = fmaxf(mm, a.sink[h]);
     float ll = 0.f, v = 0.f;
@@ -422,15 +426,16 @@ window_attn_tokens_kernel(const WinArgs a, const int* __restrict__ first_pos, co
     for (int w = 0; w < 4; ++w) {
       const float f = red_m[w][r] == -INFINITY ? 0.f : __expf(red_m[w][r] - mm);
       ll = fmaf(f, red_l[w][r], ll);
-      v = fmaf(f, ob[(w * 16 + r) * a.D + c], v);
+      v = fmaf(f, ob[(w * 16 + r) * a.V + c], v);
     }
     if (splits == 1) {
       if (a.sink != nullptr) ll += __expf(a.sink[h] - mm);
-      reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h * a.D + c] = __float2bfloat16(v / ll);
+      reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h * a.V + c] =
+          __float2bfloat16(v / ll * win_factor<__nv_bfloat16>(a, t, h, c));
     } else {
-      float* p = part + ((static_cast<long long>(split) * T + t) * a.H + h) * (a.D + 2);
+      float* p = part + ((static_cast<long long>(split) * T + t) * a.H + h) * (a.V + 2);
       p[c] = v;
-      if (c == 0) { p[a.D] = mm; p[a.D + 1] = ll; }
+      if (c == 0) { p[a.V] = mm; p[a.V + 1] = ll; }
     }
   }
 }
@@ -443,12 +448,12 @@ window_attn_combine_kernel(const WinArgs a, const int* __restrict__ first_pos, c
   __shared__ float s_m[64], s_w[64], s_l[64];                               // at most 64 ranges
   const int h = blockIdx.x, t = blockIdx.y;
   if (a.tok_req[t] < 0 || a.positions[t] < 0 || last_pos[t] - first_pos[t] + 1 > max_span) return;
-  const long long step = static_cast<long long>(T) * a.H * (a.D + 2);
-  const float* p = part + (static_cast<long long>(t) * a.H + h) * (a.D + 2);
+  const long long step = static_cast<long long>(T) * a.H * (a.V + 2);
+  const float* p = part + (static_cast<long long>(t) * a.H + h) * (a.V + 2);
   const int s = threadIdx.x;
   if (s < splits) {
-    s_m[s] = p[s * step + a.D];
-    s_l[s] = p[s * step + a.D + 1];
+    s_m[s] = p[s * step + a.V];
+    s_l[s] = p[s * step + a.V + 1];
   }
   __syncthreads();
   float m = a.sink != nullptr ? a.sink[h] : -INFINITY;
@@ -458,11 +463,12 @@ window_attn_combine_kernel(const WinArgs a, const int* __restrict__ first_pos, c
   float l = a.sink != nullptr ? __expf(a.sink[h] - m) : 0.f;
   for (int i = 0; i < splits; ++i) l = fmaf(s_w[i], s_l[i], l);
   const float inv = 1.f / l;
-  for (int c = s; c < a.D; c += blockDim.x) {
+  for (int c = s; c < a.V; c += blockDim.x) {
     float v = 0.f;
 #pragma unroll 8
     for (int i = 0; i < splits; ++i) v = fmaf(s_w[i], p[i * step + c], v);
-    reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h * a.D + c] = __float2bfloat16(v * inv);
+    reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + h * a.V + c] =
+        __float2bfloat16(v * inv * win_factor<__nv_bfloat16>(a, t, h, c));
   }
 }
 
@@ -509,7 +515,7 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
   fill_queries(qs, stride, a, kRows, gs, reinterpret_cast<float2*>(st), tok_of, head_of, kThreads);
   __syncthreads();
   zero_pad_columns(st, 2 * kPage, stride, a.row, kThreads);
-  const int ks0 = a.rd / 16, ks1 = (a.D + a.rd + 15) / 16;
+  const int ks0 = a.k_col / 16, ks1 = (a.D + a.k_col + 15) / 16;
   const bool capped = a.softcap > 0.f;
   const float c_in = capped ? a.scale * 2.f * kLog2e / a.softcap : a.scale * kLog2e;
   const float c_cap = a.softcap * kLog2e, c_two = -2.f * c_cap;
@@ -609,7 +615,7 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
             s[i][j][k] = p;
             l[k >> 1] += p;
           }
-        value16<NV>(o, s[i], keys + i * 16 * stride, stride, a.D, lane);
+        value16<NV>(o, s[i], keys + i * 16 * stride, stride, a.V, lane);
       }
     }
   }
@@ -622,17 +628,20 @@ window_attn_tiles_kernel(const WinArgs a, const int* __restrict__ query_start, c
     const int h = head_of(row);
     if (h < 0) continue;
     const float inv = 1.f / l[r];
-    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + tok_of(row) * a.ldo + h * a.D;
-    const bool pair = (a.D & 1) == 0 && (a.ldo & 1) == 0;
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + tok_of(row) * a.ldo + h * a.V;
+    const long long t = tok_of(row);
+    const bool pair = (a.V & 1) == 0 && (a.ldo & 1) == 0;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
       const int c = j * 8 + (lane & 3) * 2;
-      const float x = o[j][2 * r] * inv, y = o[j][2 * r + 1] * inv;
-      if (c + 1 < a.D && pair) {
+      float x = o[j][2 * r] * inv, y = o[j][2 * r + 1] * inv;
+      if (c < a.V) x *= win_factor<__nv_bfloat16>(a, t, h, c);
+      if (c + 1 < a.V) y *= win_factor<__nv_bfloat16>(a, t, h, c + 1);
+      if (c + 1 < a.V && pair) {
         *reinterpret_cast<__nv_bfloat162*>(out + c) = __floats2bfloat162_rn(x, y);
       } else {
-        if (c < a.D) out[c] = __float2bfloat16(x);
-        if (c + 1 < a.D) out[c + 1] = __float2bfloat16(y);
+        if (c < a.V) out[c] = __float2bfloat16(x);
+        if (c + 1 < a.V) out[c + 1] = __float2bfloat16(y);
       }
     }
   }
@@ -664,10 +673,12 @@ STK_API int stk_window_kv_insert(const void* proj, long long ldp, int q_off, int
 STK_API int stk_window_attention_simt(const void* proj, long long ldp, int q_off, int k_off, const int64_t* positions,
                                       const int* tok_req, const int* table, int bt_stride, void* cache, int row, const float* freq, int rd, float mag,
                                       int heads, int kv_heads, int dim,
+                                      int k_col, int vdim, int q_step, const void* gate, long long ldg, float out_scale,
                                       int window, float scale, float softcap, const float* sink, void* out, long long ldo,
                                       int fp32, int T, void* stream) {
   if (T <= 0) return 0;
-  const WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
+  WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
+  win_layout(a, k_col, vdim, q_step, gate, ldg, out_scale);
   if (!win_ok(a) || window < 1 || heads > 65535) return -1;
   cudaStream_t st = (cudaStream_t)stream;
   if (fp32) launch_pdl(window_attn_simt_kernel<float>, dim3(T, heads), dim3(128), 0, st, a);
@@ -687,19 +698,27 @@ STK_API int stk_window_attention_splits(int T, int heads, int kv_heads, int wind
   return s < 1 ? 1 : static_cast<int>(s);
 }
 
+// Whether the tensor-core kernels of this file cover a layer whose rows are [value | key].
+STK_API int stk_window_attention_mma_ok(int heads, int kv_heads, int dim, int vdim, int k_col, int row) {
+  return heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim <= 256 && vdim <= 256 && k_col % 16 == 0 && row % 8 == 0 &&
+         static_cast<size_t>((vdim <= 128 ? 128 : 64) + 2 * kPage) * win_stride(row) * 2 <= 220 * 1024;
+}
+
 #define STK_WIN_DIM(CALL)      \
-  if (dim <= 64) { CALL(8) }   \
-  else if (dim <= 128) { CALL(16) } \
+  if (vdim <= 64) { CALL(8) }   \
+  else if (vdim <= 128) { CALL(16) } \
   else { CALL(32) }
 
 STK_API int stk_window_attention_tokens(const void* proj, long long ldp, int q_off, int k_off, const int64_t* positions,
                                         const int* tok_req, const int* table, int bt_stride, void* cache, int row, const float* freq, int rd, float mag,
                                         int heads, int kv_heads, int dim,
+                                        int k_col, int vdim, int q_step, const void* gate, long long ldg, float out_scale,
                                         int window, float scale, float softcap, const float* sink, void* out, long long ldo,
                                         const int* first_pos, const int* last_pos, int max_span, int splits, float* part, int T,
                                         void* stream) {
   if (T <= 0) return 0;
-  const WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
+  WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
+  win_layout(a, k_col, vdim, q_step, gate, ldg, out_scale);
   if (!win_mma_ok(a) || window < 1 || splits < 1 || splits > 64 || (splits > 1 && part == nullptr) || T > 65535) return -1;
   const int sub = (heads / kv_heads + 15) / 16;
   if (kv_heads * sub > 65535) return -2;
@@ -721,14 +740,16 @@ STK_API int stk_window_attention_tokens(const void* proj, long long ldp, int q_o
 STK_API int stk_window_attention_tiles(const void* proj, long long ldp, int q_off, int k_off, const int64_t* positions,
                                        const int* tok_req, const int* table, int bt_stride, void* cache, int row, const float* freq, int rd, float mag,
                                        int heads, int kv_heads, int dim,
+                                       int k_col, int vdim, int q_step, const void* gate, long long ldg, float out_scale,
                                        int window, float scale, float softcap, const float* sink, void* out, long long ldo,
                                        const int* query_start, const int* req_rows, const int* start_pos, int n_req, int min_span, int max_span,
                                        int T, void* stream) {
   if (T <= 0) return 0;
-  const WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
+  WinArgs a = win_args(STK_WIN_CALL, window, scale, softcap, sink, out, ldo);
+  win_layout(a, k_col, vdim, q_step, gate, ldg, out_scale);
   if (!win_mma_ok(a) || window < 1 || n_req < 1) return -1;
   // eight warps of rows up to 128-wide heads, four above (their output accumulators fill the register file)
-  const int rows = dim <= 128 ? 128 : 64;
+  const int rows = vdim <= 128 ? 128 : 64;
   const int hg = heads / kv_heads, gs = hg < rows ? hg : rows, sub = (hg + gs - 1) / gs, bq = rows / gs;
   if (kv_heads * sub > 65535) return -2;
   const size_t smem = static_cast<size_t>(rows + 2 * kPage) * win_stride(row) * 2;

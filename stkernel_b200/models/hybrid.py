@@ -1,4 +1,4 @@
-"""Decoder described layer by layer (`HybridConfig`): attention and recurrent mixers, in parallel or post-norm blocks.
+"""Decoder described layer by layer (`HybridConfig`): attention and recurrent mixers, in parallel, post-norm or streams blocks.
 
 Parallel block: a layer is two matrix products.  Everything that reads the layer's norm (mixer projections, feed-forward gate and up) is one
 weight `w_in`; everything that is added to the residual (mixer output and feed-forward down projection) is one weight `w_out`
@@ -12,6 +12,13 @@ output, adds it to the fp32 residual and leaves the next copy; a mixture of expe
 
     h = x += norm1(mixer(h));  h = x += norm2(ff(h))
 
+Streams block: several fp32 residual streams; one kernel per sublayer writes the previous sublayer's output into all of them (the
+weighted sum over a token's experts on the way), forms the next sublayer's weighted sum of the new streams and norms it:
+
+    x_t = sum_s mix[s, t] x_s + write[t] y;  h = norm(sum_s read[s] x_s);  y = sublayer(h)
+
+A parallel mixer (two mixers over the same input) is one product in and one product out, like the parallel block's sublayers.
+
 Segments of both weights start on 16-column boundaries (zero-padded), whatever the configured sizes.
 """
 from __future__ import annotations
@@ -21,12 +28,14 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import HybridConfig, HybridLayer
+from ..config import HybridConfig, HybridLayer, recurrent_part
 from ..ops import attention as A
 from ..ops import functional as Fn
+from ..ops import grouped as GA
 from ..ops import hybrid as HB
 from ..ops import latent as LA
 from ..ops import moe as MO
+from ..ops import recurrence as RC
 from ..ops.functional import LinearWeight
 from ..utils.spans import span
 from .decoder import Decoder
@@ -49,8 +58,20 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
         if l.weights_of is not None:
             continue
         m, p = l.mixer, f"l{i}"
-        out[f"{p}.norm1"] = ((W,), "bf16")
-        if m.kind == "attention":
+        streams = cfg.block == "streams"
+        for q in (1, 2) if l.mlp is not None else (1,):
+            if q == 1 or cfg.block != "parallel":
+                out[f"{p}.norm{q}"] = ((W,), "bf16")
+            if streams:
+                out[f"{p}.norm{q}.b"] = ((W,), "bf16")
+                out[f"{p}.hc{q}.in"] = ((cfg.streams,), "bf16")
+                out[f"{p}.hc{q}.out"] = ((cfg.streams,), "bf16")
+                out[f"{p}.hc{q}.mix"] = ((cfg.streams, cfg.streams), "bf16")
+        if m.kind == "parallel":
+            out.update(_parallel_shapes(f"{p}.mix", m, W))
+        elif m.kind == "mamba2":
+            out.update(_mamba2_shapes(f"{p}.mix", m, W))
+        elif m.kind == "attention":
             out[f"{p}.mix.q"] = ((m.heads * m.dim, W), "bf16")
             out[f"{p}.mix.k"] = ((m.kv_heads * m.dim, W), "bf16")
             out[f"{p}.mix.sink"] = ((m.heads,), "bf16")
@@ -73,10 +94,9 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
             for g in ("i", "f"):
                 out[f"{p}.mix.{g}"] = ((m.heads, W), "bf16")
                 out[f"{p}.mix.{g}.b"] = ((m.heads,), "bf16")
-        out[f"{p}.mix.o"] = ((W, m.out_dim), "bf16")
+        if m.kind != "parallel":
+            out[f"{p}.mix.o"] = ((W, m.out_dim), "bf16")
         if l.mlp is not None:
-            if cfg.block == "post_norm":
-                out[f"{p}.norm2"] = ((W,), "bf16")
             if l.mlp.kind == "dense":
                 out[f"{p}.mlp.gate"] = ((l.mlp.ff, W), "bf16")
                 out[f"{p}.mlp.up"] = ((l.mlp.ff, W), "bf16")
@@ -86,20 +106,56 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
                     out[f"{p}.mlp.e{e}.up"] = ((l.mlp.ff, W), "bf16")
                     out[f"{p}.mlp.e{e}.down"] = ((W, l.mlp.ff), "bf16")
                 out[f"{p}.mlp.router"] = ((l.mlp.experts, W), "bf16")
-                out[f"{p}.mlp.router.b"] = ((l.mlp.experts,), "bf16")
+                if l.mlp.router_bias:
+                    out[f"{p}.mlp.router.b"] = ((l.mlp.experts,), "bf16")
+                if l.mlp.shared_ff:
+                    out[f"{p}.mlp.shared.up"] = ((l.mlp.shared_ff, W), "bf16")
+                    out[f"{p}.mlp.shared.down"] = ((W, l.mlp.shared_ff), "bf16")
     out["final.norm"] = ((W,), "bf16")
-    out["head"] = ((cfg.vocab_size, W), "bf16")
+    if cfg.block == "streams":
+        out["final.norm.b"] = ((W,), "bf16")
+    if not cfg.tied_head:
+        out["head"] = ((cfg.vocab_size, W), "bf16")
+    return out
+
+
+def _parallel_shapes(p: str, m, W: int) -> Dict[str, Tuple[Tuple[int, ...], str]]:
+    out = {}
+    a, r = m.left, m.right
+    for n, rows in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
+        out[f"{p}.left.{n}"] = ((rows, W), "bf16")
+        if a.bias:
+            out[f"{p}.left.{n}.b"] = ((rows,), "bf16")
+    if a.gate:
+        out[f"{p}.left.g"] = ((a.out_dim, W), "bf16")
+    for n, rows in (("q", r.heads * r.dim), ("k", r.heads * r.dim), ("v", r.out_dim), ("g", r.out_dim)):
+        out[f"{p}.right.{n}"] = ((rows, W), "bf16")
+    out[f"{p}.left.o"] = ((W, a.out_dim), "bf16")
+    out[f"{p}.right.o"] = ((W, r.out_dim), "bf16")
+    return out
+
+
+def _mamba2_shapes(p: str, m, W: int) -> Dict[str, Tuple[Tuple[int, ...], str]]:
+    out = {f"{p}.in": ((m.out_dim + m.conv_dim + m.heads, W), "bf16"), f"{p}.conv": ((m.conv_dim, m.conv), "bf16"),
+           f"{p}.conv.b": ((m.conv_dim,), "bf16"), f"{p}.norm": ((m.out_dim,), "bf16")}
+    for n in ("dt_bias", "A_log", "D"):
+        out[f"{p}.{n}"] = ((m.heads,), "bf16")
     return out
 
 
 def init_random_weights(cfg: HybridConfig, seed: int = 0, std: Optional[float] = None) -> Dict[str, torch.Tensor]:
-    """Random master weights: matrices ~N(0, std) (default: fan-in scaled), norms around 1, forget biases positive."""
+    """Random master weights: matrices ~N(0, std) (default: fan-in scaled), norms around 1, forget biases positive, residual streams
+    that mostly stay themselves, step sizes around 0.1."""
     g = torch.Generator().manual_seed(seed)
     w: Dict[str, torch.Tensor] = {}
     for name, (shape, _) in weight_shapes(cfg).items():
         r = torch.randn(shape, generator=g)
-        if len(shape) == 1 and "norm" in name:
+        if len(shape) == 1 and "norm" in name and not name.endswith(".b"):
             t = 1.0 + 0.2 * r
+        elif ".hc" in name:
+            t = 0.3 * r + (torch.eye(shape[0]) if len(shape) == 2 else 0.6)
+        elif name.endswith(".dt_bias"):
+            t = 0.7 * r - 2.0
         elif name.endswith(".f.b"):
             t = 3.0 + r
         elif len(shape) == 1:
@@ -123,8 +179,15 @@ class BlockWeights:
     attention: Optional[HB.AttentionParams] = None
     mlstm: Optional[HB.MlstmParams] = None
     latent: Optional[LA.LatentParams] = None
+    grouped: Optional[GA.GroupedParams] = None
+    retention: Optional[RC.RetentionParams] = None
+    mamba2: Optional[RC.Mamba2Params] = None
     w_gates: Optional[LinearWeight] = None  # [2 * heads, pad(W)]: input and forget gate of the recurrence (fp32 results)
-    # post-norm blocks: the feed-forward has weights of its own
+    # streams blocks: norm biases and how the sublayers read and write the streams
+    norm_b: Optional[torch.Tensor] = None
+    norm2_b: Optional[torch.Tensor] = None
+    streams: Tuple[HB.StreamWeights, ...] = ()          # mixer's, feed-forward's
+    # post-norm and streams blocks: the feed-forward has weights of its own
     norm2: Optional[torch.Tensor] = None    # fp32 [W]
     w_gate_up: Optional[LinearWeight] = None
     w_down: Optional[LinearWeight] = None
@@ -140,6 +203,7 @@ class HybridWeights:
     norm: torch.Tensor                      # fp32 [W]
     layers: List[BlockWeights]              # one entry per layer; `weights_of` layers repeat an entry
     layer_offset: int = 0
+    norm_b: Optional[torch.Tensor] = None   # fp32 [W]
 
 
 def _stack(parts: List[Tuple[str, torch.Tensor]], width: int, dtype) -> Tuple[LinearWeight, Dict[str, int]]:
@@ -187,6 +251,28 @@ def build_latent(cfg: HybridConfig, get, m, dt, device) -> LA.LatentParams:
                            LinearWeight(w_uk), LinearWeight(w_uv), w_ukv)
 
 
+def _parallel_params(cfg: HybridConfig, m, f32, device) -> Tuple[GA.GroupedParams, RC.RetentionParams]:
+    a, r = m.left, m.right
+    bias = torch.cat([f32(f"mix.left.{n}.b") for n in ("q", "k", "v")]).contiguous() if a.bias else None
+    temp = (a.q_temp.coef, a.q_temp.every) if a.q_temp is not None else (0.0, 1.0)
+    sink = torch.zeros(a.heads, dtype=F32, device=device) if a.null_sink else None
+    left = GA.GroupedParams(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, bias, cfg.norm_eps if a.qk_norm else None, temp, sink, a.gate,
+                            m.left_scale)
+    freq = r.rotary.frequencies()[0] if r.rotary is not None else []
+    log_decay = torch.tensor(r.decay, dtype=torch.float64).log().to(F32).to(device)
+    return left, RC.RetentionParams(r.heads, r.dim, r.vdim, log_decay, LA.split_frequencies(r.decay, device), LA.split_frequencies(freq, device), cfg.norm_eps, m.right_scale)
+
+
+def _mamba2_params(cfg: HybridConfig, m, get, f32) -> RC.Mamba2Params:
+    return RC.Mamba2Params(m.heads, m.vdim, m.state, m.groups, m.norm_groups, get("mix.conv").to(F32).t().contiguous(), f32("mix.conv.b"),
+                           f32("mix.dt_bias"), (-torch.exp(get("mix.A_log").double())).to(F32).contiguous(), f32("mix.D"),
+                           f32("mix.norm"), cfg.norm_eps)
+
+
+def _stream_weights(f32, q: int) -> HB.StreamWeights:
+    return HB.StreamWeights(f32(f"hc{q}.in"), f32(f"hc{q}.out"), f32(f"hc{q}.mix"))
+
+
 def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWeights:
     l: HybridLayer = cfg.layers[i]
     shapes = weight_shapes(cfg)
@@ -197,9 +283,14 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
     joined = l.mlp if cfg.block == "parallel" else None              # the feed-forward shares the mixer's two products
     if m.kind == "latent_attention":
         names = ["dq", "dkv", "g"] if m.kv_from is None else ["dq", "g"]
+    elif m.kind == "parallel":
+        names = ["left.q", "left.k", "left.v"] + (["left.g"] if m.left.gate else []) + [f"right.{n}" for n in "qkvg"]
     else:
         names = ["q", "k"] + (["v", "g"] if m.kind == "mlstm" else [])
-    parts = [(n, get(f"mix.{n}")) for n in names]
+    if m.kind == "mamba2":
+        parts = list(zip(("z", "xbc", "dt"), get("mix.in").split([m.out_dim, m.conv_dim, m.heads])))
+    else:
+        parts = [(n, get(f"mix.{n}")) for n in names]
     if joined is not None:
         parts += [("gate", get("mlp.gate")), ("up", get("mlp.up"))]
     w_in, seg = _stack(parts, _pad(W), dt)
@@ -208,6 +299,11 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
         w_out = torch.zeros(W, m.heads, vp, dtype=dt, device=device)
         w_out[:, :, :m.vdim] = get("mix.o").view(W, m.heads, m.vdim).to(dt)
         w_out = w_out.view(W, m.heads * vp)
+    elif m.kind == "parallel":
+        off = HB.out_offset(m.left.out_dim)
+        w_out = torch.zeros(W, off + _pad(m.right.out_dim), dtype=dt, device=device)
+        w_out[:, :m.left.out_dim] = get("mix.left.o").to(dt)
+        w_out[:, off:off + m.right.out_dim] = get("mix.right.o").to(dt)
     else:
         off = HB.out_offset(m.out_dim)
         w_out = torch.zeros(W, off + (_pad(joined.ff) if joined is not None else 0), dtype=dt, device=device)
@@ -222,11 +318,21 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
                                          f32("mix.sink") if m.sink else None)
     elif m.kind == "latent_attention":
         b.latent = build_latent(cfg, get, m, dt, device)
+    elif m.kind == "parallel":
+        b.grouped, b.retention = _parallel_params(cfg, m, f32, device)
+    elif m.kind == "mamba2":
+        b.mamba2 = _mamba2_params(cfg, m, get, f32)
     else:
         b.w_gates, _ = _stack([("i", torch.cat([get("mix.i"), get("mix.f")], 0))], _pad(W), dt)
         b.w_gates = LinearWeight(b.w_gates.w[:2 * m.heads])
         b.mlstm = HB.MlstmParams(m.heads, m.dim, m.vdim, m.gate_cap, torch.cat([f32("mix.i.b"), f32("mix.f.b")]).contiguous(),
                                  f32("mix.norm"), cfg.norm_eps)
+    if cfg.block == "streams":
+        b.norm_b = f32("norm1.b")
+        b.streams = (_stream_weights(f32, 1),)
+        if l.mlp is not None:
+            b.norm2_b = f32("norm2.b")
+            b.streams += (_stream_weights(f32, 2),)
     if l.mlp is not None and joined is None:
         build_feed_forward(b, l.mlp, get, W, dt, device)
     return b
@@ -242,15 +348,23 @@ def build_feed_forward(b: BlockWeights, mlp, get, W: int, dt, device) -> None:
         down[:, :mlp.ff] = get("mlp.down").to(dt)
         b.w_down = LinearWeight(down)
         return
-    up = torch.zeros(mlp.experts, ff, _pad(W), dtype=dt, device=device)
-    down = torch.zeros(mlp.experts, _pad(W), ff, dtype=dt, device=device)
+    # the shared expert's columns in equal parts, each an expert that every token takes
+    ff, n = _pad(mlp.expert_width), mlp.experts + mlp.shared_parts
+    up = torch.zeros(n, ff, _pad(W), dtype=dt, device=device)
+    down = torch.zeros(n, _pad(W), ff, dtype=dt, device=device)
     for e in range(mlp.experts):
         up[e, :mlp.ff, :W] = get(f"mlp.e{e}.up").to(dt)
         down[e, :W, :mlp.ff] = get(f"mlp.e{e}.down").to(dt)
-    b.experts = MO.PlainExperts(up, down)
+    if mlp.shared_parts:
+        wide = mlp.expert_width
+        rows, cols = get("mlp.shared.up").split(wide), get("mlp.shared.down").split(wide, 1)
+        for j, (r, c) in enumerate(zip(rows, cols)):
+            up[mlp.experts + j, :r.shape[0], :W] = r.to(dt)
+            down[mlp.experts + j, :W, :c.shape[1]] = c.to(dt)
+    b.experts = MO.PlainExperts(up, down, mlp.act)
     router, _ = _stack([("router", get("mlp.router"))], _pad(W), dt)
     b.router = LinearWeight(router.w[:mlp.experts])
-    b.router_bias = get("mlp.router.b").to(F32).contiguous()
+    b.router_bias = get("mlp.router.b").to(F32).contiguous() if mlp.router_bias else None
 
 
 def build_hybrid_weights(cfg: HybridConfig, src: WeightSource, device) -> HybridWeights:
@@ -261,10 +375,16 @@ def build_hybrid_weights(cfg: HybridConfig, src: WeightSource, device) -> Hybrid
         j = cfg.weight_layer(i)
         if j not in blocks:
             blocks[j] = build_block(cfg, src, j, device)
-    head, _ = _stack([("head", src.get("head", (V, W), device))], _pad(W), dt)
-    return HybridWeights(src.get("embed", (V, W), device).to(dt).contiguous(), LinearWeight(head.w[:V]),
-                         src.get("final.norm", (W,), device).to(F32).contiguous(),
-                         [blocks[cfg.weight_layer(i)] for i in range(len(cfg.layers))])
+    embed = src.get("embed", (V, W), device).to(dt).contiguous()
+    if cfg.tied_head and _pad(W) == W:
+        head = LinearWeight(embed)
+    else:
+        table = embed if cfg.tied_head else src.get("head", (V, W), device)
+        head = LinearWeight(_stack([("head", table)], _pad(W), dt)[0].w[:V])
+    # a factor on the logits is one on the norm in front of the head
+    norm = lambda n: (src.get(n, (W,), device).to(F32) * cfg.logit_scale).contiguous()
+    return HybridWeights(embed, head, norm("final.norm"), [blocks[cfg.weight_layer(i)] for i in range(len(cfg.layers))],
+                         norm_b=norm("final.norm.b") if cfg.block == "streams" else None)
 
 
 # ----------------------------------------------------------------------------
@@ -278,8 +398,9 @@ class HybridModel(Decoder):
         self.kv = kv
         self.act = HB.act_dtype(cfg.dtype, self.device)
         self.width = _pad(cfg.hidden_size)
-        self.recurrent = any(l.mixer.kind == "mlstm" for l in cfg.layers)
-        self.on_layer = None                # optional hook (layer index, residual [T, W] fp32) after each layer
+        self.recurrent = any(recurrent_part(l.mixer) is not None for l in cfg.layers)
+        self.on_layer = None                # optional hook (layer index, residual [T, W] fp32; streams: their sum) after each layer
+        self.read_sum = torch.ones(cfg.streams, dtype=F32, device=self.device)
 
     def build_meta(self, buf, t_pad: int, n_req: int, max_comp_rows: int, pure_decode: bool = False,
                    spans: Tuple = (1, 1)) -> HB.HybridMeta:
@@ -322,7 +443,17 @@ class HybridModel(Decoder):
                 return LA.latent_attention(q, p[:, b.seg["g"]:b.seg["g"] + m.heads], b.latent, meta, table, cache)
         p = Fn.linear(h, b.w_in, tag="in")
         c = torch.empty(t, b.w_out.in_features, dtype=self.act, device=h.device)
-        if m.kind == "attention":
+        if m.kind == "parallel":
+            with span("parallel_mixer", t):
+                s, table, cache = b.seg, self.kv.group_of(li).table_dev, self.kv.kv_cache[li]
+                q = GA.grouped_prep(p, s["left.q"], s["left.k"], s["left.v"], b.grouped, meta, table, cache)
+                GA.grouped_attention(p, q, s.get("left.g", 0), b.grouped, meta, table, cache, c)
+                RC.retention(p, s["right.q"], s["right.k"], s["right.v"], s["right.g"], b.retention, meta, self.kv.state[li], c,
+                             m.left.out_dim)
+        elif m.kind == "mamba2":
+            with span("mamba2", t):
+                RC.mamba2(p, b.seg["z"], b.seg["xbc"], b.seg["dt"], b.mamba2, meta, self.kv.state[li], c)
+        elif m.kind == "attention":
             with span("window_attention", t):
                 HB.window_attention(p, b.seg["q"], b.seg["k"], b.attention, meta, self.kv.group_of(li).table_dev,
                                     self.kv.kv_cache[li], c)
@@ -334,7 +465,7 @@ class HybridModel(Decoder):
         return c
 
     def feed_forward(self, li: int, h: torch.Tensor):
-        """Feed-forward output of a post-norm layer: fp32 rows, or expert rows whose sum the norm forms."""
+        """Feed-forward output of a post-norm or streams layer: fp32 rows, or expert rows whose sum the next kernel forms."""
         b, mlp = self.w.layers[li], self.cfg.layers[li].mlp
         if mlp.kind == "dense":
             p = Fn.linear(h, b.w_gate_up, tag="gate_up")
@@ -342,10 +473,11 @@ class HybridModel(Decoder):
             HB.join_glu(p, c, 0, (b.seg["gate"], b.seg["up"], mlp.ff), mlp.act)
             return Fn.linear(c, b.w_down, out_dtype=F32, tag="down")
         with span("experts", h.shape[0]):
-            routed = Fn.gate_route(h, b.router, b.router_bias, mlp.top, "softmax_topk", True, 1.0)
+            always = mlp.shared_parts
+            routed = Fn.gate_route(h, b.router, b.router_bias, mlp.top, "softmax_topk", True, 1.0, always=always) if h.is_cuda else None
             if routed is None:
                 logits = Fn.linear(h, b.router, out_dtype=F32, tag="router")
-                routed = MO.router(logits, b.router_bias, mlp.top, "softmax_topk", True, 1.0)
+                routed = MO.router(logits, b.router_bias, mlp.top, "softmax_topk", True, 1.0, always=always)
             return MO.plain_experts(h, *routed, b.experts)
 
     def post_norm_layer(self, li: int, x: torch.Tensor, h: torch.Tensor, meta: HB.HybridMeta) -> torch.Tensor:
@@ -357,10 +489,28 @@ class HybridModel(Decoder):
             h = HB.post_norm_add(x, self.feed_forward(li, h), b.norm2, cfg.norm_eps, self.width, self.act)
         return h
 
+    def streams_hidden(self, meta: HB.HybridMeta):
+        """-> (streams before the last sublayer's output, (that output, how it enters them))."""
+        cfg = self.cfg
+        x = HB.embed_scaled(meta.token_ids, self.w.embed, cfg.embedding_scale, streams=cfg.streams)
+        y, after = None, None
+        for li, b in enumerate(self.w.layers):
+            h = HB.stream_norm(x, y, after, b.streams[0].read, b.norm, b.norm_b, cfg.norm_eps, self.width, self.act)
+            y, after = Fn.linear(self.mix(li, h, meta), b.w_out, out_dtype=F32, tag="out"), b.streams[0]
+            if cfg.layers[li].mlp is not None:
+                h = HB.stream_norm(x, y, after, b.streams[1].read, b.norm2, b.norm2_b, cfg.norm_eps, self.width, self.act)
+                y, after = self.feed_forward(li, h), b.streams[1]
+            if self.on_layer is not None:
+                rows = HB.expert_sum(y, cfg.hidden_size)[:, :cfg.hidden_size]
+                self.on_layer(li, (torch.einsum("sr,tsw->tw", after.mix, x) + after.write.sum() * rows))
+        return x, (y, after)
+
     def forward_hidden(self, meta: HB.HybridMeta):
         """-> (residual before the last layer's output, that output), both [T, W] fp32: the sum is formed where it is normed.
-        Post-norm blocks: (residual, None)."""
+        Post-norm blocks: (residual, None); streams blocks: see `streams_hidden`."""
         cfg = self.cfg
+        if cfg.block == "streams":
+            return self.streams_hidden(meta)
         if cfg.block == "post_norm":
             h = torch.empty(meta.token_ids.shape[0], self.width, dtype=self.act, device=self.device)
             x = HB.embed_scaled(meta.token_ids, self.w.embed, cfg.embedding_scale, h)
@@ -379,6 +529,8 @@ class HybridModel(Decoder):
 
     def head_hidden(self, X, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         x, y = X
+        if self.cfg.block == "streams":
+            return HB.stream_norm(x, *y, self.read_sum, self.w.norm, self.w.norm_b, self.cfg.norm_eps, self.width, self.act, rows=rows)
         return HB.add_layer_norm(x, y, self.w.norm, self.cfg.norm_eps, self.width, self.act, rows=rows,
                                  center=self.cfg.block == "parallel")
 

@@ -13,7 +13,8 @@ from typing import Any, Callable, Dict, Mapping, Optional, Tuple
 
 import torch
 
-from ..config import ConfigError, EngineConfig, domilix_config_from_json, model_config_from_hf, timalorn_config_from_json
+from ..config import (ConfigError, EngineConfig, domilix_config_from_json, fanulix_config_from_json, model_config_from_hf,
+                      timalorn_config_from_json)
 
 
 @dataclass(frozen=True)
@@ -105,12 +106,14 @@ def _hybrid_model(cfg: EngineConfig, weights, kv, comm, tp_rank: int):
 _HYBRID_SOURCES = ("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", "linear_f32.cu", "hybrid_block.cu", "sampler.cu")
 _MECHANISM_SOURCES = {"attention": ("window_attention.cu", "window_attention_tc.cu"), "mlstm": ("mlstm.cu",), "dense": (),
                       "latent_attention": ("latent_attention.cu", "latent_tokens_tc.cu", "latent_prompt_tc.cu"),
+                      "grouped_attention": ("window_attention.cu", "latent_prompt_tc.cu", "grouped_attention.cu"),
+                      "retention": ("linear_scan.cu", "retention.cu"), "mamba2": ("linear_scan.cu", "mamba2.cu"),
                       "moe": ("moe.cu", "moe_plain.cu", "gate_cluster.cu")}
 
 
 def _hybrid_sources(cfg) -> Tuple[str, Tuple[str, ...]]:
     kinds = [k for k in cfg.mechanisms() if _MECHANISM_SOURCES[k]]
-    return "-".join(["hybrid"] + kinds), _HYBRID_SOURCES + tuple(f for k in kinds for f in _MECHANISM_SOURCES[k])
+    return "-".join(["hybrid"] + kinds), _HYBRID_SOURCES + tuple(dict.fromkeys(f for k in kinds for f in _MECHANISM_SOURCES[k]))
 
 
 FAMILIES: Dict[str, ModelFamily] = {
@@ -123,6 +126,7 @@ FAMILIES: Dict[str, ModelFamily] = {
 ARCHITECTURES: Dict[str, Callable[..., Any]] = {
     "Timalorn": timalorn_config_from_json,
     "Domilix": domilix_config_from_json,
+    "Fanulix": fanulix_config_from_json,
 }
 
 

@@ -1,6 +1,6 @@
-"""Ops of the layer-by-layer decoders: scaled embedding, add + norm and norm + add on an fp32 residual, paged windowed attention
-whose values are the unrotated keys, mLSTM recurrence, and the parallel block's joined sublayer outputs.  (Latent attention:
-`ops/latent.py`; experts: `ops/moe.py`.)
+"""Ops of the layer-by-layer decoders: scaled embedding, add + norm and norm + add on an fp32 residual, residual streams, paged windowed
+attention whose values are the unrotated keys, mLSTM recurrence, and the parallel block's joined sublayer outputs.  (Latent attention:
+`ops/latent.py`; grouped attention: `ops/grouped.py`; retention and Mamba-2: `ops/recurrence.py`; experts: `ops/moe.py`.)
 
 Activations are bf16, or fp32 in a float32 model (every kernel here has both forms; the fp32 forms use no reduced-precision
 products).  Residual, norms, scores and softmax, gates and recurrent state are fp32 in either.
@@ -43,9 +43,10 @@ def _is32(t: torch.Tensor) -> int:
 # ----------------------------------------------------------------------------
 # residual
 # ----------------------------------------------------------------------------
-def embed_scaled(ids: torch.Tensor, embed: torch.Tensor, scale: float, h: Optional[torch.Tensor] = None) -> torch.Tensor:
+def embed_scaled(ids: torch.Tensor, embed: torch.Tensor, scale: float, h: Optional[torch.Tensor] = None,
+                 streams: Optional[int] = None) -> torch.Tensor:
     """ids [T] -> fp32 residual [T, W] = embed[id] * scale.  h [T, width]: receives the rows in the compute type as well,
-    zero-padded."""
+    zero-padded.  streams: that many equal copies, [T, streams, W]."""
     t, w = ids.shape[0], embed.shape[1]
     if not ids.is_cuda:
         ok = (ids >= 0) & (ids < embed.shape[0])
@@ -53,11 +54,59 @@ def embed_scaled(ids: torch.Tensor, embed: torch.Tensor, scale: float, h: Option
         if h is not None:
             h.zero_()
             h[:, :w] = x.to(h.dtype)
-        return x
-    x = torch.empty(t, w, dtype=F32, device=ids.device)
-    _lib.call("stk_embed_scaled", ids, embed, _is32(embed), x, w, t, w, embed.shape[0], float(scale), h,
+        return x if streams is None else x[:, None].repeat(1, streams, 1)
+    n = streams or 1
+    x = torch.empty(t, n * w, dtype=F32, device=ids.device)
+    _lib.call("stk_embed_scaled", ids, embed, _is32(embed), x, n * w, n, t, w, embed.shape[0], float(scale), h,
               h.stride(0) if h is not None else 0, h.shape[1] if h is not None else 0, _lib.status_buffer(), _lib.stream())
-    return x
+    return x if streams is None else x.view(t, n, w)
+
+
+@dataclass
+class StreamWeights:
+    """How one sublayer reads and writes the residual streams (fp32): u = sum_s read[s] x_s before, x_t <- sum_s mix[s, t] x_s +
+    write[t] y after it."""
+    read: torch.Tensor             # [s]
+    write: torch.Tensor            # [s]
+    mix: torch.Tensor              # [s, s], [from, to]
+
+
+def expert_sum(y, w_n: int) -> torch.Tensor:
+    """CPU: fp32 rows [T, W] of a sublayer's output (`ExpertRows`: the weighted sum over each token's pairs)."""
+    if isinstance(y, torch.Tensor):
+        return y
+    t, k = y.weights.shape
+    at = y.pair_row.long() if y.pair_row is not None else torch.arange(t * k)
+    return (y.y[at].to(F32).view(t, k, -1)[..., :w_n] * y.weights[..., None]).sum(1)
+
+
+def stream_norm(x: torch.Tensor, y, after: Optional[StreamWeights], read: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float,
+                width: int, dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Streams x [T, s, W] fp32: the previous sublayer's output y (fp32 rows or `ExpertRows`; None: nothing to add) goes into them as
+    `after` says, in place, then the layer norm (weight w, bias b) of sum_s read[s] x_s in `dtype`, zero-padded to `width` columns.
+    rows: only these rows are normed, and the streams are not written back."""
+    t, s, w_n = x.shape
+    if not x.is_cuda:
+        if y is not None:
+            y = expert_sum(y, w_n)[:, :w_n]
+            new = R.stream_mix(x if rows is None else x[rows], y if rows is None else y[rows], after.mix, after.write)
+            if rows is None:
+                x.copy_(new)
+        else:
+            new = x if rows is None else x[rows]
+        h = torch.zeros(new.shape[0], width, dtype=dtype)
+        h[:, :w_n] = (R.layer_norm(torch.einsum("s,tsw->tw", read, new), w, eps) + b).to(dtype)
+        return h
+    n = t if rows is None else rows.shape[0]
+    h = torch.empty(n, width, dtype=dtype, device=x.device)
+    pairs = y if y is not None and not isinstance(y, torch.Tensor) else None
+    plain = y if pairs is None else None
+    _lib.call("stk_stream_norm", x, s, plain, plain.stride(0) if plain is not None else 0, pairs.y if pairs is not None else None,
+              pairs.y.stride(0) if pairs is not None else 0, pairs.pair_row if pairs is not None else None,
+              pairs.weights if pairs is not None else None, pairs.weights.shape[1] if pairs is not None else 0,
+              after.mix if y is not None else None, after.write if y is not None else None, read, w, b, float(eps), h, h.stride(0), w_n,
+              width, _is32(h), rows, n, _lib.stream())
+    return h
 
 
 def add_layer_norm(x: torch.Tensor, y: Optional[torch.Tensor], w: torch.Tensor, eps: float, width: int, dtype: torch.dtype,
@@ -87,11 +136,7 @@ def post_norm_add(x: torch.Tensor, y, w: torch.Tensor, eps: float, width: int, d
     t, w_n = x.shape
     rows = None if isinstance(y, torch.Tensor) else y
     if not x.is_cuda:
-        if rows is not None:
-            k = rows.weights.shape[1]
-            at = rows.pair_row.long() if rows.pair_row is not None else torch.arange(t * k)
-            y = (rows.y[at].to(F32).view(t, k, -1)[..., :w_n] * rows.weights[..., None]).sum(1)
-        x += R.rms_norm(y, w, eps)
+        x += R.rms_norm(expert_sum(y, w_n), w, eps)
         h = torch.zeros(t, width, dtype=dtype)
         h[:, :w_n] = x.to(dtype)
         return h
@@ -164,20 +209,21 @@ def window_attention(proj: torch.Tensor, q_off: int, k_off: int, a: AttentionPar
               a.freq, rd, float(a.mag), h, g, d)
     _lib.call("stk_window_kv_insert", *common, _is32(proj), t, _lib.stream())
     tail = (a.window, float(a.scale), float(a.softcap), a.sink, out, out.stride(0))
+    rows = (rd, d, d, None, 0, 1.0)                      # scores from column rd, values as wide as keys, dense queries, no gate
     if _is32(proj) or d > 256 or cache.shape[3] % 8:
-        _lib.call("stk_window_attention_simt", *common, *tail, _is32(proj), t, _lib.stream())
+        _lib.call("stk_window_attention_simt", *common, *rows, *tail, _is32(proj), t, _lib.stream())
         return
     token_span = ATTN_TOKEN_SPAN if meta.max_span > ATTN_TOKEN_SPAN else meta.max_span
     if meta.min_span <= token_span:
         splits = _lib.query("stk_window_attention_splits", t, h, g, a.window, _lib.sm_count())
         part = scratch("wattn.part", (splits * t * h * (d + 2),), F32, proj.device) if splits > 1 else None
-        _lib.call("stk_window_attention_tokens", *common, *tail, meta.first_pos, meta.last_pos, token_span, splits, part, t,
+        _lib.call("stk_window_attention_tokens", *common, *rows, *tail, meta.first_pos, meta.last_pos, token_span, splits, part, t,
                   _lib.stream())
     spans = (meta.query_start, meta.req_rows, meta.start_pos, meta.n_req)
     tc = (meta.max_span >= ATTN_TC_SPAN and out.stride(0) % 8 == 0
           and _lib.query("stk_window_attention_tc_ok", h, g, d, rd, cache.shape[3]) == 1)
     if meta.max_span > token_span and not (tc and meta.min_span >= ATTN_TC_SPAN):
-        _lib.call("stk_window_attention_tiles", *common, *tail, *spans, token_span + 1, ATTN_TC_SPAN - 1 if tc else 1 << 30, t,
+        _lib.call("stk_window_attention_tiles", *common, *rows, *tail, *spans, token_span + 1, ATTN_TC_SPAN - 1 if tc else 1 << 30, t,
                   _lib.stream())
     if tc:
         _lib.call("stk_window_attention_tc", *common, *tail, *spans, ATTN_TC_SPAN, cache.shape[0], t, _lib.status_buffer(),

@@ -140,7 +140,7 @@ def latent_attention(q: torch.Tensor, gate: Optional[torch.Tensor], a: LatentPar
         rows = meta.gathered.get(cache.data_ptr())
         if rows is None:
             rows = torch.empty(n_rows, row, dtype=q.dtype, device=q.device)
-            _lib.call("stk_latent_rows", *spans, PROMPT_SPAN, table, table.stride(0), cache, row, rows, n_rows, _lib.stream())
+            _lib.call("stk_latent_rows", *spans, PROMPT_SPAN, table, table.stride(0), cache, 1, row, rows, n_rows, _lib.stream())
             meta.gathered.clear()
             meta.gathered[cache.data_ptr()] = rows
         width = a.w_ukv.out_features // a.heads

@@ -721,14 +721,124 @@ def latent_attention(qa: torch.Tensor, qr: torch.Tensor, rot_off: int, positions
     return out
 
 
-def plain_experts(x: torch.Tensor, ids: torch.Tensor, up: torch.Tensor, down: torch.Tensor, act_dtype) -> torch.Tensor:
-    """x [T, K] through expert ids [T, k] of up [E, F, K], down [E, W, F]: relu squared between them -> pair rows [T * k, W]."""
+def expert_act(z: torch.Tensor, act: str) -> torch.Tensor:
+    """"relu2" (relu squared) or "gelu" (exact), fp32."""
+    return torch.relu(z) ** 2 if act == "relu2" else torch.nn.functional.gelu(z)
+
+
+def plain_experts(x: torch.Tensor, ids: torch.Tensor, up: torch.Tensor, down: torch.Tensor, act_dtype, act: str = "relu2"
+                  ) -> torch.Tensor:
+    """x [T, K] through expert ids [T, k] of up [E, F, K], down [E, W, F]: act between them -> pair rows [T * k, W]."""
     t, k = ids.shape
     out = torch.zeros(t * k, down.shape[1], dtype=act_dtype)
     flat = ids.reshape(-1).long()
     xp = x.to(F32).repeat_interleave(k, 0)
     for e in flat.unique().tolist():
         at = (flat == e).nonzero().flatten()
-        z = torch.relu(xp[at] @ up[e].to(F32).t())
-        out[at] = ((z * z).to(act_dtype).to(F32) @ down[e].to(F32).t()).to(act_dtype)
+        z = expert_act(xp[at] @ up[e].to(F32).t(), act)
+        out[at] = (z.to(act_dtype).to(F32) @ down[e].to(F32).t()).to(act_dtype)
     return out
+
+
+# ----------------------------------------------------------------------------
+# residual streams, grouped attention over the full context, linear recurrences with a scalar decay
+# ----------------------------------------------------------------------------
+def stream_mix(x: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """x [T, s, W] fp32, y [T, W]: every stream t becomes sum_s mix[s, t] x_s + out[t] y."""
+    return torch.einsum("sr,tsw->trw", mix.to(F32), x) + out.to(F32)[None, :, None] * y.to(F32)[:, None]
+
+
+def unit_rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: float) -> torch.Tensor:
+    n = torch.floor((positions.clamp(min=0) + 1).to(torch.float64) / every) + 1.0
+    return (1.0 + coef * torch.log(n)).to(F32)
+
+
+def grouped_kv_insert(k: torch.Tensor, v: torch.Tensor, k_col: int, positions, tok_req, table, cache) -> None:
+    """k [T, G, D], v [T, G, V] -> cache [pages, G, PAGE, row]: value, zeros, key from column k_col on, zeros."""
+    page_rows = cache.shape[2]
+    for t in range(k.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        pg = int(table[r, p // page_rows])
+        if pg < 0:
+            continue
+        dst = cache[pg, :, p % page_rows]
+        dst.zero_()
+        dst[:, :v.shape[-1]] = v[t].to(cache.dtype)
+        dst[:, k_col:k_col + k.shape[-1]] = k[t].to(cache.dtype)
+
+
+def grouped_attention(q: torch.Tensor, vdim: int, k_col: int, positions, tok_req, table, cache, scale: float,
+                      null_sink: bool) -> torch.Tensor:
+    """q [T, H, D] against every cached row up to each token's position -> [T, H, V] fp32."""
+    t_n, h, d = q.shape
+    g, page_rows = cache.shape[1], cache.shape[2]
+    out = torch.zeros(t_n, h, vdim, dtype=F32)
+    for t in range(t_n):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        at = torch.arange(0, p + 1)
+        rows = cache[table[r, at // page_rows].long(), :, at % page_rows].to(F32)        # [n, G, row]
+        s = (torch.einsum("ghd,ngd->ghn", q[t].to(F32).view(g, h // g, d), rows[..., k_col:k_col + d]) * scale).view(h, -1)
+        if null_sink:
+            s = torch.cat([s, torch.zeros(h, 1)], -1)
+        w = torch.softmax(s, -1)[:, :at.numel()]
+        out[t] = torch.einsum("ghn,ngv->ghv", w.view(g, h // g, -1), rows[..., :vdim]).reshape(h, vdim)
+    return out
+
+
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, tok_req, positions,
+                S: torch.Tensor) -> torch.Tensor:
+    """One step's tokens through S <- exp(log_decay) S + k v^T, o = S^T q per head.  q, k [T, H, D], v [T, H, V], log_decay [T, H],
+    state S [rows, H, D, V] updated in place; a span that starts at position 0 starts from zeros.  -> [T, H, V] fp32."""
+    out = torch.zeros(v.shape, dtype=F32)
+    for t in range(q.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        if p == 0:
+            S[r].zero_()
+        S[r] = torch.exp(log_decay[t].to(F32))[:, None, None] * S[r] + k[t].to(F32)[:, :, None] * v[t].to(F32)[:, None, :]
+        out[t] = torch.einsum("hdv,hd->hv", S[r], q[t].to(F32))
+    return out
+
+
+def rotate_half_split(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
+    """x [T, heads, D]: dimension i rotated with i + n by position * (freq[0, i] + freq[1, i]), n = freq.shape[1]; fp32."""
+    n = freq.shape[1]
+    xf = x.to(F32)
+    a = positions.to(torch.float64)[:, None] * (freq[0].double() + freq[1].double())[None]
+    c, s = torch.cos(a).to(F32)[:, None], torch.sin(a).to(F32)[:, None]
+    u, v = xf[..., :n], xf[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, xf[..., 2 * n:]], -1)
+
+
+def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor, tok_req, positions, first_pos, ring: torch.Tensor
+                ) -> torch.Tensor:
+    """x [T, C] -> bias + sum_j taps[:, n - 1 - j] x(position - j) per channel, fp32.  Inputs before the step's span come from
+    ring [rows, n - 1, C] (position p at p mod n - 1), inputs before position 0 are zero."""
+    n = taps.shape[1]
+    out = bias.to(F32)[None].repeat(x.shape[0], 1)
+    for t in range(x.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        for j in range(min(n, p + 1)):
+            past = x[t - j] if p - j >= int(first_pos[t]) else ring[r, (p - j) % (n - 1)]
+            out[t] += taps[:, n - 1 - j].to(F32) * past.to(F32)
+    return out
+
+
+def keep_conv_inputs(x: torch.Tensor, tok_req, positions, last_pos, ring: torch.Tensor) -> None:
+    """The last n - 1 inputs of every span into its request's ring."""
+    keep = ring.shape[1]
+    for t in range(x.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r >= 0 and p >= 0 and p > int(last_pos[t]) - keep:
+            ring[r, p % keep] = x[t].to(ring.dtype)

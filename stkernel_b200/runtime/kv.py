@@ -25,8 +25,9 @@ from typing import Callable, Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import FULL_CONTEXT, HybridConfig, ModelConfig
+from ..config import FULL_CONTEXT, HybridConfig, ModelConfig, attention_part, recurrent_part
 from ..ops.cache import PAGE, PagedCache
+from ..ops.grouped import grouped_row
 from ..ops.latent import latent_row
 from .planning import dcp_owner
 
@@ -352,8 +353,13 @@ class HybridKVManager(CacheManager):
       the key, so nothing is stored twice.  Pages are released as they leave the window.
     * latent-attention layers: paged rows of one latent and one rotated key part (`ops/latent.py`), in the page group of the
       full context, whose pages stay until the request ends.  A layer that attends over another layer's latents has none.
+    * grouped-attention layers: paged rows `[kv_heads, PAGE, row]` of value and key (`ops/grouped.py`), in the full-context group.
     * mLSTM layers: per request row the matrix memory `[heads, dim, vdim]`, the normaliser `[heads, dim]` and the running
       maximum `[heads]`, fp32.  Nothing is cleared when a row changes hands: a span that starts at position 0 reads zeros.
+    * retention and Mamba-2 layers: per request row the matrix state `[heads, dim, vdim]` in fp32, and for Mamba-2 the last inputs
+      of the convolution `[taps - 1, channels]` as projected (position p at p mod taps - 1); not cleared either.
+
+    A parallel mixer's two sides have their cache and state under the same layer.
 
     pool_tokens caps the full-context group at this many tokens over all requests together; admission then promises every
     request the pages of its whole context and makes others wait.
@@ -377,26 +383,34 @@ class HybridKVManager(CacheManager):
             self.by_window[w] = GroupTable(name, pages, max_requests, pages_ctx, self.device, 1.0)
         self.full = self.by_window.get(FULL_CONTEXT)
         self.kv_cache: Dict[int, torch.Tensor] = {}
-        self.state: Dict[int, Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = {}
+        self.state: Dict[int, Tuple[torch.Tensor, ...]] = {}
         for li, l in enumerate(cfg.layers):
-            m = l.mixer
-            if m.kind == "attention":
+            m, r = attention_part(l.mixer), recurrent_part(l.mixer)
+            if m is not None and m.kind == "attention":
                 g = self.by_window[m.window]
                 self.kv_cache[li] = torch.zeros(g.num_pages, m.kv_heads, PAGE, kv_row_width(m.dim, m.rot_dims), dtype=dt,
                                                 device=self.device)
-            elif m.kind == "latent_attention":
-                if m.kv_from is None:
-                    self.kv_cache[li] = torch.zeros(self.full.num_pages, PAGE, latent_row(m.kv_rank, m.rot_dim)[0], dtype=dt,
-                                                    device=self.device)
+            elif m is not None and m.kind == "grouped_attention":
+                self.kv_cache[li] = torch.zeros(self.full.num_pages, m.kv_heads, PAGE, grouped_row(m.dim, m.vdim)[0], dtype=dt,
+                                                device=self.device)
+            elif m is not None and m.kv_from is None:
+                self.kv_cache[li] = torch.zeros(self.full.num_pages, PAGE, latent_row(m.kv_rank, m.rot_dim)[0], dtype=dt,
+                                                device=self.device)
+            if r is None:
+                continue
+            z = lambda *s: torch.zeros(max_requests, r.heads, *s, dtype=torch.float32, device=self.device)
+            if r.kind == "mlstm":
+                self.state[li] = (z(r.dim, r.vdim), z(r.dim), z())
+            elif r.kind == "retention":
+                self.state[li] = (z(r.dim, r.vdim),)
             else:
-                z = lambda *s: torch.zeros(max_requests, m.heads, *s, dtype=torch.float32, device=self.device)
-                self.state[li] = (z(m.dim, m.vdim), z(m.dim), z())
+                self.state[li] = (z(r.state, r.vdim), torch.zeros(max_requests, r.conv - 1, r.conv_dim, dtype=dt, device=self.device))
 
     def groups(self) -> List[GroupTable]:
         return list(self.by_window.values())
 
     def group_of(self, layer: int) -> GroupTable:
-        return self.by_window[self.cfg.layers[layer].mixer.window]
+        return self.by_window[attention_part(self.cfg.layers[layer].mixer).window]
 
     def prepare(self, row: int, start_pos: int, n_tokens: int, lookback: Optional[int] = None) -> None:
         end = start_pos + n_tokens
@@ -435,14 +449,20 @@ class HybridKVManager(CacheManager):
 
     def bytes_allocated(self) -> int:
         n = sum(t.numel() * t.element_size() for t in self.kv_cache.values())
-        return n + sum(t.numel() * 4 for st in self.state.values() for t in st)
+        return n + sum(t.numel() * t.element_size() for st in self.state.values() for t in st)
 
 
 def hybrid_bytes_per_context_token(cfg: HybridConfig) -> int:
     """Bytes of full-context cache that one token of context costs (windows and recurrent states are bounded)."""
     es = 4 if cfg.dtype == "float32" else 2
-    return sum(latent_row(l.mixer.kv_rank, l.mixer.rot_dim)[0] * es for l in cfg.layers
-               if l.mixer.kind == "latent_attention" and l.mixer.kv_from is None)
+    n = 0
+    for l in cfg.layers:
+        m = attention_part(l.mixer)
+        if m is not None and m.kind == "latent_attention" and m.kv_from is None:
+            n += latent_row(m.kv_rank, m.rot_dim)[0] * es
+        elif m is not None and m.kind == "grouped_attention":
+            n += m.kv_heads * grouped_row(m.dim, m.vdim)[0] * es
+    return n
 
 
 def kv_row_width(dim: int, rot_dims: int) -> int:
