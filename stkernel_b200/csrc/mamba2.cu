@@ -55,7 +55,9 @@ struct Mamba2Front {
       else if (e < 2 * N) k[e - N] = conv_at<A>(c, t, i, pos, row, b0 + e - N) * dt;
       else x[e - 2 * N] = conv_at<A>(c, t, i, pos, row, h * V + col0 + e - 2 * N);
     }
-    return make_float2(expf(c.neg_a[h] * dt), 0.f);
+    // slow decays as 1 and the (small) difference from it: a rounded factor close to 1 would be off in the same direction for long
+    const float lg = c.neg_a[h] * dt;
+    return lg > -0.25f ? make_float2(1.f, expm1f(lg)) : make_float2(expf(lg), 0.f);
   }
 };
 

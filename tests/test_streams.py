@@ -1,0 +1,437 @@
+"""The streams decoder (Fanulix) against the plain oracle: whole prompts, portions, decoding, batches, reused pages and rows, far keys,
+far tokens in the recurrent states, generation through the scheduler.  Runs on the CPU reference ops and, marked `gpu`, on the kernels
+in both compute types."""
+import dataclasses
+import json
+import os
+
+import pytest
+import torch
+
+import fanulix_oracle as O
+import streams_util as U
+from stkernel_b200.config import CacheConfig, EngineConfig, SchedulerConfig, fanulix_config_to_json
+from stkernel_b200.runtime.engine import SamplingParams
+from streams_util import att, both, config, error, feed, make_engine, mixed, moe, oracle, plain, ret, ssm, tokens, weights
+
+CPU = pytest.param(("cpu", "float32"), id="cpu")
+G32 = pytest.param(("cuda:0", "float32"), id="gpu-f32", marks=pytest.mark.gpu)
+G16 = pytest.param(("cuda:0", "bfloat16"), id="gpu-bf16", marks=pytest.mark.gpu)
+ALL = pytest.mark.parametrize("where", [CPU, G32, G16])
+EXACT = pytest.mark.parametrize("where", [CPU, G32])
+TOL = {k: v[0] for k, v in U.LIMITS.items()}
+
+
+def close(got, ref, where, factor=1.0):
+    U.close(got, ref, where[1], factor)
+
+
+SHAPES = {
+    "plain": lambda d: plain(d),
+    "mixed": lambda d: mixed(d),
+    "one_stream": lambda d: config(both(), ssm(), dtype=d, streams=1),
+    "five_streams": lambda d: config(ssm(), both(), dtype=d, streams=5, logit_scale=2.0),
+    "odd_sizes": lambda d: config((both(att(3, 3, 13, 11), ret(5, 9, 7, 6)), moe(3, 3, 19, 31)),
+                                  (ssm(3, 7, 11, 3, 5, 7), moe(2, 2, 21, 5)), dtype=d, width=77, vocab=101),
+    "one_head": lambda d: config(both(att(1, 1, 16, 8), ret(1, 8, 24, 8)), ssm(1, 16, 8, 1, 2, 1), dtype=d, width=48),
+    "no_taps_before": lambda d: config(ssm(conv=1), both(), dtype=d),
+    "aligned": lambda d: config((both(att(8, 2, 64, 64), ret(4, 64, 64, 64)), moe(8, 8, 64, 128)),
+                                (ssm(8, 64, 64, 2, 4, 2), moe(4, 4, 64, 64)), dtype=d, width=256),
+    "wide_values": lambda d: config(both(att(2, 1, 40, 136), ret(2, 24, 136, 10)), ssm(2, 136, 136, 1, 4, 1), dtype=d),
+    "no_feed_forwards": lambda d: config((both(), None), (ssm(), None), dtype=d),
+}
+
+
+@ALL
+@pytest.mark.parametrize("shape", list(SHAPES))
+def test_prompt_then_decoding(where, shape):
+    cfg = SHAPES[shape](where[1])
+    w = weights(cfg, 1)
+    toks = tokens(cfg, 180 if where[0] != "cpu" else 100, 2)
+    n = len(toks) if where[1] == "float32" else U.clear_routing(cfg, w, toks, 0.1)
+    toks = toks[:max(n, 1)]
+    ref = oracle(cfg, w, toks)[:n]
+    eng = make_engine(cfg, w, where[0])
+    for cuts in (None, [161, 1], [63, 2, 66, 3, 2, 1]) if where[0] != "cpu" else ([63, 2, 20, 1],):
+        if n:
+            close(feed(eng, toks, cuts)[:n], ref, where)
+
+
+def test_bf16_activations_on_the_reference_path():
+    cfg = plain("bfloat16")
+    w, toks = weights(cfg, 1), tokens(cfg, 50, 2)
+    U.close(feed(make_engine(cfg, w), toks), oracle(cfg, w, toks), "bfloat16")
+
+
+@ALL
+def test_residual_stream_after_every_layer(where):
+    cfg = plain(where[1])
+    w, toks = weights(cfg, 4), tokens(cfg, 45, 5)
+    ref = O.hidden_states(fanulix_config_to_json(cfg), w, toks)
+    eng = make_engine(cfg, w, where[0])
+    got = []
+    eng.model.on_layer = lambda i, x: got.append(x.double().cpu())
+    feed(eng, toks)
+    assert len(got) == len(ref) == 4
+    for a, b in zip(got, ref):
+        assert ((a - b).norm() / b.norm()).item() < {"float32": 1e-5, "bfloat16": 2e-2}[where[1]]
+
+
+@ALL
+@pytest.mark.parametrize("cuts", [[2], [3, 5], [7, 64, 1, 1, 30], [24], [65, 2], [64, 1, 63, 2]])
+def test_portions(where, cuts):
+    cfg = plain(where[1])
+    n = 200 if where[0] != "cpu" else 90
+    w, toks = weights(cfg, 6), tokens(cfg, n, 7)
+    close(feed(make_engine(cfg, w, where[0]), toks, cuts), oracle(cfg, w, toks), where)
+
+
+@ALL
+def test_long_decoding(where):
+    cfg = config((both(att(2, 1, 16, 16, every=60), ret(2, 8, 16, 8, decay=(0.999, 0.9))), None), (ssm(2, 16, 12, 1, 3, 1), moe(2, 2, 24, 24)),
+                 dtype=where[1], width=48, vocab=97)
+    n = 420 if where[0] != "cpu" else 150
+    w, toks = weights(cfg, 8), tokens(cfg, n, 9)
+    close(feed(make_engine(cfg, w, where[0]), toks, [9, 1]), oracle(cfg, w, toks), where)
+
+
+# ---- batches ----------------------------------------------------------------------------------------------
+@ALL
+def test_unequal_requests_in_one_step(where):
+    """Prompt portions (long and short) and decode rows of several requests share steps; each sees only its own tokens."""
+    cfg = plain(where[1])
+    w = weights(cfg, 10)
+    eng = make_engine(cfg, w, where[0], seqs=5)
+    lens = [1, 250, 37, 190, 64] if where[0] != "cpu" else [1, 100, 37, 90, 24]
+    seqs = [tokens(cfg, n, 20 + i) for i, n in enumerate(lens)]
+    plans = [[1], [64, 3, 130, 1], [35, 1], [2, 1, 1, 180, 1], [64]] if where[0] != "cpu" else [[1], [64, 3, 30, 1], [35, 1], [2, 1, 1, 80, 1], [24]]
+    reqs = [eng.open_sequence() for _ in lens]
+    got, at, turn = [[] for _ in lens], [0] * 5, [0] * 5
+    while any(a < n for a, n in zip(at, lens)):
+        spans = []
+        for i in range(5):
+            if at[i] < lens[i]:
+                spans.append((i, min(plans[i][min(turn[i], len(plans[i]) - 1)], lens[i] - at[i])))
+        rows = eng.feed([(reqs[i], seqs[i][at[i]:at[i] + n], list(range(n))) for i, n in spans]).double().cpu()
+        for i, n in spans:
+            got[i].append(rows[:n])
+            rows, at[i], turn[i] = rows[n:], at[i] + n, turn[i] + 1
+    for i in range(5):
+        close(torch.cat(got[i]), oracle(cfg, w, seqs[i]), where)
+
+
+@ALL
+def test_pages_and_rows_are_reused(where):
+    """Later requests run in pages and rows that earlier ones filled; a diverged predecessor leaves nothing behind."""
+    cfg = plain(where[1])
+    w = weights(cfg, 11)
+    eng = make_engine(cfg, w, where[0], ctx=256, seqs=1, chunk=256)
+    n = 190 if where[0] != "cpu" else 80
+    toks = tokens(cfg, n, 12)
+    ref = oracle(cfg, w, toks)
+    pages = eng.kv.full.num_pages
+    assert sorted(eng.kv.kv_cache) == [0, 2] and sorted(eng.kv.state) == [0, 1, 2, 3]
+    for i in range(3):
+        feed(eng, tokens(cfg, n - 31 * i, 30 + i), [50, 1, 20])
+    for cuts in ([100, 7, 1], [80, 110], [2, 1], [1]) if where[0] != "cpu" else ([50, 7, 1], [1]):
+        for t in list(eng.kv.kv_cache.values()) + [t for st in eng.kv.state.values() for t in st]:
+            t.fill_(float("nan"))                           # whatever is left behind must not be read
+        close(feed(eng, toks, cuts), ref, where)
+    assert len(eng.kv.full.free) == pages and len(eng.kv.free_rows) == 1
+
+
+@ALL
+def test_a_short_request_takes_over_a_row(where):
+    """Requests shorter than the convolution, one after the other in one row: the earlier one's last inputs are still there."""
+    cfg = config((ssm(conv=4), None), (both(), None), dtype=where[1])
+    w = weights(cfg, 12)
+    eng = make_engine(cfg, w, where[0], seqs=1)
+    feed(eng, tokens(cfg, 40, 1))
+    for n in (1, 2, 3, 5):
+        toks = tokens(cfg, n, n)
+        for cuts in (None, [1]):
+            close(feed(eng, toks, cuts), oracle(cfg, w, toks), where)
+
+
+# ---- what a position sees -----------------------------------------------------------------------------------
+@ALL
+def test_far_key_on_both_sides_of_page_borders(where):
+    """A key that stands out is found at page and block borders, in a prompt, a short portion and in decoding."""
+    cfg = config((both(att(2, 1, 32, 32, coef=0.1, every=64), ret(2, 8, 16, 8)), None), dtype=where[1])
+    n = 300 if where[0] != "cpu" else 150
+    eng = None
+    _, without = U.needle(cfg, None, n)
+    for at in (0, 1, 63, 64, 127, 128, 191, 255, 256, 298) if where[0] != "cpu" else (0, 63, 64, 128):
+        w, toks = U.needle(cfg, at, n)
+        eng = eng or make_engine(cfg, w, where[0])
+        ref = oracle(cfg, w, toks)[-1:]
+        for cuts in (None, [n - 1, 1], [n - 3, 3], [n - 100, 100]):
+            got = feed(eng, toks, cuts)[-1:]
+            close(got, ref, where)
+            assert error(got, feed(eng, without, cuts)[-1:]) > 0.3
+
+
+@ALL
+@pytest.mark.parametrize("kind", ["retention", "mamba2"])
+def test_far_token_through_the_state(where, kind):
+    """One token's trace in a slowly decaying state reaches the last position, wherever chunks and portions are cut."""
+    cfg = config((both(att(1, 1, 8, 8), ret(2, 16, 16, 8, decay=(0.9995, 0.999)), 0.0, 1.5), None) if kind == "retention" else
+                 (ssm(2, 24, 20, 1, 3, 1), None), dtype=where[1])
+    n = 200 if where[0] != "cpu" else 100
+    w = weights(cfg, 13)
+    w["embed"][2] = 10.0 * w["embed"][2].sign()
+    if kind == "mamba2":
+        w["l0.mix.A_log"].fill_(-6.0)
+        w["l0.mix.o"] = 3.0 * w["l0.mix.o"]
+    w = {k: t.to(torch.bfloat16).float() for k, t in w.items()}
+    eng = make_engine(cfg, w, where[0])
+    for at in (0, 22, 23, 63, 64, 65, n - 2):
+        toks = [3 + x % (cfg.vocab_size - 3) for x in tokens(cfg, n, 14)]
+        ref0 = oracle(cfg, w, toks)[-1:]
+        toks[at] = 2
+        ref = oracle(cfg, w, toks)
+        assert error(ref[-1:], ref0) > 3 * TOL[where[1]]
+        for cuts in (None, [at + 1, n], [max(at, 1), 1, 2, n]):
+            close(feed(eng, toks, cuts), ref, where)
+
+
+@ALL
+def test_first_tokens(where):
+    cfg = plain(where[1])
+    w, toks = weights(cfg, 15), tokens(cfg, 6, 16)
+    eng = make_engine(cfg, w, where[0])
+    for cuts in (None, [1], [2]):
+        close(feed(eng, toks, cuts), oracle(cfg, w, toks), where)
+
+
+CONSTANTS = {
+    "scale": (0, "mixer", "left", "scale", 0.05), "negative scale": (0, "mixer", "left", "scale", -0.3), "coef": (0, "mixer", "left", "q_temp", "coef", 2.5),
+    "every": (0, "mixer", "left", "q_temp", "every", 3), "left_scale": (0, "mixer", "left_scale", 1.9), "right_scale": (0, "mixer", "right_scale", -0.9),
+    "decay": (0, "mixer", "right", "decay", [0.999, 0.2, 0.6]), "rot.base": (0, "mixer", "right", "rot", "base", 20.0),
+    "rot.dims": (0, "mixer", "right", "rot", "dims", 4), "norm_groups": (1, "mixer", "norm_groups", 1), "groups": None,
+    "top": (0, "mlp", "router", "top", 1), "logit_scale": None, "eps": None,
+}
+
+
+@ALL
+@pytest.mark.parametrize("part", [k for k, v in CONSTANTS.items() if v or k in ("logit_scale", "eps")])
+def test_every_constant_counts(where, part):
+    """The logits follow each constant of the configuration."""
+    from stkernel_b200.models.registry import config_from_json
+    cfg = plain(where[1])
+    other = json.loads(json.dumps(fanulix_config_to_json(cfg)))
+    if part == "logit_scale":
+        other["logit_scale"] = 1.3
+    elif part == "eps":
+        other["norm"]["eps"] = 0.5
+    else:
+        li, *path, key, value = CONSTANTS[part]
+        d = other["layers"][li]
+        for k in path:
+            d = d[k]
+        assert d[key] != value
+        d[key] = value
+    cfg2 = config_from_json(other, where[1])
+    w, toks = weights(cfg, 17), tokens(cfg, 80, 18)
+    if part == "top":
+        w["l0.mlp.router"] *= 4.0
+        if where[1] != "float32":
+            toks = toks[:max(1, U.clear_routing(cfg2, w, toks, 0.2))]
+    ref = O.logits(other, w, toks)
+    close(feed(make_engine(cfg2, w, where[0]), toks), ref, where)
+    assert error(oracle(cfg, w, toks), ref) > 2 * TOL[where[1]]
+
+
+# ---- generation -----------------------------------------------------------------------------------------------
+@EXACT
+@pytest.mark.parametrize("sched", [dict(), dict(chunk=24), dict(seqs=2), dict(async_scheduling=True)])
+def test_greedy_generation_equals_the_oracle(where, sched):
+    cfg = mixed(where[1])
+    w = weights(cfg, 19)
+    prompts = [tokens(cfg, n, 40 + n) for n in (5, 1, 61, 26)]
+    eng = make_engine(cfg, w, where[0], graph_cap=4, **sched)
+    got = eng.generate(prompts, SamplingParams(max_tokens=7))
+    for p, g in zip(prompts, got):
+        assert g == O.greedy(fanulix_config_to_json(cfg), w, p, 7)
+    assert eng.kv.full.pages_in_use == 0 and not eng.kv.reserved
+    assert len(eng.kv.free_rows) == eng.cfg.sched.max_num_seqs
+
+
+@ALL
+def test_batch_and_alone_sample_the_same_text(where):
+    cfg = plain(where[1])
+    w = weights(cfg, 20)
+    prompts = [tokens(cfg, n, 60 + n) for n in (30, 4, 77)]
+    par = SamplingParams(temperature=0.7, seed=5, max_tokens=12, top_k=20)
+    alone = [make_engine(cfg, w, where[0], graph_cap=4).generate([p], par)[0] for p in prompts]
+    together = make_engine(cfg, w, where[0], graph_cap=4, chunk=40).generate(prompts, par)
+    if where[1] == "float32":
+        assert together == alone
+    else:                       # rounding may flip a sampled token; the first ones agree
+        assert all(a[:2] == b[:2] for a, b in zip(alone, together))
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_captured_decode_steps_follow_eager_ones(dtype):
+    """Graphs of several batch sizes and context buckets, replayed in turn, give what eager steps give (capturing one advances no
+    state)."""
+    cfg = plain(dtype)
+    w = weights(cfg, 21)
+    prompts = [tokens(cfg, n, 80 + n) for n in (1000, 1015, 30, 2)]
+    outs = []
+    for cap in (0, 4):
+        eng = make_engine(cfg, w, "cuda:0", ctx=1200, chunk=1200, graph_cap=cap)
+        outs.append([eng.generate(prompts[:k], SamplingParams(max_tokens=20)) for k in (1, 4, 2, 1)])
+    flat = [[t for run in o for text in run for t in text] for o in outs]
+    same = sum(a == b for a, b in zip(*flat)) / len(flat[0])
+    assert len(flat[0]) == len(flat[1]) and same > (0.99 if dtype == "float32" else 0.7)
+    assert outs[1][0][0] == outs[1][3][0]                   # the same graph before and after the larger ones were captured
+
+
+@EXACT
+def test_requests_wait_for_pages(where):
+    """A pool smaller than all contexts together: requests are admitted as others end, and give the same text."""
+    from stkernel_b200.models.hybrid import build_hybrid_weights
+    from stkernel_b200.models.sources import DictSource
+    from stkernel_b200.runtime.engine import Engine
+    cfg = plain(where[1])
+    w = weights(cfg, 22)
+    prompts = [tokens(cfg, n, 90 + n) for n in (120, 60, 100, 10)]
+    want = make_engine(cfg, w, where[0]).generate(prompts, SamplingParams(max_tokens=6))
+    ec = EngineConfig(model=cfg, sched=SchedulerConfig(max_model_len=192, max_num_seqs=4, max_num_batched_tokens=64, graph_cap=0),
+                      cache=CacheConfig(kv_pool_tokens=256)).validate()
+    eng = Engine(ec, build_hybrid_weights(cfg, DictSource(w), where[0]), where[0], max_context=192)
+    assert eng.kv.full.num_pages <= 5 and not eng.kv.fits(1000)
+    ids = [eng.add_request(p, SamplingParams(max_tokens=6)) for p in prompts]
+    most = 0
+    while eng.has_work():
+        eng.step()
+        most = max(most, eng.sched.num_running)
+    assert [eng.requests[i].output for i in ids] == want and 1 < most < 4
+    assert eng.kv.full.pages_in_use == 0 and eng.kv.usage() == 0
+
+
+# ---- product interfaces -----------------------------------------------------------------------------------------
+def save_model(path, cfg, w):
+    from stkernel_b200.models.loader import write_safetensors
+    os.makedirs(path, exist_ok=True)
+    write_safetensors(os.path.join(path, "model.safetensors"), {k: t.to(torch.bfloat16).contiguous() for k, t in w.items()}, {})
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(fanulix_config_to_json(cfg), f)
+
+
+@ALL
+def test_trace_replay(where, tmp_path):
+    """Logits of a replayed trace are the engine's; requests come and go, portions longer than a step are cut."""
+    import numpy as np
+    from stkernel_b200.models.loader import CheckpointSource
+    from stkernel_b200.models.registry import family_of, load_model_config
+    from stkernel_b200.runtime.engine import Engine
+    from stkernel_b200.serve.trace_run import run
+    cfg = plain(where[1])
+    w = weights(cfg, 23)
+    save_model(tmp_path / "m", cfg, w)
+    loaded = load_model_config(str(tmp_path / "m"), where[1])
+    assert loaded == cfg
+    src = CheckpointSource(str(tmp_path / "m"))
+    assert not src.missing(loaded) and not src.unexpected(loaded)
+    ec = make_engine(cfg, w, "cpu", chunk=90, seqs=2).cfg
+    eng = Engine(ec, family_of(loaded).build_weights(loaded, src, where[0]), where[0], max_context=640)
+    a, b = tokens(cfg, 110, 1), tokens(cfg, 30, 2)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:100], "want": [99, 0, 41]}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": b[:20], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": a[100:], "want": [3]}, {"id": "b", "tokens": b[20:], "want": [9]}],
+              "end": ["a", "b"]},
+             {"step": 3, "entries": [{"id": "a", "tokens": b, "want": [5]}], "end": ["a"]}]
+    done = []
+    run(eng, [json.dumps(s) for s in steps], str(tmp_path), done.append)
+    assert done == [0, 1, 2, 3] and not (tmp_path / "1.f32").exists()
+    ra, rb = oracle(cfg, w, a), oracle(cfg, w, b)
+    for n, ref in ((0, ra[[99, 0, 41]]), (2, torch.stack([ra[103], rb[29]])), (3, rb[[5]])):
+        got = torch.from_numpy(np.fromfile(tmp_path / f"{n}.f32", dtype="<f4").copy()).view(-1, cfg.vocab_size).double()
+        assert error(got, ref) < TOL[where[1]]
+    assert len(eng.kv.free_rows) == 2
+
+
+def test_greedy_text_over_http(tmp_path):
+    """The server command on a checkpoint of weights alone: tokens are the oracle's."""
+    from fastapi.testclient import TestClient
+    from stkernel_b200.serve.api_server import create_app
+    from stkernel_b200.serve.tp_worker import build_engine, make_parser, make_tokenizer
+    cfg = mixed("float32", vocab=400)
+    w = weights(cfg, 24)
+    save_model(tmp_path, cfg, w)
+    a = make_parser().parse_args(["--model", str(tmp_path), "--dtype", "float32", "--max-model-len", "256", "--max-num-seqs", "3",
+                                  "--max-num-batched-tokens", "64"])
+    eng, mcfg = build_engine(a, 0, 1, torch.device("cpu"))
+    assert mcfg == cfg
+    tok = make_tokenizer(a, mcfg)
+    with TestClient(create_app(eng, tok, "fanulix")) as c:
+        ids = tok.encode("a text to continue")
+        want = tok.decode(O.greedy(fanulix_config_to_json(cfg), w, ids, 6))
+        body = {"prompt": ["a text to continue", "b"], "max_tokens": 6, "temperature": 0, "ignore_eos": True}
+        r = c.post("/v1/completions", json=body).json()
+        assert r["choices"][0]["text"].rstrip("�") == want.rstrip("�")
+        assert "vllm:gpu_cache_usage_perc" in c.get("/metrics").text
+
+
+@pytest.mark.parametrize("path,value,word", [
+    (("layers", 0, "type"), "attention", "mixer"), (("layers", 0, "type"), "mamba2", "unknown|missing"), (("streams",), 0, "streams"),
+    (("streams",), 9, "streams"), (("logit_scale",), "x", "logit_scale"), (("layers", 0, "mixer", "left", "kv_heads"), 3, "kv_heads"),
+    (("layers", 0, "mixer", "left", "q_temp", "every"), 0, "every"), (("layers", 0, "mixer", "left", "q_temp"), {}, "coef"),
+    (("layers", 0, "mixer", "left", "vdim"), -1, "vdim"), (("layers", 0, "mixer", "right", "decay"), [0.5], "decay"),
+    (("layers", 0, "mixer", "right", "decay"), [0.5, 0.0, 0.1], "decay"), (("layers", 0, "mixer", "right", "rot", "dims"), 18, "rot.dims"),
+    (("layers", 0, "mixer", "left_scale"), None, "left_scale"), (("layers", 0, "mixer", "extra"), 1, "extra"),
+    (("layers", 1, "mixer", "groups"), 3, "groups"), (("layers", 1, "mixer", "norm_groups"), 5, "norm_groups"),
+    (("layers", 1, "mixer", "conv"), 0, "conv"), (("layers", 1, "mixer", "state"), 2.5, "state"), (("layers", 0, "mlp", "kind"), "dense", "feed-forward"),
+    (("layers", 0, "mlp", "router", "top"), 7, "top"), (("layers", 0, "mlp", "shared"), {}, "ff"), (("layers", 0, "mlp", "shared", "ff"), 0, "shared"),
+    (("layers", 0, "mlp", "expert", "ff"), "8", "expert"), (("norm", "eps"), 0, "eps"), (("vocab",), None, "vocab")])
+def test_bad_configurations_name_the_field(path, value, word):
+    from stkernel_b200.config import ConfigError, tiny_streams_config
+    from stkernel_b200.models.registry import config_from_json
+    d = json.loads(json.dumps(fanulix_config_to_json(tiny_streams_config())))
+    assert config_from_json(d) == tiny_streams_config()
+    at = d
+    for k in path[:-1]:
+        at = at[k]
+    at[path[-1]] = value
+    with pytest.raises(ConfigError, match=word):
+        config_from_json(d)
+
+
+def test_mixers_that_this_build_does_not_combine_are_refused():
+    from stkernel_b200.config import ConfigError, HybridConfig, HybridLayer, ParallelMixer
+    for m, block in ((ssm(), "parallel"), (both(), "parallel"), (att(), "streams"), (ret(), "streams"), (ParallelMixer(ret(), att()), "streams")):
+        with pytest.raises(ConfigError):
+            HybridConfig(64, 32, (HybridLayer(m),), block=block).validate()
+
+
+def test_configuration_round_trips_and_sources_follow_the_mechanisms():
+    from stkernel_b200.config import streams_stack, tiny_latent_config, tiny_streams_config
+    from stkernel_b200.csrc.build import sources
+    from stkernel_b200.models.registry import config_from_json, family_of
+    cfg = tiny_streams_config()
+    e = EngineConfig(model=cfg, sched=SchedulerConfig(max_num_seqs=3)).validate()
+    assert EngineConfig.from_dict(json.loads(e.resolved())) == e
+    assert config_from_json(fanulix_config_to_json(cfg), "float32") == dataclasses.replace(cfg, dtype="float32")
+    big = streams_stack(4, 256, 4, 4, 2, 64, 64, 2, 64, 128, 8, 64, 64, 2, 8, 2, 64, 128, 512)
+    assert config_from_json(fanulix_config_to_json(big)) == big
+    name, files = family_of(cfg).native_sources(cfg)
+    other, theirs = family_of(tiny_latent_config()).native_sources(tiny_latent_config())
+    assert name != other and len(set(files)) == len(files) and "mamba2.cu" in files and "mamba2.cu" not in theirs
+    assert all(f.exists() for f in sources(files) + sources(theirs))
+    only_ssm = dataclasses.replace(cfg, layers=cfg.layers[1:])
+    assert "grouped_attention.cu" not in family_of(only_ssm).native_sources(only_ssm)[1]
+
+
+@EXACT
+def test_a_model_without_attention_needs_no_pages(where):
+    """Only recurrent layers: requests are bounded by rows, and generate as the oracle does."""
+    cfg = config(ssm(), (ssm(2, 16, 12, 1, 3, 1), None), dtype=where[1])
+    w = weights(cfg, 25)
+    eng = make_engine(cfg, w, where[0], seqs=2, graph_cap=4)
+    assert eng.kv.full is None and not eng.kv.kv_cache
+    prompts = [tokens(cfg, n, n) for n in (40, 3, 9)]
+    for p, g in zip(prompts, eng.generate(prompts, SamplingParams(max_tokens=5))):
+        assert g == O.greedy(fanulix_config_to_json(cfg), w, p, 5)
