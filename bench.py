@@ -106,6 +106,16 @@ def latent_arm(args) -> None:
     print(json.dumps({"metric": "latent_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
 
 
+def streams_arm(args) -> None:
+    import torch
+    from stkernel_b200.bench import hybrid_bench, streams_bench
+    torch.cuda.set_device(0)
+    with ClockSampler(0) as clocks:
+        res = streams_bench.run([int(x) for x in args.streams_sizes.split(",")], beside=not args.streams_alone)
+    print(hybrid_bench.render(res), file=sys.stderr)
+    print(json.dumps({"metric": "streams_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -127,7 +137,14 @@ def main() -> None:
                          "and expert counts, prefill, decode and per-kernel rooflines (one JSON line; table on stderr)")
     ap.add_argument("--latent-sizes", default="2048,4096", help="widths for --latent")
     ap.add_argument("--latent-alone", action="store_true", help="with --latent: without the flagship's architecture beside it")
+    ap.add_argument("--streams", action="store_true",
+                    help="instead of the flagship: the Fanulix decoder beside Timalorn and Domilix at equal width and depth, prefill, "
+                         "decode and per-kernel rooflines (one JSON line; table on stderr)")
+    ap.add_argument("--streams-sizes", default="2048,4096", help="widths for --streams")
+    ap.add_argument("--streams-alone", action="store_true", help="with --streams: without the other decoders beside it")
     args = ap.parse_args()
+    if args.streams:
+        return streams_arm(args)
     if args.hybrid:
         return hybrid_arm(args)
     if args.latent:

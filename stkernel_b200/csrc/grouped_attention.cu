@@ -104,6 +104,64 @@ grouped_prep_kernel(const GqArgs a, int vec_in, int vec_row) {
   gq_store(row + a.k_col, k, kb, a.D, a.row - a.k_col, a.norm ? gq_inv_rms(k, kb, a.D, a.eps, vec_in, lane) : 1.f, vec_row, lane);
 }
 
+// bf16 with everything in whole groups of eight: one CTA per token, L lanes per head, eight columns a lane.
+template <int L>
+__global__ void __launch_bounds__(512)
+grouped_prep_vec_kernel(const GqArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.x;
+  const int group = threadIdx.x / L, l = threadIdx.x % L, groups = blockDim.x / L, c = l * 8;
+  const int req = a.tok_req[t];
+  const long long pos = a.positions[t];
+  const bool live = req >= 0 && pos >= 0;
+  const int page = live ? a.table[static_cast<long long>(req) * a.bt_stride + pos / kGqPage] : -1;
+  const float temp = live && a.coef != 0.f ? 1.f + a.coef * logf(static_cast<float>(floor(static_cast<double>(pos + 1) / a.every)) + 1.f) : 1.f;
+  const __nv_bfloat16* p = reinterpret_cast<const __nv_bfloat16*>(a.proj) + t * a.ldp;
+  const int units = a.H + 2 * a.G, rounds = (units + groups - 1) / groups;
+  for (int i = 0; i < rounds; ++i) {                                  // query heads, key heads, value heads
+    const int u = i * groups + group;
+    const bool q = u < a.H, k = !q && u < a.H + a.G, ok = u < units;
+    const int g = q ? u : k ? u - a.H : u - a.H - a.G, n = q || k ? a.D : a.V;
+    float x[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] = 0.f;
+    if (ok && c < n) {
+      const uint4 v = *reinterpret_cast<const uint4*>(p + (q ? a.q_off : k ? a.k_off : a.v_off) + g * n + c);
+      const float* b = a.bias != nullptr ? a.bias + (q ? 0 : k ? a.H * a.D : (a.H + a.G) * a.D) + g * n + c : nullptr;
+      float4 b0 = make_float4(0.f, 0.f, 0.f, 0.f), b1 = b0;
+      if (b != nullptr) {
+        b0 = *reinterpret_cast<const float4*>(b);
+        b1 = *reinterpret_cast<const float4*>(b + 4);
+      }
+      const float bb[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
+        x[2 * j] = f.x + bb[2 * j];
+        x[2 * j + 1] = f.y + bb[2 * j + 1];
+      }
+    }
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s = fmaf(x[j], x[j], s);
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    float f = a.norm && (q || k) ? 1.f / sqrtf(s / static_cast<float>(n) + a.eps) : 1.f;
+    if (q) f = live ? f * temp : 0.f;
+    uint4 r;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) reinterpret_cast<__nv_bfloat162*>(&r)[j] = __floats2bfloat162_rn(x[2 * j] * f, x[2 * j + 1] * f);
+    if (!ok) continue;
+    if (q) {
+      if (c < a.dp) *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(a.q) + (t * a.H + g) * a.dp + c) = r;
+    } else if (page >= 0) {
+      __nv_bfloat16* row = reinterpret_cast<__nv_bfloat16*>(a.cache) + ((static_cast<long long>(page) * a.G + g) * kGqPage + pos % kGqPage) * a.row;
+      if (c < (k ? a.row - a.k_col : a.k_col)) *reinterpret_cast<uint4*>(row + (k ? a.k_col : 0) + c) = r;
+    }
+  }
+}
+
 }  // namespace stk
 
 using namespace stk;
@@ -125,6 +183,14 @@ STK_API int stk_grouped_prep(const void* proj, long long ldp, int q_off, int k_o
   const uintptr_t at = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache);
   const int vec_in = !fp32 && dim % 4 == 0 && dp % 4 == 0 && ldp % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && (at & 7) == 0;
   const int vec_row = vec_in && vdim % 4 == 0 && v_off % 4 == 0 && k_col % 4 == 0 && row % 4 == 0;
+  const int widest = dp > row - k_col ? (dp > k_col ? dp : k_col) : (row - k_col > k_col ? row - k_col : k_col);
+  if (!fp32 && (dim | vdim | dp | row | k_col | q_off | k_off | v_off) % 8 == 0 && ldp % 8 == 0 && widest <= 256 &&
+      ((at | reinterpret_cast<uintptr_t>(bias)) & 15) == 0) {
+    const int threads = T <= 148 ? 512 : 256;                        // few tokens: a token's heads side by side
+    if (widest <= 128) launch_pdl(grouped_prep_vec_kernel<16>, dim3(T), dim3(threads), 0, (cudaStream_t)stream, a);
+    else launch_pdl(grouped_prep_vec_kernel<32>, dim3(T), dim3(threads), 0, (cudaStream_t)stream, a);
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  }
   const long long warps = static_cast<long long>(T) * (heads + kv_heads);
   const dim3 grid(static_cast<unsigned>((warps + kGqWarps - 1) / kGqWarps));
   cudaStream_t st = (cudaStream_t)stream;

@@ -231,46 +231,58 @@ struct StreamArgs {
   const int64_t* rows;
 };
 
-// N consecutive columns of one row: the sublayer's output, all streams, their update; returns u in `row` and adds its sum.
-template <typename A, int S, int N>
-__device__ __forceinline__ float stream_columns(const StreamArgs<A>& a, float* xr, long long r, int i, const long long* src,
-                                                const float* wt, const float (&mix)[S][S], const float (&write)[S],
-                                                const float (&read)[S], float* row, bool has_y, bool store) {
-  float v[S][N], y[N];
+// N consecutive columns of one row in all streams, before their update.
+template <int S, int N>
+__device__ __forceinline__ void load_streams(const float* xr, int W, int i, float (&v)[S][N]) {
 #pragma unroll
   for (int s = 0; s < S; ++s) {
     if constexpr (N == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(xr + s * a.W + i);
+      const float4 f = *reinterpret_cast<const float4*>(xr + s * W + i);
       v[s][0] = f.x; v[s][1] = f.y; v[s][2] = f.z; v[s][3] = f.w;
     } else {
-      v[s][0] = xr[s * a.W + i];
+      v[s][0] = xr[s * W + i];
     }
   }
-  if (has_y) {
+}
+
+// The same columns of the sublayer's output.
+template <typename A, int N>
+__device__ __forceinline__ void load_output(const StreamArgs<A>& a, long long r, int i, const long long* src, const float* wt, float (&y)[N]) {
 #pragma unroll
-    for (int k = 0; k < N; ++k) y[k] = 0.f;
-    if (a.pairs != nullptr) {
-      for (int j = 0; j < a.top; ++j) {
-        const A* p = a.pairs + src[j] + i;
-        if constexpr (N == 4 && sizeof(A) == 2) {
-          const uint2 q = *reinterpret_cast<const uint2*>(p);
-          const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
-          const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
-          y[0] = fmaf(wt[j], f0.x, y[0]); y[1] = fmaf(wt[j], f0.y, y[1]);
-          y[2] = fmaf(wt[j], f1.x, y[2]); y[3] = fmaf(wt[j], f1.y, y[3]);
-        } else {
+  for (int k = 0; k < N; ++k) y[k] = 0.f;
+  if (a.pairs != nullptr) {
+    if constexpr (N == 4 && sizeof(A) == 2) {
+      for (int j0 = 0; j0 < a.top; j0 += 4) {                     // four rows in flight
+        uint2 q[4];
 #pragma unroll
-          for (int k = 0; k < N; ++k) y[k] = fmaf(wt[j], ld_act(p + k), y[k]);
+        for (int j = 0; j < 4; ++j)
+          q[j] = j0 + j < a.top ? *reinterpret_cast<const uint2*>(a.pairs + src[j0 + j] + i) : make_uint2(0, 0);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float w = j0 + j < a.top ? wt[j0 + j] : 0.f;
+          const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j].x));
+          const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j].y));
+          y[0] = fmaf(w, f0.x, y[0]); y[1] = fmaf(w, f0.y, y[1]);
+          y[2] = fmaf(w, f1.x, y[2]); y[3] = fmaf(w, f1.y, y[3]);
         }
       }
-    } else if constexpr (N == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(a.y + r * a.ldy + i);
-      y[0] = f.x; y[1] = f.y; y[2] = f.z; y[3] = f.w;
     } else {
-      y[0] = a.y[r * a.ldy + i];
+      for (int j = 0; j < a.top; ++j)
+#pragma unroll
+        for (int k = 0; k < N; ++k) y[k] = fmaf(wt[j], ld_act(a.pairs + src[j] + i + k), y[k]);
     }
+  } else if constexpr (N == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(a.y + r * a.ldy + i);
+    y[0] = f.x; y[1] = f.y; y[2] = f.z; y[3] = f.w;
+  } else {
+    y[0] = a.y[r * a.ldy + i];
   }
-  float u[N], sum = 0.f;
+}
+
+// Streams after the update (stored if `store`) and u = sum_s read[s] x_s.
+template <int S, int N>
+__device__ __forceinline__ void mix_streams(float* xr, int W, int i, const float (&v)[S][N], const float (&y)[N], const float (&mix)[S][S],
+                                            const float (&write)[S], const float (&read)[S], float (&u)[N], bool has_y, bool store) {
 #pragma unroll
   for (int k = 0; k < N; ++k) u[k] = 0.f;
 #pragma unroll
@@ -288,19 +300,15 @@ __device__ __forceinline__ float stream_columns(const StreamArgs<A>& a, float* x
       u[k] = fmaf(read[t], n[k], u[k]);
     }
     if (store) {
-      if constexpr (N == 4) *reinterpret_cast<float4*>(xr + t * a.W + i) = make_float4(n[0], n[1], n[2], n[3]);
-      else xr[t * a.W + i] = n[0];
+      if constexpr (N == 4) *reinterpret_cast<float4*>(xr + t * W + i) = make_float4(n[0], n[1], n[2], n[3]);
+      else xr[t * W + i] = n[0];
     }
   }
-#pragma unroll
-  for (int k = 0; k < N; ++k) {
-    row[i + k] = u[k];
-    sum += u[k];
-  }
-  return sum;
 }
 
-template <typename A, int S>
+// NIT > 0: a thread's NIT groups of four columns stay in registers (W a multiple of 4, at most NIT * 4 * blockDim.x); 0: any width, the
+// row in shared memory.
+template <typename A, int S, int NIT>
 __global__ void __launch_bounds__(1024)
 stream_norm_kernel(const StreamArgs<A> a) {
   extern __shared__ __align__(16) float row[];
@@ -311,14 +319,11 @@ stream_norm_kernel(const StreamArgs<A> a) {
   pdl_trigger();
   const long long r = a.rows != nullptr ? a.rows[blockIdx.x] : static_cast<long long>(blockIdx.x);
   const bool has_y = a.y != nullptr || a.pairs != nullptr, store = has_y && a.rows == nullptr;
-  if (a.pairs != nullptr) {
-    if (static_cast<int>(threadIdx.x) < a.top) {
-      const long long p = r * a.top + threadIdx.x;
-      const int at = a.pair_row != nullptr ? a.pair_row[p] : static_cast<int>(p);
-      src[threadIdx.x] = at < 0 ? 0 : at * a.ldp;
-      wt[threadIdx.x] = at < 0 ? 0.f : a.weights[p];
-    }
-    __syncthreads();
+  if (a.pairs != nullptr && static_cast<int>(threadIdx.x) < a.top) {
+    const long long p = r * a.top + threadIdx.x;
+    const int at = a.pair_row != nullptr ? a.pair_row[p] : static_cast<int>(p);
+    src[threadIdx.x] = at < 0 ? 0 : at * a.ldp;
+    wt[threadIdx.x] = at < 0 ? 0.f : a.weights[p];
   }
   float mix[S][S], write[S], read[S];
 #pragma unroll
@@ -329,29 +334,83 @@ stream_norm_kernel(const StreamArgs<A> a) {
     for (int t = 0; t < S; ++t) mix[s][t] = has_y ? a.mix[s * S + t] : 0.f;
   }
   float* xr = a.x + r * S * a.W;
-  float sum = 0.f;
-  if ((a.W & 3) == 0 && (a.ldy & 3) == 0 && (a.ldp & 3) == 0) {
-    for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4)
-      sum += stream_columns<A, S, 4>(a, xr, r, i, src, wt, mix, write, read, row, has_y, store);
-  } else {
-    for (int i = threadIdx.x; i < a.W; i += blockDim.x)
-      sum += stream_columns<A, S, 1>(a, xr, r, i, src, wt, mix, write, read, row, has_y, store);
-  }
-  const float mean = block_sum(sum, red) / static_cast<float>(a.W);          // also publishes the row
-  float q = 0.f;
-  for (int i = threadIdx.x; i < a.W; i += blockDim.x) {
-    const float d = row[i] - mean;
-    q = fmaf(d, d, q);
-  }
-  const float inv = 1.f / sqrtf(block_sum(q, red) / static_cast<float>(a.W) + a.eps);
   A* hr = a.h + blockIdx.x * a.ldh;
-  if (sizeof(A) == 2 && (a.width & 1) == 0 && (a.ldh & 1) == 0) {
-    for (int i = threadIdx.x * 2; i < a.width; i += blockDim.x * 2) {
-      const float c = i < a.W ? fmaf((row[i] - mean) * inv, a.w[i], a.b[i]) : 0.f;
-      const float d = i + 1 < a.W ? fmaf((row[i + 1] - mean) * inv, a.w[i + 1], a.b[i + 1]) : 0.f;
-      *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(hr) + i) = __floats2bfloat162_rn(c, d);
+  const float n = static_cast<float>(a.W);
+  if constexpr (NIT > 0) {
+    float u[NIT][4], sum = 0.f;
+    float4 w = make_float4(0.f, 0.f, 0.f, 0.f), b = w;
+    float v[S][4], y[4];
+    const int i0 = threadIdx.x * 4;
+    if (i0 < a.W) {                                                      // before the wait for the expert rows' places
+      load_streams<S, 4>(xr, a.W, i0, v);
+      if (NIT == 1) {
+        w = *reinterpret_cast<const float4*>(a.w + i0);
+        b = *reinterpret_cast<const float4*>(a.b + i0);
+      }
     }
+    if (a.pairs != nullptr) __syncthreads();
+#pragma unroll
+    for (int e = 0; e < NIT; ++e) {
+      const int i = i0 + e * blockDim.x * 4;
+      if (i < a.W) {
+        if (e > 0) load_streams<S, 4>(xr, a.W, i, v);
+        if (has_y) load_output<A, 4>(a, r, i, src, wt, y);
+        mix_streams<S, 4>(xr, a.W, i, v, y, mix, write, read, u[e], has_y, store);
+        sum += (u[e][0] + u[e][1]) + (u[e][2] + u[e][3]);
+      } else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) u[e][k] = 0.f;
+      }
+    }
+    const float mean = block_sum(sum, red) / n;
+    float q = 0.f;
+#pragma unroll
+    for (int e = 0; e < NIT; ++e)
+      if (i0 + e * static_cast<int>(blockDim.x) * 4 < a.W) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          u[e][k] -= mean;
+          q = fmaf(u[e][k], u[e][k], q);
+        }
+      }
+    const float inv = 1.f / sqrtf(block_sum(q, red) / n + a.eps);
+#pragma unroll
+    for (int e = 0; e < NIT; ++e) {
+      const int i = i0 + e * blockDim.x * 4;
+      if (i >= a.W) continue;
+      if (NIT > 1) {
+        w = *reinterpret_cast<const float4*>(a.w + i);
+        b = *reinterpret_cast<const float4*>(a.b + i);
+      }
+      const float o[4] = {fmaf(u[e][0] * inv, w.x, b.x), fmaf(u[e][1] * inv, w.y, b.y), fmaf(u[e][2] * inv, w.z, b.z),
+                          fmaf(u[e][3] * inv, w.w, b.w)};
+      if (sizeof(A) == 2 && (a.ldh & 3) == 0) {
+        __align__(8) __nv_bfloat162 pk[2] = {__floats2bfloat162_rn(o[0], o[1]), __floats2bfloat162_rn(o[2], o[3])};
+        *reinterpret_cast<uint2*>(hr + i) = *reinterpret_cast<const uint2*>(pk);
+      } else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) st_act(hr + i + k, o[k]);
+      }
+    }
+    for (int i = a.W + threadIdx.x; i < a.width; i += blockDim.x) st_act(hr + i, 0.f);
   } else {
+    if (a.pairs != nullptr) __syncthreads();
+    float sum = 0.f;
+    for (int i = threadIdx.x; i < a.W; i += blockDim.x) {
+      float v[S][1], y[1], u[1];
+      load_streams<S, 1>(xr, a.W, i, v);
+      if (has_y) load_output<A, 1>(a, r, i, src, wt, y);
+      mix_streams<S, 1>(xr, a.W, i, v, y, mix, write, read, u, has_y, store);
+      row[i] = u[0];
+      sum += u[0];
+    }
+    const float mean = block_sum(sum, red) / n;                          // also publishes the row
+    float q = 0.f;
+    for (int i = threadIdx.x; i < a.W; i += blockDim.x) {
+      const float d = row[i] - mean;
+      q = fmaf(d, d, q);
+    }
+    const float inv = 1.f / sqrtf(block_sum(q, red) / n + a.eps);
     for (int i = threadIdx.x; i < a.width; i += blockDim.x)
       st_act(hr + i, i < a.W ? fmaf((row[i] - mean) * inv, a.w[i], a.b[i]) : 0.f);
   }
@@ -359,12 +418,19 @@ stream_norm_kernel(const StreamArgs<A> a) {
 
 template <typename A, int S>
 static int launch_stream_norm(const StreamArgs<A>& a, int T, cudaStream_t st) {
-  const size_t smem = static_cast<size_t>(a.W) * sizeof(float);
-  if (smem > 40 * 1024 &&
-      cudaFuncSetAttribute(stream_norm_kernel<A, S>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
-    return -3;
   const int threads = T > 148 || a.W <= 1024 ? 256 : (a.W <= 2048 ? 512 : 1024);
-  launch_pdl(stream_norm_kernel<A, S>, dim3(T), dim3(threads), smem, st, a);
+  const int its = a.W % 4 == 0 && a.ldy % 4 == 0 && a.ldp % 4 == 0 ? (a.W / 4 + threads - 1) / threads : 99;
+  if (its == 1) launch_pdl(stream_norm_kernel<A, S, 1>, dim3(T), dim3(threads), 0, st, a);
+  else if (its == 2) launch_pdl(stream_norm_kernel<A, S, 2>, dim3(T), dim3(threads), 0, st, a);
+  else if (its <= 4) launch_pdl(stream_norm_kernel<A, S, 4>, dim3(T), dim3(threads), 0, st, a);
+  else if (its <= 8) launch_pdl(stream_norm_kernel<A, S, 8>, dim3(T), dim3(threads), 0, st, a);
+  else {
+    const size_t smem = static_cast<size_t>(a.W) * sizeof(float);
+    if (smem > 40 * 1024 &&
+        cudaFuncSetAttribute(stream_norm_kernel<A, S, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return -3;
+    launch_pdl(stream_norm_kernel<A, S, 0>, dim3(T), dim3(threads), smem, st, a);
+  }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -412,7 +412,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         const float g = (a.gate != nullptr ? lat_sigmoid(a.gate[t * a.ldg + h]) : 1.f) * a.out_scale / l;
         __nv_bfloat16* out = a.out + t * a.ldo + h * a.vp;
         const __nv_bfloat16* og = a.ogate != nullptr ? a.ogate + t * a.ldog + h * a.vp : nullptr;
-        const bool vec = ((a.vp | a.vw) & 7) == 0 && (a.ldo & 7) == 0 && (og == nullptr || ((a.ldog & 7) == 0 && (reinterpret_cast<uintptr_t>(og) & 15) == 0));
+        const bool vec = ((a.vp | a.vw) & 7) == 0 && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(og)) & 15) == 0;
         for (int c = 0; c < a.v_panels * 64; c += 16) {
           uint32_t o[16];
           __syncwarp();
@@ -550,7 +550,6 @@ STK_API int stk_prompt_attention(const void* q, long long ldq, const int* query_
   a.h0_kv = 0; a.heads_per_kv = heads / kv_heads; a.kv_step = row; a.k_off = k_col; a.v_off = 0;
   a.sink = sink; a.ogate = (const __nv_bfloat16*)gate; a.ldog = ldg; a.out_scale = out_scale;
   a.slots = lp_slots(dp, 0, vdim);
-  if (reinterpret_cast<uintptr_t>(out) & 15) return -1;
   CUtensorMap tq, te;
   const long long cols = static_cast<long long>(kv_heads) * row;
   if (make_tmap_2d(&tq, q, 2, T, static_cast<long long>(heads) * dp, ldq, kLpTile) != 0) return -3;

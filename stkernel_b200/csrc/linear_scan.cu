@@ -4,12 +4,14 @@
 //   o_t   = exp(F_t) S_start^T q_t + sum_{j <= t} exp(F_t - F_j) w_j (k_j . q_t) v_j  (+ skip v_t)
 //   S_end = exp(F_end) S_start + sum_j exp(F_end - F_j) w_j k_j v_j^T
 //
-//   linear_chunk_state     one CTA per 64 x 64 block of a head's state walks the chunks of a request with the block in its
-//                          accumulators and leaves the state before each chunk as bf16 pairs (high part and remainder)
-//   linear_chunk_out       per chunk, head and 64 or 128 value columns: the outputs
+//   linear_chunk_state     one CTA per 64 x 64 block of a head's state (transposed: 16 value rows per warp) walks the chunks of a
+//                          request with the block in its accumulators and leaves the state before each chunk
+//   linear_chunk_out       per chunk, head and 64 or 128 value columns: the outputs, 16 columns per warp
 //
-// Both run on the tensor cores.  fp32 operands (weighted keys, weighted scores, the state; queries and keys where they come as
-// pairs) enter the products as bf16 pairs, so they keep 16 mantissa bits.
+// Both run on the tensor cores.  fp32 operands (weighted values, weighted scores, the state; queries and keys where they come as
+// pairs) enter the products as bf16 pairs, high part and remainder, so they keep 16 mantissa bits.  A state is kept as it leaves the
+// accumulators: per block of 16 value rows x 16 state rows 32 lanes x 16 bytes of high parts, then of remainders.  An accumulator
+// tile of the transposed state has the layout of the B operand that the outputs need, so a lane writes and reads its own 16 bytes.
 #define STK_PDL_CLASS 16
 #include "chunk_mma.cuh"
 #include "linear_scan.cuh"
@@ -29,9 +31,10 @@ struct ChunkArgs {
   int T;
 };
 
-// A chunk's state before its first token: [D][Vp] high parts, then [D][Vp] remainders; Vp = V rounded up to 8.
+__host__ __device__ inline int blocks16(int n) { return (n + 15) / 16; }
+constexpr int kBlockFloats = 256;                // a 16 x 16 block as a bf16 pair
 __host__ __device__ inline long long linear_slot_floats(int D, int V) {
-  return (static_cast<long long>(D) * ((V + 7) / 8 * 8) + 3) / 4 * 4;
+  return static_cast<long long>(blocks16(D)) * blocks16(V) * kBlockFloats;
 }
 
 // Tokens 2 * lane and 2 * lane + 1 of a chunk of n: running sums of the log decays (F) and input weights (w, 0 behind the chunk).
@@ -72,17 +75,14 @@ __device__ __forceinline__ ChunkGates chunk_gates(const ChunkArgs& a, const Chun
   return c;
 }
 
+constexpr int kLsStages = 3;
+
 template <bool kPair>
 __global__ void __launch_bounds__(128)
 linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  __shared__ float s_w[kChunk];
-  __shared__ float s_fs;
-  constexpr int kTile = kChunk * kStStride, kParts = kPair ? 2 : 1;
-  bf16* kt = reinterpret_cast<bf16*>(smem_raw);                         // [2 stages][parts][64 tokens][72]
-  bf16* vt = kt + 2 * kParts * kTile;                                   // [2 stages][64][72]
-  bf16* wh = vt + 2 * kTile;                                            // weighted keys, high part
-  bf16* wl = wh + kTile;                                                // remainder
+  constexpr int kTile = kChunk * kStStride, kParts = kPair ? 2 : 1, kStage = (kParts + 1) * kTile;
+  bf16* tiles = reinterpret_cast<bf16*>(smem_raw);                      // [stages]{values, keys (, their remainders)}[64 tokens][72]
   pdl_wait();
   pdl_trigger();
   const ScanArgs& s = a.s;
@@ -93,8 +93,8 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
   const long long row = s.req_rows[ri];
   const bool fresh = s.start_pos[ri] == 0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int d0 = db * 64 + warp * 16 + (lane >> 2), c0 = vb * 64 + (lane & 3) * 2;
-  const int Vp = (s.V + 7) / 8 * 8;
+  const int v0 = vb * 64 + warp * 16 + (lane >> 2), d0 = db * 64 + (lane & 3) * 2;     // accumulator rows v0 (+ 8), columns d0 + 8 j (+ 1)
+  const int nd = blocks16(s.D);
   const long long slot_f = linear_slot_floats(s.D, s.V);
   float* gS = s.S + (row * s.H + h) * static_cast<long long>(s.D) * s.V;
   const int kn = max(0, min(64, a.width - db * 64)), vn = min(64, s.V - vb * 64);
@@ -103,120 +103,120 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
   for (int j = 0; j < 8; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const int d = d0 + (i >> 1) * 8, c = c0 + j * 8 + (i & 1);
-      acc[j][i] = !fresh && d < s.D && c < s.V ? gS[static_cast<long long>(d) * s.V + c] : 0.f;
+      const int v = v0 + (i >> 1) * 8, d = d0 + j * 8 + (i & 1);
+      acc[j][i] = !fresh && d < s.D && v < s.V ? gS[static_cast<long long>(d) * s.V + v] : 0.f;
     }
   const int kc = h / a.hpg * a.step + db * 64;
   auto load = [&](int c) {
-    const int n = min(kChunk, span - c * kChunk), st = c & 1;
+    const int n = min(kChunk, span - c * kChunk);
     const long long t0 = q0 + c * kChunk;
-    load_rows_async(kt + st * kParts * kTile, kStStride, 64, a.kh + t0 * a.ldqk + kc, a.ldqk, n, kn, 128);
-    if (kPair) load_rows_async(kt + (st * kParts + 1) * kTile, kStStride, 64, a.kl + t0 * a.ldqk + kc, a.ldqk, n, kn, 128);
-    load_rows_async(vt + st * kTile, kStStride, 64, a.v + t0 * a.ldv + a.v_off + h * s.V + vb * 64, a.ldv, n, vn, 128);
+    bf16* to = tiles + c % kLsStages * kStage;
+    load_rows_async(to, kStStride, 64, a.v + t0 * a.ldv + a.v_off + h * s.V + vb * 64, a.ldv, n, vn, 128);
+    load_rows_async(to + kTile, kStStride, 64, a.kh + t0 * a.ldqk + kc, a.ldqk, n, kn, 128);
+    if (kPair) load_rows_async(to + 2 * kTile, kStStride, 64, a.kl + t0 * a.ldqk + kc, a.ldqk, n, kn, 128);
   };
-  ChunkRaw raw = {};
   load(0);
   mls_commit();
-  if (warp == 0) raw = load_gates(a, h, q0, min(kChunk, span), lane);
+  if (nc > 1) load(1);
+  mls_commit();
+  ChunkRaw raw = load_gates(a, h, q0, min(kChunk, span), lane);
+  const bool block_ok = vb * 64 + warp * 16 < s.V;                      // warp-uniform: its 16 rows exist
   for (int c = 0; c < nc; ++c) {
     const int n = min(kChunk, span - c * kChunk);
-    if (warp == 0) {
-      const ChunkGates g = chunk_gates(a, raw, n, lane);
-      s_w[2 * lane] = 2 * lane < n ? g.w0 * expf(g.end - g.F0) : 0.f;
-      s_w[2 * lane + 1] = 2 * lane + 1 < n ? g.w1 * expf(g.end - g.F1) : 0.f;
-      if (lane == 0) s_fs = expf(g.end);
-    }
-    if (c + 1 < nc) load(c + 1);
-    mls_commit();
+    const ChunkGates g = chunk_gates(a, raw, n, lane);
+    const float w0 = g.w0 * expf(g.end - g.F0), w1 = g.w1 * expf(g.end - g.F1), fs = expf(g.end);   // of tokens 2 lane, 2 lane + 1
     mls_wait<1>();
-    __syncthreads();
-    if (warp == 0 && c + 1 < nc) raw = load_gates(a, h, q0 + (c + 1) * kChunk, min(kChunk, span - (c + 1) * kChunk), lane);
+    __syncthreads();                                                    // chunk c is in, the stage before it is free
+    if (c + 2 < nc) load(c + 2);
+    mls_commit();
+    if (c + 1 < nc) raw = load_gates(a, h, q0 + (c + 1) * kChunk, min(kChunk, span - (c + 1) * kChunk), lane);
     // the state before this chunk
-    {
-      bf16* sh = reinterpret_cast<bf16*>(states + (static_cast<long long>(first + c) * s.H + h) * slot_f);
-      bf16* sl = sh + static_cast<long long>(s.D) * Vp;
+    if (block_ok) {
+      float* slot = states + (static_cast<long long>(first + c) * s.H + h) * slot_f +
+                    (static_cast<long long>(vb * 4 + warp) * nd + db * 4) * kBlockFloats;
 #pragma unroll
-      for (int j = 0; j < 8; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int d = d0 + r * 8, col = c0 + j * 8;
-          if (d < s.D && col < Vp) {
-            uint32_t hi, lo;
-            mls_split2(acc[j][2 * r], acc[j][2 * r + 1], hi, lo);
-            *reinterpret_cast<uint32_t*>(sh + static_cast<long long>(d) * Vp + col) = hi;
-            *reinterpret_cast<uint32_t*>(sl + static_cast<long long>(d) * Vp + col) = lo;
-          }
+      for (int p = 0; p < 4; ++p) {
+        if (db * 4 + p < nd) {
+          uint4 hi, lo;
+          mls_split2(acc[2 * p][0], acc[2 * p][1], hi.x, lo.x);
+          mls_split2(acc[2 * p + 1][0], acc[2 * p + 1][1], hi.y, lo.y);
+          mls_split2(acc[2 * p][2], acc[2 * p][3], hi.z, lo.z);
+          mls_split2(acc[2 * p + 1][2], acc[2 * p + 1][3], hi.w, lo.w);
+          uint4* to = reinterpret_cast<uint4*>(slot + p * kBlockFloats);
+          to[lane] = hi;
+          to[32 + lane] = lo;
         }
-    }
-    const bf16* k = kt + (c & 1) * kParts * kTile;
-    const bf16* v = vt + (c & 1) * kTile;
-    for (int e = threadIdx.x; e < kChunk * 32; e += 128) {
-      const int r = e >> 5, cc = (e & 31) * 2;
-      float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + r * kStStride + cc));
-      if (kPair) {
-        const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + kTile + r * kStStride + cc));
-        x.x += y.x;
-        x.y += y.y;
       }
-      const float w = s_w[r];
-      uint32_t hi, lo;
-      mls_split2(x.x * w, x.y * w, hi, lo);
-      *reinterpret_cast<uint32_t*>(wh + r * kStStride + cc) = hi;
-      *reinterpret_cast<uint32_t*>(wl + r * kStStride + cc) = lo;
     }
-    const float fs = s_fs;
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[j][i] *= fs;
-    __syncthreads();
+    const bf16* v = tiles + c % kLsStages * kStage;
+    const bf16* k = v + kTile;
 #pragma unroll
     for (int kk = 0; kk < kChunk / 16; ++kk) {
-      uint32_t ah[4], al[4];
-      const int ao = (kk * 16 + (lane & 7) + (lane >> 4) * 8) * kStStride + warp * 16 + ((lane >> 3) & 1) * 8;
-      mls_ldsm4_t(ah, wh + ao);
-      mls_ldsm4_t(al, wl + ao);
+      uint32_t af[4], ah[4], al[4];
+      mls_ldsm4_t(af, v + (kk * 16 + (lane & 7) + (lane >> 4) * 8) * kStStride + warp * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {                                     // the operand's token pairs: 2 (lane & 3) and 8 further
+        const int from = kk * 8 + i * 4 + (lane & 3);
+        const float x0 = __shfl_sync(0xffffffffu, w0, from), x1 = __shfl_sync(0xffffffffu, w1, from);
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&af[2 * i + r]));
+          mls_split2(f.x * x0, f.y * x1, ah[2 * i + r], al[2 * i + r]);
+        }
+      }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         uint32_t b[4];
-        mls_ldsm4_t(b, v + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kStStride + j * 16 + (lane >> 4) * 8);
+        const int off = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kStStride + j * 16 + (lane >> 4) * 8;
+        mls_ldsm4_t(b, k + off);
         mls_mma(acc[2 * j], ah, b[0], b[1]);
         mls_mma(acc[2 * j + 1], ah, b[2], b[3]);
         mls_mma(acc[2 * j], al, b[0], b[1]);
         mls_mma(acc[2 * j + 1], al, b[2], b[3]);
+        if (kPair) {
+          uint32_t bl[4];
+          mls_ldsm4_t(bl, k + kTile + off);
+          mls_mma(acc[2 * j], ah, bl[0], bl[1]);
+          mls_mma(acc[2 * j + 1], ah, bl[2], bl[3]);
+        }
       }
     }
-    __syncthreads();
   }
   mls_wait<0>();
 #pragma unroll
   for (int j = 0; j < 8; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const int d = d0 + (i >> 1) * 8, c = c0 + j * 8 + (i & 1);
-      if (d < s.D && c < s.V) gS[static_cast<long long>(d) * s.V + c] = acc[j][i];
+      const int v = v0 + (i >> 1) * 8, d = d0 + j * 8 + (i & 1);
+      if (d < s.D && v < s.V) gS[static_cast<long long>(d) * s.V + v] = acc[j][i];
     }
 }
 
-constexpr int kLoRows = 32;                      // state rows per stage
+// Row and column of the b-th 16 x 16 block on or below the diagonal.
+__device__ __forceinline__ void low_block(int b, int& rb, int& kb) {
+  rb = b < 1 ? 0 : b < 3 ? 1 : b < 6 ? 2 : 3;
+  kb = b - rb * (rb + 1) / 2;
+}
 
-// Eight warps: four blocks of 16 tokens x two halves of the columns (of the keys while the scores are formed).
 template <bool kPair, int COLS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(COLS * 2)
 linear_chunk_out_kernel(const ChunkArgs a, int min_span, const float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ float s_F[kChunk], s_w[kChunk], s_in[kChunk];
   __shared__ ChunkRef s_c;
   __shared__ int s_ok;
-  constexpr int kVs = COLS + 8, kHalf = COLS / 2, kParts = kPair ? 2 : 1;
+  constexpr int kVs = COLS + 8, kParts = kPair ? 2 : 1, kThreads = COLS * 2, kWarps = COLS / 16, kMine = (10 + kWarps - 1) / kWarps;
   const ScanArgs& s = a.s;
-  const int Dp = (s.D + 15) / 16 * 16, ks = Dp + 8;
+  const int Dp = blocks16(s.D) * 16, ks = Dp + 8;
   bf16* q = reinterpret_cast<bf16*>(smem_raw);                          // [parts][64][Dp + 8]
   bf16* v = q + kParts * kChunk * ks;                                   // [64][COLS + 8]
-  bf16* ph = v + kChunk * kVs;                                          // [64][72] weighted scores, high part
-  bf16* pl = ph + kChunk * kStStride;                                   // remainder
-  bf16* k = pl + kChunk * kStStride;                                    // [parts][64][Dp + 8], then two stages of state rows:
-  bf16* st = k;                                                         // {high, remainder} x [32][COLS + 8]
+  bf16* k = v + kChunk * kVs;                                           // [parts][64][Dp + 8], then the weighted scores:
+  bf16* ph = k;                                                         // [64][72] high parts
+  bf16* pl = ph + kChunk * kStStride;                                   // remainders
   pdl_wait();
   pdl_trigger();
   const int vb = blockIdx.x, ci = blockIdx.y, h = blockIdx.z;
@@ -224,22 +224,34 @@ linear_chunk_out_kernel(const ChunkArgs a, int min_span, const float* __restrict
   __syncthreads();
   if (!s_ok) return;
   const ChunkRef c = s_c;
-  const int Vp = (s.V + 7) / 8 * 8, qc = h / a.hpg * a.step, vn = min(COLS, s.V - vb * COLS);
-  const bf16* Sh = reinterpret_cast<const bf16*>(states + (static_cast<long long>(ci) * s.H + h) * linear_slot_floats(s.D, s.V));
-  const bf16* Sl = Sh + static_cast<long long>(s.D) * Vp;
-  // a request's very first chunk starts from zeros: nothing comes from the state
-  const bool has_state = !(s.start_pos[c.ri] == 0 && c.first == ci);
-  const long long at = c.t0 * a.ldqk + qc;
-  load_rows_async(q, ks, Dp, a.qh + at, a.ldqk, c.n, a.width, 256);
-  load_rows_async(k, ks, Dp, a.kh + at, a.ldqk, c.n, a.width, 256);
-  if (kPair) {
-    load_rows_async(q + kChunk * ks, ks, Dp, a.ql + at, a.ldqk, c.n, a.width, 256);
-    load_rows_async(k + kChunk * ks, ks, Dp, a.kl + at, a.ldqk, c.n, a.width, 256);
-  }
-  load_rows_async(v, kVs, COLS, a.v + c.t0 * a.ldv + a.v_off + h * s.V + vb * COLS, a.ldv, c.n, vn, 256);
-  mls_commit();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int rb = warp & 3, half = warp >> 2;
+  const int qc = h / a.hpg * a.step, vn = min(COLS, s.V - vb * COLS);
+  // a request's very first chunk starts from zeros: nothing comes from the state
+  const bool mine = vb * COLS + warp * 16 < s.V;                        // warp-uniform: its 16 columns exist
+  const bool has_state = mine && !(s.start_pos[c.ri] == 0 && c.first == ci);
+  const long long at = c.t0 * a.ldqk + qc;
+  load_rows_async(q, ks, Dp, a.qh + at, a.ldqk, c.n, a.width, kThreads);
+  load_rows_async(k, ks, Dp, a.kh + at, a.ldqk, c.n, a.width, kThreads);
+  if (kPair) {
+    load_rows_async(q + kChunk * ks, ks, Dp, a.ql + at, a.ldqk, c.n, a.width, kThreads);
+    load_rows_async(k + kChunk * ks, ks, Dp, a.kl + at, a.ldqk, c.n, a.width, kThreads);
+  }
+  load_rows_async(v, kVs, COLS, a.v + c.t0 * a.ldv + a.v_off + h * s.V + vb * COLS, a.ldv, c.n, vn, kThreads);
+  mls_commit();
+  // this warp's state blocks, a few ahead of the products
+  const int nd = Dp / 16;
+  constexpr int kAhead = 4;
+  const uint4* S = reinterpret_cast<const uint4*>(states + (static_cast<long long>(ci) * s.H + h) * linear_slot_floats(s.D, s.V) +
+                                                  static_cast<long long>(vb * kWarps + warp) * nd * kBlockFloats) + lane;
+  uint4 sh[kAhead], sl[kAhead];
+  if (has_state) {
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+      if (i < nd) {
+        sh[i] = __ldcs(S + i * 64);
+        sl[i] = __ldcs(S + i * 64 + 32);
+      }
+  }
   if (warp == 0) {
     const ChunkGates g = chunk_gates(a, load_gates(a, h, c.t0, c.n, lane), c.n, lane);
     s_F[2 * lane] = g.F0;
@@ -251,164 +263,166 @@ linear_chunk_out_kernel(const ChunkArgs a, int min_span, const float* __restrict
   }
   mls_wait<0>();
   __syncthreads();
-  int row[2];
+  // weighted scores: the ten blocks on or below the diagonal, in turns over the warps
+  uint32_t wh[kMine][4], wl[kMine][4];
 #pragma unroll
-  for (int r = 0; r < 2; ++r) row[r] = rb * 16 + (lane >> 2) + r * 8;
-  // weighted scores of this warp's tokens against every other block of 16 keys
-  {
-    const float F[2] = {s_F[row[0]], s_F[row[1]]};
-    for (int kb = half; kb <= rb; kb += 2) {
-      float x[2][4];
+  for (int m = 0; m < kMine; ++m) {
+    const int b = warp + m * kWarps;
+    if (b >= 10) continue;
+    int rb, kb;
+    low_block(b, rb, kb);
+    float x[2][4];
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) x[j][i] = 0.f;
-      const int qo = (rb * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
-      const int ko = (kb * 16 + (lane >> 4) * 8 + (lane & 7)) * ks + ((lane >> 3) & 1) * 8;
-      for (int kk = 0; kk < Dp / 16; ++kk) {
-        uint32_t af[4], bf[4];
-        mls_ldsm4(af, q + qo + kk * 16);
-        mls_ldsm4(bf, k + ko + kk * 16);
-        mls_mma(x[0], af, bf[0], bf[1]);
-        mls_mma(x[1], af, bf[2], bf[3]);
-        if (kPair) {
-          uint32_t al[4], bl[4];
-          mls_ldsm4(al, q + kChunk * ks + qo + kk * 16);
-          mls_ldsm4(bl, k + kChunk * ks + ko + kk * 16);
-          mls_mma(x[0], al, bf[0], bf[1]);
-          mls_mma(x[1], al, bf[2], bf[3]);
-          mls_mma(x[0], af, bl[0], bl[1]);
-          mls_mma(x[1], af, bl[2], bl[3]);
-        }
+      for (int i = 0; i < 4; ++i) x[j][i] = 0.f;
+    const int qo = (rb * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
+    const int ko = (kb * 16 + (lane >> 4) * 8 + (lane & 7)) * ks + ((lane >> 3) & 1) * 8;
+    for (int kk = 0; kk < nd; ++kk) {
+      uint32_t af[4], bf[4];
+      mls_ldsm4(af, q + qo + kk * 16);
+      mls_ldsm4(bf, k + ko + kk * 16);
+      mls_mma(x[0], af, bf[0], bf[1]);
+      mls_mma(x[1], af, bf[2], bf[3]);
+      if (kPair) {
+        uint32_t al[4], bl[4];
+        mls_ldsm4(al, q + kChunk * ks + qo + kk * 16);
+        mls_ldsm4(bl, k + kChunk * ks + ko + kk * 16);
+        mls_mma(x[0], al, bf[0], bf[1]);
+        mls_mma(x[1], al, bf[2], bf[3]);
+        mls_mma(x[0], af, bl[0], bl[1]);
+        mls_mma(x[1], af, bl[2], bl[3]);
       }
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int col = kb * 16 + j * 8 + (lane & 3) * 2;
-          float p[2];
-#pragma unroll
-          for (int i = 0; i < 2; ++i)
-            p[i] = col + i <= row[r] ? x[j][2 * r + i] * (s_w[col + i] * expf(F[r] - s_F[col + i])) : 0.f;
-          uint32_t hi, lo;
-          mls_split2(p[0], p[1], hi, lo);
-          *reinterpret_cast<uint32_t*>(ph + row[r] * kStStride + col) = hi;
-          *reinterpret_cast<uint32_t*>(pl + row[r] * kStStride + col) = lo;
-        }
     }
-  }
-  __syncthreads();                                                       // k is free, the weighted scores are complete
-  float o[COLS / 16][4];
 #pragma unroll
-  for (int j = 0; j < COLS / 16; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
-  if (has_state) {
-    const int slices = (Dp + kLoRows - 1) / kLoRows;
-    constexpr int kCh = COLS / 8;
-    auto load_slice = [&](int sl) {
-      bf16* dst = st + (sl & 1) * 2 * kLoRows * kVs;
-      for (int e = threadIdx.x; e < 2 * kLoRows * kCh; e += 256) {
-        const int part = e / (kLoRows * kCh), r = e / kCh % kLoRows, cc = e % kCh * 8;
-        const int d = sl * kLoRows + r, col = vb * COLS + cc;
-        const bool ok = d < s.D && col < Vp;
-        const bf16* src = (part ? Sl : Sh) + (ok ? static_cast<long long>(d) * Vp + col : 0);
-        mls_cp16(dst + (part * kLoRows + r) * kVs + cc, src, ok);
+      for (int r = 0; r < 2; ++r) {
+        const int t = rb * 16 + (lane >> 2) + r * 8, col = kb * 16 + j * 8 + (lane & 3) * 2;
+        float p[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) p[i] = col + i <= t ? x[j][2 * r + i] * (s_w[col + i] * expf(s_F[t] - s_F[col + i])) : 0.f;
+        mls_split2(p[0], p[1], wh[m][2 * j + r], wl[m][2 * j + r]);
       }
-    };
-    load_slice(0);
-    mls_commit();
-    for (int sl = 0; sl < slices; ++sl) {
-      if (sl + 1 < slices) load_slice(sl + 1);
-      mls_commit();
-      mls_wait<1>();
-      __syncthreads();
-      const bf16* hi = st + (sl & 1) * 2 * kLoRows * kVs;
-      const bf16* lo = hi + kLoRows * kVs;
+  }
+  __syncthreads();                                                       // the keys are done with
 #pragma unroll
-      for (int kk = 0; kk < kLoRows / 16; ++kk) {
-        if (sl * kLoRows + kk * 16 < Dp) {
-          uint32_t af[4], al[4];
-          const int qo = (rb * 16 + (lane & 15)) * ks + sl * kLoRows + kk * 16 + (lane >> 4) * 8;
-          mls_ldsm4(af, q + qo);
-          if (kPair) mls_ldsm4(al, q + kChunk * ks + qo);
+  for (int m = 0; m < kMine; ++m) {
+    const int b = warp + m * kWarps;
+    if (b >= 10) continue;
+    int rb, kb;
+    low_block(b, rb, kb);
 #pragma unroll
-          for (int j = 0; j < COLS / 32; ++j) {
-            uint32_t bh[4], bl[4];
-            const int off = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kVs + half * kHalf + j * 16 + (lane >> 4) * 8;
-            mls_ldsm4_t(bh, hi + off);
-            mls_ldsm4_t(bl, lo + off);
-            mls_mma(o[2 * j], af, bh[0], bh[1]);
-            mls_mma(o[2 * j + 1], af, bh[2], bh[3]);
-            mls_mma(o[2 * j], af, bl[0], bl[1]);
-            mls_mma(o[2 * j + 1], af, bl[2], bl[3]);
-            if (kPair) {
-              mls_mma(o[2 * j], al, bh[0], bh[1]);
-              mls_mma(o[2 * j + 1], al, bh[2], bh[3]);
-            }
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int off = (rb * 16 + (lane >> 2) + r * 8) * kStStride + kb * 16 + j * 8 + (lane & 3) * 2;
+        *reinterpret_cast<uint32_t*>(ph + off) = wh[m][2 * j + r];
+        *reinterpret_cast<uint32_t*>(pl + off) = wl[m][2 * j + r];
+      }
+  }
+  float o[4][2][4];
+#pragma unroll
+  for (int rb = 0; rb < 4; ++rb)
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) o[rb][j][i] = 0.f;
+  if (has_state) {
+    const bf16* qa = q + (lane & 15) * ks + (lane >> 4) * 8;
+    for (int k0 = 0; k0 < nd; k0 += kAhead) {
+#pragma unroll
+      for (int i = 0; i < kAhead; ++i) {
+        const int kk = k0 + i;
+        if (kk >= nd) continue;
+        const uint4 hi = sh[i], lo = sl[i];
+        if (kk + kAhead < nd) {
+          sh[i] = __ldcs(S + (kk + kAhead) * 64);
+          sl[i] = __ldcs(S + (kk + kAhead) * 64 + 32);
+        }
+#pragma unroll
+        for (int rb = 0; rb < 4; ++rb) {
+          uint32_t af[4];
+          mls_ldsm4(af, qa + rb * 16 * ks + kk * 16);
+          mls_mma(o[rb][0], af, hi.x, hi.y);
+          mls_mma(o[rb][1], af, hi.z, hi.w);
+          mls_mma(o[rb][0], af, lo.x, lo.y);
+          mls_mma(o[rb][1], af, lo.z, lo.w);
+          if (kPair) {
+            uint32_t al[4];
+            mls_ldsm4(al, qa + (kChunk + rb * 16) * ks + kk * 16);
+            mls_mma(o[rb][0], al, hi.x, hi.y);
+            mls_mma(o[rb][1], al, hi.z, hi.w);
           }
         }
       }
-      __syncthreads();
     }
-    mls_wait<0>();
 #pragma unroll
-    for (int j = 0; j < COLS / 16; ++j)
+    for (int rb = 0; rb < 4; ++rb)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) o[j][i] *= s_in[row[i >> 1]];
+      for (int i = 0; i < 4; ++i) {
+        const float f = s_in[rb * 16 + (lane >> 2) + (i >> 1) * 8];
+        o[rb][0][i] *= f;
+        o[rb][1][i] *= f;
+      }
   }
-  for (int kb = 0; kb <= rb; ++kb) {
-    uint32_t hi[4], lo[4];
-    const int off = (rb * 16 + (lane & 15)) * kStStride + kb * 16 + (lane >> 4) * 8;
-    mls_ldsm4(hi, ph + off);
-    mls_ldsm4(lo, pl + off);
+  __syncthreads();                                                       // the weighted scores are complete
+  if (!mine) return;
 #pragma unroll
-    for (int j = 0; j < COLS / 32; ++j) {
-      uint32_t bf[4];
-      mls_ldsm4_t(bf, v + (kb * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kVs + half * kHalf + j * 16 + (lane >> 4) * 8);
-      mls_mma(o[2 * j], hi, bf[0], bf[1]);
-      mls_mma(o[2 * j + 1], hi, bf[2], bf[3]);
-      mls_mma(o[2 * j], lo, bf[0], bf[1]);
-      mls_mma(o[2 * j + 1], lo, bf[2], bf[3]);
+  for (int kb = 0; kb < 4; ++kb) {
+    uint32_t b[4];
+    mls_ldsm4_t(b, v + (kb * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kVs + warp * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int rb = kb; rb < 4; ++rb) {
+      uint32_t hi[4], lo[4];
+      const int off = (rb * 16 + (lane & 15)) * kStStride + kb * 16 + (lane >> 4) * 8;
+      mls_ldsm4(hi, ph + off);
+      mls_ldsm4(lo, pl + off);
+      mls_mma(o[rb][0], hi, b[0], b[1]);
+      mls_mma(o[rb][1], hi, b[2], b[3]);
+      mls_mma(o[rb][0], lo, b[0], b[1]);
+      mls_mma(o[rb][1], lo, b[2], b[3]);
     }
   }
   const float skip = a.skip != nullptr ? a.skip[h] : 0.f;
+  const bool pair = (s.V & 1) == 0;
 #pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    if (row[r] >= c.n) continue;
-    const long long t = c.t0 + row[r];
-    const int lc = half * kHalf + (lane & 3) * 2, c0 = vb * COLS + lc;
-    float* out = s.o + (t * s.H + h) * s.V + c0;
-    const bool pair = (s.V & 1) == 0;
+  for (int rb = 0; rb < 4; ++rb)
 #pragma unroll
-    for (int j = 0; j < COLS / 16; ++j) {
-      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v + row[r] * kVs + lc + j * 8));
-      const float y0 = fmaf(skip, x.x, o[j][2 * r]), y1 = fmaf(skip, x.y, o[j][2 * r + 1]);
-      if (pair && c0 + j * 8 + 1 < s.V) {
-        *reinterpret_cast<float2*>(out + j * 8) = make_float2(y0, y1);
-      } else {
-        if (c0 + j * 8 < s.V) out[j * 8] = y0;
-        if (c0 + j * 8 + 1 < s.V) out[j * 8 + 1] = y1;
+    for (int r = 0; r < 2; ++r) {
+      const int t = rb * 16 + (lane >> 2) + r * 8;
+      if (t >= c.n) continue;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int lc = warp * 16 + j * 8 + (lane & 3) * 2, col = vb * COLS + lc;
+        const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v + t * kVs + lc));
+        const float y0 = fmaf(skip, x.x, o[rb][j][2 * r]), y1 = fmaf(skip, x.y, o[rb][j][2 * r + 1]);
+        float* out = s.o + ((c.t0 + t) * static_cast<long long>(s.H) + h) * s.V + col;
+        if (pair && col + 1 < s.V) {
+          *reinterpret_cast<float2*>(out) = make_float2(y0, y1);
+        } else {
+          if (col < s.V) out[0] = y0;
+          if (col + 1 < s.V) out[1] = y1;
+        }
       }
     }
-  }
 }
 
 template <bool kPair, int COLS>
 static int launch_chunks(const ChunkArgs& a, int min_span, float* states, int max_chunks, cudaStream_t st) {
   constexpr int kParts = kPair ? 2 : 1, kVs = COLS + 8;
   const ScanArgs& s = a.s;
-  const int ks = (s.D + 15) / 16 * 16 + 8;
-  const size_t smem_s = static_cast<size_t>(2 * kParts + 2 + 2) * kChunk * kStStride * 2;
-  const size_t keys = static_cast<size_t>(kParts) * kChunk * ks, rows = static_cast<size_t>(4) * kLoRows * kVs;
-  const size_t smem_o = (keys + static_cast<size_t>(kChunk) * (kVs + 2 * kStStride) + (keys > rows ? keys : rows)) * 2;
+  const int ks = blocks16(s.D) * 16 + 8;
+  const size_t smem_s = static_cast<size_t>(kLsStages) * (kParts + 1) * kChunk * kStStride * 2;
+  const size_t keys = static_cast<size_t>(kParts) * kChunk * ks, scores = static_cast<size_t>(2) * kChunk * kStStride;
+  const size_t smem_o = (keys + static_cast<size_t>(kChunk) * kVs + (keys > scores ? keys : scores)) * 2;
   if (smem_o > 220 * 1024) return -5;
-  if (cudaFuncSetAttribute(linear_chunk_state_kernel<kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, 80 * 1024) != cudaSuccess ||
+  if (cudaFuncSetAttribute(linear_chunk_state_kernel<kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, 84 * 1024) != cudaSuccess ||
       cudaFuncSetAttribute(linear_chunk_out_kernel<kPair, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess)
     return -3;
   launch_pdl(linear_chunk_state_kernel<kPair>, dim3((s.V + 63) / 64, (s.D + 63) / 64, s.H * s.n_req), dim3(128), smem_s, st, a, min_span,
              states);
-  launch_pdl(linear_chunk_out_kernel<kPair, COLS>, dim3((s.V + COLS - 1) / COLS, max_chunks, s.H), dim3(256), smem_o, st, a, min_span,
+  launch_pdl(linear_chunk_out_kernel<kPair, COLS>, dim3((s.V + COLS - 1) / COLS, max_chunks, s.H), dim3(COLS * 2), smem_o, st, a, min_span,
              states);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

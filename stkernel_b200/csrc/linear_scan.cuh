@@ -5,8 +5,8 @@
 // shared by retention (retention.cu) and Mamba-2 (mamba2.cu).  A span that starts at position 0 starts from a zero state.
 //
 //   linear_scan_kernel     token by token, any size and type: one CTA per (32 or 64 value columns, head, request), the block of the
-//                          state in registers.  A `Front` supplies a token's q and k (in shared memory), v and decay: rotation,
-//                          convolution and step sizes happen on the way in.
+//                          state in registers.  A `Front` supplies a token's q and k (in shared memory), v and decay, so that
+//                          rotations and input weights happen on the way in.
 //   linear_chunk_*         spans of some length, bf16 operands (linear_scan.cu)
 #pragma once
 #include "hybrid_block.cuh"
@@ -21,11 +21,11 @@ struct ScanArgs {
 
 constexpr int kScanThreads = 256, kScanRows = 8;
 
-// Front: static constexpr bool kValues (v comes through shared memory);
-//   float2 fill(t, i, pos, row, h, col0, cols, q, k, x)  token t = the i-th of its span; all threads; returns the decay and what its
-//                                                        rounding left over (a fixed decay's error would add up over the tokens)
-//   float value(t, h, col)                               v when !kValues
-//   float skip(h)                                        factor of v in the output
+// Front:
+//   float2 fill(t, pos, h, q, k)   token t at position pos, all threads; returns the decay and what its rounding left over (the same
+//                                  small error at every token would add up over many)
+//   float value(t, h, col)         v
+//   float skip(h)                  factor of v in the output
 template <typename Front, int NR, int VEC>
 __global__ void __launch_bounds__(kScanThreads)
 linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) {
@@ -33,7 +33,7 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
   constexpr int kCols = 32 * VEC;
   float* q = sm;                                  // [D]
   float* k = q + a.D;                             // [D]
-  float* x = k + a.D;                             // [kCols]
+  float* x = k + a.D;                             // [kCols] v
   float* part = x + kCols;                        // [8][kCols]
   pdl_wait();
   pdl_trigger();
@@ -63,17 +63,14 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
   for (int i = 0; i < span; ++i) {
     const long long t = q0 + i;
     __syncthreads();
-    const float2 decay = f.fill(t, i, start + i, row, h, vb * kCols, min(kCols, a.V - vb * kCols), q, k, x);
+    const float2 decay = f.fill(t, start + i, h, q, k);
     float v[VEC];
-    if (!Front::kValues) {
 #pragma unroll
-      for (int c = 0; c < VEC; ++c) v[c] = col + c < a.V ? f.value(t, h, col + c) : 0.f;
+    for (int c = 0; c < VEC; ++c) {
+      v[c] = col + c < a.V ? f.value(t, h, col + c) : 0.f;
+      if (r == 0) x[lane * VEC + c] = v[c];
     }
     __syncthreads();
-    if (Front::kValues) {
-#pragma unroll
-      for (int c = 0; c < VEC; ++c) v[c] = col + c < a.V ? x[lane * VEC + c] : 0.f;
-    }
     float acc[VEC];
 #pragma unroll
     for (int c = 0; c < VEC; ++c) acc[c] = 0.f;
@@ -97,8 +94,7 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
       float s = 0.f;
 #pragma unroll
       for (int w = 0; w < kScanRows; ++w) s += part[w * kCols + oc];
-      if (Front::kValues) s = fmaf(skip, x[oc], s);
-      a.o[(t * a.H + h) * a.V + vb * kCols + oc] = s;
+      a.o[(t * a.H + h) * a.V + vb * kCols + oc] = fmaf(skip, x[oc], s);
     }
   }
 #pragma unroll

@@ -1,8 +1,8 @@
 // Mamba-2: a linear recurrence (linear_scan.cuh) with k = dt B, q = C, v = x and log decay -exp(A) dt, whose operands x, B and C come
 // through a short causal convolution per channel and silu.
 //
-//   mamba2_scan        decode rows, short spans, float32: convolution and step size on the way into the recurrence
-//   mamba2_conv        long spans: convolved operands in bf16, step sizes and log decays for the chunked form
+//   mamba2_conv        convolved operands in the compute type, step sizes and log decays
+//   mamba2_scan        decode rows, short spans, float32 (long spans: linear_scan.cu)
 //   mamba2_finish      gate silu(z), RMS norm in equal parts, and the last convolution inputs of every span into its request's ring
 //
 // Convolution inputs before a span come from ring [rows][taps - 1][channels] (position p at p mod (taps - 1)), those before
@@ -23,62 +23,47 @@ struct ConvArgs {
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
-// Channel ch of token t, the i-th of its span, at position pos.
-template <typename A>
-__device__ __forceinline__ float conv_at(const ConvArgs& a, long long t, int i, long long pos, long long row, int ch) {
-  const A* x = reinterpret_cast<const A*>(a.proj) + t * a.ldp + a.x_off + ch;
-  const int keep = a.n - 1;
-  float s = a.bias[ch];
-  for (int j = 0; j < a.n; ++j) {
-    float in = 0.f;
-    if (j <= i) in = ld_act(x - j * a.ldp);
-    else if (pos >= j) in = ld_act(reinterpret_cast<const A*>(a.ring) + (row * keep + (pos - j) % keep) * a.channels + ch);
-    s = fmaf(a.taps[(a.n - 1 - j) * a.channels + ch], in, s);
-  }
-  return silu_f(s);
-}
-
 template <typename A>
 struct Mamba2Front {
-  static constexpr bool kValues = true;
-  ConvArgs c;
-  int N, V, inner, groups, hpg;
+  const A* xbc; long long ld;                     // [T, ld]: x | B | C, convolved
+  const float* steps;                             // [2][H][T]: log decays, step sizes
+  int N, V, inner, groups, hpg, H, T;
   const float* skips;
   __device__ __forceinline__ float skip(int h) const { return skips[h]; }
-  __device__ __forceinline__ float value(long long, int, int) const { return 0.f; }
-  __device__ __forceinline__ float2 fill(long long t, int i, long long pos, long long row, int h, int col0, int cols, float* q, float* k,
-                                         float* x) const {
-    const float dt = softplus_f(ld_act(reinterpret_cast<const A*>(c.proj) + t * c.ldp + c.dt_off + h) + c.dt_bias[h]);
-    const int g = h / hpg, b0 = inner + g * N, c0 = inner + (groups + g) * N;
-    for (int e = threadIdx.x; e < 2 * N + cols; e += kScanThreads) {
-      if (e < N) q[e] = conv_at<A>(c, t, i, pos, row, c0 + e);
-      else if (e < 2 * N) k[e - N] = conv_at<A>(c, t, i, pos, row, b0 + e - N) * dt;
-      else x[e - 2 * N] = conv_at<A>(c, t, i, pos, row, h * V + col0 + e - 2 * N);
+  __device__ __forceinline__ float value(long long t, int h, int col) const { return ld_act(xbc + t * ld + h * V + col); }
+  __device__ __forceinline__ float2 fill(long long t, long long, int h, float* q, float* k) const {
+    const long long at = static_cast<long long>(h) * T + t;
+    const float lg = steps[at], dt = steps[static_cast<long long>(H) * T + at];
+    const A* p = xbc + t * ld + inner + h / hpg * N;
+    for (int e = threadIdx.x; e < 2 * N; e += kScanThreads) {
+      if (e < N) k[e] = ld_act(p + e) * dt;
+      else q[e - N] = ld_act(p + groups * N + e - N);
     }
     // slow decays as 1 and the (small) difference from it: a rounded factor close to 1 would be off in the same direction for long
-    const float lg = c.neg_a[h] * dt;
     return lg > -0.25f ? make_float2(1.f, expm1f(lg)) : make_float2(expf(lg), 0.f);
   }
 };
 
 constexpr int kConvTok = 8;
 
-// Eight channels x kConvTok tokens per thread; the inputs slide through registers where the taps are few (NT), otherwise they are
-// read again for every tap.  The grid's last column of blocks forms the step sizes.
-template <int NT>
+// Eight channels x kConvTok tokens per thread.  NT > 0 taps: the inputs of tokens that follow one another in one span are all in
+// flight together and stay in registers; otherwise (spans that meet inside the group, many taps) every tap is read where it is
+// used.  The grid's last column of blocks forms the step sizes.
+template <typename A, int NT>
 __global__ void __launch_bounds__(128)
 mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, const int* __restrict__ tok_req,
-                   const int* __restrict__ first_pos, __nv_bfloat16* __restrict__ out, long long ldo, float* __restrict__ steps, int H,
-                   int T, int vec) {
+                   const int* __restrict__ first_pos, A* __restrict__ out, long long ldo, float* __restrict__ steps, int H, int T,
+                   int vec) {
   pdl_wait();
   pdl_trigger();
-  const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(a.proj);
+  const A* proj = reinterpret_cast<const A*>(a.proj);
+  const int t0 = blockIdx.y * kConvTok, t1 = min(T, t0 + kConvTok);
   if (blockIdx.x == gridDim.x - 1) {
-    // steps [0][H][T]: log decays, [1][H][T]: input weights
+    // steps [0][H][T]: log decays, [1][H][T]: step sizes
     for (int e = threadIdx.x; e < kConvTok * H; e += 128) {
-      const int h = e / kConvTok, t = blockIdx.y * kConvTok + e % kConvTok;
+      const int h = e / kConvTok, t = t0 + e % kConvTok;
       if (t >= T) continue;
-      const float dt = softplus_f(bf16_to_f(proj[t * a.ldp + a.dt_off + h]) + a.dt_bias[h]);
+      const float dt = softplus_f(ld_act(proj + t * a.ldp + a.dt_off + h) + a.dt_bias[h]);
       steps[static_cast<long long>(h) * T + t] = dt * a.neg_a[h];
       steps[(static_cast<long long>(H) + h) * T + t] = dt;
     }
@@ -86,17 +71,13 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
   }
   const int ch = (blockIdx.x * 128 + threadIdx.x) * 8;
   if (ch >= ldo) return;
-  const int nc = min(8, a.channels - ch), t0 = blockIdx.y * kConvTok, keep = a.n - 1;
-  const __nv_bfloat16* ring = reinterpret_cast<const __nv_bfloat16*>(a.ring);
-  // input j tokens before token t: its own span's row, the ring, or zero
-  auto input = [&](int t, int j, float (&f)[8]) {
-    const int first = first_pos[t];
-    const long long pos = positions[t];
-    const __nv_bfloat16* src = nullptr;
-    if (pos - j >= first) src = proj + (t - j) * a.ldp + a.x_off + ch;
-    else if (pos >= j) src = ring + (static_cast<long long>(tok_req[t]) * keep + (pos - j) % keep) * a.channels + ch;
-    if (src != nullptr && vec) {
-      const uint4 v = *reinterpret_cast<const uint4*>(src);
+  const int nc = min(8, a.channels - ch), keep = a.n - 1;
+  const A* x = proj + a.x_off + ch;
+  const A* ring = reinterpret_cast<const A*>(a.ring) + ch;
+  auto fetch = [&](const A* src, float (&f)[8]) {
+    if (sizeof(A) == 2 && vec) {
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (src != nullptr) v = *reinterpret_cast<const uint4*>(src);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const float2 u = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[c]);
@@ -105,63 +86,146 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
       }
     } else {
 #pragma unroll
-      for (int c = 0; c < 8; ++c) f[c] = src != nullptr && c < nc ? bf16_to_f(src[c]) : 0.f;
+      for (int c = 0; c < 8; ++c) f[c] = src != nullptr && c < nc ? ld_act(src + c) : 0.f;
     }
   };
-  float w[NT > 0 ? NT : 1][8], bias[8];
+  // where the input j tokens before token t is: its own span's row, the ring, or nowhere (zero)
+  auto where = [&](int t, int j, int req, long long pos, int first) -> const A* {
+    if (pos - j >= first) return x + (t - j) * a.ldp;
+    if (pos >= j) return ring + (static_cast<long long>(req) * keep + (pos - j) % keep) * a.channels;
+    return nullptr;
+  };
+  auto put = [&](int t, const float (&s)[8]) {
+    if (sizeof(A) == 2) {
+      __align__(16) __nv_bfloat162 b[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const float y = s[2 * c], z = s[2 * c + 1];
+        b[c] = __floats2bfloat162_rn(2 * c < nc ? y / (1.f + __expf(-y)) : 0.f, 2 * c + 1 < nc ? z / (1.f + __expf(-z)) : 0.f);
+      }
+      *reinterpret_cast<uint4*>(out + t * ldo + ch) = *reinterpret_cast<const uint4*>(b);
+    } else {
+#pragma unroll
+      for (int c = 0; c < 8; ++c) st_act(out + t * ldo + ch + c, c < nc ? silu_f(s[c]) : 0.f);
+    }
+  };
+  float bias[8];
 #pragma unroll
   for (int c = 0; c < 8; ++c) bias[c] = c < nc ? a.bias[ch + c] : 0.f;
-  if (NT > 0) {
+  const int req0 = tok_req[t0], first0 = first_pos[t0];
+  const long long pos0 = positions[t0];
+  if (NT > 0 && req0 >= 0 && pos0 >= 0 && tok_req[t1 - 1] == req0 && positions[t1 - 1] == pos0 + (t1 - 1 - t0)) {
+    constexpr int kN = NT > 0 ? NT : 1;
+    float w[kN][8];
 #pragma unroll
-    for (int j = 0; j < (NT > 0 ? NT : 1); ++j)
+    for (int j = 0; j < kN; ++j)
 #pragma unroll
       for (int c = 0; c < 8; ++c) w[j][c] = c < nc ? a.taps[(a.n - 1 - j) * a.channels + ch + c] : 0.f;
+    float in[kConvTok + kN - 1][8];                       // inputs of tokens t0 - (n - 1) .. t0 + 7
+#pragma unroll
+    for (int i = 0; i < kConvTok + kN - 1; ++i) {
+      const int j = kN - 1 - i;                           // tokens before t0
+      fetch(j > 0 ? where(t0, j, req0, pos0, first0) : t0 - j < t1 ? x + (t0 - j) * a.ldp : nullptr, in[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < kConvTok; ++i) {
+      if (t0 + i < t1) {
+        float s[8];
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          s[c] = bias[c];
+#pragma unroll
+          for (int j = 0; j < kN; ++j) s[c] = fmaf(w[j][c], in[i + kN - 1 - j][c], s[c]);
+        }
+        put(t0 + i, s);
+      }
+    }
+    return;
   }
-  float past[NT > 0 ? NT : 1][8];                       // past[j]: input j tokens before the current one
-  int prev_req = -2;
-  long long prev_pos = -2;
-  for (int t = t0; t < min(T, t0 + kConvTok); ++t) {
-    const int req = tok_req[t];
+  for (int t = t0; t < t1; ++t) {
+    const int req = tok_req[t], first = first_pos[t];
     const long long pos = positions[t];
     float s[8];
 #pragma unroll
     for (int c = 0; c < 8; ++c) s[c] = bias[c];
     if (req >= 0 && pos >= 0) {
-      if (NT > 0) {
-        constexpr int kN = NT > 0 ? NT : 1;
-        if (req == prev_req && pos == prev_pos + 1) {
+#pragma unroll 4
+      for (int j = 0; j < a.n; ++j) {
+        float f[8];
+        fetch(where(t, j, req, pos, first), f);
 #pragma unroll
-          for (int j = kN - 1; j > 0; --j)
-#pragma unroll
-            for (int c = 0; c < 8; ++c) past[j][c] = past[j - 1][c];
-        } else {
-#pragma unroll
-          for (int j = 1; j < kN; ++j) input(t, j, past[j]);
-        }
-        input(t, 0, past[0]);
-#pragma unroll
-        for (int j = 0; j < kN; ++j)
-#pragma unroll
-          for (int c = 0; c < 8; ++c) s[c] = fmaf(w[j][c], past[j][c], s[c]);
-      } else {
-        for (int j = 0; j < a.n; ++j) {
-          float f[8];
-          input(t, j, f);
-#pragma unroll
-          for (int c = 0; c < 8; ++c)
-            if (c < nc) s[c] = fmaf(a.taps[(a.n - 1 - j) * a.channels + ch + c], f[c], s[c]);
-        }
+        for (int c = 0; c < 8; ++c)
+          if (c < nc) s[c] = fmaf(a.taps[(a.n - 1 - j) * a.channels + ch + c], f[c], s[c]);
       }
     }
-    prev_req = req;
-    prev_pos = pos;
-    __align__(16) __nv_bfloat162 b[4];
+    put(t, s);
+  }
+}
+
+// Convolution inputs of one of a span's last tokens, into its request's ring: this caller's share (part of parts, `threads` wide).
+template <typename A>
+__device__ __forceinline__ void keep_inputs(const A* x, A* ring, int req, long long pos, int last, int keep, int channels, int part,
+                                            int parts, int thread, int threads) {
+  if (keep <= 0 || pos <= last - keep) return;
+  A* dst = ring + (static_cast<long long>(req) * keep + pos % keep) * channels;
+  for (int c = part * threads + thread; c < channels; c += parts * threads) dst[c] = x[c];
+}
+
+// One warp per (token, norm part) of at most 128 * NV columns, which stay in registers.
+template <int NV>
+__global__ void __launch_bounds__(256)
+mamba2_finish_warp_kernel(const float* __restrict__ o, const __nv_bfloat16* __restrict__ proj, long long ldp, int z_off, int x_off,
+                          int channels, const float* __restrict__ w, float eps, const int* __restrict__ tok_req,
+                          const int64_t* __restrict__ positions, const int* __restrict__ last_pos, __nv_bfloat16* __restrict__ ring,
+                          int taps, __nv_bfloat16* __restrict__ out, long long ldo, int cols, int inner, int part, int parts, int T) {
+  pdl_wait();
+  pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const long long u = blockIdx.x * 8ll + (threadIdx.x >> 5), t = u / parts;
+  if (t >= T) return;
+  const int g = static_cast<int>(u - t * parts), c0 = g * part, req = tok_req[t];
+  const long long pos = positions[t];
+  __nv_bfloat16* to = out + t * ldo;
+  if (g == parts - 1)
+    for (int c = inner + lane; c < cols; c += 32) to[c] = __float2bfloat16(0.f);
+  if (req < 0 || pos < 0) {
+    for (int c = lane; c < part; c += 32) to[c0 + c] = __float2bfloat16(0.f);
+    return;
+  }
+  const __nv_bfloat16* p = proj + t * ldp;
+  const float4* x = reinterpret_cast<const float4*>(o + t * inner + c0);
+  const uint2* z = reinterpret_cast<const uint2*>(p + z_off + c0);
+  float4 y[NV];
+  uint2 zu[NV];
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const float x = s[2 * c], y = s[2 * c + 1];
-      b[c] = __floats2bfloat162_rn(2 * c < nc ? x / (1.f + __expf(-x)) : 0.f, 2 * c + 1 < nc ? y / (1.f + __expf(-y)) : 0.f);
-    }
-    *reinterpret_cast<uint4*>(out + t * ldo + ch) = *reinterpret_cast<const uint4*>(b);
+  for (int i = 0; i < NV; ++i) {
+    const int c = i * 32 + lane;
+    const bool ok = c * 4 < part;
+    y[i] = ok ? x[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    zu[i] = ok ? z[c] : make_uint2(0, 0);
+  }
+  keep_inputs(p + x_off, ring, req, pos, last_pos[t], taps - 1, channels, g, parts, lane, 32);
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const float2 z0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zu[i].x));
+    const float2 z1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zu[i].y));
+    y[i].x *= z0.x / (1.f + __expf(-z0.x));
+    y[i].y *= z0.y / (1.f + __expf(-z0.y));
+    y[i].z *= z1.x / (1.f + __expf(-z1.x));
+    y[i].w *= z1.y / (1.f + __expf(-z1.y));
+    ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+  }
+  const float r = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(part) + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = i * 32 + lane;
+    if (c * 4 >= part) continue;
+    const float4 f = reinterpret_cast<const float4*>(w + c0)[c];
+    uint2 pk;
+    *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(y[i].x * r * f.x, y[i].y * r * f.y);
+    *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(y[i].z * r * f.z, y[i].w * r * f.w);
+    reinterpret_cast<uint2*>(to + c0)[c] = pk;
   }
 }
 
@@ -187,11 +251,7 @@ mamba2_finish_kernel(const float* __restrict__ o, const A* __restrict__ proj, lo
     return;
   }
   const A* p = proj + t * ldp;
-  const int keep = taps - 1;
-  if (keep > 0 && pos > last_pos[t] - keep) {
-    A* dst = ring + (static_cast<long long>(req) * keep + pos % keep) * channels;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) dst[c] = p[x_off + c];
-  }
+  keep_inputs(p + x_off, ring, req, pos, last_pos[t], taps - 1, channels, blockIdx.y, gridDim.y, threadIdx.x, blockDim.x);
   const float* x = o + t * inner + c0;
   const A* z = p + z_off + c0;
   float ss = 0.f;
@@ -232,26 +292,27 @@ mamba2_finish_kernel(const float* __restrict__ o, const A* __restrict__ proj, lo
 
 using namespace stk;
 
-// Spans of min_span .. max_span tokens, token by token.
-STK_API int stk_mamba2_scan(const void* proj, long long ldp, int x_off, int dt_off, const float* taps, const float* conv_bias, int n_taps,
-                            const void* ring, const float* dt_bias, const float* neg_a, const float* skip, const int* query_start,
+// Spans of min_span .. max_span tokens, token by token, over the operands of stk_mamba2_conv.
+STK_API int stk_mamba2_scan(const void* xbc, long long ld, const float* steps, const float* skip, const int* query_start,
                             const int* req_rows, const int* start_pos, int n_req, float* S, float* o, int heads, int state, int vdim,
                             int groups, int fp32, int min_span, int max_span, int T, void* stream) {
   if (T <= 0) return 0;
-  if (n_taps < 1 || groups < 1 || heads % groups) return -1;
+  if (groups < 1 || heads % groups) return -1;
   const ScanArgs a{query_start, req_rows, start_pos, n_req, S, o, heads, state, vdim};
-  const int inner = heads * vdim;
-  const ConvArgs c{proj, ldp, x_off, dt_off, taps, conv_bias, n_taps, ring, dt_bias, neg_a, inner + 2 * groups * state};
+  const int inner = heads * vdim, hpg = heads / groups;
   if (fp32)
-    return launch_scan(Mamba2Front<float>{c, state, vdim, inner, groups, heads / groups, skip}, a, min_span, max_span, (cudaStream_t)stream);
-  return launch_scan(Mamba2Front<__nv_bfloat16>{c, state, vdim, inner, groups, heads / groups, skip}, a, min_span, max_span,
-                     (cudaStream_t)stream);
+    return launch_scan(Mamba2Front<float>{(const float*)xbc, ld, steps, state, vdim, inner, groups, hpg, heads, T, skip}, a, min_span,
+                       max_span, (cudaStream_t)stream);
+  return launch_scan(Mamba2Front<__nv_bfloat16>{(const __nv_bfloat16*)xbc, ld, steps, state, vdim, inner, groups, hpg, heads, T, skip}, a,
+                     min_span, max_span, (cudaStream_t)stream);
 }
 
-// bf16.  out [T, ldo]: convolved channels, zeros up to ldo (a multiple of 8); steps fp32 [2, heads, T]: log decays, step sizes.
+// out [T, ldo] in the compute type: convolved channels, zeros up to ldo (a multiple of 8); steps fp32 [2, heads, T]: log decays, step
+// sizes.
 STK_API int stk_mamba2_conv(const void* proj, long long ldp, int x_off, int dt_off, const float* taps, const float* conv_bias, int n_taps,
                             const void* ring, const float* dt_bias, const float* neg_a, const int64_t* positions, const int* tok_req,
-                            const int* first_pos, void* out, long long ldo, float* steps, int heads, int channels, int T, void* stream) {
+                            const int* first_pos, void* out, long long ldo, float* steps, int heads, int channels, int fp32, int T,
+                            void* stream) {
   if (T <= 0) return 0;
   if (n_taps < 1 || ldo % 8 || ldo < channels || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
   const ConvArgs c{proj, ldp, x_off, dt_off, taps, conv_bias, n_taps, ring, dt_bias, neg_a, channels};
@@ -259,13 +320,17 @@ STK_API int stk_mamba2_conv(const void* proj, long long ldp, int x_off, int dt_o
                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(ring)) & 15) == 0;
   const dim3 grid(static_cast<unsigned>((ldo + 1023) / 1024 + 1), (T + kConvTok - 1) / kConvTok);
   cudaStream_t st = (cudaStream_t)stream;
-#define STK_CONV(N) \
-  launch_pdl(mamba2_conv_kernel<N>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (__nv_bfloat16*)out, ldo, steps, heads, T, vec)
-  switch (n_taps) {
-    case 2: STK_CONV(2); break;
-    case 3: STK_CONV(3); break;
-    case 4: STK_CONV(4); break;
-    default: STK_CONV(0); break;
+#define STK_CONV(A, N) \
+  launch_pdl(mamba2_conv_kernel<A, N>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec)
+  if (fp32) {
+    STK_CONV(float, 0);
+  } else {
+    switch (n_taps) {
+      case 2: STK_CONV(__nv_bfloat16, 2); break;
+      case 3: STK_CONV(__nv_bfloat16, 3); break;
+      case 4: STK_CONV(__nv_bfloat16, 4); break;
+      default: STK_CONV(__nv_bfloat16, 0); break;
+    }
   }
 #undef STK_CONV
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -285,6 +350,18 @@ STK_API int stk_mamba2_finish(const float* o, const void* proj, long long ldp, i
     return -3;
   const dim3 grid(T, norm_groups);
   cudaStream_t st = (cudaStream_t)stream;
+  if (!fp32 && part <= 1024 && part % 4 == 0 && ldp % 4 == 0 && ldo % 4 == 0 && z_off % 4 == 0 &&
+      ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(out)) & 7) == 0) {
+    const dim3 warps(static_cast<unsigned>((static_cast<long long>(T) * norm_groups + 7) / 8));
+#define STK_FINISH(NV)                                                                                                             \
+  launch_pdl(mamba2_finish_warp_kernel<NV>, warps, dim3(256), 0, st, o, (const __nv_bfloat16*)proj, ldp, z_off, x_off, channels, norm_w, \
+             eps, tok_req, positions, last_pos, (__nv_bfloat16*)ring, n_taps, (__nv_bfloat16*)out, ldo, cols, inner, part, norm_groups, T)
+    if (part <= 256) STK_FINISH(2);
+    else if (part <= 512) STK_FINISH(4);
+    else STK_FINISH(8);
+#undef STK_FINISH
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  }
   if (fp32)
     launch_pdl(mamba2_finish_kernel<float>, grid, dim3(256), smem, st, o, (const float*)proj, ldp, z_off, x_off, channels, norm_w, eps,
                tok_req, positions, last_pos, (float*)ring, n_taps, (float*)out, ldo, cols, inner, part);

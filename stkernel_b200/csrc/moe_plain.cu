@@ -37,10 +37,19 @@ template <> struct Vec16<__nv_bfloat16> {
 
 constexpr int kRowsPerWarp = 4, kExpertWarps = 8;
 
-// act 0: none, 1: relu squared, 2: gelu (exact)
+// act 0: none, 1: relu squared, 2: gelu (exact).  kRounded: the result is rounded to bf16, so the gelu's erfc may come from the rational
+// approximation 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions (absolute error 1.5e-7).
+template <bool kRounded = true>
 __device__ __forceinline__ float expert_act(float v, int act) {
   if (act == 1) return v > 0.f ? v * v : 0.f;
-  if (act == 2) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  if (act == 2) {
+    if (!kRounded) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+    const float z = fabsf(v) * 0.70710678118654752f;
+    const float t = __fdividef(1.f, fmaf(0.3275911f, z, 1.f));
+    const float p = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+    const float half = 0.5f * v * p * __expf(-z * z);       // v erfc(|v| / sqrt 2) / 2
+    return v < 0.f ? half : v - half;
+  }
   return v;
 }
 
@@ -76,7 +85,7 @@ expert_rows_kernel(const A* __restrict__ x, long long ldx, int div, const A* __r
 #pragma unroll
   for (int r = 0; r < kRowsPerWarp; ++r) {
     float v = warp_sum(acc[r]);
-    v = expert_act(v, act);
+    v = expert_act<sizeof(A) == 2>(v, act);
     if (lane == 0 && n0 + r < n_pad) out[pair * ldo + n0 + r] = V::round(ok && n0 + r < N ? v : 0.f);
   }
 }

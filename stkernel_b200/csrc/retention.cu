@@ -27,7 +27,6 @@ __device__ __forceinline__ float rotated(const RotArgs& r, const A* x, int d, lo
 
 template <typename A>
 struct RetentionFront {
-  static constexpr bool kValues = false;
   RotArgs r;
   int v_off, D, V;
   const float* decay;                             // [2][H]: the decays and what their rounding left over
@@ -36,7 +35,7 @@ struct RetentionFront {
   __device__ __forceinline__ float value(long long t, int h, int col) const {
     return ld_act(reinterpret_cast<const A*>(r.proj) + t * r.ldp + v_off + h * V + col);
   }
-  __device__ __forceinline__ float2 fill(long long t, int, long long pos, long long, int h, int, int, float* q, float* k, float*) const {
+  __device__ __forceinline__ float2 fill(long long t, long long pos, int h, float* q, float* k) const {
     const A* p = reinterpret_cast<const A*>(r.proj) + t * r.ldp;
     for (int e = threadIdx.x; e < 2 * D; e += kScanThreads) {
       if (e < D) q[e] = rotated(r, p + r.q_off + h * D, e, pos);
@@ -46,10 +45,33 @@ struct RetentionFront {
   }
 };
 
+// Eight fp32 values as bf16 high parts and remainders, `n` elements apart.
+__device__ __forceinline__ void store_pair8(__nv_bfloat16* dst, int n, const float (&y)[8]) {
+  uint4 hi, lo;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(y[2 * j], y[2 * j + 1]);
+    const float2 f = __bfloat1622float2(h);
+    reinterpret_cast<__nv_bfloat162*>(&hi)[j] = h;
+    reinterpret_cast<__nv_bfloat162*>(&lo)[j] = __floats2bfloat162_rn(y[2 * j] - f.x, y[2 * j + 1] - f.y);
+  }
+  *reinterpret_cast<uint4*>(dst) = hi;
+  *reinterpret_cast<uint4*>(dst + n) = lo;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 v = *reinterpret_cast<const uint4*>(p);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 u = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
+    f[2 * j] = u.x;
+    f[2 * j + 1] = u.y;
+  }
+}
+
 // out [T][q high | q remainder | k high | k remainder][H * D8], zeros behind each head's D columns.  One CTA per token; the cos and
-// sin of its position are formed once for all heads.
+// sin of its position are formed once for all heads.  vec: heads, rotated pairs and rows in whole groups of eight.
 __global__ void __launch_bounds__(256)
-rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bfloat16* __restrict__ out, int H, int D, int D8) {
+rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bfloat16* __restrict__ out, int H, int D, int D8, int vec) {
   extern __shared__ float2 cs[];
   pdl_wait();
   pdl_trigger();
@@ -60,6 +82,35 @@ rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bf
   const __nv_bfloat16* p = reinterpret_cast<const __nv_bfloat16*>(r.proj) + t * r.ldp;
   const int n = H * D8;
   __nv_bfloat16* o = out + t * 4 * n;
+  if (vec) {
+    const int turned = r.pairs >> 3, items = turned + ((D - 2 * r.pairs) >> 3);      // per head: pairs of groups, then plain groups
+    for (int e = threadIdx.x; e < 2 * H * items; e += blockDim.x) {
+      const int u = e / items, i = e - u * items, isk = u >= H ? 1 : 0, h = u - isk * H;
+      const __nv_bfloat16* x = p + (isk ? r.k_off : r.q_off) + h * D;
+      __nv_bfloat16* dst = o + isk * 2 * n + h * D8;
+      const float f = isk ? r.k_scale : 1.f;
+      float a[8], b[8], y[8], z[8];
+      if (i < turned) {
+        load8(x + i * 8, a);
+        load8(x + r.pairs + i * 8, b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float2 w = cs[i * 8 + j];
+          y[j] = (a[j] * w.x - b[j] * w.y) * f;
+          z[j] = (b[j] * w.x + a[j] * w.y) * f;
+        }
+        store_pair8(dst + i * 8, n, y);
+        store_pair8(dst + r.pairs + i * 8, n, z);
+      } else {
+        const int d = 2 * r.pairs + (i - turned) * 8;
+        load8(x + d, a);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[j] = a[j] * f;
+        store_pair8(dst + d, n, y);
+      }
+    }
+    return;
+  }
   for (int e = threadIdx.x; e < n; e += blockDim.x) {               // two columns, e / (D8 / 2) the (q or k, head)
     const int half = D8 / 2, u = e / half, d0 = (e - u * half) * 2, isk = u >= H ? 1 : 0, h = u - isk * H;
     const __nv_bfloat16* x = p + (isk ? r.k_off : r.q_off) + h * D;
@@ -164,8 +215,10 @@ STK_API int stk_rotate_qk(const void* proj, long long ldp, int q_off, int k_off,
   if (T <= 0) return 0;
   if (pairs < 0 || 2 * pairs > dim || d8 < dim || d8 % 8) return -1;
   const RotArgs r{proj, ldp, q_off, k_off, freq, pairs, k_scale};
+  const int vec = pairs % 8 == 0 && dim % 8 == 0 && ldp % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 &&
+                  ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   launch_pdl(rotate_qk_kernel, dim3(T), dim3(256), static_cast<size_t>(pairs) * sizeof(float2), (cudaStream_t)stream, r, positions,
-             (__nv_bfloat16*)out, heads, dim, d8);
+             (__nv_bfloat16*)out, heads, dim, d8, vec);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

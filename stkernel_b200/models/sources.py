@@ -50,4 +50,9 @@ class RandomSource(WeightSource):
             return torch.zeros(shape, device=dev)
         if name.endswith("gate.bias"):
             return torch.rand(shape, generator=g, device=dev) * 0.2 - 0.1
-        return torch.randn(shape, generator=g, device=dev) * self.std
+        noise = torch.randn(shape, generator=g, device=dev) * self.std
+        if name.endswith((".hc1.mix", ".hc2.mix")):
+            return noise + torch.eye(shape[0], device=dev)                     # residual streams mostly stay themselves
+        if ".hc" in name or name.endswith(".dt_bias"):
+            return noise + (0.5 if ".hc" in name else -2.0)
+        return noise

@@ -1,9 +1,9 @@
 """Linear recurrences with a scalar decay per head and token, S <- a S + k v^T, o = S^T q (state fp32): retention (fixed decay, rotated
 queries and keys) and Mamba-2 (decay and input weight from a step size, operands behind a short causal convolution).
 
-Short spans and float32 models run token by token (`*_scan`: rotation, convolution and step sizes on the way in); longer spans of bf16
-models in chunks on the tensor cores (`stk_linear_chunks`, common to both).  What enters the recurrence in fp32 (rotated queries and
-keys, decays, weighted keys, the state) meets the tensor cores as bf16 pairs, high part and remainder.
+Short spans and float32 models run token by token (`*_scan`); longer spans of bf16 models in chunks on the tensor cores
+(`stk_linear_chunks`, common to both).  What enters the recurrence in fp32 (rotated queries and keys, decays, weighted values, the
+state) meets the tensor cores as bf16 pairs, high part and remainder.
 """
 from __future__ import annotations
 
@@ -139,16 +139,15 @@ def mamba2(p: torch.Tensor, z_off: int, x_off: int, dt_off: int, a: Mamba2Params
         return
     o = scratch("scan.out", (t, inner), F32, p.device)
     chunked = _chunked(p, meta, n)
-    conv = (a.taps, a.conv_bias, taps, ring, a.dt_bias, a.neg_a)
+    ld = _up8(cd)
+    xbc = scratch("scan.xbc", (t, ld), p.dtype, p.device)
+    step = scratch("scan.steps", (2, h, t), F32, p.device)
+    _lib.call("stk_mamba2_conv", p, p.stride(0), x_off, dt_off, a.taps, a.conv_bias, taps, ring, a.dt_bias, a.neg_a, meta.positions,
+              meta.tok_req, meta.first_pos, xbc, ld, step, h, cd, _is32(p), t, _lib.stream())
     if not chunked or meta.min_span < CHUNK_SPAN:
-        _lib.call("stk_mamba2_scan", p, p.stride(0), x_off, dt_off, *conv, a.skip, meta.query_start, meta.req_rows, meta.start_pos,
-                  meta.n_req, S, o, h, n, v, g, _is32(p), 1, (CHUNK_SPAN - 1) if chunked else 1 << 30, t, _lib.stream())
+        _lib.call("stk_mamba2_scan", xbc, ld, step, a.skip, meta.query_start, meta.req_rows, meta.start_pos, meta.n_req, S, o, h, n, v, g,
+                  _is32(p), 1, (CHUNK_SPAN - 1) if chunked else 1 << 30, t, _lib.stream())
     if chunked:
-        ld = _up8(cd)
-        xbc = scratch("scan.xbc", (t, ld), BF16, p.device)
-        step = scratch("scan.steps", (2, h, t), F32, p.device)
-        _lib.call("stk_mamba2_conv", p, p.stride(0), x_off, dt_off, *conv, meta.positions, meta.tok_req, meta.first_pos, xbc, ld, step,
-                  h, cd, t, _lib.stream())
         _chunks((xbc[:, inner + g * n:], None, xbc[:, inner:], None, ld, n, n), xbc, 0, h // g, None, (step[0], step[1]), a.skip, meta,
                 S, o)
     _lib.call("stk_mamba2_finish", o, p, p.stride(0), z_off, x_off, cd, a.norm, float(a.eps), a.norm_groups, meta.tok_req,

@@ -9,6 +9,8 @@ replay a CUDA graph per batch-size bucket.
 """
 from __future__ import annotations
 
+import contextlib
+import gc
 import time
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Sequence, Tuple
@@ -966,6 +968,20 @@ def _capture_stream(device) -> "torch.cuda.Stream":
     return _CAPTURE_STREAMS[idx]
 
 
+@contextlib.contextmanager
+def _capturing(graph: "torch.cuda.CUDAGraph", device):
+    """Capture into `graph` without cyclic garbage collection: a collector that runs in the middle may release an earlier engine's
+    graphs and events, which is not permitted while a stream is being captured."""
+    was = gc.isenabled()
+    gc.disable()
+    try:
+        with torch.cuda.graph(graph, stream=_capture_stream(device)):
+            yield
+    finally:
+        if was:
+            gc.enable()
+
+
 def _after_capture_rendezvous(eng: "Engine") -> None:
     """Capturing a step takes a rank-dependent amount of host time (hundreds of milliseconds for a deep model).  The
     kernels of the first replay poll their peers with a bounded budget, so the ranks meet on the host before any of
@@ -989,7 +1005,7 @@ class SpecGraph:
         torch.cuda.synchronize()
         before = _lib.launch_count
         self.graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self.graph, stream=_capture_stream(eng.device)):
+        with _capturing(self.graph, eng.device):
             self.out = eng._spec_device(t, n_req, ns, nb, rows_bucket)
         self.launches_per_replay = _lib.launch_count - before
         _after_capture_rendezvous(eng)
@@ -1023,7 +1039,7 @@ class DecodeGraph:
         from ..ops import _lib
         before = _lib.launch_count
         self.graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self.graph, stream=_capture_stream(eng.device)):
+        with _capturing(self.graph, eng.device):
             self.out = eng._run_model(bucket, bucket, bucket, rows_bucket, identity_rows=True)
         self.launches_per_replay = _lib.launch_count - before
         if ranges is not None:
