@@ -4,7 +4,7 @@
 //   o_t   = exp(F_t) S_start^T q_t + sum_{j <= t} exp(F_t - F_j) w_j (k_j . q_t) v_j  (+ skip v_t)
 //   S_end = exp(F_end) S_start + sum_j exp(F_end - F_j) w_j k_j v_j^T
 //
-//   linear_chunk_state     one CTA per 64 x 64 block of a head's state (transposed: 16 value rows per warp) walks the chunks of a
+//   linear_chunk_state     one CTA per 64 x 64 block of a head's state (transposed: 16 value rows x 32 state rows per warp) walks the chunks of a
 //                          request with the block in its accumulators and leaves the state before each chunk
 //   linear_chunk_out       per chunk, head and 64 or 128 value columns: the outputs, 16 columns per warp
 //
@@ -78,7 +78,7 @@ __device__ __forceinline__ ChunkGates chunk_gates(const ChunkArgs& a, const Chun
 constexpr int kLsStages = 3;
 
 template <bool kPair>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   constexpr int kTile = kChunk * kStStride, kParts = kPair ? 2 : 1, kStage = (kParts + 1) * kTile;
@@ -93,14 +93,15 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
   const long long row = s.req_rows[ri];
   const bool fresh = s.start_pos[ri] == 0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int v0 = vb * 64 + warp * 16 + (lane >> 2), d0 = db * 64 + (lane & 3) * 2;     // accumulator rows v0 (+ 8), columns d0 + 8 j (+ 1)
+  const int vw = warp & 3, dw = warp >> 2;                              // the warp's 16 rows, its half of the 64 columns
+  const int v0 = vb * 64 + vw * 16 + (lane >> 2), d0 = db * 64 + dw * 32 + (lane & 3) * 2;   // accumulator rows v0 (+ 8), columns d0 + 8 j (+ 1)
   const int nd = blocks16(s.D);
   const long long slot_f = linear_slot_floats(s.D, s.V);
   float* gS = s.S + (row * s.H + h) * static_cast<long long>(s.D) * s.V;
   const int kn = max(0, min(64, a.width - db * 64)), vn = min(64, s.V - vb * 64);
-  float acc[8][4];
+  float acc[4][4];
 #pragma unroll
-  for (int j = 0; j < 8; ++j)
+  for (int j = 0; j < 4; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int v = v0 + (i >> 1) * 8, d = d0 + j * 8 + (i & 1);
@@ -111,16 +112,16 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
     const int n = min(kChunk, span - c * kChunk);
     const long long t0 = q0 + c * kChunk;
     bf16* to = tiles + c % kLsStages * kStage;
-    load_rows_async(to, kStStride, 64, a.v + t0 * a.ldv + a.v_off + h * s.V + vb * 64, a.ldv, n, vn, 128);
-    load_rows_async(to + kTile, kStStride, 64, a.kh + t0 * a.ldqk + kc, a.ldqk, n, kn, 128);
-    if (kPair) load_rows_async(to + 2 * kTile, kStStride, 64, a.kl + t0 * a.ldqk + kc, a.ldqk, n, kn, 128);
+    load_rows_async(to, kStStride, 64, a.v + t0 * a.ldv + a.v_off + h * s.V + vb * 64, a.ldv, n, vn, 256);
+    load_rows_async(to + kTile, kStStride, 64, a.kh + t0 * a.ldqk + kc, a.ldqk, n, kn, 256);
+    if (kPair) load_rows_async(to + 2 * kTile, kStStride, 64, a.kl + t0 * a.ldqk + kc, a.ldqk, n, kn, 256);
   };
   load(0);
   mls_commit();
   if (nc > 1) load(1);
   mls_commit();
   ChunkRaw raw = load_gates(a, h, q0, min(kChunk, span), lane);
-  const bool block_ok = vb * 64 + warp * 16 < s.V;                      // warp-uniform: its 16 rows exist
+  const bool block_ok = vb * 64 + vw * 16 < s.V;                      // warp-uniform: its 16 rows exist
   for (int c = 0; c < nc; ++c) {
     const int n = min(kChunk, span - c * kChunk);
     const ChunkGates g = chunk_gates(a, raw, n, lane);
@@ -133,10 +134,10 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
     // the state before this chunk
     if (block_ok) {
       float* slot = states + (static_cast<long long>(first + c) * s.H + h) * slot_f +
-                    (static_cast<long long>(vb * 4 + warp) * nd + db * 4) * kBlockFloats;
+                    (static_cast<long long>(vb * 4 + vw) * nd + db * 4 + dw * 2) * kBlockFloats;
 #pragma unroll
-      for (int p = 0; p < 4; ++p) {
-        if (db * 4 + p < nd) {
+      for (int p = 0; p < 2; ++p) {
+        if (db * 4 + dw * 2 + p < nd) {
           uint4 hi, lo;
           mls_split2(acc[2 * p][0], acc[2 * p][1], hi.x, lo.x);
           mls_split2(acc[2 * p + 1][0], acc[2 * p + 1][1], hi.y, lo.y);
@@ -149,7 +150,7 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
       }
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[j][i] *= fs;
     const bf16* v = tiles + c % kLsStages * kStage;
@@ -157,7 +158,7 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
 #pragma unroll
     for (int kk = 0; kk < kChunk / 16; ++kk) {
       uint32_t af[4], ah[4], al[4];
-      mls_ldsm4_t(af, v + (kk * 16 + (lane & 7) + (lane >> 4) * 8) * kStStride + warp * 16 + ((lane >> 3) & 1) * 8);
+      mls_ldsm4_t(af, v + (kk * 16 + (lane & 7) + (lane >> 4) * 8) * kStStride + vw * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
       for (int i = 0; i < 2; ++i) {                                     // the operand's token pairs: 2 (lane & 3) and 8 further
         const int from = kk * 8 + i * 4 + (lane & 3);
@@ -169,9 +170,9 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
         }
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
+      for (int j = 0; j < 2; ++j) {
         uint32_t b[4];
-        const int off = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kStStride + j * 16 + (lane >> 4) * 8;
+        const int off = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kStStride + dw * 32 + j * 16 + (lane >> 4) * 8;
         mls_ldsm4_t(b, k + off);
         mls_mma(acc[2 * j], ah, b[0], b[1]);
         mls_mma(acc[2 * j + 1], ah, b[2], b[3]);
@@ -188,7 +189,7 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
   }
   mls_wait<0>();
 #pragma unroll
-  for (int j = 0; j < 8; ++j)
+  for (int j = 0; j < 4; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int v = v0 + (i >> 1) * 8, d = d0 + j * 8 + (i & 1);
@@ -420,7 +421,7 @@ static int launch_chunks(const ChunkArgs& a, int min_span, float* states, int ma
   if (cudaFuncSetAttribute(linear_chunk_state_kernel<kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, 84 * 1024) != cudaSuccess ||
       cudaFuncSetAttribute(linear_chunk_out_kernel<kPair, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess)
     return -3;
-  launch_pdl(linear_chunk_state_kernel<kPair>, dim3((s.V + 63) / 64, (s.D + 63) / 64, s.H * s.n_req), dim3(128), smem_s, st, a, min_span,
+  launch_pdl(linear_chunk_state_kernel<kPair>, dim3((s.V + 63) / 64, (s.D + 63) / 64, s.H * s.n_req), dim3(256), smem_s, st, a, min_span,
              states);
   launch_pdl(linear_chunk_out_kernel<kPair, COLS>, dim3((s.V + COLS - 1) / COLS, max_chunks, s.H), dim3(COLS * 2), smem_o, st, a, min_span,
              states);

@@ -44,12 +44,12 @@ struct Mamba2Front {
   }
 };
 
-constexpr int kConvTok = 8;
+constexpr int kConvTok = 16, kConvBatch = 8;
 
-// Eight channels x kConvTok tokens per thread.  NT > 0 taps: the inputs of tokens that follow one another in one span are all in
-// flight together and stay in registers; otherwise (spans that meet inside the group, many taps) every tap is read where it is
-// used.  The grid's last column of blocks forms the step sizes.
-template <typename A, int NT>
+// Eight channels x TOK tokens per thread.  NT > 0 taps: the inputs of tokens that follow one another in one span are fetched
+// kConvBatch at a time and slide through registers; otherwise (spans that meet inside the group, many taps) every tap is read where it
+// is used.  The grid's last column of blocks forms the step sizes.
+template <typename A, int NT, int TOK>
 __global__ void __launch_bounds__(128)
 mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, const int* __restrict__ tok_req,
                    const int* __restrict__ first_pos, A* __restrict__ out, long long ldo, float* __restrict__ steps, int H, int T,
@@ -57,11 +57,11 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
   pdl_wait();
   pdl_trigger();
   const A* proj = reinterpret_cast<const A*>(a.proj);
-  const int t0 = blockIdx.y * kConvTok, t1 = min(T, t0 + kConvTok);
+  const int t0 = blockIdx.y * TOK, t1 = min(T, t0 + TOK);
   if (blockIdx.x == gridDim.x - 1) {
     // steps [0][H][T]: log decays, [1][H][T]: step sizes
-    for (int e = threadIdx.x; e < kConvTok * H; e += 128) {
-      const int h = e / kConvTok, t = t0 + e % kConvTok;
+    for (int e = threadIdx.x; e < TOK * H; e += 128) {
+      const int h = e / TOK, t = t0 + e % TOK;
       if (t >= T) continue;
       const float dt = softplus_f(ld_act(proj + t * a.ldp + a.dt_off + h) + a.dt_bias[h]);
       steps[static_cast<long long>(h) * T + t] = dt * a.neg_a[h];
@@ -89,6 +89,15 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
       for (int c = 0; c < 8; ++c) f[c] = src != nullptr && c < nc ? ld_act(src + c) : 0.f;
     }
   };
+  auto coeff = [&](const float* src, float (&f)[8]) {
+    if (vec) {
+      const float4 u = *reinterpret_cast<const float4*>(src), v = *reinterpret_cast<const float4*>(src + 4);
+      f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w; f[4] = v.x; f[5] = v.y; f[6] = v.z; f[7] = v.w;
+    } else {
+#pragma unroll
+      for (int c = 0; c < 8; ++c) f[c] = c < nc ? src[c] : 0.f;
+    }
+  };
   // where the input j tokens before token t is: its own span's row, the ring, or nowhere (zero)
   auto where = [&](int t, int j, int req, long long pos, int first) -> const A* {
     if (pos - j >= first) return x + (t - j) * a.ldp;
@@ -101,7 +110,8 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const float y = s[2 * c], z = s[2 * c + 1];
-        b[c] = __floats2bfloat162_rn(2 * c < nc ? y / (1.f + __expf(-y)) : 0.f, 2 * c + 1 < nc ? z / (1.f + __expf(-z)) : 0.f);
+        b[c] = __floats2bfloat162_rn(2 * c < nc ? __fdividef(y, 1.f + __expf(-y)) : 0.f,
+                                     2 * c + 1 < nc ? __fdividef(z, 1.f + __expf(-z)) : 0.f);
       }
       *reinterpret_cast<uint4*>(out + t * ldo + ch) = *reinterpret_cast<const uint4*>(b);
     } else {
@@ -109,35 +119,37 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
       for (int c = 0; c < 8; ++c) st_act(out + t * ldo + ch + c, c < nc ? silu_f(s[c]) : 0.f);
     }
   };
-  float bias[8];
-#pragma unroll
-  for (int c = 0; c < 8; ++c) bias[c] = c < nc ? a.bias[ch + c] : 0.f;
   const int req0 = tok_req[t0], first0 = first_pos[t0];
   const long long pos0 = positions[t0];
+  float bias[8];
+  coeff(a.bias + ch, bias);
   if (NT > 0 && req0 >= 0 && pos0 >= 0 && tok_req[t1 - 1] == req0 && positions[t1 - 1] == pos0 + (t1 - 1 - t0)) {
-    constexpr int kN = NT > 0 ? NT : 1;
+    constexpr int kN = NT > 0 ? NT : 1, kB = TOK < kConvBatch ? TOK : kConvBatch;
     float w[kN][8];
 #pragma unroll
-    for (int j = 0; j < kN; ++j)
+    for (int j = 0; j < kN; ++j) coeff(a.taps + (a.n - 1 - j) * a.channels + ch, w[j]);
+    float in[kB + kN - 1][8];                             // inputs of the kN - 1 tokens before a batch, then the batch's
 #pragma unroll
-      for (int c = 0; c < 8; ++c) w[j][c] = c < nc ? a.taps[(a.n - 1 - j) * a.channels + ch + c] : 0.f;
-    float in[kConvTok + kN - 1][8];                       // inputs of tokens t0 - (n - 1) .. t0 + 7
+    for (int i = 0; i < kN - 1; ++i) fetch(where(t0, kN - 1 - i, req0, pos0, first0), in[kB + i]);
+    for (int b0 = t0; b0 < t1; b0 += kB) {
 #pragma unroll
-    for (int i = 0; i < kConvTok + kN - 1; ++i) {
-      const int j = kN - 1 - i;                           // tokens before t0
-      fetch(j > 0 ? where(t0, j, req0, pos0, first0) : t0 - j < t1 ? x + (t0 - j) * a.ldp : nullptr, in[i]);
-    }
+      for (int i = 0; i < kN - 1; ++i)
 #pragma unroll
-    for (int i = 0; i < kConvTok; ++i) {
-      if (t0 + i < t1) {
-        float s[8];
+        for (int c = 0; c < 8; ++c) in[i][c] = in[kB + i][c];
 #pragma unroll
-        for (int c = 0; c < 8; ++c) {
-          s[c] = bias[c];
+      for (int i = 0; i < kB; ++i) fetch(b0 + i < t1 ? x + (b0 + i) * a.ldp : nullptr, in[kN - 1 + i]);
 #pragma unroll
-          for (int j = 0; j < kN; ++j) s[c] = fmaf(w[j][c], in[i + kN - 1 - j][c], s[c]);
+      for (int i = 0; i < kB; ++i) {
+        if (b0 + i < t1) {
+          float s[8];
+#pragma unroll
+          for (int c = 0; c < 8; ++c) {
+            s[c] = bias[c];
+#pragma unroll
+            for (int j = 0; j < kN; ++j) s[c] = fmaf(w[j][c], in[i + kN - 1 - j][c], s[c]);
+          }
+          put(b0 + i, s);
         }
-        put(t0 + i, s);
       }
     }
     return;
@@ -151,11 +163,11 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
     if (req >= 0 && pos >= 0) {
 #pragma unroll 4
       for (int j = 0; j < a.n; ++j) {
-        float f[8];
+        float f[8], w[8];
         fetch(where(t, j, req, pos, first), f);
+        coeff(a.taps + (a.n - 1 - j) * a.channels + ch, w);
 #pragma unroll
-        for (int c = 0; c < 8; ++c)
-          if (c < nc) s[c] = fmaf(a.taps[(a.n - 1 - j) * a.channels + ch + c], f[c], s[c]);
+        for (int c = 0; c < 8; ++c) s[c] = fmaf(w[c], f[c], s[c]);
       }
     }
     put(t, s);
@@ -168,6 +180,12 @@ __device__ __forceinline__ void keep_inputs(const A* x, A* ring, int req, long l
                                             int parts, int thread, int threads) {
   if (keep <= 0 || pos <= last - keep) return;
   A* dst = ring + (static_cast<long long>(req) * keep + pos % keep) * channels;
+  constexpr int kVec = 16 / sizeof(A);
+  if (channels % kVec == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(dst)) & 15) == 0) {
+    for (int c = part * threads + thread; c < channels / kVec; c += parts * threads)
+      reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(x)[c];
+    return;
+  }
   for (int c = part * threads + thread; c < channels; c += parts * threads) dst[c] = x[c];
 }
 
@@ -317,11 +335,15 @@ STK_API int stk_mamba2_conv(const void* proj, long long ldp, int x_off, int dt_o
   if (n_taps < 1 || ldo % 8 || ldo < channels || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
   const ConvArgs c{proj, ldp, x_off, dt_off, taps, conv_bias, n_taps, ring, dt_bias, neg_a, channels};
   const int vec = channels % 8 == 0 && ldp % 8 == 0 && x_off % 8 == 0 &&
-                  ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(ring)) & 15) == 0;
-  const dim3 grid(static_cast<unsigned>((ldo + 1023) / 1024 + 1), (T + kConvTok - 1) / kConvTok);
+                  ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(taps) |
+                    reinterpret_cast<uintptr_t>(conv_bias)) & 15) == 0;
+  const bool few = T <= 256;                               // one token per thread
+  const int tok = few ? 1 : kConvTok;
+  const dim3 grid(static_cast<unsigned>((ldo + 1023) / 1024 + 1), (T + tok - 1) / tok);
   cudaStream_t st = (cudaStream_t)stream;
-#define STK_CONV(A, N) \
-  launch_pdl(mamba2_conv_kernel<A, N>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec)
+#define STK_CONV(A, N)                                                                                                               \
+  if (few) launch_pdl(mamba2_conv_kernel<A, N, 1>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec); \
+  else launch_pdl(mamba2_conv_kernel<A, N, kConvTok>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec)
   if (fp32) {
     STK_CONV(float, 0);
   } else {
