@@ -11,6 +11,14 @@ template <typename T> __device__ __forceinline__ void st_act(T* p, float v);
 template <> __device__ __forceinline__ void st_act<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void st_act<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
+// x sigmoid(x) for results that are rounded to bf16: one exponential and one reciprocal of the special-function unit.
+__device__ __forceinline__ float silu_bf16(float x) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return x * r;
+}
+
 // o[j] = act(gate_j) * up_j for j < ff, zero for ff <= j < n: the eight columns from `base` on.  vec: 16-byte accesses allowed.
 // relu: act is relu, else silu.
 template <typename A>

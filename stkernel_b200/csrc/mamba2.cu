@@ -44,13 +44,13 @@ struct Mamba2Front {
   }
 };
 
-constexpr int kConvTok = 16, kConvBatch = 8;
+constexpr int kConvTok = 32, kConvBatch = 8, kConvCh = 4, kConvThreads = 256;
 
-// Eight channels x TOK tokens per thread.  NT > 0 taps: the inputs of tokens that follow one another in one span are fetched
-// kConvBatch at a time and slide through registers; otherwise (spans that meet inside the group, many taps) every tap is read where it
-// is used.  The grid's last column of blocks forms the step sizes.
+// Four channels x TOK tokens per thread.  NT > 0 taps: the inputs of tokens that follow one another in one span slide through
+// registers, a batch of kConvBatch in flight while the one before is summed; otherwise (spans that meet inside the group, many
+// taps, unaligned rows) every tap is read where it is used.  The grid's last column of blocks forms the step sizes.
 template <typename A, int NT, int TOK>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kConvThreads)
 mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, const int* __restrict__ tok_req,
                    const int* __restrict__ first_pos, A* __restrict__ out, long long ldo, float* __restrict__ steps, int H, int T,
                    int vec) {
@@ -60,7 +60,7 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
   const int t0 = blockIdx.y * TOK, t1 = min(T, t0 + TOK);
   if (blockIdx.x == gridDim.x - 1) {
     // steps [0][H][T]: log decays, [1][H][T]: step sizes
-    for (int e = threadIdx.x; e < TOK * H; e += 128) {
+    for (int e = threadIdx.x; e < TOK * H; e += kConvThreads) {
       const int h = e / TOK, t = t0 + e % TOK;
       if (t >= T) continue;
       const float dt = softplus_f(ld_act(proj + t * a.ldp + a.dt_off + h) + a.dt_bias[h]);
@@ -69,33 +69,33 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
     }
     return;
   }
-  const int ch = (blockIdx.x * 128 + threadIdx.x) * 8;
+  const int ch = (blockIdx.x * kConvThreads + threadIdx.x) * kConvCh;
   if (ch >= ldo) return;
-  const int nc = min(8, a.channels - ch), keep = a.n - 1;
+  const int nc = min(kConvCh, a.channels - ch), keep = a.n - 1;
   const A* x = proj + a.x_off + ch;
   const A* ring = reinterpret_cast<const A*>(a.ring) + ch;
-  auto fetch = [&](const A* src, float (&f)[8]) {
+  auto fetch = [&](const A* src, float (&f)[kConvCh]) {
     if (sizeof(A) == 2 && vec) {
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (src != nullptr) v = *reinterpret_cast<const uint4*>(src);
+      uint2 v = make_uint2(0, 0);
+      if (src != nullptr) v = *reinterpret_cast<const uint2*>(src);
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < kConvCh / 2; ++c) {
         const float2 u = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[c]);
         f[2 * c] = u.x;
         f[2 * c + 1] = u.y;
       }
     } else {
 #pragma unroll
-      for (int c = 0; c < 8; ++c) f[c] = src != nullptr && c < nc ? ld_act(src + c) : 0.f;
+      for (int c = 0; c < kConvCh; ++c) f[c] = src != nullptr && c < nc ? ld_act(src + c) : 0.f;
     }
   };
-  auto coeff = [&](const float* src, float (&f)[8]) {
+  auto coeff = [&](const float* src, float (&f)[kConvCh]) {
     if (vec) {
-      const float4 u = *reinterpret_cast<const float4*>(src), v = *reinterpret_cast<const float4*>(src + 4);
-      f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w; f[4] = v.x; f[5] = v.y; f[6] = v.z; f[7] = v.w;
+      const float4 u = *reinterpret_cast<const float4*>(src);
+      f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
     } else {
 #pragma unroll
-      for (int c = 0; c < 8; ++c) f[c] = c < nc ? src[c] : 0.f;
+      for (int c = 0; c < kConvCh; ++c) f[c] = c < nc ? src[c] : 0.f;
     }
   };
   // where the input j tokens before token t is: its own span's row, the ring, or nowhere (zero)
@@ -104,46 +104,59 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
     if (pos >= j) return ring + (static_cast<long long>(req) * keep + (pos - j) % keep) * a.channels;
     return nullptr;
   };
-  auto put = [&](int t, const float (&s)[8]) {
+  auto put = [&](int t, const float (&s)[kConvCh]) {
     if (sizeof(A) == 2) {
-      __align__(16) __nv_bfloat162 b[4];
+      // behind the last channel the sums are zero, and so is silu
+      __align__(8) __nv_bfloat162 b[kConvCh / 2];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < kConvCh / 2; ++c) {
         const float y = s[2 * c], z = s[2 * c + 1];
-        b[c] = __floats2bfloat162_rn(2 * c < nc ? __fdividef(y, 1.f + __expf(-y)) : 0.f,
-                                     2 * c + 1 < nc ? __fdividef(z, 1.f + __expf(-z)) : 0.f);
+        b[c] = __floats2bfloat162_rn(silu_bf16(y), silu_bf16(z));
       }
-      *reinterpret_cast<uint4*>(out + t * ldo + ch) = *reinterpret_cast<const uint4*>(b);
+      *reinterpret_cast<uint2*>(out + t * ldo + ch) = *reinterpret_cast<const uint2*>(b);
     } else {
 #pragma unroll
-      for (int c = 0; c < 8; ++c) st_act(out + t * ldo + ch + c, c < nc ? silu_f(s[c]) : 0.f);
+      for (int c = 0; c < kConvCh; ++c) st_act(out + t * ldo + ch + c, c < nc ? silu_f(s[c]) : 0.f);
     }
   };
   const int req0 = tok_req[t0], first0 = first_pos[t0];
   const long long pos0 = positions[t0];
-  float bias[8];
+  float bias[kConvCh];
   coeff(a.bias + ch, bias);
-  if (NT > 0 && req0 >= 0 && pos0 >= 0 && tok_req[t1 - 1] == req0 && positions[t1 - 1] == pos0 + (t1 - 1 - t0)) {
+  if (NT > 0 && vec && req0 >= 0 && pos0 >= 0 && tok_req[t1 - 1] == req0 && positions[t1 - 1] == pos0 + (t1 - 1 - t0)) {
     constexpr int kN = NT > 0 ? NT : 1, kB = TOK < kConvBatch ? TOK : kConvBatch;
-    float w[kN][8];
+    float w[kN][kConvCh];
 #pragma unroll
     for (int j = 0; j < kN; ++j) coeff(a.taps + (a.n - 1 - j) * a.channels + ch, w[j]);
-    float in[kB + kN - 1][8];                             // inputs of the kN - 1 tokens before a batch, then the batch's
+    float in[kB + kN - 1][kConvCh];                       // inputs of the kN - 1 tokens before a batch, then the batch's
 #pragma unroll
     for (int i = 0; i < kN - 1; ++i) fetch(where(t0, kN - 1 - i, req0, pos0, first0), in[kB + i]);
+    uint2 ahead[kB];
+    auto request = [&](int b0) {
+#pragma unroll
+      for (int i = 0; i < kB; ++i)
+        ahead[i] = b0 + i < t1 ? *reinterpret_cast<const uint2*>(x + (b0 + i) * a.ldp) : make_uint2(0, 0);
+    };
+    request(t0);
     for (int b0 = t0; b0 < t1; b0 += kB) {
 #pragma unroll
       for (int i = 0; i < kN - 1; ++i)
 #pragma unroll
-        for (int c = 0; c < 8; ++c) in[i][c] = in[kB + i][c];
+        for (int c = 0; c < kConvCh; ++c) in[i][c] = in[kB + i][c];
 #pragma unroll
-      for (int i = 0; i < kB; ++i) fetch(b0 + i < t1 ? x + (b0 + i) * a.ldp : nullptr, in[kN - 1 + i]);
+      for (int i = 0; i < kB; ++i) {
+        const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&ahead[i].x));
+        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&ahead[i].y));
+        float (&f)[kConvCh] = in[kN - 1 + i];
+        f[0] = u.x; f[1] = u.y; f[2] = v.x; f[3] = v.y;
+      }
+      if (b0 + kB < t1) request(b0 + kB);
 #pragma unroll
       for (int i = 0; i < kB; ++i) {
         if (b0 + i < t1) {
-          float s[8];
+          float s[kConvCh];
 #pragma unroll
-          for (int c = 0; c < 8; ++c) {
+          for (int c = 0; c < kConvCh; ++c) {
             s[c] = bias[c];
 #pragma unroll
             for (int j = 0; j < kN; ++j) s[c] = fmaf(w[j][c], in[i + kN - 1 - j][c], s[c]);
@@ -157,17 +170,17 @@ mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, cons
   for (int t = t0; t < t1; ++t) {
     const int req = tok_req[t], first = first_pos[t];
     const long long pos = positions[t];
-    float s[8];
+    float s[kConvCh];
 #pragma unroll
-    for (int c = 0; c < 8; ++c) s[c] = bias[c];
+    for (int c = 0; c < kConvCh; ++c) s[c] = bias[c];
     if (req >= 0 && pos >= 0) {
 #pragma unroll 4
       for (int j = 0; j < a.n; ++j) {
-        float f[8], w[8];
+        float f[kConvCh], w[kConvCh];
         fetch(where(t, j, req, pos, first), f);
         coeff(a.taps + (a.n - 1 - j) * a.channels + ch, w);
 #pragma unroll
-        for (int c = 0; c < 8; ++c) s[c] = fmaf(w[c], f[c], s[c]);
+        for (int c = 0; c < kConvCh; ++c) s[c] = fmaf(w[c], f[c], s[c]);
       }
     }
     put(t, s);
@@ -228,10 +241,10 @@ mamba2_finish_warp_kernel(const float* __restrict__ o, const __nv_bfloat16* __re
   for (int i = 0; i < NV; ++i) {
     const float2 z0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zu[i].x));
     const float2 z1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zu[i].y));
-    y[i].x *= z0.x / (1.f + __expf(-z0.x));
-    y[i].y *= z0.y / (1.f + __expf(-z0.y));
-    y[i].z *= z1.x / (1.f + __expf(-z1.x));
-    y[i].w *= z1.y / (1.f + __expf(-z1.y));
+    y[i].x *= silu_bf16(z0.x);
+    y[i].y *= silu_bf16(z0.y);
+    y[i].z *= silu_bf16(z1.x);
+    y[i].w *= silu_bf16(z1.y);
     ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
   }
   const float r = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(part) + eps);
@@ -280,8 +293,8 @@ mamba2_finish_kernel(const float* __restrict__ o, const A* __restrict__ proj, lo
       const uint2 u = *reinterpret_cast<const uint2*>(z + c);
       const float2 z0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
       const float2 z1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-      const float4 y = make_float4(v.x * z0.x / (1.f + __expf(-z0.x)), v.y * z0.y / (1.f + __expf(-z0.y)),
-                                   v.z * z1.x / (1.f + __expf(-z1.x)), v.w * z1.y / (1.f + __expf(-z1.y)));
+      const float4 y = make_float4(v.x * silu_bf16(z0.x), v.y * silu_bf16(z0.y),
+                                   v.z * silu_bf16(z1.x), v.w * silu_bf16(z1.y));
       *reinterpret_cast<float4*>(row + c) = y;
       ss = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, fmaf(y.w, y.w, ss))));
     }
@@ -334,16 +347,17 @@ STK_API int stk_mamba2_conv(const void* proj, long long ldp, int x_off, int dt_o
   if (T <= 0) return 0;
   if (n_taps < 1 || ldo % 8 || ldo < channels || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
   const ConvArgs c{proj, ldp, x_off, dt_off, taps, conv_bias, n_taps, ring, dt_bias, neg_a, channels};
-  const int vec = channels % 8 == 0 && ldp % 8 == 0 && x_off % 8 == 0 &&
+  const int vec = channels % kConvCh == 0 && ldp % kConvCh == 0 && x_off % kConvCh == 0 &&
                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(taps) |
                     reinterpret_cast<uintptr_t>(conv_bias)) & 15) == 0;
   const bool few = T <= 256;                               // one token per thread
   const int tok = few ? 1 : kConvTok;
-  const dim3 grid(static_cast<unsigned>((ldo + 1023) / 1024 + 1), (T + tok - 1) / tok);
+  constexpr int kBlock = kConvThreads * kConvCh;
+  const dim3 grid(static_cast<unsigned>((ldo + kBlock - 1) / kBlock + 1), (T + tok - 1) / tok);
   cudaStream_t st = (cudaStream_t)stream;
 #define STK_CONV(A, N)                                                                                                               \
-  if (few) launch_pdl(mamba2_conv_kernel<A, N, 1>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec); \
-  else launch_pdl(mamba2_conv_kernel<A, N, kConvTok>, grid, dim3(128), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec)
+  if (few) launch_pdl(mamba2_conv_kernel<A, N, 1>, grid, dim3(kConvThreads), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec); \
+  else launch_pdl(mamba2_conv_kernel<A, N, kConvTok>, grid, dim3(kConvThreads), 0, st, c, positions, tok_req, first_pos, (A*)out, ldo, steps, heads, T, vec)
   if (fp32) {
     STK_CONV(float, 0);
   } else {

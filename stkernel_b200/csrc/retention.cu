@@ -138,8 +138,8 @@ rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bf
 }
 
 // out[t, col + h * V + c] = o / rms(o over the head) * silu(g) * scale: one warp per (token, head).  Zeros into the columns left .. col
-// and behind the last head.
-template <typename A>
+// and behind the last head.  NV > 0: bf16 heads of at most 128 * NV columns in whole groups of four, which stay in registers.
+template <typename A, int NV>
 __global__ void __launch_bounds__(256)
 retention_finish_kernel(const float* __restrict__ o, float eps, const int* __restrict__ tok_req, const int64_t* __restrict__ positions,
                         const A* __restrict__ proj, long long ldp, int g_off, float scale, A* __restrict__ out, long long ldo, int left,
@@ -152,6 +152,18 @@ retention_finish_kernel(const float* __restrict__ o, float eps, const int* __res
   const long long t = th / H;
   const int h = static_cast<int>(th - t * H);
   A* to = out + t * ldo;
+  const float* x = o + th * V;
+  const A* g = proj + t * ldp + g_off + h * V;
+  float4 v[NV > 0 ? NV : 1];
+  uint2 gu[NV > 0 ? NV : 1];
+  if (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      v[i] = c < V ? *reinterpret_cast<const float4*>(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      gu[i] = c < V ? *reinterpret_cast<const uint2*>(g + c) : make_uint2(0, 0);
+    }
+  }
   if (h == 0)
     for (int c = left + lane; c < col; c += 32) st_act(to + c, 0.f);
   if (h == H - 1)
@@ -161,25 +173,20 @@ retention_finish_kernel(const float* __restrict__ o, float eps, const int* __res
     for (int c = lane; c < V; c += 32) st_act(to + c, 0.f);
     return;
   }
-  const float* x = o + th * V;
-  const A* g = proj + t * ldp + g_off + h * V;
   float ss = 0.f;
-  if (sizeof(A) == 2 && ((V | ldp | ldo | g_off | col) & 3) == 0) {
-    for (int c = lane * 4; c < V; c += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(x + c);
-      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
-    }
+  if (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
     const float r = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
-    for (int c = lane * 4; c < V; c += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(x + c);
-      const uint2 gu = *reinterpret_cast<const uint2*>(g + c);
-      const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu.x));
-      const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu.y));
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      if (c >= V) continue;
+      const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu[i].x));
+      const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu[i].y));
       uint2 pk;
-      *reinterpret_cast<__nv_bfloat162*>(&pk.x) =
-          __floats2bfloat162_rn(v.x * r * g0.x / (1.f + __expf(-g0.x)), v.y * r * g0.y / (1.f + __expf(-g0.y)));
-      *reinterpret_cast<__nv_bfloat162*>(&pk.y) =
-          __floats2bfloat162_rn(v.z * r * g1.x / (1.f + __expf(-g1.x)), v.w * r * g1.y / (1.f + __expf(-g1.y)));
+      *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(v[i].x * r * silu_bf16(g0.x), v[i].y * r * silu_bf16(g0.y));
+      *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(v[i].z * r * silu_bf16(g1.x), v[i].w * r * silu_bf16(g1.y));
       *reinterpret_cast<uint2*>(to + c) = pk;
     }
     return;
@@ -228,11 +235,16 @@ STK_API int stk_retention_finish(const float* o, float eps, const int* tok_req, 
   if (T <= 0) return 0;
   const dim3 grid(static_cast<unsigned>((static_cast<long long>(T) * heads + 7) / 8));
   cudaStream_t st = (cudaStream_t)stream;
-  if (fp32)
-    launch_pdl(retention_finish_kernel<float>, grid, dim3(256), 0, st, o, eps, tok_req, positions, (const float*)proj, ldp, g_off, scale,
-               (float*)out, ldo, left, col, cols, heads, vdim, T);
-  else
-    launch_pdl(retention_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, eps, tok_req, positions, (const __nv_bfloat16*)proj, ldp,
-               g_off, scale, (__nv_bfloat16*)out, ldo, left, col, cols, heads, vdim, T);
+  const bool vec = !fp32 && vdim <= 512 && ((vdim | g_off | col) & 3) == 0 && ((ldp | ldo) & 3) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(out)) & 7) == 0;
+#define STK_FINISH(A, NV)                                                                                                          \
+  launch_pdl(retention_finish_kernel<A, NV>, grid, dim3(256), 0, st, o, eps, tok_req, positions, (const A*)proj, ldp, g_off, scale, (A*)out, \
+             ldo, left, col, cols, heads, vdim, T)
+  if (fp32) STK_FINISH(float, 0);
+  else if (!vec) STK_FINISH(__nv_bfloat16, 0);
+  else if (vdim <= 128) STK_FINISH(__nv_bfloat16, 1);
+  else if (vdim <= 256) STK_FINISH(__nv_bfloat16, 2);
+  else STK_FINISH(__nv_bfloat16, 4);
+#undef STK_FINISH
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
