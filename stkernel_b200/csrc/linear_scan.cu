@@ -38,7 +38,14 @@ __host__ __device__ inline long long linear_slot_floats(int D, int V) {
 }
 
 // Tokens 2 * lane and 2 * lane + 1 of a chunk of n: running sums of the log decays (F) and input weights (w, 0 behind the chunk).
-struct ChunkGates { float F0, F1, w0, w1, end; };
+// One token may decay by thousands and the next ones by thousandths, so sums are formed in fp64 and kept as integer part (x) and
+// remainder (y): differences lose nothing.
+struct ChunkGates { float2 F0, F1, end; float w0, w1; };
+__device__ __forceinline__ float2 int_and_rest(double v) {
+  const double i = rint(v);
+  return make_float2(static_cast<float>(i), static_cast<float>(v - i));
+}
+__device__ __forceinline__ float decay_between(float2 later, float2 earlier) { return expf((later.x - earlier.x) + (later.y - earlier.y)); }
 struct ChunkRaw { float g0, g1, w0, w1; };
 
 __device__ __forceinline__ ChunkRaw load_gates(const ChunkArgs& a, int h, long long t0, int n, int lane) {
@@ -54,22 +61,27 @@ __device__ __forceinline__ ChunkRaw load_gates(const ChunkArgs& a, int h, long l
 }
 __device__ __forceinline__ ChunkGates chunk_gates(const ChunkArgs& a, const ChunkRaw& r, int n, int lane) {
   ChunkGates c;
+  double F0, F1, end;
   if (a.fixed != nullptr) {
-    c.F0 = r.g0 * static_cast<float>(2 * lane + 1);
-    c.F1 = r.g0 * static_cast<float>(2 * lane + 2);
-    c.end = r.g0 * static_cast<float>(n);
+    const double g = r.g0;
+    F0 = g * (2 * lane + 1);
+    F1 = g * (2 * lane + 2);
+    end = g * n;
   } else {
-    const float pair = r.g0 + r.g1;
-    float inc = pair;
+    const double pair = static_cast<double>(r.g0) + r.g1;
+    double inc = pair;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float up = __shfl_up_sync(0xffffffffu, inc, o);
+      const double up = __shfl_up_sync(0xffffffffu, inc, o);
       if (lane >= o) inc += up;
     }
-    c.F0 = inc - r.g1;
-    c.F1 = inc;
-    c.end = __shfl_sync(0xffffffffu, inc, 31);                          // absent tokens add nothing
+    F0 = inc - r.g1;
+    F1 = inc;
+    end = __shfl_sync(0xffffffffu, inc, 31);                             // absent tokens add nothing
   }
+  c.F0 = int_and_rest(F0);
+  c.F1 = int_and_rest(F1);
+  c.end = int_and_rest(end);
   c.w0 = 2 * lane < n ? r.w0 : 0.f;
   c.w1 = 2 * lane + 1 < n ? r.w1 : 0.f;
   return c;
@@ -125,7 +137,8 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
   for (int c = 0; c < nc; ++c) {
     const int n = min(kChunk, span - c * kChunk);
     const ChunkGates g = chunk_gates(a, raw, n, lane);
-    const float w0 = g.w0 * expf(g.end - g.F0), w1 = g.w1 * expf(g.end - g.F1), fs = expf(g.end);   // of tokens 2 lane, 2 lane + 1
+    const float w0 = g.w0 * decay_between(g.end, g.F0), w1 = g.w1 * decay_between(g.end, g.F1);      // of tokens 2 lane, 2 lane + 1
+    const float fs = expf(g.end.x + g.end.y);
     mls_wait<1>();
     __syncthreads();                                                    // chunk c is in, the stage before it is free
     if (c + 2 < nc) load(c + 2);
@@ -207,7 +220,8 @@ template <bool kPair, int COLS>
 __global__ void __launch_bounds__(COLS * 2)
 linear_chunk_out_kernel(const ChunkArgs a, int min_span, const float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  __shared__ float s_F[kChunk], s_w[kChunk], s_in[kChunk];
+  __shared__ float2 s_F[kChunk];
+  __shared__ float s_w[kChunk], s_in[kChunk];
   __shared__ ChunkRef s_c;
   __shared__ int s_ok;
   constexpr int kVs = COLS + 8, kParts = kPair ? 2 : 1, kThreads = COLS * 2, kWarps = COLS / 16, kMine = (10 + kWarps - 1) / kWarps;
@@ -259,8 +273,8 @@ linear_chunk_out_kernel(const ChunkArgs a, int min_span, const float* __restrict
     s_F[2 * lane + 1] = g.F1;
     s_w[2 * lane] = g.w0;
     s_w[2 * lane + 1] = g.w1;
-    s_in[2 * lane] = expf(g.F0);
-    s_in[2 * lane + 1] = expf(g.F1);
+    s_in[2 * lane] = expf(g.F0.x + g.F0.y);
+    s_in[2 * lane + 1] = expf(g.F1.x + g.F1.y);
   }
   mls_wait<0>();
   __syncthreads();
@@ -302,7 +316,7 @@ linear_chunk_out_kernel(const ChunkArgs a, int min_span, const float* __restrict
         const int t = rb * 16 + (lane >> 2) + r * 8, col = kb * 16 + j * 8 + (lane & 3) * 2;
         float p[2];
 #pragma unroll
-        for (int i = 0; i < 2; ++i) p[i] = col + i <= t ? x[j][2 * r + i] * (s_w[col + i] * expf(s_F[t] - s_F[col + i])) : 0.f;
+        for (int i = 0; i < 2; ++i) p[i] = col + i <= t ? x[j][2 * r + i] * (s_w[col + i] * decay_between(s_F[t], s_F[col + i])) : 0.f;
         mls_split2(p[0], p[1], wh[m][2 * j + r], wl[m][2 * j + r]);
       }
   }

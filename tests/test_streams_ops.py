@@ -229,8 +229,9 @@ def run_plan(plan, data, refs, state, call, width, tol, dev, dt):
         call(p, meta, state, out)
         for r in range(2):
             got = out[:sizes[0]] if r == 0 else out[sizes[0]:]
-            e = worst_row(got[:, :width], refs[r][at[r]:at[r] + sizes[r]])
-            assert e < tol, (plan[:4], sizes, r, e)
+            ref = refs[r][at[r]:at[r] + sizes[r]]
+            e = worst_row(got[:, :width], ref)
+            assert e < tol and (sizes[r] == 1 or rel(got[:, :width], ref) < tol / 3), (plan[:4], sizes, r, e)
             at[r] += sizes[r]
         assert not out[:, width:].any()
     for s in state:
@@ -263,7 +264,7 @@ def test_retention(where, c):
     for plan in plans(dev):
         state = (torch.full((3, H, D, V), float("nan"), device=dev),)
         run_plan(plan, data, refs, state, lambda p, meta, st, out: RC.retention(p, *offs, a, meta, st, out, 0), H * V,
-                 5e-5 if dt == F32 else 1e-2, dev, dt)
+                 1e-4 if dt == F32 else 2e-2, dev, dt)
 
 
 SSM = [dict(H=4, V=24, N=16, G=2, taps=4, NG=2), dict(H=2, V=5, N=9, G=1, taps=3, NG=1), dict(H=3, V=64, N=64, G=3, taps=2, NG=1),
@@ -289,10 +290,16 @@ def test_mamba2(where, c):
     H, V, N, G, n = c["H"], c["V"], c["N"], c["G"], 170
     inner = H * V
     a, w = ssm_params(c, dev)
+    w["a"][0] = 6.0                                           # one head whose decays differ by thousands
+    a.neg_a[0] = -float(torch.exp(w["a"][0]))
+    w["dt"][0] = -9.0
+    a.dt_bias[0] = -9.0
     m = {"heads": H, "groups": G, "norm_groups": c["NG"]}
     data, refs = [], []
     for r in range(2):
         z, x, t = rand(n, inner, seed=90 + r), rand(n, inner + 2 * G * N, seed=94 + r), rand(n, H, seed=98 + r)
+        t[11::37] += 30.0                                     # all but forgets what was before; its neighbours decay slowly
+        t = t.to(BF16).double()
         p, offs = columns((z, x, t), dt)
         y = O.silu(O.causal_conv(x, w["conv"], w["bias"])).split([inner, G * N, G * N], -1)
         y = O.mamba2_heads(y[0].reshape(n, H, V), y[1].reshape(n, G, N), y[2].reshape(n, G, N), O.softplus(t + w["dt"]), w["a"], w["d"], m)
@@ -302,7 +309,7 @@ def test_mamba2(where, c):
         nan = lambda *s, d=F32: torch.full((3,) + s, float("nan"), dtype=d, device=dev)
         state = (nan(H, N, V), nan(c["taps"] - 1, inner + 2 * G * N, d=dt))
         run_plan(plan, data, refs, state, lambda p, meta, st, out: RC.mamba2(p, *offs, a, meta, st, out), inner,
-                 5e-5 if dt == F32 else 3e-2, dev, dt)
+                 1e-4 if dt == F32 else 0.1, dev, dt)
 
 
 @WHERE
