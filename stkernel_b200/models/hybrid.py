@@ -58,11 +58,9 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
         if l.weights_of is not None:
             continue
         m, p = l.mixer, f"l{i}"
-        streams = cfg.block == "streams"
-        for q in (1, 2) if l.mlp is not None else (1,):
-            if q == 1 or cfg.block != "parallel":
-                out[f"{p}.norm{q}"] = ((W,), "bf16")
-            if streams:
+        out[f"{p}.norm1"] = ((W,), "bf16")
+        if cfg.block == "streams":
+            for q in (1, 2) if l.mlp is not None else (1,):
                 out[f"{p}.norm{q}.b"] = ((W,), "bf16")
                 out[f"{p}.hc{q}.in"] = ((cfg.streams,), "bf16")
                 out[f"{p}.hc{q}.out"] = ((cfg.streams,), "bf16")
@@ -97,6 +95,8 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
         if m.kind != "parallel":
             out[f"{p}.mix.o"] = ((W, m.out_dim), "bf16")
         if l.mlp is not None:
+            if cfg.block != "parallel":
+                out[f"{p}.norm2"] = ((W,), "bf16")
             if l.mlp.kind == "dense":
                 out[f"{p}.mlp.gate"] = ((l.mlp.ff, W), "bf16")
                 out[f"{p}.mlp.up"] = ((l.mlp.ff, W), "bf16")

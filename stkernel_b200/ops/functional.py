@@ -193,7 +193,7 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
             _lib.call("stk_skinny_linear_fused", lw.w, lw.w.stride(0), 1 if lw.is_fp8 else 0, lw.scale,
                       lw.scale.stride(0) if lw.is_fp8 else 0, x, x.stride(0), o, o.stride(0) if o is not None else 0, t0, n0, k0,
                       0, _lib.sm_count(), norm[0] if norm is not None else None, float(norm[1]) if norm is not None else 0.0,
-                      ll.ctx if ll is not None else None, 0, None, None, None, None, 0, None, None, 0, 0, 0, 0.0,
+                      ll.ctx if ll is not None else None, 0, None, None, None, None, 0, None, None, 0, 0, 0, 0, 0.0,
                       _lib.status_buffer(), _lib.stream())
             return LLPending(ll, t0, n0, x.device) if ll is not None else o
     if norm is not None:

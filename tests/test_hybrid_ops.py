@@ -246,7 +246,7 @@ def test_attention_kernels_agree_over_many_pages(c, cap, sink):
     HB.window_attention(proj, 0, ko, a, meta, table, cache, out)
     ref = torch.empty_like(out)
     _lib.call("stk_window_attention_simt", proj, proj.stride(0), 0, ko, meta.positions, meta.tok_req, table, table.stride(0), cache,
-              cache.shape[3], freq, R, 1.1, H, G, D, win, D ** -0.5, cap, sk, ref, ref.stride(0), 0, n, _lib.stream())
+              cache.shape[3], freq, R, 1.1, H, G, D, R, D, D, None, 0, 1.0, win, D ** -0.5, cap, sk, ref, ref.stride(0), 0, n, _lib.stream())
     x, y = out[:, :H * D].float(), ref[:, :H * D].float()
     assert torch.isfinite(x).all()
     err = ((x - y).view(n, H, D).norm(dim=-1) / y.view(n, H, D).norm(dim=-1).clamp(min=1e-3)).amax(1)
