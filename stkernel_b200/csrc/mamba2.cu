@@ -44,13 +44,13 @@ struct Mamba2Front {
   }
 };
 
-constexpr int kConvTok = 32, kConvBatch = 8, kConvCh = 4, kConvThreads = 256;
+constexpr int kConvTok = 32, kConvBatch = 4, kConvCh = 4, kConvThreads = 256;
 
 // Four channels x TOK tokens per thread.  NT > 0 taps: the inputs of tokens that follow one another in one span slide through
 // registers, a batch of kConvBatch in flight while the one before is summed; otherwise (spans that meet inside the group, many
 // taps, unaligned rows) every tap is read where it is used.  The grid's last column of blocks forms the step sizes.
 template <typename A, int NT, int TOK>
-__global__ void __launch_bounds__(kConvThreads)
+__global__ void __launch_bounds__(kConvThreads, TOK > 1 && NT > 0 ? 4 : 1)
 mamba2_conv_kernel(const ConvArgs a, const int64_t* __restrict__ positions, const int* __restrict__ tok_req,
                    const int* __restrict__ first_pos, A* __restrict__ out, long long ldo, float* __restrict__ steps, int H, int T,
                    int vec) {
