@@ -239,12 +239,18 @@ class YarnScaling:
 
 
 @dataclass(frozen=True)
+class LinearScaling:
+    """Linear context extension of a rotary embedding: every frequency is divided by `factor`."""
+    factor: float
+
+
+@dataclass(frozen=True)
 class RotaryConfig:
     """Rotation of the first `dims` dimensions of a head: dimension i paired with i + dims/2, or with its neighbour
     (2i with 2i + 1) when `interleaved`."""
     base: float
     dims: int
-    scaling: Optional[YarnScaling] = None
+    scaling: Optional[Union[YarnScaling, LinearScaling]] = None
     interleaved: bool = False
 
     def frequencies(self) -> Tuple[List[float], float]:
@@ -254,6 +260,8 @@ class RotaryConfig:
         s = self.scaling
         if s is None:
             return f, 1.0
+        if isinstance(s, LinearScaling):
+            return [x / s.factor for x in f], 1.0
         at = lambda turns: d * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
         lo = max(math.floor(at(s.fast)), 0)
         hi = min(math.ceil(at(s.slow)), d - 1)
@@ -360,6 +368,56 @@ class GroupedAttentionMixer:
 
 
 @dataclass(frozen=True)
+class TalkingAttentionMixer:
+    """Grouped-query attention whose heads' scaled scores are mixed by a matrix [heads, heads] before the softmax.
+
+    chunk: a position sees the earlier positions of its own chunk only (chunks of that many positions, counted from position 0; None:
+    the full context); bias: q, k and v projections have biases; qk_norm: queries and keys are RMS-normed per head, with a weight that
+    the heads share, before their rotation; sink: one score without key and value per head, learned; gate: every head's output is
+    multiplied with the sigmoid of one number that is projected from the same input."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: Optional[int] = None
+    rotary: Optional[RotaryConfig] = None
+    bias: bool = True
+    qk_norm: bool = True
+    sink: bool = True
+    gate: bool = True
+    kind = "talking_attention"
+
+    @property
+    def window(self) -> int:
+        return FULL_CONTEXT if self.chunk is None else self.chunk
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class TimeMixMixer:
+    """Linear attention with a decay per head and key channel that the token chooses, S <- diag(w) S + k v^T, read out before the update
+    with a bonus u for the current token, o = (S + diag(u) k v^T)^T r.  Every projection reads a blend of its own between the token's
+    input and the previous token's; log w = -exp(W2 tanh(W1 x) + w0), W1 with `rank` rows (None: as many as the checkpoint has).  A
+    head's read-out is divided by its root mean square, weighted, and multiplied with silu of a gate."""
+    heads: int
+    dim: int
+    rank: Optional[int] = None
+    kind = "time_mix"
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.dim
+
+
+@dataclass(frozen=True)
 class RetentionMixer:
     """Linear attention with a fixed decay per head: S <- decay S + k v^T, read with the query; queries and keys are rotated,
     every head's read-out is divided by its root mean square and multiplied with silu of a gate."""
@@ -399,11 +457,12 @@ class Mamba2Mixer:
 @dataclass(frozen=True)
 class ParallelMixer:
     """Two mixers over the same input: left_scale * left + right_scale * right.  At most one of them keeps a cache and at most
-    one a recurrent state."""
-    left: GroupedAttentionMixer
-    right: RetentionMixer
+    one a recurrent state.  out_norm: each side's output is RMS-normed over the model width first, with a weight of its own."""
+    left: Union[GroupedAttentionMixer, TalkingAttentionMixer]
+    right: Union[RetentionMixer, TimeMixMixer]
     left_scale: float = 1.0
     right_scale: float = 1.0
+    out_norm: bool = False
     kind = "parallel"
 
     @property
@@ -413,24 +472,41 @@ class ParallelMixer:
 
 @dataclass(frozen=True)
 class DenseMlp:
-    """W_down(act(W_gate h) * W_up h)."""
+    """W_down(act(W_gate h) * W_up h), or W_down act(W_up h) for an activation without a gate.  "xielu" has two learned numbers (a, b):
+    softplus(a) z^2 + z / 2 for z > 0, (softplus(b) + 1/2) (exp(z) - 1 - z) + z / 2 otherwise."""
     ff: int
-    act: str = "silu"                     # "silu" | "relu"
+    act: str = "silu"                     # "silu" | "relu" (gated), "xielu" (no gate)
     kind = "dense"
+
+    @property
+    def gated(self) -> bool:
+        return self.act != "xielu"
 
 
 @dataclass(frozen=True)
 class MoeMlp:
     """`top` of `experts` feed-forward layers W_down act(W_up h) per token, chosen by the largest router logits (bias included)
     and weighted by the softmax over the chosen logits (which is the softmax over all of them, renormalised); a shared expert of
-    the same form, if there is one, is added for every token."""
+    the same form, if there is one, is added for every token.
+
+    act "silu" has a gate: W_down (silu(W_gate h) * W_up h).  scoring "sigmoid": experts are chosen by the sigmoid of their logit plus a
+    correction (with groups > 1 only experts of the `keep` best of that many equal groups of neighbours, a group's score being the
+    sum of its two largest), and weighted by the sigmoid alone, renormalised over the chosen, times `scale`."""
     experts: int
     top: int
     ff: int
-    act: str = "relu2"                    # "relu2" (relu squared) | "gelu" (exact)
+    act: str = "relu2"                    # "relu2" (relu squared) | "gelu" (exact) | "silu" (gated)
     router_bias: bool = True
     shared_ff: int = 0                    # 0: no shared expert
+    scoring: str = "softmax_topk"         # "softmax_topk" | "sigmoid"
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
     kind = "moe"
+
+    @property
+    def gated(self) -> bool:
+        return self.act == "silu"
 
     @property
     def shared_parts(self) -> int:
@@ -443,11 +519,12 @@ class MoeMlp:
         return self.ff if not self.shared_ff else max(self.ff, -(-self.shared_ff // self.shared_parts))
 
 
-Mixer = Union[AttentionMixer, MlstmMixer, LatentAttentionMixer, GroupedAttentionMixer, RetentionMixer, Mamba2Mixer, ParallelMixer]
+Mixer = Union[AttentionMixer, MlstmMixer, LatentAttentionMixer, GroupedAttentionMixer, TalkingAttentionMixer, RetentionMixer,
+              TimeMixMixer, Mamba2Mixer, ParallelMixer]
 Mlp = Union[DenseMlp, MoeMlp]
 
-ATTENTION_KINDS = ("attention", "latent_attention", "grouped_attention")
-RECURRENT_KINDS = ("mlstm", "retention", "mamba2")
+ATTENTION_KINDS = ("attention", "latent_attention", "grouped_attention", "talking_attention")
+RECURRENT_KINDS = ("mlstm", "retention", "mamba2", "time_mix")
 
 
 def mixer_parts(m: Mixer) -> Tuple[Mixer, ...]:
@@ -473,6 +550,15 @@ class HybridLayer:
 
 
 @dataclass(frozen=True)
+class BigramTable:
+    """A second embedding, of the token and the one before it: row (previous * mul_prev + token * mul_cur) mod buckets; a sequence's
+    first token takes row `buckets`, the table's last."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
 class HybridConfig:
     """A decoder given as a list of layers, each with its own mixer (attention or recurrence) and optional feed-forward.
 
@@ -481,7 +567,9 @@ class HybridConfig:
                        they are added to it;
     block "streams":   several residual streams; a sublayer reads the layer norm (with bias) of a weighted sum of them, and every
                        stream becomes a weighted sum of all of them plus a multiple of the sublayer's output.  The model's
-                       output is the sum of the streams."""
+                       output is the sum of the streams;
+    block "shifted":   both sublayers read one RMS norm's output and are added to the fp32 residual together; what the mixer reads
+                       is blended, element by element, with the previous token's norm output (token shift)."""
     vocab_size: int
     hidden_size: int
     layers: Tuple[HybridLayer, ...]
@@ -490,10 +578,11 @@ class HybridConfig:
     dtype: str = "bfloat16"               # "bfloat16": projections and activations; "float32": everything
     max_position_embeddings: int = 1 << 30
     architecture: str = "Timalorn"
-    block: str = "parallel"               # "parallel" | "post_norm" | "streams"
+    block: str = "parallel"               # "parallel" | "post_norm" | "streams" | "shifted"
     streams: int = 1                      # residual streams ("streams" blocks)
     tied_head: bool = False               # logits are read with the embedding table
     logit_scale: float = 1.0
+    bigram: Optional[BigramTable] = None  # added to the embedding ("shifted" blocks)
     family = "hybrid"
     # fields of the other family that family-neutral code asks for
     n_mtp_layers = 0
@@ -526,7 +615,8 @@ class HybridConfig:
     def mechanisms(self) -> Tuple[str, ...]:
         """Kinds of mixers and feed-forwards in this model, which decide what kernels it needs."""
         return tuple(sorted({p.kind for l in self.layers for p in mixer_parts(l.mixer)}
-                            | {l.mlp.kind for l in self.layers if l.mlp is not None}))
+                            | {l.mlp.kind for l in self.layers if l.mlp is not None}
+                            | ({"token_shift"} if self.block == "shifted" else set())))
 
     def validate(self) -> None:
         def positive(name: str, v: Any, integer: bool = True) -> None:
@@ -550,8 +640,16 @@ class HybridConfig:
             raise ConfigError(f"unknown dtype {self.dtype!r}")
         if not self.layers:
             raise ConfigError("layers must not be empty")
-        if self.block not in ("parallel", "post_norm", "streams"):
+        if self.block not in ("parallel", "post_norm", "streams", "shifted"):
             raise ConfigError(f"unknown block {self.block!r}")
+        if self.bigram is not None:
+            if self.block != "shifted":
+                raise ConfigError("a bigram embedding is available in shifted blocks")
+            positive("embedding.bigram.buckets", self.bigram.buckets)
+            for f in ("mul_prev", "mul_cur"):
+                v = getattr(self.bigram, f)
+                if not isinstance(v, int) or isinstance(v, bool) or not 0 <= v < 1 << 31:
+                    raise ConfigError(f"embedding.bigram.{f}: {v!r} must be an integer from 0 to 2^31 - 1")
 
         def rotary(at: str, r: RotaryConfig, dim: int, of: str) -> None:
             positive(f"{at}.rot.base", r.base, False)
@@ -559,8 +657,8 @@ class HybridConfig:
             if r.dims % 2 or r.dims > dim:
                 raise ConfigError(f"{at}.rot.dims must be even and at most {of}")
             if r.scaling is not None:
-                for f in ("factor", "original", "fast", "slow"):
-                    positive(f"{at}.rot.scaling.{f}", getattr(r.scaling, f), False)
+                for f in dataclasses.fields(r.scaling):
+                    positive(f"{at}.rot.scaling.{f.name}", getattr(r.scaling, f.name), False)
 
         def mixer(at: str, i: int, m: Mixer) -> None:
             """at: name of the mixer's section."""
@@ -610,6 +708,20 @@ class HybridConfig:
                 if m.q_temp is not None:
                     number(f"{at}.q_temp.coef", m.q_temp.coef)
                     positive(f"{at}.q_temp.every", m.q_temp.every, False)
+            elif m.kind == "talking_attention":
+                positive(f"{at}.kv_heads", m.kv_heads)
+                positive(f"{at}.vdim", m.vdim)
+                if m.chunk is not None:
+                    positive(f"{at}.mask.size", m.chunk)
+                if m.vdim > 1024:
+                    raise ConfigError(f"{at}.vdim: at most 1024")
+                if m.heads % m.kv_heads:
+                    raise ConfigError(f"{at}: kv_heads must divide heads")
+                if m.rotary is not None:
+                    rotary(at, m.rotary, m.dim, "dim")
+            elif m.kind == "time_mix":
+                if m.rank is not None:
+                    positive(f"{at}.rank", m.rank)
             elif m.kind == "retention":
                 positive(f"{at}.vdim", m.vdim)
                 if not isinstance(m.decay, tuple) or len(m.decay) != m.heads:
@@ -638,25 +750,44 @@ class HybridConfig:
             if m.kind == "parallel":
                 number(f"{at}.mixer.left_scale", m.left_scale)
                 number(f"{at}.mixer.right_scale", m.right_scale)
-                if m.left.kind != "grouped_attention" or m.right.kind != "retention":
-                    raise ConfigError(f"{at}.mixer: grouped attention beside retention is what this build combines")
+                sides = (m.left.kind, m.right.kind)
+                if sides == ("talking_attention", "time_mix"):
+                    if self.block != "shifted" or not m.out_norm:
+                        raise ConfigError(f"{at}.mixer: talking attention beside time mixing needs shifted blocks and norms on the outputs")
+                elif sides != ("grouped_attention", "retention"):
+                    raise ConfigError(f"{at}.mixer: this build combines grouped attention with retention, and talking attention with "
+                                      "time mixing")
+                elif m.out_norm or self.block == "shifted":
+                    raise ConfigError(f"{at}.mixer: grouped attention beside retention has no norms on its outputs and no token shift")
                 mixer(f"{at}.mixer.left", i, m.left)
                 mixer(f"{at}.mixer.right", i, m.right)
             else:
-                if m.kind in ("grouped_attention", "retention"):
+                if m.kind in ("grouped_attention", "retention", "talking_attention", "time_mix"):
                     raise ConfigError(f"{at}.type: {m.kind} is one side of a parallel mixer")
                 mixer(f"{at}.mixer", i, m)
             if l.mlp is not None:
                 positive(f"{at}.mlp.ff", l.mlp.ff)
                 if l.mlp.kind == "dense":
-                    if l.mlp.act not in ("silu", "relu"):
+                    if l.mlp.act not in ("silu", "relu", "xielu") or (l.mlp.act == "xielu" and self.block == "parallel"):
                         raise ConfigError(f"{at}.mlp.act: unknown activation {l.mlp.act!r}")
                 else:
                     p = l.mlp
                     positive(f"{at}.mlp.router.experts", p.experts)
                     positive(f"{at}.mlp.router.top", p.top)
-                    if p.act not in ("relu2", "gelu"):
+                    if p.act not in ("relu2", "gelu", "silu"):
                         raise ConfigError(f"{at}.mlp.act: unknown activation {p.act!r}")
+                    if p.scoring not in ("softmax_topk", "sigmoid"):
+                        raise ConfigError(f"{at}.mlp.router: unknown scoring {p.scoring!r}")
+                    number(f"{at}.mlp.router.scale", p.scale)
+                    positive(f"{at}.mlp.router.groups.count", p.groups)
+                    positive(f"{at}.mlp.router.groups.keep", p.keep)
+                    if p.groups > 1 and (p.scoring != "sigmoid" or p.groups > 32 or p.experts % p.groups
+                                         or p.experts // p.groups < 2):
+                        raise ConfigError(f"{at}.mlp.router.groups: at most 32 equal groups of two experts or more, with sigmoid scores")
+                    if p.keep > p.groups or p.experts // p.groups * p.keep < p.top:
+                        raise ConfigError(f"{at}.mlp.router.groups.keep: at most count, and enough for `top` experts")
+                    if p.shared_ff and (p.gated or p.scoring != "softmax_topk"):
+                        raise ConfigError(f"{at}.mlp.shared: not available with gated experts or sigmoid scores")
                     if p.shared_ff != 0:
                         positive(f"{at}.mlp.shared.ff", p.shared_ff)
                     most = 31 if p.shared_ff else 32
@@ -880,6 +1011,72 @@ def fanulix_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
             "layers": layers, "norm": {"eps": cfg.norm_eps}, "logit_scale": cfg.logit_scale}
 
 
+def fogizen_config_from_json(d: Mapping[str, Any], dtype: str = "bfloat16") -> HybridConfig:
+    """The `config.json` of a Fogizen model: shifted blocks of talking-heads attention beside time mixing, with a dense feed-forward, a
+    mixture of experts or none, over token and bigram embeddings."""
+    _check_model_keys(d)
+    layers: List[HybridLayer] = []
+    for i, l in enumerate(d["layers"]):
+        at = f"layers[{i}]"
+        l = _take(l, at, ("type", "mixer"), ("mlp",))
+        if l["type"] != "parallel":
+            raise ConfigError(f"{at}.type: unknown mixer {l['type']!r}")
+        m = _take(l["mixer"], f"{at}.mixer", ("left", "right"))
+        a = _take(m["left"], f"{at}.mixer.left", ("heads", "kv_heads", "dim", "vdim", "scale", "mask", "rot"))
+        chunk = _take(a.pop("mask"), f"{at}.mixer.left.mask", ("size",))["size"]
+        if chunk is None:
+            raise ConfigError(f"{at}.mixer.left.mask.size: None must be a positive integer")
+        r = _take(a.pop("rot"), f"{at}.mixer.left.rot", ("base", "dims"), ("scaling",))
+        sc = r.get("scaling")
+        if sc is not None:
+            sc = LinearScaling(**_take(sc, f"{at}.mixer.left.rot.scaling", ("factor",)))
+        left = TalkingAttentionMixer(**a, chunk=chunk, rotary=RotaryConfig(r["base"], r["dims"], sc, interleaved=True))
+        right = TimeMixMixer(**_take(m["right"], f"{at}.mixer.right", ("heads", "dim")))
+        mlp: Optional[Mlp] = None
+        if l.get("mlp") is not None:
+            p = l["mlp"]
+            kind = p.get("kind") if isinstance(p, Mapping) else None
+            if kind == "dense":
+                mlp = DenseMlp(_take(p, f"{at}.mlp", ("kind", "ff"))["ff"], "xielu")
+            elif kind == "moe":
+                p = _take(p, f"{at}.mlp", ("kind", "expert", "router"))
+                r = _take(p["router"], f"{at}.mlp.router", ("experts", "top", "scale"), ("groups",))
+                g = _take(r["groups"], f"{at}.mlp.router.groups", ("count", "keep")) if r.get("groups") is not None else {"count": 1, "keep": 1}
+                mlp = MoeMlp(r["experts"], r["top"], _take(p["expert"], f"{at}.mlp.expert", ("ff",))["ff"], "silu", False,
+                             scoring="sigmoid", groups=g["count"], keep=g["keep"], scale=r["scale"])
+            else:
+                raise ConfigError(f"{at}.mlp.kind: unknown feed-forward {kind!r}")
+        layers.append(HybridLayer(ParallelMixer(left, right, 0.5, 0.5, True), mlp))
+    e = _take(d["embedding"], "embedding", ("bigram",))
+    cfg = HybridConfig(d["vocab"], d["width"], tuple(layers), _take(d["norm"], "norm", ("eps",))["eps"], 1.0, dtype,
+                       architecture="Fogizen", block="shifted",
+                       bigram=BigramTable(**_take(e["bigram"], "embedding.bigram", ("buckets", "mul_prev", "mul_cur"))))
+    cfg.validate()
+    return cfg
+
+
+def fogizen_config_to_json(cfg: HybridConfig) -> Dict[str, Any]:
+    """The inverse of `fogizen_config_from_json` (the decay's rank is the checkpoint's)."""
+    layers = []
+    for l in cfg.layers:
+        a, r, p = l.mixer.left, l.mixer.right, l.mlp
+        left = {k: getattr(a, k) for k in ("heads", "kv_heads", "dim", "vdim", "scale")}
+        left["mask"] = {"size": a.chunk}
+        left["rot"] = {"base": a.rotary.base, "dims": a.rotary.dims}
+        if a.rotary.scaling is not None:
+            left["rot"]["scaling"] = dataclasses.asdict(a.rotary.scaling)
+        if p is None:
+            mlp = None
+        elif p.kind == "dense":
+            mlp = {"kind": "dense", "ff": p.ff}
+        else:
+            mlp = {"kind": "moe", "expert": {"ff": p.ff}, "router": {"experts": p.experts, "top": p.top, "scale": p.scale,
+                                                                     "groups": {"count": p.groups, "keep": p.keep}}}
+        layers.append({"type": "parallel", "mixer": {"left": left, "right": {"heads": r.heads, "dim": r.dim}}, "mlp": mlp})
+    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "layers": layers,
+            "norm": {"eps": cfg.norm_eps}, "embedding": {"bigram": dataclasses.asdict(cfg.bigram)}}
+
+
 def _mixer_from_dict(d: Mapping[str, Any]) -> Mixer:
     m = dict(d)
     if "left" in m:
@@ -888,9 +1085,15 @@ def _mixer_from_dict(d: Mapping[str, Any]) -> Mixer:
     if r is not None:
         r = dict(r)
         sc = r.pop("scaling", None)
-        r = RotaryConfig(**r, scaling=YarnScaling(**sc) if sc is not None else None)
+        if sc is not None:
+            sc = YarnScaling(**sc) if "original" in sc else LinearScaling(**sc)
+        r = RotaryConfig(**r, scaling=sc)
     if "q_temp" in m:
         return GroupedAttentionMixer(**{**m, "q_temp": QueryTemperature(**m["q_temp"]) if m["q_temp"] is not None else None})
+    if "chunk" in m:
+        return TalkingAttentionMixer(**m, rotary=r)
+    if "rank" in m:
+        return TimeMixMixer(**m)
     if "decay" in m:
         return RetentionMixer(**{**m, "decay": tuple(m["decay"])}, rotary=r)
     if "state" in m:
@@ -910,6 +1113,8 @@ def hybrid_config_from_dict(d: Mapping[str, Any]) -> HybridConfig:
         p = l.get("mlp")
         mlp: Optional[Mlp] = None if p is None else MoeMlp(**p) if "experts" in p else DenseMlp(**p)
         layers.append(HybridLayer(_mixer_from_dict(l["mixer"]), mlp, l.get("weights_of")))
+    if d.get("bigram") is not None:
+        d["bigram"] = BigramTable(**d["bigram"])
     cfg = HybridConfig(layers=tuple(layers), **d)
     cfg.validate()
     return cfg
@@ -958,6 +1163,34 @@ def streams_stack(n_layers: int, width: int, streams: int, heads: int, kv_heads:
     layers = tuple(HybridLayer(both if i % parallel_every == parallel_every - 1 else ssm, mlp) for i in range(n_layers))
     cfg = HybridConfig(vocab, width, layers, 1e-6, 1.0, dtype, architecture="Fanulix", block="streams", streams=streams, tied_head=True,
                        logit_scale=0.5)
+    cfg.validate()
+    return cfg
+
+
+def shifted_stack(n_layers: int, width: int, heads: int, kv_heads: int, dim: int, vdim: int, chunk: int, mix_heads: int, mix_dim: int,
+                  rank: int, ff: int, experts: int, top: int, groups: int, keep: int, expert_ff: int, vocab: int,
+                  dtype: str = "bfloat16") -> HybridConfig:
+    """A Fogizen-shaped decoder: the first layer's feed-forward is dense, the others' are mixtures of experts (experts 0: all dense)."""
+    both = ParallelMixer(TalkingAttentionMixer(heads, kv_heads, dim, vdim, dim ** -0.5, chunk,
+                                               RotaryConfig(10000.0, dim, LinearScaling(4.0), interleaved=True)),
+                         TimeMixMixer(mix_heads, mix_dim, rank), 0.5, 0.5, True)
+    moe = MoeMlp(experts, top, expert_ff, "silu", False, scoring="sigmoid", groups=groups, keep=keep, scale=1.5) if experts else None
+    layers = tuple(HybridLayer(both, DenseMlp(ff, "xielu") if i == 0 or moe is None else moe) for i in range(n_layers))
+    cfg = HybridConfig(vocab, width, layers, 1e-5, 1.0, dtype, architecture="Fogizen", block="shifted", bigram=BigramTable(vocab - 1, 31, 7))
+    cfg.validate()
+    return cfg
+
+
+def tiny_shifted_config(**over: Any) -> HybridConfig:
+    """CPU-sized Fogizen-shaped decoder: a dense layer, a mixture of experts in groups, and a layer without feed-forward."""
+    both = ParallelMixer(TalkingAttentionMixer(4, 2, 20, 28, 0.21, 24, RotaryConfig(3000.0, 12, LinearScaling(2.5), interleaved=True)),
+                         TimeMixMixer(3, 20, 12), 0.5, 0.5, True)
+    moe = MoeMlp(6, 2, 40, "silu", False, scoring="sigmoid", groups=3, keep=2, scale=1.3)
+    kw: Dict[str, Any] = dict(vocab_size=300, hidden_size=88, norm_eps=2e-5, architecture="Fogizen", block="shifted",
+                              bigram=BigramTable(97, 13, 5),
+                              layers=(HybridLayer(both, DenseMlp(104, "xielu")), HybridLayer(both, moe), HybridLayer(both, None)))
+    kw.update(over)
+    cfg = HybridConfig(**kw)
     cfg.validate()
     return cfg
 

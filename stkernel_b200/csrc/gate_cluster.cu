@@ -157,9 +157,9 @@ STK_API int stk_gate_route_cluster_ok() { return gate_cluster_launchable() ? 1 :
 // 16-byte aligned); the caller then uses the grid-wide path.
 STK_API int stk_gate_route_cluster(const void* W, long long ldw, const void* x, long long ldx, int T, int E, int K,
                                    const float* bias, const int* tid2eid, const int64_t* token_ids, int vocab, int* ids,
-                                   float* weights, int topk, int always, int scoring, int renorm, float scaling, int* status,
+                                   float* weights, int topk, int always, int groups, int keep, int scoring, int renorm, float scaling, int* status,
                                    void* stream) {
-  if (T < 1 || T > kGcMaxT || K % 8 || K > kGcIters * 32 * 8 || E < 1 || E > kGcMaxE || topk < 1 || always < 0 || topk + always > 32) return -1;
+  if (T < 1 || T > kGcMaxT || K % 8 || K > kGcIters * 32 * 8 || E < 1 || E > kGcMaxE || topk < 1 || always < 0 || topk + always > 32 || groups < 1 || groups > 32 || keep < 1) return -1;
   if ((ldw % 8) || (ldx % 8) || (reinterpret_cast<uintptr_t>(W) & 15) || (reinterpret_cast<uintptr_t>(x) & 15)) return -1;
   if ((E + kGcCluster - 1) / kGcCluster > 2 * kGcWarps) return -1;
   if (!gate_cluster_launchable()) return -1;
@@ -169,7 +169,7 @@ STK_API int stk_gate_route_cluster(const void* W, long long ldw, const void* x, 
   a.x = static_cast<const __nv_bfloat16*>(x);
   a.ldx = ldx;
   a.T = T; a.E = E; a.K = K;
-  a.router = RouterArgs{bias, tid2eid, token_ids, vocab, ids, weights, E, topk, always, scoring, renorm, scaling, status};
+  a.router = RouterArgs{bias, tid2eid, token_ids, vocab, ids, weights, E, topk, always, groups, keep, scoring, renorm, scaling, status};
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(kGcCluster);
   cfg.blockDim = dim3(kGcWarps * 32);

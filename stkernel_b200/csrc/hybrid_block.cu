@@ -465,9 +465,49 @@ join_glu_kernel(const A* __restrict__ proj, long long ldp, int go, int uo, int f
   glu_columns(pg, pu, o + o0, base, ff, cols - o0, (ldo & 7) == 0 && (ldp & 7) == 0, relu);
 }
 
+// out[t, c] = xIELU(z[t, c]) = (z > 0 ? a z^2 : b (exp(z) - 1 - z)) + z / 2 for c < ff, zero up to `width`; eight columns per thread.
+template <typename A>
+__global__ void __launch_bounds__(256)
+xielu_kernel(const A* __restrict__ z, long long ldz, int ff, float a, float b, A* __restrict__ out, long long ldo, int width, int T) {
+  pdl_wait();
+  pdl_trigger();
+  const int per = (width + 7) / 8;
+  const long long e = blockIdx.x * 256ll + threadIdx.x, t = e / per;
+  if (t >= T) return;
+  const int c0 = static_cast<int>(e - t * per) * 8;
+  auto f = [&](float x) { return fmaf(x, 0.5f, x > 0.f ? a * x * x : b * (expm1f(x) - x)); };
+  const A* p = z + t * ldz + c0;
+  A* o = out + t * ldo + c0;
+  if (sizeof(A) == 2 && c0 + 8 <= ff && ((ldz | ldo) & 7) == 0) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    uint4 r;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 x = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
+      reinterpret_cast<__nv_bfloat162*>(&r)[j] = __floats2bfloat162_rn(f(x.x), f(x.y));
+    }
+    *reinterpret_cast<uint4*>(o) = r;
+    return;
+  }
+  for (int j = 0; j < 8 && c0 + j < width; ++j) st_act(o + j, c0 + j < ff ? f(ld_act(p + j)) : 0.f);
+}
+
 }  // namespace stk
 
 using namespace stk;
+
+// z and out rows start on 16 bytes.
+STK_API int stk_xielu(const void* z, long long ldz, int ff, float a, float b, void* out, long long ldo, int width, int fp32, int T,
+                      void* stream) {
+  if (T <= 0) return 0;
+  if (width < ff || ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
+  const long long n = static_cast<long long>(T) * ((width + 7) / 8);
+  const dim3 grid(static_cast<unsigned>((n + 255) / 256));
+  cudaStream_t st = (cudaStream_t)stream;
+  if (fp32) launch_pdl(xielu_kernel<float>, grid, dim3(256), 0, st, (const float*)z, ldz, ff, a, b, (float*)out, ldo, width, T);
+  else launch_pdl(xielu_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, ff, a, b, (__nv_bfloat16*)out, ldo, width, T);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
 
 STK_API int stk_embed_scaled(const int64_t* ids, const void* embed, int embed_fp32, float* x, long long ldx, int copies, int T, int W,
                              int vocab, float scale, void* h, long long ldh, int width, int* status, void* stream) {

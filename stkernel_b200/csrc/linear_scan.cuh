@@ -2,7 +2,8 @@
 //
 //   S_t = exp(g_t) S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t  (+ skip v_t)        S [D, V] fp32 per head and request row
 //
-// shared by retention (retention.cu) and Mamba-2 (mamba2.cu).  A span that starts at position 0 starts from a zero state.
+// shared by retention (retention.cu) and Mamba-2 (mamba2.cu), and with a decay per key channel and a bonus for the current token, read out
+// before the update, by time mixing (time_mix.cu).  A span that starts at position 0 starts from a zero state.
 //
 //   linear_scan_kernel     token by token, any size and type: one CTA per (32 or 64 value columns, head, request), the block of the
 //                          state in registers.  A `Front` supplies a token's q and k (in shared memory), v and decay, so that
@@ -24,6 +25,7 @@ constexpr int kScanThreads = 256, kScanRows = 8;
 // Front:
 //   float2 fill(t, pos, h, q, k)   token t at position pos, all threads; returns the decay and what its rounding left over (the same
 //                                  small error at every token would add up over many)
+//   or, kPerChannel: void fill(t, h, q, k, uk, w) with the bonus' keys and the channels' decays as well
 //   float value(t, h, col)         v
 //   float skip(h)                  factor of v in the output
 template <typename Front, int NR, int VEC>
@@ -35,6 +37,8 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
   float* k = q + a.D;                             // [D]
   float* x = k + a.D;                             // [kCols] v
   float* part = x + kCols;                        // [8][kCols]
+  float* uk = part + kScanRows * kCols;           // per channel: [D] bonus' keys, [D] decays
+  float2* w = reinterpret_cast<float2*>(uk + (a.D + 1) / 2 * 2);
   pdl_wait();
   pdl_trigger();
   const int vb = blockIdx.x, h = blockIdx.y, ri = blockIdx.z;
@@ -63,7 +67,9 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
   for (int i = 0; i < span; ++i) {
     const long long t = q0 + i;
     __syncthreads();
-    const float2 decay = f.fill(t, start + i, h, q, k);
+    float2 decay = make_float2(0.f, 0.f);
+    if constexpr (Front::kPerChannel) f.fill(t, h, q, k, uk, w);
+    else decay = f.fill(t, start + i, h, q, k);
     float v[VEC];
 #pragma unroll
     for (int c = 0; c < VEC; ++c) {
@@ -79,6 +85,16 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
       const int d = r + j * kScanRows;
       if (d < a.D) {
         const float kd = k[d], qd = q[d];
+        if constexpr (Front::kPerChannel) {
+          const float ud = uk[d];
+          const float2 wd = w[d];
+#pragma unroll
+          for (int c = 0; c < VEC; ++c) {
+            acc[c] = fmaf(qd, fmaf(ud, v[c], S[j][c]), acc[c]);
+            S[j][c] = fmaf(wd.x, S[j][c], fmaf(wd.y, S[j][c], kd * v[c]));
+          }
+          continue;
+        }
 #pragma unroll
         for (int c = 0; c < VEC; ++c) {
           S[j][c] = fmaf(decay.x, S[j][c], fmaf(decay.y, S[j][c], kd * v[c]));
@@ -114,7 +130,8 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
 template <typename Front, int NR, int VEC>
 static int launch_scan_as(const Front& f, const ScanArgs& a, int min_span, int max_span, cudaStream_t st) {
   constexpr int kCols = 32 * VEC;
-  const size_t smem = static_cast<size_t>(2 * a.D + (1 + kScanRows) * kCols) * sizeof(float);
+  // kCols is even: everything behind q, k starts on 8 bytes when D is rounded up to even
+  const size_t smem = static_cast<size_t>(2 * a.D + (1 + kScanRows) * kCols + (Front::kPerChannel ? 3 * a.D + 2 : 0)) * sizeof(float);
   launch_pdl(linear_scan_kernel<Front, NR, VEC>, dim3((a.V + kCols - 1) / kCols, a.H, a.n_req), dim3(kScanThreads), smem, st, f, a,
              min_span, max_span);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;

@@ -25,6 +25,7 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + lo
 
 template <typename A>
 struct Mamba2Front {
+  static constexpr bool kPerChannel = false;
   const A* xbc; long long ld;                     // [T, ld]: x | B | C, convolved
   const float* steps;                             // [2][H][T]: log decays, step sizes
   int N, V, inner, groups, hpg, H, T;

@@ -25,13 +25,13 @@ namespace stk {
 // One warp per token, E <= 512 (the selection itself lives in router.cuh, shared with the gate projection's epilogue).
 __global__ void router_kernel(const float* __restrict__ logits, long long ldl, const float* __restrict__ bias,
                               const int* __restrict__ tid2eid, const int64_t* __restrict__ token_ids, int vocab,
-                              int* __restrict__ ids, float* __restrict__ weights, int T, int E, int topk, int always, int scoring,
+                              int* __restrict__ ids, float* __restrict__ weights, int T, int E, int topk, int always, int groups, int keep, int scoring,
                               int renorm, float scaling, int* status) {
   pdl_wait();
   pdl_trigger();
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   if (t >= T) return;
-  RouterArgs r{bias, tid2eid, token_ids, vocab, ids, weights, E, topk, always, scoring, renorm, scaling, status};
+  RouterArgs r{bias, tid2eid, token_ids, vocab, ids, weights, E, topk, always, groups, keep, scoring, renorm, scaling, status};
   route_token(r, logits + t * ldl, t, threadIdx.x & 31);
 }
 
@@ -416,12 +416,12 @@ expert_fc2_kernel(const __half* __restrict__ act, ExpertW w2, const int* __restr
 using namespace stk;
 
 STK_API int stk_router(const float* logits, long long ldl, const float* bias, const int* tid2eid,
-                       const int64_t* token_ids, int vocab, int* ids, float* weights, int T, int E, int topk, int always,
+                       const int64_t* token_ids, int vocab, int* ids, float* weights, int T, int E, int topk, int always, int groups, int keep,
                        int scoring, int renorm, float scaling, int* status, void* stream) {
   if (T <= 0) return 0;
-  if (E > 512 || always < 0 || topk + always > 32) return -1;
+  if (E > 512 || always < 0 || topk + always > 32 || groups < 1 || groups > 32 || keep < 1) return -1;
   launch_pdl(router_kernel, dim3((T + 7) / 8), dim3(256), 0, (cudaStream_t)stream, logits, ldl, bias, tid2eid, token_ids, vocab, ids,
-                                                               weights, T, E, topk, always, scoring, renorm, scaling, status);
+                                                               weights, T, E, topk, always, groups, keep, scoring, renorm, scaling, status);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

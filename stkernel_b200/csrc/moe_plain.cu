@@ -1,5 +1,5 @@
-// Mixture-of-experts feed-forward with ungated experts, y = W_down act(W_up x), act relu squared or the exact gelu, weights in the
-// compute type (bf16 or fp32).
+// Mixture-of-experts feed-forward, y = W_down act(W_up x) with act relu squared or the exact gelu, or y = W_down (silu(W_gate x) * W_up x)
+// with the rows of W_gate and W_up in turns (so that one tile has both); weights in the compute type (bf16 or fp32).
 //
 //   expert_rows      one CTA per (pair, block of output rows): a warp streams whole weight rows and dots them with the pair's
 //                    activations, fp32 accumulation.  A handful of pairs, and every batch of a float32 model.
@@ -36,6 +36,12 @@ template <> struct Vec16<__nv_bfloat16> {
 };
 
 constexpr int kRowsPerWarp = 4, kExpertWarps = 8;
+
+constexpr int kActGated = 3;                     // N weight rows give N / 2 results
+
+// silu(gate) * up.
+__device__ __forceinline__ float expert_glu(float gate, float up) { return gate / (1.f + expf(-gate)) * up; }
+__device__ __forceinline__ float expert_glu_fast(float gate, float up) { return __fdividef(gate, 1.f + __expf(-gate)) * up; }
 
 // act 0: none, 1: relu squared, 2: gelu (exact).  kRounded: the result is rounded to bf16, so the gelu's erfc may come from the rational
 // approximation 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions (absolute error 1.5e-7).
@@ -81,6 +87,14 @@ expert_rows_kernel(const A* __restrict__ x, long long ldx, int div, const A* __r
     for (int r = 0; r < kRowsPerWarp; ++r)
 #pragma unroll
       for (int i = 0; i < V::kN; ++i) acc[r] = fmaf(wv[r][i], xv[i], acc[r]);
+  }
+  if (act == kActGated) {
+#pragma unroll
+    for (int r = 0; r < kRowsPerWarp; r += 2) {
+      const float v = expert_glu(warp_sum(acc[r]), warp_sum(acc[r + 1]));
+      if (lane == 0 && n0 + r < n_pad) out[pair * ldo + (n0 + r) / 2] = V::round(ok && n0 + r < N ? v : 0.f);
+    }
+    return;
   }
 #pragma unroll
   for (int r = 0; r < kRowsPerWarp; ++r) {
@@ -241,7 +255,15 @@ experts_slim_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
         uint32_t v[16];
         tmem_ld_32x16(tmem + (i & 1) * BT + c + (static_cast<uint32_t>(q * 32) << 16), v);
         tmem_ld_wait();
-        if (n < a.N) {
+        if (a.act == kActGated) {
+          // an odd lane's row is the value that belongs to the gate of the lane before it
+          __nv_bfloat16* og = a.out + (static_cast<long long>(a.offsets[e]) + tt * BT) * a.ldo + (n >> 1);
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const float up = __shfl_down_sync(0xffffffffu, __uint_as_float(v[j]), 1);
+            if ((lane & 1) == 0 && n < a.N && c + j < valid) og[(c + j) * a.ldo] = __float2bfloat16(expert_glu_fast(__uint_as_float(v[j]), up));
+          }
+        } else if (n < a.N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             if (c + j < valid) o[(c + j) * a.ldo] = __float2bfloat16(expert_act(__uint_as_float(v[j]), a.act));
@@ -358,7 +380,19 @@ experts_wide_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
           const int col = half * 128 + c * 32;
           tmem_ld_32x32(tmem + m * 256 + col + (static_cast<uint32_t>(q * 32) << 16), v);
           tmem_ld_wait();
-          if (t < left) {
+          if (t < left && a.act == kActGated) {
+            __nv_bfloat16* og = a.out + static_cast<long long>(row0 + t) * a.ldo + (tn * 256 + col) / 2;
+#pragma unroll
+            for (int j = 0; j < 32; j += 8)
+              if (tn * 256 + col + j < a.N) {
+                __align__(8) __nv_bfloat162 b[2];
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+                  b[k] = __floats2bfloat162_rn(expert_glu_fast(__uint_as_float(v[j + 4 * k]), __uint_as_float(v[j + 4 * k + 1])),
+                                               expert_glu_fast(__uint_as_float(v[j + 4 * k + 2]), __uint_as_float(v[j + 4 * k + 3])));
+                *reinterpret_cast<uint2*>(og + j / 2) = *reinterpret_cast<const uint2*>(b);
+              }
+          } else if (t < left) {
 #pragma unroll
             for (int j = 0; j < 32; j += 8)
               if (tn * 256 + col + j < a.N)                          // N is a multiple of 8
@@ -394,12 +428,12 @@ static int launch_slim(const CUtensorMap& tw, const CUtensorMap& tx, const Exper
 
 using namespace stk;
 
-// x rows of K elements (K a multiple of 16 bytes' worth, rows 16-byte aligned), W [E, N, K].
+// act 3: `out` has N / 2 columns (n_pad / 2 of them are written), N even.  x rows of K elements (K a multiple of 16 bytes' worth, rows 16-byte aligned), W [E, N, K].
 STK_API int stk_expert_rows(const void* x, long long ldx, int div, const void* W, const int* ids, int E, void* out, long long ldo,
                             int N, int n_pad, int K, int act, int fp32, int n_pairs, void* stream) {
   if (n_pairs <= 0) return 0;
   const int v = fp32 ? 4 : 8;
-  if (K % v || ldx % v || div < 1 || N < 1 || n_pad < N || E < 1) return -1;
+  if (K % v || ldx % v || div < 1 || N < 1 || n_pad < N || E < 1 || (act == kActGated && (N | n_pad) % 2)) return -1;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) return -1;
   const int bx = (n_pad + kExpertWarps * kRowsPerWarp - 1) / (kExpertWarps * kRowsPerWarp);
   cudaStream_t st = (cudaStream_t)stream;
@@ -425,7 +459,7 @@ STK_API int stk_expert_gather(const void* x, long long ldx, const int* sorted, i
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-// xs [n_pairs, K] sorted by expert, W [E, N, K], out [n_pairs, ldo]; bf16.  The tile follows the average number of pairs an expert has.
+// xs [n_pairs, K] sorted by expert, W [E, N, K], out [n_pairs, ldo] (act 3: N / 2 columns); bf16.  The tile follows the average number of pairs an expert has.
 STK_API int stk_experts(const void* xs, int n_pairs, const void* W, const int* offsets, int E, int N, int K, void* out, long long ldo,
                         int act, int sm_count, int* status, void* stream) {
   if (n_pairs <= 0) return 0;

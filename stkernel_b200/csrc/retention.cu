@@ -3,7 +3,7 @@
 //
 //   retention_scan       decode rows, short spans, float32: rotation in fp32 on the way into the recurrence
 //   rotate_qk            long spans: rotated queries and scaled, rotated keys as bf16 pairs for the chunked form
-//   retention_finish     head norm, gate, factor
+//   retention_finish     head norm (weighted, if there is a weight), gate, factor; time mixing ends with it as well
 #define STK_PDL_CLASS 16
 #include "linear_scan.cuh"
 
@@ -27,6 +27,7 @@ __device__ __forceinline__ float rotated(const RotArgs& r, const A* x, int d, lo
 
 template <typename A>
 struct RetentionFront {
+  static constexpr bool kPerChannel = false;
   RotArgs r;
   int v_off, D, V;
   const float* decay;                             // [2][H]: the decays and what their rounding left over
@@ -137,11 +138,11 @@ rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bf
   }
 }
 
-// out[t, col + h * V + c] = o / rms(o over the head) * silu(g) * scale: one warp per (token, head).  Zeros into the columns left .. col
+// out[t, col + h * V + c] = o / rms(o over the head) * weight * silu(g) * scale (weight null: 1): one warp per (token, head).  Zeros into the columns left .. col
 // and behind the last head.  NV > 0: bf16 heads of at most 128 * NV columns in whole groups of four, which stay in registers.
 template <typename A, int NV>
 __global__ void __launch_bounds__(256)
-retention_finish_kernel(const float* __restrict__ o, float eps, const int* __restrict__ tok_req, const int64_t* __restrict__ positions,
+retention_finish_kernel(const float* __restrict__ o, float eps, const float* __restrict__ weight, const int* __restrict__ tok_req, const int64_t* __restrict__ positions,
                         const A* __restrict__ proj, long long ldp, int g_off, float scale, A* __restrict__ out, long long ldo, int left,
                         int col, int cols, int H, int V, int T) {
   pdl_wait();
@@ -184,6 +185,10 @@ retention_finish_kernel(const float* __restrict__ o, float eps, const int* __res
       if (c >= V) continue;
       const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu[i].x));
       const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu[i].y));
+      if (weight != nullptr) {
+        const float4 w = *reinterpret_cast<const float4*>(weight + h * V + c);
+        v[i].x *= w.x; v[i].y *= w.y; v[i].z *= w.z; v[i].w *= w.w;
+      }
       uint2 pk;
       *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(v[i].x * r * silu_bf16(g0.x), v[i].y * r * silu_bf16(g0.y));
       *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(v[i].z * r * silu_bf16(g1.x), v[i].w * r * silu_bf16(g1.y));
@@ -195,7 +200,7 @@ retention_finish_kernel(const float* __restrict__ o, float eps, const int* __res
   const float r = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
   for (int c = lane; c < V; c += 32) {
     const float z = ld_act(g + c);
-    st_act(to + c, x[c] * r * z / (1.f + expf(-z)));
+    st_act(to + c, x[c] * r * (weight != nullptr ? weight[h * V + c] : 1.f) * z / (1.f + expf(-z)));
   }
 }
 
@@ -229,7 +234,7 @@ STK_API int stk_rotate_qk(const void* proj, long long ldp, int q_off, int k_off,
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-STK_API int stk_retention_finish(const float* o, float eps, const int* tok_req, const int64_t* positions, const void* proj, long long ldp,
+STK_API int stk_retention_finish(const float* o, float eps, const float* weight, const int* tok_req, const int64_t* positions, const void* proj, long long ldp,
                                  int g_off, float scale, void* out, long long ldo, int left, int col, int cols, int fp32, int heads,
                                  int vdim, int T, void* stream) {
   if (T <= 0) return 0;
@@ -238,7 +243,7 @@ STK_API int stk_retention_finish(const float* o, float eps, const int* tok_req, 
   const bool vec = !fp32 && vdim <= 512 && ((vdim | g_off | col) & 3) == 0 && ((ldp | ldo) & 3) == 0 &&
                    ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(out)) & 7) == 0;
 #define STK_FINISH(A, NV)                                                                                                          \
-  launch_pdl(retention_finish_kernel<A, NV>, grid, dim3(256), 0, st, o, eps, tok_req, positions, (const A*)proj, ldp, g_off, scale, (A*)out, \
+  launch_pdl(retention_finish_kernel<A, NV>, grid, dim3(256), 0, st, o, eps, weight, tok_req, positions, (const A*)proj, ldp, g_off, scale, (A*)out, \
              ldo, left, col, cols, heads, vdim, T)
   if (fp32) STK_FINISH(float, 0);
   else if (!vec) STK_FINISH(__nv_bfloat16, 0);

@@ -6,6 +6,7 @@
 // with bounds checks); weights from the unbiased score, renormalised and scaled (topkGatingSoftplusSqrt /
 // fused_topk_bias and the hash-MoE lookup of overlay/nvidia_model.py:806-827).
 // `always` experts E, E + 1, ... are taken by every token with weight 1, behind the chosen ones.
+// groups > 1: only experts of the `keep` groups (equal, of neighbours) with the largest sums of two selection scores can be selected.
 // Scoring 2 (softmax over the chosen): score = logit + bias, weights = softmax of the selected scores.
 #pragma once
 #include "common.cuh"
@@ -19,7 +20,7 @@ struct RouterArgs {
   int vocab;
   int* ids;                   // [T, topk + always]
   float* weights;             // [T, topk + always]
-  int E, topk, always, scoring, renorm;
+  int E, topk, always, groups, keep, scoring, renorm;
   float scaling;
   int* status;
 };
@@ -49,6 +50,38 @@ __device__ __forceinline__ void route_token_impl(const RouterArgs& r, const floa
     } else {
       sc[i] = 0.f;
       sel[i] = -INFINITY;
+    }
+  }
+  if (r.groups > 1) {
+    const int size = r.E / r.groups;
+    float score = -INFINITY;                             // lane g: group g's score (at most 32 groups)
+    for (int g = 0; g < r.groups; ++g) {
+      float sum = 0.f;
+      int first = -1;
+      for (int j = 0; j < 2; ++j) {
+        float best = -INFINITY;
+        int best_e = 0x7fffffff;
+#pragma unroll
+        for (int i = 0; i < kPer; ++i) {
+          const int e = i * 32 + lane;
+          if (e / size == g && e < r.E && e != first && sel[i] > best) { best = sel[i]; best_e = e; }
+        }
+        const uint32_t key = ordered_key(best), kmax = __reduce_max_sync(0xffffffffu, key);
+        first = __reduce_min_sync(0xffffffffu, key == kmax ? best_e : 0x7fffffff);
+        sum += (kmax & 0x80000000u) ? __uint_as_float(kmax & 0x7fffffffu) : __uint_as_float(~kmax);
+      }
+      if (lane == g) score = sum;
+    }
+    uint32_t kept = 0;
+    for (int j = 0; j < r.keep; ++j) {
+      const bool open = lane < r.groups && !((kept >> lane) & 1u);
+      const uint32_t key = open ? ordered_key(score) : 0u, kmax = __reduce_max_sync(0xffffffffu, key);
+      kept |= 1u << __reduce_min_sync(0xffffffffu, open && key == kmax ? lane : 31);
+    }
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int e = i * 32 + lane;
+      if (e < r.E && !((kept >> (e / size)) & 1u)) sel[i] = -INFINITY;
     }
   }
   float wsum = 0.f, top = 0.f;

@@ -442,7 +442,7 @@ STK_API int stk_skinny_linear_fused(const void* W, long long ldw, int is_fp8, co
                                     const void* x, long long ldx, void* out, long long ldo, int T, int N, int K,
                                     int out_fp32, int sm_count, const void* norm_w, float norm_eps, const void* ll_ctx,
                                     int route, int* route_counter, const float* bias, const int* tid2eid,
-                                    const int64_t* token_ids, int vocab, int* ids, float* weights, int topk, int always, int scoring,
+                                    const int64_t* token_ids, int vocab, int* ids, float* weights, int topk, int always, int groups, int keep, int scoring,
                                     int renorm, float scaling, int* status, void* stream) {
   SkinnyExtra ex;
   memset(&ex, 0, sizeof(ex));
@@ -453,13 +453,13 @@ STK_API int stk_skinny_linear_fused(const void* W, long long ldw, int is_fp8, co
     ex.use_ll = 1;
   }
   if (route) {
-    if (always < 0 || topk + always > 32) return -9;
+    if (always < 0 || topk + always > 32 || groups < 1 || groups > 32 || keep < 1) return -9;
     // a narrow projection (a few hundred rows) leaves most SMs idle: two CTAs per row block, half of K each
     const int n_chunks = K / (is_fp8 ? 16 : 8);
     ex.k_split = (route == 2 && (n_chunks / 2) % 32 == 0) ? 2 : 1;
     ex.route = 1;
     ex.route_counter = route_counter;
-    ex.router = RouterArgs{bias, tid2eid, token_ids, vocab, ids, weights, N, topk, always, scoring, renorm, scaling, status};
+    ex.router = RouterArgs{bias, tid2eid, token_ids, vocab, ids, weights, N, topk, always, groups, keep, scoring, renorm, scaling, status};
   }
   return skinny_launch(W, ldw, is_fp8, w_scale, w_scale_ld, x, ldx, out, ldo, T, N, K, out_fp32, sm_count, 1, 0, 0.f, ex,
                        stream);

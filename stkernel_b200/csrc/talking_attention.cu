@@ -1,0 +1,274 @@
+// Grouped-query attention whose heads' scores are mixed before the softmax (ops/talking.py).
+//
+// A cached row holds the values of all key/value heads (vp columns each), then from k_col on their keys (kp columns each); pages are
+// [64][row].  A mixed query has G * kp columns: in the part of key/value head c the sum of talk[h, g] q_g over the heads g that read c.
+//
+//   talking_prep         one CTA per token: biases, weighted RMS norms, rotation, the token's row, mixed queries, gate logits
+//   talking_simt         any size and type, fp32 arithmetic throughout: one CTA per (token, head)
+#define STK_PDL_CLASS 8
+#include "hybrid_block.cuh"
+#include "talking_attention.cuh"
+
+namespace stk {
+
+struct TalkPrepArgs {
+  const void* proj; long long ldp; int q_off, k_off, v_off, g_off;
+  const float* bias;                                   // [H * D | G * D | G * V] or nullptr
+  const float* q_norm; const float* k_norm; float eps; // [D] or nullptr
+  const float* freq; int pairs;                        // [2][pairs]
+  const float* talk;                                   // [H, H]
+  const int64_t* positions; const int* tok_req; const int* table; int bt_stride;
+  void* cache; int row, k_col, kp, vp;
+  int H, G, D, V;
+  void* q; float* gate;
+};
+
+constexpr int kTkThreads = 256;
+
+// HG: heads per key/value head (their queries stay in registers while all heads' mixtures are formed), 0: any number.
+template <typename A, int HG>
+__global__ void __launch_bounds__(kTkThreads)
+talking_prep_kernel(const TalkPrepArgs a) {
+  extern __shared__ __align__(16) float sm[];
+  const int D2 = (a.D + 1) & ~1;
+  float* x = sm;                                       // [H + G][D2]: queries, keys
+  float* talk = x + (a.H + a.G) * D2;                  // [H][H], transposed: talk[g][h]
+  float2* cs = reinterpret_cast<float2*>(talk + ((a.H * a.H + 1) & ~1));      // [pairs]
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, KD = a.G * a.kp;
+  const int req = a.tok_req[t];
+  const long long pos = a.positions[t];
+  A* q = reinterpret_cast<A*>(a.q) + t * a.H * KD;
+  const A* p = reinterpret_cast<const A*>(a.proj) + t * a.ldp;
+  if (a.gate != nullptr)
+    for (int h = threadIdx.x; h < a.H; h += kTkThreads) a.gate[t * a.H + h] = ld_act(p + a.g_off + h);
+  if (req < 0 || pos < 0) {
+    for (int i = threadIdx.x; i < a.H * KD; i += kTkThreads) st_act(q + i, 0.f);
+    return;
+  }
+  for (int i = threadIdx.x; i < a.pairs; i += kTkThreads) cs[i] = cos_sin_split(pos, a.freq[i], a.freq[a.pairs + i]);
+  for (int i = threadIdx.x; i < a.H * a.H; i += kTkThreads) talk[(i % a.H) * a.H + i / a.H] = a.talk[i];
+  for (int u = warp; u < a.H + a.G; u += kTkThreads / 32) {
+    const bool isq = u < a.H;
+    const A* src = p + (isq ? a.q_off + u * a.D : a.k_off + (u - a.H) * a.D);
+    const float* w = isq ? a.q_norm : a.k_norm;
+    float* dst = x + u * D2;
+    float s = 0.f;
+    for (int d = lane; d < a.D; d += 32) {
+      const float v = ld_act(src + d) + (a.bias != nullptr ? a.bias[u * a.D + d] : 0.f);
+      dst[d] = v;
+      s = fmaf(v, v, s);
+    }
+    if (w != nullptr) {
+      const float f = 1.f / sqrtf(warp_sum(s) / static_cast<float>(a.D) + a.eps);
+      for (int d = lane; d < a.D; d += 32) dst[d] *= f * w[d];
+    }
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < (a.H + a.G) * a.pairs; e += kTkThreads) {
+    const int u = e / a.pairs, i = e - u * a.pairs;
+    float* v = x + u * D2 + 2 * i;
+    const float c0 = v[0], c1 = v[1];
+    const float2 w = cs[i];
+    v[0] = c0 * w.x - c1 * w.y;
+    v[1] = c1 * w.x + c0 * w.y;
+  }
+  __syncthreads();
+  const int page = a.table[static_cast<long long>(req) * a.bt_stride + pos / kTkPage];
+  if (page >= 0) {
+    A* row = reinterpret_cast<A*>(a.cache) + (static_cast<long long>(page) * kTkPage + pos % kTkPage) * a.row;
+    for (int e = threadIdx.x; e < a.G * a.vp; e += kTkThreads) {
+      const int g = e / a.vp, d = e - g * a.vp;
+      st_act(row + e, d < a.V ? ld_act(p + a.v_off + g * a.V + d) + (a.bias != nullptr ? a.bias[(a.H + a.G) * a.D + g * a.V + d] : 0.f) : 0.f);
+    }
+    for (int e = threadIdx.x; e < KD; e += kTkThreads) {
+      const int g = e / a.kp, d = e - g * a.kp;
+      st_act(row + a.k_col + e, d < a.D ? x[(a.H + g) * D2 + d] : 0.f);
+    }
+  }
+  const int hg = HG > 0 ? HG : a.H / a.G, half = a.kp >> 1;
+  for (int e = threadIdx.x; e < a.G * half; e += kTkThreads) {          // two columns of every head's mixture
+    const int c = e / half, d = (e - c * half) * 2;
+    const bool in0 = d < a.D, in1 = d + 1 < a.D;
+    const float* qc = x + c * hg * D2 + d;
+    float q0[HG > 0 ? HG : 1], q1[HG > 0 ? HG : 1];
+    if (HG > 0) {
+#pragma unroll
+      for (int g = 0; g < HG; ++g) {
+        q0[g] = in0 ? qc[g * D2] : 0.f;
+        q1[g] = in1 ? qc[g * D2 + 1] : 0.f;
+      }
+    }
+    for (int h = 0; h < a.H; ++h) {
+      float s0 = 0.f, s1 = 0.f;
+      if (HG > 0) {
+#pragma unroll
+        for (int g = 0; g < HG; ++g) {
+          const float w = talk[(c * HG + g) * a.H + h];
+          s0 = fmaf(w, q0[g], s0);
+          s1 = fmaf(w, q1[g], s1);
+        }
+      } else {
+        for (int g = 0; g < hg; ++g) {
+          const float w = talk[(c * hg + g) * a.H + h];
+          s0 = fmaf(w, in0 ? qc[g * D2] : 0.f, s0);
+          s1 = fmaf(w, in1 ? qc[g * D2 + 1] : 0.f, s1);
+        }
+      }
+      A* to = q + static_cast<long long>(h) * KD + c * a.kp + d;
+      if (sizeof(A) == 2) {
+        *reinterpret_cast<__nv_bfloat162*>(to) = __floats2bfloat162_rn(s0, s1);
+      } else {
+        st_act(to, s0);
+        st_act(to + 1, s1);
+      }
+    }
+  }
+}
+
+// ---- any size, fp32 arithmetic ------------------------------------------------------------------
+constexpr int kTkKeys = 512;
+
+template <typename A>
+__global__ void __launch_bounds__(128)
+talking_simt_kernel(const TalkArgs a, const int* __restrict__ first_pos, const int* __restrict__ last_pos, int max_span) {
+  extern __shared__ __align__(16) float q[];           // [G * kp]
+  __shared__ float sc[kTkKeys];
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x, h = blockIdx.y, KD = a.G * a.kp, vc = h / (a.H / a.G) * a.vp;
+  const int req = a.tok_req[t];
+  const long long pos = a.positions[t];
+  A* out = reinterpret_cast<A*>(a.out) + t * a.ldo;
+  if (req >= 0 && pos >= 0 && last_pos[t] - first_pos[t] + 1 > max_span) return;
+  if (h == a.H - 1)
+    for (int d = a.H * a.V + threadIdx.x; d < a.out_cols; d += blockDim.x) st_act(out + d, 0.f);
+  out += h * a.V;
+  if (req < 0 || pos < 0) {
+    for (int d = threadIdx.x; d < a.V; d += blockDim.x) st_act(out + d, 0.f);
+    return;
+  }
+  const A* qg = reinterpret_cast<const A*>(a.q) + t * a.ldq + static_cast<long long>(h) * KD;
+  for (int d = threadIdx.x; d < KD; d += blockDim.x) q[d] = ld_act(qg + d);
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long lo = talk_first(a, pos);
+  const int* bt = a.table + static_cast<long long>(req) * a.bt_stride;
+  const A* cache = reinterpret_cast<const A*>(a.cache);
+  auto row_of = [&](long long p) {
+    const int page = bt[p / kTkPage];
+    return cache + (static_cast<long long>(page < 0 ? 0 : page) * kTkPage + p % kTkPage) * a.row;
+  };
+  float m = a.sink != nullptr ? a.sink[h] : -INFINITY, l = a.sink != nullptr ? 1.f : 0.f, acc[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+  for (long long k0 = lo; k0 <= pos; k0 += kTkKeys) {
+    const int n = static_cast<int>(pos + 1 - k0 < kTkKeys ? pos + 1 - k0 : kTkKeys);
+    float mx = -INFINITY;
+    for (int j = warp; j < n; j += 4) {
+      const A* r = row_of(k0 + j) + a.k_col;
+      float s = 0.f;
+      for (int d = lane; d < KD; d += 32) s = fmaf(q[d], ld_act(r + d), s);
+      s = warp_sum(s) * a.scale;
+      if (lane == 0) sc[j] = s;
+      mx = fmaxf(mx, s);
+    }
+    const float m_new = fmaxf(m, block_max(mx, red));
+    float sum = 0.f;
+    for (int j = threadIdx.x; j < n; j += blockDim.x) {
+      const float p = expf(sc[j] - m_new);
+      sc[j] = p;
+      sum += p;
+    }
+    const float f = expf(m - m_new);
+    l = l * f + block_sum(sum, red);
+    m = m_new;
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] *= f;
+    for (int j = 0; j < n; ++j) {
+      const A* r = row_of(k0 + j) + vc;
+      const float p = sc[j];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int d = threadIdx.x + i * 128;
+        if (d < a.V) acc[i] = fmaf(p, ld_act(r + d), acc[i]);
+      }
+    }
+    __syncthreads();
+  }
+  const float g = talk_gate(a, t, h) / l;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int d = threadIdx.x + i * 128;
+    if (d < a.V) st_act(out + d, acc[i] * g);
+  }
+}
+
+template <typename A>
+static int launch_talk_prep(const TalkPrepArgs& a, int T, cudaStream_t st) {
+  const size_t smem = (static_cast<size_t>(a.H + a.G) * ((a.D + 1) & ~1) + ((a.H * a.H + 1) & ~1) + 2 * a.pairs) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+#define STK_TALK_PREP(HG)                                                                                                       \
+  {                                                                                                                             \
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(talking_prep_kernel<A, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
+                                                 200 * 1024) != cudaSuccess)                                                    \
+      return -3;                                                                                                                \
+    launch_pdl(talking_prep_kernel<A, HG>, dim3(T), dim3(kTkThreads), smem, st, a);                                             \
+  }
+  switch (a.H / a.G) {
+    case 1: STK_TALK_PREP(1) break;
+    case 2: STK_TALK_PREP(2) break;
+    case 4: STK_TALK_PREP(4) break;
+    case 8: STK_TALK_PREP(8) break;
+    default: STK_TALK_PREP(0) break;
+  }
+#undef STK_TALK_PREP
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+}  // namespace stk
+
+using namespace stk;
+
+// q: [T, heads * kv_heads * kp] in the type of proj; gate [T, heads] fp32 or null (no gate).
+STK_API int stk_talking_prep(const void* proj, long long ldp, int q_off, int k_off, int v_off, int g_off, const float* bias,
+                             const float* q_norm, const float* k_norm, float eps, const float* freq, int pairs, const float* talk,
+                             const int64_t* positions, const int* tok_req, const int* table, int bt_stride, void* cache, int row, int k_col,
+                             int kp, int vp, int heads, int kv_heads, int dim, int vdim, void* q, float* gate, int fp32, int T,
+                             void* stream) {
+  if (T <= 0) return 0;
+  if (heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || kp < dim || (kp & 1) || vp < vdim || k_col != kv_heads * vp ||
+      row < k_col + kv_heads * kp || pairs < 0 || 2 * pairs > dim || (q_norm == nullptr) != (k_norm == nullptr))
+    return -1;
+  TalkPrepArgs a;
+  a.proj = proj; a.ldp = ldp; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.g_off = g_off;
+  a.bias = bias; a.q_norm = q_norm; a.k_norm = k_norm; a.eps = eps; a.freq = freq; a.pairs = pairs; a.talk = talk;
+  a.positions = positions; a.tok_req = tok_req; a.table = table; a.bt_stride = bt_stride;
+  a.cache = cache; a.row = row; a.k_col = k_col; a.kp = kp; a.vp = vp;
+  a.H = heads; a.G = kv_heads; a.D = dim; a.V = vdim; a.q = q; a.gate = gate;
+  return fp32 ? launch_talk_prep<float>(a, T, (cudaStream_t)stream) : launch_talk_prep<__nv_bfloat16>(a, T, (cudaStream_t)stream);
+}
+
+// Spans of at most max_span tokens.
+STK_API int stk_talking_simt(const void* q, long long ldq, const float* gate, const float* sink, const int64_t* positions, const int* tok_req,
+                             const int* table, int bt_stride, const void* cache, int row, int k_col, int kp, int vp, int heads, int kv_heads,
+                             int vdim, int chunk, float scale, void* out, long long ldo, int out_cols, int fp32, const int* first_pos,
+                             const int* last_pos, int max_span, int T, void* stream) {
+  if (T <= 0) return 0;
+  const TalkArgs a = {q, ldq, gate, sink, positions, tok_req, table, bt_stride, cache, row, k_col, kp, vp, heads, kv_heads, vdim, chunk,
+                      scale, out, ldo, out_cols};
+  const size_t smem = static_cast<size_t>(kv_heads) * kp * sizeof(float);
+  if (!talk_ok(a) || vdim > 1024 || heads > 65535 || smem > 200 * 1024) return -1;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (smem > 40 * 1024 &&
+      (cudaFuncSetAttribute(talking_simt_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess ||
+       cudaFuncSetAttribute(talking_simt_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess))
+    return -3;
+  if (fp32) launch_pdl(talking_simt_kernel<float>, dim3(T, heads), dim3(128), smem, st, a, first_pos, last_pos, max_span);
+  else launch_pdl(talking_simt_kernel<__nv_bfloat16>, dim3(T, heads), dim3(128), smem, st, a, first_pos, last_pos, max_span);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}

@@ -1,4 +1,4 @@
-"""Decoder described layer by layer (`HybridConfig`): attention and recurrent mixers, in parallel, post-norm or streams blocks.
+"""Decoder described layer by layer (`HybridConfig`): attention and recurrent mixers, in parallel, post-norm, streams or shifted blocks.
 
 Parallel block: a layer is two matrix products.  Everything that reads the layer's norm (mixer projections, feed-forward gate and up) is one
 weight `w_in`; everything that is added to the residual (mixer output and feed-forward down projection) is one weight `w_out`
@@ -16,6 +16,11 @@ Streams block: several fp32 residual streams; one kernel per sublayer writes the
 weighted sum over a token's experts on the way), forms the next sublayer's weighted sum of the new streams and norms it:
 
     x_t = sum_s mix[s, t] x_s + write[t] y;  h = norm(sum_s read[s] x_s);  y = sublayer(h)
+
+Shifted block: one kernel per layer adds what the layer before left (both sides of its mixer, each normed, and its feed-forward) to the
+fp32 residual, norms it, and forms the token-shifted input of the mixer and the blends that time mixing projects:
+
+    h = norm(x += y_prev);  s = h + (h' - h) shift;  y = mixer(s) + ff(h)          (h': the previous token's h)
 
 A parallel mixer (two mixers over the same input) is one product in and one product out, like the parallel block's sublayers.
 
@@ -36,10 +41,12 @@ from ..ops import hybrid as HB
 from ..ops import latent as LA
 from ..ops import moe as MO
 from ..ops import recurrence as RC
+from ..ops import shifted as SH
+from ..ops import talking as TK
 from ..ops.functional import LinearWeight
 from ..utils.spans import span
 from .decoder import Decoder
-from .sources import WeightSource
+from .sources import RANDOM_EXTENT, WeightSource
 
 BF16 = torch.bfloat16
 F32 = torch.float32
@@ -59,6 +66,8 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
             continue
         m, p = l.mixer, f"l{i}"
         out[f"{p}.norm1"] = ((W,), "bf16")
+        if cfg.block == "shifted":
+            out[f"{p}.shift"] = ((W,), "bf16")
         if cfg.block == "streams":
             for q in (1, 2) if l.mlp is not None else (1,):
                 out[f"{p}.norm{q}.b"] = ((W,), "bf16")
@@ -95,22 +104,31 @@ def weight_shapes(cfg: HybridConfig) -> Dict[str, Tuple[Tuple[int, ...], str]]:
         if m.kind != "parallel":
             out[f"{p}.mix.o"] = ((W, m.out_dim), "bf16")
         if l.mlp is not None:
-            if cfg.block != "parallel":
+            if cfg.block not in ("parallel", "shifted"):
                 out[f"{p}.norm2"] = ((W,), "bf16")
             if l.mlp.kind == "dense":
-                out[f"{p}.mlp.gate"] = ((l.mlp.ff, W), "bf16")
+                if l.mlp.gated:
+                    out[f"{p}.mlp.gate"] = ((l.mlp.ff, W), "bf16")
+                else:
+                    out[f"{p}.mlp.act"] = ((2,), "bf16")
                 out[f"{p}.mlp.up"] = ((l.mlp.ff, W), "bf16")
                 out[f"{p}.mlp.down"] = ((W, l.mlp.ff), "bf16")
             else:
                 for e in range(l.mlp.experts):
+                    if l.mlp.gated:
+                        out[f"{p}.mlp.e{e}.gate"] = ((l.mlp.ff, W), "bf16")
                     out[f"{p}.mlp.e{e}.up"] = ((l.mlp.ff, W), "bf16")
                     out[f"{p}.mlp.e{e}.down"] = ((W, l.mlp.ff), "bf16")
                 out[f"{p}.mlp.router"] = ((l.mlp.experts, W), "bf16")
                 if l.mlp.router_bias:
                     out[f"{p}.mlp.router.b"] = ((l.mlp.experts,), "bf16")
+                if l.mlp.scoring == "sigmoid":
+                    out[f"{p}.mlp.correction"] = ((l.mlp.experts,), "bf16")
                 if l.mlp.shared_ff:
                     out[f"{p}.mlp.shared.up"] = ((l.mlp.shared_ff, W), "bf16")
                     out[f"{p}.mlp.shared.down"] = ((W, l.mlp.shared_ff), "bf16")
+    if cfg.bigram is not None:
+        out["bigram"] = ((cfg.bigram.buckets + 1, W), "bf16")
     out["final.norm"] = ((W,), "bf16")
     if cfg.block == "streams":
         out["final.norm.b"] = ((W,), "bf16")
@@ -127,9 +145,28 @@ def _parallel_shapes(p: str, m, W: int) -> Dict[str, Tuple[Tuple[int, ...], str]
         if a.bias:
             out[f"{p}.left.{n}.b"] = ((rows,), "bf16")
     if a.gate:
-        out[f"{p}.left.g"] = ((a.out_dim, W), "bf16")
-    for n, rows in (("q", r.heads * r.dim), ("k", r.heads * r.dim), ("v", r.out_dim), ("g", r.out_dim)):
-        out[f"{p}.right.{n}"] = ((rows, W), "bf16")
+        out[f"{p}.left.g"] = ((a.heads if a.kind == "talking_attention" else a.out_dim, W), "bf16")
+    if a.kind == "talking_attention":
+        if a.qk_norm:
+            out[f"{p}.left.q.norm"] = out[f"{p}.left.k.norm"] = ((a.dim,), "bf16")
+        out[f"{p}.left.talk"] = ((a.heads, a.heads), "bf16")
+        if a.sink:
+            out[f"{p}.left.sink"] = ((a.heads,), "bf16")
+    if m.out_norm:
+        out[f"{p}.left.out"] = out[f"{p}.right.out"] = ((W,), "bf16")
+    if r.kind == "time_mix":
+        N = r.out_dim
+        for n in "rkvg":
+            out[f"{p}.right.{n}"] = ((N, W), "bf16")
+        for n in "rkvgw":
+            out[f"{p}.right.mu.{n}"] = ((W,), "bf16")
+        out[f"{p}.right.w1"] = ((r.rank, W), "bf16")
+        out[f"{p}.right.w2"] = ((N, r.rank), "bf16")
+        out[f"{p}.right.w0"] = out[f"{p}.right.norm"] = ((N,), "bf16")
+        out[f"{p}.right.u"] = ((r.heads, r.dim), "bf16")
+    else:
+        for n, rows in (("q", r.heads * r.dim), ("k", r.heads * r.dim), ("v", r.out_dim), ("g", r.out_dim)):
+            out[f"{p}.right.{n}"] = ((rows, W), "bf16")
     out[f"{p}.left.o"] = ((W, a.out_dim), "bf16")
     out[f"{p}.right.o"] = ((W, r.out_dim), "bf16")
     return out
@@ -145,10 +182,11 @@ def _mamba2_shapes(p: str, m, W: int) -> Dict[str, Tuple[Tuple[int, ...], str]]:
 
 def init_random_weights(cfg: HybridConfig, seed: int = 0, std: Optional[float] = None) -> Dict[str, torch.Tensor]:
     """Random master weights: matrices ~N(0, std) (default: fan-in scaled), norms around 1, forget biases positive, residual streams
-    that mostly stay themselves, step sizes around 0.1."""
+    that mostly stay themselves, step sizes around 0.1, blends between a token and its predecessor from 0 to 0.8, decays from fast to slow."""
     g = torch.Generator().manual_seed(seed)
     w: Dict[str, torch.Tensor] = {}
     for name, (shape, _) in weight_shapes(cfg).items():
+        shape = tuple(RANDOM_EXTENT if n is None else n for n in shape)
         r = torch.randn(shape, generator=g)
         if len(shape) == 1 and "norm" in name and not name.endswith(".b"):
             t = 1.0 + 0.2 * r
@@ -158,6 +196,16 @@ def init_random_weights(cfg: HybridConfig, seed: int = 0, std: Optional[float] =
             t = 0.7 * r - 2.0
         elif name.endswith(".f.b"):
             t = 3.0 + r
+        elif name.endswith(".shift") or ".mu." in name:
+            t = 0.4 + 0.4 * torch.tanh(r)
+        elif name.endswith((".left.out", ".right.out")):
+            t = 1.0 + 0.2 * r
+        elif name.endswith(".w0"):
+            t = -3.0 + 1.5 * r
+        elif name.endswith(".talk"):
+            t = torch.eye(shape[0]) + 0.3 * r
+        elif name.endswith(".correction"):
+            t = 0.3 * r - 1.0
         elif len(shape) == 1:
             t = 0.5 * r
         else:
@@ -182,6 +230,16 @@ class BlockWeights:
     grouped: Optional[GA.GroupedParams] = None
     retention: Optional[RC.RetentionParams] = None
     mamba2: Optional[RC.Mamba2Params] = None
+    talking: Optional[TK.TalkingParams] = None
+    time_mix: Optional[RC.TimeMixParams] = None
+    # parallel mixers whose sides have products of their own
+    w_mixes: Optional[LinearWeight] = None  # [4 * np, pad(W)]: r, k, v, gate of time mixing, each from its own blend
+    w_decay: Tuple[LinearWeight, ...] = ()  # [pad(rank), pad(W)], [np, pad(rank) or twice that]
+    w_sides: Tuple[LinearWeight, ...] = ()  # output projections, left and right
+    out_norms: Tuple[torch.Tensor, ...] = ()            # fp32 [W] each
+    # shifted blocks
+    shift: Optional[torch.Tensor] = None    # fp32 [W]
+    mu: Optional[torch.Tensor] = None       # fp32 [blends, W]
     w_gates: Optional[LinearWeight] = None  # [2 * heads, pad(W)]: input and forget gate of the recurrence (fp32 results)
     # streams blocks: norm biases and how the sublayers read and write the streams
     norm_b: Optional[torch.Tensor] = None
@@ -189,7 +247,8 @@ class BlockWeights:
     streams: Tuple[HB.StreamWeights, ...] = ()          # mixer's, feed-forward's
     # post-norm and streams blocks: the feed-forward has weights of its own
     norm2: Optional[torch.Tensor] = None    # fp32 [W]
-    w_gate_up: Optional[LinearWeight] = None
+    w_gate_up: Optional[LinearWeight] = None            # gate and up, or up alone
+    xielu: Tuple[float, float] = (0.0, 0.0)
     w_down: Optional[LinearWeight] = None
     router: Optional[LinearWeight] = None   # [experts, pad(W)]
     router_bias: Optional[torch.Tensor] = None          # fp32 [experts]
@@ -204,6 +263,7 @@ class HybridWeights:
     layers: List[BlockWeights]              # one entry per layer; `weights_of` layers repeat an entry
     layer_offset: int = 0
     norm_b: Optional[torch.Tensor] = None   # fp32 [W]
+    bigram: Optional[torch.Tensor] = None   # [buckets + 1, W]
 
 
 def _stack(parts: List[Tuple[str, torch.Tensor]], width: int, dtype) -> Tuple[LinearWeight, Dict[str, int]]:
@@ -263,6 +323,35 @@ def _parallel_params(cfg: HybridConfig, m, f32, device) -> Tuple[GA.GroupedParam
     return left, RC.RetentionParams(r.heads, r.dim, r.vdim, log_decay, LA.split_frequencies(r.decay, device), LA.split_frequencies(freq, device), cfg.norm_eps, m.right_scale)
 
 
+def _padded(w: torch.Tensor, rows: int, width: int, dtype) -> torch.Tensor:
+    out = torch.zeros(rows, width, dtype=dtype, device=w.device)
+    out[:w.shape[0], :w.shape[1]] = w.to(dtype)
+    return out
+
+
+def build_talking_time_mix(cfg: HybridConfig, b: BlockWeights, m, get, f32, dt, device) -> None:
+    """Talking-heads attention beside time mixing."""
+    a, r, W = m.left, m.right, cfg.hidden_size
+    bias = torch.cat([f32(f"mix.left.{n}.b") for n in ("q", "k", "v")]).contiguous() if a.bias else None
+    freq = a.rotary.frequencies()[0] if a.rotary is not None else []
+    norms = [f32(f"mix.left.{n}.norm") for n in "qk"] if a.qk_norm else [None, None]
+    b.talking = TK.TalkingParams(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.chunk or 0, cfg.norm_eps, bias, *norms,
+                                 LA.split_frequencies(freq, device), f32("mix.left.talk"), f32("mix.left.sink") if a.sink else None, a.gate)
+    N, np = r.out_dim, _pad(r.out_dim)
+    b.w_mixes = LinearWeight(torch.cat([_padded(get(f"mix.right.{n}"), np, _pad(W), dt) for n in "rkvg"]))
+    w1, w2 = get("mix.right.w1"), get("mix.right.w2")
+    if w1.shape[0] != w2.shape[1]:
+        raise ValueError(f"mix.right.w1 has {w1.shape[0]} rows, mix.right.w2 {w2.shape[1]} columns")
+    rp = _pad(w1.shape[0])
+    w2 = _padded(w2, np, rp, dt)
+    # bf16: tanh comes as high part and remainder, both meet the same weights
+    b.w_decay = (LinearWeight(_padded(w1, rp, _pad(W), dt)), LinearWeight(torch.cat([w2, w2], 1) if dt == BF16 and RC.tanh_pair(device) else w2))
+    b.time_mix = RC.TimeMixParams(r.heads, r.dim, np, f32("mix.right.w0"), f32("mix.right.u").view(-1), f32("mix.right.norm"), cfg.norm_eps)
+    b.w_sides = tuple(LinearWeight(_padded(get(f"mix.{s}.o"), W, _pad(p.out_dim), dt)) for s, p in (("left", a), ("right", r)))
+    b.out_norms = (f32("mix.left.out"), f32("mix.right.out"))
+    b.mu = torch.stack([f32(f"mix.right.mu.{n}") for n in "rkvgw"]).contiguous()
+
+
 def _mamba2_params(cfg: HybridConfig, m, get, f32) -> RC.Mamba2Params:
     return RC.Mamba2Params(m.heads, m.vdim, m.state, m.groups, m.norm_groups, get("mix.conv").to(F32).t().contiguous(), f32("mix.conv.b"),
                            f32("mix.dt_bias"), (-torch.exp(get("mix.A_log").double())).to(F32).contiguous(), f32("mix.D"),
@@ -283,6 +372,8 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
     joined = l.mlp if cfg.block == "parallel" else None              # the feed-forward shares the mixer's two products
     if m.kind == "latent_attention":
         names = ["dq", "dkv", "g"] if m.kv_from is None else ["dq", "g"]
+    elif m.kind == "parallel" and m.left.kind == "talking_attention":
+        names = ["left.q", "left.k", "left.v"] + (["left.g"] if m.left.gate else [])
     elif m.kind == "parallel":
         names = ["left.q", "left.k", "left.v"] + (["left.g"] if m.left.gate else []) + [f"right.{n}" for n in "qkvg"]
     else:
@@ -299,6 +390,8 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
         w_out = torch.zeros(W, m.heads, vp, dtype=dt, device=device)
         w_out[:, :, :m.vdim] = get("mix.o").view(W, m.heads, m.vdim).to(dt)
         w_out = w_out.view(W, m.heads * vp)
+    elif m.kind == "parallel" and m.left.kind == "talking_attention":
+        w_out = None                                       # each side has its own
     elif m.kind == "parallel":
         off = HB.out_offset(m.left.out_dim)
         w_out = torch.zeros(W, off + _pad(m.right.out_dim), dtype=dt, device=device)
@@ -310,7 +403,7 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
         w_out[:, :m.out_dim] = get("mix.o").to(dt)
         if joined is not None:
             w_out[:, off:off + joined.ff] = get("mlp.down").to(dt)
-    b = BlockWeights(f32("norm1"), w_in, LinearWeight(w_out), seg)
+    b = BlockWeights(f32("norm1"), w_in, LinearWeight(w_out) if w_out is not None else None, seg)
     if m.kind == "attention":
         freq, mag = m.rotary.frequencies() if m.rotary is not None else ([], 1.0)
         b.attention = HB.AttentionParams(m.heads, m.kv_heads, m.dim, m.window, m.scale, m.softcap,
@@ -318,6 +411,8 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
                                          f32("mix.sink") if m.sink else None)
     elif m.kind == "latent_attention":
         b.latent = build_latent(cfg, get, m, dt, device)
+    elif m.kind == "parallel" and m.left.kind == "talking_attention":
+        build_talking_time_mix(cfg, b, m, get, f32, dt, device)
     elif m.kind == "parallel":
         b.grouped, b.retention = _parallel_params(cfg, m, f32, device)
     elif m.kind == "mamba2":
@@ -333,16 +428,22 @@ def build_block(cfg: HybridConfig, src: WeightSource, i: int, device) -> BlockWe
         if l.mlp is not None:
             b.norm2_b = f32("norm2.b")
             b.streams += (_stream_weights(f32, 2),)
+    if cfg.block == "shifted":
+        b.shift = f32("shift")
     if l.mlp is not None and joined is None:
+        if cfg.block != "shifted":
+            b.norm2 = f32("norm2")
         build_feed_forward(b, l.mlp, get, W, dt, device)
     return b
 
 
 def build_feed_forward(b: BlockWeights, mlp, get, W: int, dt, device) -> None:
-    b.norm2 = get("norm2").to(F32).contiguous()
     ff = _pad(mlp.ff)
     if mlp.kind == "dense":
-        b.w_gate_up, seg = _stack([("gate", get("mlp.gate")), ("up", get("mlp.up"))], _pad(W), dt)
+        b.w_gate_up, seg = _stack(([("gate", get("mlp.gate"))] if mlp.gated else []) + [("up", get("mlp.up"))], _pad(W), dt)
+        if mlp.act == "xielu":
+            sp = torch.nn.functional.softplus(get("mlp.act").double().cpu()).tolist()
+            b.xielu = (sp[0], sp[1] + 0.5)
         b.seg.update(seg)
         down = torch.zeros(W, ff, dtype=dt, device=device)
         down[:, :mlp.ff] = get("mlp.down").to(dt)
@@ -350,10 +451,14 @@ def build_feed_forward(b: BlockWeights, mlp, get, W: int, dt, device) -> None:
         return
     # the shared expert's columns in equal parts, each an expert that every token takes
     ff, n = _pad(mlp.expert_width), mlp.experts + mlp.shared_parts
-    up = torch.zeros(n, ff, _pad(W), dtype=dt, device=device)
+    up = torch.zeros(n, (2 if mlp.gated else 1) * ff, _pad(W), dtype=dt, device=device)
     down = torch.zeros(n, _pad(W), ff, dtype=dt, device=device)
     for e in range(mlp.experts):
-        up[e, :mlp.ff, :W] = get(f"mlp.e{e}.up").to(dt)
+        if mlp.gated:
+            up[e, 0:2 * mlp.ff:2, :W] = get(f"mlp.e{e}.gate").to(dt)
+            up[e, 1:2 * mlp.ff:2, :W] = get(f"mlp.e{e}.up").to(dt)
+        else:
+            up[e, :mlp.ff, :W] = get(f"mlp.e{e}.up").to(dt)
         down[e, :W, :mlp.ff] = get(f"mlp.e{e}.down").to(dt)
     if mlp.shared_parts:
         wide = mlp.expert_width
@@ -364,7 +469,8 @@ def build_feed_forward(b: BlockWeights, mlp, get, W: int, dt, device) -> None:
     b.experts = MO.PlainExperts(up, down, mlp.act)
     router, _ = _stack([("router", get("mlp.router"))], _pad(W), dt)
     b.router = LinearWeight(router.w[:mlp.experts])
-    b.router_bias = get("mlp.router.b").to(F32).contiguous() if mlp.router_bias else None
+    bias = "mlp.correction" if mlp.scoring == "sigmoid" else "mlp.router.b" if mlp.router_bias else None
+    b.router_bias = get(bias).to(F32).contiguous() if bias is not None else None
 
 
 def build_hybrid_weights(cfg: HybridConfig, src: WeightSource, device) -> HybridWeights:
@@ -384,7 +490,8 @@ def build_hybrid_weights(cfg: HybridConfig, src: WeightSource, device) -> Hybrid
     # a factor on the logits is one on the norm in front of the head
     norm = lambda n: (src.get(n, (W,), device).to(F32) * cfg.logit_scale).contiguous()
     return HybridWeights(embed, head, norm("final.norm"), [blocks[cfg.weight_layer(i)] for i in range(len(cfg.layers))],
-                         norm_b=norm("final.norm.b") if cfg.block == "streams" else None)
+                         norm_b=norm("final.norm.b") if cfg.block == "streams" else None,
+                         bigram=src.get("bigram", (cfg.bigram.buckets + 1, W), device).to(dt).contiguous() if cfg.bigram is not None else None)
 
 
 # ----------------------------------------------------------------------------
@@ -398,7 +505,7 @@ class HybridModel(Decoder):
         self.kv = kv
         self.act = HB.act_dtype(cfg.dtype, self.device)
         self.width = _pad(cfg.hidden_size)
-        self.recurrent = any(recurrent_part(l.mixer) is not None for l in cfg.layers)
+        self.recurrent = cfg.block == "shifted" or any(recurrent_part(l.mixer) is not None for l in cfg.layers)
         self.on_layer = None                # optional hook (layer index, residual [T, W] fp32; streams: their sum) after each layer
         self.read_sum = torch.ones(cfg.streams, dtype=F32, device=self.device)
 
@@ -469,15 +576,17 @@ class HybridModel(Decoder):
         b, mlp = self.w.layers[li], self.cfg.layers[li].mlp
         if mlp.kind == "dense":
             p = Fn.linear(h, b.w_gate_up, tag="gate_up")
+            if not mlp.gated:
+                return Fn.linear(HB.xielu_rows(p, mlp.ff, b.xielu, b.w_down.in_features), b.w_down, out_dtype=F32, tag="down")
             c = torch.empty(h.shape[0], b.w_down.in_features, dtype=self.act, device=h.device)
             HB.join_glu(p, c, 0, (b.seg["gate"], b.seg["up"], mlp.ff), mlp.act)
             return Fn.linear(c, b.w_down, out_dtype=F32, tag="down")
         with span("experts", h.shape[0]):
-            always = mlp.shared_parts
-            routed = Fn.gate_route(h, b.router, b.router_bias, mlp.top, "softmax_topk", True, 1.0, always=always) if h.is_cuda else None
+            how = (b.router_bias, mlp.top, mlp.scoring, True, mlp.scale)
+            kw = dict(always=mlp.shared_parts, groups=mlp.groups, keep=mlp.keep)
+            routed = Fn.gate_route(h, b.router, *how, **kw) if h.is_cuda else None
             if routed is None:
-                logits = Fn.linear(h, b.router, out_dtype=F32, tag="router")
-                routed = MO.router(logits, b.router_bias, mlp.top, "softmax_topk", True, 1.0, always=always)
+                routed = MO.router(Fn.linear(h, b.router, out_dtype=F32, tag="router"), *how, **kw)
             return MO.plain_experts(h, *routed, b.experts)
 
     def post_norm_layer(self, li: int, x: torch.Tensor, h: torch.Tensor, meta: HB.HybridMeta) -> torch.Tensor:
@@ -488,6 +597,45 @@ class HybridModel(Decoder):
         if cfg.layers[li].mlp is not None:
             h = HB.post_norm_add(x, self.feed_forward(li, h), b.norm2, cfg.norm_eps, self.width, self.act)
         return h
+
+    def sides(self, li: int, s: torch.Tensor, blends: Optional[torch.Tensor], meta: HB.HybridMeta) -> SH.Pending:
+        """Outputs of layer li's mixer on the shifted rows s (and their blends, for time mixing), as the next norm adds them."""
+        b, m = self.w.layers[li], self.cfg.layers[li].mixer
+        if m.kind != "parallel":
+            return SH.Pending([(Fn.linear(self.mix(li, s, meta), b.w_out, out_dtype=F32, tag="out"), None, 1.0)])
+        t, width, sg = s.shape[0], self.width, b.seg
+        p = Fn.linear(s, b.w_in, tag="in")
+        table, cache = self.kv.group_of(li).table_dev, self.kv.kv_cache[li]
+        with span("talking_attention", t):
+            q, gate = TK.talking_prep(p, sg["left.q"], sg["left.k"], sg["left.v"], sg.get("left.g", 0), b.talking, meta, table, cache)
+            c = torch.empty(t, b.w_sides[0].in_features, dtype=self.act, device=s.device)
+            TK.talking_attention(q, gate, b.talking, meta, table, cache, c)
+        left = Fn.linear(c, b.w_sides[0], out_dtype=F32, tag="out")
+        with span("time_mix", t):
+            p = Fn.linear(blends[:, :4 * width], b.w_mixes, groups=4, tag="mixes")
+            z = RC.tanh_rows(Fn.linear(blends[:, 4 * width:], b.w_decay[0], out_dtype=F32, tag="decay1"), self.act)
+            z = Fn.linear(z, b.w_decay[1], out_dtype=F32, tag="decay2")
+            c = torch.empty(t, b.w_sides[1].in_features, dtype=self.act, device=s.device)
+            RC.time_mix(p, z, b.time_mix, meta, self.kv.state[li], c)
+        right = Fn.linear(c, b.w_sides[1], out_dtype=F32, tag="out")
+        return SH.Pending([(left, b.out_norms[0], m.left_scale), (right, b.out_norms[1], m.right_scale)])
+
+    def shifted_hidden(self, meta: HB.HybridMeta):
+        """-> (residual before the last layer's outputs, those outputs)."""
+        cfg, st = self.cfg, self.kv.shift
+        x = SH.embed_bigram(meta, self.w.embed, cfg.embedding_scale, self.w.bigram, cfg.bigram, st)
+        pending = None
+        for li, b in enumerate(self.w.layers):
+            x, h, s, blends = SH.shifted_norm(x, pending, b.norm, cfg.norm_eps, self.width, self.act, b.shift, b.mu, st, li, meta)
+            if self.on_layer is not None and li:
+                self.on_layer(li - 1, x.clone())
+            pending = self.sides(li, s, blends, meta)
+            if cfg.layers[li].mlp is not None:
+                pending.ff = self.feed_forward(li, h)
+        if self.on_layer is not None:
+            self.on_layer(len(self.w.layers) - 1, SH.shifted_norm(x, pending, self.w.norm, cfg.norm_eps, self.width, self.act)[0])
+        SH.commit(st, meta)
+        return x, pending
 
     def streams_hidden(self, meta: HB.HybridMeta):
         """-> (streams before the last sublayer's output, (that output, how it enters them))."""
@@ -507,10 +655,12 @@ class HybridModel(Decoder):
 
     def forward_hidden(self, meta: HB.HybridMeta):
         """-> (residual before the last layer's output, that output), both [T, W] fp32: the sum is formed where it is normed.
-        Post-norm blocks: (residual, None); streams blocks: see `streams_hidden`."""
+        Post-norm blocks: (residual, None); streams and shifted blocks: see `streams_hidden`, `shifted_hidden`."""
         cfg = self.cfg
         if cfg.block == "streams":
             return self.streams_hidden(meta)
+        if cfg.block == "shifted":
+            return self.shifted_hidden(meta)
         if cfg.block == "post_norm":
             h = torch.empty(meta.token_ids.shape[0], self.width, dtype=self.act, device=self.device)
             x = HB.embed_scaled(meta.token_ids, self.w.embed, cfg.embedding_scale, h)
@@ -531,6 +681,10 @@ class HybridModel(Decoder):
         x, y = X
         if self.cfg.block == "streams":
             return HB.stream_norm(x, *y, self.read_sum, self.w.norm, self.w.norm_b, self.cfg.norm_eps, self.width, self.act, rows=rows)
+        if self.cfg.block == "shifted":
+            if rows is None:
+                rows = torch.arange(x.shape[0], device=x.device)
+            return SH.shifted_norm(x, y, self.w.norm, self.cfg.norm_eps, self.width, self.act, rows=rows)[1]
         return HB.add_layer_norm(x, y, self.w.norm, self.cfg.norm_eps, self.width, self.act, rows=rows,
                                  center=self.cfg.block == "parallel")
 

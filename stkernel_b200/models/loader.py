@@ -31,7 +31,7 @@ import torch
 from ..config import FP8_BLOCK, ModelConfig
 from ..ops import reference as R
 from .registry import family_of, load_model_config  # noqa: F401
-from .sources import WeightSource
+from .sources import WeightSource, fits
 from .weights import weight_shapes
 
 _DTYPES = {"F32": (torch.float32, 4), "F16": (torch.float16, 2), "BF16": (torch.bfloat16, 2), "I64": (torch.int64, 8),
@@ -191,7 +191,7 @@ class CheckpointSource(WeightSource):
             out = R.dequant_mxfp4(w.view(torch.uint8).to(device), scale.view(torch.uint8).to(device))
         else:
             out = w.to(device)
-        if tuple(out.shape) != tuple(shape):
+        if not fits(out.shape, shape):
             raise ValueError(f"{name}: checkpoint shape {tuple(out.shape)} != expected {tuple(shape)}")
         return out
 

@@ -13,8 +13,8 @@ from typing import Any, Callable, Dict, Mapping, Optional, Tuple
 
 import torch
 
-from ..config import (ConfigError, EngineConfig, domilix_config_from_json, fanulix_config_from_json, model_config_from_hf,
-                      timalorn_config_from_json)
+from ..config import (ConfigError, EngineConfig, domilix_config_from_json, fanulix_config_from_json, fogizen_config_from_json,
+                      model_config_from_hf, timalorn_config_from_json)
 
 
 @dataclass(frozen=True)
@@ -107,6 +107,8 @@ _HYBRID_SOURCES = ("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", 
 _MECHANISM_SOURCES = {"attention": ("window_attention.cu", "window_attention_tc.cu"), "mlstm": ("mlstm.cu",), "dense": (),
                       "latent_attention": ("latent_attention.cu", "latent_tokens_tc.cu", "latent_prompt_tc.cu"),
                       "grouped_attention": ("window_attention.cu", "latent_prompt_tc.cu", "grouped_attention.cu"),
+                      "talking_attention": ("talking_attention.cu",),
+                      "time_mix": ("linear_scan.cu", "retention.cu", "time_mix.cu"), "token_shift": ("token_shift.cu",),
                       "retention": ("linear_scan.cu", "retention.cu"), "mamba2": ("linear_scan.cu", "mamba2.cu"),
                       "moe": ("moe.cu", "moe_plain.cu", "gate_cluster.cu")}
 
@@ -127,6 +129,7 @@ ARCHITECTURES: Dict[str, Callable[..., Any]] = {
     "Timalorn": timalorn_config_from_json,
     "Domilix": domilix_config_from_json,
     "Fanulix": fanulix_config_from_json,
+    "Fogizen": fogizen_config_from_json,
 }
 
 

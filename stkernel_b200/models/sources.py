@@ -2,13 +2,21 @@
 from __future__ import annotations
 
 import hashlib
-from typing import Dict, Tuple
+from typing import Dict, Optional, Sequence, Tuple
 
 import torch
 
 
+RANDOM_EXTENT = 32           # of an extent that only a checkpoint could tell
+
+
+def fits(shape: Sequence[int], want: Sequence[Optional[int]]) -> bool:
+    """Whether a tensor's shape is the wanted one (None: any extent)."""
+    return len(shape) == len(want) and all(w is None or s == w for s, w in zip(shape, want))
+
+
 class WeightSource:
-    """Hands out fp32 master tensors by checkpoint name."""
+    """Hands out fp32 master tensors by checkpoint name.  An extent of None in a wanted shape is whatever the source has."""
 
     def get(self, name: str, shape: Tuple[int, ...], device) -> torch.Tensor:
         raise NotImplementedError
@@ -20,7 +28,7 @@ class DictSource(WeightSource):
 
     def get(self, name, shape, device):
         t = self.t[name]
-        assert tuple(t.shape) == tuple(shape), (name, t.shape, shape)
+        assert fits(t.shape, shape), (name, t.shape, shape)
         return t.to(device)
 
 
@@ -39,6 +47,7 @@ class RandomSource(WeightSource):
 
     def get(self, name, shape, device):
         dev = torch.device(device)
+        shape = tuple(RANDOM_EXTENT if n is None else n for n in shape)
         g = self._gen(name, dev)
         if name.endswith("tid2eid"):
             return torch.randint(0, 1 << 30, shape, generator=g, device=dev, dtype=torch.int64)
@@ -55,4 +64,12 @@ class RandomSource(WeightSource):
             return noise + torch.eye(shape[0], device=dev)                     # residual streams mostly stay themselves
         if ".hc" in name or name.endswith(".dt_bias"):
             return noise + (0.5 if ".hc" in name else -2.0)
+        if name.endswith(".talk"):
+            return noise + torch.eye(shape[0], device=dev)                     # heads mostly keep their own scores
+        if name.endswith(".mix.right.w0"):
+            return noise - 4.0                                                 # decays near one
+        if name.endswith((".q.norm", ".k.norm", ".left.out", ".right.out")):
+            return torch.ones(shape, device=dev)
+        if name.endswith((".shift", ".mu.r", ".mu.k", ".mu.v", ".mu.g", ".mu.w")):
+            return noise + 0.3
         return noise

@@ -193,7 +193,7 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
             _lib.call("stk_skinny_linear_fused", lw.w, lw.w.stride(0), 1 if lw.is_fp8 else 0, lw.scale,
                       lw.scale.stride(0) if lw.is_fp8 else 0, x, x.stride(0), o, o.stride(0) if o is not None else 0, t0, n0, k0,
                       0, _lib.sm_count(), norm[0] if norm is not None else None, float(norm[1]) if norm is not None else 0.0,
-                      ll.ctx if ll is not None else None, 0, None, None, None, None, 0, None, None, 0, 0, 0, 0, 0.0,
+                      ll.ctx if ll is not None else None, 0, None, None, None, None, 0, None, None, 0, 0, 1, 1, 0, 0, 0.0,
                       _lib.status_buffer(), _lib.stream())
             return LLPending(ll, t0, n0, x.device) if ll is not None else o
     if norm is not None:
@@ -299,10 +299,10 @@ SCORING = {"sigmoid": 0, "sqrtsoftplus": 1, "softmax_topk": 2}
 
 
 def gate_route(x: torch.Tensor, w_gate: LinearWeight, bias, top_k: int, scoring: str, renorm: bool, scaling: float,
-               tid2eid=None, token_ids=None, always: int = 0):
+               tid2eid=None, token_ids=None, always: int = 0, groups: int = 1, keep: int = 1):
     """Router gate projection and expert selection in one launch for decode-sized batches (the CTA that finishes the
     projection last routes the tokens); returns (ids i32 [T, k + always], weights f32 likewise) or None when that kernel does
-    not apply (the caller then runs the projection and the router separately).  always: see `moe.router`."""
+    not apply (the caller then runs the projection and the router separately).  always, groups, keep: see `moe.router`."""
     t, k = x.shape
     e = w_gate.w.shape[0]
     if not _skinny_ok(x, t, k, w_gate.is_fp8) or e > 512 or top_k + always > 32:
@@ -316,7 +316,7 @@ def gate_route(x: torch.Tensor, w_gate: LinearWeight, bias, top_k: int, scoring:
             and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and _gate_cluster_ok()):
         # one 16-CTA cluster: the logits meet in distributed shared memory instead of global memory
         _lib.call("stk_gate_route_cluster", w, w.stride(0), x, x.stride(0), t, e, k, bias, tid2eid, token_ids, vocab, ids,
-                  wts, top_k, always, SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(),
+                  wts, top_k, always, groups, keep, SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(),
                   _lib.stream())
         return ids, wts
     cnt = _route_counters.get(dev.index)
@@ -325,7 +325,7 @@ def gate_route(x: torch.Tensor, w_gate: LinearWeight, bias, top_k: int, scoring:
     logits = scratch("gate.logits", (t, e), F32, dev, zero=True)      # zero on entry, left zero by the kernel
     _lib.call("stk_skinny_linear_fused", w_gate.w, w_gate.w.stride(0), 1 if w_gate.is_fp8 else 0, w_gate.scale,
               w_gate.scale.stride(0) if w_gate.is_fp8 else 0, x, x.stride(0), logits, logits.stride(0), t, e, k, 1,
-              _lib.sm_count(), None, 0.0, None, 2, cnt, bias, tid2eid, token_ids, vocab, ids, wts, top_k, always,
+              _lib.sm_count(), None, 0.0, None, 2, cnt, bias, tid2eid, token_ids, vocab, ids, wts, top_k, always, groups, keep,
               SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(), _lib.stream())
     return ids, wts
 

@@ -285,6 +285,16 @@ def out_offset(mixer_dim: int) -> int:
     return (mixer_dim + 15) // 16 * 16
 
 
+def xielu_rows(p: torch.Tensor, ff: int, act: Tuple[float, float], width: int) -> torch.Tensor:
+    """xIELU of p[:, :ff] in p's type, zero-padded to `width` columns.  act: the factors of the positive and the negative side."""
+    t = p.shape[0]
+    if not p.is_cuda:
+        return torch.nn.functional.pad(R.xielu(p[:, :ff], *act), (0, width - ff)).to(p.dtype)
+    out = torch.empty(t, width, dtype=p.dtype, device=p.device)
+    _lib.call("stk_xielu", p, p.stride(0), ff, float(act[0]), float(act[1]), out, out.stride(0), width, _is32(p), t, _lib.stream())
+    return out
+
+
 def join_glu(proj: torch.Tensor, out: torch.Tensor, mixer_dim: int, glu: Optional[Tuple[int, int, int]],
              act: str = "silu") -> None:
     """out[:, out_offset(mixer_dim):] = act(gate) * up with (gate, up) at columns glu[0], glu[1] of proj, glu[2] wide (None:

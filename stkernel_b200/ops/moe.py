@@ -71,20 +71,20 @@ class ExpertWeights:
 
 
 def router(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str, renorm: bool, scaling: float,
-           tid2eid: Optional[torch.Tensor] = None, token_ids: Optional[torch.Tensor] = None, always: int = 0
-           ) -> Tuple[torch.Tensor, torch.Tensor]:
+           tid2eid: Optional[torch.Tensor] = None, token_ids: Optional[torch.Tensor] = None, always: int = 0,
+           groups: int = 1, keep: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
     """fp32 gate logits [T, E] -> (expert ids i32 [T, k + always], weights f32 likewise); always: experts E, E + 1, ... that every
-    token takes with weight 1, behind the k chosen ones."""
+    token takes with weight 1, behind the k chosen ones; groups, keep: see `reference.route`."""
     t, e = logits.shape
     if not logits.is_cuda:
         hash_ids = tid2eid[token_ids.long()] if tid2eid is not None else None
-        ids, w = R.route(logits, bias, top_k, scoring, renorm, scaling, hash_ids)
+        ids, w = R.route(logits, bias, top_k, scoring, renorm, scaling, hash_ids, groups, keep)
         more = torch.arange(e, e + always, dtype=I32).expand(t, -1)
         return torch.cat([ids, more], 1), torch.cat([w, torch.ones(t, always)], 1)
     ids = torch.empty(t, top_k + always, dtype=I32, device=logits.device)
     w = torch.empty(t, top_k + always, dtype=F32, device=logits.device)
     vocab = tid2eid.shape[0] if tid2eid is not None else 0
-    _lib.call("stk_router", logits, logits.stride(0), bias, tid2eid, token_ids, vocab, ids, w, t, e, top_k, always,
+    _lib.call("stk_router", logits, logits.stride(0), bias, tid2eid, token_ids, vocab, ids, w, t, e, top_k, always, groups, keep,
               SCORING[scoring], 1 if renorm else 0, float(scaling), _lib.status_buffer(), _lib.stream())
     return ids, w
 
@@ -152,15 +152,16 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, ew: E
 
 
 # ----------------------------------------------------------------------------
-# experts without a gate, in the compute type
+# experts in the compute type
 # ----------------------------------------------------------------------------
-ACTS = {"relu2": 1, "gelu": 2}
+ACTS = {"relu2": 1, "gelu": 2, "silu": 3}
 
 
 @dataclass
 class PlainExperts:
     """y = W_down act(W_up x) per expert: up [E, F, K], down [E, W, F], bf16 or fp32, K and F padded to whole 16-byte units.
-    act: "relu2" (relu squared) or "gelu" (exact)."""
+    act: "relu2" (relu squared), "gelu" (exact), or "silu": up [E, 2 F, K] holds rows of W_gate and W_up in turns, y = W_down
+    (silu(W_gate x) * W_up x)."""
     up: torch.Tensor
     down: torch.Tensor
     act: str = "relu2"
@@ -181,7 +182,7 @@ class ExpertRows:
 def plain_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, ex: PlainExperts) -> ExpertRows:
     """x [T, K] through its chosen experts ids [T, k]; the weighted sum is left to the consumer."""
     t, k = ids.shape
-    n_pairs, (e_n, inter, width), out_w = t * k, ex.up.shape, ex.down.shape[1]
+    n_pairs, (e_n, rows, width), (out_w, inter) = t * k, ex.up.shape, ex.down.shape[1:]
     if not x.is_cuda:
         return ExpertRows(R.plain_experts(x, ids, ex.up, ex.down, x.dtype, ex.act), None, weights)
     st, f32, code = _lib.stream(), 1 if x.dtype == F32 else 0, ACTS[ex.act]
@@ -197,11 +198,11 @@ def plain_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, ex:
         act = scratch("moe.plain.act", (n_pairs, inter), BF16, dev)
         y = torch.empty(n_pairs, out_w, dtype=BF16, device=dev)
         _lib.call("stk_expert_gather", x, x.stride(0), sorted_p, k, xs, width, n_pairs, st)
-        for a, w, o, n, kk, f in ((xs, ex.up, act, inter, width, code), (act, ex.down, y, out_w, inter, 0)):
-            _lib.call("stk_experts", a, n_pairs, w, offsets, e_n, n, kk, o, n, f, _lib.sm_count(), _lib.status_buffer(), st)
+        for a, w, o, n, kk, f in ((xs, ex.up, act, rows, width, code), (act, ex.down, y, out_w, inter, 0)):
+            _lib.call("stk_experts", a, n_pairs, w, offsets, e_n, n, kk, o, o.shape[1], f, _lib.sm_count(), _lib.status_buffer(), st)
         return ExpertRows(y, pair_row, weights)
     act = torch.empty(n_pairs, inter, dtype=x.dtype, device=x.device)
     y = torch.empty(n_pairs, out_w, dtype=x.dtype, device=x.device)
-    _lib.call("stk_expert_rows", x, x.stride(0), k, ex.up, ids, e_n, act, inter, inter, inter, width, code, f32, n_pairs, st)
+    _lib.call("stk_expert_rows", x, x.stride(0), k, ex.up, ids, e_n, act, inter, rows, rows, width, code, f32, n_pairs, st)
     _lib.call("stk_expert_rows", act, inter, 1, ex.down, ids, e_n, y, out_w, out_w, out_w, inter, 0, f32, n_pairs, st)
     return ExpertRows(y, None, weights)

@@ -1,5 +1,6 @@
-"""Linear recurrences with a scalar decay per head and token, S <- a S + k v^T, o = S^T q (state fp32): retention (fixed decay, rotated
-queries and keys) and Mamba-2 (decay and input weight from a step size, operands behind a short causal convolution).
+"""Linear recurrences S <- a S + k v^T, o = S^T q (state fp32).  With a scalar decay per head and token: retention (fixed decay, rotated
+queries and keys) and Mamba-2 (decay and input weight from a step size, operands behind a short causal convolution).  With a decay
+per key channel and a bonus for the current token: time mixing.
 
 Short spans and float32 models run token by token (`*_scan`); longer spans of bf16 models in chunks on the tensor cores
 (`stk_linear_chunks`, common to both).  What enters the recurrence in fp32 (rotated queries and keys, decays, weighted values, the
@@ -14,6 +15,7 @@ import torch
 
 from . import _lib
 from . import reference as R
+from .functional import cpu_act_dtype
 from .hybrid import HybridMeta, _is32, out_offset
 from .scratch import scratch
 
@@ -91,8 +93,65 @@ def retention(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, a
         rot = scratch("scan.rotated", (t, 4, h * d8), BF16, p.device)
         _lib.call("stk_rotate_qk", p, p.stride(0), q_off, k_off, a.freq, pairs, scale, meta.positions, rot, h, d, d8, t, _lib.stream())
         _chunks((rot[:, 0], rot[:, 1], rot[:, 2], rot[:, 3], 4 * h * d8, d8, d8), p, v_off, 1, a.log_decay, None, None, meta, S, o)
-    _lib.call("stk_retention_finish", o, float(a.eps), meta.tok_req, meta.positions, p, p.stride(0), g_off, float(a.out_scale), out,
+    _lib.call("stk_retention_finish", o, float(a.eps), None, meta.tok_req, meta.positions, p, p.stride(0), g_off, float(a.out_scale), out,
               out.stride(0), left, col, out.shape[1], _is32(p), h, v, t, _lib.stream())
+
+
+# ----------------------------------------------------------------------------
+# time mixing
+# ----------------------------------------------------------------------------
+@dataclass
+class TimeMixParams:
+    heads: int
+    dim: int
+    np: int                        # columns of a projection (heads * dim, padded)
+    w0: torch.Tensor               # [heads * dim] fp32: added to the decay's projection
+    bonus: torch.Tensor            # [heads * dim] fp32
+    norm: torch.Tensor             # [heads * dim] fp32
+    eps: float
+
+
+def tanh_pair(device) -> bool:
+    """Whether a bf16 model on this device takes tanh as high part and remainder (the CPU path of a model with bf16 weights does so
+    only when its activations are bf16 as well)."""
+    return torch.device(device).type == "cuda" or cpu_act_dtype() == BF16
+
+
+def tanh_rows(z: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """tanh(z [T, n] fp32): [T, n] in fp32 models; in bf16 models its high part and remainder side by side, [T, 2 n]."""
+    t, n = z.shape
+    pair = dtype == BF16
+    if not z.is_cuda:
+        y = torch.tanh(z)
+        hi = y.to(dtype)
+        return torch.cat([hi, (y - hi.to(F32)).to(dtype)], 1) if pair else y
+    out = torch.empty(t, 2 * n if pair else n, dtype=dtype, device=z.device)
+    _lib.call("stk_tanh_rows", z, z.stride(0), n, out, _is32(out), t, _lib.stream())
+    return out
+
+
+def time_mix(p: torch.Tensor, z: torch.Tensor, a: TimeMixParams, meta: HybridMeta, state: Tuple[torch.Tensor], out: torch.Tensor) -> None:
+    """p [T, 4 * np]: r, k, v and the gate as projected; z [T, >= heads * dim] fp32: the decay's projection, log w = -exp(z + w0).
+    Runs the step's tokens through the recurrence (state updated) and writes norm(o) * weight * silu(gate) into
+    out[:, : heads * dim], zeros behind it."""
+    t = p.shape[0]
+    h, d, n = a.heads, a.dim, a.heads * a.dim
+    S, = state
+    if not p.is_cuda:
+        r, k, v = (p[:, i * a.np:i * a.np + n].reshape(t, h, d) for i in range(3))
+        log_decay = -torch.exp(z[:, :n] + a.w0).view(t, h, d)
+        o = R.bonus_scan(r, k, v, log_decay, a.bonus.view(h, d), meta.tok_req, meta.positions, S)
+        gate = torch.nn.functional.silu(p[:, 3 * a.np:3 * a.np + n].to(F32))
+        out[:, n:] = 0
+        out[:, :n] = (R.unit_rms(o, a.eps).flatten(1) * a.norm * gate).to(out.dtype)
+        return
+    o = scratch("scan.out", (t, n), F32, p.device)
+    chunked = False
+    if not chunked or meta.min_span < CHUNK_SPAN:
+        _lib.call("stk_time_mix_scan", p, p.stride(0), a.np, z, z.stride(0), a.w0, a.bonus, meta.query_start, meta.req_rows, meta.start_pos,
+                  meta.n_req, S, o, h, d, _is32(p), 1, (CHUNK_SPAN - 1) if chunked else 1 << 30, t, _lib.stream())
+    _lib.call("stk_retention_finish", o, float(a.eps), a.norm, meta.tok_req, meta.positions, p, p.stride(0), 3 * a.np, 1.0, out, out.stride(0),
+              0, 0, out.shape[1], _is32(p), h, d, t, _lib.stream())
 
 
 # ----------------------------------------------------------------------------

@@ -419,9 +419,10 @@ def router_scores(logits: torch.Tensor, scoring: str) -> torch.Tensor:
 
 
 def route(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scoring: str, renorm: bool,
-          scaling: float, hash_ids: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+          scaling: float, hash_ids: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
     """-> (expert ids [T, k] int32, weights [T, k] fp32).  Selection uses score+bias,
-    weights use the unbiased score (except "softmax_topk").  hash_ids [T, k] (already looked up) overrides selection."""
+    weights use the unbiased score (except "softmax_topk").  hash_ids [T, k] (already looked up) overrides selection.
+    groups > 1: only experts of the `keep` groups with the largest sums of two selection scores can be selected."""
     scores = router_scores(logits, scoring)
     if scoring == "softmax_topk":
         # the bias belongs to the logits: the softmax over the chosen ones sees it too
@@ -432,6 +433,11 @@ def route(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, scorin
         ids = hash_ids.long()
     else:
         sel = scores + bias.to(F32)[None] if bias is not None else scores
+        if groups > 1:
+            best = sel.view(sel.shape[0], groups, -1).topk(2, -1).values.sum(-1)
+            kept = torch.argsort(best, dim=-1, descending=True, stable=True)[:, :keep]
+            shut = torch.ones_like(best, dtype=torch.bool).scatter_(1, kept, False)
+            sel = sel.masked_fill(shut.repeat_interleave(sel.shape[1] // groups, 1), float("-inf"))
         # ties broken toward the lower expert id
         ids = torch.argsort(sel, dim=-1, descending=True, stable=True)[:, :top_k]
     w = torch.gather(scores, 1, ids)
@@ -722,7 +728,9 @@ def latent_attention(qa: torch.Tensor, qr: torch.Tensor, rot_off: int, positions
 
 
 def expert_act(z: torch.Tensor, act: str) -> torch.Tensor:
-    """"relu2" (relu squared) or "gelu" (exact), fp32."""
+    """"relu2" (relu squared), "gelu" (exact) or "silu" (columns of gate and value in turns, half as many result), fp32."""
+    if act == "silu":
+        return torch.nn.functional.silu(z[..., 0::2]) * z[..., 1::2]
     return torch.relu(z) ** 2 if act == "relu2" else torch.nn.functional.gelu(z)
 
 
@@ -842,3 +850,66 @@ def keep_conv_inputs(x: torch.Tensor, tok_req, positions, last_pos, ring: torch.
         r, p = int(tok_req[t]), int(positions[t])
         if r >= 0 and p >= 0 and p > int(last_pos[t]) - keep:
             ring[r, p % keep] = x[t].to(ring.dtype)
+
+
+# ----------------------------------------------------------------------------
+# talking-heads attention, time mixing, xIELU
+# ----------------------------------------------------------------------------
+def talking_kv_insert(k: torch.Tensor, v: torch.Tensor, k_col: int, kp: int, vp: int, positions, tok_req, table, cache) -> None:
+    """k [T, G, D], v [T, G, V] -> cache [pages, PAGE, row]: every head's value in vp columns, then every head's key in kp columns."""
+    page_rows = cache.shape[1]
+    for t in range(k.shape[0]):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        pg = int(table[r, p // page_rows])
+        if pg < 0:
+            continue
+        dst = cache[pg, p % page_rows]
+        dst.zero_()
+        dst[:k_col].view(-1, vp)[:, :v.shape[-1]] = v[t].to(cache.dtype)
+        dst[k_col:].view(-1, kp)[:, :k.shape[-1]] = k[t].to(cache.dtype)
+
+
+def talking_attention(q: torch.Tensor, vdim: int, vp: int, groups: int, k_col: int, positions, tok_req, table, cache, scale: float, chunk: int,
+                      sink: Optional[torch.Tensor]) -> torch.Tensor:
+    """Mixed queries q [T, H, kv_heads * kp] against the cached rows of each token's chunk (0: the whole context) -> [T, H, V] fp32."""
+    t_n, h, _ = q.shape
+    page_rows = cache.shape[1]
+    out = torch.zeros(t_n, h, vdim, dtype=F32)
+    for t in range(t_n):
+        r, p = int(tok_req[t]), int(positions[t])
+        if r < 0 or p < 0:
+            continue
+        at = torch.arange(p // chunk * chunk if chunk else 0, p + 1)
+        rows = cache[table[r, at // page_rows].long(), at % page_rows].to(F32)
+        s = q[t].to(F32) @ rows[:, k_col:].t() * scale
+        if sink is not None:
+            s = torch.cat([s, sink[:, None]], -1)
+        w = torch.softmax(s, -1)[:, :at.numel()]
+        v = rows[:, :k_col].view(-1, groups, vp)[..., :vdim]
+        out[t] = torch.einsum("ghn,ngv->ghv", w.view(groups, h // groups, -1), v).reshape(h, vdim)
+    return out
+
+
+def bonus_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, u: torch.Tensor, tok_req, positions,
+               S: torch.Tensor) -> torch.Tensor:
+    """One step's tokens through o = (S + diag(u) k v^T)^T r, S <- diag(exp(log_decay)) S + k v^T per head.  r, k, log_decay [T, H, D],
+    v [T, H, V], u [H, D], state S [rows, H, D, V] updated in place; a span that starts at position 0 starts from zeros."""
+    out = torch.zeros(v.shape, dtype=F32)
+    for t in range(r.shape[0]):
+        n, p = int(tok_req[t]), int(positions[t])
+        if n < 0 or p < 0:
+            continue
+        if p == 0:
+            S[n].zero_()
+        new = k[t].to(F32)[:, :, None] * v[t].to(F32)[:, None, :]
+        out[t] = torch.einsum("hdv,hd->hv", S[n] + u[:, :, None] * new, r[t].to(F32))
+        S[n] = torch.exp(log_decay[t])[:, :, None] * S[n] + new
+    return out
+
+
+def xielu(z: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    """a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise."""
+    z = z.to(F32)
+    return torch.where(z > 0, a * z * z, b * (torch.expm1(z.clamp(max=0.0)) - z)) + 0.5 * z

@@ -29,6 +29,8 @@ from ..config import FULL_CONTEXT, HybridConfig, ModelConfig, attention_part, re
 from ..ops.cache import PAGE, PagedCache
 from ..ops.grouped import grouped_row
 from ..ops.latent import latent_row
+from ..ops.shifted import shift_state
+from ..ops.talking import talking_row
 from .planning import dcp_owner
 
 
@@ -356,6 +358,10 @@ class HybridKVManager(CacheManager):
     * grouped-attention layers: paged rows `[kv_heads, PAGE, row]` of value and key (`ops/grouped.py`), in the full-context group.
     * mLSTM layers: per request row the matrix memory `[heads, dim, vdim]`, the normaliser `[heads, dim]` and the running
       maximum `[heads]`, fp32.  Nothing is cleared when a row changes hands: a span that starts at position 0 reads zeros.
+    * talking-heads attention: paged rows `[PAGE, row]` of all heads' values and keys (`ops/talking.py`).  Chunks of n positions use the
+      page group of a window of n, which holds whatever a chunk can see.
+    * time-mixing layers: the matrix state as for retention.  "shifted" blocks: per request row the last token, and per layer the last
+      norm output and shifted row (`ops/shifted.py`).
     * retention and Mamba-2 layers: per request row the matrix state `[heads, dim, vdim]` in fp32, and for Mamba-2 the last inputs
       of the convolution `[taps - 1, channels]` as projected (position p at p mod taps - 1); not cleared either.
 
@@ -393,6 +399,9 @@ class HybridKVManager(CacheManager):
             elif m is not None and m.kind == "grouped_attention":
                 self.kv_cache[li] = torch.zeros(self.full.num_pages, m.kv_heads, PAGE, grouped_row(m.dim, m.vdim)[0], dtype=dt,
                                                 device=self.device)
+            elif m is not None and m.kind == "talking_attention":
+                g = self.by_window[m.window]
+                self.kv_cache[li] = torch.zeros(g.num_pages, PAGE, talking_row(m.kv_heads, m.dim, m.vdim)[0], dtype=dt, device=self.device)
             elif m is not None and m.kv_from is None:
                 self.kv_cache[li] = torch.zeros(self.full.num_pages, PAGE, latent_row(m.kv_rank, m.rot_dim)[0], dtype=dt,
                                                 device=self.device)
@@ -401,10 +410,12 @@ class HybridKVManager(CacheManager):
             z = lambda *s: torch.zeros(max_requests, r.heads, *s, dtype=torch.float32, device=self.device)
             if r.kind == "mlstm":
                 self.state[li] = (z(r.dim, r.vdim), z(r.dim), z())
-            elif r.kind == "retention":
+            elif r.kind in ("retention", "time_mix"):
                 self.state[li] = (z(r.dim, r.vdim),)
             else:
                 self.state[li] = (z(r.state, r.vdim), torch.zeros(max_requests, r.conv - 1, r.conv_dim, dtype=dt, device=self.device))
+
+        self.shift = shift_state(len(cfg.layers), max_requests, cfg.hidden_size, self.device) if cfg.block == "shifted" else None
 
     def groups(self) -> List[GroupTable]:
         return list(self.by_window.values())
@@ -449,6 +460,8 @@ class HybridKVManager(CacheManager):
 
     def bytes_allocated(self) -> int:
         n = sum(t.numel() * t.element_size() for t in self.kv_cache.values())
+        if self.shift is not None:
+            n += sum(t.numel() * t.element_size() for t in (self.shift.token, self.shift.now, self.shift.then))
         return n + sum(t.numel() * t.element_size() for st in self.state.values() for t in st)
 
 
@@ -462,6 +475,8 @@ def hybrid_bytes_per_context_token(cfg: HybridConfig) -> int:
             n += latent_row(m.kv_rank, m.rot_dim)[0] * es
         elif m is not None and m.kind == "grouped_attention":
             n += m.kv_heads * grouped_row(m.dim, m.vdim)[0] * es
+        elif m is not None and m.kind == "talking_attention" and m.chunk is None:
+            n += talking_row(m.kv_heads, m.dim, m.vdim)[0] * es
     return n
 
 
