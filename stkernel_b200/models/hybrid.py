@@ -337,7 +337,7 @@ def build_talking_time_mix(cfg: HybridConfig, b: BlockWeights, m, get, f32, dt, 
     norms = [f32(f"mix.left.{n}.norm") for n in "qk"] if a.qk_norm else [None, None]
     b.talking = TK.TalkingParams(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.chunk or 0, cfg.norm_eps, bias, *norms,
                                  LA.split_frequencies(freq, device), f32("mix.left.talk"), f32("mix.left.sink") if a.sink else None, a.gate)
-    N, np = r.out_dim, _pad(r.out_dim)
+    N, np = r.out_dim, (r.out_dim + 127) // 128 * 128       # whole tiles of a block-diagonal product
     b.w_mixes = LinearWeight(torch.cat([_padded(get(f"mix.right.{n}"), np, _pad(W), dt) for n in "rkvg"]))
     w1, w2 = get("mix.right.w1"), get("mix.right.w2")
     if w1.shape[0] != w2.shape[1]:
@@ -612,7 +612,7 @@ class HybridModel(Decoder):
             TK.talking_attention(q, gate, b.talking, meta, table, cache, c)
         left = Fn.linear(c, b.w_sides[0], out_dtype=F32, tag="out")
         with span("time_mix", t):
-            p = Fn.linear(blends[:, :4 * width], b.w_mixes, groups=4, tag="mixes")
+            p = Fn.linear_blocks(blends[:, :4 * width], b.w_mixes, 4, tag="mixes")
             z = RC.tanh_rows(Fn.linear(blends[:, 4 * width:], b.w_decay[0], out_dtype=F32, tag="decay1"), self.act)
             z = Fn.linear(z, b.w_decay[1], out_dtype=F32, tag="decay2")
             c = torch.empty(t, b.w_sides[1].in_features, dtype=self.act, device=s.device)

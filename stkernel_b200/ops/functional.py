@@ -259,6 +259,19 @@ def linear(x, lw: LinearWeight, out: Optional[torch.Tensor] = None, out_dtype=BF
     return out
 
 
+def linear_blocks(x: torch.Tensor, lw: LinearWeight, groups: int, tag: str = "lin") -> torch.Tensor:
+    """Block-diagonal product of a few large blocks (see `linear`, groups): one launch for decode-sized batches, a product of its own
+    per block for longer ones (which then run on the widest tiles) and where a block does not fall on whole tiles."""
+    t, (n, k) = x.shape[0], lw.w.shape
+    m = n // groups
+    if not x.is_cuda or lw.w.dtype == F32 or (t <= 128 and k % 64 == 0 and m % 128 == 0):
+        return linear(x, lw, groups=groups, tag=tag)
+    out = torch.empty(t, n, dtype=x.dtype, device=x.device)
+    for g in range(groups):
+        linear(x[:, g * k:(g + 1) * k], LinearWeight(lw.w[g * m:(g + 1) * m]), out[:, g * m:(g + 1) * m], tag=tag)
+    return out
+
+
 def _linear_f32(x: torch.Tensor, lw: LinearWeight, out: Optional[torch.Tensor], groups: int = 1) -> torch.Tensor:
     """fp32 x fp32 -> fp32 on the CUDA cores (no tf32 anywhere): models that run in float32."""
     t, (n, k) = x.shape[0], lw.w.shape
