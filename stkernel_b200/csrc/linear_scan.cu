@@ -27,15 +27,10 @@ struct ChunkArgs {
   const float* fixed;                            // [H] log decay of every token, or
   const float* g; const float* w;                // [H, T] log decay and input weight
   const float* skip;                             // [H] or null
+  const float* channel;                          // or, for the states alone, [chunk][H][D] decays of whole chunks per state row
   ScanArgs s;
   int T;
 };
-
-__host__ __device__ inline int blocks16(int n) { return (n + 15) / 16; }
-constexpr int kBlockFloats = 256;                // a 16 x 16 block as a bf16 pair
-__host__ __device__ inline long long linear_slot_floats(int D, int V) {
-  return static_cast<long long>(blocks16(D)) * blocks16(V) * kBlockFloats;
-}
 
 // Tokens 2 * lane and 2 * lane + 1 of a chunk of n: running sums of the log decays (F) and input weights (w, 0 behind the chunk).
 // One token may decay by thousands and the next ones by thousandths, so sums are formed in fp64 and kept as integer part (x) and
@@ -52,7 +47,7 @@ __device__ __forceinline__ ChunkRaw load_gates(const ChunkArgs& a, int h, long l
   ChunkRaw r = {0.f, 0.f, 1.f, 1.f};
   if (a.fixed != nullptr) {
     r.g0 = r.g1 = a.fixed[h];
-  } else {
+  } else if (a.g != nullptr) {
     const long long at = static_cast<long long>(h) * a.T + t0 + 2 * lane;
     if (2 * lane < n) { r.g0 = a.g[at]; r.w0 = a.w[at]; }
     if (2 * lane + 1 < n) { r.g1 = a.g[at + 1]; r.w1 = a.w[at + 1]; }
@@ -89,7 +84,8 @@ __device__ __forceinline__ ChunkGates chunk_gates(const ChunkArgs& a, const Chun
 
 constexpr int kLsStages = 3;
 
-template <bool kPair>
+// kChannel: every state row decays by a factor of its own per chunk, and the keys come with the decays up to the end of their chunk.
+template <bool kPair, bool kChannel>
 __global__ void __launch_bounds__(256)
 linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -133,17 +129,28 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
   if (nc > 1) load(1);
   mls_commit();
   ChunkRaw raw = load_gates(a, h, q0, min(kChunk, span), lane);
+  float2 fc[4];                                                       // factors of state columns d0 + 8 j (+ 1)
+  auto load_factors = [&](int c) {
+    const float* p = a.channel + (static_cast<long long>(first + c) * s.H + h) * s.D;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) fc[j] = make_float2(d0 + 8 * j < s.D ? p[d0 + 8 * j] : 0.f, d0 + 8 * j + 1 < s.D ? p[d0 + 8 * j + 1] : 0.f);
+  };
+  if (kChannel) load_factors(0);
   const bool block_ok = vb * 64 + vw * 16 < s.V;                      // warp-uniform: its 16 rows exist
   for (int c = 0; c < nc; ++c) {
     const int n = min(kChunk, span - c * kChunk);
-    const ChunkGates g = chunk_gates(a, raw, n, lane);
-    const float w0 = g.w0 * decay_between(g.end, g.F0), w1 = g.w1 * decay_between(g.end, g.F1);      // of tokens 2 lane, 2 lane + 1
-    const float fs = expf(g.end.x + g.end.y);
+    float w0 = 1.f, w1 = 1.f, fs = 1.f;                                  // weights of tokens 2 lane, 2 lane + 1
+    if (!kChannel) {
+      const ChunkGates g = chunk_gates(a, raw, n, lane);
+      w0 = g.w0 * decay_between(g.end, g.F0);
+      w1 = g.w1 * decay_between(g.end, g.F1);
+      fs = expf(g.end.x + g.end.y);
+    }
     mls_wait<1>();
     __syncthreads();                                                    // chunk c is in, the stage before it is free
     if (c + 2 < nc) load(c + 2);
     mls_commit();
-    if (c + 1 < nc) raw = load_gates(a, h, q0 + (c + 1) * kChunk, min(kChunk, span - (c + 1) * kChunk), lane);
+    if (!kChannel && c + 1 < nc) raw = load_gates(a, h, q0 + (c + 1) * kChunk, min(kChunk, span - (c + 1) * kChunk), lane);
     // the state before this chunk
     if (block_ok) {
       float* slot = states + (static_cast<long long>(first + c) * s.H + h) * slot_f +
@@ -165,7 +172,8 @@ linear_chunk_state_kernel(const ChunkArgs a, int min_span, float* __restrict__ s
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[j][i] *= fs;
+      for (int i = 0; i < 4; ++i) acc[j][i] *= kChannel ? ((i & 1) ? fc[j].y : fc[j].x) : fs;
+    if (kChannel && c + 1 < nc) load_factors(c + 1);
     const bf16* v = tiles + c % kLsStages * kStage;
     const bf16* k = v + kTile;
 #pragma unroll
@@ -432,12 +440,25 @@ static int launch_chunks(const ChunkArgs& a, int min_span, float* states, int ma
   const size_t keys = static_cast<size_t>(kParts) * kChunk * ks, scores = static_cast<size_t>(2) * kChunk * kStStride;
   const size_t smem_o = (keys + static_cast<size_t>(kChunk) * kVs + (keys > scores ? keys : scores)) * 2;
   if (smem_o > 220 * 1024) return -5;
-  if (cudaFuncSetAttribute(linear_chunk_state_kernel<kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, 84 * 1024) != cudaSuccess ||
+  if (cudaFuncSetAttribute(linear_chunk_state_kernel<kPair, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 84 * 1024) != cudaSuccess ||
       cudaFuncSetAttribute(linear_chunk_out_kernel<kPair, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess)
     return -3;
-  launch_pdl(linear_chunk_state_kernel<kPair>, dim3((s.V + 63) / 64, (s.D + 63) / 64, s.H * s.n_req), dim3(256), smem_s, st, a, min_span,
+  launch_pdl(linear_chunk_state_kernel<kPair, false>, dim3((s.V + 63) / 64, (s.D + 63) / 64, s.H * s.n_req), dim3(256), smem_s, st, a, min_span,
              states);
   launch_pdl(linear_chunk_out_kernel<kPair, COLS>, dim3((s.V + COLS - 1) / COLS, max_chunks, s.H), dim3(COLS * 2), smem_o, st, a, min_span,
+             states);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+int linear_states_per_channel(const bf16* kh, const bf16* kl, long long ldk, int step, int width, const bf16* v, long long ldv, int v_off,
+                              const float* channel, const ScanArgs& s, int min_span, float* states, int T, cudaStream_t st) {
+  ChunkArgs a = {};
+  a.kh = kh; a.kl = kl; a.ldqk = ldk; a.step = step; a.width = width; a.hpg = 1;
+  a.v = v; a.ldv = ldv; a.v_off = v_off; a.channel = channel; a.s = s; a.T = T;
+  const size_t smem = static_cast<size_t>(kLsStages) * 3 * kChunk * kStStride * 2;
+  if (cudaFuncSetAttribute(linear_chunk_state_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 84 * 1024) != cudaSuccess)
+    return -3;
+  launch_pdl(linear_chunk_state_kernel<true, true>, dim3((s.V + 63) / 64, (s.D + 63) / 64, s.H * s.n_req), dim3(256), smem, st, a, min_span,
              states);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
@@ -465,7 +486,7 @@ STK_API int stk_linear_chunks(const void* qh, const void* ql, const void* kh, co
   a.qh = (const bf16*)qh; a.ql = (const bf16*)ql; a.kh = (const bf16*)kh; a.kl = (const bf16*)kl;
   a.ldqk = ldqk; a.step = step; a.width = width; a.hpg = hpg;
   a.v = (const bf16*)v; a.ldv = ldv; a.v_off = v_off;
-  a.fixed = log_decay; a.g = g; a.w = w; a.skip = skip;
+  a.fixed = log_decay; a.g = g; a.w = w; a.skip = skip; a.channel = nullptr;
   a.s = ScanArgs{query_start, req_rows, start_pos, n_req, S, o, heads, dim, vdim};
   a.T = T;
   cudaStream_t st = (cudaStream_t)stream;

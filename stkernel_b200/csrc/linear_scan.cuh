@@ -22,6 +22,20 @@ struct ScanArgs {
 
 constexpr int kScanThreads = 256, kScanRows = 8;
 
+// ---- chunked form: the states before every chunk (linear_scan.cu) --------------------------------
+// A state is kept in the layout of the B operand of the output products: per block of 16 value rows x 16 state rows 32 lanes x 16 bytes of
+// high parts, then of remainders.
+__host__ __device__ inline int blocks16(int n) { return (n + 15) / 16; }
+constexpr int kBlockFloats = 256;                // a 16 x 16 block as a bf16 pair
+__host__ __device__ inline long long linear_slot_floats(int D, int V) {
+  return static_cast<long long>(blocks16(D)) * blocks16(V) * kBlockFloats;
+}
+// States of a recurrence whose state rows decay by factors of their own (channel [chunk][H][D]) from chunk to chunk: S_end = diag(f) S +
+// sum_j k_j v_j^T with keys (high parts kh, remainders kl) that already carry the decay from their token to the end of the chunk.
+int linear_states_per_channel(const __nv_bfloat16* kh, const __nv_bfloat16* kl, long long ldk, int step, int width, const __nv_bfloat16* v,
+                              long long ldv, int v_off, const float* channel, const ScanArgs& s, int min_span, float* states, int T,
+                              cudaStream_t st);
+
 // Front:
 //   float2 fill(t, pos, h, q, k)   token t at position pos, all threads; returns the decay and what its rounding left over (the same
 //                                  small error at every token would add up over many)

@@ -4,7 +4,16 @@
 //   o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,   S_t = diag(w_t) S_{t-1} + k_t v_t^T,   log w = -exp(z + w0)
 //
 //   time_mix_scan        decode rows, short spans, float32: linear_scan.cuh with the decay in the front
+//   time_mix_keys        long spans: per chunk of 64 tokens the keys with their decays up to the end of the chunk, as bf16 pairs, and the
+//                        chunk's decays; the states before every chunk follow from them (linear_states_per_channel)
+//   time_mix_out         per chunk and head the outputs, on the tensor cores
 //   tanh_rows            the decay projection's activation
+//
+// Inside a chunk the weight of token j's key for token i > j is, per channel, the product of the decays between them.  A chunk is cut
+// into four blocks of 16 tokens.  Between blocks it factors at the block borders into parts that are at most one, r~_i = r_i times
+// the decays from its block's start and k^_j = k_j times those to its block's end, with the decays of whole blocks in between.  Inside a
+// block the weighted key of a column moves on from row to row, p <- p w_i, in fp32.  Nothing is divided by a decay, so strong
+// ones underflow to zero and lose nothing.
 #define STK_PDL_CLASS 16
 #include "chunk_mma.cuh"
 #include "linear_scan.cuh"
@@ -35,6 +44,319 @@ struct TimeMixFront {
     }
   }
 };
+
+// ---- chunked form ----------------------------------------------------------------------------------
+struct TmArgs {
+  const __nv_bfloat16* proj; long long ldp; int np;
+  const float* z; long long ldz;
+  const float* w0; const float* u;
+  ScanArgs s;                                     // V = D
+};
+constexpr int kTmSub = 16, kTmBlocks = kChunk / kTmSub;
+
+__device__ __forceinline__ float tm_log_decay(const TmArgs& a, long long t, int h, int d) {
+  return -__expf(a.z[t * a.ldz + h * a.s.D + d] + a.w0[h * a.s.D + d]);
+}
+
+// keys [T][2][H * D8]: high parts, remainders; channel [chunk][H][D].  One CTA per (chunk, head); a thread takes a block's 16 tokens of a channel.
+__global__ void __launch_bounds__(256)
+time_mix_keys_kernel(const TmArgs a, int min_span, __nv_bfloat16* __restrict__ keys, int D8, float* __restrict__ channel) {
+  extern __shared__ __align__(16) float ends[];   // [4][D8]
+  __shared__ ChunkRef s_c;
+  __shared__ int s_ok;
+  pdl_wait();
+  pdl_trigger();
+  const int ci = blockIdx.x, h = blockIdx.y, D = a.s.D, n8 = a.s.H * D8;
+  if (threadIdx.x == 0) s_ok = find_chunk(a.s.query_start, a.s.n_req, min_span, ci, s_c) ? 1 : 0;
+  __syncthreads();
+  if (!s_ok) return;
+  const ChunkRef c = s_c;
+  for (int e0 = 0; e0 < kTmBlocks * D8; e0 += blockDim.x) {
+    const int e = e0 + threadIdx.x, b = e / D8, d = e - b * D8;
+    if (e >= kTmBlocks * D8) continue;
+    float sum = 0.f;
+    if (d < D)
+#pragma unroll
+      for (int i = 0; i < kTmSub; ++i)
+        if (b * kTmSub + i < c.n) sum += tm_log_decay(a, c.t0 + b * kTmSub + i, h, d);
+    ends[b * D8 + d] = sum;
+  }
+  __syncthreads();
+  for (int e0 = 0; e0 < kTmBlocks * D8; e0 += blockDim.x) {
+    const int e = e0 + threadIdx.x, b = e / D8, d = e - b * D8;
+    if (e >= kTmBlocks * D8) continue;
+    float left = 0.f;                             // decays behind the token, up to the end of the chunk
+    for (int m = kTmBlocks - 1; m > b; --m) left += ends[m * D8 + d];
+#pragma unroll
+    for (int i = kTmSub - 1; i >= 0; --i) {
+      const int n = b * kTmSub + i;
+      if (n >= c.n) continue;
+      const long long t = c.t0 + n;
+      const float k = d < D ? bf16_to_f(a.proj[t * a.ldp + a.np + h * D + d]) * __expf(left) : 0.f;
+      const __nv_bfloat16 hi = __float2bfloat16(k);
+      keys[t * 2 * n8 + h * D8 + d] = hi;
+      keys[t * 2 * n8 + n8 + h * D8 + d] = __float2bfloat16(k - bf16_to_f(hi));
+      if (d < D) left += tm_log_decay(a, t, h, d);
+    }
+    if (b == 0 && d < D) channel[(static_cast<long long>(ci) * a.s.H + h) * D + d] = __expf(left);
+  }
+}
+
+constexpr int kTmOutThreads = 256;
+struct TmOutLayout { int ks, q, k, r, kr, v, w, f, p, bytes; };                   // byte offsets
+__host__ __device__ inline TmOutLayout tm_out_layout(int D) {
+  TmOutLayout l;
+  const int Dp = blocks16(D) * 16;
+  l.ks = Dp + 8;
+  const int tile = kChunk * l.ks * 2;
+  l.q = 0;                                        // [2][64][ks] r~ as pair
+  l.k = 2 * tile;                                 // [2][64][ks] k^ as pair, later the weighted scores [2][64][72]
+  const int scores = 2 * kChunk * kStStride * 2;
+  l.r = l.k + (2 * tile > scores ? 2 * tile : scores);          // [64][ks]
+  l.kr = l.r + tile;
+  l.v = l.kr + tile;
+  l.w = l.v + tile;                               // [64][Dp] fp32 decays
+  l.f = l.w + kChunk * Dp * 4;                    // [6][Dp] fp32: decays of blocks 1, 2, 1 and 2, 0, 0 and 1, 0 to 2
+  l.p = l.f + 6 * Dp * 4;                         // [4][Dp] sums of the blocks
+  l.bytes = l.p + 4 * Dp * 4;
+  return l;
+}
+
+// An operand pair times a factor per column (columns 2 (lane & 3), + 1, and 8 further).
+__device__ __forceinline__ void tm_scale_pair(uint32_t (&hi)[4], uint32_t (&lo)[4], const float* f) {
+  const float2 f0 = *reinterpret_cast<const float2*>(f), f1 = *reinterpret_cast<const float2*>(f + 8);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi[i]));
+    const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&lo[i]));
+    const float2 g = i < 2 ? f0 : f1;
+    mls_split2((x.x + y.x) * g.x, (x.y + y.y) * g.y, hi[i], lo[i]);
+  }
+}
+
+// One CTA per (chunk, head).
+__global__ void __launch_bounds__(kTmOutThreads)
+time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ states) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  __shared__ ChunkRef s_c;
+  __shared__ int s_ok;
+  const int D = a.s.D, nd = blocks16(D), Dp = nd * 16;
+  const TmOutLayout L = tm_out_layout(D);
+  const int ks = L.ks, part = kChunk * ks;
+  __nv_bfloat16* q = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.q);
+  __nv_bfloat16* k = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.k);
+  __nv_bfloat16* ph = k;
+  __nv_bfloat16* pl = ph + kChunk * kStStride;
+  __nv_bfloat16* r = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.r);
+  __nv_bfloat16* kr = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.kr);
+  __nv_bfloat16* v = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.v);
+  float* w = reinterpret_cast<float*>(smem_raw + L.w);
+  float* f = reinterpret_cast<float*>(smem_raw + L.f);
+  float* sums = reinterpret_cast<float*>(smem_raw + L.p);
+  pdl_wait();
+  pdl_trigger();
+  const int ci = blockIdx.x, h = blockIdx.y;
+  if (threadIdx.x == 0) s_ok = find_chunk(a.s.query_start, a.s.n_req, min_span, ci, s_c) ? 1 : 0;
+  __syncthreads();
+  if (!s_ok) return;
+  const ChunkRef c = s_c;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const __nv_bfloat16* p = a.proj + c.t0 * a.ldp + h * D;
+  load_rows_async(r, ks, Dp, p, a.ldp, c.n, D, kTmOutThreads);
+  load_rows_async(kr, ks, Dp, p + a.np, a.ldp, c.n, D, kTmOutThreads);
+  load_rows_async(v, ks, Dp, p + 2 * a.np, a.ldp, c.n, D, kTmOutThreads);
+  mls_commit();
+  mls_wait<0>();
+  __syncthreads();
+  // r~ and k^ of every block, the decays themselves
+  for (int e = threadIdx.x; e < kTmBlocks * Dp; e += kTmOutThreads) {
+    const int b = e / Dp, d = e - b * Dp;
+    float g[kTmSub], sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kTmSub; ++i) g[i] = d < D && b * kTmSub + i < c.n ? tm_log_decay(a, c.t0 + b * kTmSub + i, h, d) : 0.f;
+#pragma unroll
+    for (int i = 0; i < kTmSub; ++i) {
+      const int n = b * kTmSub + i;
+      mls_split(bf16_to_f(r[n * ks + d]) * __expf(sum), q[n * ks + d], q[part + n * ks + d]);
+      w[n * Dp + d] = __expf(g[i]);
+      sum += g[i];
+    }
+    sums[b * Dp + d] = sum;
+    float left = 0.f;
+#pragma unroll
+    for (int i = kTmSub - 1; i >= 0; --i) {
+      const int n = b * kTmSub + i;
+      mls_split(bf16_to_f(kr[n * ks + d]) * __expf(left), k[n * ks + d], k[part + n * ks + d]);
+      left += g[i];
+    }
+  }
+  __syncthreads();
+  for (int d = threadIdx.x; d < Dp; d += kTmOutThreads) {
+    const float s0 = sums[d], s1 = sums[Dp + d], s2 = sums[2 * Dp + d];
+    f[d] = __expf(s1);
+    f[Dp + d] = __expf(s2);
+    f[2 * Dp + d] = __expf(s1 + s2);
+    f[3 * Dp + d] = __expf(s0);
+    f[4 * Dp + d] = __expf(s0 + s1);
+    f[5 * Dp + d] = __expf(s0 + s1 + s2);
+  }
+  // the blocks on the diagonal: four lanes per column, each four channels of every 16
+  float acc[kTmSub];
+  const int jb = warp >> 1, j = (warp & 1) * 8 + (lane >> 2), seg = lane & 3;
+#pragma unroll
+  for (int i = 0; i < kTmSub; ++i) acc[i] = 0.f;
+  for (int c0 = seg * 4; c0 < Dp; c0 += 16) {
+    auto four = [&](const __nv_bfloat16* src, float (&x)[4]) {
+      const uint2 y = *reinterpret_cast<const uint2*>(src);
+      const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.x));
+      const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.y));
+      x[0] = lo.x; x[1] = lo.y; x[2] = hi.x; x[3] = hi.y;
+    };
+    float x[4];
+    four(kr + (jb * kTmSub + j) * ks + c0, x);
+#pragma unroll
+    for (int i = 0; i < kTmSub; ++i) {
+      if (i < j) continue;
+      float y[4];
+      four(r + (jb * kTmSub + i) * ks + c0, y);
+      if (i == j) {
+#pragma unroll
+        for (int m = 0; m < 4; ++m) acc[i] = fmaf(y[m] * (c0 + m < D ? a.u[h * D + c0 + m] : 0.f), x[m], acc[i]);
+      } else {
+        const float4 wi = *reinterpret_cast<const float4*>(w + (jb * kTmSub + i) * Dp + c0);
+#pragma unroll
+        for (int m = 0; m < 4; ++m) acc[i] = fmaf(y[m], x[m], acc[i]);
+        x[0] *= wi.x; x[1] *= wi.y; x[2] *= wi.z; x[3] *= wi.w;
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kTmSub; ++i) {
+    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 1);
+    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 2);
+  }
+  __syncthreads();                                                       // the factors are in
+  // the six blocks below the diagonal, one per warp
+  uint32_t wh[4], wl[4];
+  int rb = 0, kb = 0;
+  if (warp < 6) {
+    rb = warp < 1 ? 1 : warp < 3 ? 2 : 3;
+    kb = warp - rb * (rb - 1) / 2;
+    const float* g = rb - kb == 1 ? nullptr : rb - kb == 3 ? f + 2 * Dp : kb == 0 ? f : f + Dp;
+    float x[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[n][i] = 0.f;
+    const int qo = (rb * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
+    const int ko = (kb * 16 + (lane >> 4) * 8 + (lane & 7)) * ks + ((lane >> 3) & 1) * 8;
+    for (int kk = 0; kk < nd; ++kk) {
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      mls_ldsm4(ah, q + qo + kk * 16);
+      mls_ldsm4(al, q + part + qo + kk * 16);
+      mls_ldsm4(bh, k + ko + kk * 16);
+      mls_ldsm4(bl, k + part + ko + kk * 16);
+      if (g != nullptr) tm_scale_pair(ah, al, g + kk * 16 + (lane & 3) * 2);
+      mls_mma(x[0], ah, bh[0], bh[1]);
+      mls_mma(x[1], ah, bh[2], bh[3]);
+      mls_mma(x[0], al, bh[0], bh[1]);
+      mls_mma(x[1], al, bh[2], bh[3]);
+      mls_mma(x[0], ah, bl[0], bl[1]);
+      mls_mma(x[1], ah, bl[2], bl[3]);
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) mls_split2(x[n][2 * i], x[n][2 * i + 1], wh[2 * n + i], wl[2 * n + i]);
+  }
+  __syncthreads();                                                       // k^ is done with
+  if (warp < 6) {
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int off = (rb * 16 + (lane >> 2) + i * 8) * kStStride + kb * 16 + n * 8 + (lane & 3) * 2;
+        *reinterpret_cast<uint32_t*>(ph + off) = wh[2 * n + i];
+        *reinterpret_cast<uint32_t*>(pl + off) = wl[2 * n + i];
+      }
+  }
+#pragma unroll
+  for (int i = 0; i < kTmSub; ++i) {
+    if ((i & 3) != seg) continue;
+    const int off = (jb * kTmSub + i) * kStStride + jb * kTmSub + j;
+    mls_split(i >= j ? acc[i] : 0.f, ph[off], pl[off]);
+  }
+  __syncthreads();                                                       // the weighted scores are complete
+  const bool has_state = !(a.s.start_pos[c.ri] == 0 && c.first == ci);
+  const uint4* S0 = reinterpret_cast<const uint4*>(states + (static_cast<long long>(ci) * a.s.H + h) * linear_slot_floats(D, D)) + lane;
+  for (int unit = warp; unit < 2 * nd; unit += kTmOutThreads / 32) {     // 16 columns, 32 rows
+    const int cg = unit >> 1, rh = unit & 1;
+    float o[2][2][4];
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int y = 0; y < 2; ++y)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[x][y][i] = 0.f;
+    if (has_state) {
+      const uint4* S = S0 + static_cast<long long>(cg) * nd * 64;
+#pragma unroll 4
+      for (int kk = 0; kk < nd; ++kk) {
+        const uint4 hi = __ldcs(S + kk * 64), lo = __ldcs(S + kk * 64 + 32);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int rb2 = rh * 2 + x;
+          uint32_t ah[4], al[4];
+          const int qo = (rb2 * 16 + (lane & 15)) * ks + (lane >> 4) * 8 + kk * 16;
+          mls_ldsm4(ah, q + qo);
+          mls_ldsm4(al, q + part + qo);
+          if (rb2 > 0) tm_scale_pair(ah, al, f + (2 + rb2) * Dp + kk * 16 + (lane & 3) * 2);
+          mls_mma(o[x][0], ah, hi.x, hi.y);
+          mls_mma(o[x][1], ah, hi.z, hi.w);
+          mls_mma(o[x][0], ah, lo.x, lo.y);
+          mls_mma(o[x][1], ah, lo.z, lo.w);
+          mls_mma(o[x][0], al, hi.x, hi.y);
+          mls_mma(o[x][1], al, hi.z, hi.w);
+        }
+      }
+    }
+    for (int b = 0; b <= rh * 2 + 1; ++b) {
+      uint32_t bv[4];
+      mls_ldsm4_t(bv, v + (b * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ks + cg * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int rb2 = rh * 2 + x;
+        if (b > rb2) continue;
+        uint32_t hi[4], lo[4];
+        const int off = (rb2 * 16 + (lane & 15)) * kStStride + b * 16 + (lane >> 4) * 8;
+        mls_ldsm4(hi, ph + off);
+        mls_ldsm4(lo, pl + off);
+        mls_mma(o[x][0], hi, bv[0], bv[1]);
+        mls_mma(o[x][1], hi, bv[2], bv[3]);
+        mls_mma(o[x][0], lo, bv[0], bv[1]);
+        mls_mma(o[x][1], lo, bv[2], bv[3]);
+      }
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = (rh * 2 + x) * 16 + (lane >> 2) + i * 8;
+        if (t >= c.n) continue;
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          const int col = cg * 16 + y * 8 + (lane & 3) * 2;
+          float* to = a.s.o + ((c.t0 + t) * static_cast<long long>(a.s.H) + h) * D + col;
+          if ((D & 1) == 0 && col + 1 < D) {
+            *reinterpret_cast<float2*>(to) = make_float2(o[x][y][2 * i], o[x][y][2 * i + 1]);
+          } else {
+            if (col < D) to[0] = o[x][y][2 * i];
+            if (col + 1 < D) to[1] = o[x][y][2 * i + 1];
+          }
+        }
+      }
+  }
+}
 
 // tanh of fp32 rows; kPair: bf16 high parts, then the remainders n columns further.
 template <bool kPair>
@@ -78,5 +400,33 @@ STK_API int stk_tanh_rows(const float* z, long long ldz, int n, void* out, int f
   const dim3 grid(static_cast<unsigned>((total + 255) / 256));
   if (fp32) launch_pdl(tanh_rows_kernel<false>, grid, dim3(256), 0, (cudaStream_t)stream, z, ldz, n, out, total);
   else launch_pdl(tanh_rows_kernel<true>, grid, dim3(256), 0, (cudaStream_t)stream, z, ldz, n, out, total);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// Whether `stk_time_mix_chunks` covers a head size.
+STK_API int stk_time_mix_chunks_ok(int dim) { return dim >= 1 && dim <= 128 ? 1 : 0; }
+
+// Spans of at least min_span tokens, bf16.  keys: work space [T, 2, heads * d8] bf16 (d8: dim rounded up to 8); channel: fp32
+// [max_chunks, heads, dim]; states: fp32 [max_chunks * heads * stk_linear_state_slot()]; max_chunks bounds the chunks over all requests.
+STK_API int stk_time_mix_chunks(const void* proj, long long ldp, int np, const float* z, long long ldz, const float* w0, const float* u,
+                                const int* query_start, const int* req_rows, const int* start_pos, int n_req, float* S, float* o, int heads,
+                                int dim, int min_span, void* keys, float* channel, float* states, int max_chunks, int T, void* stream) {
+  if (T <= 0 || n_req <= 0 || max_chunks <= 0) return 0;
+  if (!stk_time_mix_chunks_ok(dim) || heads < 1 || static_cast<long long>(heads) * n_req > 65535 || min_span < 1 ||
+      ((reinterpret_cast<uintptr_t>(states) | reinterpret_cast<uintptr_t>(keys)) & 15))
+    return -1;
+  const int d8 = (dim + 7) / 8 * 8, n8 = heads * d8;
+  TmArgs a;
+  a.proj = (const __nv_bfloat16*)proj; a.ldp = ldp; a.np = np; a.z = z; a.ldz = ldz; a.w0 = w0; a.u = u;
+  a.s = ScanArgs{query_start, req_rows, start_pos, n_req, S, o, heads, dim, dim};
+  cudaStream_t st = (cudaStream_t)stream;
+  __nv_bfloat16* kp = (__nv_bfloat16*)keys;
+  launch_pdl(time_mix_keys_kernel, dim3(max_chunks, heads), dim3(256), static_cast<size_t>(kTmBlocks) * d8 * sizeof(float), st, a, min_span, kp,
+             d8, channel);
+  const int rc = linear_states_per_channel(kp, kp + n8, 2ll * n8, d8, d8, a.proj, ldp, 2 * np, channel, a.s, min_span, states, T, st);
+  if (rc != 0) return rc;
+  if (cudaFuncSetAttribute(time_mix_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return -3;
+  launch_pdl(time_mix_out_kernel, dim3(max_chunks, heads), dim3(kTmOutThreads), static_cast<size_t>(tm_out_layout(dim).bytes), st, a, min_span,
+             (const float*)states);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -107,7 +107,7 @@ _HYBRID_SOURCES = ("elementwise.cu", "meta.cu", "gemm_tcgen05.cu", "skinny.cu", 
 _MECHANISM_SOURCES = {"attention": ("window_attention.cu", "window_attention_tc.cu"), "mlstm": ("mlstm.cu",), "dense": (),
                       "latent_attention": ("latent_attention.cu", "latent_tokens_tc.cu", "latent_prompt_tc.cu"),
                       "grouped_attention": ("window_attention.cu", "latent_prompt_tc.cu", "grouped_attention.cu"),
-                      "talking_attention": ("talking_attention.cu",),
+                      "talking_attention": ("talking_attention.cu", "talking_tokens_tc.cu", "talking_prompt_tc.cu"),
                       "time_mix": ("linear_scan.cu", "retention.cu", "time_mix.cu"), "token_shift": ("token_shift.cu",),
                       "retention": ("linear_scan.cu", "retention.cu"), "mamba2": ("linear_scan.cu", "mamba2.cu"),
                       "moe": ("moe.cu", "moe_plain.cu", "gate_cluster.cu")}

@@ -146,10 +146,17 @@ def time_mix(p: torch.Tensor, z: torch.Tensor, a: TimeMixParams, meta: HybridMet
         out[:, :n] = (R.unit_rms(o, a.eps).flatten(1) * a.norm * gate).to(out.dtype)
         return
     o = scratch("scan.out", (t, n), F32, p.device)
-    chunked = False
+    chunked = not _is32(p) and meta.max_span >= CHUNK_SPAN and _lib.query("stk_time_mix_chunks_ok", d) == 1
     if not chunked or meta.min_span < CHUNK_SPAN:
         _lib.call("stk_time_mix_scan", p, p.stride(0), a.np, z, z.stride(0), a.w0, a.bonus, meta.query_start, meta.req_rows, meta.start_pos,
                   meta.n_req, S, o, h, d, _is32(p), 1, (CHUNK_SPAN - 1) if chunked else 1 << 30, t, _lib.stream())
+    if chunked:
+        chunks = t // CHUNK + meta.n_req
+        keys = scratch("scan.rotated", (t, 2, h * _up8(d)), BF16, p.device)
+        channel = scratch("scan.channel", (chunks, h, d), F32, p.device)
+        ws = scratch("scan.states", (chunks * h * _lib.query("stk_linear_state_slot", d, d),), F32, p.device)
+        _lib.call("stk_time_mix_chunks", p, p.stride(0), a.np, z, z.stride(0), a.w0, a.bonus, meta.query_start, meta.req_rows, meta.start_pos,
+                  meta.n_req, S, o, h, d, CHUNK_SPAN, keys, channel, ws, chunks, t, _lib.stream())
     _lib.call("stk_retention_finish", o, float(a.eps), a.norm, meta.tok_req, meta.positions, p, p.stride(0), 3 * a.np, 1.0, out, out.stride(0),
               0, 0, out.shape[1], _is32(p), h, d, t, _lib.stream())
 

@@ -70,7 +70,7 @@ def talking_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int
         out = torch.zeros(t, h, g, kp, dtype=p.dtype)
         out[..., :d] = torch.einsum("hcj,tcjd->thcd", a.talk.view(h, g, h // g), q.view(t, g, h // g, d)).to(p.dtype)
         return out.flatten(1), p[:, g_off:g_off + h].to(F32) if a.gated else None
-    out = torch.empty(t, h * g * kp, dtype=p.dtype, device=p.device)
+    out = torch.empty(t, h * g * kp, dtype=p.dtype, device=p.device)       # whole 16-byte units: kp is a multiple of 16
     gate = torch.empty(t, h, dtype=F32, device=p.device) if a.gated else None
     _lib.call("stk_talking_prep", p, p.stride(0), q_off, k_off, v_off, g_off, a.bias, a.q_norm, a.k_norm, float(a.eps), a.freq, a.freq.shape[1],
               a.talk, meta.positions, meta.tok_req, table, table.stride(0), cache, row, k_col, kp, vp, h, g, d, v, out, gate, _is32(p), t,
@@ -91,6 +91,30 @@ def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], a: TalkingP
         out[:, h * v:] = 0
         out[:, :h * v] = o.flatten(1).to(out.dtype)
         return
-    common = (q, q.stride(0), gate, a.sink, meta.positions, meta.tok_req, table, table.stride(0), cache, row, k_col, kp, vp, h, g, v, a.chunk,
-              float(a.scale), out, out.stride(0), out.shape[1])
-    _lib.call("stk_talking_simt", *common, _is32(q), meta.first_pos, meta.last_pos, 1 << 30, t, _lib.stream())
+    shape = (row, k_col, kp, vp, h, g, v, a.chunk, float(a.scale), out, out.stride(0), out.shape[1])
+    common = (q, q.stride(0), gate, a.sink, meta.positions, meta.tok_req, table, table.stride(0), cache, *shape)
+    prompt = (not _is32(q) and meta.max_span >= PROMPT_SPAN and meta.spans is not None
+              and _lib.query("stk_talking_prompt_ok", h, g, kp, vp, v) == 1)
+    if not prompt or meta.min_span < PROMPT_SPAN:
+        max_span = PROMPT_SPAN - 1 if prompt else meta.max_span
+        if _is32(q) or _lib.query("stk_talking_tokens_ok", h, g, kp, vp, max_span) == 0:
+            _lib.call("stk_talking_simt", *common, _is32(q), meta.first_pos, meta.last_pos, max_span, t, _lib.stream())
+        else:
+            context = min(meta.max_context, table.shape[1] * PAGE)
+            keys = min(a.chunk, context) if a.chunk else context
+            splits = _lib.query("stk_talking_tokens_splits", t, h, g, kp, vp, max_span, keys, _lib.sm_count())
+            part = scratch("talking.part", (splits * t * h * (v + 2),), F32, q.device)
+            _lib.call("stk_talking_tokens", *common, meta.query_start, meta.req_rows, meta.start_pos, meta.n_req, meta.first_pos,
+                      meta.last_pos, max_span, cache.shape[0], splits, part, t, _lib.status_buffer(), _lib.stream())
+    if prompt:
+        n_rows = sum(_up(start + n - _rows_base(a.chunk, start), PROMPT_ROWS) for start, n in meta.spans if n >= PROMPT_SPAN)
+        rows = torch.empty(n_rows, row, dtype=q.dtype, device=q.device)
+        _lib.call("stk_talking_rows", meta.query_start, meta.req_rows, meta.start_pos, meta.n_req, PROMPT_SPAN, a.chunk, table, table.stride(0),
+                  cache, row, rows, n_rows, _lib.stream())
+        _lib.call("stk_talking_prompt", q, q.stride(0), gate, a.sink, rows, n_rows, *shape, meta.query_start, meta.start_pos, meta.n_req,
+                  PROMPT_SPAN, t, _lib.status_buffer(), _lib.stream())
+
+
+def _rows_base(chunk: int, start: int) -> int:
+    """First position whose row a long span starting at `start` gathers."""
+    return start // chunk * chunk // PROMPT_ROWS * PROMPT_ROWS if chunk else 0
