@@ -116,6 +116,16 @@ def streams_arm(args) -> None:
     print(json.dumps({"metric": "streams_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
 
 
+def shifted_arm(args) -> None:
+    import torch
+    from stkernel_b200.bench import hybrid_bench, shifted_bench
+    torch.cuda.set_device(0)
+    with ClockSampler(0) as clocks:
+        res = shifted_bench.run([int(x) for x in args.shifted_sizes.split(",")], beside=not args.shifted_alone)
+    print(hybrid_bench.render(res), file=sys.stderr)
+    print(json.dumps({"metric": "shifted_decoder", "data": "synthetic", "clocks": clocks.summary(), **res}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -142,7 +152,14 @@ def main() -> None:
                          "decode and per-kernel rooflines (one JSON line; table on stderr)")
     ap.add_argument("--streams-sizes", default="2048,4096", help="widths for --streams")
     ap.add_argument("--streams-alone", action="store_true", help="with --streams: without the other decoders beside it")
+    ap.add_argument("--shifted", action="store_true",
+                    help="instead of the flagship: the Fogizen decoder beside Fanulix and Domilix at equal width and depth, prefill, "
+                         "decode and per-kernel rooflines (one JSON line; table on stderr)")
+    ap.add_argument("--shifted-sizes", default="2048,4096", help="widths for --shifted")
+    ap.add_argument("--shifted-alone", action="store_true", help="with --shifted: without the other decoders beside it")
     args = ap.parse_args()
+    if args.shifted:
+        return shifted_arm(args)
     if args.streams:
         return streams_arm(args)
     if args.hybrid:

@@ -1184,7 +1184,7 @@ def shifted_stack(n_layers: int, width: int, heads: int, kv_heads: int, dim: int
 def tiny_shifted_config(**over: Any) -> HybridConfig:
     """CPU-sized Fogizen-shaped decoder: a dense layer, a mixture of experts in groups, and a layer without feed-forward."""
     both = ParallelMixer(TalkingAttentionMixer(4, 2, 20, 28, 0.21, 24, RotaryConfig(3000.0, 12, LinearScaling(2.5), interleaved=True)),
-                         TimeMixMixer(3, 20, 12), 0.5, 0.5, True)
+                         TimeMixMixer(3, 20), 0.5, 0.5, True)
     moe = MoeMlp(6, 2, 40, "silu", False, scoring="sigmoid", groups=3, keep=2, scale=1.3)
     kw: Dict[str, Any] = dict(vocab_size=300, hidden_size=88, norm_eps=2e-5, architecture="Fogizen", block="shifted",
                               bigram=BigramTable(97, 13, 5),
