@@ -475,7 +475,12 @@ xielu_kernel(const A* __restrict__ z, long long ldz, int ff, float a, float b, A
   const long long e = blockIdx.x * 256ll + threadIdx.x, t = e / per;
   if (t >= T) return;
   const int c0 = static_cast<int>(e - t * per) * 8;
-  auto f = [&](float x) { return fmaf(x, 0.5f, x > 0.f ? a * x * x : b * (expm1f(x) - x)); };
+  auto f = [&](float x) {
+    if (sizeof(A) == 4) return fmaf(x, 0.5f, x > 0.f ? a * x * x : b * (expm1f(x) - x));
+    // rounded results: exp(x) - 1 - x from its series where the difference would cancel
+    const float near = x * x * fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f), far = __expf(x) - 1.f - x;
+    return fmaf(x, 0.5f, x > 0.f ? a * x * x : b * (x > -0.25f ? near : far));
+  };
   const A* p = z + t * ldz + c0;
   A* o = out + t * ldo + c0;
   if (sizeof(A) == 2 && c0 + 8 <= ff && ((ldz | ldo) & 7) == 0) {

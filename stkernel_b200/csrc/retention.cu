@@ -139,17 +139,24 @@ rotate_qk_kernel(const RotArgs r, const int64_t* __restrict__ positions, __nv_bf
 }
 
 // out[t, col + h * V + c] = o / rms(o over the head) * weight * silu(g) * scale (weight null: 1): one warp per (token, head).  Zeros into the columns left .. col
-// and behind the last head.  NV > 0: bf16 heads of at most 128 * NV columns in whole groups of four, which stay in registers.
-template <typename A, int NV>
+// and behind the last head.  NV > 0: bf16 heads of at most 4 * LPH * NV columns in whole groups of
+// four, which stay in registers, LPH lanes per (token, head).
+template <typename A, int NV, int LPH>
 __global__ void __launch_bounds__(256)
 retention_finish_kernel(const float* __restrict__ o, float eps, const float* __restrict__ weight, const int* __restrict__ tok_req, const int64_t* __restrict__ positions,
                         const A* __restrict__ proj, long long ldp, int g_off, float scale, A* __restrict__ out, long long ldo, int left,
                         int col, int cols, int H, int V, int T) {
   pdl_wait();
   pdl_trigger();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long th = blockIdx.x * 8ll + warp;
+  const int lane = threadIdx.x & (LPH - 1);
+  const long long th = blockIdx.x * (256ll / LPH) + threadIdx.x / LPH;
   if (th >= static_cast<long long>(T) * H) return;
+  const unsigned mates = LPH == 32 ? 0xffffffffu : 0xffffu << (threadIdx.x & 16);
+  auto head_sum = [&](float v) {
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) v += __shfl_xor_sync(mates, v, o);
+    return v;
+  };
   const long long t = th / H;
   const int h = static_cast<int>(th - t * H);
   A* to = out + t * ldo;
@@ -160,28 +167,28 @@ retention_finish_kernel(const float* __restrict__ o, float eps, const float* __r
   if (NV > 0) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * 32 + lane) * 4;
+      const int c = (i * LPH + lane) * 4;
       v[i] = c < V ? *reinterpret_cast<const float4*>(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
       gu[i] = c < V ? *reinterpret_cast<const uint2*>(g + c) : make_uint2(0, 0);
     }
   }
   if (h == 0)
-    for (int c = left + lane; c < col; c += 32) st_act(to + c, 0.f);
+    for (int c = left + lane; c < col; c += LPH) st_act(to + c, 0.f);
   if (h == H - 1)
-    for (int c = col + H * V + lane; c < cols; c += 32) st_act(to + c, 0.f);
+    for (int c = col + H * V + lane; c < cols; c += LPH) st_act(to + c, 0.f);
   to += col + h * V;
   if (tok_req[t] < 0 || positions[t] < 0) {
-    for (int c = lane; c < V; c += 32) st_act(to + c, 0.f);
+    for (int c = lane; c < V; c += LPH) st_act(to + c, 0.f);
     return;
   }
   float ss = 0.f;
   if (NV > 0) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
-    const float r = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
+    const float r = scale / sqrtf(head_sum(ss) / static_cast<float>(V) + eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * 32 + lane) * 4;
+      const int c = (i * LPH + lane) * 4;
       if (c >= V) continue;
       const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu[i].x));
       const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gu[i].y));
@@ -196,9 +203,9 @@ retention_finish_kernel(const float* __restrict__ o, float eps, const float* __r
     }
     return;
   }
-  for (int c = lane; c < V; c += 32) ss = fmaf(x[c], x[c], ss);
-  const float r = scale / sqrtf(warp_sum(ss) / static_cast<float>(V) + eps);
-  for (int c = lane; c < V; c += 32) {
+  for (int c = lane; c < V; c += LPH) ss = fmaf(x[c], x[c], ss);
+  const float r = scale / sqrtf(head_sum(ss) / static_cast<float>(V) + eps);
+  for (int c = lane; c < V; c += LPH) {
     const float z = ld_act(g + c);
     st_act(to + c, x[c] * r * (weight != nullptr ? weight[h * V + c] : 1.f) * z / (1.f + expf(-z)));
   }
@@ -238,18 +245,18 @@ STK_API int stk_retention_finish(const float* o, float eps, const float* weight,
                                  int g_off, float scale, void* out, long long ldo, int left, int col, int cols, int fp32, int heads,
                                  int vdim, int T, void* stream) {
   if (T <= 0) return 0;
-  const dim3 grid(static_cast<unsigned>((static_cast<long long>(T) * heads + 7) / 8));
   cudaStream_t st = (cudaStream_t)stream;
-  const bool vec = !fp32 && vdim <= 512 && ((vdim | g_off | col) & 3) == 0 && ((ldp | ldo) & 3) == 0 &&
+  const bool vec = !fp32 && vdim <= 512 && ((vdim | g_off | col) & 3) == 0 && (reinterpret_cast<uintptr_t>(weight) & 15) == 0 && ((ldp | ldo) & 3) == 0 &&
                    ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(out)) & 7) == 0;
-#define STK_FINISH(A, NV)                                                                                                          \
-  launch_pdl(retention_finish_kernel<A, NV>, grid, dim3(256), 0, st, o, eps, weight, tok_req, positions, (const A*)proj, ldp, g_off, scale, (A*)out, \
+#define STK_FINISH(A, NV, LPH)                                                                                                     \
+  launch_pdl(retention_finish_kernel<A, NV, LPH>, dim3(static_cast<unsigned>((static_cast<long long>(T) * heads + 256 / LPH - 1) / (256 / LPH))), dim3(256), 0, st, o, eps, weight, tok_req, positions, (const A*)proj, ldp, g_off, scale, (A*)out, \
              ldo, left, col, cols, heads, vdim, T)
-  if (fp32) STK_FINISH(float, 0);
-  else if (!vec) STK_FINISH(__nv_bfloat16, 0);
-  else if (vdim <= 128) STK_FINISH(__nv_bfloat16, 1);
-  else if (vdim <= 256) STK_FINISH(__nv_bfloat16, 2);
-  else STK_FINISH(__nv_bfloat16, 4);
+  if (fp32) STK_FINISH(float, 0, 32);
+  else if (!vec) STK_FINISH(__nv_bfloat16, 0, 32);
+  else if (vdim <= 64) STK_FINISH(__nv_bfloat16, 1, 16);
+  else if (vdim <= 128) STK_FINISH(__nv_bfloat16, 1, 32);
+  else if (vdim <= 256) STK_FINISH(__nv_bfloat16, 2, 32);
+  else STK_FINISH(__nv_bfloat16, 4, 32);
 #undef STK_FINISH
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -3,7 +3,7 @@
 // A cached row holds the values of all key/value heads (vp columns each), then from k_col on their keys (kp columns each); pages are
 // [64][row].  A mixed query has G * kp columns: in the part of key/value head c the sum of talk[h, g] q_g over the heads g that read c.
 //
-//   talking_prep         one CTA per token: biases, weighted RMS norms, rotation, the token's row, mixed queries, gate logits
+//   talking_prep         one CTA per token, or a few where there are few tokens: biases, weighted RMS norms, rotation, the token's row, mixed queries, gate logits
 //   talking_simt         any size and type, fp32 arithmetic throughout: one CTA per (token, head)
 #define STK_PDL_CLASS 8
 #include "hybrid_block.cuh"
@@ -19,45 +19,47 @@ struct TalkPrepArgs {
   const float* talk;                                   // [H, H]
   const int64_t* positions; const int* tok_req; const int* table; int bt_stride;
   void* cache; int row, k_col, kp, vp;
-  int H, G, D, V;
+  int H, G, D, V, T;
   void* q; float* gate;
 };
 
-constexpr int kTkThreads = 256;
-
-// HG: heads per key/value head (their queries stay in registers while all heads' mixtures are formed), 0: any number.
+// HG: heads per key/value head (their queries stay in registers while the heads' mixtures are formed), 0: any number.  grid (T, parts): a
+// part forms the mixtures of its share of the heads; the first one also writes the cached row and the gate logits.
 template <typename A, int HG>
-__global__ void __launch_bounds__(kTkThreads)
+__global__ void __launch_bounds__(512)
 talking_prep_kernel(const TalkPrepArgs a) {
   extern __shared__ __align__(16) float sm[];
-  const int D2 = (a.D + 1) & ~1;
+  const int D2 = (a.D + 3) & ~3, H4 = (a.H + 3) & ~3;
   float* x = sm;                                       // [H + G][D2]: queries, keys
-  float* talk = x + (a.H + a.G) * D2;                  // [H][H], transposed: talk[g][h]
-  float2* cs = reinterpret_cast<float2*>(talk + ((a.H * a.H + 1) & ~1));      // [pairs]
+  float* talk = x + (a.H + a.G) * D2;                  // [heads of this part][H4]
+  const int per = (a.H + gridDim.y - 1) / gridDim.y, h0 = blockIdx.y * per, h1 = min(a.H, h0 + per);
+  float2* cs = reinterpret_cast<float2*>(talk + per * H4);      // [pairs]
   pdl_wait();
   pdl_trigger();
   const long long t = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, KD = a.G * a.kp;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, KD = a.G * a.kp, warps = blockDim.x >> 5;
+  const bool lead = blockIdx.y == 0;
   const int req = a.tok_req[t];
   const long long pos = a.positions[t];
-  A* q = reinterpret_cast<A*>(a.q) + t * a.H * KD;
+  A* q = reinterpret_cast<A*>(a.q) + t * KD;           // head h: h * T * KD further
+  const long long hstep = static_cast<long long>(a.T) * KD;
   const A* p = reinterpret_cast<const A*>(a.proj) + t * a.ldp;
-  if (a.gate != nullptr)
-    for (int h = threadIdx.x; h < a.H; h += kTkThreads) a.gate[t * a.H + h] = ld_act(p + a.g_off + h);
+  if (lead && a.gate != nullptr)
+    for (int h = threadIdx.x; h < a.H; h += blockDim.x) a.gate[t * a.H + h] = ld_act(p + a.g_off + h);
   if (req < 0 || pos < 0) {
-    for (int i = threadIdx.x; i < a.H * KD; i += kTkThreads) st_act(q + i, 0.f);
+    for (int h = h0; h < h1; ++h)
+      for (int i = threadIdx.x; i < KD; i += blockDim.x) st_act(q + h * hstep + i, 0.f);
     return;
   }
-  for (int i = threadIdx.x; i < a.pairs; i += kTkThreads) cs[i] = cos_sin_split(pos, a.freq[i], a.freq[a.pairs + i]);
-  for (int i = threadIdx.x; i < a.H * a.H; i += kTkThreads) talk[(i % a.H) * a.H + i / a.H] = a.talk[i];
-  for (int u = warp; u < a.H + a.G; u += kTkThreads / 32) {
-    const bool isq = u < a.H;
-    const A* src = p + (isq ? a.q_off + u * a.D : a.k_off + (u - a.H) * a.D);
+  const int page = a.table[static_cast<long long>(req) * a.bt_stride + pos / kTkPage];
+  for (int u0 = warp; u0 < a.H + a.G; u0 += warps) {
+    const bool isq = u0 < a.H;
+    const A* src = p + (isq ? a.q_off + u0 * a.D : a.k_off + (u0 - a.H) * a.D);
     const float* w = isq ? a.q_norm : a.k_norm;
-    float* dst = x + u * D2;
+    float* dst = x + u0 * D2;
     float s = 0.f;
-    for (int d = lane; d < a.D; d += 32) {
-      const float v = ld_act(src + d) + (a.bias != nullptr ? a.bias[u * a.D + d] : 0.f);
+    for (int d = lane; d < D2; d += 32) {
+      const float v = d < a.D ? ld_act(src + d) + (a.bias != nullptr ? a.bias[u0 * a.D + d] : 0.f) : 0.f;
       dst[d] = v;
       s = fmaf(v, v, s);
     }
@@ -66,63 +68,61 @@ talking_prep_kernel(const TalkPrepArgs a) {
       for (int d = lane; d < a.D; d += 32) dst[d] *= f * w[d];
     }
   }
+  for (int i = threadIdx.x; i < a.pairs; i += blockDim.x) cs[i] = cos_sin_split(pos, a.freq[i], a.freq[a.pairs + i]);
+  for (int i = threadIdx.x; i < (h1 - h0) * a.H; i += blockDim.x) talk[i / a.H * H4 + i % a.H] = a.talk[h0 * a.H + i];
   __syncthreads();
-  for (int e = threadIdx.x; e < (a.H + a.G) * a.pairs; e += kTkThreads) {
+  for (int e = threadIdx.x; e < (a.H + a.G) * a.pairs; e += blockDim.x) {
     const int u = e / a.pairs, i = e - u * a.pairs;
-    float* v = x + u * D2 + 2 * i;
-    const float c0 = v[0], c1 = v[1];
-    const float2 w = cs[i];
-    v[0] = c0 * w.x - c1 * w.y;
-    v[1] = c1 * w.x + c0 * w.y;
+    float2* v = reinterpret_cast<float2*>(x + u * D2 + 2 * i);
+    const float2 c = *v, w = cs[i];
+    *v = make_float2(c.x * w.x - c.y * w.y, c.y * w.x + c.x * w.y);
   }
   __syncthreads();
-  const int page = a.table[static_cast<long long>(req) * a.bt_stride + pos / kTkPage];
-  if (page >= 0) {
+  if (lead && page >= 0) {
     A* row = reinterpret_cast<A*>(a.cache) + (static_cast<long long>(page) * kTkPage + pos % kTkPage) * a.row;
-    for (int e = threadIdx.x; e < a.G * a.vp; e += kTkThreads) {
+    for (int e = threadIdx.x; e < a.G * a.vp; e += blockDim.x) {
       const int g = e / a.vp, d = e - g * a.vp;
       st_act(row + e, d < a.V ? ld_act(p + a.v_off + g * a.V + d) + (a.bias != nullptr ? a.bias[(a.H + a.G) * a.D + g * a.V + d] : 0.f) : 0.f);
     }
-    for (int e = threadIdx.x; e < KD; e += kTkThreads) {
+    for (int e = threadIdx.x; e < KD; e += blockDim.x) {
       const int g = e / a.kp, d = e - g * a.kp;
       st_act(row + a.k_col + e, d < a.D ? x[(a.H + g) * D2 + d] : 0.f);
     }
   }
-  const int hg = HG > 0 ? HG : a.H / a.G, half = a.kp >> 1;
-  for (int e = threadIdx.x; e < a.G * half; e += kTkThreads) {          // two columns of every head's mixture
-    const int c = e / half, d = (e - c * half) * 2;
-    const bool in0 = d < a.D, in1 = d + 1 < a.D;
+  // four columns of the mixtures of every other, fourth, ... head (kp is a multiple of 4)
+  const int hg = HG > 0 ? HG : a.H / a.G, quads = a.kp >> 2, items = a.G * quads;
+  const int lots = max(1, min(h1 - h0, static_cast<int>(blockDim.x) / items));
+  for (int e = threadIdx.x; e < items * lots; e += blockDim.x) {
+    const int lot = e / items, i = e - lot * items, c = i / quads, d = (i - c * quads) * 4;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     const float* qc = x + c * hg * D2 + d;
-    float q0[HG > 0 ? HG : 1], q1[HG > 0 ? HG : 1];
+    float4 qv[HG > 0 ? HG : 1];
     if (HG > 0) {
 #pragma unroll
-      for (int g = 0; g < HG; ++g) {
-        q0[g] = in0 ? qc[g * D2] : 0.f;
-        q1[g] = in1 ? qc[g * D2 + 1] : 0.f;
-      }
+      for (int g = 0; g < HG; ++g) qv[g] = d < a.D ? *reinterpret_cast<const float4*>(qc + g * D2) : zero;
     }
-    for (int h = 0; h < a.H; ++h) {
-      float s0 = 0.f, s1 = 0.f;
+    for (int h = h0 + lot; h < h1; h += lots) {
+      const float* w = talk + (h - h0) * H4 + c * hg;
+      float4 s = zero;
       if (HG > 0) {
 #pragma unroll
         for (int g = 0; g < HG; ++g) {
-          const float w = talk[(c * HG + g) * a.H + h];
-          s0 = fmaf(w, q0[g], s0);
-          s1 = fmaf(w, q1[g], s1);
+          s.x = fmaf(w[g], qv[g].x, s.x); s.y = fmaf(w[g], qv[g].y, s.y);
+          s.z = fmaf(w[g], qv[g].z, s.z); s.w = fmaf(w[g], qv[g].w, s.w);
         }
-      } else {
+      } else if (d < a.D) {
         for (int g = 0; g < hg; ++g) {
-          const float w = talk[(c * hg + g) * a.H + h];
-          s0 = fmaf(w, in0 ? qc[g * D2] : 0.f, s0);
-          s1 = fmaf(w, in1 ? qc[g * D2 + 1] : 0.f, s1);
+          const float4 y = *reinterpret_cast<const float4*>(qc + g * D2);
+          s.x = fmaf(w[g], y.x, s.x); s.y = fmaf(w[g], y.y, s.y);
+          s.z = fmaf(w[g], y.z, s.z); s.w = fmaf(w[g], y.w, s.w);
         }
       }
-      A* to = q + static_cast<long long>(h) * KD + c * a.kp + d;
-      if (sizeof(A) == 2) {
-        *reinterpret_cast<__nv_bfloat162*>(to) = __floats2bfloat162_rn(s0, s1);
+      A* to = q + h * hstep + c * a.kp + d;
+      if constexpr (sizeof(A) == 2) {
+        __align__(8) const __nv_bfloat162 b[2] = {__floats2bfloat162_rn(s.x, s.y), __floats2bfloat162_rn(s.z, s.w)};
+        *reinterpret_cast<uint2*>(to) = *reinterpret_cast<const uint2*>(b);
       } else {
-        st_act(to, s0);
-        st_act(to + 1, s1);
+        *reinterpret_cast<float4*>(to) = s;
       }
     }
   }
@@ -151,7 +151,7 @@ talking_simt_kernel(const TalkArgs a, const int* __restrict__ first_pos, const i
     for (int d = threadIdx.x; d < a.V; d += blockDim.x) st_act(out + d, 0.f);
     return;
   }
-  const A* qg = reinterpret_cast<const A*>(a.q) + t * a.ldq + static_cast<long long>(h) * KD;
+  const A* qg = reinterpret_cast<const A*>(a.q) + (static_cast<long long>(h) * a.T + t) * KD;
   for (int d = threadIdx.x; d < KD; d += blockDim.x) q[d] = ld_act(qg + d);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -210,14 +210,15 @@ talking_simt_kernel(const TalkArgs a, const int* __restrict__ first_pos, const i
 
 template <typename A>
 static int launch_talk_prep(const TalkPrepArgs& a, int T, cudaStream_t st) {
-  const size_t smem = (static_cast<size_t>(a.H + a.G) * ((a.D + 1) & ~1) + ((a.H * a.H + 1) & ~1) + 2 * a.pairs) * sizeof(float);
+  const int parts = T >= 148 ? 1 : min((a.H + 3) / 4, 8), per = (a.H + parts - 1) / parts, threads = T >= 148 ? 256 : 512;
+  const size_t smem = (static_cast<size_t>(a.H + a.G) * ((a.D + 3) & ~3) + per * ((a.H + 3) & ~3) + 2 * a.pairs) * sizeof(float);
   if (smem > 200 * 1024) return -2;
 #define STK_TALK_PREP(HG)                                                                                                       \
   {                                                                                                                             \
     if (smem > 40 * 1024 && cudaFuncSetAttribute(talking_prep_kernel<A, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
                                                  200 * 1024) != cudaSuccess)                                                    \
       return -3;                                                                                                                \
-    launch_pdl(talking_prep_kernel<A, HG>, dim3(T), dim3(kTkThreads), smem, st, a);                                             \
+    launch_pdl(talking_prep_kernel<A, HG>, dim3(T, parts), dim3(threads), smem, st, a);                                            \
   }
   switch (a.H / a.G) {
     case 1: STK_TALK_PREP(1) break;
@@ -234,32 +235,32 @@ static int launch_talk_prep(const TalkPrepArgs& a, int T, cudaStream_t st) {
 
 using namespace stk;
 
-// q: [T, heads * kv_heads * kp] in the type of proj; gate [T, heads] fp32 or null (no gate).
+// q: [heads, T, kv_heads * kp] in the type of proj, 16-byte aligned; gate [T, heads] fp32 or null (no gate).
 STK_API int stk_talking_prep(const void* proj, long long ldp, int q_off, int k_off, int v_off, int g_off, const float* bias,
                              const float* q_norm, const float* k_norm, float eps, const float* freq, int pairs, const float* talk,
                              const int64_t* positions, const int* tok_req, const int* table, int bt_stride, void* cache, int row, int k_col,
                              int kp, int vp, int heads, int kv_heads, int dim, int vdim, void* q, float* gate, int fp32, int T,
                              void* stream) {
   if (T <= 0) return 0;
-  if (heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || kp < dim || (kp & 1) || vp < vdim || k_col != kv_heads * vp ||
-      row < k_col + kv_heads * kp || pairs < 0 || 2 * pairs > dim || (q_norm == nullptr) != (k_norm == nullptr))
+  if (heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || kp < dim || (kp & 15) || vp < vdim || k_col != kv_heads * vp ||
+      row < k_col + kv_heads * kp || pairs < 0 || 2 * pairs > dim || (q_norm == nullptr) != (k_norm == nullptr) || (reinterpret_cast<uintptr_t>(q) & 15))
     return -1;
   TalkPrepArgs a;
   a.proj = proj; a.ldp = ldp; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.g_off = g_off;
   a.bias = bias; a.q_norm = q_norm; a.k_norm = k_norm; a.eps = eps; a.freq = freq; a.pairs = pairs; a.talk = talk;
   a.positions = positions; a.tok_req = tok_req; a.table = table; a.bt_stride = bt_stride;
   a.cache = cache; a.row = row; a.k_col = k_col; a.kp = kp; a.vp = vp;
-  a.H = heads; a.G = kv_heads; a.D = dim; a.V = vdim; a.q = q; a.gate = gate;
+  a.H = heads; a.G = kv_heads; a.D = dim; a.V = vdim; a.T = T; a.q = q; a.gate = gate;
   return fp32 ? launch_talk_prep<float>(a, T, (cudaStream_t)stream) : launch_talk_prep<__nv_bfloat16>(a, T, (cudaStream_t)stream);
 }
 
 // Spans of at most max_span tokens.
-STK_API int stk_talking_simt(const void* q, long long ldq, const float* gate, const float* sink, const int64_t* positions, const int* tok_req,
+STK_API int stk_talking_simt(const void* q, const float* gate, const float* sink, const int64_t* positions, const int* tok_req,
                              const int* table, int bt_stride, const void* cache, int row, int k_col, int kp, int vp, int heads, int kv_heads,
                              int vdim, int chunk, float scale, void* out, long long ldo, int out_cols, int fp32, const int* first_pos,
                              const int* last_pos, int max_span, int T, void* stream) {
   if (T <= 0) return 0;
-  const TalkArgs a = {q, ldq, gate, sink, positions, tok_req, table, bt_stride, cache, row, k_col, kp, vp, heads, kv_heads, vdim, chunk,
+  const TalkArgs a = {q, T, gate, sink, positions, tok_req, table, bt_stride, cache, row, k_col, kp, vp, heads, kv_heads, vdim, chunk,
                       scale, out, ldo, out_cols};
   const size_t smem = static_cast<size_t>(kv_heads) * kp * sizeof(float);
   if (!talk_ok(a) || vdim > 1024 || heads > 65535 || smem > 200 * 1024) return -1;

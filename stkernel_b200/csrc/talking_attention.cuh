@@ -8,7 +8,7 @@ namespace stk {
 constexpr int kTkPage = 64;
 
 struct TalkArgs {
-  const void* q; long long ldq;                   // mixed queries: head h at columns h * G * kp
+  const void* q; int T;                           // mixed queries [H, T, G * kp]
   const float* gate; const float* sink;           // [T, H] gate logits, [H] scores without a key (nullptr: none)
   const int64_t* positions; const int* tok_req;
   const int* table; int bt_stride;

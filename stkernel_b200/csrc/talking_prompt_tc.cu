@@ -9,7 +9,7 @@
 //                      ring of 16 KB panels [128 rows x 64 columns], keys and values in the order in which they are used
 //     MMA warp         S[query, key] = Q . K^T, then O[query, v] += P . V with P read from tensor memory.  Blocks take turns between two
 //                      sets of accumulators, so one block's softmax runs under the products of the next
-//     softmax warps    four per set, one row per thread: running maximum (O rescaled only when a row's maximum grew by more than 2^8),
+//     softmax warps    eight per set, half of a row's scores per thread: running maximum (O rescaled only when a row's maximum grew by more than 2^8),
 //                      probabilities written over the scores as bf16 pairs (high part and remainder, two products)
 //
 // The two sets hold partial results of the same rows with maxima and denominators of their own; they are joined at the end.
@@ -22,7 +22,7 @@ namespace stk {
 
 int make_tmap_2d(CUtensorMap* tm, const void* base, int elem_bytes, long long rows, long long cols, long long ld, int box_rows);
 
-constexpr int kTpTile = 128, kTpPanel = kTpTile * 128, kTpThreads = 320, kTpMaxSlots = 12, kTpMaxQ = 10;
+constexpr int kTpTile = 128, kTpPanel = kTpTile * 128, kTpThreads = 576, kTpMaxSlots = 12, kTpMaxQ = 10;
 constexpr float kTpLog2e = 1.4426950408889634f;
 
 struct alignas(8) TpBars {
@@ -31,14 +31,16 @@ struct alignas(8) TpBars {
   uint32_t tmem_base;
   int find[2];
   long long seg;
+  float row_max[4 * 128];                                          // [set][half][row]
 };
+constexpr int kTpBarBytes = 3072;
 
 struct TpArgs {
   TalkArgs a;
   const int* query_start; const int* start_pos;
   int n_req, min_span;
   int k_panels, v_panels, q_kept;        // panels of 64 columns; whether the queries stay in shared memory
-  int slots;
+  int slots, T;
   int* status;
 };
 
@@ -56,11 +58,22 @@ __device__ __forceinline__ float tp_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// Barrier `id` of `n` threads that also tells whether all of them are fine.
+__device__ __forceinline__ bool tp_bar_all(int id, bool ok, int n = 256) {
+  int r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.s32 p, %1, 0;\n\t"
+      "barrier.cta.red.and.pred q, %2, %3, p;\n\t"
+      "selp.s32 %0, 1, 0, q;\n\t}"
+      : "=r"(r) : "r"(ok ? 1 : 0), "r"(id), "r"(n) : "memory");
+  return r != 0;
+}
 // First row that a span starting at `start` needs: its chunk's first position, on a 128-row border.
 __host__ __device__ inline int tp_base(int chunk, int start) { return chunk > 0 ? start / chunk * chunk / kTpTile * kTpTile : 0; }
 
 // kTpParts CTAs per 128 rows of the gathered matrix.
-constexpr int kTpParts = 8;
+constexpr int kTpParts = 32;
 __global__ void __launch_bounds__(256)
 talking_rows_kernel(const int* __restrict__ query_start, const int* __restrict__ req_rows, const int* __restrict__ start_pos, int n_req,
                     int min_span, int chunk, const int* __restrict__ table, int bt_stride, const __nv_bfloat16* __restrict__ cache, int row,
@@ -102,14 +115,18 @@ talking_rows_kernel(const int* __restrict__ query_start, const int* __restrict__
 
 __global__ void __launch_bounds__(kTpThreads, 1)
 talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_r, const TpArgs x) {
-  extern __shared__ uint8_t smem_raw[];
+  extern __shared__ __align__(1024) uint8_t smem[];
   const TalkArgs& a = x.a;
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  if ((smem_u32(smem) & 1023) != 0) {                              // the panels' swizzle needs it; there is no room to round up
+    pdl_wait();
+    set_status(x.status, kBadIndex, 859);
+    return;
+  }
   const int kp = x.k_panels;
   uint8_t* q_s = smem;                                             // [kp][128 rows x 128 B] when the queries are kept
   uint8_t* ring = q_s + (x.q_kept ? kp * kTpPanel : 0);            // [slots][128 rows x 128 B]
   TpBars* bars = reinterpret_cast<TpBars*>(ring + x.slots * kTpPanel);
-  float* join = reinterpret_cast<float*>(ring);                    // at the end: [128][2] maxima and denominators of the second set
+  float* row_sum = reinterpret_cast<float*>(ring);                 // [set][half][row], when nothing uses the ring any more
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   pdl_trigger();
@@ -134,7 +151,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&bars->s_full[i], 1);
-      mbar_init(&bars->p_full[i], 4);
+      mbar_init(&bars->p_full[i], 8);
       mbar_init(&bars->o_full[i], 1);
     }
     fence_barrier_init();
@@ -142,11 +159,11 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
   __syncthreads();
   const int ri = bars->find[0];
   if (ri < 0) return;
-  if (warp == 9) {
+  if (warp == 17) {
     tmem_alloc(&bars->tmem_base, 512);
     tmem_relinquish();
   }
-  const int h = blockIdx.y, KD = a.G * a.kp;
+  const int h = blockIdx.y;
   const int q0 = x.query_start[ri], span = x.query_start[ri + 1] - q0, off = bars->find[1] * kTpTile;
   const int n_tok = min(kTpTile, span - off), first = x.start_pos[ri] + off, last = first + n_tok - 1;
   const int base = tp_base(a.chunk, x.start_pos[ri]), seg = static_cast<int>(bars->seg);
@@ -156,14 +173,14 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
   tc_fence_after();
   const uint32_t tmem = bars->tmem_base;                           // scores of set i: i * 128; outputs: 256 + i * 128
 
-  if (warp == 8) {
+  if (warp == 16) {
     // ------------------------------- loader -------------------------------
     if (lane == 0) {
       bool ok = true;
       int seq = 0;
       if (x.q_kept) {
         mbar_expect_tx(&bars->q_full, kp * kTpPanel);
-        for (int p = 0; p < kp; ++p) tma_load_2d(q_s + p * kTpPanel, &tm_q, &bars->q_full, h * KD + p * 64, q0 + off);
+        for (int p = 0; p < kp; ++p) tma_load_2d(q_s + p * kTpPanel, &tm_q, &bars->q_full, p * 64, h * x.T + q0 + off);
       }
       auto load = [&](const CUtensorMap* tm, int col, int y) {
         const int st = seq % x.slots;
@@ -175,7 +192,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
       };
       auto keys = [&](int b) {
         for (int j = 0; j < kp && ok; ++j) {
-          if (!x.q_kept) load(&tm_q, h * KD + j * 64, q0 + off);
+          if (!x.q_kept) load(&tm_q, j * 64, h * x.T + q0 + off);
           if (ok) load(&tm_r, a.k_col + j * 64, seg + (b0 + b) * kTpTile);
         }
       };
@@ -193,7 +210,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
       }
     }
     __syncwarp();
-  } else if (warp == 9) {
+  } else if (warp == 17) {
     // ------------------------------- MMA issuer -------------------------------
     const uint32_t lead = elect_one() ? 1u : 0u, tm = __shfl_sync(0xffffffffu, tmem, 0);
     constexpr uint32_t kIdescS = umma_idesc(1u, 1u, 128, 128);
@@ -276,49 +293,46 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
     __syncwarp();
   } else {
     // ------------------------------- softmax -------------------------------
-    const int set = warp >> 2, r = (warp & 3) * 32 + lane;
+    const int set = warp >> 3, half = (warp >> 2) & 1, r = (warp & 3) * 32 + lane;
     const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
-    const uint32_t ts = tmem + set * 128 + lanes, to = tmem + 256 + set * 128 + lanes;
+    const uint32_t ts = tmem + set * 128 + half * 64 + lanes, to = tmem + 256 + set * 128 + half * x.v_panels * 32 + lanes;
+    float* peer = bars->row_max + (set * 2) * kTpTile;             // [2 halves][128]
     const float c_in = a.scale * kTpLog2e;
     const bool flip = c_in < 0.f;                                  // a negative scale: the largest score is the smallest product
     const uint32_t masked = __float_as_uint(flip ? INFINITY : -INFINITY);
     // the sink counts once, in the first set
     const bool sunk = set == 0 && a.sink != nullptr;
-    float m = sunk ? a.sink[h] * kTpLog2e : -INFINITY, l = sunk ? 1.f : 0.f;
+    float m = sunk ? a.sink[h] * kTpLog2e : -INFINITY, l = sunk && half == 0 ? 1.f : 0.f;
     const int pos = first + r, lo = talk_first(a, pos), lo_last = talk_first(a, last);
     const int mine = nb > set ? (nb - set + 1) >> 1 : 0;           // blocks of this set
     bool ok = true;
-    for (int n = 0; n < mine && ok; ++n) {
-      const int k0 = base + (b0 + 2 * n + set) * kTpTile;          // position of the block's first key
-      ok = mbar_wait(&bars->s_full[set], n & 1, x.status, 870);
-      if (!ok) break;
+    for (int n = 0; n < mine; ++n) {
+      const int k0 = base + (b0 + 2 * n + set) * kTpTile + half * 64;      // position of the half block's first key
+      ok = ok && mbar_wait(&bars->s_full[set], n & 1, x.status, 870);
       tc_fence_after();
-      const int d1 = pos - k0, d0 = lo - k0;                       // keys d0 .. d1 of the block are visible
-      const bool edge = k0 + kTpTile - 1 > first || k0 < lo_last;
-      uint32_t s[2][32];                                           // 64 scores of the row at a time
-      auto fetch = [&](int half) {
-        tmem_ld_32x32(ts + half * 64, s[0]);
-        tmem_ld_32x32(ts + half * 64 + 32, s[1]);
-        tmem_ld_wait();
-        if (edge) {
+      const int d1 = pos - k0, d0 = lo - k0;                       // keys d0 .. d1 of the half block are visible
+      uint32_t s[2][32];                                           // the row's 64 scores
+      tmem_ld_32x32(ts, s[0]);
+      tmem_ld_32x32(ts + 32, s[1]);
+      tmem_ld_wait();
+      if (k0 + 63 > first || k0 < lo_last) {
 #pragma unroll
-          for (int j = 0; j < 64; ++j)
-            if (half * 64 + j > d1 || half * 64 + j < d0) s[j >> 5][j & 31] = masked;
-        }
-      };
-      auto largest = [&]() {
-        float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        for (int j = 0; j < 64; ++j)
+          if (j > d1 || j < d0) s[j >> 5][j & 31] = masked;
+      }
+      float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      if (flip) {
 #pragma unroll
-        for (int j = 0; j < 64; ++j) {
-          const float v = __uint_as_float(s[j >> 5][j & 31]);
-          m4[j & 3] = fmaxf(m4[j & 3], flip ? -v : v);
-        }
-        return fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
-      };
-      fetch(0);
-      float mx = largest();
-      fetch(1);
-      mx = fmaxf(mx, largest()) * fabsf(c_in);
+        for (int j = 0; j < 64; ++j) m4[j & 3] = fmaxf(m4[j & 3], -__uint_as_float(s[j >> 5][j & 31]));
+      } else {
+#pragma unroll
+        for (int j = 0; j < 64; ++j) m4[j & 3] = fmaxf(m4[j & 3], __uint_as_float(s[j >> 5][j & 31]));
+      }
+      float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+      peer[half * kTpTile + r] = mx;
+      ok = tp_bar_all(1 + set, ok);                                // the set's warps leave together
+      if (!ok) break;
+      mx = fmaxf(mx, peer[(half ^ 1) * kTpTile + r]) * fabsf(c_in);
       const bool grow = mx > m + 8.f || (m == -INFINITY && mx > -INFINITY);
       if (__any_sync(0xffffffffu, grow)) {
         const float f = grow ? (m == -INFINITY ? 0.f : tp_ex2(m - mx)) : 1.f;
@@ -326,7 +340,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
         l *= f;
         if (n > 0) {
           // the products that fed these scores were issued after the set's previous P . V: that one is complete
-          for (int c = 0; c < x.v_panels * 64; c += 16) {
+          for (int c = 0; c < x.v_panels * 32; c += 16) {
             uint32_t o[16];
             tmem_ld_32x16(to + c, o);
             tmem_ld_wait();
@@ -334,38 +348,32 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
             for (int j = 0; j < 16; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * f);
             tp_st16(to + c, o);
           }
-          tp_st_wait();
         }
       }
       const float ms = m == -INFINITY ? 0.f : m;
       const uint64_t c2 = pack2(c_in, c_in), m2 = pack2(-ms, -ms), minus = pack2(-1.f, -1.f);
       uint64_t sum2[2] = {0ull, 0ull};
-      auto weigh = [&](int half) {
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          uint32_t hi[16], lw[16];
+      for (int c = 0; c < 2; ++c) {
+        uint32_t hi[16], lw[16];
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            float p0, p1;
-            unpack2(fma2(pack2(__uint_as_float(s[c][2 * j]), __uint_as_float(s[c][2 * j + 1])), c2, m2), p0, p1);
-            p0 = tp_ex2(p0);
-            p1 = tp_ex2(p1);
-            const uint64_t p2 = pack2(p0, p1);
-            sum2[j & 1] = add2(sum2[j & 1], p2);
-            const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
-            hi[j] = *reinterpret_cast<const uint32_t*>(&hb);
-            float r0, r1;
-            unpack2(fma2(pack2(__uint_as_float(hi[j] << 16), __uint_as_float(hi[j] & 0xffff0000u)), minus, p2), r0, r1);
-            const __nv_bfloat162 lb = __floats2bfloat162_rn(r0, r1);
-            lw[j] = *reinterpret_cast<const uint32_t*>(&lb);
-          }
-          tp_st16(ts + (half * 2 + c) * 32, hi);
-          tp_st16(ts + (half * 2 + c) * 32 + 16, lw);
+        for (int j = 0; j < 16; ++j) {
+          float p0, p1;
+          unpack2(fma2(pack2(__uint_as_float(s[c][2 * j]), __uint_as_float(s[c][2 * j + 1])), c2, m2), p0, p1);
+          p0 = tp_ex2(p0);
+          p1 = tp_ex2(p1);
+          const uint64_t p2 = pack2(p0, p1);
+          sum2[j & 1] = add2(sum2[j & 1], p2);
+          const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
+          hi[j] = *reinterpret_cast<const uint32_t*>(&hb);
+          float r0, r1;
+          unpack2(fma2(pack2(__uint_as_float(hi[j] << 16), __uint_as_float(hi[j] & 0xffff0000u)), minus, p2), r0, r1);
+          const __nv_bfloat162 lb = __floats2bfloat162_rn(r0, r1);
+          lw[j] = *reinterpret_cast<const uint32_t*>(&lb);
         }
-      };
-      weigh(1);
-      fetch(0);
-      weigh(0);
+        tp_st16(ts + c * 32, hi);
+        tp_st16(ts + c * 32 + 16, lw);
+      }
       float ls[4];
       unpack2(sum2[0], ls[0], ls[1]);
       unpack2(sum2[1], ls[2], ls[3]);
@@ -375,40 +383,35 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->p_full[set]);
     }
-    if (ok && mine > 0) {
-      ok = mbar_wait(&bars->o_full[set], 0, x.status, 871);
-      tc_fence_after();
-    }
-    const bool two = nb > 1;
-    if (two) {
-      // both outputs are complete, so nothing uses the ring any more: the second set's maxima and denominators go through it
-      ok = ok && mbar_wait(&bars->o_full[set ^ 1], 0, x.status, 872);
-      if (set == 1) {
-        join[2 * r] = ok ? m : -INFINITY;
-        join[2 * r + 1] = ok ? l : 0.f;
-      }
-      tc_fence_before();
-      asm volatile("bar.sync 1, 256;" ::: "memory");
-      tc_fence_after();
-    }
-    if (set == 0 && ok && mine > 0) {
-      const float m1 = two ? join[2 * r] : -INFINITY, l1 = two ? join[2 * r + 1] : 0.f;
-      const float mm = fmaxf(m, m1);
-      const float f0 = m == -INFINITY ? 0.f : tp_ex2(m - mm), f1 = m1 == -INFINITY ? 0.f : tp_ex2(m1 - mm);
+    // both outputs complete: their maxima and denominators meet, and each warp writes a quarter of the columns
+    if (ok) ok = mbar_wait(&bars->o_full[0], 0, x.status, 871) && (nb < 2 || mbar_wait(&bars->o_full[1], 0, x.status, 872));
+    if (half == 0) bars->row_max[set * 2 * kTpTile + r] = m;
+    row_sum[(set * 2 + half) * kTpTile + r] = l;
+    tc_fence_before();
+    ok = tp_bar_all(3, ok, 512);
+    tc_fence_after();
+    if (ok) {
+      const bool two = nb > 1;
+      const float m0 = bars->row_max[r], m1 = bars->row_max[2 * kTpTile + r];
+      const float l0 = row_sum[r] + row_sum[kTpTile + r], l1 = row_sum[2 * kTpTile + r] + row_sum[3 * kTpTile + r];
+      const float mm = fmaxf(m0, m1);
+      const float f0 = m0 == -INFINITY ? 0.f : tp_ex2(m0 - mm), f1 = m1 == -INFINITY ? 0.f : tp_ex2(m1 - mm);
       const bool row_ok = r < n_tok;
       const long long t = q0 + off + (row_ok ? r : 0);
-      const float g = talk_gate(a, t, h) / (f0 * l + f1 * l1);
+      const float g = talk_gate(a, t, h) / (f0 * l0 + f1 * l1);
       const float g0 = f0 * g, g1 = f1 * g;
       __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + t * a.ldo;
-      if (h == a.H - 1 && row_ok)
+      if (h == a.H - 1 && row_ok && warp < 4)
         for (int c = a.H * a.V; c < a.out_cols; ++c) out[c] = __float2bfloat16(0.f);
       out += h * a.V;
       const bool vec = (a.V & 7) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
-      for (int c = 0; c < x.v_panels * 64; c += 16) {
+      const uint32_t tj = tmem + 256 + lanes;
+      const int part = x.v_panels * 16;                            // columns of this warp
+      for (int c = (warp >> 2) * part; c < ((warp >> 2) + 1) * part; c += 16) {
         uint32_t o[16], p[16];
         __syncwarp();
-        tmem_ld_32x16(to + c, o);
-        if (two) tmem_ld_32x16(to + 128 + c, p);
+        tmem_ld_32x16(tj + c, o);
+        if (two) tmem_ld_32x16(tj + 128 + c, p);
         tmem_ld_wait();
         if (!row_ok) continue;
         float y[16];
@@ -419,15 +422,15 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
         }
         if (vec) {
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            if (c + half * 8 >= a.V) continue;
+          for (int q = 0; q < 2; ++q) {
+            if (c + q * 8 >= a.V) continue;
             uint32_t pk[4];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-              const __nv_bfloat162 v = __floats2bfloat162_rn(y[half * 8 + 2 * j], y[half * 8 + 2 * j + 1]);
+              const __nv_bfloat162 v = __floats2bfloat162_rn(y[q * 8 + 2 * j], y[q * 8 + 2 * j + 1]);
               pk[j] = *reinterpret_cast<const uint32_t*>(&v);
             }
-            *reinterpret_cast<uint4*>(out + c + half * 8) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+            *reinterpret_cast<uint4*>(out + c + q * 8) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
           }
         } else {
 #pragma unroll
@@ -439,7 +442,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 9) {
+  if (warp == 17) {
     tc_fence_after();
     tmem_dealloc(tmem, 512);
   }
@@ -451,7 +454,7 @@ static TpShape tp_shape(int G, int kp, int V) {
   s.k_panels = (G * kp + 63) / 64;
   s.v_panels = (V + 63) / 64;
   s.q_kept = s.k_panels <= kTpMaxQ ? 1 : 0;
-  s.slots = (225 * 1024 - (s.q_kept ? s.k_panels * kTpPanel : 0)) / kTpPanel;
+  s.slots = (227 * 1024 - kTpBarBytes - (s.q_kept ? s.k_panels * kTpPanel : 0)) / kTpPanel;
   if (s.slots > kTpMaxSlots) s.slots = kTpMaxSlots;
   return s;
 }
@@ -476,26 +479,26 @@ STK_API int stk_talking_rows(const int* query_start, const int* req_rows, const 
 }
 
 // Spans of at least min_span tokens.  rows [n_rows, row]: `stk_talking_rows`.
-STK_API int stk_talking_prompt(const void* q, long long ldq, const float* gate, const float* sink, const void* rows, long long n_rows, int row,
+STK_API int stk_talking_prompt(const void* q, const float* gate, const float* sink, const void* rows, long long n_rows, int row,
                                int k_col, int kp, int vp, int heads, int kv_heads, int vdim, int chunk, float scale, void* out, long long ldo,
                                int out_cols, const int* query_start, const int* start_pos, int n_req, int min_span, int T, int* status,
                                void* stream) {
   if (T <= 0) return 0;
   TpArgs x = {};
-  x.a.q = q; x.a.ldq = ldq; x.a.gate = gate; x.a.sink = sink; x.a.row = row; x.a.k_col = k_col; x.a.kp = kp; x.a.vp = vp;
+  x.a.q = q; x.a.T = T; x.a.gate = gate; x.a.sink = sink; x.a.row = row; x.a.k_col = k_col; x.a.kp = kp; x.a.vp = vp;
   x.a.H = heads; x.a.G = kv_heads; x.a.V = vdim; x.a.chunk = chunk; x.a.scale = scale; x.a.out = out; x.a.ldo = ldo; x.a.out_cols = out_cols;
   if (!talk_ok(x.a) || !stk_talking_prompt_ok(heads, kv_heads, kp, vp, vdim) || n_req < 1 || n_rows < 1 || n_rows >= (1ll << 31) ||
-      heads > 65535 || ldq % 8 || row % 8 || row != k_col + kv_heads * kp ||
+      heads > 65535 || static_cast<long long>(heads) * T >= (1ll << 31) || row % 8 || row != k_col + kv_heads * kp ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(rows)) & 15))
     return -1;
   const TpShape s = tp_shape(kv_heads, kp, vdim);
   x.query_start = query_start; x.start_pos = start_pos; x.n_req = n_req; x.min_span = min_span;
-  x.k_panels = s.k_panels; x.v_panels = s.v_panels; x.q_kept = s.q_kept; x.slots = s.slots; x.status = status;
+  x.k_panels = s.k_panels; x.v_panels = s.v_panels; x.q_kept = s.q_kept; x.slots = s.slots; x.T = T; x.status = status;
   CUtensorMap tq, tr;
-  if (make_tmap_2d(&tq, q, 2, T, static_cast<long long>(heads) * kv_heads * kp, ldq, kTpTile) != 0) return -3;
+  if (make_tmap_2d(&tq, q, 2, static_cast<long long>(heads) * T, kv_heads * kp, kv_heads * kp, kTpTile) != 0) return -3;
   if (make_tmap_2d(&tr, rows, 2, n_rows, row, row, kTpTile) != 0) return -3;
-  int smem = (s.q_kept ? s.k_panels * kTpPanel : 0) + s.slots * kTpPanel + 1024 + 1024;
-  static_assert(sizeof(TpBars) <= 1024, "barrier block");
+  int smem = (s.q_kept ? s.k_panels * kTpPanel : 0) + s.slots * kTpPanel + kTpBarBytes;
+  static_assert(sizeof(TpBars) <= kTpBarBytes, "barrier block");
   if (cudaFuncSetAttribute(talking_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -3;
   if (smem < 118 * 1024) smem = 118 * 1024;                          // one CTA per SM: it owns all of tensor memory
   launch_pdl(talking_prompt_tc_kernel, dim3(T / kTpTile + n_req, heads), dim3(kTpThreads), smem, (cudaStream_t)stream, tq, tr, x);

@@ -173,6 +173,12 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
       tma_load_2d(dst + j * kTtPanel + kTtPanel / 2, &tm_rows, &bars->full[st], col + j * 64, pg1 * kTkPage);
     }
   };
+  // the first block's keys are on their way while the queries are laid out
+  const int early = min(x.k_pairs, x.slots);
+  if (warp == 8 && lane == 0) {
+    const int pg0 = page_of(2 * b0), pg1 = page_of(2 * b0 + 1);
+    for (int d = 0; d < early; ++d) load_pair(d, a.k_col + d * 128, pg0, pg1);
+  }
   if (warp == 9) {
     tmem_alloc(&bars->tmem_base, 512);
     tmem_relinquish();
@@ -182,7 +188,7 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
   for (int n = warp; n < N; n += kTtThreads / 32) {
     const int q = n / x.hs, hh = n - q * x.hs;
     const bool valid = q < ntok && hh < nh;
-    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(a.q) + (valid ? (tok0 + q) * a.ldq + static_cast<long long>(h0 + hh) * KD : 0);
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(a.q) + (valid ? (static_cast<long long>(h0 + hh) * x.T + tok0 + q) * KD : 0);
     for (int cc = lane; cc < q_panels * 8; cc += 32) {
       uint4 v = make_uint4(0, 0, 0, 0);
       if (valid && cc * 8 < KD) v = *reinterpret_cast<const uint4*>(src + cc * 8);
@@ -211,7 +217,7 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
   if (warp == 8) {
     // ------------------------------- loader -------------------------------
     bool ok = true;
-    int seq = 0;
+    int seq = early;
     auto load = [&](int col, int pg0, int pg1) {                    // one pair, lane 0
       const int st = seq % x.slots;
       if (seq >= x.slots) ok = mbar_wait(&bars->empty[st], ((seq / x.slots) - 1) & 1, x.status, 930);
@@ -220,14 +226,14 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
         ++seq;
       }
     };
-    auto load_keys = [&](int b) {
+    auto load_keys = [&](int b, int done) {
       const int pg0 = page_of(2 * b), pg1 = page_of(2 * b + 1);
-      for (int d = 0; d < x.k_pairs && ok; ++d) load(a.k_col + d * 128, pg0, pg1);
+      for (int d = done; d < x.k_pairs && ok; ++d) load(a.k_col + d * 128, pg0, pg1);
     };
-    if (lane == 0) load_keys(b0);
+    if (lane == 0) load_keys(b0, early);
     for (int b = b0; b < b1; ++b) {
       if (lane == 0) {
-        if (ok && b + 1 < b1) load_keys(b + 1);
+        if (ok && b + 1 < b1) load_keys(b + 1, 0);
         const int pg0 = page_of(2 * b), pg1 = page_of(2 * b + 1);
         for (int j = 0; j < x.v_tiles && ok; ++j) load(j * 128, pg0, pg1);
       }
@@ -538,17 +544,17 @@ STK_API int stk_talking_tokens_splits(int T, int heads, int kv_heads, int kp, in
 }
 
 // Spans of at most max_span tokens.  part: [splits][T][heads][vdim + 2] fp32.
-STK_API int stk_talking_tokens(const void* q, long long ldq, const float* gate, const float* sink, const int64_t* positions, const int* tok_req,
+STK_API int stk_talking_tokens(const void* q, const float* gate, const float* sink, const int64_t* positions, const int* tok_req,
                                const int* table, int bt_stride, const void* cache, int row, int k_col, int kp, int vp, int heads, int kv_heads,
                                int vdim, int chunk, float scale, void* out, long long ldo, int out_cols, const int* query_start,
                                const int* req_rows, const int* start_pos, int n_req, const int* first_pos, const int* last_pos, int max_span,
                                long long num_pages, int splits, float* part, int T, int* status, void* stream) {
   if (T <= 0) return 0;
   TtArgs x;
-  x.a = {q, ldq, gate, sink, positions, tok_req, table, bt_stride, cache, row, k_col, kp, vp, heads, kv_heads, vdim, chunk, scale, out, ldo,
+  x.a = {q, T, gate, sink, positions, tok_req, table, bt_stride, cache, row, k_col, kp, vp, heads, kv_heads, vdim, chunk, scale, out, ldo,
          out_cols};
   const TtShape s = tt_shape(heads, kv_heads, kp, vp, max_span);
-  if (!talk_ok(x.a) || s.n == 0 || splits < 1 || splits > kTtMaxSplits || n_req < 1 || num_pages < 1 || ldq % 8 || row % 8 || kp % 8 || vp % 8 ||
+  if (!talk_ok(x.a) || s.n == 0 || splits < 1 || splits > kTtMaxSplits || n_req < 1 || num_pages < 1 || row % 8 || kp % 8 || vp % 8 ||
       heads > 65535 || row != k_col + kv_heads * kp || num_pages * kTkPage >= (1ll << 31) ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15))
     return -1;

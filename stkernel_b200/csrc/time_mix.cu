@@ -54,51 +54,78 @@ struct TmArgs {
 };
 constexpr int kTmSub = 16, kTmBlocks = kChunk / kTmSub;
 
-__device__ __forceinline__ float tm_log_decay(const TmArgs& a, long long t, int h, int d) {
-  return -__expf(a.z[t * a.ldz + h * a.s.D + d] + a.w0[h * a.s.D + d]);
-}
-
-// keys [T][2][H * D8]: high parts, remainders; channel [chunk][H][D].  One CTA per (chunk, head); a thread takes a block's 16 tokens of a channel.
+// keys [T][2][H * D8]: high parts, remainders; channel [chunk][H][D].  One CTA per (chunk, head); a thread takes a block's 16 tokens of two
+// channels.  vec: channels come in whole aligned pairs.
 __global__ void __launch_bounds__(256)
-time_mix_keys_kernel(const TmArgs a, int min_span, __nv_bfloat16* __restrict__ keys, int D8, float* __restrict__ channel) {
+time_mix_keys_kernel(const TmArgs a, int min_span, __nv_bfloat16* __restrict__ keys, int D8, float* __restrict__ channel, int vec) {
   extern __shared__ __align__(16) float ends[];   // [4][D8]
   __shared__ ChunkRef s_c;
   __shared__ int s_ok;
   pdl_wait();
   pdl_trigger();
-  const int ci = blockIdx.x, h = blockIdx.y, D = a.s.D, n8 = a.s.H * D8;
+  const int ci = blockIdx.x, h = blockIdx.y, D = a.s.D, n8 = a.s.H * D8, pairs = D8 >> 1;
   if (threadIdx.x == 0) s_ok = find_chunk(a.s.query_start, a.s.n_req, min_span, ci, s_c) ? 1 : 0;
   __syncthreads();
   if (!s_ok) return;
   const ChunkRef c = s_c;
-  for (int e0 = 0; e0 < kTmBlocks * D8; e0 += blockDim.x) {
-    const int e = e0 + threadIdx.x, b = e / D8, d = e - b * D8;
-    if (e >= kTmBlocks * D8) continue;
-    float sum = 0.f;
-    if (d < D)
+  const int b = threadIdx.x / pairs, d = (threadIdx.x - b * pairs) * 2;      // blockDim.x = 4 * pairs
+  const bool in0 = d < D, in1 = d + 1 < D;
+  const float w0 = in0 ? a.w0[h * D + d] : 0.f, w1 = in1 ? a.w0[h * D + d + 1] : 0.f;
+  float2 g[kTmSub], sum = make_float2(0.f, 0.f);
+  __nv_bfloat162 k[kTmSub];
 #pragma unroll
-      for (int i = 0; i < kTmSub; ++i)
-        if (b * kTmSub + i < c.n) sum += tm_log_decay(a, c.t0 + b * kTmSub + i, h, d);
-    ends[b * D8 + d] = sum;
-  }
-  __syncthreads();
-  for (int e0 = 0; e0 < kTmBlocks * D8; e0 += blockDim.x) {
-    const int e = e0 + threadIdx.x, b = e / D8, d = e - b * D8;
-    if (e >= kTmBlocks * D8) continue;
-    float left = 0.f;                             // decays behind the token, up to the end of the chunk
-    for (int m = kTmBlocks - 1; m > b; --m) left += ends[m * D8 + d];
-#pragma unroll
-    for (int i = kTmSub - 1; i >= 0; --i) {
-      const int n = b * kTmSub + i;
-      if (n >= c.n) continue;
-      const long long t = c.t0 + n;
-      const float k = d < D ? bf16_to_f(a.proj[t * a.ldp + a.np + h * D + d]) * __expf(left) : 0.f;
-      const __nv_bfloat16 hi = __float2bfloat16(k);
-      keys[t * 2 * n8 + h * D8 + d] = hi;
-      keys[t * 2 * n8 + n8 + h * D8 + d] = __float2bfloat16(k - bf16_to_f(hi));
-      if (d < D) left += tm_log_decay(a, t, h, d);
+  for (int i = 0; i < kTmSub; ++i) {
+    const int n = b * kTmSub + i;
+    const long long t = c.t0 + n;
+    float2 z = make_float2(0.f, 0.f);
+    k[i] = __floats2bfloat162_rn(0.f, 0.f);
+    if (n < c.n) {
+      const float* zp = a.z + t * a.ldz + h * D + d;
+      const __nv_bfloat16* kp = a.proj + t * a.ldp + a.np + h * D + d;
+      if (vec && in1) {
+        z = *reinterpret_cast<const float2*>(zp);
+        k[i] = *reinterpret_cast<const __nv_bfloat162*>(kp);
+      } else {
+        if (in0) { z.x = zp[0]; k[i].x = kp[0]; }
+        if (in1) { z.y = zp[1]; k[i].y = kp[1]; }
+      }
     }
-    if (b == 0 && d < D) channel[(static_cast<long long>(ci) * a.s.H + h) * D + d] = __expf(left);
+    g[i] = z;
+  }
+#pragma unroll
+  for (int i = 0; i < kTmSub; ++i) {
+    const bool live = b * kTmSub + i < c.n;
+    g[i].x = live && in0 ? -__expf(g[i].x + w0) : 0.f;
+    g[i].y = live && in1 ? -__expf(g[i].y + w1) : 0.f;
+    sum.x += g[i].x;
+    sum.y += g[i].y;
+  }
+  *reinterpret_cast<float2*>(ends + b * D8 + d) = sum;
+  __syncthreads();
+  float2 left = make_float2(0.f, 0.f);            // decays behind the token, up to the end of the chunk
+  for (int m = kTmBlocks - 1; m > b; --m) {
+    const float2 e = *reinterpret_cast<const float2*>(ends + m * D8 + d);
+    left.x += e.x;
+    left.y += e.y;
+  }
+#pragma unroll
+  for (int i = kTmSub - 1; i >= 0; --i) {
+    const int n = b * kTmSub + i;
+    if (n < c.n) {
+      const float2 kf = __bfloat1622float2(k[i]);
+      uint32_t hi, lo;
+      mls_split2(kf.x * __expf(left.x), kf.y * __expf(left.y), hi, lo);
+      __nv_bfloat16* to = keys + (c.t0 + n) * 2 * n8 + h * D8 + d;
+      *reinterpret_cast<uint32_t*>(to) = hi;
+      *reinterpret_cast<uint32_t*>(to + n8) = lo;
+    }
+    left.x += g[i].x;
+    left.y += g[i].y;
+  }
+  if (b == 0) {
+    float* to = channel + (static_cast<long long>(ci) * a.s.H + h) * D + d;
+    if (in0) to[0] = __expf(left.x);
+    if (in1) to[1] = __expf(left.y);
   }
 }
 
@@ -116,8 +143,8 @@ __host__ __device__ inline TmOutLayout tm_out_layout(int D) {
   l.kr = l.r + tile;
   l.v = l.kr + tile;
   l.w = l.v + tile;                               // [64][Dp] fp32 decays
-  l.f = l.w + kChunk * Dp * 4;                    // [6][Dp] fp32: decays of blocks 1, 2, 1 and 2, 0, 0 and 1, 0 to 2
-  l.p = l.f + 6 * Dp * 4;                         // [4][Dp] sums of the blocks
+  l.f = l.w + kChunk * Dp * 4;                    // [7][Dp] fp32: decays of blocks 1, 2, 1 and 2, 0, 0 and 1, 0 to 2; the bonus
+  l.p = l.f + 7 * Dp * 4;                         // [4][Dp] sums of the blocks
   l.bytes = l.p + 4 * Dp * 4;
   return l;
 }
@@ -166,14 +193,24 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
   load_rows_async(kr, ks, Dp, p + a.np, a.ldp, c.n, D, kTmOutThreads);
   load_rows_async(v, ks, Dp, p + 2 * a.np, a.ldp, c.n, D, kTmOutThreads);
   mls_commit();
+  for (int d = threadIdx.x; d < Dp; d += kTmOutThreads) f[6 * Dp + d] = d < D ? a.u[h * D + d] : 0.f;
+  float g[kTmSub], w0 = 0.f;
+  auto fetch = [&](int e) {
+    const int b = e / Dp, d = e - b * Dp;
+#pragma unroll
+    for (int i = 0; i < kTmSub; ++i) g[i] = d < D && b * kTmSub + i < c.n ? a.z[(c.t0 + b * kTmSub + i) * a.ldz + h * D + d] : 0.f;
+    w0 = d < D ? a.w0[h * D + d] : 0.f;
+  };
+  if (threadIdx.x < kTmBlocks * Dp) fetch(threadIdx.x);
   mls_wait<0>();
   __syncthreads();
   // r~ and k^ of every block, the decays themselves
   for (int e = threadIdx.x; e < kTmBlocks * Dp; e += kTmOutThreads) {
     const int b = e / Dp, d = e - b * Dp;
-    float g[kTmSub], sum = 0.f;
+    if (e >= kTmOutThreads) fetch(e);
+    float sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < kTmSub; ++i) g[i] = d < D && b * kTmSub + i < c.n ? tm_log_decay(a, c.t0 + b * kTmSub + i, h, d) : 0.f;
+    for (int i = 0; i < kTmSub; ++i) g[i] = d < D && b * kTmSub + i < c.n ? -__expf(g[i] + w0) : 0.f;
 #pragma unroll
     for (int i = 0; i < kTmSub; ++i) {
       const int n = b * kTmSub + i;
@@ -201,7 +238,7 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
     f[5 * Dp + d] = __expf(s0 + s1 + s2);
   }
   // the blocks on the diagonal: four lanes per column, each four channels of every 16
-  float acc[kTmSub];
+  float acc[kTmSub], bonus = 0.f;
   const int jb = warp >> 1, j = (warp & 1) * 8 + (lane >> 2), seg = lane & 3;
 #pragma unroll
   for (int i = 0; i < kTmSub; ++i) acc[i] = 0.f;
@@ -212,24 +249,27 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
       const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.y));
       x[0] = lo.x; x[1] = lo.y; x[2] = hi.x; x[3] = hi.y;
     };
-    float x[4];
+    float x[4], y[4];
     four(kr + (jb * kTmSub + j) * ks + c0, x);
+    four(r + (jb * kTmSub + j) * ks + c0, y);
+    const float4 u = *reinterpret_cast<const float4*>(f + 6 * Dp + c0);
+    bonus = fmaf(y[0] * u.x, x[0], fmaf(y[1] * u.y, x[1], fmaf(y[2] * u.z, x[2], fmaf(y[3] * u.w, x[3], bonus))));
 #pragma unroll
-    for (int i = 0; i < kTmSub; ++i) {
-      if (i < j) continue;
-      float y[4];
+    for (int i = 1; i < kTmSub; ++i) {
+      if (i < 9 && (warp & 1)) continue;                                 // the warp's columns start behind these rows
+      const float4 wi = *reinterpret_cast<const float4*>(w + (jb * kTmSub + i) * Dp + c0);
       four(r + (jb * kTmSub + i) * ks + c0, y);
-      if (i == j) {
-#pragma unroll
-        for (int m = 0; m < 4; ++m) acc[i] = fmaf(y[m] * (c0 + m < D ? a.u[h * D + c0 + m] : 0.f), x[m], acc[i]);
-      } else {
-        const float4 wi = *reinterpret_cast<const float4*>(w + (jb * kTmSub + i) * Dp + c0);
-#pragma unroll
-        for (int m = 0; m < 4; ++m) acc[i] = fmaf(y[m], x[m], acc[i]);
-        x[0] *= wi.x; x[1] *= wi.y; x[2] *= wi.z; x[3] *= wi.w;
-      }
+      const bool below = i > j;
+      const float s = fmaf(y[0], x[0], fmaf(y[1], x[1], fmaf(y[2], x[2], y[3] * x[3])));
+      acc[i] += below ? s : 0.f;
+      x[0] = below ? x[0] * wi.x : x[0];
+      x[1] = below ? x[1] * wi.y : x[1];
+      x[2] = below ? x[2] * wi.z : x[2];
+      x[3] = below ? x[3] * wi.w : x[3];
     }
   }
+  bonus += __shfl_xor_sync(0xffffffffu, bonus, 1);
+  bonus += __shfl_xor_sync(0xffffffffu, bonus, 2);
 #pragma unroll
   for (int i = 0; i < kTmSub; ++i) {
     acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 1);
@@ -284,7 +324,7 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
   for (int i = 0; i < kTmSub; ++i) {
     if ((i & 3) != seg) continue;
     const int off = (jb * kTmSub + i) * kStStride + jb * kTmSub + j;
-    mls_split(i >= j ? acc[i] : 0.f, ph[off], pl[off]);
+    mls_split(i > j ? acc[i] : i == j ? bonus : 0.f, ph[off], pl[off]);
   }
   __syncthreads();                                                       // the weighted scores are complete
   const bool has_state = !(a.s.start_pos[c.ri] == 0 && c.first == ci);
@@ -416,13 +456,15 @@ STK_API int stk_time_mix_chunks(const void* proj, long long ldp, int np, const f
       ((reinterpret_cast<uintptr_t>(states) | reinterpret_cast<uintptr_t>(keys)) & 15))
     return -1;
   const int d8 = (dim + 7) / 8 * 8, n8 = heads * d8;
+  const int vec = dim % 2 == 0 && ldp % 2 == 0 && np % 2 == 0 && ldz % 2 == 0 && (reinterpret_cast<uintptr_t>(proj) & 3) == 0 &&
+                  (reinterpret_cast<uintptr_t>(z) & 7) == 0;
   TmArgs a;
   a.proj = (const __nv_bfloat16*)proj; a.ldp = ldp; a.np = np; a.z = z; a.ldz = ldz; a.w0 = w0; a.u = u;
   a.s = ScanArgs{query_start, req_rows, start_pos, n_req, S, o, heads, dim, dim};
   cudaStream_t st = (cudaStream_t)stream;
   __nv_bfloat16* kp = (__nv_bfloat16*)keys;
-  launch_pdl(time_mix_keys_kernel, dim3(max_chunks, heads), dim3(256), static_cast<size_t>(kTmBlocks) * d8 * sizeof(float), st, a, min_span, kp,
-             d8, channel);
+  launch_pdl(time_mix_keys_kernel, dim3(max_chunks, heads), dim3(2 * d8), static_cast<size_t>(kTmBlocks) * d8 * sizeof(float), st, a, min_span, kp,
+             d8, channel, vec);
   const int rc = linear_states_per_channel(kp, kp + n8, 2ll * n8, d8, d8, a.proj, ldp, 2 * np, channel, a.s, min_span, states, T, st);
   if (rc != 0) return rc;
   if (cudaFuncSetAttribute(time_mix_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return -3;

@@ -5,6 +5,8 @@
 //                     and s' are the previous token's h and s
 //   shift_commit      the last h, s and token of every request's span become its state
 //
+//   shift_blend       s and the blends of a long step, after its sums and norms
+//
 // shifted_norm: a CTA walks a run of consecutive tokens with h' and s' in registers.  At the start of a run it forms h of the two tokens
 // before it once more (s' needs the h before that), at the start of a span it takes h' and s' from the request's state.  The new
 // state goes to a second buffer: other CTAs of the step may still read the first.
@@ -74,6 +76,7 @@ struct ShiftArgs {
   const int* tok_req; const int64_t* positions; const int* first_pos; const int* last_pos;
   const int64_t* rows;
   int T, W, width, run;
+  float* inv;                                     // [T] receives 1 / rms(x) (or null)
 };
 
 // N columns (4, or 1 for widths that are not multiples of 4) from p.
@@ -115,8 +118,8 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
   return make_float2(warp_sum(a), warp_sum(b));
 }
 
-template <typename A, int N, int NIT>
-__global__ void __launch_bounds__(1024)
+template <typename A, int N, int NIT, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 shifted_norm_kernel(const ShiftArgs<A> a) {
   __shared__ float red[64], red1[32];
   __shared__ long long src[32];
@@ -218,6 +221,14 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       }
     }
     float f0 = a.o[0].f, f1 = a.o[1].f;
+    float u0[NIT][N], u1[NIT][N];                                       // the outputs' weights, before the wait as well
+#pragma unroll
+    for (int e = 0; e < NIT; ++e) {
+      const int i = i0 + e * step;
+      if (NIT > 1 || i >= a.W) continue;
+      if (a.o[0].w != nullptr) sh_load<N>(a.o[0].w + i, u0[e]);
+      if (a.o[1].w != nullptr) sh_load<N>(a.o[1].w + i, u1[e]);
+    }
     if (a.o[0].w != nullptr || a.o[1].w != nullptr) {
       const float2 q = block_sum2(q0, q1, red);
       if (a.o[0].w != nullptr) f0 /= sqrtf(q.x * inv_w + a.eps);
@@ -229,22 +240,30 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       const int i = i0 + e * step;
       if (i >= a.W) continue;
       if (a.o[0].y != nullptr) {
-        float w[N];
-        if (a.o[0].w != nullptr) sh_load<N>(a.o[0].w + i, w);
+        if (NIT > 1 && a.o[0].w != nullptr) sh_load<N>(a.o[0].w + i, u0[e]);
 #pragma unroll
-        for (int k = 0; k < N; ++k) v[e][k] = fmaf(y0[e][k] * f0, a.o[0].w != nullptr ? w[k] : 1.f, v[e][k]);
+        for (int k = 0; k < N; ++k) v[e][k] = fmaf(y0[e][k] * f0, a.o[0].w != nullptr ? u0[e][k] : 1.f, v[e][k]);
       }
       if (a.o[1].y != nullptr) {
-        float w[N];
-        if (a.o[1].w != nullptr) sh_load<N>(a.o[1].w + i, w);
+        if (NIT > 1 && a.o[1].w != nullptr) sh_load<N>(a.o[1].w + i, u1[e]);
 #pragma unroll
-        for (int k = 0; k < N; ++k) v[e][k] = fmaf(y1[e][k] * f1, a.o[1].w != nullptr ? w[k] : 1.f, v[e][k]);
+        for (int k = 0; k < N; ++k) v[e][k] = fmaf(y1[e][k] * f1, a.o[1].w != nullptr ? u1[e][k] : 1.f, v[e][k]);
       }
       if (own && a.x_out != nullptr) sh_store<N>(a.x_out + r * a.W + i, v[e]);
 #pragma unroll
       for (int k = 0; k < N; ++k) ss = fmaf(v[e][k], v[e][k], ss);
     }
+    // what the rest needs is asked for before the wait
+    float wn[NIT][N], ws[NIT][N];
+#pragma unroll
+    for (int e = 0; e < NIT; ++e) {
+      const int i = i0 + e * step;
+      if (NIT > 1 || i >= a.W) continue;
+      sh_load<N>(a.norm + i, wn[e]);
+      if (shifted) sh_load<N>(a.shift + i, ws[e]);
+    }
     const float inv = 1.f / sqrtf(block_sum(ss, red1) * inv_w + a.eps);
+    if (a.inv != nullptr && own && threadIdx.x == 0) a.inv[t] = inv;
     const bool keep = own && req >= 0 && pos == a.last_pos[t];
     float* st = keep ? a.then + static_cast<long long>(req) * 2 * a.W : nullptr;
 #pragma unroll
@@ -252,14 +271,14 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       const int i = i0 + e * step;
       if (i >= a.W) continue;
       float w[N], h[N], s[N];
-      sh_load<N>(a.norm + i, w);
+      if (NIT > 1) sh_load<N>(a.norm + i, wn[e]);
 #pragma unroll
-      for (int k = 0; k < N; ++k) h[k] = v[e][k] * inv * w[k];
+      for (int k = 0; k < N; ++k) h[k] = v[e][k] * inv * wn[e][k];
       if (own) sh_store_act<A, N>(a.h + static_cast<long long>(t) * a.width + i, h);
       if (!shifted) continue;
-      sh_load<N>(a.shift + i, w);
+      if (NIT > 1) sh_load<N>(a.shift + i, ws[e]);
 #pragma unroll
-      for (int k = 0; k < N; ++k) s[k] = fmaf(hp[e][k] - h[k], w[k], h[k]);
+      for (int k = 0; k < N; ++k) s[k] = fmaf(hp[e][k] - h[k], ws[e][k], h[k]);
       if (own) {
         sh_store_act<A, N>(a.s + static_cast<long long>(t) * a.width + i, s);
         for (int j = 0; j < a.blends; ++j) {
@@ -287,22 +306,115 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
   }
 }
 
+// Long steps: the sums and norms first (shifted_norm_kernel without a shift, which leaves 1 / rms of every token), then the shifted rows and
+// blends of four columns per thread over a run of tokens.  h is formed again from the residual, in fp32.
 template <typename A>
-static int launch_shifted(ShiftArgs<A> a, int decode, int sm_count, cudaStream_t st) {
+struct BlendArgs {
+  const float* x; const float* inv;
+  const float* norm; const float* shift; const float* mu;
+  A* s; A* mix;
+  const float* now; float* then;
+  const int* tok_req; const int64_t* positions; const int* first_pos; const int* last_pos;
+  int T, W, width, run;
+};
+
+template <typename A, int N, int BLENDS>
+__global__ void __launch_bounds__(256)
+shift_blend_kernel(const BlendArgs<A> a) {
+  pdl_wait();
+  pdl_trigger();
+  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * N;
+  const int r0 = blockIdx.y * a.run, r1 = min(a.T, r0 + a.run);
+  if (i >= a.W) {
+    // zeros behind the last column
+    for (int t = r0; i < a.width && t < r1; ++t)
+      for (int k = 0; k < N && i + k < a.width; ++k) {
+        st_act(a.s + static_cast<long long>(t) * a.width + i + k, 0.f);
+        for (int j = 0; j < BLENDS; ++j) st_act(a.mix + (static_cast<long long>(t) * BLENDS + j) * a.width + i + k, 0.f);
+      }
+    return;
+  }
+  float norm[N], shift[N], mu[BLENDS > 0 ? BLENDS : 1][N], hp[N], sp[N];
+  sh_load<N>(a.norm + i, norm);
+  sh_load<N>(a.shift + i, shift);
+#pragma unroll
+  for (int j = 0; j < BLENDS; ++j) sh_load<N>(a.mu + static_cast<long long>(j) * a.W + i, mu[j]);
+#pragma unroll
+  for (int k = 0; k < N; ++k) hp[k] = sp[k] = 0.f;
+  int begin = r0;
+  if (a.tok_req[r0] >= 0 && a.positions[r0] >= 0)
+    begin = r0 - static_cast<int>(min(2ll, static_cast<long long>(a.positions[r0]) - a.first_pos[r0]));
+  float next[N];
+  sh_load<N>(a.x + static_cast<long long>(begin) * a.W + i, next);
+  for (int t = begin; t < r1; ++t) {
+    const int req = a.tok_req[t];
+    const long long pos = a.positions[t];
+    const float inv = a.inv[t];
+    float h[N], s[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) h[k] = next[k] * inv * norm[k];
+    if (t + 1 < r1) sh_load<N>(a.x + (t + 1ll) * a.W + i, next);
+    if (req >= 0 && pos == a.first_pos[t]) {
+      if (pos > 0) {
+        const float* st = a.now + static_cast<long long>(req) * 2 * a.W;
+        sh_load<N>(st + i, hp);
+        sh_load<N>(st + a.W + i, sp);
+      } else {
+#pragma unroll
+        for (int k = 0; k < N; ++k) hp[k] = sp[k] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k) s[k] = fmaf(hp[k] - h[k], shift[k], h[k]);
+    if (t >= r0) {
+      sh_store_act<A, N>(a.s + static_cast<long long>(t) * a.width + i, s);
+#pragma unroll
+      for (int j = 0; j < BLENDS; ++j) {
+        float b[N];
+#pragma unroll
+        for (int k = 0; k < N; ++k) b[k] = fmaf(sp[k] - s[k], mu[j][k], s[k]);
+        sh_store_act<A, N>(a.mix + (static_cast<long long>(t) * BLENDS + j) * a.width + i, b);
+      }
+      if (req >= 0 && pos == a.last_pos[t]) {
+        float* st = a.then + static_cast<long long>(req) * 2 * a.W;
+        sh_store<N>(st + i, h);
+        sh_store<N>(st + a.W + i, s);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k) { hp[k] = h[k]; sp[k] = s[k]; }
+  }
+}
+
+constexpr int kBlendRun = 16;
+
+template <typename A>
+static int launch_shifted(ShiftArgs<A> a, float* inv, int decode, int sm_count, cudaStream_t st) {
   const bool vec = a.W % 4 == 0 && a.o[0].ld % 4 == 0 && a.o[1].ld % 4 == 0 && a.ldf % 4 == 0 && a.ldp % 4 == 0 && a.width % 4 == 0;
   const bool walk = a.shift != nullptr && !decode;
+  const ShiftArgs<A> all = a;
+  const bool split = walk && inv != nullptr && a.T > 2 * sm_count && (a.blends == 0 || a.blends == 5);
+  if (split) {
+    a.shift = nullptr;
+    a.blends = 0;
+    a.inv = inv;
+  }
   // runs: long enough that the two tokens formed again cost little, short enough to fill the SMs
   a.run = 1;
-  if (walk) {
+  if (walk && !split) {
     a.run = a.T / (2 * sm_count);
     a.run = a.run < 2 ? 2 : a.run > 16 ? 16 : a.run;
   }
   const int need = (a.W + (vec ? 4 : 1) - 1) / (vec ? 4 : 1);
   int threads = need <= 256 ? 256 : need <= 512 ? 512 : 1024;
-  if (!walk && a.T > sm_count && need <= 1024) threads = 256;
+  if ((!walk || split) && a.T > sm_count && need <= 1024) threads = 256;
   const int its = (need + threads - 1) / threads;
   const dim3 grid((a.T + a.run - 1) / a.run);
-#define STK_SHIFT(N, NIT) launch_pdl(shifted_norm_kernel<A, N, NIT>, grid, dim3(threads), 0, st, a)
+#define STK_SHIFT(N, NIT)                                                                                             \
+  do {                                                                                                                \
+    if (threads == 256) launch_pdl(shifted_norm_kernel<A, N, NIT, 256>, grid, dim3(threads), 0, st, a);               \
+    else launch_pdl(shifted_norm_kernel<A, N, NIT, 1024>, grid, dim3(threads), 0, st, a);                             \
+  } while (0)
   if (vec) {
     if (its == 1) STK_SHIFT(4, 1);
     else if (its == 2) STK_SHIFT(4, 2);
@@ -315,6 +427,18 @@ static int launch_shifted(ShiftArgs<A> a, int decode, int sm_count, cudaStream_t
     else return -2;
   }
 #undef STK_SHIFT
+  if (split) {
+    const BlendArgs<A> b{all.x_out != nullptr ? all.x_out : all.x, inv, all.norm, all.shift, all.mu, all.s, all.mix, all.now, all.then, all.tok_req,
+                         all.positions, all.first_pos, all.last_pos, all.T, all.W, all.width, kBlendRun};
+    const int n = vec ? 4 : 1, cols = (a.width + n - 1) / n;
+    const dim3 g((cols + 255) / 256, (a.T + kBlendRun - 1) / kBlendRun);
+#define STK_BLEND(N, B) launch_pdl(shift_blend_kernel<A, N, B>, g, dim3(256), 0, st, b)
+    if (vec && all.blends == 5) STK_BLEND(4, 5);
+    else if (vec) STK_BLEND(4, 0);
+    else if (all.blends == 5) STK_BLEND(1, 5);
+    else STK_BLEND(1, 0);
+#undef STK_BLEND
+  }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -359,13 +483,13 @@ STK_API int stk_embed_bigram(const int64_t* ids, const void* embed, int embed_fp
 }
 
 // y0, y1: mixer outputs (w: weight of their RMS norm, null for none); ff [T, W] fp32 rows or pairs: a token's `top` expert rows; all may be
-// null.  x_out null: the sum is not kept.  shift null: h only; rows: of these T rows.  decode: every span is one token.
+// null.  x_out null: the sum is not kept.  inv: work space [T] (or null).  shift null: h only; rows: of these T rows.  decode: every span is one token.
 STK_API int stk_shifted_norm(const float* x, float* x_out, const float* y0, long long ld0, const float* w0, float f0, const float* y1,
                              long long ld1, const float* w1, float f1, const float* ff, long long ldf, const void* pairs, long long ldp,
                              const int* pair_row, const float* weights, int top, const float* norm, float eps, const float* shift,
                              const float* mu, int blends, void* h, void* s, void* mix, int width, int fp32, const float* now, float* then,
                              const int* tok_req, const int64_t* positions, const int* first_pos, const int* last_pos, const int64_t* rows,
-                             int T, int W, int decode, int sm_count, void* stream) {
+                             float* inv, int T, int W, int decode, int sm_count, void* stream) {
   if (T <= 0) return 0;
   if (top > 32 || (pairs != nullptr && ff != nullptr) || (shift != nullptr && rows != nullptr) || blends < 0 || (rows != nullptr && x_out != nullptr) ||
       x == x_out)
@@ -373,13 +497,13 @@ STK_API int stk_shifted_norm(const float* x, float* x_out, const float* y0, long
   const ShiftOut o0{y0, ld0, w0, f0}, o1{y1, ld1, w1, f1};
   if (fp32) {
     const ShiftArgs<float> a{x, x_out, {o0, o1}, ff, ldf, (const float*)pairs, ldp, pair_row, weights, top, norm, eps, shift, mu, blends,
-                             (float*)h, (float*)s, (float*)mix, now, then, tok_req, positions, first_pos, last_pos, rows, T, W, width, 1};
-    return launch_shifted(a, decode, sm_count, (cudaStream_t)stream);
+                             (float*)h, (float*)s, (float*)mix, now, then, tok_req, positions, first_pos, last_pos, rows, T, W, width, 1, nullptr};
+    return launch_shifted(a, inv, decode, sm_count, (cudaStream_t)stream);
   }
   const ShiftArgs<__nv_bfloat16> a{x, x_out, {o0, o1}, ff, ldf, (const __nv_bfloat16*)pairs, ldp, pair_row, weights, top, norm, eps, shift, mu,
                                    blends, (__nv_bfloat16*)h, (__nv_bfloat16*)s, (__nv_bfloat16*)mix, now, then, tok_req, positions,
-                                   first_pos, last_pos, rows, T, W, width, 1};
-  return launch_shifted(a, decode, sm_count, (cudaStream_t)stream);
+                                   first_pos, last_pos, rows, T, W, width, 1, nullptr};
+  return launch_shifted(a, inv, decode, sm_count, (cudaStream_t)stream);
 }
 
 // then, now [layers, n_rows, n].

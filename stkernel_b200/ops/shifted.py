@@ -16,6 +16,7 @@ import torch
 from . import _lib
 from .hybrid import HybridMeta, _is32, expert_sum
 from .moe import ExpertRows
+from .scratch import scratch
 
 F32 = torch.float32
 
@@ -128,7 +129,8 @@ def shifted_norm(x: torch.Tensor, p: Optional[Pending], norm: torch.Tensor, eps:
               pairs.weights if pairs is not None else None, pairs.weights.shape[1] if pairs is not None else 0, norm, float(eps), shift, mu, blends,
               h, s, mix, width, _is32(h), st.now[layer] if shift is not None else None, st.then[layer] if shift is not None else None,
               meta.tok_req if shift is not None else None, meta.positions if shift is not None else None,
-              meta.first_pos if shift is not None else None, meta.last_pos if shift is not None else None, rows, n, w_n,
+              meta.first_pos if shift is not None else None, meta.last_pos if shift is not None else None, rows,
+              scratch("shift.inv", (n,), F32, dev) if shift is not None else None, n, w_n,
               1 if meta is not None and meta.pure_decode else 0, _lib.sm_count(), _lib.stream())
     return (out if out is not None else x if rows is None else None), h, s, mix
 

@@ -52,7 +52,7 @@ class TalkingParams:
 
 def talking_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, a: TalkingParams, meta: HybridMeta, table: torch.Tensor,
                  cache: torch.Tensor) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
-    """Inserts the tokens' rows into the paged cache; -> (mixed queries [T, heads * kv_heads * kp], gate logits [T, heads] fp32)."""
+    """Inserts the tokens' rows into the paged cache; -> (mixed queries [heads, T, kv_heads * kp], gate logits [T, heads] fp32)."""
     t = p.shape[0]
     h, g, d, v = a.heads, a.kv_heads, a.dim, a.vdim
     row, k_col, kp, vp = talking_row(g, d, v)
@@ -67,10 +67,10 @@ def talking_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int
         q = torch.cat([R.rotate_pairs(q[..., :n], meta.positions, a.freq), q[..., n:]], -1)
         k = torch.cat([R.rotate_pairs(k[..., :n], meta.positions, a.freq), k[..., n:]], -1)
         R.talking_kv_insert(k, vv, k_col, kp, vp, meta.positions, meta.tok_req, table, cache)
-        out = torch.zeros(t, h, g, kp, dtype=p.dtype)
-        out[..., :d] = torch.einsum("hcj,tcjd->thcd", a.talk.view(h, g, h // g), q.view(t, g, h // g, d)).to(p.dtype)
-        return out.flatten(1), p[:, g_off:g_off + h].to(F32) if a.gated else None
-    out = torch.empty(t, h * g * kp, dtype=p.dtype, device=p.device)       # whole 16-byte units: kp is a multiple of 16
+        out = torch.zeros(h, t, g, kp, dtype=p.dtype)
+        out[..., :d] = torch.einsum("hcj,tcjd->htcd", a.talk.view(h, g, h // g), q.view(t, g, h // g, d)).to(p.dtype)
+        return out.flatten(2), p[:, g_off:g_off + h].to(F32) if a.gated else None
+    out = torch.empty(h, t, g * kp, dtype=p.dtype, device=p.device)
     gate = torch.empty(t, h, dtype=F32, device=p.device) if a.gated else None
     _lib.call("stk_talking_prep", p, p.stride(0), q_off, k_off, v_off, g_off, a.bias, a.q_norm, a.k_norm, float(a.eps), a.freq, a.freq.shape[1],
               a.talk, meta.positions, meta.tok_req, table, table.stride(0), cache, row, k_col, kp, vp, h, g, d, v, out, gate, _is32(p), t,
@@ -81,18 +81,20 @@ def talking_prep(p: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int
 def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], a: TalkingParams, meta: HybridMeta, table: torch.Tensor,
                       cache: torch.Tensor, out: torch.Tensor) -> None:
     """q, gate: `talking_prep` of the step.  Writes the gated heads' outputs into out[:, : heads * vdim], zeros behind them."""
-    t = q.shape[0]
+    t = out.shape[0]
     h, g, d, v = a.heads, a.kv_heads, a.dim, a.vdim
     row, k_col, kp, vp = talking_row(g, d, v)
+    if q.shape != (h, t, g * kp) or out.shape[1] < h * v:
+        raise ValueError(f"mixed queries {tuple(q.shape)} do not fit outputs {tuple(out.shape)}")
     if not q.is_cuda:
-        o = R.talking_attention(q.view(t, h, g * kp), v, vp, g, k_col, meta.positions, meta.tok_req, table, cache, a.scale, a.chunk, a.sink)
+        o = R.talking_attention(q.transpose(0, 1), v, vp, g, k_col, meta.positions, meta.tok_req, table, cache, a.scale, a.chunk, a.sink)
         if gate is not None:
             o = o * torch.sigmoid(gate)[..., None]
         out[:, h * v:] = 0
         out[:, :h * v] = o.flatten(1).to(out.dtype)
         return
     shape = (row, k_col, kp, vp, h, g, v, a.chunk, float(a.scale), out, out.stride(0), out.shape[1])
-    common = (q, q.stride(0), gate, a.sink, meta.positions, meta.tok_req, table, table.stride(0), cache, *shape)
+    common = (q, gate, a.sink, meta.positions, meta.tok_req, table, table.stride(0), cache, *shape)
     prompt = (not _is32(q) and meta.max_span >= PROMPT_SPAN and meta.spans is not None
               and _lib.query("stk_talking_prompt_ok", h, g, kp, vp, v) == 1)
     if not prompt or meta.min_span < PROMPT_SPAN:
@@ -111,7 +113,7 @@ def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], a: TalkingP
         rows = torch.empty(n_rows, row, dtype=q.dtype, device=q.device)
         _lib.call("stk_talking_rows", meta.query_start, meta.req_rows, meta.start_pos, meta.n_req, PROMPT_SPAN, a.chunk, table, table.stride(0),
                   cache, row, rows, n_rows, _lib.stream())
-        _lib.call("stk_talking_prompt", q, q.stride(0), gate, a.sink, rows, n_rows, *shape, meta.query_start, meta.start_pos, meta.n_req,
+        _lib.call("stk_talking_prompt", q, gate, a.sink, rows, n_rows, *shape, meta.query_start, meta.start_pos, meta.n_req,
                   PROMPT_SPAN, t, _lib.status_buffer(), _lib.stream())
 
 

@@ -224,7 +224,7 @@ def test_attention_kernels_agree_over_many_pages(c, chunk):
     out = torch.full((n, al(H * V)), float("nan"), dtype=BF16, device=dev)
     TK.talking_attention(q, gate, a, meta, table, cache, out)
     ref = torch.empty_like(out)
-    _lib.call("stk_talking_simt", q, q.stride(0), gate, a.sink, meta.positions, meta.tok_req, table, table.stride(0), cache, row, k_col, kp, vp, H, G,
+    _lib.call("stk_talking_simt", q, gate, a.sink, meta.positions, meta.tok_req, table, table.stride(0), cache, row, k_col, kp, vp, H, G,
               V, chunk, a.scale, ref, ref.stride(0), ref.shape[1], 0, meta.first_pos, meta.last_pos, 1 << 30, n, _lib.stream())
     x, y = out[:, :H * V].float(), ref[:, :H * V].float()
     assert torch.isfinite(x).all()
