@@ -107,12 +107,12 @@ linear_scan_kernel(const Front f, const ScanArgs a, int min_span, int max_span) 
             acc[c] = fmaf(qd, fmaf(ud, v[c], S[j][c]), acc[c]);
             S[j][c] = fmaf(wd.x, S[j][c], fmaf(wd.y, S[j][c], kd * v[c]));
           }
-          continue;
-        }
+        } else {
 #pragma unroll
-        for (int c = 0; c < VEC; ++c) {
-          S[j][c] = fmaf(decay.x, S[j][c], fmaf(decay.y, S[j][c], kd * v[c]));
-          acc[c] = fmaf(qd, S[j][c], acc[c]);
+          for (int c = 0; c < VEC; ++c) {
+            S[j][c] = fmaf(decay.x, S[j][c], fmaf(decay.y, S[j][c], kd * v[c]));
+            acc[c] = fmaf(qd, S[j][c], acc[c]);
+          }
         }
       }
     }

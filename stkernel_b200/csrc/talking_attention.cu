@@ -23,9 +23,21 @@ struct TalkPrepArgs {
   void* q; float* gate;
 };
 
+__device__ __forceinline__ void talk_load4(const float* p, float (&v)[4]) {
+  const float4 f = *reinterpret_cast<const float4*>(p);
+  v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void talk_load4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+}
+
 // HG: heads per key/value head (their queries stay in registers while the heads' mixtures are formed), 0: any number.  grid (T, parts): a
 // part forms the mixtures of its share of the heads; the first one also writes the cached row and the gate logits.
-template <typename A, int HG>
+// VEC: heads of at most 128 columns in whole aligned groups of four.
+template <typename A, int HG, bool VEC>
 __global__ void __launch_bounds__(512)
 talking_prep_kernel(const TalkPrepArgs a) {
   extern __shared__ __align__(16) float sm[];
@@ -52,41 +64,76 @@ talking_prep_kernel(const TalkPrepArgs a) {
     return;
   }
   const int page = a.table[static_cast<long long>(req) * a.bt_stride + pos / kTkPage];
-  for (int u0 = warp; u0 < a.H + a.G; u0 += warps) {
-    const bool isq = u0 < a.H;
-    const A* src = p + (isq ? a.q_off + u0 * a.D : a.k_off + (u0 - a.H) * a.D);
-    const float* w = isq ? a.q_norm : a.k_norm;
-    float* dst = x + u0 * D2;
-    float s = 0.f;
-    for (int d = lane; d < D2; d += 32) {
-      const float v = d < a.D ? ld_act(src + d) + (a.bias != nullptr ? a.bias[u0 * a.D + d] : 0.f) : 0.f;
-      dst[d] = v;
-      s = fmaf(v, v, s);
-    }
-    if (w != nullptr) {
-      const float f = 1.f / sqrtf(warp_sum(s) / static_cast<float>(a.D) + a.eps);
-      for (int d = lane; d < a.D; d += 32) dst[d] *= f * w[d];
-    }
-  }
   for (int i = threadIdx.x; i < a.pairs; i += blockDim.x) cs[i] = cos_sin_split(pos, a.freq[i], a.freq[a.pairs + i]);
-  for (int i = threadIdx.x; i < (h1 - h0) * a.H; i += blockDim.x) talk[i / a.H * H4 + i % a.H] = a.talk[h0 * a.H + i];
+  for (int h = h0 + warp; h < h1; h += warps)
+    for (int i = lane; i < a.H; i += 32) talk[(h - h0) * H4 + i] = a.talk[h * a.H + i];
   __syncthreads();
-  for (int e = threadIdx.x; e < (a.H + a.G) * a.pairs; e += blockDim.x) {
-    const int u = e / a.pairs, i = e - u * a.pairs;
-    float2* v = reinterpret_cast<float2*>(x + u * D2 + 2 * i);
-    const float2 c = *v, w = cs[i];
-    *v = make_float2(c.x * w.x - c.y * w.y, c.y * w.x + c.x * w.y);
+  if (VEC) {
+    // four neighbouring columns per lane: norm and rotation in registers
+    for (int u0 = warp; u0 < a.H + a.G; u0 += warps) {
+      const bool isq = u0 < a.H;
+      const A* src = p + (isq ? a.q_off + u0 * a.D : a.k_off + (u0 - a.H) * a.D);
+      const float* w = isq ? a.q_norm : a.k_norm;
+      const int d = lane * 4;
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+      if (d < a.D) {
+        talk_load4(src + d, v);
+        if (a.bias != nullptr) {
+          const float4 b = *reinterpret_cast<const float4*>(a.bias + u0 * a.D + d);
+          v[0] += b.x; v[1] += b.y; v[2] += b.z; v[3] += b.w;
+        }
+      }
+      if (w != nullptr) {
+        const float s = fmaf(v[0], v[0], fmaf(v[1], v[1], fmaf(v[2], v[2], v[3] * v[3])));
+        const float f = 1.f / sqrtf(warp_sum(s) / static_cast<float>(a.D) + a.eps);
+        if (d < a.D) {
+          const float4 y = *reinterpret_cast<const float4*>(w + d);
+          v[0] *= f * y.x; v[1] *= f * y.y; v[2] *= f * y.z; v[3] *= f * y.w;
+        }
+      }
+      if (d >= a.D) continue;
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (lane * 2 + j < a.pairs) {
+          const float2 c = cs[lane * 2 + j];
+          const float x0 = v[2 * j], x1 = v[2 * j + 1];
+          v[2 * j] = x0 * c.x - x1 * c.y;
+          v[2 * j + 1] = x1 * c.x + x0 * c.y;
+        }
+      *reinterpret_cast<float4*>(x + u0 * D2 + d) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+  } else {
+    for (int u0 = warp; u0 < a.H + a.G; u0 += warps) {
+      const bool isq = u0 < a.H;
+      const A* src = p + (isq ? a.q_off + u0 * a.D : a.k_off + (u0 - a.H) * a.D);
+      const float* w = isq ? a.q_norm : a.k_norm;
+      float* dst = x + u0 * D2;
+      float s = 0.f;
+      for (int d = lane; d < D2; d += 32) {
+        const float v = d < a.D ? ld_act(src + d) + (a.bias != nullptr ? a.bias[u0 * a.D + d] : 0.f) : 0.f;
+        dst[d] = v;
+        s = fmaf(v, v, s);
+      }
+      if (w != nullptr) {
+        const float f = 1.f / sqrtf(warp_sum(s) / static_cast<float>(a.D) + a.eps);
+        for (int d = lane; d < a.D; d += 32) dst[d] *= f * w[d];
+      }
+      __syncwarp();
+      for (int i = lane; i < a.pairs; i += 32) {
+        float2* v = reinterpret_cast<float2*>(dst + 2 * i);
+        const float2 c = *v, w2 = cs[i];
+        *v = make_float2(c.x * w2.x - c.y * w2.y, c.y * w2.x + c.x * w2.y);
+      }
+    }
   }
   __syncthreads();
   if (lead && page >= 0) {
     A* row = reinterpret_cast<A*>(a.cache) + (static_cast<long long>(page) * kTkPage + pos % kTkPage) * a.row;
-    for (int e = threadIdx.x; e < a.G * a.vp; e += blockDim.x) {
-      const int g = e / a.vp, d = e - g * a.vp;
-      st_act(row + e, d < a.V ? ld_act(p + a.v_off + g * a.V + d) + (a.bias != nullptr ? a.bias[(a.H + a.G) * a.D + g * a.V + d] : 0.f) : 0.f);
-    }
-    for (int e = threadIdx.x; e < KD; e += blockDim.x) {
-      const int g = e / a.kp, d = e - g * a.kp;
-      st_act(row + a.k_col + e, d < a.D ? x[(a.H + g) * D2 + d] : 0.f);
+    for (int g = warp; g < a.G; g += warps) {
+      const A* v = p + a.v_off + g * a.V;
+      const float* b = a.bias != nullptr ? a.bias + (a.H + a.G) * a.D + g * a.V : nullptr;
+      for (int d = lane; d < a.vp; d += 32) st_act(row + g * a.vp + d, d < a.V ? ld_act(v + d) + (b != nullptr ? b[d] : 0.f) : 0.f);
+      for (int d = lane; d < a.kp; d += 32) st_act(row + a.k_col + g * a.kp + d, d < a.D ? x[(a.H + g) * D2 + d] : 0.f);
     }
   }
   // four columns of the mixtures of every other, fourth, ... head (kp is a multiple of 4)
@@ -104,7 +151,19 @@ talking_prep_kernel(const TalkPrepArgs a) {
     for (int h = h0 + lot; h < h1; h += lots) {
       const float* w = talk + (h - h0) * H4 + c * hg;
       float4 s = zero;
-      if (HG > 0) {
+      if (HG > 0 && HG % 4 == 0) {
+#pragma unroll
+        for (int g0 = 0; g0 < HG; g0 += 4) {
+          const float4 wv = *reinterpret_cast<const float4*>(w + g0);
+          const float wg[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            const float4 y = qv[HG > 0 ? g0 + g : 0];
+            s.x = fmaf(wg[g], y.x, s.x); s.y = fmaf(wg[g], y.y, s.y);
+            s.z = fmaf(wg[g], y.z, s.z); s.w = fmaf(wg[g], y.w, s.w);
+          }
+        }
+      } else if (HG > 0) {
 #pragma unroll
         for (int g = 0; g < HG; ++g) {
           s.x = fmaf(w[g], qv[g].x, s.x); s.y = fmaf(w[g], qv[g].y, s.y);
@@ -213,13 +272,19 @@ static int launch_talk_prep(const TalkPrepArgs& a, int T, cudaStream_t st) {
   const int parts = T >= 148 ? 1 : min((a.H + 3) / 4, 8), per = (a.H + parts - 1) / parts, threads = T >= 148 ? 256 : 512;
   const size_t smem = (static_cast<size_t>(a.H + a.G) * ((a.D + 3) & ~3) + per * ((a.H + 3) & ~3) + 2 * a.pairs) * sizeof(float);
   if (smem > 200 * 1024) return -2;
-#define STK_TALK_PREP(HG)                                                                                                       \
+  const uintptr_t at = reinterpret_cast<uintptr_t>(a.proj);
+  const bool vec = a.D % 4 == 0 && a.D <= 128 && a.ldp % 4 == 0 && (a.q_off | a.k_off) % 4 == 0 && (at & 15) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.bias) | reinterpret_cast<uintptr_t>(a.q_norm) | reinterpret_cast<uintptr_t>(a.k_norm)) & 15) == 0;
+#define STK_TALK_PREP_AS(HG, VEC)                                                                                               \
   {                                                                                                                             \
-    if (smem > 40 * 1024 && cudaFuncSetAttribute(talking_prep_kernel<A, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(talking_prep_kernel<A, HG, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
                                                  200 * 1024) != cudaSuccess)                                                    \
       return -3;                                                                                                                \
-    launch_pdl(talking_prep_kernel<A, HG>, dim3(T, parts), dim3(threads), smem, st, a);                                            \
+    launch_pdl(talking_prep_kernel<A, HG, VEC>, dim3(T, parts), dim3(threads), smem, st, a);                                    \
   }
+#define STK_TALK_PREP(HG)                 \
+  if (vec) STK_TALK_PREP_AS(HG, true)     \
+  else STK_TALK_PREP_AS(HG, false)
   switch (a.H / a.G) {
     case 1: STK_TALK_PREP(1) break;
     case 2: STK_TALK_PREP(2) break;
@@ -228,6 +293,7 @@ static int launch_talk_prep(const TalkPrepArgs& a, int T, cudaStream_t st) {
     default: STK_TALK_PREP(0) break;
   }
 #undef STK_TALK_PREP
+#undef STK_TALK_PREP_AS
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -130,23 +130,43 @@ time_mix_keys_kernel(const TmArgs a, int min_span, __nv_bfloat16* __restrict__ k
 }
 
 constexpr int kTmOutThreads = 256;
-struct TmOutLayout { int ks, q, k, r, kr, v, w, f, p, bytes; };                   // byte offsets
+struct TmOutLayout { int ks, q, r, v, wk, w, f, p, bytes; };                      // byte offsets
 __host__ __device__ inline TmOutLayout tm_out_layout(int D) {
   TmOutLayout l;
   const int Dp = blocks16(D) * 16;
   l.ks = Dp + 8;
-  const int tile = kChunk * l.ks * 2;
+  const int tile = kChunk * l.ks * 2, scores = 2 * kChunk * kStStride * 2;
   l.q = 0;                                        // [2][64][ks] r~ as pair
-  l.k = 2 * tile;                                 // [2][64][ks] k^ as pair, later the weighted scores [2][64][72]
-  const int scores = 2 * kChunk * kStStride * 2;
-  l.r = l.k + (2 * tile > scores ? 2 * tile : scores);          // [64][ks]
-  l.kr = l.r + tile;
-  l.v = l.kr + tile;
-  l.w = l.v + tile;                               // [64][Dp] fp32 decays
-  l.f = l.w + kChunk * Dp * 4;                    // [7][Dp] fp32: decays of blocks 1, 2, 1 and 2, 0, 0 and 1, 0 to 2; the bonus
+  l.r = 2 * tile;                                 // [64][ks]
+  l.v = l.r + tile;                               // [64][ks]
+  l.wk = l.v + tile;                              // k [64][ks], then at w decays [64][Dp] fp32; later k^ as pair [2][64][ks]; then the weighted
+  l.w = l.wk + tile;                              // scores [2][64][72]
+  const int first = tile + kChunk * Dp * 4, second = 2 * tile > scores ? 2 * tile : scores;
+  l.f = l.wk + (first > second ? first : second); // [7][Dp] fp32: decays of blocks 1, 2, 1 and 2, 0, 0 and 1, 0 to 2; the bonus
   l.p = l.f + 7 * Dp * 4;                         // [4][Dp] sums of the blocks
   l.bytes = l.p + 4 * Dp * 4;
   return l;
+}
+// packed pairs of fp32
+__device__ __forceinline__ uint64_t tm_pack2(float x, float y) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void tm_unpack2(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
+__device__ __forceinline__ uint64_t tm_fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t tm_mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+// Two bf16 as a pair of fp32.
+__device__ __forceinline__ uint64_t tm_widen2(uint32_t v) {
+  return tm_pack2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
 }
 
 // An operand pair times a factor per column (columns 2 (lane & 3), + 1, and 8 further).
@@ -162,7 +182,7 @@ __device__ __forceinline__ void tm_scale_pair(uint32_t (&hi)[4], uint32_t (&lo)[
 }
 
 // One CTA per (chunk, head).
-__global__ void __launch_bounds__(kTmOutThreads)
+__global__ void __launch_bounds__(kTmOutThreads, 3)
 time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ states) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ ChunkRef s_c;
@@ -171,12 +191,12 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
   const TmOutLayout L = tm_out_layout(D);
   const int ks = L.ks, part = kChunk * ks;
   __nv_bfloat16* q = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.q);
-  __nv_bfloat16* k = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.k);
-  __nv_bfloat16* ph = k;
-  __nv_bfloat16* pl = ph + kChunk * kStStride;
   __nv_bfloat16* r = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.r);
-  __nv_bfloat16* kr = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.kr);
   __nv_bfloat16* v = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.v);
+  __nv_bfloat16* kr = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.wk);
+  __nv_bfloat16* k = kr;                                                 // k^, after the keys and the decays are done with
+  __nv_bfloat16* ph = kr;                                                // weighted scores, after k^
+  __nv_bfloat16* pl = ph + kChunk * kStStride;
   float* w = reinterpret_cast<float*>(smem_raw + L.w);
   float* f = reinterpret_cast<float*>(smem_raw + L.f);
   float* sums = reinterpret_cast<float*>(smem_raw + L.p);
@@ -194,39 +214,29 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
   load_rows_async(v, ks, Dp, p + 2 * a.np, a.ldp, c.n, D, kTmOutThreads);
   mls_commit();
   for (int d = threadIdx.x; d < Dp; d += kTmOutThreads) f[6 * Dp + d] = d < D ? a.u[h * D + d] : 0.f;
-  float g[kTmSub], w0 = 0.f;
-  auto fetch = [&](int e) {
-    const int b = e / Dp, d = e - b * Dp;
+  // a thread's (block, channel) in every round: at most two rounds, up to 128 channels
+  float g[2][kTmSub];
 #pragma unroll
-    for (int i = 0; i < kTmSub; ++i) g[i] = d < D && b * kTmSub + i < c.n ? a.z[(c.t0 + b * kTmSub + i) * a.ldz + h * D + d] : 0.f;
-    w0 = d < D ? a.w0[h * D + d] : 0.f;
-  };
-  if (threadIdx.x < kTmBlocks * Dp) fetch(threadIdx.x);
-  mls_wait<0>();
-  __syncthreads();
-  // r~ and k^ of every block, the decays themselves
-  for (int e = threadIdx.x; e < kTmBlocks * Dp; e += kTmOutThreads) {
-    const int b = e / Dp, d = e - b * Dp;
-    if (e >= kTmOutThreads) fetch(e);
-    float sum = 0.f;
+  for (int m = 0; m < 2; ++m) {
+    const int e = threadIdx.x + m * kTmOutThreads, b = e / Dp, d = e - b * Dp;
+    const bool in = e < kTmBlocks * Dp && d < D;
+    if (m > 0 && Dp <= 64) continue;
+    const float w0 = in ? a.w0[h * D + d] : 0.f;
 #pragma unroll
-    for (int i = 0; i < kTmSub; ++i) g[i] = d < D && b * kTmSub + i < c.n ? -__expf(g[i] + w0) : 0.f;
+    for (int i = 0; i < kTmSub; ++i) g[m][i] = in && b * kTmSub + i < c.n ? a.z[(c.t0 + b * kTmSub + i) * a.ldz + h * D + d] : 0.f;
 #pragma unroll
-    for (int i = 0; i < kTmSub; ++i) {
-      const int n = b * kTmSub + i;
-      mls_split(bf16_to_f(r[n * ks + d]) * __expf(sum), q[n * ks + d], q[part + n * ks + d]);
-      w[n * Dp + d] = __expf(g[i]);
-      sum += g[i];
-    }
-    sums[b * Dp + d] = sum;
-    float left = 0.f;
+    for (int i = 0; i < kTmSub; ++i) g[m][i] = in && b * kTmSub + i < c.n ? -__expf(g[m][i] + w0) : 0.f;
+    if (e < kTmBlocks * Dp) {
+      float sum = 0.f;
 #pragma unroll
-    for (int i = kTmSub - 1; i >= 0; --i) {
-      const int n = b * kTmSub + i;
-      mls_split(bf16_to_f(kr[n * ks + d]) * __expf(left), k[n * ks + d], k[part + n * ks + d]);
-      left += g[i];
+      for (int i = 0; i < kTmSub; ++i) {
+        w[(b * kTmSub + i) * Dp + d] = __expf(g[m][i]);
+        sum += g[m][i];
+      }
+      sums[b * Dp + d] = sum;
     }
   }
+  mls_wait<0>();
   __syncthreads();
   for (int d = threadIdx.x; d < Dp; d += kTmOutThreads) {
     const float s0 = sums[d], s1 = sums[Dp + d], s2 = sums[2 * Dp + d];
@@ -243,39 +253,72 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
 #pragma unroll
   for (int i = 0; i < kTmSub; ++i) acc[i] = 0.f;
   for (int c0 = seg * 4; c0 < Dp; c0 += 16) {
-    auto four = [&](const __nv_bfloat16* src, float (&x)[4]) {
-      const uint2 y = *reinterpret_cast<const uint2*>(src);
-      const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.x));
-      const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.y));
-      x[0] = lo.x; x[1] = lo.y; x[2] = hi.x; x[3] = hi.y;
-    };
-    float x[4], y[4];
-    four(kr + (jb * kTmSub + j) * ks + c0, x);
-    four(r + (jb * kTmSub + j) * ks + c0, y);
-    const float4 u = *reinterpret_cast<const float4*>(f + 6 * Dp + c0);
-    bonus = fmaf(y[0] * u.x, x[0], fmaf(y[1] * u.y, x[1], fmaf(y[2] * u.z, x[2], fmaf(y[3] * u.w, x[3], bonus))));
+    const uint2 kv = *reinterpret_cast<const uint2*>(kr + (jb * kTmSub + j) * ks + c0);
+    const uint2 rv = *reinterpret_cast<const uint2*>(r + (jb * kTmSub + j) * ks + c0);
+    uint64_t x0 = tm_widen2(kv.x), x1 = tm_widen2(kv.y);
+    const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(f + 6 * Dp + c0);
+    float s0, s1;
+    tm_unpack2(tm_fma2(tm_mul2(tm_widen2(rv.x), u.x), x0, tm_mul2(tm_mul2(tm_widen2(rv.y), u.y), x1)), s0, s1);
+    bonus += s0 + s1;
 #pragma unroll
     for (int i = 1; i < kTmSub; ++i) {
       if (i < 9 && (warp & 1)) continue;                                 // the warp's columns start behind these rows
-      const float4 wi = *reinterpret_cast<const float4*>(w + (jb * kTmSub + i) * Dp + c0);
-      four(r + (jb * kTmSub + i) * ks + c0, y);
+      const ulonglong2 wi = *reinterpret_cast<const ulonglong2*>(w + (jb * kTmSub + i) * Dp + c0);
+      const uint2 y = *reinterpret_cast<const uint2*>(r + (jb * kTmSub + i) * ks + c0);
+      tm_unpack2(tm_fma2(tm_widen2(y.x), x0, tm_mul2(tm_widen2(y.y), x1)), s0, s1);
       const bool below = i > j;
-      const float s = fmaf(y[0], x[0], fmaf(y[1], x[1], fmaf(y[2], x[2], y[3] * x[3])));
-      acc[i] += below ? s : 0.f;
-      x[0] = below ? x[0] * wi.x : x[0];
-      x[1] = below ? x[1] * wi.y : x[1];
-      x[2] = below ? x[2] * wi.z : x[2];
-      x[3] = below ? x[3] * wi.w : x[3];
+      acc[i] += below ? s0 + s1 : 0.f;
+      x0 = below ? tm_mul2(x0, wi.x) : x0;
+      x1 = below ? tm_mul2(x1, wi.y) : x1;
     }
   }
   bonus += __shfl_xor_sync(0xffffffffu, bonus, 1);
   bonus += __shfl_xor_sync(0xffffffffu, bonus, 2);
+  // k^ of every block in registers, r~ to its place
+  uint32_t kh[2][kTmSub / 2], kl[2][kTmSub / 2];                         // two tokens each
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const int e = threadIdx.x + m * kTmOutThreads, b = e / Dp, d = e - b * Dp;
+    if ((m > 0 && Dp <= 64) || e >= kTmBlocks * Dp) continue;
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kTmSub; ++i) {
+      const int n = b * kTmSub + i;
+      mls_split(bf16_to_f(r[n * ks + d]) * __expf(sum), q[n * ks + d], q[part + n * ks + d]);
+      sum += g[m][i];
+    }
+    float left = 0.f;
+#pragma unroll
+    for (int i = kTmSub / 2 - 1; i >= 0; --i) {
+      const int n = b * kTmSub + 2 * i;
+      const float y1 = bf16_to_f(kr[(n + 1) * ks + d]) * __expf(left);
+      left += g[m][2 * i + 1];
+      const float y0 = bf16_to_f(kr[n * ks + d]) * __expf(left);
+      left += g[m][2 * i];
+      mls_split2(y0, y1, kh[m][i], kl[m][i]);
+    }
+  }
 #pragma unroll
   for (int i = 0; i < kTmSub; ++i) {
     acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 1);
     acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 2);
   }
-  __syncthreads();                                                       // the factors are in
+  __syncthreads();                                                       // keys and decays are done with
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const int e = threadIdx.x + m * kTmOutThreads, b = e / Dp, d = e - b * Dp;
+    if ((m > 0 && Dp <= 64) || e >= kTmBlocks * Dp) continue;
+#pragma unroll
+    for (int i = 0; i < kTmSub / 2; ++i) {
+      __nv_bfloat16* to = k + (b * kTmSub + 2 * i) * ks + d;
+      const __nv_bfloat162 hi = *reinterpret_cast<const __nv_bfloat162*>(&kh[m][i]), lo = *reinterpret_cast<const __nv_bfloat162*>(&kl[m][i]);
+      to[0] = hi.x;
+      to[ks] = hi.y;
+      to[part] = lo.x;
+      to[part + ks] = lo.y;
+    }
+  }
+  __syncthreads();
   // the six blocks below the diagonal, one per warp
   uint32_t wh[4], wl[4];
   int rb = 0, kb = 0;

@@ -5,7 +5,8 @@
 //                     and s' are the previous token's h and s
 //   shift_commit      the last h, s and token of every request's span become its state
 //
-//   shift_blend       s and the blends of a long step, after its sums and norms
+//   sum_norm          x and h alone: the model's last norm, and the first half of long steps
+//   shift_blend       s and the blends of long steps, from x and 1 / rms
 //
 // shifted_norm: a CTA walks a run of consecutive tokens with h' and s' in registers.  At the start of a run it forms h of the two tokens
 // before it once more (s' needs the h before that), at the start of a span it takes h' and s' from the request's state.  The new
@@ -118,6 +119,44 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
   return make_float2(warp_sum(a), warp_sum(b));
 }
 
+// v += N columns of the feed-forward's output: a row, or the weighted sum of a token's expert rows.
+template <typename A, int N>
+__device__ __forceinline__ void sh_tail(const ShiftArgs<A>& a, long long r, int i, const long long* src, const float* wt, float (&v)[N]) {
+  if (a.ff != nullptr) {
+    float f[N];
+    sh_load<N>(a.ff + r * a.ldf + i, f);
+#pragma unroll
+    for (int k = 0; k < N; ++k) v[k] += f[k];
+  }
+  if (a.pairs != nullptr) {
+    float f[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) f[k] = 0.f;
+    if constexpr (N == 4 && sizeof(A) == 2) {
+      for (int j0 = 0; j0 < a.top; j0 += 4) {                 // four rows in flight
+        uint2 q[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          q[j] = j0 + j < a.top ? *reinterpret_cast<const uint2*>(a.pairs + src[j0 + j] + i) : make_uint2(0, 0);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float w = j0 + j < a.top ? wt[j0 + j] : 0.f;
+          const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j].x));
+          const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j].y));
+          f[0] = fmaf(w, f0.x, f[0]); f[1] = fmaf(w, f0.y, f[1]);
+          f[2] = fmaf(w, f1.x, f[2]); f[3] = fmaf(w, f1.y, f[3]);
+        }
+      }
+    } else {
+      for (int j = 0; j < a.top; ++j)
+#pragma unroll
+        for (int k = 0; k < N; ++k) f[k] = fmaf(wt[j], ld_act(a.pairs + src[j] + i + k), f[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k) v[k] += f[k];
+  }
+}
+
 template <typename A, int N, int NIT, int THREADS>
 __global__ void __launch_bounds__(THREADS)
 shifted_norm_kernel(const ShiftArgs<A> a) {
@@ -128,10 +167,9 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
   pdl_trigger();
   const int step = blockDim.x * N, i0 = threadIdx.x * N;
   const int r0 = blockIdx.x * a.run, r1 = min(a.T, r0 + a.run);
-  const bool shifted = a.shift != nullptr;
   const float inv_w = 1.f / static_cast<float>(a.W);
   int begin = r0;
-  if (shifted && a.run > 1 && a.tok_req[r0] >= 0 && a.positions[r0] >= 0)
+  if (a.run > 1 && a.tok_req[r0] >= 0 && a.positions[r0] >= 0)
     begin = r0 - static_cast<int>(min(2ll, static_cast<long long>(a.positions[r0]) - a.first_pos[r0]));
   float hp[NIT][N], sp[NIT][N];
 #pragma unroll
@@ -140,24 +178,20 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
     for (int k = 0; k < N; ++k) hp[e][k] = sp[e][k] = 0.f;
   for (int t = begin; t < r1; ++t) {
     const bool own = t >= r0;
-    const long long r = a.rows != nullptr ? a.rows[t] : static_cast<long long>(t);
-    int req = -1;
-    long long pos = -1;
-    if (shifted) {
-      req = a.tok_req[t];
-      pos = a.positions[t];
-      if (req >= 0 && pos == a.first_pos[t]) {
-        const float* st = a.now + static_cast<long long>(req) * 2 * a.W;
+    const long long r = t;
+    const int req = a.tok_req[t];
+    const long long pos = a.positions[t];
+    if (req >= 0 && pos == a.first_pos[t]) {
+      const float* st = a.now + static_cast<long long>(req) * 2 * a.W;
 #pragma unroll
-        for (int e = 0; e < NIT; ++e) {
-          const int i = i0 + e * step;
-          if (pos > 0 && i < a.W) {
-            sh_load<N>(st + i, hp[e]);
-            sh_load<N>(st + a.W + i, sp[e]);
-          } else {
+      for (int e = 0; e < NIT; ++e) {
+        const int i = i0 + e * step;
+        if (pos > 0 && i < a.W) {
+          sh_load<N>(st + i, hp[e]);
+          sh_load<N>(st + a.W + i, sp[e]);
+        } else {
 #pragma unroll
-            for (int k = 0; k < N; ++k) hp[e][k] = sp[e][k] = 0.f;
-          }
+          for (int k = 0; k < N; ++k) hp[e][k] = sp[e][k] = 0.f;
         }
       }
     }
@@ -181,39 +215,7 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       sh_load<N>(a.x + r * a.W + i, v[e]);
       if (a.o[0].y != nullptr) sh_load<N>(a.o[0].y + r * a.o[0].ld + i, y0[e]);
       if (a.o[1].y != nullptr) sh_load<N>(a.o[1].y + r * a.o[1].ld + i, y1[e]);
-      if (a.ff != nullptr) {
-        float f[N];
-        sh_load<N>(a.ff + r * a.ldf + i, f);
-#pragma unroll
-        for (int k = 0; k < N; ++k) v[e][k] += f[k];
-      }
-      if (a.pairs != nullptr) {
-        float f[N];
-#pragma unroll
-        for (int k = 0; k < N; ++k) f[k] = 0.f;
-        if constexpr (N == 4 && sizeof(A) == 2) {
-          for (int j0 = 0; j0 < a.top; j0 += 4) {                 // four rows in flight
-            uint2 q[4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-              q[j] = j0 + j < a.top ? *reinterpret_cast<const uint2*>(a.pairs + src[j0 + j] + i) : make_uint2(0, 0);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const float w = j0 + j < a.top ? wt[j0 + j] : 0.f;
-              const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j].x));
-              const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j].y));
-              f[0] = fmaf(w, f0.x, f[0]); f[1] = fmaf(w, f0.y, f[1]);
-              f[2] = fmaf(w, f1.x, f[2]); f[3] = fmaf(w, f1.y, f[3]);
-            }
-          }
-        } else {
-          for (int j = 0; j < a.top; ++j)
-#pragma unroll
-            for (int k = 0; k < N; ++k) f[k] = fmaf(wt[j], ld_act(a.pairs + src[j] + i + k), f[k]);
-        }
-#pragma unroll
-        for (int k = 0; k < N; ++k) v[e][k] += f[k];
-      }
+      sh_tail<A, N>(a, r, i, src, wt, v[e]);
 #pragma unroll
       for (int k = 0; k < N; ++k) {
         q0 = fmaf(y0[e][k], y0[e][k], q0);
@@ -260,10 +262,9 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       const int i = i0 + e * step;
       if (NIT > 1 || i >= a.W) continue;
       sh_load<N>(a.norm + i, wn[e]);
-      if (shifted) sh_load<N>(a.shift + i, ws[e]);
+      sh_load<N>(a.shift + i, ws[e]);
     }
     const float inv = 1.f / sqrtf(block_sum(ss, red1) * inv_w + a.eps);
-    if (a.inv != nullptr && own && threadIdx.x == 0) a.inv[t] = inv;
     const bool keep = own && req >= 0 && pos == a.last_pos[t];
     float* st = keep ? a.then + static_cast<long long>(req) * 2 * a.W : nullptr;
 #pragma unroll
@@ -275,7 +276,6 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
 #pragma unroll
       for (int k = 0; k < N; ++k) h[k] = v[e][k] * inv * wn[e][k];
       if (own) sh_store_act<A, N>(a.h + static_cast<long long>(t) * a.width + i, h);
-      if (!shifted) continue;
       if (NIT > 1) sh_load<N>(a.shift + i, ws[e]);
 #pragma unroll
       for (int k = 0; k < N; ++k) s[k] = fmaf(hp[e][k] - h[k], ws[e][k], h[k]);
@@ -299,15 +299,93 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
     if (own)
       for (int i = a.W + threadIdx.x; i < a.width; i += blockDim.x) {
         st_act(a.h + static_cast<long long>(t) * a.width + i, 0.f);
-        if (!shifted) continue;
         st_act(a.s + static_cast<long long>(t) * a.width + i, 0.f);
         for (int j = 0; j < a.blends; ++j) st_act(a.mix + (static_cast<long long>(t) * a.blends + j) * a.width + i, 0.f);
       }
   }
 }
 
-// Long steps: the sums and norms first (shifted_norm_kernel without a shift, which leaves 1 / rms of every token), then the shifted rows and
-// blends of four columns per thread over a run of tokens.  h is formed again from the residual, in fp32.
+// The sum and the norm alone: the first half of a long step, and the model's last norm (rows: only of these tokens, the sum is not kept).
+template <typename A, int N, int NIT, int THREADS>
+__global__ void __launch_bounds__(THREADS, 1024 / THREADS)
+sum_norm_kernel(const ShiftArgs<A> a) {
+  __shared__ float red[64], red1[32];
+  __shared__ long long src[32];
+  __shared__ float wt[32];
+  pdl_wait();
+  pdl_trigger();
+  const int step = blockDim.x * N, i0 = threadIdx.x * N;
+  const float inv_w = 1.f / static_cast<float>(a.W);
+  const long long r = a.rows != nullptr ? a.rows[blockIdx.x] : static_cast<long long>(blockIdx.x);
+  if (a.pairs != nullptr && static_cast<int>(threadIdx.x) < a.top) {
+    const long long p = r * a.top + threadIdx.x;
+    const int at = a.pair_row != nullptr ? a.pair_row[p] : static_cast<int>(p);
+    src[threadIdx.x] = at < 0 ? 0 : at * a.ldp;
+    wt[threadIdx.x] = at < 0 ? 0.f : a.weights[p];
+  }
+  float v[NIT][N], y0[NIT][N], y1[NIT][N], q0 = 0.f, q1 = 0.f;
+#pragma unroll
+  for (int e = 0; e < NIT; ++e) {
+    const int i = i0 + e * step;
+#pragma unroll
+    for (int k = 0; k < N; ++k) v[e][k] = y0[e][k] = y1[e][k] = 0.f;
+    if (i >= a.W) continue;
+    sh_load<N>(a.x + r * a.W + i, v[e]);
+    if (a.o[0].y != nullptr) sh_load<N>(a.o[0].y + r * a.o[0].ld + i, y0[e]);
+    if (a.o[1].y != nullptr) sh_load<N>(a.o[1].y + r * a.o[1].ld + i, y1[e]);
+  }
+  if (a.pairs != nullptr) __syncthreads();
+#pragma unroll
+  for (int e = 0; e < NIT; ++e) {
+    const int i = i0 + e * step;
+    if (i >= a.W) continue;
+    sh_tail<A, N>(a, r, i, src, wt, v[e]);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      q0 = fmaf(y0[e][k], y0[e][k], q0);
+      q1 = fmaf(y1[e][k], y1[e][k], q1);
+    }
+  }
+  float f0 = a.o[0].f, f1 = a.o[1].f;
+  if (a.o[0].w != nullptr || a.o[1].w != nullptr) {
+    const float2 q = block_sum2(q0, q1, red);
+    if (a.o[0].w != nullptr) f0 /= sqrtf(q.x * inv_w + a.eps);
+    if (a.o[1].w != nullptr) f1 /= sqrtf(q.y * inv_w + a.eps);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < NIT; ++e) {
+    const int i = i0 + e * step;
+    if (i >= a.W) continue;
+    float u0[N], u1[N];
+    if (a.o[0].w != nullptr) sh_load<N>(a.o[0].w + i, u0);
+    if (a.o[1].w != nullptr) sh_load<N>(a.o[1].w + i, u1);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      if (a.o[0].y != nullptr) v[e][k] = fmaf(y0[e][k] * f0, a.o[0].w != nullptr ? u0[k] : 1.f, v[e][k]);
+      if (a.o[1].y != nullptr) v[e][k] = fmaf(y1[e][k] * f1, a.o[1].w != nullptr ? u1[k] : 1.f, v[e][k]);
+      ss = fmaf(v[e][k], v[e][k], ss);
+    }
+    if (a.x_out != nullptr) sh_store<N>(a.x_out + r * a.W + i, v[e]);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red1) * inv_w + a.eps);
+  if (a.inv != nullptr && threadIdx.x == 0) a.inv[blockIdx.x] = inv;
+  A* to = a.h + static_cast<long long>(blockIdx.x) * a.width;
+#pragma unroll
+  for (int e = 0; e < NIT; ++e) {
+    const int i = i0 + e * step;
+    if (i >= a.W) continue;
+    float w[N], h[N];
+    sh_load<N>(a.norm + i, w);
+#pragma unroll
+    for (int k = 0; k < N; ++k) h[k] = v[e][k] * inv * w[k];
+    sh_store_act<A, N>(to + i, h);
+  }
+  for (int i = a.W + threadIdx.x; i < a.width; i += blockDim.x) st_act(to + i, 0.f);
+}
+
+// The second half of a long step: shifted rows and blends of N columns per thread over a run of tokens.  h is formed again from the residual and
+// 1 / rms, in fp32.
 template <typename A>
 struct BlendArgs {
   const float* x; const float* inv;
@@ -315,17 +393,45 @@ struct BlendArgs {
   A* s; A* mix;
   const float* now; float* then;
   const int* tok_req; const int64_t* positions; const int* first_pos; const int* last_pos;
-  int T, W, width, run;
+  int T, W, width;
 };
+constexpr int kBlendRun = 16, kBlendAhead = 4;
 
 template <typename A, int N, int BLENDS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 4)
 shift_blend_kernel(const BlendArgs<A> a) {
+  __shared__ __align__(16) float wts[2 + BLENDS][256 * N];        // norm, shift, mu of the thread's columns
+  __shared__ float s_inv[kBlendRun + 2];
+  __shared__ int s_req[kBlendRun + 2], s_kind[kBlendRun + 2];     // kind: 1 first of its span with a state, 2 first without, 4 last
   pdl_wait();
   pdl_trigger();
-  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * N;
-  const int r0 = blockIdx.y * a.run, r1 = min(a.T, r0 + a.run);
-  if (i >= a.W) {
+  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * N, at = threadIdx.x * N;
+  const int r0 = blockIdx.y * kBlendRun, r1 = min(a.T, r0 + kBlendRun);
+  int begin = r0;
+  if (a.tok_req[r0] >= 0 && a.positions[r0] >= 0)
+    begin = r0 - static_cast<int>(min(2ll, static_cast<long long>(a.positions[r0]) - a.first_pos[r0]));
+  if (static_cast<int>(threadIdx.x) < r1 - begin) {
+    const int t = begin + threadIdx.x, req = a.tok_req[t];
+    const long long pos = a.positions[t];
+    s_inv[threadIdx.x] = a.inv[t];
+    s_req[threadIdx.x] = req;
+    s_kind[threadIdx.x] = req < 0 ? 0 : (pos == a.first_pos[t] ? (pos > 0 ? 1 : 2) : 0) | (pos == a.last_pos[t] ? 4 : 0);
+  }
+  const bool in = i < a.W;
+  if (in) {
+    float w[N];
+    sh_load<N>(a.norm + i, w);
+    sh_store<N>(&wts[0][at], w);
+    sh_load<N>(a.shift + i, w);
+    sh_store<N>(&wts[1][at], w);
+#pragma unroll
+    for (int j = 0; j < BLENDS; ++j) {
+      sh_load<N>(a.mu + static_cast<long long>(j) * a.W + i, w);
+      sh_store<N>(&wts[2 + j][at], w);
+    }
+  }
+  __syncthreads();
+  if (!in) {
     // zeros behind the last column
     for (int t = r0; i < a.width && t < r1; ++t)
       for (int k = 0; k < N && i + k < a.width; ++k) {
@@ -334,81 +440,116 @@ shift_blend_kernel(const BlendArgs<A> a) {
       }
     return;
   }
-  float norm[N], shift[N], mu[BLENDS > 0 ? BLENDS : 1][N], hp[N], sp[N];
-  sh_load<N>(a.norm + i, norm);
-  sh_load<N>(a.shift + i, shift);
-#pragma unroll
-  for (int j = 0; j < BLENDS; ++j) sh_load<N>(a.mu + static_cast<long long>(j) * a.W + i, mu[j]);
+  float hp[N], sp[N], x[kBlendAhead][N];
 #pragma unroll
   for (int k = 0; k < N; ++k) hp[k] = sp[k] = 0.f;
-  int begin = r0;
-  if (a.tok_req[r0] >= 0 && a.positions[r0] >= 0)
-    begin = r0 - static_cast<int>(min(2ll, static_cast<long long>(a.positions[r0]) - a.first_pos[r0]));
-  float next[N];
-  sh_load<N>(a.x + static_cast<long long>(begin) * a.W + i, next);
-  for (int t = begin; t < r1; ++t) {
-    const int req = a.tok_req[t];
-    const long long pos = a.positions[t];
-    const float inv = a.inv[t];
-    float h[N], s[N];
 #pragma unroll
-    for (int k = 0; k < N; ++k) h[k] = next[k] * inv * norm[k];
-    if (t + 1 < r1) sh_load<N>(a.x + (t + 1ll) * a.W + i, next);
-    if (req >= 0 && pos == a.first_pos[t]) {
-      if (pos > 0) {
-        const float* st = a.now + static_cast<long long>(req) * 2 * a.W;
-        sh_load<N>(st + i, hp);
-        sh_load<N>(st + a.W + i, sp);
-      } else {
+  for (int j = 0; j < kBlendAhead; ++j)
+    if (begin + j < r1) sh_load<N>(a.x + (begin + static_cast<long long>(j)) * a.W + i, x[j]);
+  for (int t0 = begin; t0 < r1; t0 += kBlendAhead) {
 #pragma unroll
-        for (int k = 0; k < N; ++k) hp[k] = sp[k] = 0.f;
+    for (int u = 0; u < kBlendAhead; ++u) {
+      const int t = t0 + u;
+      if (t >= r1) break;
+      const float inv = s_inv[t - begin];
+      const int kind = s_kind[t - begin];
+      float h[N], s[N], w[N];
+      sh_load<N>(&wts[0][at], w);
+#pragma unroll
+      for (int k = 0; k < N; ++k) h[k] = x[u][k] * inv * w[k];
+      if (t + kBlendAhead < r1) sh_load<N>(a.x + (t + static_cast<long long>(kBlendAhead)) * a.W + i, x[u]);
+      if (kind & 3) {
+        if (kind & 1) {
+          const float* st = a.now + static_cast<long long>(s_req[t - begin]) * 2 * a.W;
+          sh_load<N>(st + i, hp);
+          sh_load<N>(st + a.W + i, sp);
+        } else {
+#pragma unroll
+          for (int k = 0; k < N; ++k) hp[k] = sp[k] = 0.f;
+        }
       }
+      sh_load<N>(&wts[1][at], w);
+#pragma unroll
+      for (int k = 0; k < N; ++k) s[k] = fmaf(hp[k] - h[k], w[k], h[k]);
+      if (t >= r0) {
+        sh_store_act<A, N>(a.s + static_cast<long long>(t) * a.width + i, s);
+#pragma unroll
+        for (int j = 0; j < BLENDS; ++j) {
+          float b[N];
+          sh_load<N>(&wts[2 + j][at], w);
+#pragma unroll
+          for (int k = 0; k < N; ++k) b[k] = fmaf(sp[k] - s[k], w[k], s[k]);
+          sh_store_act<A, N>(a.mix + (static_cast<long long>(t) * BLENDS + j) * a.width + i, b);
+        }
+        if (kind & 4) {
+          float* st = a.then + static_cast<long long>(s_req[t - begin]) * 2 * a.W;
+          sh_store<N>(st + i, h);
+          sh_store<N>(st + a.W + i, s);
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < N; ++k) { hp[k] = h[k]; sp[k] = s[k]; }
     }
-#pragma unroll
-    for (int k = 0; k < N; ++k) s[k] = fmaf(hp[k] - h[k], shift[k], h[k]);
-    if (t >= r0) {
-      sh_store_act<A, N>(a.s + static_cast<long long>(t) * a.width + i, s);
-#pragma unroll
-      for (int j = 0; j < BLENDS; ++j) {
-        float b[N];
-#pragma unroll
-        for (int k = 0; k < N; ++k) b[k] = fmaf(sp[k] - s[k], mu[j][k], s[k]);
-        sh_store_act<A, N>(a.mix + (static_cast<long long>(t) * BLENDS + j) * a.width + i, b);
-      }
-      if (req >= 0 && pos == a.last_pos[t]) {
-        float* st = a.then + static_cast<long long>(req) * 2 * a.W;
-        sh_store<N>(st + i, h);
-        sh_store<N>(st + a.W + i, s);
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < N; ++k) { hp[k] = h[k]; sp[k] = s[k]; }
   }
 }
 
-constexpr int kBlendRun = 16;
+
+template <typename A>
+static int launch_sum_norm(const ShiftArgs<A>& a, bool vec, cudaStream_t st) {
+  const int need = (a.W + (vec ? 4 : 1) - 1) / (vec ? 4 : 1);
+  // many tokens: two groups of columns per thread keep enough loads in flight; few: a wide row is spread over more threads
+  const int threads = need <= 256 ? 256 : a.T > 148 ? (need <= 512 ? 256 : need <= 1024 ? 512 : 1024) : need <= 512 ? 512 : 1024;
+  const int its = (need + threads - 1) / threads;
+#define STK_SUM(N, NIT)                                                                                              \
+  do {                                                                                                               \
+    if (threads == 256) launch_pdl(sum_norm_kernel<A, N, NIT, 256>, dim3(a.T), dim3(256), 0, st, a);                 \
+    else if (threads == 512) launch_pdl(sum_norm_kernel<A, N, NIT, 512>, dim3(a.T), dim3(512), 0, st, a);            \
+    else launch_pdl(sum_norm_kernel<A, N, NIT, 1024>, dim3(a.T), dim3(1024), 0, st, a);                              \
+  } while (0)
+  if (vec) {
+    if (its == 1) STK_SUM(4, 1);
+    else if (its == 2) STK_SUM(4, 2);
+    else if (its <= 4) STK_SUM(4, 4);
+    else return -2;
+  } else {
+    if (its == 1) STK_SUM(1, 1);
+    else if (its <= 4) STK_SUM(1, 4);
+    else if (its <= 16) STK_SUM(1, 16);
+    else return -2;
+  }
+#undef STK_SUM
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
 
 template <typename A>
 static int launch_shifted(ShiftArgs<A> a, float* inv, int decode, int sm_count, cudaStream_t st) {
   const bool vec = a.W % 4 == 0 && a.o[0].ld % 4 == 0 && a.o[1].ld % 4 == 0 && a.ldf % 4 == 0 && a.ldp % 4 == 0 && a.width % 4 == 0;
-  const bool walk = a.shift != nullptr && !decode;
-  const ShiftArgs<A> all = a;
-  const bool split = walk && inv != nullptr && a.T > 2 * sm_count && (a.blends == 0 || a.blends == 5);
-  if (split) {
-    a.shift = nullptr;
-    a.blends = 0;
-    a.inv = inv;
+  if (a.shift == nullptr) return launch_sum_norm(a, vec, st);
+  if (!decode && inv != nullptr && a.T > 2 * sm_count && (a.blends == 0 || a.blends == 5)) {
+    ShiftArgs<A> sum = a;
+    sum.inv = inv;
+    const int rc = launch_sum_norm(sum, vec, st);
+    if (rc != 0) return rc;
+    const BlendArgs<A> b{a.x_out != nullptr ? a.x_out : a.x, inv, a.norm, a.shift, a.mu, a.s, a.mix, a.now, a.then, a.tok_req, a.positions,
+                         a.first_pos, a.last_pos, a.T, a.W, a.width};
+    const int n = vec ? 4 : 1, cols = (a.width + n - 1) / n;
+    const dim3 g((cols + 255) / 256, (a.T + kBlendRun - 1) / kBlendRun);
+#define STK_BLEND(N, B) launch_pdl(shift_blend_kernel<A, N, B>, g, dim3(256), 0, st, b)
+    if (vec && a.blends == 5) STK_BLEND(4, 5);
+    else if (vec) STK_BLEND(4, 0);
+    else if (a.blends == 5) STK_BLEND(1, 5);
+    else STK_BLEND(1, 0);
+#undef STK_BLEND
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
   }
   // runs: long enough that the two tokens formed again cost little, short enough to fill the SMs
   a.run = 1;
-  if (walk && !split) {
+  if (!decode) {
     a.run = a.T / (2 * sm_count);
     a.run = a.run < 2 ? 2 : a.run > 16 ? 16 : a.run;
   }
   const int need = (a.W + (vec ? 4 : 1) - 1) / (vec ? 4 : 1);
-  int threads = need <= 256 ? 256 : need <= 512 ? 512 : 1024;
-  if ((!walk || split) && a.T > sm_count && need <= 1024) threads = 256;
-  const int its = (need + threads - 1) / threads;
+  const int threads = need <= 256 ? 256 : need <= 512 ? 512 : 1024, its = (need + threads - 1) / threads;
   const dim3 grid((a.T + a.run - 1) / a.run);
 #define STK_SHIFT(N, NIT)                                                                                             \
   do {                                                                                                                \
@@ -417,28 +558,14 @@ static int launch_shifted(ShiftArgs<A> a, float* inv, int decode, int sm_count, 
   } while (0)
   if (vec) {
     if (its == 1) STK_SHIFT(4, 1);
-    else if (its == 2) STK_SHIFT(4, 2);
     else if (its <= 4) STK_SHIFT(4, 4);
     else return -2;
   } else {
     if (its == 1) STK_SHIFT(1, 1);
-    else if (its <= 4) STK_SHIFT(1, 4);
     else if (its <= 16) STK_SHIFT(1, 16);
     else return -2;
   }
 #undef STK_SHIFT
-  if (split) {
-    const BlendArgs<A> b{all.x_out != nullptr ? all.x_out : all.x, inv, all.norm, all.shift, all.mu, all.s, all.mix, all.now, all.then, all.tok_req,
-                         all.positions, all.first_pos, all.last_pos, all.T, all.W, all.width, kBlendRun};
-    const int n = vec ? 4 : 1, cols = (a.width + n - 1) / n;
-    const dim3 g((cols + 255) / 256, (a.T + kBlendRun - 1) / kBlendRun);
-#define STK_BLEND(N, B) launch_pdl(shift_blend_kernel<A, N, B>, g, dim3(256), 0, st, b)
-    if (vec && all.blends == 5) STK_BLEND(4, 5);
-    else if (vec) STK_BLEND(4, 0);
-    else if (all.blends == 5) STK_BLEND(1, 5);
-    else STK_BLEND(1, 0);
-#undef STK_BLEND
-  }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -114,7 +114,7 @@ def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], a: TalkingP
         _lib.call("stk_talking_rows", meta.query_start, meta.req_rows, meta.start_pos, meta.n_req, PROMPT_SPAN, a.chunk, table, table.stride(0),
                   cache, row, rows, n_rows, _lib.stream())
         _lib.call("stk_talking_prompt", q, gate, a.sink, rows, n_rows, *shape, meta.query_start, meta.start_pos, meta.n_req,
-                  PROMPT_SPAN, t, _lib.status_buffer(), _lib.stream())
+                  PROMPT_SPAN, t, _lib.sm_count(), _lib.status_buffer(), _lib.stream())
 
 
 def _rows_base(chunk: int, start: int) -> int:
