@@ -26,7 +26,7 @@ GROUPS = [("attention, prompt", ("talking_prompt_tc",)), ("attention, tokens", (
           ("attention, merge", ("talking_merge",)), ("cached rows gather", ("talking_rows",)), ("attention prep + insert", ("talking_prep",)),
           ("time mixing scan", ("TimeMixFront",)), ("time mixing chunk keys", ("time_mix_keys",)),
           ("time mixing chunk states", ("linear_chunk_state_kernel",)), ("time mixing chunk outputs", ("time_mix_out",)),
-          ("time mixing finish", ("retention_finish",)), ("decay tanh", ("tanh_rows",)), ("shifted norm", ("shifted_norm", "shift_blend")),
+          ("time mixing finish", ("retention_finish",)), ("decay tanh", ("tanh_rows",)), ("shifted norm", ("shifted_norm", "sum_norm", "shift_blend")),
           ("state commit", ("shift_commit",)), ("experts", ("experts_wide", "experts_slim", "expert_rows")),
           ("expert sort + gather", ("moe_align", "expert_gather")), ("router", ("router_kernel", "gate_route")), ("xielu", ("xielu",)),
           ("embedding", ("embed_bigram",)), ("projections", ("gemm", "skinny"))]

@@ -23,7 +23,7 @@ namespace stk {
 
 int make_tmap_2d(CUtensorMap* tm, const void* base, int elem_bytes, long long rows, long long cols, long long ld, int box_rows);
 
-constexpr int kTpTile = 128, kTpPanel = kTpTile * 128, kTpThreads = 576, kTpMaxSlots = 12, kTpMaxQ = 10;
+constexpr int kTpTile = 128, kTpPanel = kTpTile * 128, kTpThreads = 608, kTpMaxSlots = 12, kTpMaxQ = 10;
 constexpr float kTpLog2e = 1.4426950408889634f;
 
 struct alignas(8) TpBars {
@@ -185,27 +185,32 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
   tc_fence_after();
   const uint32_t tmem = bars->tmem_base;                           // scores of set i: i * 128; outputs: 256 + i * 128
 
-  if (warp == 16) {
+  if (warp == 16 || warp == 18) {
     // ------------------------------- loader -------------------------------
     if (lane == 0) {
-      bool ok = true;
-      int seq = 0, asked = 0;                                      // panels, and tiles whose queries were asked for
+      bool ok = true, wrapped = false, turn = warp == 16;          // the two loaders take the panels in turn
+      int asked = 0, slot = 0;                                     // tiles whose queries were asked for; the next slot and
+      uint32_t par = 1u;                                           // the parity of its release (a fresh barrier passes for 1)
+      const int slots = x.slots;
       auto load = [&](const CUtensorMap* tm, int col, int y) {
-        const int st = seq % x.slots;
-        if (seq >= x.slots) ok = mbar_wait(&bars->empty[st], ((seq / x.slots) - 1) & 1, x.status, 860);
-        if (!ok) return;
-        mbar_expect_tx(&bars->full[st], kTpPanel);
-        tma_load_2d(ring + st * kTpPanel, tm, &bars->full[st], col, y);
-        ++seq;
+        if (turn) {
+          uint64_t* full = bars->full + slot;
+          if (!mbar_wait(bars->empty + slot, par, x.status, 860)) { ok = false; return; }
+          mbar_expect_tx(full, kTpPanel);
+          tma_load_2d(ring + slot * kTpPanel, tm, full, col, y);
+        }
+        turn = !turn;
+        if (++slot == slots) { slot = 0; par ^= 1u; wrapped = true; }
       };
       for (int items = 0; ok; ++items) {
         const TpItem t = tp_item(x, items);
         if (t.nb == 0) break;
         const int qy = t.h * x.T + t.row0, vc = t.h / (a.H / a.G) * a.vp;
+        const int y0 = t.seg + t.b0 * kTpTile;
         auto keys = [&](int b, int j0, int j1) {
           for (int j = j0; j < j1 && ok; ++j) {
             if (!x.q_kept) load(&tm_q, j * 64, qy);
-            if (ok) load(&tm_r, a.k_col + j * 64, t.seg + (t.b0 + b) * kTpTile);
+            if (ok) load(&tm_r, a.k_col + j * 64, y0 + b * kTpTile);
           }
         };
         int ahead = 0;
@@ -213,23 +218,25 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
           // as many keys as the ring takes without the products' help, then the queries in place of the previous tile's
           ahead = min(kp, x.slots);
           keys(0, 0, ahead);
-          if (ok && items > 0) ok = mbar_wait(&bars->q_empty, (items - 1) & 1, x.status, 861);
+          if (ok && items > 0 && warp == 16) ok = mbar_wait(&bars->q_empty, (items - 1) & 1, x.status, 861);
           if (!ok) break;
-          mbar_expect_tx(&bars->q_full, kp * kTpPanel);
-          for (int p = 0; p < kp; ++p) tma_load_2d(q_s + p * kTpPanel, &tm_q, &bars->q_full, p * 64, qy);
-          ++asked;
+          if (warp == 16) {
+            mbar_expect_tx(&bars->q_full, kp * kTpPanel);
+            for (int p = 0; p < kp; ++p) tma_load_2d(q_s + p * kTpPanel, &tm_q, &bars->q_full, p * 64, qy);
+            ++asked;
+          }
         }
         keys(0, ahead, kp);
         if (t.nb > 1) keys(1, 0, kp);
         for (int b = 0; b < t.nb && ok; ++b) {
-          for (int j = 0; j < x.v_panels && ok; ++j) load(&tm_r, vc + j * 64, t.seg + (t.b0 + b) * kTpTile);
+          for (int j = 0; j < x.v_panels && ok; ++j) load(&tm_r, vc + j * 64, y0 + b * kTpTile);
           if (b + 2 < t.nb) keys(b + 2, 0, kp);
         }
       }
       if (!ok) {
         // leave no copy in flight: what was asked for lands before the CTA's shared memory goes away
         if (asked > 0) mbar_wait(&bars->q_full, (asked - 1) & 1, nullptr, 0);
-        for (int s = max(0, seq - x.slots); s < seq; ++s) mbar_wait(&bars->full[s % x.slots], (s / x.slots) & 1, nullptr, 0);
+        for (int s = 0; s < (wrapped ? slots : slot); ++s) mbar_wait(&bars->full[s], s < slot ? par ^ 1u : par, nullptr, 0);
       }
     }
     __syncwarp();
