@@ -4,6 +4,7 @@
 // joined sublayer buffer.
 #define STK_PDL_CLASS 4
 #include "hybrid_block.cuh"
+#include "pairs.cuh"
 
 namespace stk {
 
@@ -471,10 +472,9 @@ __global__ void __launch_bounds__(256)
 xielu_kernel(const A* __restrict__ z, long long ldz, int ff, float a, float b, A* __restrict__ out, long long ldo, int width, int T) {
   pdl_wait();
   pdl_trigger();
-  const int per = (width + 7) / 8;
-  const long long e = blockIdx.x * 256ll + threadIdx.x, t = e / per;
-  if (t >= T) return;
-  const int c0 = static_cast<int>(e - t * per) * 8;
+  const int c0 = (blockIdx.y * 256 + threadIdx.x) * 8;
+  if (c0 >= width) return;
+  const long long t = blockIdx.x;
   auto f = [&](float x) {
     if (sizeof(A) == 4) return fmaf(x, 0.5f, x > 0.f ? a * x * x : b * (expm1f(x) - x));
     // rounded results: exp(x) - 1 - x from its series where the difference would cancel
@@ -489,7 +489,18 @@ xielu_kernel(const A* __restrict__ z, long long ldz, int ff, float a, float b, A
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const float2 x = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[j]);
-      reinterpret_cast<__nv_bfloat162*>(&r)[j] = __floats2bfloat162_rn(f(x.x), f(x.y));
+      // two at a time: the series and the difference of f in packed arithmetic
+      const uint64_t xx = pack2(x.x, x.y), sq = mul2(xx, xx);
+      const uint64_t near = mul2(sq, fma2(xx, fma2(xx, fma2(xx, pack2(1.f / 120.f, 1.f / 120.f), pack2(1.f / 24.f, 1.f / 24.f)),
+                                                   pack2(1.f / 6.f, 1.f / 6.f)), pack2(0.5f, 0.5f)));
+      float n0, n1, q0, q1, y0, y1;
+      unpack2(near, n0, n1);
+      unpack2(sq, q0, q1);
+      const float e0 = __expf(x.x) - 1.f - x.x, e1 = __expf(x.y) - 1.f - x.y;
+      const uint64_t by = pack2(x.x > 0.f ? a : b, x.y > 0.f ? a : b);
+      const uint64_t part = pack2(x.x > 0.f ? q0 : x.x > -0.25f ? n0 : e0, x.y > 0.f ? q1 : x.y > -0.25f ? n1 : e1);
+      unpack2(fma2(part, by, mul2(xx, pack2(0.5f, 0.5f))), y0, y1);
+      reinterpret_cast<__nv_bfloat162*>(&r)[j] = __floats2bfloat162_rn(y0, y1);
     }
     *reinterpret_cast<uint4*>(o) = r;
     return;
@@ -506,8 +517,7 @@ STK_API int stk_xielu(const void* z, long long ldz, int ff, float a, float b, vo
                       void* stream) {
   if (T <= 0) return 0;
   if (width < ff || ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
-  const long long n = static_cast<long long>(T) * ((width + 7) / 8);
-  const dim3 grid(static_cast<unsigned>((n + 255) / 256));
+  const dim3 grid(static_cast<unsigned>(T), static_cast<unsigned>((width + 2047) / 2048));
   cudaStream_t st = (cudaStream_t)stream;
   if (fp32) launch_pdl(xielu_kernel<float>, grid, dim3(256), 0, st, (const float*)z, ldz, ff, a, b, (float*)out, ldo, width, T);
   else launch_pdl(xielu_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, ff, a, b, (__nv_bfloat16*)out, ldo, width, T);

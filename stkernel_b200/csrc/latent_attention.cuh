@@ -4,6 +4,7 @@
 // in columns [rot_off, rot_off + R), zeros to the end of the row.
 #pragma once
 #include "common.cuh"
+#include "pairs.cuh"
 
 namespace stk {
 
@@ -62,24 +63,6 @@ __device__ __forceinline__ void mma_commit(uint64_t* bar, uint32_t lead) {
       "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
       "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
       ::"r"(smem_u32(bar)), "r"(lead) : "memory");
-}
-
-// packed pairs of fp32
-__device__ __forceinline__ uint64_t pack2(float x, float y) {
-  uint64_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
-  return r;
-}
-__device__ __forceinline__ void unpack2(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
-  uint64_t r;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
 }
 
 }  // namespace stk

@@ -17,6 +17,7 @@
 #define STK_PDL_CLASS 16
 #include "chunk_mma.cuh"
 #include "linear_scan.cuh"
+#include "pairs.cuh"
 
 namespace stk {
 
@@ -147,27 +148,6 @@ __host__ __device__ inline TmOutLayout tm_out_layout(int D) {
   l.bytes = l.p + 4 * Dp * 4;
   return l;
 }
-// packed pairs of fp32
-__device__ __forceinline__ uint64_t tm_pack2(float x, float y) {
-  uint64_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
-  return r;
-}
-__device__ __forceinline__ void tm_unpack2(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
-__device__ __forceinline__ uint64_t tm_fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ uint64_t tm_mul2(uint64_t a, uint64_t b) {
-  uint64_t r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-// Two bf16 as a pair of fp32.
-__device__ __forceinline__ uint64_t tm_widen2(uint32_t v) {
-  return tm_pack2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
-}
 
 // An operand pair times a factor per column (columns 2 (lane & 3), + 1, and 8 further).
 __device__ __forceinline__ void tm_scale_pair(uint32_t (&hi)[4], uint32_t (&lo)[4], const float* f) {
@@ -255,21 +235,21 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
   for (int c0 = seg * 4; c0 < Dp; c0 += 16) {
     const uint2 kv = *reinterpret_cast<const uint2*>(kr + (jb * kTmSub + j) * ks + c0);
     const uint2 rv = *reinterpret_cast<const uint2*>(r + (jb * kTmSub + j) * ks + c0);
-    uint64_t x0 = tm_widen2(kv.x), x1 = tm_widen2(kv.y);
+    uint64_t x0 = widen2(kv.x), x1 = widen2(kv.y);
     const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(f + 6 * Dp + c0);
     float s0, s1;
-    tm_unpack2(tm_fma2(tm_mul2(tm_widen2(rv.x), u.x), x0, tm_mul2(tm_mul2(tm_widen2(rv.y), u.y), x1)), s0, s1);
+    unpack2(fma2(mul2(widen2(rv.x), u.x), x0, mul2(mul2(widen2(rv.y), u.y), x1)), s0, s1);
     bonus += s0 + s1;
 #pragma unroll
     for (int i = 1; i < kTmSub; ++i) {
       if (i < 9 && (warp & 1)) continue;                                 // the warp's columns start behind these rows
       const ulonglong2 wi = *reinterpret_cast<const ulonglong2*>(w + (jb * kTmSub + i) * Dp + c0);
       const uint2 y = *reinterpret_cast<const uint2*>(r + (jb * kTmSub + i) * ks + c0);
-      tm_unpack2(tm_fma2(tm_widen2(y.x), x0, tm_mul2(tm_widen2(y.y), x1)), s0, s1);
+      unpack2(fma2(widen2(y.x), x0, mul2(widen2(y.y), x1)), s0, s1);
       const bool below = i > j;
       acc[i] += below ? s0 + s1 : 0.f;
-      x0 = below ? tm_mul2(x0, wi.x) : x0;
-      x1 = below ? tm_mul2(x1, wi.y) : x1;
+      x0 = below ? mul2(x0, wi.x) : x0;
+      x1 = below ? mul2(x1, wi.y) : x1;
     }
   }
   bonus += __shfl_xor_sync(0xffffffffu, bonus, 1);
@@ -369,8 +349,31 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
     const int off = (jb * kTmSub + i) * kStStride + jb * kTmSub + j;
     mls_split(i > j ? acc[i] : i == j ? bonus : 0.f, ph[off], pl[off]);
   }
-  __syncthreads();                                                       // the weighted scores are complete
   const bool has_state = !(a.s.start_pos[c.ri] == 0 && c.first == ci);
+  if (has_state) {
+    // r~ decayed from the chunk's start on, for the state: blocks 1 to 3
+    const int per = Dp / 8;
+    for (int e = threadIdx.x; e < 48 * per; e += kTmOutThreads) {
+      const int t = e / per + 16, c0 = (e % per) * 8;
+      uint4* at = reinterpret_cast<uint4*>(q + t * ks + c0);
+      uint4* rest = reinterpret_cast<uint4*>(q + part + t * ks + c0);
+      const ulonglong2* by = reinterpret_cast<const ulonglong2*>(f + (2 + (t >> 4)) * Dp + c0);
+      const ulonglong2 g0 = by[0], g1 = by[1];
+      uint4 hi = *at, lo = *rest;
+      auto scale = [&](uint32_t& x, uint32_t& y, uint64_t g) {
+        float s0, s1;
+        unpack2(mul2(add2(widen2(x), widen2(y)), g), s0, s1);
+        mls_split2(s0, s1, x, y);
+      };
+      scale(hi.x, lo.x, g0.x);
+      scale(hi.y, lo.y, g0.y);
+      scale(hi.z, lo.z, g1.x);
+      scale(hi.w, lo.w, g1.y);
+      *at = hi;
+      *rest = lo;
+    }
+  }
+  __syncthreads();                                                       // the weighted scores are complete
   const uint4* S0 = reinterpret_cast<const uint4*>(states + (static_cast<long long>(ci) * a.s.H + h) * linear_slot_floats(D, D)) + lane;
   for (int unit = warp; unit < 2 * nd; unit += kTmOutThreads / 32) {     // 16 columns, 32 rows
     const int cg = unit >> 1, rh = unit & 1;
@@ -393,7 +396,6 @@ time_mix_out_kernel(const TmArgs a, int min_span, const float* __restrict__ stat
           const int qo = (rb2 * 16 + (lane & 15)) * ks + (lane >> 4) * 8 + kk * 16;
           mls_ldsm4(ah, q + qo);
           mls_ldsm4(al, q + part + qo);
-          if (rb2 > 0) tm_scale_pair(ah, al, f + (2 + rb2) * Dp + kk * 16 + (lane & 3) * 2);
           mls_mma(o[x][0], ah, hi.x, hi.y);
           mls_mma(o[x][1], ah, hi.z, hi.w);
           mls_mma(o[x][0], ah, lo.x, lo.y);
