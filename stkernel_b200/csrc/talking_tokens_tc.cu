@@ -31,7 +31,7 @@ struct TtArgs {
   const int* query_start; const int* req_rows; const int* start_pos;
   int n_req, max_span;
   int tq, hs;                            // tokens per tile, heads per group (tq * hs <= N)
-  int k_pairs, v_tiles, slots;           // panel pairs of a row's keys, 128-dim tiles of its values, ring size
+  int k_pairs, slots;                    // panel pairs of a row's keys, ring size
   float* part;                           // [splits][T][H][V + 2]
   int T;
   int* status;
@@ -148,6 +148,8 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
   if (ri < 0) return;
   const int off = bars->find[1];
   const int h0 = blockIdx.z * x.hs, nh = min(x.hs, a.H - h0);
+  // 128-dim tiles of the values of the group's key/value heads
+  const int v0 = h0 / (a.H / a.G) * a.vp / kTtBlock, v_tiles = ((h0 + nh - 1) / (a.H / a.G) * a.vp + a.vp - 1) / kTtBlock + 1 - v0;
   const int tok0 = x.query_start[ri] + off, ntok = min(x.tq, x.query_start[ri + 1] - tok0);
   const int p0 = x.start_pos[ri] + off, p_last = p0 + ntok - 1;
   const int k_first = talk_first(a, p0), first_b = k_first / kTtBlock, end_b = p_last / kTtBlock + 1, blocks = end_b - first_b;
@@ -235,14 +237,14 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
       if (lane == 0) {
         if (ok && b + 1 < b1) load_keys(b + 1, 0);
         const int pg0 = page_of(2 * b), pg1 = page_of(2 * b + 1);
-        for (int j = 0; j < x.v_tiles && ok; ++j) load(j * 128, pg0, pg1);
+        for (int j = 0; j < v_tiles && ok; ++j) load((v0 + j) * 128, pg0, pg1);
       }
       ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
       if (!ok) break;
       if (dirty(b)) {
         const int last = __shfl_sync(0xffffffffu, seq, 0);
         const int r0 = b == b0 ? front : 0, r1 = b == b1 - 1 && back > 0 ? back : kTtBlock;
-        for (int s = last - x.v_tiles; s < last && ok; ++s) {
+        for (int s = last - v_tiles; s < last && ok; ++s) {
           const int st = s % x.slots;
           ok = mbar_wait(&bars->full[st], (s / x.slots) & 1, x.status, 931);
           ok = __all_sync(0xffffffffu, ok);
@@ -302,7 +304,7 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
       }
       if (!ok) break;
       tc_fence_after();
-      for (int j = 0; j < x.v_tiles; ++j) {
+      for (int j = 0; j < v_tiles; ++j) {
         if (!mbar_wait(&bars->full[slot], par, x.status, 935)) { ok = false; break; }
         tc_fence_after();
         const uint32_t al = v_lo + slot * 2 * kStep, dj = tm + 2 * N + j * 2 * N;
@@ -371,7 +373,7 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
         if (i > 0) {
           // high parts for the first four warps, remainders for the others
           const uint32_t to = tmem_o + (warp >> 2) * N + lanes;
-          for (int j = 0; j < x.v_tiles; ++j)
+          for (int j = 0; j < v_tiles; ++j)
 #pragma unroll
             for (int c = 0; c < N; c += 16) {
               uint32_t o[16];
@@ -407,8 +409,8 @@ talking_tokens_tc_kernel(const __grid_constant__ CUtensorMap tm_rows, const TtAr
     tt_bar_sync();
     if (ok) {
       // the two halves of the warps take every other 128 dims
-      for (int j = warp >> 2; j < x.v_tiles; j += 2) {
-        const int d = j * 128 + row;
+      for (int j = warp >> 2; j < v_tiles; j += 2) {
+        const int d = (v0 + j) * 128 + row;
 #pragma unroll
         for (int c = 0; c < N; c += 16) {
           uint32_t u[16], w[16];
@@ -498,16 +500,16 @@ talking_merge_kernel(const TalkArgs a, const float* __restrict__ part, int split
 
 struct TtShape { int n, hs, k_pairs, v_tiles, slots; };
 static int tt_fixed(const TtShape& s) { return 2 * s.k_pairs * s.n * 128 + 4 * s.n * 128 + 256 + 10 * s.n * 4 + 64 + 1024; }
-// n 0: the kernel does not cover the layer.
-static TtShape tt_shape(int H, int G, int kp, int vp, int max_span) {
+// Groups of `hs` heads; 0: as many as fit.  n 0: the kernel does not cover the layer.
+static TtShape tt_shape(int H, int G, int kp, int vp, int max_span, int hs = 0) {
   TtShape s = {};
   s.k_pairs = (G * kp + 127) / 128;
   s.v_tiles = (G * vp + 127) / 128;
-  const bool wide = H > 16 || (max_span > 1 && 2 * H > 16);
-  for (int n = wide ? 32 : 16; n >= 16; n -= 16) {
+  const bool wide = hs > 0 ? hs > 16 : H > 16 || (max_span > 1 && 2 * H > 16);
+  for (int n = wide ? 32 : 16; n >= 16 && hs <= n; n -= 16) {
     s.n = n;
     const int groups = (H + n - 1) / n;
-    s.hs = (H + groups - 1) / groups;
+    s.hs = hs > 0 ? hs : (H + groups - 1) / groups;
     s.slots = (227 * 1024 - tt_fixed(s)) / (2 * kTtPanel);
     if (s.slots > kTtMaxPairs) s.slots = kTtMaxPairs;
     // the values of a block lie in the ring while rows that nobody sees are zeroed
@@ -527,33 +529,39 @@ STK_API int stk_talking_tokens_ok(int heads, int kv_heads, int kp, int vp, int m
   return tt_shape(heads, kv_heads, kp, vp, max_span).n > 0 ? 1 : 0;
 }
 
-// Splits of the key range for T tokens that see at most `keys` keys: the smallest number of block steps.
-STK_API int stk_talking_tokens_splits(int T, int heads, int kv_heads, int kp, int vp, int max_span, int keys, int sm_count) {
-  const TtShape s = tt_shape(heads, kv_heads, kp, vp, max_span);
-  if (s.n == 0) return 0;
-  const int groups = (heads + s.hs - 1) / s.hs, tq = max_span < 2 ? 1 : s.n / s.hs;
-  const int tiles = ((T + tq - 1) / tq) * groups, blocks = (keys + kTtBlock - 2) / kTtBlock + 1;
-  int best = 1;
+// Splits of the key range for T tokens that see at most `keys` keys, and whether every key/value head is a group of its own, which reads
+// the keys once per group and of the values only its own: the smallest number of block steps.  splits + 256 * that; 0: not covered.
+STK_API int stk_talking_tokens_plan(int T, int heads, int kv_heads, int kp, int vp, int max_span, int keys, int sm_count) {
+  int best = 0;
   double cost = 1e30;
-  for (int n = 1; n <= kTtMaxSplits && n <= blocks; ++n) {
-    const int waves = (tiles * n + sm_count - 1) / sm_count;
-    const double c = static_cast<double>(waves) * ((blocks + n - 1) / n + 1.5) + 0.03 * n;
-    if (c < cost - 1e-9) { cost = c; best = n; }
+  for (int own = 0; own < (max_span < 2 && kv_heads > 1 ? 2 : 1); ++own) {
+    const TtShape s = tt_shape(heads, kv_heads, kp, vp, max_span, own ? heads / kv_heads : 0);
+    if (s.n == 0 || (own && best == 0)) continue;
+    const int groups = (heads + s.hs - 1) / s.hs, tq = max_span < 2 ? 1 : s.n / s.hs;
+    const int tiles = ((T + tq - 1) / tq) * groups, blocks = (keys + kTtBlock - 2) / kTtBlock + 1;
+    const int held = (s.hs + heads / kv_heads - 1) / (heads / kv_heads);                // key/value heads whose values a group reads
+    const double step = static_cast<double>(kv_heads * kp + held * vp) / (kv_heads * (kp + vp));
+    for (int n = 1; n <= kTtMaxSplits && n <= blocks; ++n) {
+      const int waves = (tiles * n + sm_count - 1) / sm_count;
+      const double c = static_cast<double>(waves) * ((blocks + n - 1) / n * step + 1.5) + 0.03 * n;
+      if (c < cost - 1e-9) { cost = c; best = n + 256 * own; }
+    }
   }
   return best;
 }
 
-// Spans of at most max_span tokens.  part: [splits][T][heads][vdim + 2] fp32.
+// Spans of at most max_span tokens.  plan: of stk_talking_tokens_plan.  part: [splits][T][heads][vdim + 2] fp32.
 STK_API int stk_talking_tokens(const void* q, const float* gate, const float* sink, const int64_t* positions, const int* tok_req,
                                const int* table, int bt_stride, const void* cache, int row, int k_col, int kp, int vp, int heads, int kv_heads,
                                int vdim, int chunk, float scale, void* out, long long ldo, int out_cols, const int* query_start,
                                const int* req_rows, const int* start_pos, int n_req, const int* first_pos, const int* last_pos, int max_span,
-                               long long num_pages, int splits, float* part, int T, int* status, void* stream) {
+                               long long num_pages, int plan, float* part, int T, int* status, void* stream) {
   if (T <= 0) return 0;
+  const int splits = plan & 255;
   TtArgs x;
   x.a = {q, T, gate, sink, positions, tok_req, table, bt_stride, cache, row, k_col, kp, vp, heads, kv_heads, vdim, chunk, scale, out, ldo,
          out_cols};
-  const TtShape s = tt_shape(heads, kv_heads, kp, vp, max_span);
+  const TtShape s = tt_shape(heads, kv_heads, kp, vp, max_span, plan >= 256 ? heads / kv_heads : 0);
   if (!talk_ok(x.a) || s.n == 0 || splits < 1 || splits > kTtMaxSplits || n_req < 1 || num_pages < 1 || row % 8 || kp % 8 || vp % 8 ||
       heads > 65535 || row != k_col + kv_heads * kp || num_pages * kTkPage >= (1ll << 31) ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15))
@@ -562,7 +570,7 @@ STK_API int stk_talking_tokens(const void* q, const float* gate, const float* si
   x.hs = s.hs;
   x.tq = max_span < 2 ? 1 : s.n / s.hs;
   x.query_start = query_start; x.req_rows = req_rows; x.start_pos = start_pos; x.n_req = n_req; x.max_span = max_span;
-  x.k_pairs = s.k_pairs; x.v_tiles = s.v_tiles; x.slots = s.slots;
+  x.k_pairs = s.k_pairs; x.slots = s.slots;
   x.part = part; x.T = T; x.status = status;
   static_assert(sizeof(TtBars) <= 256, "barrier block");
   CUtensorMap tm;

@@ -157,12 +157,25 @@ __device__ __forceinline__ void sh_tail(const ShiftArgs<A>& a, long long r, int 
   }
 }
 
+__device__ __forceinline__ void sh_prefetch(const float* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 template <typename A, int N, int NIT, int THREADS>
 __global__ void __launch_bounds__(THREADS)
 shifted_norm_kernel(const ShiftArgs<A> a) {
   __shared__ float red[64], red1[32];
   __shared__ long long src[32];
   __shared__ float wt[32];
+  constexpr int kMu = NIT > 1 ? 0 : THREADS > 256 ? 2 : 5;                // blends whose weights are asked for before the last wait
+  if (blockIdx.x == 0) {
+    // the weights come from HBM while the kernel before is at work
+    for (int i = threadIdx.x * 32; i < a.W; i += blockDim.x * 32) {
+      if (a.o[0].w != nullptr) sh_prefetch(a.o[0].w + i);
+      if (a.o[1].w != nullptr) sh_prefetch(a.o[1].w + i);
+      sh_prefetch(a.norm + i);
+      sh_prefetch(a.shift + i);
+      for (int j = 0; j < a.blends; ++j) sh_prefetch(a.mu + static_cast<long long>(j) * a.W + i);
+    }
+  }
   pdl_wait();
   pdl_trigger();
   const int step = blockDim.x * N, i0 = threadIdx.x * N;
@@ -256,11 +269,14 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       for (int k = 0; k < N; ++k) ss = fmaf(v[e][k], v[e][k], ss);
     }
     // what the rest needs is asked for before the wait
-    float wn[NIT][N], ws[NIT][N];
+    float wn[NIT][N], ws[NIT][N], wm[kMu > 0 ? kMu : 1][N];
 #pragma unroll
     for (int e = 0; e < NIT; ++e) {
       const int i = i0 + e * step;
       if (NIT > 1 || i >= a.W) continue;
+#pragma unroll
+      for (int j = 0; j < kMu; ++j)
+        if (j < a.blends) sh_load<N>(a.mu + static_cast<long long>(j) * a.W + i, wm[j]);
       sh_load<N>(a.norm + i, wn[e]);
       sh_load<N>(a.shift + i, ws[e]);
     }
@@ -281,12 +297,18 @@ shifted_norm_kernel(const ShiftArgs<A> a) {
       for (int k = 0; k < N; ++k) s[k] = fmaf(hp[e][k] - h[k], ws[e][k], h[k]);
       if (own) {
         sh_store_act<A, N>(a.s + static_cast<long long>(t) * a.width + i, s);
-        for (int j = 0; j < a.blends; ++j) {
+        auto blend = [&](int j, const float (&m)[N]) {
           float b[N];
-          sh_load<N>(a.mu + static_cast<long long>(j) * a.W + i, w);
 #pragma unroll
-          for (int k = 0; k < N; ++k) b[k] = fmaf(sp[e][k] - s[k], w[k], s[k]);
+          for (int k = 0; k < N; ++k) b[k] = fmaf(sp[e][k] - s[k], m[k], s[k]);
           sh_store_act<A, N>(a.mix + (static_cast<long long>(t) * a.blends + j) * a.width + i, b);
+        };
+#pragma unroll
+        for (int j = 0; j < kMu; ++j)
+          if (j < a.blends) blend(j, wm[j]);
+        for (int j = kMu; j < a.blends; ++j) {
+          sh_load<N>(a.mu + static_cast<long long>(j) * a.W + i, w);
+          blend(j, w);
         }
         if (keep) {
           sh_store<N>(st + i, h);

@@ -104,10 +104,10 @@ def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], a: TalkingP
         else:
             context = min(meta.max_context, table.shape[1] * PAGE)
             keys = min(a.chunk, context) if a.chunk else context
-            splits = _lib.query("stk_talking_tokens_splits", t, h, g, kp, vp, max_span, keys, _lib.sm_count())
-            part = scratch("talking.part", (splits * t * h * (v + 2),), F32, q.device)
+            plan = _lib.query("stk_talking_tokens_plan", t, h, g, kp, vp, max_span, keys, _lib.sm_count())
+            part = scratch("talking.part", ((plan & 255) * t * h * (v + 2),), F32, q.device)
             _lib.call("stk_talking_tokens", *common, meta.query_start, meta.req_rows, meta.start_pos, meta.n_req, meta.first_pos,
-                      meta.last_pos, max_span, cache.shape[0], splits, part, t, _lib.status_buffer(), _lib.stream())
+                      meta.last_pos, max_span, cache.shape[0], plan, part, t, _lib.status_buffer(), _lib.stream())
     if prompt:
         n_rows = sum(_up(start + n - _rows_base(a.chunk, start), PROMPT_ROWS) for start, n in meta.spans if n >= PROMPT_SPAN)
         rows = torch.empty(n_rows, row, dtype=q.dtype, device=q.device)

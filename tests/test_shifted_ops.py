@@ -197,16 +197,11 @@ LONG = [dict(H=8, G=2, D=128, V=128, R=128), dict(H=4, G=4, D=64, V=128, R=32), 
         dict(H=16, G=4, D=128, V=128, R=64), dict(H=40, G=8, D=128, V=64, R=128), dict(H=3, G=3, D=200, V=200, R=10)]
 
 
-@pytest.mark.gpu
-@pytest.mark.parametrize("c", LONG, ids=ids)
-@pytest.mark.parametrize("chunk", [0, 256, 300, 77])
-def test_attention_kernels_agree_over_many_pages(c, chunk):
-    """Several requests in one step (long portions that begin inside a page and a chunk, short ones, single tokens): the tensor-core
-    kernels against the fp32 one."""
+def kernels_agree(c, chunk, spans, rows):
+    """The tensor-core kernels against the fp32 one over scattered pages."""
     dev = torch.device("cuda:0")
     H, G, D, V = c["H"], c["G"], c["D"], c["V"]
     g = torch.Generator(device=dev).manual_seed(1)
-    spans, rows = [(0, 777), (500, 1), (1300, 333), (130, 40), (0, 3), (64, 64), (1001, 65), (255, 2)], [0, 3, 1, 2, 4, 5, 6, 7]
     n = sum(s[1] for s in spans)
     meta = step(spans, dev, rows)
     pages, (row, k_col, kp, vp) = 27, TK.talking_row(G, D, V)
@@ -231,6 +226,24 @@ def test_attention_kernels_agree_over_many_pages(c, chunk):
     err = ((x - y).norm(dim=-1) / y.norm(dim=-1)).cpu()
     assert err.max() < 1e-2, int(err.argmax())
     _lib.check_status()
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("c", LONG, ids=ids)
+@pytest.mark.parametrize("chunk", [0, 256, 300, 77])
+def test_attention_kernels_agree_over_many_pages(c, chunk):
+    """Several requests in one step: long portions that begin inside a page and a chunk, short ones, single tokens."""
+    kernels_agree(c, chunk, [(0, 777), (500, 1), (1300, 333), (130, 40), (0, 3), (64, 64), (1001, 65), (255, 2)], [0, 3, 1, 2, 4, 5, 6, 7])
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("c", LONG, ids=ids)
+@pytest.mark.parametrize("chunk", [0, 300])
+@pytest.mark.parametrize("sms", [1, 148, 4000])
+def test_decode_rows_agree_whatever_the_split(monkeypatch, c, chunk, sms):
+    """One token per request: all heads in a CTA over the whole range, up to a CTA per key/value head and block of keys."""
+    monkeypatch.setattr(_lib, "sm_count", lambda: sms)
+    kernels_agree(c, chunk, [(1500, 1), (0, 1), (299, 1), (300, 1), (127, 1), (128, 1), (777, 1), (64, 1)], [0, 3, 1, 2, 4, 5, 6, 7])
 
 
 # ---- time mixing -----------------------------------------------------------------------------------------
