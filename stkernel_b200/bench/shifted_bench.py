@@ -1,6 +1,6 @@
 """Prefill and decode of the shifted decoder (Fogizen: talking-heads attention in chunks beside time mixing, gated experts chosen in groups, bigram
 embedding) at sizes like a real model's layers, beside the closest decoders of the same width and depth: Fanulix (attention beside
-retention, Mamba-2, gelu experts) and Domilix (full-context attention, ungated experts), with every kernel's distance from its
+retention, Mamba-2, gelu experts) and Domilix (latent attention, ungated experts), with every kernel's distance from its
 roofline.
 
     python bench.py --shifted [--shifted-sizes 2048,4096] [--shifted-alone]
